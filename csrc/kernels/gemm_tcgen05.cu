@@ -46,6 +46,13 @@ constexpr int kGemmThreads = 192;
 constexpr int kGemmThreadsScatter = 224;  // + one warp that publishes finished tiles to peer GPUs
 
 enum GemmEpilogue : int { kEpiNone = 0, kEpiResidual = 1, kEpiSwiGLU = 2, kEpiScatter = 3 };
+enum GemmAct : int { kActSilu = 0, kActGeluTanh = 1 };   // gate activation of the gated epilogue
+
+// 0.5 z (1 + tanh(a)) = z / (1 + exp(-2 a)); relative error of a few 1e-7, ahead of a bf16 rounding
+OGB_DEVICE float gelu_tanh_fast(float z) {
+  const float a = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.f + __expf(fminf(-2.f * a, 80.f)));
+}
 
 constexpr int kStagingPitch = 272;                       // bytes per staged row: 128 bf16 + 16 bytes of padding
 constexpr int kStagingWarpBytes = 32 * kStagingPitch;    // one epilogue warp: 32 rows
@@ -117,6 +124,13 @@ struct GemmWork {
   }
 };
 
+// A batch of products that share shapes: problem z reads A from column z * a_step and W from row z * N, and writes its
+// results from column z * c_step of C (per-head projections of a packed row).  Columns of A past K belong to the next
+// problem; the rows of W end at K and the loads past it read zeros, so they add nothing.
+struct GemmBatch {
+  int count = 1, a_step = 0, c_step = 0;
+};
+
 // fp32 partial accumulators of stream-K: slot = CTA, layout [BN / 32 column chunks][128 rows][32 floats], so a warp's
 // 32 rows of one chunk are 4 KB contiguous.  flags[cta * 4 + quarter] holds the sequence number of the launch whose
 // partial of that row quarter is complete.
@@ -142,7 +156,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                          const __nv_bfloat16* residual, float* __restrict__ C_f32, int M, int N, int K, int ldc, int ldr,
                          int* status, const TpScatter* __restrict__ sc, const int* __restrict__ group_tab,
                          const int* __restrict__ group_mtiles, uint32_t* a_ready, uint32_t* a_done, unsigned long long a_wait_ns,
-                         float* sk_ws, uint32_t* sk_flags, uint32_t sk_seq) {
+                         float* sk_ws, uint32_t* sk_flags, uint32_t sk_seq, const GemmBatch batch, const int act) {
   using Cfg = GemmCfg<BN>;
   const bool stream_k = sk_ws != nullptr;
   if constexpr (EPI == kEpiScatter) pdl_trigger();   // the exchange kernel may start: it waits on the tile counters this kernel bumps
@@ -164,7 +178,8 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
   // grouped (MoE) mode: the m-tile list {expert, first row, end row} and its length live in device memory
   const int m_tiles = group_tab != nullptr ? *group_mtiles : (M + kBM - 1) / kBM;
   const int n_tiles = (N + BN - 1) / BN;
-  const int num_tiles = m_tiles * n_tiles;
+  const int batch_tiles = m_tiles * n_tiles;
+  const int num_tiles = batch_tiles * batch.count;
   const int k_blocks = (K + kBK - 1) / kBK;
 
   if (threadIdx.x == 0) {
@@ -201,11 +216,13 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
       GemmWork work(stream_k, num_tiles, k_blocks);
       GemmSeg seg;
       while (ok && work.next(seg)) {
-        const int tile = seg.tile;
+        const int z = seg.tile / batch_tiles;
+        const int tile = seg.tile - z * batch_tiles;
         const int mt = tile % m_tiles;
         const int n0 = (tile / m_tiles) * BN;
         const int m0 = group_tab != nullptr ? group_tab[4 * mt + 1] : mt * kBM;
-        const int b_row = group_tab != nullptr ? group_tab[4 * mt] * N + n0 : n0;   // expert e's weights start at row e*N
+        const int b_row = group_tab != nullptr ? group_tab[4 * mt] * N + n0 : z * N + n0;   // expert e's weights start at row e*N
+        const int a_col = z * batch.a_step;
         if (a_ready != nullptr && !(mt < 64 && ((seen_ready >> mt) & 1ull))) {
           // The rows of A are delivered by other GPUs (the all-gather half of a tensor-parallel exchange): every 8
           // rows that land bump the tile's counter.  Wait, bounded, until the whole tile is here; the loads below
@@ -228,7 +245,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
           uint8_t* sa = smem + stage * Cfg::kStage;
           uint8_t* sb = sa + Cfg::kStageA;
           mbar_expect_tx(&full_bar[stage], Cfg::kStage);
-          tma_load_2d(sa, &tmap_a, &full_bar[stage], kb * kBK, m0);
+          tma_load_2d(sa, &tmap_a, &full_bar[stage], a_col + kb * kBK, m0);
           tma_load_2d(sb, &tmap_b, &full_bar[stage], kb * kBK, b_row);
           if (++stage == Cfg::kStages) { stage = 0; phase ^= 1; }
         }
@@ -279,7 +296,9 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
     GemmSeg seg;
     const long long sk_total = static_cast<long long>(num_tiles) * k_blocks;
     for (; ok && work.next(seg); ++it) {
-      const int tile = seg.tile;
+      const int z = seg.tile / batch_tiles;
+      const int tile = seg.tile - z * batch_tiles;
+      const size_t c_off = static_cast<size_t>(z) * batch.c_step;
       const int acc = it & 1;
       const uint32_t acc_phase = (it >> 1) & 1;
       const int mt = tile % m_tiles;
@@ -319,7 +338,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
           continue;
         }
         if (seg.kb0 > 0) {
-          fix_lo = GemmWork::owner(sk_total, gridDim.x, static_cast<long long>(tile) * k_blocks);
+          fix_lo = GemmWork::owner(sk_total, gridDim.x, static_cast<long long>(seg.tile) * k_blocks);
           fix_hi = blockIdx.x;
           for (int x = fix_lo; x < fix_hi && ok; ++x) {
             const uint64_t t0 = global_timer_ns();
@@ -343,7 +362,14 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
           for (int x = fix_lo; x < fix_hi; ++x) sk_add32(r, sk_slot<BN>(sk_ws, x, c, q * 32 + lane));
           const int col = n0 + c * 32;
           if (row < m_end && col < N) {
-            float* dst = C_f32 + static_cast<size_t>(row) * ldc + col;
+            float* dst = C_f32 + static_cast<size_t>(row) * ldc + c_off + col;
+            if (EPI == kEpiNone && bias == nullptr && col + 32 <= N && (ldc & 3) == 0 && (c_off & 3) == 0) {
+#pragma unroll
+              for (int v = 0; v < 8; ++v)
+                *reinterpret_cast<float4*>(dst + 4 * v) = make_float4(__uint_as_float(r[4 * v]), __uint_as_float(r[4 * v + 1]),
+                                                                    __uint_as_float(r[4 * v + 2]), __uint_as_float(r[4 * v + 3]));
+              continue;
+            }
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               if (col + j < N) {
@@ -383,7 +409,8 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
               for (int j = 0; j < 16; ++j) {
                 const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
                 const float u0 = __uint_as_float(u[2 * j]), u1 = __uint_as_float(u[2 * j + 1]);
-                o[j] = pack_bf16(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
+                o[j] = act == kActGeluTanh ? pack_bf16(gelu_tanh_fast(g0) * u0, gelu_tanh_fast(g1) * u1)
+                                           : pack_bf16(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
               }
             } else {
               uint32_t r[32];
@@ -454,7 +481,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                     dst = sc->staging[sc->rank] + static_cast<size_t>(grow) * N + gcol;
                   }
                 } else {
-                  dst = C + static_cast<size_t>(grow) * ldc + gcol;
+                  dst = C + static_cast<size_t>(grow) * ldc + c_off + gcol;
                 }
                 const bool full = (gcol + 8 <= out_cols);
                 if constexpr (EPI == kEpiResidual) {
@@ -729,12 +756,12 @@ static int launch_gemm(const void* A, const void* W, void* C, const void* bias, 
                        int N, int K, int lda, int ldw, int ldc, int ldr, int* status, cudaStream_t stream,
                        const TpScatter* sc = nullptr, const int* group_tab = nullptr, const int* group_mtiles = nullptr,
                        int experts = 1, int max_mtiles = 0, uint32_t* a_ready = nullptr, uint32_t* a_done = nullptr,
-                       unsigned long long a_wait_ns = 0) {
+                       unsigned long long a_wait_ns = 0, GemmBatch batch = GemmBatch(), int act = kActSilu) {
   using Cfg = GemmCfg<BN>;
   CUtensorMap ta, tb;
-  int rc = make_tmap_bf16_2d(&ta, A, M, K, lda, kBM, kBK);
+  int rc = make_tmap_bf16_2d(&ta, A, M, static_cast<uint64_t>(batch.count - 1) * batch.a_step + K, lda, kBM, kBK);
   if (rc != 0) return rc;
-  rc = make_tmap_bf16_2d(&tb, W, static_cast<uint64_t>(N) * experts, K, ldw, BN, kBK);
+  rc = make_tmap_bf16_2d(&tb, W, static_cast<uint64_t>(N) * experts * batch.count, K, ldw, BN, kBK);
   if (rc != 0) return rc;
   static bool attr_set = false;
   if (!attr_set) {
@@ -743,7 +770,7 @@ static int launch_gemm(const void* A, const void* W, void* C, const void* bias, 
     attr_set = true;
   }
   const int m_tiles = group_tab != nullptr ? max_mtiles : (M + kBM - 1) / kBM, n_tiles = (N + BN - 1) / BN;
-  const int tiles = m_tiles * n_tiles;
+  const int tiles = m_tiles * n_tiles * batch.count;
   const int sms = ogb_num_sms();
   int grid = tiles;
   if (grid > sms) grid = sms;
@@ -770,14 +797,14 @@ static int launch_gemm(const void* A, const void* W, void* C, const void* bias, 
       gemm_bf16_tcgen05_kernel<BN, EPI>, dim3(grid), dim3(EPI == kEpiScatter ? kGemmThreadsScatter : kGemmThreads), Cfg::kSmemBytes, stream,
       pdl, ta, tb, static_cast<__nv_bfloat16*>(C), static_cast<const __nv_bfloat16*>(bias), static_cast<const __nv_bfloat16*>(residual),
       static_cast<float*>(C_f32), M, N, K, ldc, ldr, status, sc, group_tab, group_mtiles, a_ready, a_done,
-      static_cast<unsigned long long>(a_wait_ns), sk_ws, sk_flags, sk_seq));
+      static_cast<unsigned long long>(a_wait_ns), sk_ws, sk_flags, sk_seq, batch, act));
 }
 
 }  // namespace ogb
 
 using namespace ogb;
 
-#define OGB_GEMM_ARGS A, W, C, bias, residual, C_f32, M, N, K, lda, ldw, ldc, ldr, status, stream, nullptr, nullptr, nullptr, 1, 0, a_ready, a_done, a_wait_ns
+#define OGB_GEMM_ARGS A, W, C, bias, residual, C_f32, M, N, K, lda, ldw, ldc, ldr, status, stream, nullptr, nullptr, nullptr, 1, 0, a_ready, a_done, a_wait_ns, batch, act
 #define OGB_GEMM_DISPATCH_BN(EPI)                              \
   switch (bn) {                                                \
     case 32: return launch_gemm<32, EPI>(OGB_GEMM_ARGS);       \
@@ -809,9 +836,9 @@ extern "C" int ogb_gemm_bf16(const void* A, const void* W, void* C, const void* 
   return ogb_gemm_bf16_wait(A, W, C, bias, residual, C_f32, M, N, K, lda, ldw, ldc, ldr, epilogue, bn, nullptr, nullptr, 0, status, stream_);
 }
 
-extern "C" int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const void* bias, const void* residual, void* C_f32,
-                                  int M, int N, int K, int lda, int ldw, int ldc, int ldr, int epilogue, int bn,
-                                  uint32_t* a_ready, uint32_t* a_done, unsigned long long a_wait_ns, int* status, void* stream_) {
+static int gemm_bf16_dispatch(const void* A, const void* W, void* C, const void* bias, const void* residual, void* C_f32, int M, int N, int K,
+                              int lda, int ldw, int ldc, int ldr, int epilogue, int bn, uint32_t* a_ready, uint32_t* a_done,
+                              unsigned long long a_wait_ns, GemmBatch batch, int act, int* status, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (a_ready != nullptr && a_done == nullptr) return -8;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
@@ -819,6 +846,7 @@ extern "C" int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const v
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C)) & 15) return -4;
   if (epilogue == kEpiResidual && (residual == nullptr || (ldr % 8) != 0)) return -5;
   if (epilogue == kEpiSwiGLU && (bn < 64 || (N % bn) != 0 || C_f32 != nullptr)) return -6;
+  if (batch.count < 1 || (batch.a_step % 8) != 0 || (batch.c_step % 8) != 0 || (batch.count > 1 && (a_ready != nullptr || epilogue != kEpiNone))) return -9;
   if (bn == 0) {
     // Tiles are handed out round-robin to one persistent CTA per SM, so the kernel takes
     // ceil(tiles / SMs) "waves" of one tile time each.  Pick the tile width with the lowest
@@ -834,7 +862,7 @@ extern "C" int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const v
     bn = 256;
     for (int i = 0; i < 5; ++i) {
       if (cand[i] < 128 && m_tiles > 3) break;  // narrow tiles only pay off for decode-sized M
-      const int tiles = m_tiles * ((N + cand[i] - 1) / cand[i]);
+      const int tiles = m_tiles * ((N + cand[i] - 1) / cand[i]) * batch.count;
       const float t = launch_cost(tiles, (K + kBK - 1) / kBK, sms, cost[i], kSkFixPlain);
       if (t < best - 1e-6f) { best = t; bn = cand[i]; }
     }
@@ -850,6 +878,30 @@ extern "C" int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const v
     }
   }
   return -7;
+}
+
+extern "C" int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const void* bias, const void* residual, void* C_f32,
+                                  int M, int N, int K, int lda, int ldw, int ldc, int ldr, int epilogue, int bn,
+                                  uint32_t* a_ready, uint32_t* a_done, unsigned long long a_wait_ns, int* status, void* stream_) {
+  return gemm_bf16_dispatch(A, W, C, bias, residual, C_f32, M, N, K, lda, ldw, ldc, ldr, epilogue, bn, a_ready, a_done, a_wait_ns, GemmBatch(),
+                            kActSilu, status, stream_);
+}
+
+// Gated product over a packed gate | up weight with the activation chosen by `act` (0 silu, 1 tanh form of gelu).
+extern "C" int ogb_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, int bn,
+                                   int* status, void* stream) {
+  if (act != kActSilu && act != kActGeluTanh) return -7;
+  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, kEpiSwiGLU, bn, nullptr, nullptr, 0, GemmBatch(), act,
+                            status, stream);
+}
+
+// `batch` products of one shape (see GemmBatch): C[:, z*c_step : +N] = A[:, z*a_step : +K] * W[z*N : +N, :]^T.
+extern "C" int ogb_gemm_bf16_batched(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int batch,
+                                     int a_step, int c_step, int* status, void* stream) {
+  GemmBatch b;
+  b.count = batch; b.a_step = a_step; b.c_step = c_step;
+  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, kEpiNone, 0, nullptr, nullptr, 0, b, kActSilu, status,
+                            stream);
 }
 
 // Row-parallel GEMM of a tensor-parallel group: the partial product A[M,K_local] * W[N,K_local]^T of

@@ -1,0 +1,415 @@
+// Row-wise kernels of models with hyper-connected residual streams, Dynamic-Tanh norms, token shift and latent KV pages,
+// plus the fp32 matrix product of the 32-bit engine.
+//
+// hyper_step is the one pass between two matrix products: it folds a sublayer's output y into the residual streams
+// (x_t <- sum_s mix[s][t] x_s + out[t] y), reads the next sublayer's input (u = sum_s in[s] x_s), applies the
+// Dynamic-Tanh norm (tanh(alpha u) w + b) and, where the mixer wants it, the token shift (h + (h_before - h) amount).
+// Everything is elementwise in the column, so a thread keeps its columns and walks a few tokens; the row before its
+// first token is computed again from the streams the pass reads (the streams are double buffered), or comes from the
+// sequence's state.  Streams, norm and shift are fp32 whatever the activation type.
+#include <algorithm>
+
+#include "hybrid.cuh"
+#include "ogb_kernels.h"
+
+namespace ogb {
+
+constexpr int kHsThreads = 256;
+constexpr int kHsRows = 16;                   // tokens a thread walks (a 64-row scheduler tile is four such groups)
+
+struct HyperParams {
+  const float* x_in;       // [rows, S, W]
+  float* x_out;            // [rows, S, W] or null (nothing to write back)
+  const void* y;           // [rows, ldy] or null (no update)
+  const float *mix, *out_w, *in_w;             // [S, S] (from, to), [S], [S] (null: ones)
+  const float *alpha, *w, *b;                  // Dynamic-Tanh norm (alpha null: none)
+  const float* shift;      // [W] or null
+  float* prev;             // [slots, W] state of the shift: h of the sequence's last computed token
+  void* h;                 // [rows, ldh] or null
+  const int* gather;       // row r of h comes from row gather[r] (final norm of the rows that sample)
+  int rows, total_rows, S, W, ldy, ldh;
+  StepRows sr;
+  int* status;
+};
+
+template <typename T, int SMAX, int V>
+struct HyperCol {
+  const HyperParams& p;
+  int c;                                       // first column of this thread
+  float mix[SMAX][SMAX], out_w[SMAX], in_w[SMAX];
+  float alpha, w[V], b[V];
+
+  OGB_DEVICE HyperCol(const HyperParams& p_, int c_) : p(p_), c(c_) {
+#pragma unroll
+    for (int s = 0; s < SMAX; ++s) {
+      const bool live = s < p.S;
+      in_w[s] = live ? (p.in_w != nullptr ? p.in_w[s] : 1.f) : 0.f;
+      out_w[s] = (live && p.y != nullptr) ? p.out_w[s] : 0.f;
+#pragma unroll
+      for (int t = 0; t < SMAX; ++t) mix[s][t] = (live && t < p.S && p.y != nullptr) ? p.mix[s * p.S + t] : 0.f;
+    }
+    alpha = p.alpha != nullptr ? *p.alpha : 0.f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      w[i] = p.alpha != nullptr ? p.w[c + i] : 1.f;
+      b[i] = p.alpha != nullptr ? p.b[c + i] : 0.f;
+    }
+  }
+
+  // streams of row t after the update, normed read-out in hv
+  OGB_DEVICE void row(int t, bool write, float (&hv)[V]) const {
+    float x[SMAX][V], y[V], u[V];
+    const float* src = p.x_in + static_cast<size_t>(t) * p.S * p.W + c;
+#pragma unroll
+    for (int s = 0; s < SMAX; ++s)
+      if (s < p.S) load_vec<V>(src + static_cast<size_t>(s) * p.W, x[s]);
+    if (p.y != nullptr) {
+      load_vec<V>(static_cast<const T*>(p.y) + static_cast<size_t>(t) * p.ldy + c, y);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        float n[SMAX];
+#pragma unroll
+        for (int q = 0; q < SMAX; ++q) {
+          n[q] = out_w[q] * y[i];
+#pragma unroll
+          for (int s = 0; s < SMAX; ++s)
+            if (s < p.S) n[q] = fmaf(mix[s][q], x[s][i], n[q]);
+        }
+#pragma unroll
+        for (int q = 0; q < SMAX; ++q) x[q][i] = n[q];
+      }
+      if (write && p.x_out != nullptr) {
+        float* dst = p.x_out + static_cast<size_t>(t) * p.S * p.W + c;
+#pragma unroll
+        for (int s = 0; s < SMAX; ++s)
+          if (s < p.S) store_vec<V>(dst + static_cast<size_t>(s) * p.W, x[s]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      u[i] = 0.f;
+#pragma unroll
+      for (int s = 0; s < SMAX; ++s)
+        if (s < p.S) u[i] = fmaf(in_w[s], x[s][i], u[i]);
+      hv[i] = p.alpha != nullptr ? fmaf(tanhf(alpha * u[i]), w[i], b[i]) : u[i];
+    }
+  }
+};
+
+// rows are independent: no shift
+template <typename T, int SMAX, int V>
+__global__ void __launch_bounds__(kHsThreads) hyper_rows_kernel(HyperParams p) {
+  const int c = (blockIdx.y * kHsThreads + threadIdx.x) * V;
+  if (c >= p.W) return;
+  HyperCol<T, SMAX, V> col(p, c);
+  const int r0 = blockIdx.x * kHsRows;
+#pragma unroll 2
+  for (int j = 0; j < kHsRows; ++j) {
+    const int r = r0 + j;
+    if (r >= p.rows) return;
+    int t = r;
+    if (p.gather != nullptr) {
+      t = p.gather[r];
+      if (t < 0 || t >= p.total_rows) {
+        if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
+        t = 0;
+      }
+    }
+    float hv[V];
+    col.row(t, true, hv);
+    if (p.h != nullptr) store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r) * p.ldh + c, hv);
+  }
+}
+
+// with the token shift: a block is one decode row or kHsRows rows of one prefill chunk
+template <typename T, int SMAX, int V>
+__global__ void __launch_bounds__(kHsThreads) hyper_shift_kernel(HyperParams p) {
+  const int c = (blockIdx.y * kHsThreads + threadIdx.x) * V;
+  if (c >= p.W) return;
+  const StepRows& sr = p.sr;
+  int entry, base, n, j0;                      // sequence entry, its first row, its rows, first row of this block within them
+  if (static_cast<int>(blockIdx.x) < sr.num_decode) {
+    entry = blockIdx.x; base = blockIdx.x; n = 1; j0 = 0;
+  } else {
+    const int g = blockIdx.x - sr.num_decode;
+    const int tile = g / (64 / kHsRows);
+    const int s = sr.tile_seq[tile];
+    entry = sr.num_decode + s;
+    base = sr.num_decode + sr.cu_q[s];
+    n = sr.cu_q[s + 1] - sr.cu_q[s];
+    j0 = sr.tile_q0[tile] + (g % (64 / kHsRows)) * kHsRows;
+    if (j0 >= n) return;
+  }
+  int slot = sr.state_slot[entry];
+  if (slot >= sr.num_slots) {
+    if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
+    slot = -1;
+  }
+  HyperCol<T, SMAX, V> col(p, c);
+  float amount[V], before[V], hv[V], o[V];
+  load_vec<V>(p.shift + c, amount);
+  float* state = slot >= 0 ? p.prev + static_cast<size_t>(slot) * p.W + c : nullptr;
+#pragma unroll
+  for (int i = 0; i < V; ++i) before[i] = 0.f;
+  if (j0 > 0) {
+    col.row(base + j0 - 1, false, before);
+  } else {
+    if (state != nullptr && sr.ctx_len[entry] > n) load_vec<V>(state, before);
+    // this block also leaves the chunk's last h behind: it is the only one that reads the slot, so the order is safe
+    if (state != nullptr && n > kHsRows) {
+      col.row(base + n - 1, false, hv);
+      store_vec<V>(state, hv);
+    }
+  }
+  const int j1 = min(j0 + kHsRows, n);
+#pragma unroll 2
+  for (int j = j0; j < j1; ++j) {
+    col.row(base + j, true, hv);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      o[i] = fmaf(before[i] - hv[i], amount[i], hv[i]);
+      before[i] = hv[i];
+    }
+    store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(base + j) * p.ldh + c, o);
+  }
+  if (state != nullptr && j0 == 0 && n <= kHsRows) store_vec<V>(state, before);
+}
+
+template <typename T, int SMAX, int V>
+static int launch_hyper(const HyperParams& p, cudaStream_t stream) {
+  const int cols = (p.W + V * kHsThreads - 1) / (V * kHsThreads);
+  if (p.shift != nullptr) {
+    const int blocks = p.sr.num_decode + p.sr.num_tiles * (64 / kHsRows);
+    hyper_shift_kernel<T, SMAX, V><<<dim3(blocks, cols), kHsThreads, 0, stream>>>(p);
+  } else {
+    hyper_rows_kernel<T, SMAX, V><<<dim3((p.rows + kHsRows - 1) / kHsRows, cols), kHsThreads, 0, stream>>>(p);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+template <typename T, int V>
+static int dispatch_hyper(const HyperParams& p, cudaStream_t stream) {
+  if (p.S <= 2) return launch_hyper<T, 2, V>(p, stream);
+  if (p.S <= 4) return launch_hyper<T, 4, V>(p, stream);
+  return launch_hyper<T, 8, V>(p, stream);
+}
+
+// ------------------------------------------------------------------------------------------------------
+// all streams of a row start as the token's embedding
+// ------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) embed_streams_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
+                                                            int S, int W, int vocab, int* status) {
+  const int t = blockIdx.x;
+  int id = ids[t];
+  if (id < 0 || id >= vocab) {
+    if (threadIdx.x == 0) atomicOr(status, kStatusIndexOutOfRange);
+    id = 0;
+  }
+  const T* src = table + static_cast<size_t>(id) * W;
+  float* dst = x + static_cast<size_t>(t) * S * W;
+  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    const float v = to_f32<T>(src[c]);
+    for (int s = 0; s < S; ++s) dst[static_cast<size_t>(s) * W + c] = v;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------
+// latent pages: RMS norm of a projected row, written to its page.  pool [pages, 16, ldp]; one warp per token.
+// ------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128) latent_append_kernel(const T* __restrict__ c, int ldc, const float* __restrict__ w, float eps,
+                                                            const int* __restrict__ slots, T* __restrict__ pool, int tokens, int rank,
+                                                            int ldp, int64_t num_slots, int* status) {
+  const int lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (t >= tokens) return;
+  const int slot = slots[t];
+  if (slot < 0) return;                        // padding row
+  if (slot >= num_slots) {
+    if (lane == 0) atomicOr(status, kStatusIndexOutOfRange);
+    return;
+  }
+  const T* src = c + static_cast<size_t>(t) * ldc;
+  float ss = 0.f;
+  for (int i = lane; i < rank; i += 32) { const float v = to_f32<T>(src[i]); ss = fmaf(v, v, ss); }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(rank) + eps);
+  T* dst = pool + static_cast<size_t>(slot) * ldp;
+  for (int i = lane; i < rank; i += 32) dst[i] = from_f32<T>(to_f32<T>(src[i]) * inv * w[i]);
+}
+
+// ------------------------------------------------------------------------------------------------------
+// RMS norm of every group of `n` columns (a head) with one shared weight: fp32 in, activation type out; one warp per group
+// ------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, T* __restrict__ out,
+                                                           int rows, int heads, int n, int ldx, int ldo) {
+  const int lane = threadIdx.x & 31;
+  const long long g = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (g >= static_cast<long long>(rows) * heads) return;
+  const int t = static_cast<int>(g / heads), h = static_cast<int>(g % heads);
+  const float* src = x + static_cast<size_t>(t) * ldx + static_cast<size_t>(h) * n;
+  T* dst = out + static_cast<size_t>(t) * ldo + static_cast<size_t>(h) * n;
+  float ss = 0.f;
+  if ((n & 127) == 0 && n <= 512 && (ldx & 3) == 0 && (ldo & 3) == 0) {
+    float v[4][4];
+    const int per = n >> 7;
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (k < per) {
+        load_vec<4>(src + k * 128 + lane * 4, v[k]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss = fmaf(v[k][i], v[k][i], ss);
+      }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (k < per) {
+        float wv[4];
+        load_vec<4>(w + k * 128 + lane * 4, wv);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[k][i] *= inv * wv[i];
+        store_vec<4>(dst + k * 128 + lane * 4, v[k]);
+      }
+    return;
+  }
+  for (int i = lane; i < n; i += 32) ss = fmaf(src[i], src[i], ss);
+  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
+  for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(src[i] * inv * w[i]);
+}
+
+// ------------------------------------------------------------------------------------------------------
+// gated activation over tile-interleaved gate | up columns (ops.pack_gate_up): act 0 = silu, 1 = tanh form of gelu
+// ------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) act_mul_packed_kernel(const T* __restrict__ gu, T* __restrict__ out, int rows, int inter, int half, int act) {
+  const long long total = static_cast<long long>(rows) * inter;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
+    const int t = static_cast<int>(i / inter), j = static_cast<int>(i % inter);
+    const T* row = gu + static_cast<size_t>(t) * 2 * inter + static_cast<size_t>(j / half) * 2 * half + j % half;
+    const float g = to_f32<T>(row[0]), u = to_f32<T>(row[half]);
+    const float a = act == 1 ? 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.f + expf(-g));
+    out[i] = from_f32<T>(a * u);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------
+// fp32 matrix product (no reduced-precision mode): C[M,N] = A[M,K] W[N,K]^T for `batch` problems whose operands start at
+// column offsets of A and C and at row offsets of W.  64 x 64 tile, 4 x 4 results per thread.
+// ------------------------------------------------------------------------------------------------------
+constexpr int kF32Tile = 64, kF32K = 16;
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W, float* __restrict__ C, int M,
+                                                       int N, int K, int lda, int ldw, int ldc, int a_step, int c_step) {
+  __shared__ float sa[kF32K][kF32Tile + 4], sw[kF32K][kF32Tile + 4];
+  A += static_cast<size_t>(blockIdx.z) * a_step;
+  W += static_cast<size_t>(blockIdx.z) * N * ldw;
+  C += static_cast<size_t>(blockIdx.z) * c_step;
+  const int m0 = blockIdx.y * kF32Tile, n0 = blockIdx.x * kF32Tile;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kF32K) {
+    for (int i = threadIdx.x; i < kF32Tile * kF32K; i += 256) {
+      const int r = i / kF32K, k = i % kF32K;
+      sa[k][r] = (m0 + r < M && k0 + k < K) ? A[static_cast<size_t>(m0 + r) * lda + k0 + k] : 0.f;
+      sw[k][r] = (n0 + r < N && k0 + k < K) ? W[static_cast<size_t>(n0 + r) * ldw + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kF32K; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { a[i] = sa[k][ty * 4 + i]; b[i] = sw[k][tx * 4 + i]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = m0 + ty * 4 + i, c = n0 + tx * 4 + j;
+      if (r < M && c < N) C[static_cast<size_t>(r) * ldc + c] = acc[i][j];
+    }
+}
+
+}  // namespace ogb
+
+using namespace ogb;
+
+extern "C" int ogb_hyper_step(const float* x_in, float* x_out, const void* y, const float* mix, const float* out_w, const float* in_w,
+                              const float* alpha, const float* w, const float* b, const float* shift, float* prev, void* h,
+                              const int* gather, int rows, int total_rows, int S, int W, int ldy, int ldh, const int* ctx_len,
+                              const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode,
+                              int num_tiles, int num_slots, int elem, int* status, void* stream) {
+  if (rows <= 0) return 0;
+  if (S < 1 || S > 8 || W < 1 || x_in == x_out) return -3;
+  if (shift != nullptr && (prev == nullptr || h == nullptr || gather != nullptr)) return -3;
+  if (y != nullptr && (mix == nullptr || out_w == nullptr)) return -3;
+  HyperParams p{x_in, x_out, y, mix, out_w, in_w, alpha, w, b, shift, prev, h, gather, rows, total_rows, S, W, ldy, ldh,
+                StepRows{ctx_len, state_slot, cu_q, tile_seq, tile_q0, num_decode, num_tiles, num_slots}, status};
+  const bool vec = W % 4 == 0 && ldy % 4 == 0 && ldh % 4 == 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (elem == kElemBF16) return vec ? dispatch_hyper<__nv_bfloat16, 4>(p, s) : dispatch_hyper<__nv_bfloat16, 1>(p, s);
+  if (elem == kElemF32) return vec ? dispatch_hyper<float, 4>(p, s) : dispatch_hyper<float, 1>(p, s);
+  return -3;
+}
+
+extern "C" int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, int elem, int* status,
+                                 void* stream) {
+  if (tokens <= 0) return 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (elem == kElemBF16) embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const __nv_bfloat16*>(table), x, S, W, vocab, status);
+  else if (elem == kElemF32) embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const float*>(table), x, S, W, vocab, status);
+  else return -3;
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int ogb_latent_append(const void* c, int ldc, const float* w, float eps, const int* slots, void* pool, int tokens, int rank,
+                                 int ldp, int64_t num_slots, int elem, int* status, void* stream) {
+  if (tokens <= 0) return 0;
+  if (rank > ldp) return -3;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int blocks = (tokens + 3) / 4;
+  if (elem == kElemBF16)
+    latent_append_kernel<<<blocks, 128, 0, s>>>(static_cast<const __nv_bfloat16*>(c), ldc, w, eps, slots, static_cast<__nv_bfloat16*>(pool), tokens,
+                                                rank, ldp, num_slots, status);
+  else if (elem == kElemF32)
+    latent_append_kernel<<<blocks, 128, 0, s>>>(static_cast<const float*>(c), ldc, w, eps, slots, static_cast<float*>(pool), tokens, rank, ldp,
+                                                num_slots, status);
+  else return -3;
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, int elem,
+                                void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * heads + 7) / 8);
+  if (elem == kElemBF16) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo);
+  else if (elem == kElemF32) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo);
+  else return -3;
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, int elem, void* stream) {
+  if (rows <= 0) return 0;
+  if (half <= 0 || inter % half != 0 || act < 0 || act > 1) return -3;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int blocks = static_cast<int>(std::min<long long>((static_cast<long long>(rows) * inter + 255) / 256, 148 * 16));
+  if (elem == kElemBF16)
+    act_mul_packed_kernel<<<blocks, 256, 0, s>>>(static_cast<const __nv_bfloat16*>(gate_up), static_cast<__nv_bfloat16*>(out), rows, inter, half, act);
+  else if (elem == kElemF32)
+    act_mul_packed_kernel<<<blocks, 256, 0, s>>>(static_cast<const float*>(gate_up), static_cast<float*>(out), rows, inter, half, act);
+  else return -3;
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int ogb_gemm_f32(const float* A, const float* W, float* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step,
+                            int c_step, void* stream) {
+  if (M <= 0 || N <= 0 || batch <= 0) return 0;
+  const dim3 grid((N + kF32Tile - 1) / kF32Tile, (M + kF32Tile - 1) / kF32Tile, batch);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, M, N, K, lda, ldw, ldc, a_step, c_step);
+  return static_cast<int>(cudaGetLastError());
+}

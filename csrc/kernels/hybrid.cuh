@@ -1,0 +1,57 @@
+// Shared pieces of the kernels behind models with a per-layer mixer choice (hybrid.cu, recurrent.cu,
+// latent_attention.cu): the row structure of a step and loads / stores of the two activation types.
+// These files are compiled without fast math: tanh, exponentials, divisions and roots keep their full precision.
+#pragma once
+#include "common.cuh"
+
+namespace ogb {
+
+enum ElemType : int { kElemF32 = 0, kElemBF16 = 1 };
+
+template <typename T> OGB_DEVICE float to_f32(T v);
+template <> OGB_DEVICE float to_f32<float>(float v) { return v; }
+template <> OGB_DEVICE float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> OGB_DEVICE T from_f32(float v);
+template <> OGB_DEVICE float from_f32<float>(float v) { return v; }
+template <> OGB_DEVICE __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+// V consecutive elements as fp32 (one vector access where V = 4; the pointer is then aligned to it)
+template <int V, typename T>
+OGB_DEVICE void load_vec(const T* p, float (&r)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    r[0] = f.x; r[1] = f.y; r[2] = f.z; r[3] = f.w;
+  } else if constexpr (V == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16(u.x), b = unpack_bf16(u.y);
+    r[0] = a.x; r[1] = a.y; r[2] = b.x; r[3] = b.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) r[i] = to_f32<T>(p[i]);
+  }
+}
+template <int V, typename T>
+OGB_DEVICE void store_vec(T* p, const float (&r)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(r[0], r[1], r[2], r[3]);
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]));
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) p[i] = from_f32<T>(r[i]);
+  }
+}
+
+// Rows of a step: `num_decode` single-token rows (row r belongs to sequence entry r), then the packed prefill chunks
+// (sequence entry num_decode + s holds rows num_decode + cu_q[s] .. num_decode + cu_q[s + 1]).  ctx_len counts an entry's
+// tokens after the step, so its first row sits at position ctx_len - rows.
+struct StepRows {
+  const int* ctx_len;
+  const int* state_slot;
+  const int* cu_q;
+  const int* tile_seq;
+  const int* tile_q0;
+  int num_decode, num_tiles, num_slots;
+};
+
+}  // namespace ogb

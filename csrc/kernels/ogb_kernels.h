@@ -24,6 +24,16 @@ int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const void* bias, 
                        int N, int K, int lda, int ldw, int ldc, int ldr, int epilogue, int bn, uint32_t* a_ready,
                        uint32_t* a_done, unsigned long long a_wait_ns, int* status, void* stream);
 
+// Gated product over a packed gate | up weight (tile width bn), activation act: 0 = silu, 1 = tanh form of gelu.
+int ogb_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, int bn,
+                        int* status, void* stream);
+// `batch` products of one shape: C[:, z*c_step : +N] = A[:, z*a_step : +K] * W[z*N : +N, :]^T (steps are multiples of 8).
+int ogb_gemm_bf16_batched(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step,
+                          int c_step, int* status, void* stream);
+// The same in fp32 without any reduced-precision mode.
+int ogb_gemm_f32(const float* A, const float* W, float* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step, int c_step,
+                 void* stream);
+
 // Stream-K decomposition of the GEMMs (on by default; OGB_STREAM_K=0 disables it): 1 / 0 sets it, the old value is returned.
 int ogb_gemm_set_stream_k(int on);
 // Programmatic dependent launch along scatter GEMM -> exchange kernel -> consuming GEMM (off by default; OGB_TP_PDL=1
@@ -145,6 +155,31 @@ int ogb_index_share_attention(const void* q, const void* k, const void* v, const
 // cache [B,G,C,row] and int64 idx [B,G,Q,K] -> out [B,G,Q,K,row]; an index outside the row's valid length sets the status word.
 int ogb_sparse_kv_gather(const void* cache, const void* idx, const void* lengths, void* out, int B, int G, int C, int Q, int K,
                          int row_bytes, int* status, void* stream);
+
+// Models with a mixer per layer (hybrid.cu, recurrent.cu, latent_attention.cu).  elem: 0 = fp32, 1 = bf16 activations; residual
+// streams, norms, gates and recurrent state are fp32 either way.  ctx_len, state_slot and the page table have one entry per
+// sequence of the step (decode rows first); cu_q, tile_seq and tile_q0 describe the prefill chunks as everywhere else.
+// hyper_step: fold y into the streams (x_in -> x_out), read the next sublayer's input, Dynamic-Tanh norm, token shift -> h.
+int ogb_hyper_step(const float* x_in, float* x_out, const void* y, const float* mix, const float* out_w, const float* in_w, const float* alpha,
+                   const float* w, const float* b, const float* shift, float* prev, void* h, const int* gather, int rows, int total_rows, int S,
+                   int W, int ldy, int ldh, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0,
+                   int num_decode, int num_tiles, int num_slots, int elem, int* status, void* stream);
+int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, int elem, int* status, void* stream);
+int ogb_latent_append(const void* c, int ldc, const float* w, float eps, const int* slots, void* pool, int tokens, int rank, int ldp,
+                      int64_t num_slots, int elem, int* status, void* stream);
+int ogb_latent_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
+                         const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages, int num_tiles,
+                         int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml, int elem, int* status,
+                         void* stream);
+int ogb_hgrn2_state_rows(int D);
+int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D, int V,
+              const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int* status,
+              void* stream);
+int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, int elem, void* stream);
+int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, int elem, void* stream);
+int ogb_argmax_f32(const float* logits, int* out_tokens, int rows, int vocab, int ld, void* stream);
+int ogb_sample_f32(const float* logits, int* out_tokens, const float* temperature, const int* top_k, const float* top_p, const float* min_p,
+                   const float* uniform, uint32_t* work, int rows, int vocab, int ld, void* stream);
 
 // MoE: softmax router with top-k (renormalised), device-side permutation by expert, grouped GEMM, combine.
 int ogb_moe_route_topk(const void* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k,

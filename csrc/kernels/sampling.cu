@@ -46,16 +46,21 @@ OGB_DEVICE ArgMax block_argmax(ArgMax a, ArgMax* sh /*[32]*/) {
   r = warp_argmax(r);
   return r;  // identical in every thread
 }
-OGB_DEVICE ArgMax row_argmax(const __nv_bfloat16* row, int vocab, ArgMax* sh) {
+OGB_DEVICE float logit_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+OGB_DEVICE float logit_f32(float v) { return v; }
+
+template <typename T>
+OGB_DEVICE ArgMax row_argmax(const T* row, int vocab, ArgMax* sh) {
   ArgMax best{-INFINITY, 0x7fffffff};
   for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
-    const float v = __bfloat162float(row[i]);
+    const float v = logit_f32(row[i]);
     if (v > best.v) { best.v = v; best.i = i; }  // strided scan keeps the lowest index per thread on ties
   }
   return block_argmax(best, sh);
 }
 
-__global__ void __launch_bounds__(kSampleThreads) argmax_kernel(const __nv_bfloat16* __restrict__ logits,
+template <typename T>
+__global__ void __launch_bounds__(kSampleThreads) argmax_kernel(const T* __restrict__ logits,
                                                                  int* __restrict__ out, int vocab, int ld) {
   __shared__ ArgMax sh[32];
   const ArgMax r = row_argmax(logits + static_cast<size_t>(blockIdx.x) * ld, vocab, sh);
@@ -160,8 +165,9 @@ OGB_DEVICE uint32_t radix_threshold(const uint32_t* __restrict__ w, int vocab, u
   return prefix < floor_w ? floor_w : prefix;
 }
 
+template <typename T>
 __global__ void __launch_bounds__(kSampleThreads)
-sample_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out, const float* __restrict__ temperature,
+sample_kernel(const T* __restrict__ logits, int* __restrict__ out, const float* __restrict__ temperature,
               const int* __restrict__ top_k, const float* __restrict__ top_p, const float* __restrict__ min_p,
               const float* __restrict__ uniform, uint32_t* __restrict__ work, int vocab, int ld) {
   __shared__ ArgMax sh_arg[32];
@@ -170,7 +176,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out, c
   __shared__ unsigned long long sh_scan[kSampleThreads / 32];
   __shared__ int sh_pick;
   const int rowi = blockIdx.x;
-  const __nv_bfloat16* row = logits + static_cast<size_t>(rowi) * ld;
+  const T* row = logits + static_cast<size_t>(rowi) * ld;
   const ArgMax best = row_argmax(row, vocab, sh_arg);
   const float temp = temperature[rowi];
   if (!(temp > 0.f) || best.i == 0x7fffffff) {
@@ -181,7 +187,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out, c
   const float inv_t = 1.f / temp;
   unsigned long long local = 0;
   for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
-    const float l = __bfloat162float(row[i]);
+    const float l = logit_f32(row[i]);
     float e = __expf((l - best.v) * inv_t);   // in (0, 1]; NaN logits get weight 0
     if (!(e >= 0.f)) e = 0.f;
     uint32_t q = static_cast<uint32_t>(e * 1073741824.f + 0.5f);
@@ -598,6 +604,21 @@ extern "C" int ogb_sample_bf16(const void* logits, int* out_tokens, const float*
   }
   sample_kernel<<<rows, kSampleThreads, 0, static_cast<cudaStream_t>(stream)>>>(
       static_cast<const __nv_bfloat16*>(logits), out_tokens, temperature, top_k, top_p, min_p, uniform, work, vocab, ld);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// The same over fp32 logits (the 32-bit engine).
+extern "C" int ogb_argmax_f32(const float* logits, int* out_tokens, int rows, int vocab, int ld, void* stream) {
+  if (rows <= 0) return 0;
+  argmax_kernel<<<rows, kSampleThreads, 0, static_cast<cudaStream_t>(stream)>>>(logits, out_tokens, vocab, ld);
+  return static_cast<int>(cudaGetLastError());
+}
+extern "C" int ogb_sample_f32(const float* logits, int* out_tokens, const float* temperature, const int* top_k, const float* top_p,
+                              const float* min_p, const float* uniform, uint32_t* work, int rows, int vocab, int ld, void* stream) {
+  if (rows <= 0) return 0;
+  if (work == nullptr) return -4;
+  sample_kernel<<<rows, kSampleThreads, 0, static_cast<cudaStream_t>(stream)>>>(logits, out_tokens, temperature, top_k, top_p, min_p, uniform,
+                                                                               work, vocab, ld);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -142,7 +142,7 @@ static PlanLayout make_layout(const CoreConfig& c) {
   l.max_tiles = c.max_tokens_per_step / 64 + c.max_seqs + 1;
   l.tile_seq = take(l.max_tiles);
   l.tile_q0 = take(l.max_tiles);
-  l.max_rows = c.max_seqs * (1 + (c.max_draft_tokens > 0 ? c.max_draft_tokens : 0));
+  l.max_rows = std::max(c.max_logit_rows, c.max_seqs * (1 + (c.max_draft_tokens > 0 ? c.max_draft_tokens : 0)));
   l.logit_rows = take(l.max_rows);
   l.temperature = take(l.max_rows);
   l.top_k = take(l.max_rows);
@@ -150,6 +150,7 @@ static PlanLayout make_layout(const CoreConfig& c) {
   l.min_p = take(l.max_rows);
   l.uniform = take(l.max_rows);
   l.logit_seq = take(l.max_rows);
+  l.state_slot = take(c.max_seqs);
   l.copy_src = take(c.max_seqs);
   l.copy_dst = take(c.max_seqs);
   l.max_swap = c.max_seqs * c.max_pages_per_seq;
@@ -166,6 +167,41 @@ static PlanLayout make_layout(const CoreConfig& c) {
 
 Core::Core(const CoreConfig& cfg) : cfg_(cfg), layout_(make_layout(cfg)), pool_(cfg.num_pages) {
   for (int i = cfg.num_host_pages - 1; i >= 0; --i) host_free_.push_back(i);
+  for (int i = cfg.num_state_slots - 1; i >= 0; --i) state_free_.push_back(i);
+  if (stateful()) {
+    cfg_.enable_prefix_cache = false;
+    cfg_.max_draft_tokens = 0;
+    cfg_.preempt = PreemptMode::Recompute;
+  }
+}
+
+bool Core::acquire_state(Sequence& s) {
+  if (!stateful() || s.state_slot >= 0) return true;
+  if (state_free_.empty()) return false;
+  s.state_slot = state_free_.back();
+  state_free_.pop_back();
+  return true;
+}
+
+void Core::release_state(Sequence& s) {
+  if (s.state_slot < 0) return;
+  state_free_.push_back(s.state_slot);
+  s.state_slot = -1;
+}
+
+void Core::start_over(Sequence& s) {
+  free_pages(s, false);
+  s.num_computed = 0;
+  s.num_cached_prefix = 0;
+}
+
+bool Core::has_work() const {
+  if (!waiting_.empty() || !swapped_.empty()) return true;
+  for (int64_t id : running_) {
+    const Sequence* s = find(id);
+    if (s && !(s->forced && s->num_computed >= static_cast<int>(s->tokens.size()))) return true;
+  }
+  return false;
 }
 
 Sequence* Core::find(int64_t id) {
@@ -213,6 +249,23 @@ int64_t Core::add_request(const int32_t* prompt, int n, int max_new_tokens, cons
   seqs_.emplace(id, std::move(s));
   waiting_.push_back(id);
   return id;
+}
+
+int64_t Core::add_forced(const int32_t* tokens, int n) {
+  const int64_t id = add_request(tokens, n, 0, SamplingParams{}, 0, 0, true, nullptr, 0);
+  if (id > 0) find(id)->forced = true;
+  return id;
+}
+
+bool Core::want_logits(int64_t seq_id, const int32_t* positions, int n) {
+  Sequence* s = find(seq_id);
+  if (!s || !s->forced || n < 0) return false;
+  for (int i = 0; i < n; ++i)
+    if (positions[i] < s->num_computed || positions[i] >= static_cast<int>(s->tokens.size())) return false;
+  s->wanted.insert(s->wanted.end(), positions, positions + n);
+  std::sort(s->wanted.begin(), s->wanted.end());
+  s->wanted.erase(std::unique(s->wanted.begin(), s->wanted.end()), s->wanted.end());
+  return true;
 }
 
 void Core::free_pages(Sequence& s, bool publish_prefix) {
@@ -337,6 +390,7 @@ bool Core::preempt_one(Sequence* keep, std::vector<std::pair<int, int>>& swap_ou
     swapped_.push_back(v.id);
   } else {
     free_pages(v, true);
+    release_state(v);
     v.num_computed = 0;
     v.status = SeqStatus::Waiting;
     waiting_.push_front(v.id);
@@ -379,7 +433,7 @@ int Core::build_step(int32_t* plan) {
     Sequence* s = find(running_[i]);
     int remaining = static_cast<int>(s->tokens.size()) - s->num_computed;
     s->num_draft = 0;
-    if (remaining == 1 && !s->draft.empty() && cfg_.max_draft_tokens > 0) {
+    if (remaining == 1 && !s->draft.empty() && cfg_.max_draft_tokens > 0 && !s->forced) {
       // speculative verification: feed the last token and the drafts as one short chunk
       int k = std::min<int>(static_cast<int>(s->draft.size()), cfg_.max_draft_tokens);
       const int generated = static_cast<int>(s->tokens.size()) - s->prompt_len;
@@ -454,9 +508,11 @@ int Core::build_step(int32_t* plan) {
       const int remaining = static_cast<int>(s->tokens.size()) - s->num_computed;
       int n = std::min({remaining, budget, cfg_.prefill_chunk});
       if (n <= 0) break;
-      // keep one page of headroom per running sequence so decode rows are not starved next step
+      // keep one page of headroom per running sequence so decode rows are not starved next step (a forced sequence grows
+      // only when its caller feeds it, and the caller knows what the pool holds)
       const int need = (s->num_computed + n + kPageTokens - 1) / kPageTokens - static_cast<int>(s->pages.size());
-      if (need + static_cast<int>(running_.size()) > pool_.num_free()) {
+      const int headroom = s->forced ? 0 : static_cast<int>(running_.size());
+      if (need + headroom > pool_.num_free() || (stateful() && s->state_slot < 0 && state_free_.empty())) {
         if (s->num_cached_prefix > 0 && s->num_computed == s->num_cached_prefix) {  // give the cached pages back
           free_pages(*s, false);
           s->num_computed = 0;
@@ -465,6 +521,7 @@ int Core::build_step(int32_t* plan) {
         break;
       }
       if (!ensure_pages(*s, s->num_computed + n, copies)) break;
+      acquire_state(*s);
       waiting_.erase(std::find(waiting_.begin(), waiting_.end(), id));
       s->status = SeqStatus::Running;
       running_.push_back(id);
@@ -508,6 +565,7 @@ int Core::build_step(int32_t* plan) {
     max_ctx = std::max(max_ctx, ctx);
     plan[L.ctx_len + row] = ctx;
     plan[L.seq_slot + row] = static_cast<int32_t>(s->id & 0x7fffffff);
+    plan[L.state_slot + row] = s->state_slot;
     int32_t* pt = plan + L.page_table + static_cast<size_t>(row) * cfg_.max_pages_per_seq;
     const int np = static_cast<int>(s->pages.size());
     for (int j = 0; j < np; ++j) pt[j] = s->pages[j];
@@ -523,8 +581,19 @@ int Core::build_step(int32_t* plan) {
       }
     }
     const bool completes = (ctx == static_cast<int>(s->tokens.size()));
-    s->samples_this_step = completes;
-    if (completes) {
+    s->samples_this_step = completes && !s->forced;
+    if (s->forced) {
+      // rows for the positions the caller wants; they carry no sampling parameters and commit nothing
+      size_t taken = 0;
+      for (; taken < s->wanted.size() && s->wanted[taken] < ctx && nlog < L.max_rows; ++taken) {
+        plan[L.logit_rows + nlog] = t + s->wanted[taken] - start;
+        plan[L.logit_seq + nlog] = static_cast<int32_t>(s->id & 0x7fffffff);
+        for (int f : {L.temperature, L.top_k, L.top_p, L.min_p, L.uniform}) plan[f + nlog] = 0;
+        step_rows_.push_back(s->id);
+        ++nlog;
+      }
+      s->wanted.erase(s->wanted.begin(), s->wanted.begin() + taken);
+    } else if (completes) {
       // one logit row for the last position, or one per fed position when drafts are being verified
       const int first = s->num_draft > 0 ? 0 : n - 1;
       for (int j = first; j < n && nlog < L.max_rows; ++j) {
@@ -604,6 +673,7 @@ void Core::finish(Sequence& s, FinishReason why) {
   s.status = SeqStatus::Finished;
   s.scheduled = 0;
   free_pages(s, why != FinishReason::Error);
+  release_state(s);
   for (int hp : s.host_pages) if (hp >= 0) host_free_.push_back(hp);
   s.host_pages.clear();
   running_.erase(std::remove(running_.begin(), running_.end(), s.id), running_.end());
@@ -697,8 +767,10 @@ int64_t Core::fork(int64_t seq_id) {
   c.scheduled = 0;
   c.samples_this_step = false;
   c.rng_state ^= 0xD1B54A32D192ED03ull * static_cast<uint64_t>(c.id);
+  c.state_slot = -1;
+  if (stateful()) c.pages.clear();        // the state belongs to the parent: nothing of its progress can be shared
   for (int p : c.pages) if (p >= 0) pool_.retain(p);
-  if (s->status == SeqStatus::Swapped) {  // a swapped parent has no device pages to share
+  if (s->status == SeqStatus::Swapped || stateful()) {  // a swapped parent has no device pages to share
     c.pages.clear();
     c.trim_end = 0;
     c.num_computed = 0;
@@ -733,6 +805,12 @@ bool Core::swap_state(int64_t a, int64_t b) {
 bool Core::rewind(int64_t seq_id, int new_len) {
   Sequence* s = find(seq_id);
   if (!s || new_len < 1 || new_len > static_cast<int>(s->tokens.size())) return false;
+  if (stateful() && new_len < s->num_computed) {   // earlier states are gone: compute the kept tokens again
+    start_over(*s);
+    s->tokens.resize(new_len);
+    if (s->prompt_len > new_len) s->prompt_len = new_len;
+    return true;
+  }
   // keys released under the sliding window cannot come back into view
   if (s->trim_end > sink_pages_ && std::min(new_len, s->num_computed) - window_ < s->trim_end * kPageTokens) return false;
   s->tokens.resize(new_len);
@@ -749,7 +827,7 @@ bool Core::rewind(int64_t seq_id, int new_len) {
 
 bool Core::set_draft(int64_t seq_id, const int32_t* tokens, int k) {
   Sequence* s = find(seq_id);
-  if (!s || s->status == SeqStatus::Finished || k < 0) return false;
+  if (!s || s->status == SeqStatus::Finished || k < 0 || stateful()) return false;
   s->draft.assign(tokens, tokens + k);
   return true;
 }
@@ -858,7 +936,7 @@ extern "C" {
 
 void* ogb_core_create(int num_pages, int num_host_pages, int max_seqs, int max_tokens_per_step, int max_pages_per_seq,
                       int prefill_chunk, int token_multiple, int policy, int preempt_mode, int enable_prefix_cache,
-                      int eos_token, int max_draft_tokens) {
+                      int eos_token, int max_draft_tokens, int num_state_slots, int max_logit_rows) {
   CoreConfig c;
   c.num_pages = num_pages;
   c.num_host_pages = num_host_pages;
@@ -872,6 +950,8 @@ void* ogb_core_create(int num_pages, int num_host_pages, int max_seqs, int max_t
   c.enable_prefix_cache = enable_prefix_cache != 0;
   c.eos_token = eos_token;
   c.max_draft_tokens = max_draft_tokens;
+  c.num_state_slots = num_state_slots;
+  c.max_logit_rows = max_logit_rows;
   return new Core(c);
 }
 void ogb_core_destroy(void* h) { delete static_cast<Core*>(h); }
@@ -882,7 +962,8 @@ int ogb_core_layout(void* h, int32_t* out, int cap) {
   const int32_t v[] = {l.header, l.token_ids, l.positions, l.slots, l.seq_slot, l.ctx_len, l.cu_q, l.page_table,
                        l.tile_seq, l.tile_q0, l.logit_rows, l.temperature, l.top_k, l.top_p, l.min_p, l.uniform,
                        l.copy_src, l.copy_dst, l.swap_out_dev, l.swap_out_host, l.swap_in_dev, l.swap_in_host,
-                       l.total_words, l.max_tiles, l.max_swap, l.logit_seq, l.max_rows, l.move_runs, l.max_runs};
+                       l.total_words, l.max_tiles, l.max_swap, l.logit_seq, l.max_rows, l.move_runs, l.max_runs,
+                       l.state_slot};
   const int n = static_cast<int>(sizeof(v) / sizeof(v[0]));
   for (int i = 0; i < n && i < cap; ++i) out[i] = v[i];
   return n;
@@ -897,6 +978,10 @@ int64_t ogb_core_add_request(void* h, const int32_t* prompt, int n, int max_new_
   sp.min_p = min_p;
   sp.seed = seed;
   return static_cast<Core*>(h)->add_request(prompt, n, max_new_tokens, sp, priority, tenant, ignore_eos != 0, stop_ids, n_stop);
+}
+int64_t ogb_core_add_forced(void* h, const int32_t* tokens, int n) { return static_cast<Core*>(h)->add_forced(tokens, n); }
+int ogb_core_want_logits(void* h, int64_t id, const int32_t* positions, int n) {
+  return static_cast<Core*>(h)->want_logits(id, positions, n) ? 1 : 0;
 }
 int ogb_core_build_step(void* h, int32_t* plan) { return static_cast<Core*>(h)->build_step(plan); }
 int ogb_core_commit_step(void* h, const int32_t* sampled, int n, int64_t* ev_seq, int32_t* ev_token, int32_t* ev_finish,
@@ -944,6 +1029,7 @@ int64_t ogb_core_stat(void* h, int which) {
     case 9: return c->spec_accepted();
     case 10: return c->spec_steps();
     case 11: return c->num_pages();
+    case 12: return c->num_free_state_slots();
     default: return -1;
   }
 }

@@ -61,6 +61,9 @@ struct Sequence {
   bool samples_this_step = false;
   int num_draft = 0;                 // speculative tokens appended to `tokens` for the step being built
   std::vector<int32_t> draft;        // proposed continuation waiting to be verified
+  int state_slot = -1;               // slot of the recurrent-state buffers while running (models with per-sequence state)
+  bool forced = false;               // every token comes from the caller; the sequence never samples (see Core::add_forced)
+  std::vector<int32_t> wanted;       // forced sequences: positions whose logits rows the caller asked for, not yet computed
 };
 
 // Reference-counted device pages with a prefix cache over full pages.
@@ -109,6 +112,12 @@ struct CoreConfig {
   bool enable_prefix_cache = true;
   int eos_token = -1;
   int max_draft_tokens = 0;      // speculative decoding: draft tokens verified per sequence per step
+  // Models that carry recurrent state beside (or instead of) KV pages: number of state slots, 0 for none.  A running
+  // sequence owns one slot; its state starts over at position 0, so a slot needs no clearing when it is handed out again.
+  // State exists only at a sequence's last computed token.  Hence, with slots: no prefix cache, no drafts, preemption by
+  // recompute, and a fork or a rewind below the computed length starts the sequence over from its first token.
+  int num_state_slots = 0;
+  int max_logit_rows = 0;        // rows of logits per step (0: max_seqs * (1 + max_draft_tokens))
 };
 
 // Offsets (in int32 words) of the sections of a packed step plan.
@@ -122,6 +131,7 @@ struct PlanLayout {
   int logit_rows;                            // [max_seqs]
   int temperature, top_k, top_p, min_p, uniform;  // [max_rows] (floats stored by bit pattern)
   int logit_seq;                             // [max_rows] sequence id (low 31 bits) of every logit row
+  int state_slot;                            // [max_seqs] recurrent-state slot of every row's sequence (-1: none)
   int copy_src, copy_dst;                    // [max_seqs] CoW page copies to run before the step
   int swap_out_dev, swap_out_host, swap_in_dev, swap_in_host;  // [max_swap]
   int move_runs;                             // [2 * max_runs] (kind, count) pairs: the order in which the page moves above were
@@ -129,7 +139,7 @@ struct PlanLayout {
                                              // front to back, so running the runs in order reproduces the scheduler's sequence
   int total_words;
   int max_tiles, max_swap, max_runs;
-  int max_rows;                              // max_seqs * (1 + max_draft_tokens)
+  int max_rows;                              // max(max_logit_rows, max_seqs * (1 + max_draft_tokens))
 };
 
 enum PlanHeader : int {
@@ -151,6 +161,11 @@ class Core {
 
   int64_t add_request(const int32_t* prompt, int n, int max_new_tokens, const SamplingParams& sp, int priority, int tenant,
                       bool ignore_eos, const int32_t* stop_ids, int n_stop);
+  // A forced sequence runs exactly the tokens its caller brings (scoring, replaying): it computes what add_forced and
+  // append_tokens gave it, then waits for more, and it neither samples nor finishes by itself.  Logits rows are produced
+  // for the positions named with want_logits; release() ends it.
+  int64_t add_forced(const int32_t* tokens, int n);
+  bool want_logits(int64_t seq_id, const int32_t* positions, int n);
   bool cancel(int64_t seq_id);
   // Builds the next step into `plan` (layout().total_words int32 words).  Returns the number of tokens scheduled.
   int build_step(int32_t* plan);
@@ -208,7 +223,8 @@ class Core {
   int64_t prefix_hits() const { return pool_.hits(); }
   int64_t prefix_lookups() const { return pool_.lookups(); }
   int64_t num_preemptions() const { return preemptions_; }
-  bool has_work() const { return !waiting_.empty() || !running_.empty() || !swapped_.empty(); }
+  bool has_work() const;
+  int num_free_state_slots() const { return static_cast<int>(state_free_.size()); }
 
  private:
   Sequence* find(int64_t id);
@@ -221,12 +237,17 @@ class Core {
   bool preempt_one(Sequence* keep, std::vector<std::pair<int, int>>& swap_out);
   std::vector<int64_t> waiting_order();
   float next_uniform(Sequence& s);
+  bool stateful() const { return cfg_.num_state_slots > 0; }
+  bool acquire_state(Sequence& s);       // true when the model keeps no state or the sequence has a slot afterwards
+  void release_state(Sequence& s);
+  void start_over(Sequence& s);          // give back pages and slot: the sequence is computed again from its first token
   void finish(Sequence& s, FinishReason why);
 
   CoreConfig cfg_;
   PlanLayout layout_;
   BlockPool pool_;
   std::vector<int> host_free_;
+  std::vector<int> state_free_;
   std::unordered_map<int64_t, Sequence> seqs_;
   std::deque<int64_t> waiting_;
   std::vector<int64_t> running_;

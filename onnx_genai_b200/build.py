@@ -36,7 +36,12 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v",
 ]
 # --use_fast_math only affects intrinsics-free float math in glue kernels; numerically sensitive
-# paths call exp2f/__expf explicitly.
+# paths call exp2f/__expf explicitly.  Sources whose tanh, exp, divisions and roots belong to a model's 32-bit part are
+# compiled without it.
+PRECISE_SOURCES = {"hybrid.cu", "recurrent.cu", "latent_attention.cu"}
+# A library of its own for models that need only a few of the kernel sources: built when the full library is not there, so
+# that the first load compiles no more than the model uses (ops/_native.py ``prefer``).
+SUBSETS = {"hybrid": ("hybrid.cu", "recurrent.cu", "latent_attention.cu", "gemm_tcgen05.cu", "sampling.cu", "tp_comm.cu")}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-fopenmp", "-mavx2", "-mfma"]
 
 
@@ -78,12 +83,28 @@ def _stamp_ok(lib: Path, digest: str) -> bool:
     return lib.exists() and stamp.exists() and stamp.read_text().strip() == digest
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> Path:
-    srcs = cuda_sources()
+def cuda_flags(src: Path) -> list[str]:
+    return [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and src.name in PRECISE_SOURCES)]
+
+
+def _cuda_digest(srcs: list[Path]) -> str:
     hdrs = sorted((ROOT / "csrc" / "kernels").glob("*.h")) + sorted((ROOT / "csrc" / "kernels").glob("*.cuh"))
-    digest = _digest(srcs + hdrs, " ".join(NVCC_FLAGS))
-    if not force and _stamp_ok(CUDA_LIB, digest):
-        return CUDA_LIB
+    return _digest(srcs + hdrs, " ".join(NVCC_FLAGS) + " precise: " + " ".join(sorted(PRECISE_SOURCES)))
+
+
+def build_cuda(force: bool = False, verbose: bool = False, subset: str | None = None) -> Path:
+    """The kernel library.  ``subset``: a library of the named sources only (SUBSETS), unless the full one is up to date."""
+    srcs = cuda_sources()
+    lib = CUDA_LIB
+    digest = _cuda_digest(srcs)
+    if not force and _stamp_ok(lib, digest):
+        return lib
+    if subset is not None:
+        srcs = [s for s in srcs if s.name in SUBSETS[subset]]
+        lib = LIB_DIR / f"libogb_cuda_{subset}.so"
+        digest = _cuda_digest(srcs)
+        if not force and _stamp_ok(lib, digest):
+            return lib
     nvcc = _nvcc()
     LIB_DIR.mkdir(parents=True, exist_ok=True)
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
@@ -91,17 +112,17 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
 
     def one(src: Path) -> Path:
         obj = OBJ_DIR / (src.stem + ".o")
-        logs[src.name] = _run([nvcc, *NVCC_FLAGS, "-I", str(src.parent), "-c", str(src), "-o", str(obj)])
+        logs[src.name] = _run([nvcc, *cuda_flags(src), "-I", str(src.parent), "-c", str(src), "-o", str(obj)])
         return obj
 
     with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(one, srcs))
-    _run([nvcc, "-shared", "-o", str(CUDA_LIB), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a"])
+    _run([nvcc, "-shared", "-o", str(lib), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a"])
     (ROOT / "build" / "ptxas.log").write_text("\n".join(f"== {k}\n{v}" for k, v in sorted(logs.items())))
-    CUDA_LIB.with_suffix(".stamp").write_text(digest)
+    lib.with_suffix(".stamp").write_text(digest)
     if verbose:
-        print(f"built {CUDA_LIB}")
-    return CUDA_LIB
+        print(f"built {lib}")
+    return lib
 
 
 def cuda_include_dir() -> str:

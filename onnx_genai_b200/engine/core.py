@@ -27,7 +27,7 @@ HDR = dict(num_tokens=0, num_decode=1, num_prefill_seqs=2, num_tiles=3, num_logi
 _LAYOUT_FIELDS = ["header", "token_ids", "positions", "slots", "seq_slot", "ctx_len", "cu_q", "page_table", "tile_seq",
                   "tile_q0", "logit_rows", "temperature", "top_k", "top_p", "min_p", "uniform", "copy_src", "copy_dst",
                   "swap_out_dev", "swap_out_host", "swap_in_dev", "swap_in_host", "total_words", "max_tiles", "max_swap",
-                  "logit_seq", "max_rows", "move_runs", "max_runs"]
+                  "logit_seq", "max_rows", "move_runs", "max_runs", "state_slot"]
 
 
 def load_runtime():
@@ -45,7 +45,7 @@ def load_runtime():
     lib = ctypes.CDLL(str(path))
     P = c_void_p
     I32P = POINTER(c_int32)
-    lib.ogb_core_create.argtypes = [c_int] * 12
+    lib.ogb_core_create.argtypes = [c_int] * 14
     lib.ogb_core_create.restype = P
     lib.ogb_core_destroy.argtypes = [P]
     lib.ogb_core_layout.argtypes = [P, I32P, c_int]
@@ -53,6 +53,10 @@ def load_runtime():
     lib.ogb_core_add_request.argtypes = [P, I32P, c_int, c_int, c_float, c_int, c_float, c_float, c_uint64, c_int, c_int,
                                          c_int, I32P, c_int]
     lib.ogb_core_add_request.restype = c_int64
+    lib.ogb_core_add_forced.argtypes = [P, I32P, c_int]
+    lib.ogb_core_add_forced.restype = c_int64
+    lib.ogb_core_want_logits.argtypes = [P, c_int64, I32P, c_int]
+    lib.ogb_core_want_logits.restype = c_int
     lib.ogb_core_build_step.argtypes = [P, c_void_p]
     lib.ogb_core_build_step.restype = c_int
     lib.ogb_core_commit_step.argtypes = [P, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int]
@@ -111,6 +115,8 @@ class CoreConfig:
     enable_prefix_cache: bool = True
     eos_token: int = -1
     max_draft_tokens: int = 0
+    num_state_slots: int = 0       # > 0: the model keeps recurrent state; one slot per running sequence
+    max_logit_rows: int = 0        # 0: max_seqs * (1 + max_draft_tokens)
 
 
 class Layout:
@@ -128,7 +134,7 @@ class Core:
         self.h = self.lib.ogb_core_create(cfg.num_pages, cfg.num_host_pages, cfg.max_seqs, cfg.max_tokens_per_step,
                                           cfg.max_pages_per_seq, cfg.prefill_chunk, cfg.token_multiple,
                                           POLICIES[cfg.policy], PREEMPT[cfg.preempt], int(cfg.enable_prefix_cache),
-                                          cfg.eos_token, cfg.max_draft_tokens)
+                                          cfg.eos_token, cfg.max_draft_tokens, cfg.num_state_slots, cfg.max_logit_rows)
         buf = (c_int32 * 32)()
         n = self.lib.ogb_core_layout(self.h, buf, 32)
         self.layout = Layout(list(buf)[:n])
@@ -158,6 +164,20 @@ class Core:
             raise ValueError(f"prompt of {len(arr)} tokens does not fit max_pages_per_seq={self.cfg.max_pages_per_seq} "
                              f"({self.cfg.max_pages_per_seq * 16} tokens); raise it or shorten the prompt")
         return int(sid)
+
+    def add_forced(self, tokens) -> int:
+        """A sequence whose every token comes from the caller: it runs what it was given (more follows through
+        :meth:`append_tokens`), samples nothing and lives until :meth:`release`."""
+        arr = np.ascontiguousarray(tokens, dtype=np.int32)
+        sid = int(self.lib.ogb_core_add_forced(self.h, arr.ctypes.data_as(POINTER(c_int32)), len(arr)))
+        if sid < 0:
+            raise ValueError(f"a forced sequence needs 1 .. {self.cfg.max_pages_per_seq * 16 - 1} tokens to start with, got {len(arr)}")
+        return sid
+
+    def want_logits(self, sid, positions) -> bool:
+        """Ask for the logits rows of positions of a forced sequence that the coming steps will compute."""
+        arr = np.ascontiguousarray(positions, dtype=np.int32)
+        return bool(self.lib.ogb_core_want_logits(self.h, sid, arr.ctypes.data_as(POINTER(c_int32)), len(arr)))
 
     def build_step(self, plan_ptr: int) -> int:
         return self.lib.ogb_core_build_step(self.h, plan_ptr)
@@ -266,3 +286,4 @@ class Core:
     spec_accepted = property(lambda self: self._stat(9))
     spec_steps = property(lambda self: self._stat(10))
     num_pages = property(lambda self: self._stat(11))
+    num_free_state_slots = property(lambda self: self._stat(12))

@@ -18,6 +18,8 @@ same request stream, so no per-step control message crosses ranks.
 """
 from __future__ import annotations
 
+import dataclasses
+import math
 import time
 from dataclasses import dataclass, field
 
@@ -26,7 +28,9 @@ import torch
 
 from .. import ops
 from ..models.config import DecoderConfig
-from ..models.decoder import DecoderModel, DecoderWeights, KVCache, StepInputs, random_weights
+from ..models.decoder import DecoderWeights, KVCache, StepInputs
+from ..models.registry import family_of
+from ..models.state import StateCache
 from ..parallel.sharding import shard_heads
 from ..utils.trace import TRACER
 from .core import HDR, Core, CoreConfig
@@ -34,7 +38,7 @@ from .core import HDR, Core, CoreConfig
 
 @dataclass
 class EngineConfig:
-    model: DecoderConfig
+    model: DecoderConfig               # or another family's configuration (models/registry.py)
     num_pages: int = 0                 # 0: size from free device memory
     host_allocator_plugin: str = ""    # shared library implementing the memory plugin ABI: the host swap space comes from it
     kv_max_pages: int = 0              # > num_pages (CUDA, TP=1): reserve address space for this many pages, back num_pages now
@@ -51,6 +55,8 @@ class EngineConfig:
     enable_prefix_cache: bool = True
     release_window_pages: bool = True  # sliding-window models: give back the KV pages no later query can see (sinks are kept)
     kv_dtype: str = "bf16"
+    compute_dtype: str = "bf16"        # "f32": weights, activations and pages in true 32-bit (families that have it)
+    max_logit_rows: int = 0            # logits rows a step may produce (0: one per sequence and draft)
     decode_splits: int = 0             # 0: pick from batch shape
     sync_sampled_tokens: bool = True   # TP: broadcast rank 0's tokens so replicas cannot diverge
     max_draft_tokens: int = 0          # speculative decoding: drafts verified per sequence per step
@@ -80,6 +86,7 @@ class StepOutput:
     num_tokens: int = 0
     num_decode: int = 0
     num_prefill_tokens: int = 0
+    forced_logits: dict = field(default_factory=dict)   # forced sequences: seq_id -> [(position, logits row)] as asked for
 
 
 class LLMEngine:
@@ -95,15 +102,29 @@ class LLMEngine:
             raise ValueError("pipeline parallelism needs tp = 1, a communicator, and no weight paging")
         m = cfg.model
         is_cuda = self.device.type == "cuda"
+        fam = family_of(m)
+        if cfg.compute_dtype not in ("bf16", "f32") or (is_cuda and cfg.compute_dtype not in fam.compute_dtypes):
+            raise ValueError(f"compute_dtype {cfg.compute_dtype!r} is not available for {m.name} on this device; it has {', '.join(fam.compute_dtypes)}")
+        if cfg.compute_dtype == "f32":
+            cfg = self.cfg = dataclasses.replace(cfg, kv_dtype="f32")
+        if m.has_state:
+            # state exists at a sequence's last computed token only: nothing can attach to a prefix, be rolled back after a
+            # rejected draft, or leave for host memory page by page
+            for bad, what in ((cfg.max_draft_tokens > 0, "speculative decoding"), (cfg.num_host_pages > 0, "KV swap space (use preempt='recompute')"),
+                              (cfg.kv_dtype not in ("bf16", "f32"), f"kv_dtype {cfg.kv_dtype!r}"), (tp > 1 or self.pp > 1, "more than one GPU"),
+                              (cfg.weight_offload_layers > 0, "weight offload")):
+                if bad:
+                    raise ValueError(f"{m.name} keeps recurrent state per sequence: {what} is not available")
+            cfg = self.cfg = dataclasses.replace(cfg, enable_prefix_cache=False, preempt="recompute")
         shard_rank = 0 if self.pp > 1 else rank       # a pipeline stage holds whole layers: nothing is sharded within one
         if weights is None:
-            dtype = torch.bfloat16 if is_cuda else torch.float32
-            weights = random_weights(m, self.device, tp, shard_rank, seed=cfg.seed, dtype=dtype)
+            dtype = torch.bfloat16 if is_cuda and cfg.compute_dtype == "bf16" else torch.float32
+            weights = fam.random_weights(m, self.device, tp, shard_rank, cfg.seed, dtype)
         self.weights = weights
         max_pages_per_seq = (cfg.max_seq_len + ops.PAGE - 1) // ops.PAGE
         hs = shard_heads(m.num_heads, m.num_kv_heads, tp, shard_rank)
-        max_rows = cfg.max_seqs * (1 + max(0, cfg.max_draft_tokens))
-        self.model = DecoderModel(m, weights, self.device, cfg.max_tokens_per_step, max_rows, tp, shard_rank, comm)
+        max_rows = max(cfg.max_logit_rows, cfg.max_seqs * (1 + max(0, cfg.max_draft_tokens)))
+        self.model = fam.model(m, weights, self.device, cfg.max_tokens_per_step, max_rows, tp, shard_rank, comm)
         own_layers = None
         if self.pp > 1:
             from ..parallel.pipeline import plan_stages
@@ -130,8 +151,9 @@ class LLMEngine:
         self.memory.lease("activations", tier, act_bytes, "step buffers")
         num_pages = cfg.num_pages
         if num_pages <= 0:
-            kv_bytes = 1 if cfg.kv_dtype in ("fp8", "int8", "fp8_e5m2") else 2
-            page_bytes = m.num_layers * len(hs.kv_heads) * 2 * ops.PAGE * m.head_dim * kv_bytes
+            kv_bytes = {"fp8": 1, "int8": 1, "fp8_e5m2": 1, "f32": 4}.get(cfg.kv_dtype, 2)
+            shapes = [m.kv_page_shape(li, len(hs.kv_heads)) for li in range(m.num_layers)]
+            page_bytes = max(1, sum(math.prod(sh) * kv_bytes for sh in shapes if sh is not None))
             if is_cuda:
                 free, total = torch.cuda.mem_get_info(self.device)
                 budget = int(free - (1.0 - cfg.gpu_memory_utilization) * total)
@@ -154,13 +176,19 @@ class LLMEngine:
         self.kv = KVCache(m, self.num_pages, self.device, len(hs.kv_heads), cfg.kv_dtype, max_pages=kv_max, layers=own_layers,
                           allocator=self.allocator)
         self.kv_lease = self.memory.lease("kv", tier, self.kv.mapped_bytes(), f"pages of 16 tokens, {cfg.kv_dtype}")
+        self.state = None
+        if m.has_state:
+            self.state = StateCache(m, cfg.max_seqs, self.device)
+            self.model.bind_state(self.state)
+            self.memory.lease("kv", tier, self.state.nbytes(), f"recurrent state of {cfg.max_seqs} sequences")
         self.kv_grows, self.kv_grow_error = 0, None
         self.core = Core(CoreConfig(num_pages=self.num_pages, num_host_pages=cfg.num_host_pages, max_seqs=cfg.max_seqs,
                                     max_tokens_per_step=cfg.max_tokens_per_step, max_pages_per_seq=max_pages_per_seq,
                                     prefill_chunk=cfg.prefill_chunk, token_multiple=cfg.token_multiple,
                                     policy=cfg.policy, preempt=cfg.preempt,
                                     enable_prefix_cache=cfg.enable_prefix_cache, eos_token=m.eos_token,
-                                    max_draft_tokens=cfg.max_draft_tokens))
+                                    max_draft_tokens=cfg.max_draft_tokens, num_state_slots=cfg.max_seqs if m.has_state else 0,
+                                    max_logit_rows=cfg.max_logit_rows))
         if m.sliding_window > 0 and cfg.release_window_pages:
             self.core.set_window(m.sliding_window, m.attention_sinks)
         L = self.core.layout
@@ -219,7 +247,7 @@ class LLMEngine:
             slots=p[L.slots:L.slots + T], ctx_len=p[L.ctx_len:L.ctx_len + S],
             page_table=p[L.page_table:L.page_table + S * MP].view(S, MP), cu_q=p[L.cu_q:L.cu_q + S + 1],
             tile_seq=p[L.tile_seq:L.tile_seq + L.max_tiles], tile_q0=p[L.tile_q0:L.tile_q0 + L.max_tiles],
-            logit_rows=p[L.logit_rows:L.logit_rows + max_rows])
+            logit_rows=p[L.logit_rows:L.logit_rows + max_rows], state_slot=p[L.state_slot:L.state_slot + S])
         f32 = lambda off: p[off:off + max_rows].view(torch.float32)
         self.temperature, self.top_p, self.min_p, self.uniform = (f32(L.temperature), f32(L.top_p), f32(L.min_p),
                                                                   f32(L.uniform))
@@ -233,6 +261,7 @@ class LLMEngine:
             slots = sum(s.numel() for s in self.model.weight_slots)
             self.weights_lease.resize(max(0, self.weights_lease.nbytes - self.model.paged_weight_bytes + slots))   # two slots stay on the device
         self.host_samplers: dict = {}     # seq id -> fn(logits_row fp32 numpy, uniform) -> token id
+        self.forced: set = set()          # sequences whose tokens come from the caller (open_forced)
         self.proposers: dict = {}         # seq id -> SpeculativeProposer
         self.stats: dict[int, RequestStats] = {}
         self.steps = 0
@@ -256,6 +285,48 @@ class LLMEngine:
                                     ignore_eos, stop_ids)
         self.stats[sid] = RequestStats(arrival=time.perf_counter(), prompt_tokens=len(prompt_ids))
         return sid
+
+    # ---- forced sequences: the caller brings every token and asks for logits ----------------------
+    def _want(self, sid: int, start: int, want) -> None:
+        if len(want) and not self.core.want_logits(sid, [start + int(k) for k in want]):
+            raise ValueError(f"logits asked for outside the tokens just given to sequence {sid}")
+
+    def open_forced(self, tokens, want=()) -> int:
+        """A sequence that runs exactly the tokens it is given, batched with everything else by the scheduler, and samples
+        nothing.  ``want``: places among ``tokens`` whose logits rows the step that computes them returns
+        (``StepOutput.forced_logits``).  It holds its pages and state until :meth:`close_forced`."""
+        sid = self.core.add_forced(tokens)
+        self.forced.add(sid)
+        self._want(sid, 0, want)
+        return sid
+
+    def extend_forced(self, sid: int, tokens, want=()) -> None:
+        """More tokens for a forced sequence; ``want`` counts within them."""
+        start = self.core.seq_len(sid)
+        if sid not in self.forced or not self.core.append_tokens(sid, tokens):
+            raise ValueError(f"sequence {sid} is not an open forced sequence, or {len(tokens)} more tokens exceed max_seq_len")
+        self._want(sid, start, want)
+
+    def close_forced(self, sid: int) -> None:
+        self.forced.discard(sid)
+        self.core.release(sid)
+
+    def forced_pending(self, sid: int) -> int:
+        """Tokens of a forced sequence that no step has computed yet."""
+        return self.core.seq_len(sid) - self.core.seq_computed(sid)
+
+    def _collect_forced(self, out: "StepOutput", logits, r: int) -> int:
+        """Copies the rows of forced sequences out of the step's logits; returns how many of the r rows they were."""
+        L, pn = self.L, self.plan_np
+        seqs = pn[L.logit_seq:L.logit_seq + r]
+        by_key = {sid & 0x7FFFFFFF: sid for sid in self.forced}
+        rows = [i for i in range(r) if int(seqs[i]) in by_key]
+        if rows:
+            block = logits[rows].float()
+            for j, i in enumerate(rows):
+                pos = int(pn[L.positions + int(pn[L.logit_rows + i])])
+                out.forced_logits.setdefault(by_key[int(seqs[i])], []).append((pos, block[j]))
+        return len(rows)
 
     @property
     def has_work(self) -> bool:
@@ -370,6 +441,8 @@ class LLMEngine:
             return self.cfg.decode_splits
         ctas = nd * self.model.hkv
         target = 2 * (ops.num_sms() if self.device.type == "cuda" else 148)
+        if getattr(self.model, "split_by_window", False) and self.cfg.model.sliding_window > 0:
+            max_ctx = min(max_ctx, self.cfg.model.sliding_window)
         if ctas >= target or max_ctx < 256:
             return 1
         s = 1
@@ -404,6 +477,7 @@ class LLMEngine:
             pn[L.positions + r:L.positions + bucket] = 0
             pn[L.slots + r:L.slots + bucket] = -1
             pn[L.ctx_len + r:L.ctx_len + bucket] = 0
+            pn[L.state_slot + r:L.state_slot + bucket] = -1
             pn[L.logit_rows + r:L.logit_rows + bucket] = np.arange(r, bucket, dtype=np.int32)
             pn[L.temperature + r:L.temperature + bucket] = 0          # 0.0f: padded rows take the argmax path
             self.plan_dev.copy_(self.plan_host[: self.dev_words], non_blocking=True)
@@ -548,7 +622,7 @@ class LLMEngine:
         ids (4 bytes per row) replaces the broadcast that kept replicas in step.  Steps whose logits are needed on
         the host (custom samplers, log-probabilities, embeddings, speculative verification) keep all rows."""
         return (self.tp > 1 and self.cfg.shard_sampling and r >= self.tp
-                and not self.host_samplers and not self.hidden_taps and self.cfg.max_draft_tokens == 0)
+                and not self.host_samplers and not self.hidden_taps and not self.forced and self.cfg.max_draft_tokens == 0)
 
     def forward_and_sample_sharded(self, si, r: int, greedy: bool) -> None:
         """Run the step with this rank's share of the sampling rows; leaves all r token ids in sampled_dev[:r]."""
@@ -668,7 +742,10 @@ class LLMEngine:
             logits = None
         else:
             logits = self.model.forward(si, self.kv)
-        if r > 0:
+        sampling = r
+        if self.forced and r > 0:
+            sampling = r - self._collect_forced(out, logits, r)
+        if sampling > 0:
             temps = self.plan_np[self.L.temperature:self.L.temperature + r].view(np.float32)
             if graphed:
                 self._finish_device_step(r)

@@ -59,6 +59,12 @@ class DecoderConfig:
     def kv_size(self) -> int:
         return self.num_kv_heads * self.head_dim
 
+    has_state = False              # no per-sequence state beside the KV pages
+
+    def kv_page_shape(self, layer: int, kv_heads: int):
+        """Shape of one KV page of a layer ([kv heads, K | V, tokens, head dimension])."""
+        return (kv_heads, 2, 16, self.head_dim)
+
     def replace(self, **kw) -> "DecoderConfig":
         return dataclasses.replace(self, **kw)
 

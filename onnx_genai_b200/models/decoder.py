@@ -153,6 +153,7 @@ class StepInputs:
     tile_q0: torch.Tensor
     logit_rows: torch.Tensor       # [R]
     max_ctx: int = 0
+    state_slot: torch.Tensor | None = None     # [S] slot of every entry's recurrent state (models that keep some)
     # Speculative verification over long contexts: when every "prefill" sequence of the step is just a handful
     # of draft rows, the engine describes those rows as decode rows (one page-table row and context length per
     # query row) so attention runs on the split-KV decode kernel instead of walking the whole context in one CTA.
@@ -163,7 +164,8 @@ class StepInputs:
 
 
 class KVCache:
-    """Per-layer paged pools [pages, kv_heads_local, 2, 16, head_dim] (bf16, or e4m3 + scales).
+    """Per-layer paged pools [pages, *page shape] -- [pages, kv_heads_local, 2, 16, head_dim] for K/V (bf16, or e4m3 + scales);
+    ``cfg.kv_page_shape(layer, kv_heads)`` gives a layer's page, None for a layer that caches nothing of its own.
 
     With ``max_pages`` > ``num_pages`` on a CUDA device each pool (and scale table) is a view over a reserved address
     range of ``max_pages`` pages of which only the first ``num_pages`` are backed; :meth:`grow` backs more in place, so
@@ -175,14 +177,16 @@ class KVCache:
         """``layers``: the layer indices this process runs (a pipeline stage); the others get no pool.  ``allocator``: an
         engine allocator (engine/allocator.py) the fixed-size pools come from; torch's allocator when absent."""
         hkv = kv_heads_local or cfg.num_kv_heads
-        own = set(range(cfg.num_layers)) if layers is None else set(layers)
+        own = {li for li in (range(cfg.num_layers) if layers is None else layers) if cfg.kv_page_shape(li, hkv) is not None}
+        shape = {li: tuple(cfg.kv_page_shape(li, hkv)) for li in own}
         self.own_layers = sorted(own)
         self.num_pages = num_pages
         self.dtype = dtype
-        if dtype not in ("bf16", "fp8", "int8", "fp8_e5m2"):
-            raise ValueError(f"kv dtype {dtype!r} is not supported; use bf16, fp8 (e4m3 pages), fp8_e5m2 or int8")
+        if dtype not in ("bf16", "fp8", "int8", "fp8_e5m2", "f32"):
+            raise ValueError(f"kv dtype {dtype!r} is not supported; use bf16, fp8 (e4m3 pages), fp8_e5m2 or int8 (f32: the 32-bit engine)")
         # one-byte pools say their format by dtype
-        tdtype = {"bf16": torch.bfloat16, "fp8": torch.uint8, "int8": torch.int8, "fp8_e5m2": torch.float8_e5m2}[dtype]
+        tdtype = {"bf16": torch.bfloat16, "fp8": torch.uint8, "int8": torch.int8, "fp8_e5m2": torch.float8_e5m2,
+                  "f32": torch.float32}[dtype]
         if torch.device(device).type == "cpu" and dtype == "bf16":
             tdtype = torch.float32
         quant = dtype in ("fp8", "int8", "fp8_e5m2")
@@ -192,19 +196,24 @@ class KVCache:
             from ..utils.vmm import GrowableBuffer
 
             dev = torch.device(device).index or 0
-            self.page_nbytes = hkv * 2 * ops.PAGE * cfg.head_dim * torch.empty(0, dtype=tdtype).element_size()
             self.scale_nbytes = hkv * 2 * 4
-            self.buffers, self.scale_buffers, self.pools, self.scales = [], [], [], [] if quant else None
-            for _ in range(cfg.num_layers):
-                buf = GrowableBuffer(self.max_pages * self.page_nbytes, dev, num_pages * self.page_nbytes)
+            self.layer_page_nbytes, self.buffers, self.scale_buffers, self.pools, self.scales = [], [], [], [], [] if quant else None
+            for li in range(cfg.num_layers):
+                if li not in own:
+                    self.pools.append(None)
+                    continue
+                nbytes = math.prod(shape[li]) * torch.empty(0, dtype=tdtype).element_size()
+                buf = GrowableBuffer(self.max_pages * nbytes, dev, num_pages * nbytes)
+                self.layer_page_nbytes.append(nbytes)
                 self.buffers.append(buf)
                 buf.view(torch.uint8).zero_()
-                self.pools.append(buf.span(tdtype, (self.max_pages, hkv, 2, ops.PAGE, cfg.head_dim)))
+                self.pools.append(buf.span(tdtype, (self.max_pages, *shape[li])))
                 if quant:
                     sb = GrowableBuffer(self.max_pages * self.scale_nbytes, dev, num_pages * self.scale_nbytes)
                     self.scale_buffers.append(sb)
                     sb.view(torch.uint8).zero_()
                     self.scales.append(sb.span(torch.float32, (self.max_pages, hkv, 2)))
+            self.page_nbytes = max(self.layer_page_nbytes, default=0)
             self._mark_backed()
             return
         self.max_pages = num_pages
@@ -212,7 +221,7 @@ class KVCache:
             make = lambda shape, dt, tag: allocator.tensor(shape, dt, "kv", tag)
         else:
             make = lambda shape, dt, tag: torch.zeros(*shape, dtype=dt, device=device)
-        self.pools = [make((num_pages, hkv, 2, ops.PAGE, cfg.head_dim), tdtype, f"pages of layer {li}") if li in own else None
+        self.pools = [make((num_pages, *shape[li]), tdtype, f"pages of layer {li}") if li in own else None
                       for li in range(cfg.num_layers)]
         self.scales = None
         if quant:
@@ -221,7 +230,7 @@ class KVCache:
 
     def _mark_backed(self) -> None:
         """Record the mapped page count on every pool tensor: kernels bound page ids by it (ops.backed_pages)."""
-        for t in self.pools:
+        for t in self.own_pools:
             t.backed_pages = self.num_pages
 
     @property
@@ -237,9 +246,9 @@ class KVCache:
         new_pages = min(int(new_pages), self.max_pages)
         if new_pages <= self.num_pages:
             return self.num_pages
-        for buf in self.buffers:
+        for buf, nbytes in zip(self.buffers, self.layer_page_nbytes):
             old = buf.mapped
-            buf.grow(new_pages * self.page_nbytes)
+            buf.grow(new_pages * nbytes)
             if buf.mapped > old:     # scale tables rely on zero meaning "page not started"; pools are zeroed for tidiness
                 buf.view(torch.uint8, (buf.mapped - old,), old).zero_()
         for sb in self.scale_buffers:
@@ -271,8 +280,7 @@ class KVCache:
         return sum(b.mapped for b in self.buffers) + sum(b.mapped for b in self.scale_buffers)
 
     def page_bytes(self) -> int:
-        p = self.own_pools[0]
-        return p.stride(0) * p.element_size() * len(self.own_layers)
+        return sum(p.stride(0) * p.element_size() for p in self.own_pools)
 
 
 class DecoderModel:

@@ -438,8 +438,9 @@ def argmax(logits, out=None):
     rows, vocab = logits.shape
     if out is None:
         out = torch.empty(rows, dtype=torch.int32, device=logits.device)
-    rc = _native.load().ogb_argmax_bf16(logits.data_ptr(), out.data_ptr(), rows, vocab, logits.stride(0), _stream())
-    _native.check(rc, "ogb_argmax_bf16")
+    fn = _native.load().ogb_argmax_f32 if logits.dtype == torch.float32 else _native.load().ogb_argmax_bf16
+    rc = fn(logits.data_ptr(), out.data_ptr(), rows, vocab, logits.stride(0), _stream())
+    _native.check(rc, "ogb_argmax")
     launch_counts["argmax"] += 1
     return out
 
@@ -456,10 +457,10 @@ def sample(logits, temperature, top_k, top_p, min_p, uniform, work=None, out=Non
         work = torch.empty(rows * vocab, dtype=torch.int32, device=logits.device)
     if out is None:
         out = torch.empty(rows, dtype=torch.int32, device=logits.device)
-    rc = _native.load().ogb_sample_bf16(logits.data_ptr(), out.data_ptr(), temperature.data_ptr(), top_k.data_ptr(),
-                                        top_p.data_ptr(), min_p.data_ptr(), uniform.data_ptr(), work.data_ptr(), rows,
-                                        vocab, logits.stride(0), _stream())
-    _native.check(rc, "ogb_sample_bf16")
+    fn = _native.load().ogb_sample_f32 if logits.dtype == torch.float32 else _native.load().ogb_sample_bf16
+    rc = fn(logits.data_ptr(), out.data_ptr(), temperature.data_ptr(), top_k.data_ptr(), top_p.data_ptr(), min_p.data_ptr(),
+            uniform.data_ptr(), work.data_ptr(), rows, vocab, logits.stride(0), _stream())
+    _native.check(rc, "ogb_sample")
     launch_counts["sample"] += 1
     return out
 

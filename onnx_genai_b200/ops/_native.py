@@ -40,6 +40,11 @@ _SIGNATURES = {
     "ogb_rope_kv_append_q8": ([P, P, P, P, P, P, I, I, I, I, I, I, I, I, L, I, P, P], I),
     "ogb_paged_decode_q8": ([P, P, P, P, I, P, P, I, I, L, I, I, I, I, I, F, I, P, P, I, I, P, P], I),
     "ogb_paged_prefill_q8": ([P, P, P, P, I, P, P, P, P, P, I, I, I, L, I, I, I, I, I, F, I, I, P, P], I),
+    "ogb_gemm_bf16_gated": ([P, P, P, I, I, I, I, I, I, I, I, P, P], I),
+    "ogb_gemm_bf16_batched": ([P, P, P, I, I, I, I, I, I, I, I, I, P, P], I),
+    "ogb_gemm_f32": ([P, P, P, I, I, I, I, I, I, I, I, I, P], I),
+    "ogb_argmax_f32": ([P, P, I, I, I, P], I),
+    "ogb_sample_f32": ([P, P, P, P, P, P, P, P, I, I, I, P], I),
     "ogb_argmax_bf16": ([P, P, I, I, I, P], I),
     "ogb_sample_bf16": ([P, P, P, P, P, P, P, P, I, I, I, P], I),
     "ogb_spec_verify_greedy": ([P, P, P, P, I, I, I, I, P], I),
@@ -54,6 +59,16 @@ def lib_path() -> Path:
     return Path(__file__).resolve().parent.parent / "_lib" / "libogb_cuda.so"
 
 
+_SUBSET: str | None = None
+
+
+def prefer(subset: str) -> None:
+    """Name the kernel subset a model needs: if the library has to be compiled, only that subset is (build.SUBSETS)."""
+    global _SUBSET
+    if _LIB is None:
+        _SUBSET = subset
+
+
 def load() -> ctypes.CDLL:
     """Load (building first when the sources are newer and nvcc exists) the CUDA kernel library."""
     global _LIB
@@ -66,7 +81,7 @@ def load() -> ctypes.CDLL:
         try:
             from .. import build as _build
 
-            path = _build.build_cuda()
+            path = _build.build_cuda(subset=_SUBSET)
         except Exception as exc:  # nvcc missing on the run machine: fall back to the shipped .so
             if not path.exists():
                 raise RuntimeError(

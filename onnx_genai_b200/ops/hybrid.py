@@ -1,0 +1,224 @@
+"""Ops of models that choose a mixer per layer (csrc/kernels/hybrid.cu, recurrent.cu, latent_attention.cu): hyper-connected
+residual streams with a Dynamic-Tanh norm and token shift, HGRN2 recurrence over per-sequence state, attention over paged
+latents, batched per-head products, and the fp32 matrix product of the 32-bit engine.
+
+CUDA tensors run the kernels; CPU tensors run the statements in :mod:`onnx_genai_b200.ops.reference`, as the other ops do.
+``si`` is the step's :class:`~onnx_genai_b200.models.decoder.StepInputs`.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from . import _native, _ptr, _stream, _timed, backed_pages, launch_counts, reference, status_word
+from . import PAGE, gemm
+
+P, I, F, L = _native.P, _native.I, _native.F, _native.L
+_native.register("ogb_hyper_step", [P] * 13 + [I] * 6 + [P] * 5 + [I] * 4 + [P, P])
+_native.register("ogb_embed_streams", [P, P, P, I, I, I, I, I, P, P])
+_native.register("ogb_latent_append", [P, I, P, F, P, P, I, I, I, L, I, P, P])
+_native.register("ogb_latent_attention", [P] * 8 + [I] * 7 + [L, I, F, I, P, P, I, P, P])
+_native.register("ogb_hgrn2_state_rows", [I])
+_native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 3 + [P, P])
+_native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, I, P])
+_native.register("ogb_act_mul_packed", [P, P, I, I, I, I, I, P])
+
+ACTS = {"silu": 0, "gelu_tanh": 1}
+_ELEM = {torch.float32: 0, torch.bfloat16: 1}
+
+
+@dataclass
+class DynamicTanh:
+    """tanh(alpha x) w + b, all fp32 (alpha is a one-element tensor)."""
+    alpha: torch.Tensor
+    w: torch.Tensor
+    b: torch.Tensor
+
+
+@dataclass
+class HyperConnection:
+    """Weights of one sublayer over S residual streams, fp32: reads sum_s read[s] x_s, writes
+    x_t <- sum_s mix[s, t] x_s + write[t] y."""
+    read: torch.Tensor
+    write: torch.Tensor
+    mix: torch.Tensor
+
+
+def state_rows(dim: int) -> int:
+    """Row width at which the recurrence keeps a state of ``dim`` key channels."""
+    for n in (64, 128, 256):
+        if dim <= n:
+            return n
+    raise ValueError(f"recurrent key width {dim} is not supported (at most 256)")
+
+
+@_timed("linear")
+def linear(a, w, out, f32_out=False):
+    """out = a @ w^T: bf16 on the tensor cores (fp32 results with ``f32_out``), fp32 operands in true fp32."""
+    if not a.is_cuda:
+        out.copy_(reference.gemm(a, w, out_dtype=out.dtype))
+        return out
+    if a.dtype == torch.bfloat16:
+        return gemm(a, w, out=out, out_f32=f32_out)
+    return linear_batched(a, w, out, 1, 0, 0)
+
+
+@_timed("linear_batched")
+def linear_batched(a, w, out, batch, a_step, c_step):
+    """out[:, z*c_step : +N] = a[:, z*a_step : +K] @ w[z*N : +N]^T for every z < batch; w is [batch * N, K]."""
+    m, k = a.shape[0], w.shape[1]
+    n = w.shape[0] // batch
+    if not a.is_cuda:
+        for z in range(batch):
+            out[:, z * c_step:z * c_step + n] = reference.gemm(a[:, z * a_step:z * a_step + k], w[z * n:(z + 1) * n], out_dtype=out.dtype)
+        return out
+    lib = _native.load()
+    if a.dtype == torch.bfloat16:
+        rc = lib.ogb_gemm_bf16_batched(a.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, a.stride(0), w.stride(0), out.stride(0), batch,
+                                       a_step, c_step, status_word().data_ptr(), _stream())
+        _native.check(rc, "ogb_gemm_bf16_batched")
+        launch_counts["gemm_bf16_tcgen05"] += 1
+    else:
+        rc = lib.ogb_gemm_f32(a.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, a.stride(0), w.stride(0), out.stride(0), batch, a_step,
+                              c_step, _stream())
+        _native.check(rc, "ogb_gemm_f32")
+        launch_counts["gemm_f32"] += 1
+    return out
+
+
+@_timed("gated_linear")
+def gated_linear(a, w_packed, half, act, out, scratch=None):
+    """out = act(a @ gate^T) * (a @ up^T) over a weight packed by ``ops.pack_gate_up``; bf16 in one product with the gate in its
+    epilogue, fp32 through ``scratch`` [rows, 2 * inter]."""
+    if not a.is_cuda:
+        out.copy_(reference.act_mul_packed(reference.gemm(a, w_packed, out_dtype=torch.float32), half, act, out.dtype))
+        return out
+    m, n = a.shape[0], w_packed.shape[0]
+    if a.dtype == torch.bfloat16:
+        rc = _native.load().ogb_gemm_bf16_gated(a.data_ptr(), w_packed.data_ptr(), out.data_ptr(), m, n, a.shape[1], a.stride(0),
+                                                w_packed.stride(0), out.stride(0), ACTS[act], 2 * half, status_word().data_ptr(), _stream())
+        _native.check(rc, "ogb_gemm_bf16_gated")
+        launch_counts["gemm_bf16_tcgen05"] += 1
+        return out
+    gu = scratch[:m, :n]
+    assert gu.is_contiguous() and out.is_contiguous()
+    linear(a, w_packed, gu)
+    rc = _native.load().ogb_act_mul_packed(gu.data_ptr(), out.data_ptr(), m, n // 2, half, ACTS[act], _ELEM[a.dtype], _stream())
+    _native.check(rc, "ogb_act_mul_packed")
+    launch_counts["act_mul_packed"] += 1
+    return out
+
+
+@_timed("embed_streams")
+def embed_streams(ids, table, x):
+    """Every stream of row t of x [T, S, W] (fp32) becomes the embedding of ids[t]."""
+    t, s, w = x.shape
+    if not x.is_cuda:
+        x.copy_(table[ids[:t].long()].float()[:, None, :].expand(-1, s, -1))
+        return x
+    rc = _native.load().ogb_embed_streams(ids.data_ptr(), table.data_ptr(), x.data_ptr(), t, s, w, table.shape[0], _ELEM[table.dtype],
+                                          status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_embed_streams")
+    launch_counts["embed_streams"] += 1
+    return x
+
+
+@_timed("hyper_step")
+def hyper_step(x_in, x_out, y, written: HyperConnection | None, read, norm: DynamicTanh | None, h, si, shift=None, prev=None, gather=None):
+    """Fold the last sublayer's output ``y`` into the streams (weights ``written``; x_in -> x_out), read the next sublayer's
+    input (weights ``read``, None: the sum), norm it and shift it by a token where ``shift`` is given (state ``prev`` [slots, W]).
+    ``gather``: h gets the rows it names only, and nothing is written back."""
+    rows = h.shape[0] if h is not None else x_in.shape[0]
+    if not x_in.is_cuda:
+        src = x_in if gather is None else x_in[gather.long()]
+        ys = y if (y is None or gather is None) else y[gather.long()]
+        x, u = reference.hyper_step(src, ys, written.mix if y is not None else None, written.write if y is not None else None, read, norm)
+        if y is not None and x_out is not None:
+            x_out.copy_(x)
+        if h is not None:
+            if shift is not None:
+                u = reference.token_shift(u, shift, prev, si)
+            h[:, : u.shape[1]] = u.to(h.dtype)
+        return h
+    elem = _ELEM[h.dtype if h is not None else y.dtype]
+    assert y is None or h is None or y.dtype == h.dtype
+    total, s, w = x_in.shape
+    rc = _native.load().ogb_hyper_step(
+        x_in.data_ptr(), _ptr(x_out), _ptr(y), _ptr(written.mix if y is not None else None), _ptr(written.write if y is not None else None),
+        _ptr(read), _ptr(norm.alpha if norm is not None else None), _ptr(norm.w if norm is not None else None),
+        _ptr(norm.b if norm is not None else None), _ptr(shift), _ptr(prev), _ptr(h), _ptr(gather), rows, total, s, w,
+        y.stride(0) if y is not None else 0, h.stride(0) if h is not None else 0, si.ctx_len.data_ptr(), _ptr(si.state_slot),
+        si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), si.num_decode, si.num_tiles,
+        prev.shape[0] if prev is not None else 0, elem, status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_hyper_step")
+    launch_counts["hyper_step"] += 1
+    return h
+
+
+@_timed("latent_append")
+def latent_append(c, w, eps, slots, pool, rank):
+    """RMS-norm the projected latents c [T, >= rank] and write them to their slots of pool [pages, 16, ld]."""
+    t = c.shape[0]
+    if not c.is_cuda:
+        reference.latent_append(c, w, eps, slots[:t], pool, rank)
+        return
+    assert pool.dtype == c.dtype
+    rc = _native.load().ogb_latent_append(c.data_ptr(), c.stride(0), w.data_ptr(), float(eps), slots.data_ptr(), pool.data_ptr(), t, rank,
+                                          pool.shape[2], backed_pages(pool) * PAGE, _ELEM[c.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_latent_append")
+    launch_counts["latent_append"] += 1
+
+
+@_timed("latent_attention")
+def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None):
+    """Rows (token, head) of q [T * heads, ld] over the latents of their sequences' pages; window <= 0: causal only."""
+    if not q.is_cuda:
+        reference.latent_attention(q, out, pool, si, heads, rank, scale, window)
+        return out
+    lib, st = _native.load(), status_word().data_ptr()
+    nd, npf, t = si.num_decode, si.num_prefill_seqs, si.num_tokens
+    pages, mp = backed_pages(pool), si.page_table.shape[1]
+    elem = _ELEM[q.dtype]
+    if nd > 0:
+        rc = lib.ogb_latent_attention(q.data_ptr(), out.data_ptr(), pool.data_ptr(), si.page_table.data_ptr(), si.ctx_len.data_ptr(), 0, 0, 0,
+                                      nd, heads, rank, q.stride(0), pool.shape[2], mp, 0, pages, int(window), float(scale), int(splits),
+                                      _ptr(part_o), _ptr(part_ml), elem, st, _stream())
+        _native.check(rc, "ogb_latent_attention")
+        launch_counts["latent_decode"] += 1
+    if npf > 0:
+        qp, op = q[nd * heads:], out[nd * heads:]
+        rc = lib.ogb_latent_attention(qp.data_ptr(), op.data_ptr(), pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(),
+                                      si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), t - nd, heads, rank, q.stride(0),
+                                      pool.shape[2], mp, si.num_tiles, pages, int(window), float(scale), 1, 0, 0, elem, st, _stream())
+        _native.check(rc, "ogb_latent_attention")
+        launch_counts["latent_prefill"] += 1
+    return out
+
+
+@_timed("hgrn2")
+def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si):
+    """Advance the recurrence over the step's rows: qfv [T, ld] fp32 (query, gate and value projections), state
+    [slots, heads, vdim, state_rows(dim)] fp32 in place, raw head outputs to out [T, ld] fp32."""
+    if not qfv.is_cuda:
+        reference.hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si)
+        return out
+    rc = _native.load().ogb_hgrn2(qfv.data_ptr(), bias.data_ptr(), low.data_ptr(), state.data_ptr(), out.data_ptr(), qfv.stride(0),
+                                  out.stride(0), heads, dim, vdim, si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(),
+                                  si.num_decode, si.num_prefill_seqs, state.shape[0], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_hgrn2")
+    launch_counts["hgrn2"] += 1
+    return out
+
+
+@_timed("head_rmsnorm")
+def head_rmsnorm(x, w, eps, out, heads, n):
+    """RMS norm of each head's n columns of x [T, ld] (fp32) with one shared weight."""
+    if not x.is_cuda:
+        out[:, : heads * n] = reference.head_rmsnorm(x, w, eps, heads, n, out.dtype)
+        return out
+    rc = _native.load().ogb_head_rmsnorm(x.data_ptr(), w.data_ptr(), float(eps), out.data_ptr(), x.shape[0], heads, n, x.stride(0),
+                                         out.stride(0), _ELEM[out.dtype], _stream())
+    _native.check(rc, "ogb_head_rmsnorm")
+    launch_counts["head_rmsnorm"] += 1
+    return out

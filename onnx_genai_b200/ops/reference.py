@@ -338,3 +338,102 @@ def moe_route(router_logits, k, renormalize=True):
     if renormalize:
         w = w / w.sum(-1, keepdim=True)
     return ids.to(torch.int32), w
+
+
+# ------------------------------------------------------------------------------------------
+# models with a mixer per layer (ops/hybrid.py)
+# ------------------------------------------------------------------------------------------
+def gelu_tanh(z):
+    return torch.nn.functional.gelu(z, approximate="tanh")
+
+
+GATED_ACTS = {"silu": torch.nn.functional.silu, "gelu_tanh": gelu_tanh}
+
+
+def act_mul_packed(gate_up, half, act, out_dtype=None):
+    """act(gate) * up over columns interleaved by :func:`pack_gate_up`."""
+    t, n = gate_up.shape
+    y = gate_up.float().view(t, n // (2 * half), 2, half)
+    return (GATED_ACTS[act](y[:, :, 0]) * y[:, :, 1]).reshape(t, n // 2).to(out_dtype or gate_up.dtype)
+
+
+def hyper_step(x, y=None, mix=None, out_w=None, in_w=None, norm=None):
+    """Streams x [T, S, W] fp32 -> (streams after folding y in, normed read-out u [T, W] fp32)."""
+    if y is not None:
+        x = torch.einsum("tsw,sq->tqw", x, mix) + out_w[None, :, None] * y.float()[:, None, : x.shape[2]]
+    u = x.sum(1) if in_w is None else torch.einsum("tsw,s->tw", x, in_w)
+    if norm is not None:
+        u = torch.tanh(norm.alpha * u) * norm.w + norm.b
+    return x, u
+
+
+def step_entries(si):
+    """(entry, first row, rows, position of the first row, state slot) of every sequence of a step plan."""
+    nd = si.num_decode
+    cu = si.cu_q[: si.num_prefill_seqs + 1].tolist()
+    ctx, slots = si.ctx_len[: nd + si.num_prefill_seqs].tolist(), si.state_slot[: nd + si.num_prefill_seqs].tolist()
+    for e, (c, slot) in enumerate(zip(ctx, slots)):
+        base, n = (e, 1) if e < nd else (nd + cu[e - nd], cu[e - nd + 1] - cu[e - nd])
+        if n > 0 and c > 0:
+            yield e, base, n, c - n, slot
+
+
+def token_shift(u, amount, prev, si):
+    """u [T, W] fp32 -> shifted copy; prev [slots, W] holds every sequence's last row and is advanced."""
+    out = u.clone()
+    for _, base, n, start, slot in step_entries(si):
+        rows = u[base:base + n]
+        first = prev[slot] if start > 0 else torch.zeros_like(rows[0])
+        before = torch.cat([first[None], rows[:-1]])
+        out[base:base + n] = rows + (before - rows) * amount
+        prev[slot] = rows[-1]
+    return out
+
+
+def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si):
+    """Raw head outputs of the step's rows into out [T, heads * vdim]; state [slots, heads, vdim, rows >= dim] is advanced."""
+    t = qfv.shape[0]
+    hd = heads * dim
+    q = torch.nn.functional.silu(qfv[:, :hd]).view(t, heads, dim)
+    f = (low + (1 - low) * torch.sigmoid(qfv[:, hd:2 * hd] + bias)).view(t, heads, dim)
+    v = qfv[:, 2 * hd:2 * hd + heads * vdim].view(t, heads, vdim)
+    for _, base, n, start, slot in step_entries(si):
+        s = state[slot, :, :, :dim].clone() if start > 0 else torch.zeros(heads, vdim, dim)
+        for r in range(base, base + n):
+            s = s * f[r][:, None, :] + v[r][:, :, None] * (1 - f[r])[:, None, :]
+            out[r, : heads * vdim] = torch.einsum("hvd,hd->hv", s, q[r]).reshape(-1)
+        state[slot, :, :, :dim] = s
+
+
+def head_rmsnorm(x, w, eps, heads, n, out_dtype=None):
+    y = x[:, : heads * n].float().view(-1, heads, n)
+    y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w
+    return y.reshape(x.shape[0], heads * n).to(out_dtype or x.dtype)
+
+
+def latent_append(c, w, eps, slots, pool, rank):
+    """RMS norm of every row of c, written to its slot of pool [pages, 16, >= rank]."""
+    y = c[:, :rank].float()
+    y = (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w).to(pool.dtype)
+    flat = pool.view(-1, pool.shape[-1])
+    live = slots >= 0
+    flat[slots[live].long(), :rank] = y[live]
+
+
+def latent_attention(q, out, pool, si, heads, rank, scale, window):
+    """q / out [T * heads, >= rank]: every head attends to the latents of its sequence's pages (key and value alike)."""
+    for e, base, n, start, _ in step_entries(si):
+        ctx = start + n
+        lo = max(0, start - window + 1) if window > 0 else 0
+        pages = si.page_table[e, lo // PAGE:(ctx + PAGE - 1) // PAGE].long()
+        c = pool[pages].reshape(-1, pool.shape[-1])[: ctx - lo // PAGE * PAGE, :rank].float()
+        j = torch.arange(lo // PAGE * PAGE, ctx)
+        i = torch.arange(start, ctx)
+        seen = j[None, :] <= i[:, None]
+        if window > 0:
+            seen &= i[:, None] - j[None, :] < window
+        qs = q[base * heads:(base + n) * heads, :rank].float().view(n, heads, rank)
+        s = torch.einsum("nhr,kr->nhk", qs, c) * scale
+        p = torch.softmax(s.masked_fill(~seen[:, None, :], float("-inf")), -1)
+        o = torch.einsum("nhk,kr->nhr", p, c)
+        out[base * heads:(base + n) * heads, :rank] = o.reshape(n * heads, rank).to(out.dtype)
