@@ -43,6 +43,7 @@ def _add_engine(p):
                    help="native: this package's kernels and scheduler; graph: interpret the ONNX graph node by node "
                         "(any decoder architecture, `generate` only, one sequence)")
     p.add_argument("--kv-cache-dtype", default="bf16", choices=["bf16", "fp8_e4m3fn", "fp8_e5m2", "int8"])
+    p.add_argument("--compute-dtype", default="bf16", choices=["bf16", "f32"], help="f32: weights, activations and cache in true 32-bit (checkpoint architectures that have it)")
     p.add_argument("--max-batch", type=int, default=32)
     p.add_argument("--vram-limit", default="0.85", help="0.85 (fraction of the device the engine may fill), auto, or a size such as 8GiB for weights + activations + KV")
     p.add_argument("--context-cache", action="store_true", help="keep the lowered weight layout beside the model (ogb_context/) and reuse it on the next load")
@@ -121,6 +122,8 @@ def _load(args):
         extra.update(tp=tp_world, tp_rank=tp_rank, comm=tp_comm)
     if getattr(args, "context_cache", False):
         extra["context_cache"] = True
+    if getattr(args, "compute_dtype", "bf16") != "bf16":
+        extra["compute_dtype"] = args.compute_dtype
     if getattr(args, "weight_offload_layers", 0) > 0:
         extra["weight_offload_layers"] = args.weight_offload_layers
     eng = Engine.from_dir(args.model, device=dev, max_seqs=args.max_batch, kv_dtype={"fp8_e4m3fn": "fp8", "int8": "int8", "fp8_e5m2": "fp8_e5m2"}.get(args.kv_cache_dtype, "bf16"),
@@ -237,7 +240,17 @@ def cmd_generate(args, profiler):
         print(f"generate: {e}\nThe fast path does not recognise this decoder graph; it can still run node by node: add --backend graph",
               file=sys.stderr)
         return 2
-    prompt = args.prompt if args.prompt is not None else sys.stdin.read()
+    ids = None
+    if args.prompt_ids:
+        ids = [int(t) for t in args.prompt_ids.replace(",", " ").split()]
+        vocab = eng.llm.cfg.model.vocab
+        if not ids or min(ids) < 0 or max(ids) >= vocab:
+            print(f"generate: --prompt-ids takes token ids in [0, {vocab})", file=sys.stderr)
+            return 2
+    elif eng.tokenizer is None:
+        print("generate: this model directory has no tokenizer.json; give the prompt as token ids with --prompt-ids", file=sys.stderr)
+        return 2
+    prompt = "" if ids else (args.prompt if args.prompt is not None else sys.stdin.read())
     t_lat = []
     last = [time.perf_counter()]
 
@@ -245,11 +258,11 @@ def cmd_generate(args, profiler):
         now = time.perf_counter()
         t_lat.append(now - last[0])
         last[0] = now
-        sys.stdout.write(delta)
+        sys.stdout.write(delta if eng.tokenizer is not None else f"{tok} ")
         sys.stdout.flush()
 
     with profiler.span("generate"):
-        res = eng.generate(_prompt_text(eng, prompt, args.raw), _options(args), on_token=on_token)
+        res = eng.generate(ids if ids else _prompt_text(eng, prompt, args.raw), _options(args), on_token=on_token)
     sys.stdout.write("\n")
     print(_stats_line(res), file=sys.stderr)
     profiler.report(res, t_lat[1:], eng)
@@ -554,6 +567,16 @@ def cmd_show(args, profiler):
 
     d = pkg.open_model_directory(args.model)
     meta = d.load_metadata()
+    if d.native is not None:
+        import dataclasses
+
+        from .models.registry import ARCHITECTURES
+
+        cfg = ARCHITECTURES[d.native["architecture"]].read_config(d.native)
+        print(json.dumps({"model_path": d.model_path, "tokenizer": d.tokenizer_path, "metadata": d.metadata_path,
+                          "architecture": {**dataclasses.asdict(cfg), "name": d.native["architecture"]},
+                          "max_sequence_length": meta.max_sequence_length, "weight_bytes": cfg.weight_bytes()}, indent=1))
+        return 0
     model = load_any(d.model_path)
     ops_count: dict = {}
     for n in model.graph.nodes:
@@ -598,6 +621,22 @@ def cmd_validate(args, profiler):
     except Exception as exc:
         problems.append(f"metadata: {exc}")
     cfg = None
+    if d.native is not None:
+        import torch
+
+        from .models.registry import load_checkpoint
+
+        try:
+            cfg, _ = load_checkpoint(d.root, d.native, torch.bfloat16, "cpu")
+            notes.append(f"{d.native['architecture']} checkpoint: {cfg.num_layers} layers, hidden {cfg.hidden}, vocab {cfg.vocab}, every tensor read")
+            if meta is not None and meta.vocab_size and meta.vocab_size != cfg.vocab:
+                problems.append(f"metadata model.vocab_size={meta.vocab_size} but the embedding has {cfg.vocab} rows")
+        except Exception as exc:
+            problems.append(f"checkpoint: {type(exc).__name__}: {exc}")
+        if d.tokenizer_path is None:
+            notes.append("no tokenizer.json: text prompts are unavailable, token-id prompts still work")
+        print(json.dumps({"ok": not problems, "model": d.model_path, "problems": problems, "notes": notes}, indent=1))
+        return 0 if not problems else 1
     try:
         cfg, weights, _ = lower_decoder(load_any(d.model_path), keep_int4=True)
         notes.append(f"decoder graph recognised: {cfg.num_layers} layers, hidden {cfg.hidden}, {cfg.num_heads}/{cfg.num_kv_heads} heads "
@@ -655,10 +694,13 @@ def cmd_validate(args, profiler):
 
 
 def cmd_list(args, profiler):
+    from .models.registry import native_config
+
     root = args.models_dir
     for name in sorted(os.listdir(root)):
         p = os.path.join(root, name)
-        if os.path.isdir(p) and (os.path.exists(os.path.join(p, "manifest.json")) or any(f.endswith(".onnx") for f in os.listdir(p))):
+        if os.path.isdir(p) and (os.path.exists(os.path.join(p, "manifest.json")) or any(f.endswith(".onnx") for f in os.listdir(p))
+                                 or native_config(p) is not None):
             print(name)
     return 0
 
@@ -912,6 +954,7 @@ def main(argv=None):
     g = sub.add_parser("generate")
     g.add_argument("model")
     g.add_argument("--prompt", default=None)
+    g.add_argument("--prompt-ids", default="", help="the prompt as token ids (commas or spaces); without a tokenizer the output is token ids too")
     _add_sampling(g)
     _add_engine(g)
     r = sub.add_parser("run")
@@ -946,6 +989,10 @@ def main(argv=None):
     sh.add_argument("model")
     va = sub.add_parser("validate", help="check a model directory and report every problem")
     va.add_argument("model")
+    rp = sub.add_parser("replay", help="run given token ids through a checkpoint step by step (JSON lines on standard input) and write logits")
+    from . import replay
+
+    replay.add_arguments(rp)
     pm = sub.add_parser("plan-memory", help="lifetimes, arena size and lower bound of a graph's intermediates (JSON)")
     pm.add_argument("graph", help=".onnx or .onnx.textproto file")
     pm.add_argument("--bind", action="append", default=[], metavar="SYMBOL=N", help="value of a symbolic dimension (repeatable)")
@@ -988,6 +1035,8 @@ def main(argv=None):
     if args.cmd == "diagnose":
         from .utils.diagnose import main as diagnose_main
         return diagnose_main([args.trace] + (["--category", args.category] if args.category else []) + (["--peaks", args.peaks] if args.peaks else []))
+    if args.cmd == "replay":
+        return replay.run(args)
     if args.cmd == "run-workflow":
         return cmd_run_workflow(args)
     if args.cmd == "plan-memory":

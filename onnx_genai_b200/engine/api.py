@@ -123,14 +123,16 @@ class Engine:
     def from_dir(cls, model_dir: str, device=None, page_size: int | None = None, max_seqs: int = 32,
                  max_seq_len: int | None = None, num_pages: int = 0, max_tokens_per_step: int = 2048,
                  kv_dtype: str = "bf16", max_draft_tokens: int = 0, draft_model_dir: str | None = None,
-                 keep_int4: bool | None = None, context_cache=None, tp: int = 1, tp_rank: int = 0, comm=None, **engine_kw):
+                 keep_int4: bool | None = None, context_cache=None, tp: int = 1, tp_rank: int = 0, comm=None,
+                 compute_dtype: str = "bf16", **engine_kw):
         """Load a flat model directory or a model package.  ``page_size`` is accepted for API
         compatibility; pages hold 16 tokens (the attention kernels' tile).  ``context_cache``: True (or a directory) keeps the
         lowered weight layout beside the model (``ogb_context/``) and reads it back on the next load instead of parsing and
         packing the graph again; ``ONNX_GENAI_CONTEXT_CACHE=1`` turns it on for every load.  ``tp`` > 1: this process is
         rank ``tp_rank`` of a tensor-parallel group that talks over ``comm`` (engine/tp_driver.py ``bootstrap`` gives all
         three from the launcher's environment); it loads its shard of the weights, rank 0 serves and the others call
-        :meth:`follow`."""
+        :meth:`follow`.  A checkpoint directory of a registered architecture (models/registry.py) is read without a graph;
+        ``compute_dtype="f32"`` runs it in true 32-bit."""
         if page_size not in (None, 16):
             raise ValueError(f"page_size={page_size} is not supported: KV pages hold 16 tokens")
         # precedence: the caller's arguments > ONNX_GENAI_* environment (utils/runtime_config.py) > metadata > built-in
@@ -147,7 +149,11 @@ class Engine:
         d = pkg.open_model_directory(model_dir, ep="cuda" if str(device).startswith("cuda") else "cpu",
                                      device="gpu" if str(device).startswith("cuda") else "cpu")
         meta = d.load_metadata()
-        dtype = torch.bfloat16 if str(device).startswith("cuda") else torch.float32
+        dtype = torch.bfloat16 if str(device).startswith("cuda") and compute_dtype == "bf16" else torch.float32
+        if d.native is not None:
+            if tp > 1:
+                raise ValueError(f"{model_dir}: {d.native['architecture']} checkpoints run on one GPU per replica")
+            context_cache = False
         if tp > 1:
             if comm is None:
                 raise ValueError("tensor parallelism needs a communicator: use engine.tp_driver.bootstrap() under a launcher")
@@ -159,7 +165,11 @@ class Engine:
         if context_cache is None:
             context_cache = os.environ.get("ONNX_GENAI_CONTEXT_CACHE", "0") not in ("", "0")
         cache_hit = None
-        if context_cache:
+        if d.native is not None:
+            from ..models.registry import load_checkpoint
+
+            cfg, weights = load_checkpoint(d.root, d.native, dtype, device)
+        elif context_cache:
             from ..package.context_cache import lower_with_cache
 
             cfg, weights, cache_hit = lower_with_cache(d.model_path, lambda: load_any(d.model_path), dtype, device, keep_int4,
@@ -169,11 +179,14 @@ class Engine:
         if meta.vocab_size and meta.vocab_size != cfg.vocab:
             raise md.MetadataError(f"{d.metadata_path}: model.vocab_size={meta.vocab_size} but the graph's embedding has "
                                    f"{cfg.vocab} rows; fix the metadata or re-export the model")
-        if meta.sliding_window and cfg.sliding_window <= 0:
-            cfg.sliding_window = int(meta.sliding_window)         # graphs exported without local_window_size
-        if cfg.sliding_window > 0 and meta.sink_tokens:
-            cfg.attention_sinks = int(meta.sink_tokens)
+        if d.native is None:
+            if meta.sliding_window and cfg.sliding_window <= 0:
+                cfg.sliding_window = int(meta.sliding_window)         # graphs exported without local_window_size
+            if cfg.sliding_window > 0 and meta.sink_tokens:
+                cfg.attention_sinks = int(meta.sink_tokens)
         limit = meta.max_sequence_length or cfg.max_position
+        if not max_seq_len and not meta.max_sequence_length:
+            max_seq_len = getattr(cfg, "default_seq_len", None)       # models without a positional table have no limit of their own
         max_seq_len = min(max_seq_len or limit, limit, cfg.max_position)
         tok = None
         eos = []
@@ -193,7 +206,7 @@ class Engine:
         rt.apply_engine_defaults(engine_kw, str(device).startswith("cuda"))
         ecfg = EngineConfig(model=cfg, num_pages=num_pages, max_seqs=max_seqs, max_seq_len=max_seq_len,
                             max_tokens_per_step=max_tokens_per_step, prefill_chunk=meta.chunked_prefill_size or 2048,
-                            kv_dtype=kv_dtype, max_draft_tokens=max_draft_tokens, **engine_kw)
+                            kv_dtype=kv_dtype, max_draft_tokens=max_draft_tokens, compute_dtype=compute_dtype, **engine_kw)
         llm = LLMEngine(ecfg, weights=weights, device=device, tp=tp, rank=tp_rank, comm=comm)
         draft = cls.from_dir(draft_model_dir, device=device, max_seqs=max_seqs, max_seq_len=max_seq_len) if (draft_model_dir and tp == 1) else None
         eng = cls(llm, tok, d.chat_template, meta, eos, draft)

@@ -6,6 +6,8 @@ crates/onnx-model-package/src/lib.rs, docs/genai/MODEL_PACKAGE.md:66-118):
 * flat directory: ``tokenizer.json`` (mandatory), ``decoder.onnx`` or the single ``*.onnx``,
   optional ``inference_metadata.{yaml,yml,json}``, ``genai_config.json`` (import only),
   ``chat_template.jinja`` or ``tokenizer_config.json["chat_template"]``, external ``*.onnx.data``;
+* checkpoint directory: ``config.json`` naming an architecture of :mod:`onnx_genai_b200.models.registry` and
+  ``model.safetensors`` (tokenizer, metadata and template optional, as above);
 * package directory: ``manifest.json`` (``schema_version "1.x"``, ``components{model{variants
   {name: {variant_directory, ep, device, compatibility_string, executor_info}}}}``) with
   content-addressed ``shared_assets/sha256-<digest>/`` directories referenced as
@@ -36,11 +38,12 @@ class ModelDirectory:
     variant: str | None = None
     manifest: dict | None = None
     extra: dict = field(default_factory=dict)
+    native: dict | None = None             # config.json of a checkpoint read without a graph (models/registry.py)
 
     def load_metadata(self) -> md.InferenceMetadata:
         if self.metadata_path:
             return md.load(self.metadata_path)
-        if self.genai_config is not None:
+        if self.genai_config is not None and self.native is None:
             from .genai_config import graph_ports, import_genai_config
 
             graph = None
@@ -126,6 +129,12 @@ def open_model_directory(path: str, ep: str = "cuda", device: str = "gpu", varia
             return _open_package(path, manifest, ep, device, variant)
     tok = os.path.join(path, "tokenizer.json")
     gc = os.path.join(path, "genai_config.json")
+    from ..models.registry import native_config
+
+    doc = native_config(path)
+    if doc is not None:                    # a checkpoint of a registered architecture: weights and configuration, no graph
+        return ModelDirectory(root=path, model_path=os.path.join(path, "model.safetensors"), tokenizer_path=tok if os.path.exists(tok) else None,
+                              metadata_path=md.find(path), chat_template=_chat_template(path), native=doc)
     return ModelDirectory(root=path, model_path=_find_onnx(path), tokenizer_path=tok if os.path.exists(tok) else None,
                           metadata_path=md.find(path), chat_template=_chat_template(path),
                           genai_config=json.load(open(gc)) if os.path.exists(gc) else None)

@@ -38,11 +38,14 @@ class ModelRegistry:
 
     @classmethod
     def from_dir(cls, models_dir: str, **kw):
-        """Every sub-directory that holds a model (inference metadata, a manifest or an .onnx file) is one model."""
+        """Every sub-directory that holds a model (inference metadata, a manifest, an .onnx file or a native checkpoint) is one model."""
+        from ..models.registry import native_config
+
         found = {}
         for name in sorted(os.listdir(models_dir)):
             path = os.path.join(models_dir, name)
-            if os.path.isdir(path) and any(f.endswith((".onnx", ".yaml", ".yml")) or f == "manifest.json" for f in os.listdir(path)):
+            if os.path.isdir(path) and (any(f.endswith((".onnx", ".yaml", ".yml")) or f == "manifest.json" for f in os.listdir(path))
+                                        or native_config(path) is not None):
                 found[name] = path
         return cls(found, **kw)
 

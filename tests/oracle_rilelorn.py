@@ -115,3 +115,85 @@ def forward(config, tensors, tokens, dtype=torch.float64, layers_out=None):
         if layers_out is not None:
             layers_out.append(x.sum(0))
     return norm("final.norm", x.sum(0)) @ T["head"].T
+
+
+# ------------------------------------------------------------------------------------------
+# small random checkpoints
+# ------------------------------------------------------------------------------------------
+def layer_hgrn2(heads, dim, vdim, ff):
+    return {"type": "hgrn2", "mixer": {"heads": heads, "dim": dim, "vdim": vdim}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def layer_latent(heads, dim, vdim, rank, window, ff, scale=None, kv_from=None):
+    m = {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": rank, "scale": scale or dim ** -0.5, "mask": {"size": window}}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def make_config(vocab, width, streams, layers, eps=1e-5):
+    return {"architecture": "Rilelorn", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps}, "layers": layers}
+
+
+def random_tensors(config, seed=0):
+    g = torch.Generator().manual_seed(seed)
+    W, S = config["width"], config["streams"]
+    out = {}
+
+    def normal(name, *shape, gain=1.0):
+        out[name] = (torch.randn(*shape, generator=g) * gain / shape[-1] ** 0.5).to(torch.bfloat16)
+
+    def uniform(name, *shape, lo=0.0, hi=1.0):
+        out[name] = (lo + (hi - lo) * torch.rand(*shape, generator=g)).to(torch.bfloat16)
+
+    def norm(name):
+        uniform(name, W, lo=0.6, hi=1.4)
+        uniform(name + ".b", W, lo=-0.3, hi=0.3)
+        uniform(name + ".alpha", 1, lo=0.5, hi=1.1)
+        out[name + ".alpha"] = out[name + ".alpha"].reshape(())
+
+    def hyper(name):
+        uniform(name + ".in", S, lo=0.2, hi=1.2)
+        uniform(name + ".out", S, lo=-0.4, hi=1.2)
+        uniform(name + ".mix", S, S, lo=-0.2, hi=0.4)
+        out[name + ".mix"] += torch.eye(S, dtype=torch.bfloat16) * 0.5
+
+    normal("embed", config["vocab"], W, gain=W ** 0.5)
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        norm(p + "norm1")
+        uniform(p + "shift", W, lo=0.1, hi=0.9)
+        hyper(p + "hc1")
+        if layer["type"] == "hgrn2":
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            normal(p + "mix.q", hd, W, gain=1.5)
+            normal(p + "mix.f", hd, W, gain=2.0)
+            uniform(p + "mix.f.b", hd, lo=0.0, hi=4.0)
+            uniform(p + "mix.lower", hd, lo=0.0, hi=0.9)
+            normal(p + "mix.v", hv, W, gain=1.5)
+            uniform(p + "mix.norm", m["vdim"], lo=0.5, hi=1.5)
+            normal(p + "mix.o", W, hv, gain=1.5)
+        else:
+            normal(p + "mix.q", m["heads"] * m["dim"], W, gain=2.5)
+            if "kv_from" not in m:
+                normal(p + "mix.dkv", m["kv_rank"], W)
+                uniform(p + "mix.dkv.norm", m["kv_rank"], lo=0.5, hi=1.5)
+            normal(p + "mix.uk", m["heads"] * m["dim"], m["kv_rank"], gain=2.5)
+            normal(p + "mix.uv", m["heads"] * m["vdim"], m["kv_rank"], gain=1.5)
+            normal(p + "mix.o", W, m["heads"] * m["vdim"], gain=1.5)
+        if layer["mlp"]:
+            norm(p + "norm2")
+            hyper(p + "hc2")
+            ff = layer["mlp"]["ff"]
+            normal(p + "mlp.gate", ff, W, gain=1.5)
+            normal(p + "mlp.up", ff, W)
+            normal(p + "mlp.down", W, ff, gain=1.5)
+    norm("final.norm")
+    normal("head", config["vocab"], W, gain=2.0)
+    return out
+
+
+def follows_greedily(config, tensors, prompt, out):
+    """True when every token of ``out`` is the most likely one after what precedes it."""
+    logits = forward(config, tensors, list(prompt) + list(out)[:-1])
+    return logits[len(prompt) - 1:].argmax(-1).tolist() == list(out)
