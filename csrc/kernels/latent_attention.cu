@@ -4,31 +4,17 @@
 // the result is the softmax-weighted sum of the visible c_j.  A token at position i sees j with 0 <= i - j < window
 // (window <= 0: every earlier token).
 //
-// latent_attention_warp_kernel takes any rank and both activation types: one warp per query row, four keys at a time,
-// online softmax in fp32; decode rows can split their keys over `num_splits` warps (combined by a second kernel).
-#include "hybrid.cuh"
+// bf16 rows of up to 512 values run on the tensor cores (latent_attention_tc.cu).  latent_attention_warp_kernel takes any rank
+// and both activation types: one warp per query row, four keys at a time, online softmax in fp32.  Decode rows can split
+// their keys `num_splits` ways (combined by a second kernel).
+#include <stdlib.h>
+
+#include "latent_attention.cuh"
 #include "ogb_kernels.h"
 
 namespace ogb {
 
-struct LatParams {
-  const void* q;          // [rows * heads, ldq]: rows of the launch's region (decode rows, or the packed prefill rows)
-  void* out;              // same shape
-  const void* pool;       // [pages, 16, ldp]
-  const int* page_table;  // [entries, max_pages]
-  const int* ctx_len;
-  const int* cu_q;        // null: decode (entry = row)
-  const int* tile_seq;
-  const int* tile_q0;
-  int rows, heads, rank, ldq, ldp, max_pages, num_tiles, window, num_splits;
-  int64_t num_pages;
-  float scale;
-  float *part_o, *part_ml;
-  int* status;
-};
-
 constexpr int kLatWarps = 4;
-constexpr int kLatPage = 16;
 
 template <typename T, int PER>
 __global__ void __launch_bounds__(kLatWarps * 32) latent_attention_warp_kernel(LatParams p) {
@@ -171,6 +157,22 @@ static int launch_warp(const LatParams& p, cudaStream_t stream) {
 
 using namespace ogb;
 
+static int g_latent_tc = -1;    // -1: read OGB_LATENT_TC once (default on)
+static bool use_tensor_cores() {
+  if (g_latent_tc < 0) {
+    const char* e = getenv("OGB_LATENT_TC");
+    g_latent_tc = (e != nullptr && e[0] == '0') ? 0 : 1;
+  }
+  return g_latent_tc == 1;
+}
+
+// 1 / 0: bf16 latent attention on the tensor cores or on the warp kernel (comparisons); returns the old setting.
+extern "C" int ogb_latent_set_tc(int on) {
+  const int old = use_tensor_cores() ? 1 : 0;
+  g_latent_tc = on ? 1 : 0;
+  return old;
+}
+
 extern "C" int ogb_latent_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
                                     const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages,
                                     int num_tiles, int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml,
@@ -182,7 +184,9 @@ extern "C" int ogb_latent_attention(const void* q, void* out, const void* pool, 
   LatParams p{q, out, pool, page_table, ctx_len, cu_q, tile_seq, tile_q0, rows, heads, rank, ldq, ldp, max_pages, num_tiles, window,
               num_splits < 1 ? 1 : num_splits, num_pages, scale, part_o, part_ml, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int rc = elem == kElemBF16 ? launch_warp<__nv_bfloat16>(p, s) : elem == kElemF32 ? launch_warp<float>(p, s) : -3;
+  int rc = -2;                                    // the tensor-core kernel declines what it cannot take
+  if (elem == kElemBF16 && use_tensor_cores()) rc = launch_latent_tc(p, s);
+  if (rc == -2) rc = elem == kElemBF16 ? launch_warp<__nv_bfloat16>(p, s) : elem == kElemF32 ? launch_warp<float>(p, s) : -3;
   if (rc != 0 || p.num_splits == 1) return rc;
   const int blocks = (rows * heads + 3) / 4;
   if (elem == kElemBF16)
