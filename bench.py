@@ -120,9 +120,26 @@ def main():
                     help="skip the labelled library arm (cuBLAS GEMMs + ncclAllReduce) that is replayed on the same steps for vs_baseline")
     ap.add_argument("--latency-requests", type=int, default=256,
                     help="after the timed regions keep the closed loop running until this many requests have finished (TTFT / TPOT sample)")
+    ap.add_argument("--hybrid", action="store_true", help="instead of the headline workload: prefill / decode throughput of the hybrid decoder "
+                    "(Rilelorn layers) beside a dense decoder of equal size, and every kernel against its roofline (table on stderr, JSON on stdout)")
+    ap.add_argument("--hybrid-sizes", default="small,medium,large")
+    ap.add_argument("--hybrid-json", default="")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.hybrid:
+        from onnx_genai_b200.bench import hybrid_bench
+
+        sampler = ClockSampler(0)
+        sampler.start()
+        t0 = time.perf_counter()
+        doc = hybrid_bench.main(args.hybrid_sizes.split(","), args.hybrid_json)
+        t1 = time.perf_counter()
+        sampler.stop()
+        print(json.dumps({"metric": "prefill and decode tok/s, hybrid decoder beside a dense one", "unit": "tok/s", "dtype": "bf16",
+                          "data": "synthetic (random token ids and weights)", "clocks": sampler.summary(t0, t1),
+                          "sizes": {k: v["throughput"] for k, v in doc["sizes"].items()}}))
+        return 0
     args.warmup = max(args.warmup, 3)
     # stdout carries exactly one JSON line: anything libraries print (NCCL's version banner, torchrun
     # notices) is sent to stderr by pointing fd 1 at fd 2 and keeping a private handle on the real stdout

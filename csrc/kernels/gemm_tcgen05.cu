@@ -127,8 +127,10 @@ struct GemmWork {
 // A batch of products that share shapes: problem z reads A from column z * a_step and W from row z * N, and writes its
 // results from column z * c_step of C (per-head projections of a packed row).  Columns of A past K belong to the next
 // problem; the rows of W end at K and the loads past it read zeros, so they add nothing.
+// page_d > 0 (plain epilogue, one problem): row r, column n of the result belong to token r of a paged pool of [pages][N / page_d]
+// [16][page_d] and are written there.
 struct GemmBatch {
-  int count = 1, a_step = 0, c_step = 0;
+  int count = 1, a_step = 0, c_step = 0, page_d = 0;
 };
 
 // fp32 partial accumulators of stream-K: slot = CTA, layout [BN / 32 column chunks][128 rows][32 floats], so a warp's
@@ -482,6 +484,10 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                   }
                 } else {
                   dst = C + static_cast<size_t>(grow) * ldc + c_off + gcol;
+                  if constexpr (EPI == kEpiNone)
+                    if (batch.page_d > 0)
+                      dst = C + static_cast<size_t>(grow >> 4) * 16 * N + (static_cast<size_t>(gcol / batch.page_d) * 16 + (grow & 15)) * batch.page_d +
+                            gcol % batch.page_d;
                 }
                 const bool full = (gcol + 8 <= out_cols);
                 if constexpr (EPI == kEpiResidual) {
@@ -902,6 +908,15 @@ extern "C" int ogb_gemm_bf16_batched(const void* A, const void* W, void* C, int 
   b.count = batch; b.a_step = a_step; b.c_step = c_step;
   return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, kEpiNone, 0, nullptr, nullptr, 0, b, kActSilu, status,
                             stream);
+}
+
+// Result written token by token into pages [rows / 16][N / page_d][16][page_d] (page_d a multiple of 8 that divides N).
+extern "C" int ogb_gemm_bf16_paged(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int page_d, int* status,
+                                   void* stream) {
+  if (page_d <= 0 || page_d % 8 != 0 || N % page_d != 0) return -9;
+  GemmBatch b;
+  b.page_d = page_d;
+  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, N, 0, kEpiNone, 0, nullptr, nullptr, 0, b, kActSilu, status, stream);
 }
 
 // Row-parallel GEMM of a tensor-parallel group: the partial product A[M,K_local] * W[N,K_local]^T of

@@ -28,6 +28,7 @@ struct HyperParams {
   void* h;                 // [rows, ldh] or null
   const int* gather;       // row r of h comes from row gather[r] (final norm of the rows that sample)
   int rows, total_rows, S, W, ldy, ldh;
+  int rows_per_block;      // without the shift
   StepRows sr;
   int* status;
 };
@@ -102,9 +103,9 @@ __global__ void __launch_bounds__(kHsThreads) hyper_rows_kernel(HyperParams p) {
   const int c = (blockIdx.y * kHsThreads + threadIdx.x) * V;
   if (c >= p.W) return;
   HyperCol<T, SMAX, V> col(p, c);
-  const int r0 = blockIdx.x * kHsRows;
+  const int r0 = blockIdx.x * p.rows_per_block;
 #pragma unroll 2
-  for (int j = 0; j < kHsRows; ++j) {
+  for (int j = 0; j < p.rows_per_block; ++j) {
     const int r = r0 + j;
     if (r >= p.rows) return;
     int t = r;
@@ -182,7 +183,7 @@ static int launch_hyper(const HyperParams& p, cudaStream_t stream) {
     const int blocks = p.sr.num_decode + p.sr.num_tiles * (64 / kHsRows);
     hyper_shift_kernel<T, SMAX, V><<<dim3(blocks, cols), kHsThreads, 0, stream>>>(p);
   } else {
-    hyper_rows_kernel<T, SMAX, V><<<dim3((p.rows + kHsRows - 1) / kHsRows, cols), kHsThreads, 0, stream>>>(p);
+    hyper_rows_kernel<T, SMAX, V><<<dim3((p.rows + p.rows_per_block - 1) / p.rows_per_block, cols), kHsThreads, 0, stream>>>(p);
   }
   return static_cast<int>(cudaGetLastError());
 }
@@ -347,7 +348,7 @@ extern "C" int ogb_hyper_step(const float* x_in, float* x_out, const void* y, co
   if (S < 1 || S > 8 || W < 1 || x_in == x_out) return -3;
   if (shift != nullptr && (prev == nullptr || h == nullptr || gather != nullptr)) return -3;
   if (y != nullptr && (mix == nullptr || out_w == nullptr)) return -3;
-  HyperParams p{x_in, x_out, y, mix, out_w, in_w, alpha, w, b, shift, prev, h, gather, rows, total_rows, S, W, ldy, ldh,
+  HyperParams p{x_in, x_out, y, mix, out_w, in_w, alpha, w, b, shift, prev, h, gather, rows, total_rows, S, W, ldy, ldh, rows <= 1024 ? 1 : kHsRows,
                 StepRows{ctx_len, state_slot, cu_q, tile_seq, tile_q0, num_decode, num_tiles, num_slots}, status};
   const bool vec = W % 4 == 0 && ldy % 4 == 0 && ldh % 4 == 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

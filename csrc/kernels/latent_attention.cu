@@ -139,6 +139,31 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
   }
 }
 
+// Visible latents of every prefill entry, packed page by page: block b copies one 16-token page to dense rows 16 b .. 16 b + 15
+// and enters b into the entry's scratch page table.
+__global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restrict__ pool, const int* __restrict__ page_table,
+                                                            const int* __restrict__ ctx_len, const int* __restrict__ cu_q, int entries, int max_pages,
+                                                            int64_t num_pages, int window, int vecs, uint4* __restrict__ out,
+                                                            int* __restrict__ scratch_table, int* status) {
+  int b = blockIdx.x, e = 0, pi = -1;
+  for (; e < entries; ++e) {
+    const int ctx = ctx_len[e], start = ctx - (cu_q[e + 1] - cu_q[e]);
+    const int lo = (window > 0 ? max(0, start - window + 1) : 0) / kLatPage, n = (ctx + kLatPage - 1) / kLatPage - lo;
+    if (b < n) { pi = lo + b; break; }
+    b -= n;
+  }
+  if (pi < 0 || pi >= max_pages) return;
+  int64_t page = page_table[static_cast<size_t>(e) * max_pages + pi];
+  if (page < 0 || page >= num_pages) {
+    if (threadIdx.x == 0) atomicOr(status, kStatusIndexOutOfRange);
+    page = 0;
+  }
+  if (threadIdx.x == 0) scratch_table[static_cast<size_t>(e) * max_pages + pi] = blockIdx.x;
+  const uint4* src = pool + static_cast<size_t>(page) * kLatPage * vecs;
+  uint4* dst = out + static_cast<size_t>(blockIdx.x) * kLatPage * vecs;
+  for (int i = threadIdx.x; i < kLatPage * vecs; i += blockDim.x) dst[i] = src[i];
+}
+
 template <typename T>
 static int launch_warp(const LatParams& p, cudaStream_t stream) {
   const long long blocks = p.cu_q == nullptr ? (static_cast<long long>(p.rows) * p.heads + kLatWarps - 1) / kLatWarps
@@ -193,5 +218,17 @@ extern "C" int ogb_latent_attention(const void* q, void* out, const void* pool, 
     latent_combine_kernel<<<blocks, 128, 0, s>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), ctx_len, rows, heads, rank, ldq, p.num_splits);
   else
     latent_combine_kernel<<<blocks, 128, 0, s>>>(part_o, part_ml, static_cast<float*>(out), ctx_len, rows, heads, rank, ldq, p.num_splits);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Packs the visible latents (bf16, rows of ldp values, ldp a multiple of 8) of the prefill entries for an expansion to keys and
+// values; `blocks` = their pages in total.
+extern "C" int ogb_latent_gather(const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, int entries, int max_pages,
+                                 int64_t num_pages, int window, int ldp, int blocks, void* out, int* scratch_table, int* status, void* stream) {
+  if (blocks <= 0 || entries <= 0) return 0;
+  if (ldp % 8 != 0) return -3;
+  latent_gather_kernel<<<blocks, 128, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const uint4*>(pool), page_table, ctx_len, cu_q, entries,
+                                                                             max_pages, num_pages, window, ldp / 8, static_cast<uint4*>(out),
+                                                                             scratch_table, status);
   return static_cast<int>(cudaGetLastError());
 }

@@ -30,7 +30,9 @@ int ogb_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int
 // `batch` products of one shape: C[:, z*c_step : +N] = A[:, z*a_step : +K] * W[z*N : +N, :]^T (steps are multiples of 8).
 int ogb_gemm_bf16_batched(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step,
                           int c_step, int* status, void* stream);
-// The same in fp32 without any reduced-precision mode.
+// C written token by token into pages [M / 16][N / page_d][16][page_d].
+int ogb_gemm_bf16_paged(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int page_d, int* status, void* stream);
+// Products as ogb_gemm_bf16_batched in fp32 without any reduced-precision mode.
 int ogb_gemm_f32(const float* A, const float* W, float* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step, int c_step,
                  void* stream);
 
@@ -171,6 +173,9 @@ int ogb_latent_attention(const void* q, void* out, const void* pool, const int* 
                          const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages, int num_tiles,
                          int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml, int elem, int* status,
                          void* stream);
+int ogb_latent_gather(const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, int entries, int max_pages, int64_t num_pages,
+                      int window, int ldp, int blocks, void* out, int* scratch_table, int* status, void* stream);
+int ogb_latent_set_tc(int on);
 int ogb_hgrn2_state_rows(int D);
 int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D, int V,
               const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int* status,

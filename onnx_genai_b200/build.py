@@ -41,7 +41,8 @@ NVCC_FLAGS = [
 PRECISE_SOURCES = {"hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_attention_tc.cu"}
 # A library of its own for models that need only a few of the kernel sources: built when the full library is not there, so
 # that the first load compiles no more than the model uses (ops/_native.py ``prefer``).
-SUBSETS = {"hybrid": ("hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_attention_tc.cu", "gemm_tcgen05.cu", "sampling.cu", "tp_comm.cu")}
+SUBSETS = {"hybrid": ("hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_attention_tc.cu", "attention_tc.cu", "attention.cu", "gemm_tcgen05.cu",
+                      "sampling.cu", "tp_comm.cu")}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-fopenmp", "-mavx2", "-mfma"]
 
 

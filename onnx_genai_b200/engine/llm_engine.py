@@ -436,6 +436,12 @@ class LLMEngine:
             self.kv_lease.resize(kv.mapped_bytes())
             self.kv_grows += 1
 
+    def _host_entries(self, si) -> None:
+        """The prefill entries of the plan as the host knows them (executors size their work by it)."""
+        L, pn, nd, n = self.L, self.plan_np, si.num_decode, si.num_prefill_seqs
+        cu = pn[L.cu_q:L.cu_q + n + 1] if n else np.zeros(1, dtype=np.int32)
+        si.prefill_ctx, si.prefill_len = pn[L.ctx_len + nd:L.ctx_len + nd + n].copy(), np.diff(cu)
+
     def _pick_splits(self, nd: int, max_ctx: int) -> int:
         if self.cfg.decode_splits > 0:
             return self.cfg.decode_splits
@@ -724,6 +730,7 @@ class LLMEngine:
         si.num_prefill_seqs, si.num_tiles = int(hdr[HDR["num_prefill_seqs"]]), int(hdr[HDR["num_tiles"]])
         si.num_logit_rows, si.max_ctx = int(hdr[HDR["num_logit_rows"]]), int(hdr[HDR["max_ctx"]])
         r = si.num_logit_rows
+        self._host_entries(si)
         if self.device.type == "cuda":
             self.plan_dev.copy_(self.plan_host[: self.dev_words], non_blocking=True)
             self.h2d_bytes += self.dev_words * 4

@@ -154,6 +154,8 @@ class StepInputs:
     logit_rows: torch.Tensor       # [R]
     max_ctx: int = 0
     state_slot: torch.Tensor | None = None     # [S] slot of every entry's recurrent state (models that keep some)
+    prefill_ctx: object = None     # host copies (numpy) of the prefill entries' context lengths and row counts
+    prefill_len: object = None
     # Speculative verification over long contexts: when every "prefill" sequence of the step is just a handful
     # of draft rows, the engine describes those rows as decode rows (one page-table row and context length per
     # query row) so attention runs on the split-KV decode kernel instead of walking the whole context in one CTA.

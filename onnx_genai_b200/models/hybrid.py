@@ -7,7 +7,8 @@ a layer to a fixed list of launches over buffers allocated once:
 
     hyper_step (fold the last sublayer's output into the streams, read-out, norm, token shift)
     recurrent:  gemm(q | gate | v, fp32 out) | hgrn2 | head_rmsnorm | gemm(o)
-    latent:     gemm(q | latent) | latent_append | gemm per head (W_uk^T q) | latent_attention | gemm per head (W_uv o) | gemm(o)
+    latent:     gemm(q | latent) | latent_append | gemm per head (W_uk^T q) | latent_attention | gemm per head (W_uv o) | gemm(o);
+                prompts over wide latents: latent_gather | gemm (K | V pages) | paged_prefill | gemm(o)
     hyper_step | gemm(gate_up, gated epilogue) | gemm(down)
 
 The residual streams, norms, gates and recurrent state are fp32 in every engine; matrix products and the activations
@@ -172,6 +173,7 @@ class LatentWeights:
     uk: torch.Tensor              # [heads * rank_p, dim_p]: W_uk^T per head, folds the key expansion into the query
     uv: torch.Tensor              # [heads * vdim_p, rank_p]: value expansion, applied to the attended latent
     o: torch.Tensor               # [hidden, heads * vdim_p]
+    kv: torch.Tensor | None = None   # [heads * (key | value) * dim, rank_p]: both expansions, for prompts (see expand_prompts)
 
 
 @dataclass
@@ -212,6 +214,12 @@ def pack_recurrent(spec: RecurrentSpec, q, f, f_bias, low, v, norm, o) -> Recurr
                             norm=norm.float().contiguous(), o=pad_cols(o))
 
 
+def expand_prompts(spec: LatentSpec, dtype) -> bool:
+    """Whether prompts of a layer may run on expanded keys and values: the heads fit the paged prefill kernel, and a latent is
+    wider than a head (otherwise attending to the latent itself is no more work)."""
+    return dtype == torch.bfloat16 and spec.dim == spec.vdim and spec.dim in (64, 128) and spec.rank > spec.dim
+
+
 def pack_latent(spec: LatentSpec, q, dkv, dkv_norm, uk, uv, o) -> LatentWeights:
     h, dp, rp, vp = spec.heads, pad8(spec.dim), pad8(spec.rank), pad8(spec.vdim)
     qc = pad_head_rows(q, h, dp)
@@ -219,7 +227,10 @@ def pack_latent(spec: LatentSpec, q, dkv, dkv_norm, uk, uv, o) -> LatentWeights:
         qc = torch.cat([qc, pad_head_rows(dkv, 1, rp)], 0)
     ukt = uk.reshape(h, spec.dim, spec.rank).transpose(1, 2)                                   # [h, rank, dim]
     ukt = torch.nn.functional.pad(ukt, (0, dp - spec.dim, 0, rp - spec.rank)).reshape(h * rp, dp)
-    return LatentWeights(qc=pad_cols(qc), c_norm=None if dkv_norm is None else dkv_norm.float().contiguous(), uk=ukt.contiguous(),
+    kv = None
+    if expand_prompts(spec, q.dtype):
+        kv = pad_cols(torch.stack([uk.reshape(h, spec.dim, spec.rank), uv.reshape(h, spec.vdim, spec.rank)], 1).reshape(2 * h * spec.dim, spec.rank), rp)
+    return LatentWeights(kv=kv, qc=pad_cols(qc), c_norm=None if dkv_norm is None else dkv_norm.float().contiguous(), uk=ukt.contiguous(),
                          uv=pad_cols(pad_head_rows(uv, h, vp), rp),
                          o=torch.nn.functional.pad(o.reshape(o.shape[0], h, spec.vdim), (0, vp - spec.vdim)).reshape(o.shape[0], h * vp).contiguous())
 
@@ -304,6 +315,7 @@ class HybridModel:
         self.decode_splits, self._split_capacity = 1, 1
         self.part_o = self.part_ml = None
         self.state = None
+        self.scratch: dict = {}
         self.capture = None            # list: gets the summed streams [rows, hidden] after every layer (tests, debugging)
 
     # ---- the engine's view -------------------------------------------------------------------
@@ -362,13 +374,46 @@ class HybridModel:
         hops.linear(h, w.qc, qc)
         if own:
             hops.latent_append(qc[:, hp * dp:], w.c_norm, self.cfg.norm_eps, si.slots, pool, m.rank)
-        qa, oc = self._rows(self.qa, t, hp * rp), self._rows(self.oc, t, hp * rp)
-        hops.linear_batched(qc, w.uk, qa, hp, dp, rp)
-        hops.latent_attention(qa.view(t * hp, rp), oc.view(t * hp, rp), pool, si, hp, rp, m.scale, m.window, self.decode_splits, self.part_o,
-                              self.part_ml)
         attn = self._rows(self.attn, t, hp * vp)
-        hops.linear_batched(oc, w.uv, attn, hp, rp, vp)
+        pages = self._expanded_pages(m, w, si)
+        rows = si.num_decode if pages else t      # rows that attend to the latents themselves
+        if rows:
+            qa, oc = self._rows(self.qa, rows, hp * rp), self._rows(self.oc, rows, hp * rp)
+            hops.linear_batched(qc[:rows], w.uk, qa, hp, dp, rp)
+            hops.latent_attention(qa.view(rows * hp, rp), oc.view(rows * hp, rp), pool, si, hp, rp, m.scale, m.window, self.decode_splits,
+                                  self.part_o, self.part_ml, decode_only=bool(pages))
+            hops.linear_batched(oc, w.uv, attn[:rows], hp, rp, vp)
+        if pages:
+            hops.latent_prefill_expanded(qc, attn, pool, w.kv, si, hp, m.dim, m.scale, m.window, pages,
+                                         self._scratch("dense", (pages * ops.PAGE, rp), m), self._scratch("kv", (pages, hp, 2, ops.PAGE, m.dim), m),
+                                         self._scratch("table", (si.num_prefill_seqs, si.page_table.shape[1]), m, torch.int32))
         hops.linear(attn, w.o, y)
+
+    EXPAND_BYTES = 1 << 30             # most memory the expanded keys and values of a step may take
+
+    def _expanded_pages(self, m: LatentSpec, w: LatentWeights, si) -> int:
+        """Pages to expand for this step's prompts, 0 to attend to the latents: with few queries per visible latent the
+        expansion costs more than it saves."""
+        if w.kv is None or si.num_prefill_seqs == 0 or si.prefill_ctx is None or self.device.type != "cuda":
+            return 0
+        pages = hops.visible_pages(si, m.window)
+        n, start = si.prefill_len.astype("int64"), (si.prefill_ctx - si.prefill_len).astype("int64")
+        seen = start + (n + 1) // 2
+        pairs = int((n * (seen.clip(max=m.window) if m.window > 0 else seen)).sum())
+        # operations per head: the latent kernel computes scores once per 128 output columns of a wide latent
+        direct = pairs * 2 * m.rank * (1 + max(1, -(-m.rank // 128)))
+        expanded = pairs * 4 * m.dim + pages * ops.PAGE * 4 * m.dim * m.rank
+        return pages if direct > expanded and pages * ops.PAGE * m.heads * m.dim * 4 <= self.EXPAND_BYTES else 0
+
+    def _scratch(self, name, shape, m, dtype=None):
+        """Step scratch that grows to the largest step seen (prompt steps only: never inside a captured graph)."""
+        n = 1
+        for d in shape:
+            n *= d
+        buf = self.scratch.get(name)
+        if buf is None or buf.numel() < n:
+            buf = self.scratch[name] = torch.zeros(n, dtype=dtype or self.w.embed.dtype, device=self.device)
+        return buf[:n].view(shape)
 
     def forward(self, si, kv) -> torch.Tensor:
         """Runs one step; returns logits [num_logit_rows, vocab] (a view of a static buffer)."""

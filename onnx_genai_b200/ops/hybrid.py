@@ -19,6 +19,9 @@ _native.register("ogb_hyper_step", [P] * 13 + [I] * 6 + [P] * 5 + [I] * 4 + [P, 
 _native.register("ogb_embed_streams", [P, P, P, I, I, I, I, I, P, P])
 _native.register("ogb_latent_append", [P, I, P, F, P, P, I, I, I, L, I, P, P])
 _native.register("ogb_latent_attention", [P] * 8 + [I] * 7 + [L, I, F, I, P, P, I, P, P])
+_native.register("ogb_latent_gather", [P, P, P, P, I, I, L, I, I, I, P, P, P, P])
+_native.register("ogb_latent_set_tc", [I])
+_native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
 _native.register("ogb_hgrn2_state_rows", [I])
 _native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 3 + [P, P])
 _native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, I, P])
@@ -171,8 +174,9 @@ def latent_append(c, w, eps, slots, pool, rank):
 
 
 @_timed("latent_attention")
-def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None):
-    """Rows (token, head) of q [T * heads, ld] over the latents of their sequences' pages; window <= 0: causal only."""
+def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None, decode_only=False):
+    """Rows (token, head) of q [T * heads, ld] over the latents of their sequences' pages; window <= 0: causal only.
+    ``decode_only``: leave the prefill rows to :func:`latent_prefill_expanded`."""
     if not q.is_cuda:
         reference.latent_attention(q, out, pool, si, heads, rank, scale, window)
         return out
@@ -186,7 +190,7 @@ def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, par
                                       _ptr(part_o), _ptr(part_ml), elem, st, _stream())
         _native.check(rc, "ogb_latent_attention")
         launch_counts["latent_decode"] += 1
-    if npf > 0:
+    if npf > 0 and not decode_only:
         qp, op = q[nd * heads:], out[nd * heads:]
         rc = lib.ogb_latent_attention(qp.data_ptr(), op.data_ptr(), pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(),
                                       si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), t - nd, heads, rank, q.stride(0),
@@ -194,6 +198,34 @@ def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, par
         _native.check(rc, "ogb_latent_attention")
         launch_counts["latent_prefill"] += 1
     return out
+
+
+def visible_pages(si, window):
+    """KV pages that the prefill rows of a step can see, from the host's copy of the plan."""
+    start = si.prefill_ctx - si.prefill_len
+    lo = (start - window + 1).clip(0) // PAGE if window > 0 else 0
+    return int(((si.prefill_ctx + PAGE - 1) // PAGE - lo).sum())
+
+
+def latent_prefill_expanded(q, out, pool, kv_w, si, heads, d, scale, window, pages, dense, kv, table):
+    """Prefill rows with keys and values expanded: the visible latents are packed (``dense`` [16 * pages, ld]), one product with
+    ``kv_w`` [heads * (key | value) * d, ld] writes K/V pages (``kv`` [pages, heads, 2, 16, d]), and the paged prefill kernel of the
+    dense decoders runs over them through ``table``.  Worth it when many queries share a latent and the latent is wider
+    than a head: a (query, key) pair then costs 4 d instead of 4 rank operations per head."""
+    from . import paged_prefill
+
+    nd, npf, t = si.num_decode, si.num_prefill_seqs, si.num_tokens
+    lib, st = _native.load(), status_word().data_ptr()
+    mp = si.page_table.shape[1]
+    rc = lib.ogb_latent_gather(pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(), si.cu_q.data_ptr(), npf, mp,
+                               backed_pages(pool), int(window), pool.shape[2], pages, dense.data_ptr(), table.data_ptr(), st, _stream())
+    _native.check(rc, "ogb_latent_gather")
+    rc = lib.ogb_gemm_bf16_paged(dense.data_ptr(), kv_w.data_ptr(), kv.data_ptr(), pages * PAGE, kv_w.shape[0], kv_w.shape[1], dense.stride(0),
+                                 kv_w.stride(0), d, st, _stream())
+    _native.check(rc, "ogb_gemm_bf16_paged")
+    launch_counts["latent_expand"] += 1
+    paged_prefill(q[nd:t], out[nd:t], kv[:pages], table[:npf], si.ctx_len[nd:nd + npf], si.cu_q, si.tile_seq, si.tile_q0, si.num_tiles, heads, heads,
+                  d, scale, window)
 
 
 @_timed("hgrn2")

@@ -29,7 +29,10 @@ ODD = O.make_config(61, 50, 1, [O.layer_latent(1, 10, 14, 18, 1, 33), O.layer_hg
 RECURRENT = O.make_config(64, 64, 2, [O.layer_hgrn2(4, 16, 16, 64), O.layer_hgrn2(2, 130, 40, 64)])
 ATTENTION = O.make_config(80, 128, 4, [O.layer_latent(8, 32, 32, 128, 70, 128), O.layer_latent(4, 64, 64, 128, 33, 128, kv_from=0),
                                        O.layer_latent(16, 32, 16, 192, 200, 128)])
-CONFIGS = {"mixed": MIXED, "odd": ODD, "recurrent": RECURRENT, "attention": ATTENTION}
+# latents wider than a head: prompts run on expanded keys and values in bf16
+WIDE = O.make_config(90, 96, 2, [O.layer_latent(3, 64, 64, 136, 37, 64), O.layer_hgrn2(2, 24, 24, 64), O.layer_latent(2, 128, 128, 136, 90, 64, kv_from=0),
+                                 O.layer_latent(1, 64, 64, 200, 500, 0)])
+CONFIGS = {"mixed": MIXED, "odd": ODD, "recurrent": RECURRENT, "attention": ATTENTION, "wide": WIDE}
 
 
 @pytest.fixture(scope="module")
@@ -394,6 +397,28 @@ def test_far_key_and_window_edge_show_in_logits(models, where):
         for ids in (a, b):
             want = O.forward(cfg, tensors, ids)
             assert_logits(replay_cuts(eng, ids, [50, 2, 60, 1]), want, where)
+
+
+@GPU
+def test_prompts_on_expanded_latents(models):
+    """Prompts with and without a past, beside decoded tokens, on the expanded keys and values; short portions stay on the
+    latents; the two agree."""
+    cfg, tensors = models["wide"]
+    eng = make_engine(cfg, tensors, ("cuda", "bf16"), max_tokens=768)
+    ids = {k: tokens_of(cfg, 240, 90 + i) for i, k in enumerate("abc")}
+    want = {k: O.forward(cfg, tensors, v) for k, v in ids.items()}
+    rep, at, rows = replay.Replayer(eng), dict.fromkeys("abc", 0), {k: [] for k in "abc"}
+    count = lambda: ops.launch_counts["latent_expand"]
+    for portions, expanded in (({"a": 130}, True), ({"a": 1, "b": 140}, True), ({"a": 1, "b": 2, "c": 1}, False), ({"a": 108, "b": 98, "c": 120}, True),
+                               ({"c": 119}, True)):
+        c0 = count()
+        out = rep.step([{"id": k, "tokens": ids[k][at[k]:at[k] + n], "want": list(range(n))} for k, n in portions.items()], [])
+        assert (count() > c0) == expanded
+        for k, n in portions.items():
+            rows[k] += [out.pop(0) for _ in range(n)]
+            at[k] += n
+    for k in "abc":
+        assert_logits(torch.stack(rows[k]), want[k], ("cuda", "bf16"))
 
 
 # ------------------------------------------------------------------------------------------
