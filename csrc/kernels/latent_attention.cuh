@@ -24,5 +24,7 @@ struct LatParams {
 
 // Tensor-core launch; -2 when it does not take the call (rank above 512, alignment).
 int launch_latent_tc(const LatParams& p, cudaStream_t stream);
+// Decode rows (latent_decode.cu); launch_latent_tc hands them over.
+int launch_latent_decode(const LatParams& p, cudaStream_t stream);
 
 }  // namespace ogb

@@ -427,6 +427,7 @@ int launch_latent_tc(const LatParams& p, cudaStream_t stream) {
   if (p.rank > 512 || p.rank % 8 != 0 || p.ldq % 8 != 0 || p.ldp % 8 != 0 || p.num_pages <= 0) return -2;
   if ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.out) | reinterpret_cast<uintptr_t>(p.pool) |
        reinterpret_cast<uintptr_t>(p.part_o)) & 15) return -2;
+  if (p.cu_q == nullptr) return launch_latent_decode(p, stream);
   if (p.scale <= 0.f) return -2;           // the row maximum is taken before scaling
   if (p.rank <= 64) return launch_lt<64, 64, 128, 4>(p, stream);
   if (p.rank <= 128) return launch_lt<128, 128, 128, 4>(p, stream);

@@ -1,0 +1,305 @@
+// Decode attention over paged latents: one token per sequence, up to 32 heads per CTA against one stream of latents.
+//
+// A decode row has few query rows (the heads), so the 128-row tensor-memory tiles of the prefill kernel would spend most of
+// their shared-memory traffic on rows that do not exist.  Here the products run on mma.sync m16n8k16 with 16 or 32 rows and
+// the kernel is laid out around the byte stream instead:
+//
+//   warp 8    : TMA producer, 64 tokens (4 pages) x R values per stage, 128-byte swizzled column chunks
+//   warps 0-7 : S = Q' C^T split four ways over the latent's columns and two ways over the tokens (a warp keeps its slice of
+//               Q' in registers for the whole call), partial scores summed through shared memory, softmax by eight threads a
+//               row, then O += P C with a warp owning R / 8 output columns
+//
+// Keys split `num_splits` ways leave fp32 partials for latent_combine_kernel.  Waits are bounded; page ids are checked.
+#include "attention_common.cuh"
+#include "attention_tc.cuh"
+#include "latent_attention.cuh"
+#include "ogb_kernels.h"
+
+namespace ogb {
+
+constexpr int kLdKeys = 64;
+constexpr int kLdWarps = 8;
+constexpr int kLdThreads = (kLdWarps + 1) * 32;
+constexpr int kLdPitch = 72;             // floats per row of partial scores: conflict-free 8-byte stores
+
+template <int R, int MT, int ST>
+struct LdCfg {
+  static constexpr int kRows = 16 * MT;
+  static constexpr int kChunks = R / 64;
+  static constexpr int kStage = kLdKeys * R * 2;
+  static constexpr int kQBytes = kRows * R * 2;
+  static constexpr int kPBytes = kRows * 128;
+  static constexpr int kSBytes = 4 * kRows * kLdPitch * 4;
+  static constexpr int kSmemBytes = ST * kStage + kQBytes + kPBytes + kSBytes + 1024 /*alignment*/ + 512 /*barriers, row factors*/ + 256;
+  static_assert(kSmemBytes <= 227 * 1024, "shared memory");
+};
+
+// byte offset of (row, column) in a tile of [64-column chunk][rows][128 bytes], 128-byte swizzle
+OGB_DEVICE uint32_t ld_off(int rows, int row, int col) {
+  return static_cast<uint32_t>(((col >> 6) * rows + row) * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4));
+}
+
+template <int R, int MT, int ST>
+__global__ void __launch_bounds__(kLdThreads, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap c_map, const LatParams p) {
+  using Cfg = LdCfg<R, MT, ST>;
+  constexpr int KS = R / 64;             // k-steps of a warp's column slice (R / 4 columns)
+  constexpr int NT = R / 64;             // 8-column output tiles of a warp
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* sK = smem;
+  uint8_t* sQ = sK + ST * Cfg::kStage;
+  uint8_t* sP = sQ + Cfg::kQBytes;
+  float* sS = reinterpret_cast<float*>(sP + Cfg::kPBytes);
+  uint64_t* full = reinterpret_cast<uint64_t*>(sS + 4 * Cfg::kRows * kLdPitch);
+  uint64_t* empty = full + ST;
+  uint64_t* q_full = empty + ST;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(q_full + 1);
+  float* sA = reinterpret_cast<float*>(q_full + 2);      // [rows] rescale factors, at the end 1 / l or the split's (m, l)
+
+  const int entry = blockIdx.x, head0 = blockIdx.y * Cfg::kRows;
+  const int ctx = p.ctx_len[entry];
+  if (ctx <= 0) return;                                  // padding row
+  const int heads = min(Cfg::kRows, p.heads - head0);
+  const int lo = p.window > 0 ? max(0, ctx - p.window) : 0;
+  int b0 = lo / kLdKeys, b1 = (ctx + kLdKeys - 1) / kLdKeys;
+  if (p.num_splits > 1) {
+    const int per = (b1 - b0 + p.num_splits - 1) / p.num_splits;
+    b0 += static_cast<int>(blockIdx.z) * per;
+    b1 = min(b1, b0 + per);
+  }
+  const size_t row0 = static_cast<size_t>(entry) * p.heads + head0;
+  const int nblk = b1 - b0;
+  if (nblk <= 0) {
+    if (static_cast<int>(threadIdx.x) < heads) {
+      const size_t pr = (row0 + threadIdx.x) * p.num_splits + blockIdx.z;
+      p.part_ml[2 * pr] = -INFINITY;
+      p.part_ml[2 * pr + 1] = 0.f;
+    }
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < ST; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], kLdWarps); }
+    mbar_init(q_full, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  __syncthreads();
+
+  if (warp == kLdWarps) {
+    if (lane == 0) {
+      mbar_expect_tx(q_full, Cfg::kQBytes);
+      for (int h = 0; h < Cfg::kChunks; ++h) tma_load_2d(sQ + h * Cfg::kRows * 128, &q_map, q_full, h * 64, static_cast<int>(row0));
+      const int n_pages = (ctx + kLatPage - 1) / kLatPage;
+      const int* table = p.page_table + static_cast<size_t>(entry) * p.max_pages;
+      for (int it = 0; it < nblk; ++it) {
+        const int st = it % ST;
+        int row_of_page[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int pi = min(max((b0 + it) * 4 + i, lo / kLatPage), min(n_pages, p.max_pages) - 1);   // the rest is masked
+          int64_t page = table[pi];
+          if (page < 0 || page >= p.num_pages) {
+            atomicOr(p.status, kStatusIndexOutOfRange);
+            page = 0;
+          }
+          row_of_page[i] = static_cast<int>(page) * kLatPage;
+        }
+        if (!fa_wait(&empty[st], ((it / ST) & 1) ^ 1, abort_flag)) { atomicOr(p.status, kStatusWaitTimeout); *abort_flag = 1; break; }
+        mbar_expect_tx(&full[st], Cfg::kStage);
+        uint8_t* dst = sK + st * Cfg::kStage;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int h = 0; h < Cfg::kChunks; ++h) tma_load_2d(dst + h * kLdKeys * 128 + i * 2048, &c_map, &full[st], h * 64, row_of_page[i]);
+      }
+    }
+    // the copies in flight are waited for by the consumers (bounded), which leave after the last one
+    return;
+  }
+
+  // ------------------------------ consumers ------------------------------
+  const int g = lane >> 2, t = lane & 3;
+  const int ks = warp >> 1, kh = warp & 1;               // column slice and token half of the score product
+  const uint32_t aK = smem_u32(sK), aQ = smem_u32(sQ), aP = smem_u32(sP);
+  bool ok = fa_wait(q_full, 0, abort_flag);
+  uint32_t qf[MT][KS][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+      ldsm_x4(aQ + ld_off(Cfg::kRows, m * 16 + (lane & 15), ks * (R / 4) + k * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
+  float o[MT][NT][4] = {};
+  const int srow = threadIdx.x / 8, sub = threadIdx.x & 7;      // softmax: eight threads a row (rows past 16 * MT idle)
+  float m_run = -INFINITY, l_run = 0.f;
+  const float scale = p.scale * 1.4426950408889634f;
+  for (int it = 0; it < nblk; ++it) {
+    const int st = it % ST;
+    ok = __all_sync(0xffffffffu, ok && fa_wait(&full[st], (it / ST) & 1, abort_flag));
+    if (!ok && lane == 0) { atomicOr(p.status, kStatusWaitTimeout); *abort_flag = 1; }
+    const uint32_t kb = aK + st * Cfg::kStage;
+    // ---- partial scores ----
+    float s[MT][4][4] = {};
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+#pragma unroll
+      for (int n2 = 0; n2 < 2; ++n2) {
+        uint32_t b[4];
+        ldsm_x4(kb + ld_off(kLdKeys, kh * 32 + n2 * 16 + (lane >> 4) * 8 + (lane & 7), ks * (R / 4) + k * 16 + ((lane >> 3) & 1) * 8), b[0], b[1], b[2], b[3]);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16_16816(s[m][2 * n2], qf[m][k], b[0], b[1]);
+          mma_bf16_16816(s[m][2 * n2 + 1], qf[m][k], b[2], b[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        float* d = sS + (ks * Cfg::kRows + m * 16 + g) * kLdPitch + kh * 32 + n * 8 + 2 * t;
+        *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
+        *reinterpret_cast<float2*>(d + 8 * kLdPitch) = make_float2(s[m][n][2], s[m][n][3]);
+      }
+    asm volatile("bar.sync 1, 256;" ::: "memory");
+    // ---- softmax ----
+    if (srow < Cfg::kRows) {
+      float v[8];
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        float4 a = *reinterpret_cast<const float4*>(sS + srow * kLdPitch + sub * 8 + 4 * h);
+#pragma unroll
+        for (int x = 1; x < 4; ++x) {
+          const float4 b = *reinterpret_cast<const float4*>(sS + (x * Cfg::kRows + srow) * kLdPitch + sub * 8 + 4 * h);
+          a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
+        }
+        v[4 * h] = a.x; v[4 * h + 1] = a.y; v[4 * h + 2] = a.z; v[4 * h + 3] = a.w;
+      }
+      const int key0 = (b0 + it) * kLdKeys + sub * 8;
+      float mx = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        v[j] = key0 + j >= lo && key0 + j < ctx ? v[j] * scale : -INFINITY;
+        mx = fmaxf(mx, v[j]);
+      }
+      const unsigned act = __activemask();
+#pragma unroll
+      for (int x = 1; x < 8; x <<= 1) mx = fmaxf(mx, __shfl_xor_sync(act, mx, x));
+      const float m_new = fmaxf(m_run, mx);
+      const float alpha = m_run == -INFINITY ? 0.f : exp2f(m_run - m_new);
+      const float neg = m_new == -INFINITY ? 0.f : -m_new;
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) { v[j] = exp2f(v[j] + neg); sum += v[j]; }
+      l_run = l_run * alpha + sum;                       // this thread's keys; the row's sum is formed at the end
+      m_run = m_new;
+      *reinterpret_cast<uint4*>(sP + ld_off(Cfg::kRows, srow, sub * 8)) =
+          make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+      if (sub == 0) sA[srow] = alpha;
+    }
+    asm volatile("bar.sync 1, 256;" ::: "memory");
+    // ---- O += P C ----
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float a0 = sA[m * 16 + g], a1 = sA[m * 16 + g + 8];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
+      }
+    }
+#pragma unroll
+    for (int kk = 0; kk < 2; ++kk) {
+      uint32_t pf[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+          ldsm_x4(aP + ld_off(Cfg::kRows, m * 16 + (lane & 15), kk * 32 + k * 16 + (lane >> 4) * 8), pf[m][k][0], pf[m][k][1], pf[m][k][2], pf[m][k][3]);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        uint32_t b[4];
+        ldsm_x4_t(kb + ld_off(kLdKeys, kk * 32 + lane, warp * (R / 8) + n * 8), b[0], b[1], b[2], b[3]);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16_16816(o[m][n], pf[m][0], b[0], b[1]);
+          mma_bf16_16816(o[m][n], pf[m][1], b[2], b[3]);
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[st]);
+  }
+  // ---- row sums, output ----
+  asm volatile("bar.sync 1, 256;" ::: "memory");
+  const bool split = p.num_splits > 1;
+  if (srow < Cfg::kRows) {
+    const unsigned act = __activemask();
+#pragma unroll
+    for (int x = 1; x < 8; x <<= 1) l_run += __shfl_xor_sync(act, l_run, x);
+    if (sub == 0) {
+      sA[srow] = split ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
+      if (split && srow < heads) {
+        const size_t pr = (row0 + srow) * p.num_splits + blockIdx.z;
+        p.part_ml[2 * pr] = m_run * 0.6931471805599453f;
+        p.part_ml[2 * pr + 1] = l_run;
+      }
+    }
+  }
+  asm volatile("bar.sync 1, 256;" ::: "memory");
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int hrow = 0; hrow < 2; ++hrow) {
+      const int row = m * 16 + hrow * 8 + g;
+      if (row >= heads) continue;
+      const float f = sA[row];
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const int col = warp * (R / 8) + n * 8 + 2 * t;
+        if (col >= p.rank) continue;
+        const float x = o[m][n][2 * hrow] * f, y = o[m][n][2 * hrow + 1] * f;
+        if (split)
+          *reinterpret_cast<float2*>(p.part_o + ((row0 + row) * p.num_splits + blockIdx.z) * p.rank + col) = make_float2(x, y);
+        else
+          *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldq + col) = pack_bf16(x, y);
+      }
+    }
+  if (*abort_flag != 0) {
+    // a wait ran out: give copies that may still be in flight a bounded time to land
+    const uint64_t t0 = global_timer_ns();
+    while (global_timer_ns() - t0 < 200000ull) { __nanosleep(1000); }
+  }
+}
+
+template <int R, int MT, int ST>
+static int launch_ld(const LatParams& p, cudaStream_t stream) {
+  using Cfg = LdCfg<R, MT, ST>;
+  CUtensorMap q_map, c_map;
+  int rc = make_tmap_bf16_2d(&q_map, p.q, static_cast<uint64_t>(p.rows) * p.heads, p.rank, p.ldq, Cfg::kRows, 64);
+  if (rc != 0) return rc;
+  rc = make_tmap_bf16_2d(&c_map, p.pool, static_cast<uint64_t>(p.num_pages) * kLatPage, p.rank, p.ldp, kLatPage, 64);
+  if (rc != 0) return rc;
+  static bool attr_set = false;
+  if (!attr_set) {
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<R, MT, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    attr_set = true;
+  }
+  const dim3 grid(p.rows, (p.heads + Cfg::kRows - 1) / Cfg::kRows, p.num_splits);
+  latent_decode_kernel<R, MT, ST><<<grid, kLdThreads, Cfg::kSmemBytes, stream>>>(q_map, c_map, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int MT>
+static int dispatch_ld(const LatParams& p, cudaStream_t stream) {
+  if (p.rank <= 64) return launch_ld<64, MT, 4>(p, stream);
+  if (p.rank <= 128) return launch_ld<128, MT, 4>(p, stream);
+  if (p.rank <= 256) return launch_ld<256, MT, 4>(p, stream);
+  return launch_ld<512, MT, 2>(p, stream);
+}
+
+int launch_latent_decode(const LatParams& p, cudaStream_t stream) {
+  return p.heads <= 16 ? dispatch_ld<1>(p, stream) : dispatch_ld<2>(p, stream);
+}
+
+}  // namespace ogb

@@ -449,6 +449,7 @@ class LLMEngine:
         target = 2 * (ops.num_sms() if self.device.type == "cuda" else 148)
         if getattr(self.model, "split_by_window", False) and self.cfg.model.sliding_window > 0:
             max_ctx = min(max_ctx, self.cfg.model.sliding_window)
+            target //= 2                 # one CTA per SM, and a split costs fp32 partials of the latent's width
         if ctas >= target or max_ctx < 256:
             return 1
         s = 1

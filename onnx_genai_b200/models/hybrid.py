@@ -311,7 +311,8 @@ class HybridModel:
         self.h_last = self.h_last_buf[:, :hid]
         self.logits_buf = z(max_seqs, pad8(cfg.vocab) if dev.type == "cuda" else cfg.vocab)
         self.logits = self.logits_buf[:, : cfg.vocab]
-        self.hkv = max((-(-m.heads // 4) for m in lat), default=1)      # CTAs per decode row: what the engine fills the device with
+        per_cta = 32 if dt == torch.bfloat16 else 4                     # heads a decode CTA takes
+        self.hkv = max((-(-m.heads // per_cta) for m in lat), default=1)      # CTAs per decode row: what the engine fills the device with
         self.decode_splits, self._split_capacity = 1, 1
         self.part_o = self.part_ml = None
         self.state = None
