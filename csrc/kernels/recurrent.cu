@@ -2,19 +2,22 @@
 //
 //   f = low + (1 - low) sigmoid(z + bias)      S <- diag(f) S + (1 - f) v^T      o = S^T silu(q)
 //
-// One CTA owns 32 value columns of one head of one sequence and walks the sequence's rows of the step, decode rows and
-// prefill chunks alike.  A warp owns 4 columns; its 8 lane groups own every eighth quad of state rows, so a thread keeps
-// D / 8 fp32 state values of one column in registers, the state is stored with the row index contiguous ([slot][head][column]
-// [row]) and moves as coalesced 16-byte vectors, and a token costs two fused multiply-adds per state value plus a
-// three-step lane reduction.  Gates and activations of the next tokens are fetched while the current ones run.
-// All arithmetic is fp32.  The per-head norm and the cast follow in head_rmsnorm_kernel.
+// One CTA walks the rows of one (head, sequence) -- decode rows and prefill chunks alike -- with the state in registers: a warp
+// owns 16 value columns (8 when the state is 256 rows high), its 16 lane pairs own every sixteenth quad of state rows, so a
+// thread holds a block of rows x columns and three 16-byte shared-memory reads (gate, key, query of four rows) serve all
+// its columns.  The arithmetic is packed fp32 (two rows per instruction); a row's outputs are summed over the lanes by a
+// halving exchange.  Gates and activations of the next tokens are fetched while the current ones run.  The state is stored
+// with the row index contiguous ([slot][head][column][row]) and moves as 16-byte vectors.  All arithmetic is fp32.
+//
+// Long prompts with few (head, sequence) pairs are cut into segments that run side by side: every segment first runs from a
+// zero state (MODE kLocal) and leaves its state and the product of its gates, hgrn2_chain_kernel turns those into the state
+// at each segment's start, and the second pass (MODE kFull) produces the outputs from there.
+//
+// The per-head norm and the cast follow in head_rmsnorm_kernel.
 #include "hybrid.cuh"
 #include "ogb_kernels.h"
 
 namespace ogb {
-
-constexpr int kRecThreads = 256;
-constexpr int kRecCols = 32;       // value columns per CTA
 
 struct RecParams {
   const float* qfv;       // [rows, ld]: q (heads * D) | z (heads * D) | v (heads * V)
@@ -22,128 +25,244 @@ struct RecParams {
   const float* low;       // [heads * D] lower bound of the gate
   float* state;           // [slots, heads, V, DP]
   float* out;             // [rows, ldo] raw head outputs (heads * V)
-  int ld, ldo, heads, D, V;
+  float* seg_state;       // [segments, heads, V, DP] (segmented runs)
+  float* seg_gate;        // [segments, heads, DP]
+  int ld, ldo, heads, D, V, num_prefill, seg_len;   // seg_len 0: not segmented
   StepRows sr;
   int* status;
 };
 
-template <int DP>          // key channels, padded to 64, 128 or 256
-__global__ void __launch_bounds__(kRecThreads) hgrn2_kernel(RecParams p) {
-  constexpr int kRecTok = DP == 256 ? 8 : 16;    // tokens staged at a time
-  constexpr int RPT = DP / 8;                    // state rows per thread
-  constexpr int QPT = RPT / 4;                   // quads of rows
-  constexpr int LPT = kRecTok * DP / kRecThreads;  // staged q (and z) values per thread
-  __shared__ __align__(16) float sq[kRecTok][DP];
-  __shared__ __align__(16) float sf[kRecTok][DP];
-  __shared__ __align__(16) float sk[kRecTok][DP];
-  __shared__ float sv[kRecTok][kRecCols];
-  __shared__ float so[kRecTok][kRecCols];
-  const int head = blockIdx.y, entry = blockIdx.z, col0 = blockIdx.x * kRecCols;
+enum RecMode : int { kFull = 0, kLocal = 1 };
+
+OGB_DEVICE float2 f2_fma(float2 a, float2 b, float2 c) {
+  unsigned long long r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;"
+      : "=l"(r)
+      : "l"(*reinterpret_cast<unsigned long long*>(&a)), "l"(*reinterpret_cast<unsigned long long*>(&b)), "l"(*reinterpret_cast<unsigned long long*>(&c)));
+  return *reinterpret_cast<float2*>(&r);
+}
+OGB_DEVICE float2 f2_mul(float2 a, float2 b) {
+  unsigned long long r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(*reinterpret_cast<unsigned long long*>(&a)), "l"(*reinterpret_cast<unsigned long long*>(&b)));
+  return *reinterpret_cast<float2*>(&r);
+}
+
+// Rows of work item z: a decode row, or a (segment of a) prefill chunk.
+struct RecItem {
+  int entry, base, n, first, seg;        // first: tokens of the chunk before this segment; seg: global segment index
+  bool last;                             // the item ends its chunk
+};
+OGB_DEVICE bool rec_item(const RecParams& p, int z, RecItem& it) {
   const StepRows& sr = p.sr;
-  int base, n;
-  if (entry < sr.num_decode) {
-    base = entry; n = 1;
-  } else {
-    const int s = entry - sr.num_decode;
-    base = sr.num_decode + sr.cu_q[s];
-    n = sr.cu_q[s + 1] - sr.cu_q[s];
+  it.seg = -1; it.first = 0; it.last = true;
+  if (z < sr.num_decode) {
+    it.entry = z; it.base = z; it.n = 1;
+    return true;
   }
-  const int ctx = sr.ctx_len[entry];
-  const int slot = sr.state_slot[entry];
-  if (n <= 0 || ctx <= 0 || slot < 0) return;    // padding row
+  z -= sr.num_decode;
+  for (int s = 0, before = 0; s < p.num_prefill; ++s) {
+    const int len = sr.cu_q[s + 1] - sr.cu_q[s];
+    const int segs = p.seg_len > 0 ? (len + p.seg_len - 1) / p.seg_len : 1;
+    if (z < before + segs) {
+      it.entry = sr.num_decode + s;
+      it.seg = z;
+      it.first = p.seg_len > 0 ? (z - before) * p.seg_len : 0;
+      it.n = p.seg_len > 0 ? min(p.seg_len, len - it.first) : len;
+      it.last = z - before == segs - 1;
+      it.base = sr.num_decode + sr.cu_q[s] + it.first;
+      return it.n > 0;
+    }
+    before += segs;
+  }
+  return false;
+}
+
+template <int DP, int CPT, int MODE>
+__global__ void __launch_bounds__(256) hgrn2_kernel(RecParams p) {
+  constexpr int QPT = DP / 64;                   // quads of state rows per thread
+  constexpr int kTok = DP == 256 ? 8 : 16;       // tokens staged at a time
+  constexpr int kMaxCols = 8 * 2 * CPT;          // columns of a CTA of eight warps
+  __shared__ __align__(16) float sq[MODE == kFull ? kTok : 1][DP];
+  __shared__ __align__(16) float sf[kTok][DP];
+  __shared__ __align__(16) float sk[kTok][DP];
+  __shared__ __align__(16) float sv[kTok][kMaxCols];
+  __shared__ float so[MODE == kFull ? kTok : 1][kMaxCols];
+  const int threads = blockDim.x, ncols = threads / 32 * 2 * CPT;
+  const int head = blockIdx.y, col0 = blockIdx.x * ncols;
+  RecItem it;
+  if (!rec_item(p, blockIdx.z, it)) return;
+  if (MODE == kLocal && it.last) return;         // nothing follows this segment: its end state comes out of the second pass
+  const StepRows& sr = p.sr;
+  const int ctx = sr.ctx_len[it.entry];
+  const int slot = sr.state_slot[it.entry];
+  if (ctx <= 0 || slot < 0) return;              // padding row
   if (slot >= sr.num_slots) {
     if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
     return;
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int g = lane >> 2;                       // row group
-  const int lc = warp * 4 + (lane & 3);          // column within the CTA
-  const int col = col0 + lc;
-  const bool live = col < p.V;
-  float4* st = reinterpret_cast<float4*>(p.state + ((static_cast<size_t>(slot) * p.heads + head) * p.V + (live ? col : 0)) * DP);
-  float s[RPT];
-#pragma unroll
-  for (int i = 0; i < QPT; ++i) {
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (ctx > n && live) v = st[i * 8 + g];
-    s[4 * i] = v.x; s[4 * i + 1] = v.y; s[4 * i + 2] = v.z; s[4 * i + 3] = v.w;
+  const int g = lane & 15;                       // row group
+  const int lc = (warp * 2 + (lane >> 4)) * CPT; // first column within the CTA
+  const size_t head_state = static_cast<size_t>(p.V) * DP;
+  float* own = p.state + (static_cast<size_t>(slot) * p.heads + head) * head_state;
+  float* segs = it.seg >= 0 && p.seg_len > 0 ? p.seg_state + (static_cast<size_t>(it.seg) * p.heads + head) * head_state : nullptr;
+  // where the run starts: zero, the sequence's slot, or the chained state of the segment before
+  const float* init = nullptr;
+  if (MODE == kFull) {
+    if (it.first > 0) init = segs - static_cast<size_t>(p.heads) * head_state;
+    else if (ctx - (sr.num_decode > it.entry ? 1 : sr.cu_q[it.entry - sr.num_decode + 1] - sr.cu_q[it.entry - sr.num_decode]) > 0) init = own;
   }
+  float2 s[CPT][QPT][2];
+#pragma unroll
+  for (int c = 0; c < CPT; ++c)
+#pragma unroll
+    for (int i = 0; i < QPT; ++i) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (init != nullptr && col0 + lc + c < p.V) v = *reinterpret_cast<const float4*>(init + static_cast<size_t>(col0 + lc + c) * DP + (i * 16 + g) * 4);
+      s[c][i][0] = make_float2(v.x, v.y);
+      s[c][i][1] = make_float2(v.z, v.w);
+    }
+  float gate = 1.f;                              // MODE kLocal: product of the gates of row threadIdx.x
   const int HD = p.heads * p.D;
-  constexpr int VPT = kRecTok * kRecCols / kRecThreads;
-  float rq[LPT], rz[LPT], rv[VPT];
-  auto fetch = [&](int t0) {
-#pragma unroll
-    for (int e = 0; e < LPT; ++e) {
-      const int i = threadIdx.x + e * kRecThreads, t = t0 + i / DP, d = i % DP;
-      const bool in = t < n && d < p.D;
-      const float* row = p.qfv + static_cast<size_t>(base + t) * p.ld + head * p.D + d;
-      rq[e] = in ? row[0] : 0.f;
-      rz[e] = in ? row[HD] : 0.f;
-    }
-#pragma unroll
-    for (int e = 0; e < VPT; ++e) {
-      const int i = threadIdx.x + e * kRecThreads, t = t0 + i / kRecCols, c = col0 + i % kRecCols;
-      rv[e] = (t < n && c < p.V) ? p.qfv[static_cast<size_t>(base + t) * p.ld + 2 * HD + head * p.V + c] : 0.f;
-    }
-  };
-  fetch(0);
-  for (int t0 = 0; t0 < n; t0 += kRecTok) {
+  for (int t0 = 0; t0 < it.n; t0 += kTok) {
+    const int nt = min(kTok, it.n - t0);
     __syncthreads();
-#pragma unroll
-    for (int e = 0; e < LPT; ++e) {
-      const int i = threadIdx.x + e * kRecThreads, t = i / DP, d = i % DP;
+    for (int i = threadIdx.x; i < kTok * DP; i += threads) {
+      const int t = i / DP, d = i % DP;
       float q = 0.f, f = 0.f, k = 0.f;
-      if (t0 + t < n && d < p.D) {
+      if (t < nt && d < p.D) {
+        const float* row = p.qfv + static_cast<size_t>(it.base + t0 + t) * p.ld + head * p.D + d;
         const float low = p.low[head * p.D + d];
-        const float z = rz[e] + p.bias[head * p.D + d];
+        const float z = row[HD] + p.bias[head * p.D + d];
         const float ez = expf(-fabsf(z));        // sigmoid of both signs from one exponential that cannot overflow
-        const float small = ez / (1.f + ez), big = 1.f / (1.f + ez);
-        f = fmaf(1.f - low, z >= 0.f ? big : small, low);
-        k = (1.f - low) * (z >= 0.f ? small : big);   // 1 - f without the cancellation
-        q = rq[e] / (1.f + expf(-rq[e]));
+        const float r = 1.f / (1.f + ez), small = ez * r;
+        f = fmaf(1.f - low, z >= 0.f ? r : small, low);
+        k = (1.f - low) * (z >= 0.f ? small : r);     // 1 - f without the cancellation
+        if (MODE == kFull) { const float x = row[0]; q = x / (1.f + expf(-x)); }
       }
-      sq[t][d] = q; sf[t][d] = f; sk[t][d] = k;
+      if (MODE == kFull) sq[t][d] = q;
+      sf[t][d] = f; sk[t][d] = k;
     }
-#pragma unroll
-    for (int e = 0; e < VPT; ++e) {
-      const int i = threadIdx.x + e * kRecThreads;
-      sv[i / kRecCols][i % kRecCols] = rv[e];
+    for (int i = threadIdx.x; i < kTok * ncols; i += threads) {
+      const int t = i / ncols, c = i % ncols;
+      sv[t][c] = t < nt && col0 + c < p.V ? p.qfv[static_cast<size_t>(it.base + t0 + t) * p.ld + 2 * HD + head * p.V + col0 + c] : 0.f;
     }
     __syncthreads();
-    if (t0 + kRecTok < n) fetch(t0 + kRecTok);
-    const int nt = min(kRecTok, n - t0);
+    if (MODE == kLocal && blockIdx.x == 0) {
+      if (static_cast<int>(threadIdx.x) < DP)
+        for (int t = 0; t < nt; ++t) gate *= sf[t][threadIdx.x];
+    }
     for (int t = 0; t < nt; ++t) {
-      const float v = sv[t][lc];
-      float o = 0.f;
+      float2 f[QPT][2], k[QPT][2], q[QPT][2], o[CPT];
 #pragma unroll
       for (int i = 0; i < QPT; ++i) {
-        const float4 f4 = *reinterpret_cast<const float4*>(&sf[t][(i * 8 + g) * 4]);
-        const float4 k4 = *reinterpret_cast<const float4*>(&sk[t][(i * 8 + g) * 4]);
-        const float4 q4 = *reinterpret_cast<const float4*>(&sq[t][(i * 8 + g) * 4]);
-        s[4 * i] = fmaf(f4.x, s[4 * i], k4.x * v);
-        s[4 * i + 1] = fmaf(f4.y, s[4 * i + 1], k4.y * v);
-        s[4 * i + 2] = fmaf(f4.z, s[4 * i + 2], k4.z * v);
-        s[4 * i + 3] = fmaf(f4.w, s[4 * i + 3], k4.w * v);
-        o = fmaf(q4.x, s[4 * i], o);
-        o = fmaf(q4.y, s[4 * i + 1], o);
-        o = fmaf(q4.z, s[4 * i + 2], o);
-        o = fmaf(q4.w, s[4 * i + 3], o);
+        const float4 a = *reinterpret_cast<const float4*>(&sf[t][(i * 16 + g) * 4]);
+        const float4 b = *reinterpret_cast<const float4*>(&sk[t][(i * 16 + g) * 4]);
+        f[i][0] = make_float2(a.x, a.y); f[i][1] = make_float2(a.z, a.w);
+        k[i][0] = make_float2(b.x, b.y); k[i][1] = make_float2(b.z, b.w);
+        if (MODE == kFull) {
+          const float4 c = *reinterpret_cast<const float4*>(&sq[t][(i * 16 + g) * 4]);
+          q[i][0] = make_float2(c.x, c.y); q[i][1] = make_float2(c.z, c.w);
+        }
       }
-      o += __shfl_xor_sync(0xffffffffu, o, 4);
-      o += __shfl_xor_sync(0xffffffffu, o, 8);
-      o += __shfl_xor_sync(0xffffffffu, o, 16);
-      if (g == 0) so[t][lc] = o;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < nt * kRecCols; i += kRecThreads) {
-      const int t = i / kRecCols, c = col0 + i % kRecCols;
-      if (c < p.V) p.out[static_cast<size_t>(base + t0 + t) * p.ldo + head * p.V + c] = so[t][i % kRecCols];
-    }
-  }
-  if (live) {
 #pragma unroll
-    for (int i = 0; i < QPT; ++i) st[i * 8 + g] = make_float4(s[4 * i], s[4 * i + 1], s[4 * i + 2], s[4 * i + 3]);
+      for (int c4 = 0; c4 < CPT / 4; ++c4) {
+        const float4 v4 = *reinterpret_cast<const float4*>(&sv[t][lc + 4 * c4]);
+        const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) {
+          const int c = 4 * c4 + cc;
+          const float2 v = make_float2(vv[cc], vv[cc]);
+          o[c] = make_float2(0.f, 0.f);
+#pragma unroll
+          for (int i = 0; i < QPT; ++i)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              s[c][i][h] = f2_fma(f[i][h], s[c][i][h], f2_mul(k[i][h], v));
+              if (MODE == kFull) o[c] = f2_fma(q[i][h], s[c][i][h], o[c]);
+            }
+        }
+      }
+      if (MODE == kFull) {
+        // sum over the 16 row groups: halve the columns a lane carries while there are several, then plain steps
+        float r[CPT];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) r[c] = o[c].x + o[c].y;
+        int mine = 0;
+#pragma unroll
+        for (int w = CPT / 2, bit = 1; w >= 1; w >>= 1, bit <<= 1) {
+          const bool up = (g & bit) != 0;
+#pragma unroll
+          for (int c = 0; c < w; ++c) {
+            const float send = up ? r[c] : r[c + w], keep = up ? r[c + w] : r[c];
+            r[c] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+          }
+          mine += up ? w : 0;
+        }
+#pragma unroll
+        for (int bit = CPT; bit < 16; bit <<= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], bit);
+        if (g < CPT) so[t][lc + mine] = r[0];
+      }
+    }
+    if (MODE == kFull) {
+      __syncthreads();
+      for (int i = threadIdx.x; i < nt * ncols; i += threads) {
+        const int t = i / ncols, c = i % ncols;
+        if (col0 + c < p.V) p.out[static_cast<size_t>(it.base + t0 + t) * p.ldo + head * p.V + col0 + c] = so[t][c];
+      }
+    }
   }
+  float* dst = MODE == kLocal ? segs : (it.last ? own : nullptr);
+  if (dst != nullptr) {
+#pragma unroll
+    for (int c = 0; c < CPT; ++c)
+#pragma unroll
+      for (int i = 0; i < QPT; ++i)
+        if (col0 + lc + c < p.V)
+          *reinterpret_cast<float4*>(dst + static_cast<size_t>(col0 + lc + c) * DP + (i * 16 + g) * 4) =
+              make_float4(s[c][i][0].x, s[c][i][0].y, s[c][i][1].x, s[c][i][1].y);
+  }
+  if (MODE == kLocal && blockIdx.x == 0 && static_cast<int>(threadIdx.x) < DP)
+    p.seg_gate[(static_cast<size_t>(it.seg) * p.heads + head) * DP + threadIdx.x] = gate;
+}
+
+// Turns every segment's local end state into the true state at its end: S_i <- gates_i * S_(i-1) + local_i, starting from the
+// sequence's state.  One thread per four state values of a (head, chunk).
+__global__ void __launch_bounds__(256) hgrn2_chain_kernel(RecParams p, int DP) {
+  const int head = blockIdx.y, s = blockIdx.z;
+  const StepRows& sr = p.sr;
+  const int len = sr.cu_q[s + 1] - sr.cu_q[s], segs = (len + p.seg_len - 1) / p.seg_len;
+  const int entry = sr.num_decode + s, slot = sr.state_slot[entry], ctx = sr.ctx_len[entry];
+  if (segs < 2 || slot < 0 || slot >= sr.num_slots || ctx <= 0) return;
+  int seg0 = 0;
+  for (int i = 0; i < s; ++i) seg0 += (sr.cu_q[i + 1] - sr.cu_q[i] + p.seg_len - 1) / p.seg_len;
+  const int quads = p.V * DP / 4, i = blockIdx.x * 256 + threadIdx.x;
+  if (i >= quads) return;
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (ctx > len) a = reinterpret_cast<const float4*>(p.state + (static_cast<size_t>(slot) * p.heads + head) * p.V * DP)[i];
+  for (int j = 0; j < segs - 1; ++j) {
+    const size_t at = static_cast<size_t>(seg0 + j) * p.heads + head;
+    float4* u = reinterpret_cast<float4*>(p.seg_state + at * p.V * DP) + i;
+    const float4 g = reinterpret_cast<const float4*>(p.seg_gate + at * DP)[i % (DP / 4)];
+    const float4 l = *u;
+    a = make_float4(fmaf(g.x, a.x, l.x), fmaf(g.y, a.y, l.y), fmaf(g.z, a.z, l.z), fmaf(g.w, a.w, l.w));
+    *u = a;
+  }
+}
+
+template <int DP, int CPT>
+static int launch_hgrn2(const RecParams& p, int items, cudaStream_t stream) {
+  int warps = (p.V + 2 * CPT - 1) / (2 * CPT);
+  if (warps > 8) warps = 8;
+  const int need = (DP + 31) / 32;               // the gate products of a segment take one thread per state row
+  if (p.seg_len > 0 && warps < need) warps = need;
+  const dim3 grid((p.V + warps * 2 * CPT - 1) / (warps * 2 * CPT), p.heads, items);
+  if (p.seg_len > 0) {
+    hgrn2_kernel<DP, CPT, kLocal><<<grid, warps * 32, 0, stream>>>(p);
+    hgrn2_chain_kernel<<<dim3((p.V * DP / 4 + 255) / 256, p.heads, p.num_prefill), 256, 0, stream>>>(p, DP);
+  }
+  hgrn2_kernel<DP, CPT, kFull><<<grid, warps * 32, 0, stream>>>(p);
+  return static_cast<int>(cudaGetLastError());
 }
 
 }  // namespace ogb
@@ -153,18 +272,20 @@ using namespace ogb;
 // Row width of the stored state for D key channels (0: not supported).
 extern "C" int ogb_hgrn2_state_rows(int D) { return D <= 0 ? 0 : D <= 64 ? 64 : D <= 128 ? 128 : D <= 256 ? 256 : 0; }
 
+// seg_len > 0: prefill chunks run as segments of that many tokens; num_segments counts them over all chunks, and seg_state
+// [num_segments, heads, V, rows] / seg_gate [num_segments, heads, rows] are scratch.
 extern "C" int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D,
                          int V, const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots,
-                         int* status, void* stream) {
-  const int entries = num_decode + num_prefill;
-  if (entries <= 0 || heads <= 0 || V <= 0) return 0;
+                         int seg_len, int num_segments, float* seg_state, float* seg_gate, int* status, void* stream) {
+  if (num_decode + num_prefill <= 0 || heads <= 0 || V <= 0) return 0;
   const int dp = ogb_hgrn2_state_rows(D);
   if (dp == 0) return -2;
-  RecParams p{qfv, bias, low, state, out, ld, ldo, heads, D, V, StepRows{ctx_len, state_slot, cu_q, nullptr, nullptr, num_decode, 0, num_slots}, status};
-  const dim3 grid((V + kRecCols - 1) / kRecCols, heads, entries);
+  if (seg_len > 0 && (seg_state == nullptr || seg_gate == nullptr || num_segments < num_prefill)) return -3;
+  RecParams p{qfv, bias, low, state, out, seg_state, seg_gate, ld, ldo, heads, D, V, num_prefill, seg_len > 0 ? seg_len : 0,
+              StepRows{ctx_len, state_slot, cu_q, nullptr, nullptr, num_decode, 0, num_slots}, status};
+  const int items = num_decode + (seg_len > 0 ? num_segments : num_prefill);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dp == 64) hgrn2_kernel<64><<<grid, kRecThreads, 0, s>>>(p);
-  else if (dp == 128) hgrn2_kernel<128><<<grid, kRecThreads, 0, s>>>(p);
-  else hgrn2_kernel<256><<<grid, kRecThreads, 0, s>>>(p);
-  return static_cast<int>(cudaGetLastError());
+  if (dp == 64) return launch_hgrn2<64, 8>(p, items, s);
+  if (dp == 128) return launch_hgrn2<128, 8>(p, items, s);
+  return launch_hgrn2<256, 4>(p, items, s);
 }

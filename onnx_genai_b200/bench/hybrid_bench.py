@@ -127,7 +127,8 @@ def _plan(chunks, max_pages, num_pages):
     pos = [p for a, n in chunks for p in range(a, a + n)]
     return StepInputs(len(pos), nd, len(chunks) - nd, len(ts), 0, token_ids=t([0] * len(pos)), positions=t(pos), slots=t(slots),
                       ctx_len=t([a + n for a, n in chunks]), page_table=t(table), cu_q=t(cu), tile_seq=t(ts or [0]), tile_q0=t(tq or [0]),
-                      logit_rows=t([0]), state_slot=t(list(range(len(chunks)))))
+                      logit_rows=t([0]), state_slot=t(list(range(len(chunks)))), prefill_ctx=np.array([a + n for a, n in chunks[nd:]], dtype=np.int32),
+                      prefill_len=np.array([n for _, n in chunks[nd:]], dtype=np.int32))
 
 
 def seen_pairs(chunks, window):

@@ -358,7 +358,7 @@ class HybridModel:
         qfv = self._rows(self.qfv, t, pad8(n))
         hops.linear(h, w.qfv, qfv[:, :n], f32_out=True)
         raw = hops.hgrn2(qfv, w.gate_bias, w.gate_low, self.state.layers[li]["recurrent"], self._rows(self.rec_o, t, m.heads * m.vdim), m.heads,
-                         m.dim, m.vdim, si)
+                         m.dim, m.vdim, si, scratch=lambda name, shape: self._scratch(name, shape, torch.float32))
         width = m.heads * m.vdim
         attn = self._rows(self.attn, t, pad8(width))
         if pad8(width) != width:
@@ -386,8 +386,8 @@ class HybridModel:
             hops.linear_batched(oc, w.uv, attn[:rows], hp, rp, vp)
         if pages:
             hops.latent_prefill_expanded(qc, attn, pool, w.kv, si, hp, m.dim, m.scale, m.window, pages,
-                                         self._scratch("dense", (pages * ops.PAGE, rp), m), self._scratch("kv", (pages, hp, 2, ops.PAGE, m.dim), m),
-                                         self._scratch("table", (si.num_prefill_seqs, si.page_table.shape[1]), m, torch.int32))
+                                         self._scratch("dense", (pages * ops.PAGE, rp)), self._scratch("kv", (pages, hp, 2, ops.PAGE, m.dim)),
+                                         self._scratch("table", (si.num_prefill_seqs, si.page_table.shape[1]), torch.int32))
         hops.linear(attn, w.o, y)
 
     EXPAND_BYTES = 1 << 30             # most memory the expanded keys and values of a step may take
@@ -406,7 +406,7 @@ class HybridModel:
         expanded = pairs * 4 * m.dim + pages * ops.PAGE * 4 * m.dim * m.rank
         return pages if direct > expanded and pages * ops.PAGE * m.heads * m.dim * 4 <= self.EXPAND_BYTES else 0
 
-    def _scratch(self, name, shape, m, dtype=None):
+    def _scratch(self, name, shape, dtype=None):
         """Step scratch that grows to the largest step seen (prompt steps only: never inside a captured graph)."""
         n = 1
         for d in shape:

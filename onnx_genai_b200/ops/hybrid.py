@@ -23,7 +23,7 @@ _native.register("ogb_latent_gather", [P, P, P, P, I, I, L, I, I, I, P, P, P, P]
 _native.register("ogb_latent_set_tc", [I])
 _native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
 _native.register("ogb_hgrn2_state_rows", [I])
-_native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 3 + [P, P])
+_native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P] * 4)
 _native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, I, P])
 _native.register("ogb_act_mul_packed", [P, P, I, I, I, I, I, P])
 
@@ -228,16 +228,38 @@ def latent_prefill_expanded(q, out, pool, kv_w, si, heads, d, scale, window, pag
                   d, scale, window)
 
 
+def segment_length(si, heads: int, vdim: int) -> int:
+    """Tokens per segment of a step's prompts, 0 to run every chunk in one piece: chunks are cut while the (head, chunk) pairs
+    leave the device half empty (a segmented run costs two thirds of a pass more)."""
+    if si.num_prefill_seqs == 0 or si.prefill_len is None:
+        return 0
+    longest, per = int(si.prefill_len.max()), heads * max(1, -(-vdim // 128))
+    if per * si.num_prefill_seqs >= 148 or longest < 256:
+        return 0
+    seg = 1 << (longest - 1).bit_length()
+    while seg > 128 and per * int((-(-si.prefill_len // seg)).sum()) < 296:
+        seg //= 2
+    return seg if seg < longest else 0
+
+
 @_timed("hgrn2")
-def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si):
+def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si, segment=None, scratch=None):
     """Advance the recurrence over the step's rows: qfv [T, ld] fp32 (query, gate and value projections), state
-    [slots, heads, vdim, state_rows(dim)] fp32 in place, raw head outputs to out [T, ld] fp32."""
+    [slots, heads, vdim, state_rows(dim)] fp32 in place, raw head outputs to out [T, ld] fp32.  ``segment``: tokens per segment of
+    the prompts (None: chosen, 0: whole); ``scratch(name, shape)`` provides fp32 scratch for segmented runs."""
     if not qfv.is_cuda:
         reference.hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si)
         return out
+    seg = segment_length(si, heads, vdim) if segment is None else segment
+    nseg, us, ug = 0, None, None
+    if seg > 0 and si.num_prefill_seqs > 0:
+        nseg, rows = int((-(-si.prefill_len // seg)).sum()), state.shape[3]
+        make = scratch or (lambda name, shape: torch.empty(*shape, dtype=torch.float32, device=qfv.device))
+        us, ug = make("seg_state", (nseg, heads, vdim, rows)), make("seg_gate", (nseg, heads, rows))
     rc = _native.load().ogb_hgrn2(qfv.data_ptr(), bias.data_ptr(), low.data_ptr(), state.data_ptr(), out.data_ptr(), qfv.stride(0),
                                   out.stride(0), heads, dim, vdim, si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(),
-                                  si.num_decode, si.num_prefill_seqs, state.shape[0], status_word().data_ptr(), _stream())
+                                  si.num_decode, si.num_prefill_seqs, state.shape[0], seg if nseg else 0, nseg, _ptr(us), _ptr(ug),
+                                  status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_hgrn2")
     launch_counts["hgrn2"] += 1
     return out

@@ -97,7 +97,8 @@ def step_of(chunks, device, page_seed=0):
     t = lambda x: torch.tensor(x, dtype=torch.int32, device=device)
     si = StepInputs(len(pos), nd, len(order) - nd, len(ts), 0, token_ids=t([0] * len(pos)), positions=t(pos), slots=t(kv),
                     ctx_len=t([a + n for a, n in order]), page_table=perm.to(device), cu_q=t(cu), tile_seq=t(ts or [0]), tile_q0=t(tq or [0]),
-                    logit_rows=t([0]), state_slot=slots.to(device))
+                    logit_rows=t([0]), state_slot=slots.to(device), prefill_ctx=np.array([a + n for a, n in order[nd:]], dtype=np.int32),
+                    prefill_len=np.array([n for _, n in order[nd:]], dtype=np.int32))
     return si, order, len(order) * mp
 
 
@@ -141,8 +142,9 @@ def test_hyper_step_with_norm_and_shift(device, streams, width):
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("heads,dim,vdim", [(2, 48, 64), (3, 20, 36), (1, 64, 10), (2, 128, 130), (1, 200, 33), (4, 100, 32)])
-def test_hgrn2_recurrence(device, heads, dim, vdim):
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 48, 64), (3, 20, 36), (1, 64, 10), (2, 128, 130), (1, 200, 33), (4, 100, 32), (2, 256, 140)])
+@pytest.mark.parametrize("segment", [0, 32])
+def test_hgrn2_recurrence(device, heads, dim, vdim, segment):
     g = torch.Generator().manual_seed(dim)
     si, order, _ = step_of(CHUNKS, device)
     t, hd = si.num_tokens, heads * dim
@@ -154,7 +156,7 @@ def test_hgrn2_recurrence(device, heads, dim, vdim):
     start = torch.randn(len(order), heads, vdim, rows, generator=g)
     start[..., dim:] = 0
     state, out = start.to(device).clone(), torch.zeros(t, heads * vdim, device=device)
-    H.hgrn2(qfv.to(device), bias.to(device), low.to(device), state, out, heads, dim, vdim, si)
+    H.hgrn2(qfv.to(device), bias.to(device), low.to(device), state, out, heads, dim, vdim, si, segment=segment)
     base, slots = 0, si.state_slot.cpu()
     for e, (a, n) in enumerate(order):
         z = qfv[base:base + n].double()
