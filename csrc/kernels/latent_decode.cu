@@ -6,7 +6,7 @@
 //
 //   warp 8    : TMA producer, 64 tokens (4 pages) x R values per stage, 128-byte swizzled column chunks
 //   warps 0-7 : S = Q' C^T split four ways over the latent's columns and two ways over the tokens (a warp keeps its slice of
-//               Q' in registers for the whole call), partial scores summed through shared memory, softmax by eight threads a
+//               Q' in registers where they suffice), partial scores summed through shared memory, softmax by eight threads a
 //               row, then O += P C with a warp owning R / 8 output columns
 //
 // Keys split `num_splits` ways leave fp32 partials for latent_combine_kernel.  Waits are bounded; page ids are checked.
@@ -124,12 +124,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   const int ks = warp >> 1, kh = warp & 1;               // column slice and token half of the score product
   const uint32_t aK = smem_u32(sK), aQ = smem_u32(sQ), aP = smem_u32(sP);
   bool ok = fa_wait(q_full, 0, abort_flag);
-  uint32_t qf[MT][KS][4];
+  constexpr bool kQRegs = MT * KS <= 8;                  // else the registers are worth more as loads in flight
+  uint32_t qf[MT][kQRegs ? KS : 1][4];
+  auto load_q = [&](int m, int k, uint32_t (&f)[4]) {
+    ldsm_x4(aQ + ld_off(Cfg::kRows, m * 16 + (lane & 15), ks * (R / 4) + k * 16 + (lane >> 4) * 8), f[0], f[1], f[2], f[3]);
+  };
+  if constexpr (kQRegs) {
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int k = 0; k < KS; ++k)
-      ldsm_x4(aQ + ld_off(Cfg::kRows, m * 16 + (lane & 15), ks * (R / 4) + k * 16 + (lane >> 4) * 8), qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3]);
+      for (int k = 0; k < KS; ++k) load_q(m, k, qf[m][k]);
+  }
   float o[MT][NT][4] = {};
   const int srow = threadIdx.x / 8, sub = threadIdx.x & 7;      // softmax: eight threads a row (rows past 16 * MT idle)
   float m_run = -INFINITY, l_run = 0.f;
@@ -143,14 +148,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
     float s[MT][4][4] = {};
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
+      if constexpr (!kQRegs) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m) load_q(m, k, qf[m][0]);
+      }
 #pragma unroll
       for (int n2 = 0; n2 < 2; ++n2) {
         uint32_t b[4];
         ldsm_x4(kb + ld_off(kLdKeys, kh * 32 + n2 * 16 + (lane >> 4) * 8 + (lane & 7), ks * (R / 4) + k * 16 + ((lane >> 3) & 1) * 8), b[0], b[1], b[2], b[3]);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          mma_bf16_16816(s[m][2 * n2], qf[m][k], b[0], b[1]);
-          mma_bf16_16816(s[m][2 * n2 + 1], qf[m][k], b[2], b[3]);
+          mma_bf16_16816(s[m][2 * n2], qf[m][kQRegs ? k : 0], b[0], b[1]);
+          mma_bf16_16816(s[m][2 * n2 + 1], qf[m][kQRegs ? k : 0], b[2], b[3]);
         }
       }
     }

@@ -34,17 +34,22 @@ struct RecParams {
 
 enum RecMode : int { kFull = 0, kLocal = 1 };
 
-OGB_DEVICE float2 f2_fma(float2 a, float2 b, float2 c) {
-  unsigned long long r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;"
-      : "=l"(r)
-      : "l"(*reinterpret_cast<unsigned long long*>(&a)), "l"(*reinterpret_cast<unsigned long long*>(&b)), "l"(*reinterpret_cast<unsigned long long*>(&c)));
-  return *reinterpret_cast<float2*>(&r);
+// two fp32 values in one 64-bit register
+typedef unsigned long long f32x2;
+OGB_DEVICE f32x2 f2_fma(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
 }
-OGB_DEVICE float2 f2_mul(float2 a, float2 b) {
-  unsigned long long r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(*reinterpret_cast<unsigned long long*>(&a)), "l"(*reinterpret_cast<unsigned long long*>(&b)));
-  return *reinterpret_cast<float2*>(&r);
+OGB_DEVICE f32x2 f2_mul(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+OGB_DEVICE float f2_sum(f32x2 a) {
+  float x, y;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
+  return x + y;
 }
 
 // Rows of work item z: a decode row, or a (segment of a) prefill chunk.
@@ -78,14 +83,14 @@ OGB_DEVICE bool rec_item(const RecParams& p, int z, RecItem& it) {
 }
 
 template <int DP, int CPT, int MODE>
-__global__ void __launch_bounds__(256) hgrn2_kernel(RecParams p) {
+__global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
   constexpr int QPT = DP / 64;                   // quads of state rows per thread
   constexpr int kTok = DP == 256 ? 8 : 16;       // tokens staged at a time
   constexpr int kMaxCols = 8 * 2 * CPT;          // columns of a CTA of eight warps
   __shared__ __align__(16) float sq[MODE == kFull ? kTok : 1][DP];
   __shared__ __align__(16) float sf[kTok][DP];
   __shared__ __align__(16) float sk[kTok][DP];
-  __shared__ __align__(16) float sv[kTok][kMaxCols];
+  __shared__ __align__(16) float2 sv[kTok][kMaxCols];      // every value twice: the packed operand of its column
   __shared__ float so[MODE == kFull ? kTok : 1][kMaxCols];
   const int threads = blockDim.x, ncols = threads / 32 * 2 * CPT;
   const int head = blockIdx.y, col0 = blockIdx.x * ncols;
@@ -112,15 +117,15 @@ __global__ void __launch_bounds__(256) hgrn2_kernel(RecParams p) {
     if (it.first > 0) init = segs - static_cast<size_t>(p.heads) * head_state;
     else if (ctx - (sr.num_decode > it.entry ? 1 : sr.cu_q[it.entry - sr.num_decode + 1] - sr.cu_q[it.entry - sr.num_decode]) > 0) init = own;
   }
-  float2 s[CPT][QPT][2];
+  f32x2 s[CPT][QPT][2];
 #pragma unroll
   for (int c = 0; c < CPT; ++c)
 #pragma unroll
     for (int i = 0; i < QPT; ++i) {
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (init != nullptr && col0 + lc + c < p.V) v = *reinterpret_cast<const float4*>(init + static_cast<size_t>(col0 + lc + c) * DP + (i * 16 + g) * 4);
-      s[c][i][0] = make_float2(v.x, v.y);
-      s[c][i][1] = make_float2(v.z, v.w);
+      ulonglong2 v = make_ulonglong2(0ull, 0ull);
+      if (init != nullptr && col0 + lc + c < p.V) v = *reinterpret_cast<const ulonglong2*>(init + static_cast<size_t>(col0 + lc + c) * DP + (i * 16 + g) * 4);
+      s[c][i][0] = v.x;
+      s[c][i][1] = v.y;
     }
   float gate = 1.f;                              // MODE kLocal: product of the gates of row threadIdx.x
   const int HD = p.heads * p.D;
@@ -134,63 +139,72 @@ __global__ void __launch_bounds__(256) hgrn2_kernel(RecParams p) {
         const float* row = p.qfv + static_cast<size_t>(it.base + t0 + t) * p.ld + head * p.D + d;
         const float low = p.low[head * p.D + d];
         const float z = row[HD] + p.bias[head * p.D + d];
-        const float ez = expf(-fabsf(z));        // sigmoid of both signs from one exponential that cannot overflow
-        const float r = 1.f / (1.f + ez), small = ez * r;
+        const float ez = __expf(-fabsf(z));      // sigmoid of both signs from one exponential that cannot overflow
+        const float r = __fdividef(1.f, 1.f + ez), small = ez * r;
         f = fmaf(1.f - low, z >= 0.f ? r : small, low);
         k = (1.f - low) * (z >= 0.f ? small : r);     // 1 - f without the cancellation
-        if (MODE == kFull) { const float x = row[0]; q = x / (1.f + expf(-x)); }
+        if (MODE == kFull) { const float x = row[0]; q = __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
       }
       if (MODE == kFull) sq[t][d] = q;
       sf[t][d] = f; sk[t][d] = k;
     }
     for (int i = threadIdx.x; i < kTok * ncols; i += threads) {
       const int t = i / ncols, c = i % ncols;
-      sv[t][c] = t < nt && col0 + c < p.V ? p.qfv[static_cast<size_t>(it.base + t0 + t) * p.ld + 2 * HD + head * p.V + col0 + c] : 0.f;
+      const float v = t < nt && col0 + c < p.V ? p.qfv[static_cast<size_t>(it.base + t0 + t) * p.ld + 2 * HD + head * p.V + col0 + c] : 0.f;
+      sv[t][c] = make_float2(v, v);
     }
     __syncthreads();
     if (MODE == kLocal && blockIdx.x == 0) {
       if (static_cast<int>(threadIdx.x) < DP)
         for (int t = 0; t < nt; ++t) gate *= sf[t][threadIdx.x];
     }
-    for (int t = 0; t < nt; ++t) {
-      float2 f[QPT][2], k[QPT][2], q[QPT][2], o[CPT];
+    // two tokens at a time, so that their lane sums share the steps of one exchange
+    for (int t = 0; t < nt; t += 2) {
+      f32x2 o[2][CPT];
 #pragma unroll
-      for (int i = 0; i < QPT; ++i) {
-        const float4 a = *reinterpret_cast<const float4*>(&sf[t][(i * 16 + g) * 4]);
-        const float4 b = *reinterpret_cast<const float4*>(&sk[t][(i * 16 + g) * 4]);
-        f[i][0] = make_float2(a.x, a.y); f[i][1] = make_float2(a.z, a.w);
-        k[i][0] = make_float2(b.x, b.y); k[i][1] = make_float2(b.z, b.w);
-        if (MODE == kFull) {
-          const float4 c = *reinterpret_cast<const float4*>(&sq[t][(i * 16 + g) * 4]);
-          q[i][0] = make_float2(c.x, c.y); q[i][1] = make_float2(c.z, c.w);
+      for (int u = 0; u < 2; ++u) {
+        if (u == 1 && t + 1 >= nt) {
+#pragma unroll
+          for (int c = 0; c < CPT; ++c) o[1][c] = 0ull;
+          break;
         }
-      }
+        f32x2 f[QPT][2], k[QPT][2], q[QPT][2];
 #pragma unroll
-      for (int c4 = 0; c4 < CPT / 4; ++c4) {
-        const float4 v4 = *reinterpret_cast<const float4*>(&sv[t][lc + 4 * c4]);
-        const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
+        for (int i = 0; i < QPT; ++i) {
+          const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(&sf[t + u][(i * 16 + g) * 4]);
+          const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(&sk[t + u][(i * 16 + g) * 4]);
+          f[i][0] = a.x; f[i][1] = a.y;
+          k[i][0] = b.x; k[i][1] = b.y;
+          if (MODE == kFull) {
+            const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(&sq[t + u][(i * 16 + g) * 4]);
+            q[i][0] = c.x; q[i][1] = c.y;
+          }
+        }
 #pragma unroll
-        for (int cc = 0; cc < 4; ++cc) {
-          const int c = 4 * c4 + cc;
-          const float2 v = make_float2(vv[cc], vv[cc]);
-          o[c] = make_float2(0.f, 0.f);
+        for (int c2 = 0; c2 < CPT / 2; ++c2) {
+          const ulonglong2 v2 = *reinterpret_cast<const ulonglong2*>(&sv[t + u][lc + 2 * c2]);
 #pragma unroll
-          for (int i = 0; i < QPT; ++i)
+          for (int cc = 0; cc < 2; ++cc) {
+            const int c = 2 * c2 + cc;
+            const f32x2 v = cc == 0 ? v2.x : v2.y;
 #pragma unroll
-            for (int h = 0; h < 2; ++h) {
-              s[c][i][h] = f2_fma(f[i][h], s[c][i][h], f2_mul(k[i][h], v));
-              if (MODE == kFull) o[c] = f2_fma(q[i][h], s[c][i][h], o[c]);
-            }
+            for (int i = 0; i < QPT; ++i)
+#pragma unroll
+              for (int h = 0; h < 2; ++h) {
+                s[c][i][h] = f2_fma(f[i][h], s[c][i][h], f2_mul(k[i][h], v));
+                if (MODE == kFull) o[u][c] = (i | h) == 0 ? f2_mul(q[i][h], s[c][i][h]) : f2_fma(q[i][h], s[c][i][h], o[u][c]);
+              }
+          }
         }
       }
       if (MODE == kFull) {
-        // sum over the 16 row groups: halve the columns a lane carries while there are several, then plain steps
-        float r[CPT];
+        // sums over the 16 row groups: lanes halve the (token, column) values they carry, then plain steps
+        float r[2 * CPT];
 #pragma unroll
-        for (int c = 0; c < CPT; ++c) r[c] = o[c].x + o[c].y;
+        for (int c = 0; c < CPT; ++c) { r[c] = f2_sum(o[0][c]); r[CPT + c] = f2_sum(o[1][c]); }
         int mine = 0;
 #pragma unroll
-        for (int w = CPT / 2, bit = 1; w >= 1; w >>= 1, bit <<= 1) {
+        for (int w = CPT, bit = 1; w >= 1; w >>= 1, bit <<= 1) {
           const bool up = (g & bit) != 0;
 #pragma unroll
           for (int c = 0; c < w; ++c) {
@@ -200,8 +214,8 @@ __global__ void __launch_bounds__(256) hgrn2_kernel(RecParams p) {
           mine += up ? w : 0;
         }
 #pragma unroll
-        for (int bit = CPT; bit < 16; bit <<= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], bit);
-        if (g < CPT) so[t][lc + mine] = r[0];
+        for (int bit = 2 * CPT; bit < 16; bit <<= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], bit);
+        if (g < 2 * CPT) so[t + mine / CPT][lc + mine % CPT] = r[0];
       }
     }
     if (MODE == kFull) {
@@ -219,8 +233,7 @@ __global__ void __launch_bounds__(256) hgrn2_kernel(RecParams p) {
 #pragma unroll
       for (int i = 0; i < QPT; ++i)
         if (col0 + lc + c < p.V)
-          *reinterpret_cast<float4*>(dst + static_cast<size_t>(col0 + lc + c) * DP + (i * 16 + g) * 4) =
-              make_float4(s[c][i][0].x, s[c][i][0].y, s[c][i][1].x, s[c][i][1].y);
+          *reinterpret_cast<ulonglong2*>(dst + static_cast<size_t>(col0 + lc + c) * DP + (i * 16 + g) * 4) = make_ulonglong2(s[c][i][0], s[c][i][1]);
   }
   if (MODE == kLocal && blockIdx.x == 0 && static_cast<int>(threadIdx.x) < DP)
     p.seg_gate[(static_cast<size_t>(it.seg) * p.heads + head) * DP + threadIdx.x] = gate;
