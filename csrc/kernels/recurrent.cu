@@ -82,16 +82,38 @@ OGB_DEVICE bool rec_item(const RecParams& p, int z, RecItem& it) {
   return false;
 }
 
+template <int DP, int CPT>
+struct RecCfg {
+  static constexpr int kTok = DP == 256 ? 8 : 16;       // tokens staged at a time
+  static constexpr int kMaxCols = 8 * 2 * CPT;          // columns of a CTA of eight warps
+  static constexpr int kSmemBytes = 4 * (kTok * (3 * DP + 3 * kMaxCols) + 2 * DP + 2 * kTok * (2 * DP + kMaxCols));
+};
+
+template <int BYTES>
+OGB_DEVICE void cp_async(void* dst, const void* src) {
+  if constexpr (BYTES == 16)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  else
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+
 template <int DP, int CPT, int MODE>
 __global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
   constexpr int QPT = DP / 64;                   // quads of state rows per thread
-  constexpr int kTok = DP == 256 ? 8 : 16;       // tokens staged at a time
-  constexpr int kMaxCols = 8 * 2 * CPT;          // columns of a CTA of eight warps
-  __shared__ __align__(16) float sq[MODE == kFull ? kTok : 1][DP];
-  __shared__ __align__(16) float sf[kTok][DP];
-  __shared__ __align__(16) float sk[kTok][DP];
-  __shared__ __align__(16) float2 sv[kTok][kMaxCols];      // every value twice: the packed operand of its column
-  __shared__ float so[MODE == kFull ? kTok : 1][kMaxCols];
+  constexpr int kTok = RecCfg<DP, CPT>::kTok, kMaxCols = RecCfg<DP, CPT>::kMaxCols;
+  extern __shared__ __align__(16) uint8_t rec_smem[];
+  typedef float Row[DP];
+  Row* sq = reinterpret_cast<Row*>(rec_smem);                                    // [kTok][DP]: query, gate, key
+  Row* sf = sq + kTok;
+  Row* sk = sf + kTok;
+  typedef float2 VRow[kMaxCols];
+  VRow* sv = reinterpret_cast<VRow*>(sk + kTok);                                 // every value twice: the packed operand of its column
+  typedef float ORow[kMaxCols];
+  ORow* so = reinterpret_cast<ORow*>(sv + kTok);
+  float* slow = reinterpret_cast<float*>(so + kTok);                             // [DP] lower bound, bias
+  float* sbias = slow + DP;
+  float* raw = sbias + DP;                                                       // [2][kTok][2 * DP + kMaxCols]: the rows as they come
+  constexpr int kRaw = 2 * DP + kMaxCols;
   const int threads = blockDim.x, ncols = threads / 32 * 2 * CPT;
   const int head = blockIdx.y, col0 = blockIdx.x * ncols;
   RecItem it;
@@ -129,28 +151,47 @@ __global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
     }
   float gate = 1.f;                              // MODE kLocal: product of the gates of row threadIdx.x
   const int HD = p.heads * p.D;
-  for (int t0 = 0; t0 < it.n; t0 += kTok) {
+  for (int d = threadIdx.x; d < p.D; d += threads) { slow[d] = p.low[head * p.D + d]; sbias[d] = p.bias[head * p.D + d]; }
+  // rows of the next tokens on their way while the current ones run: q, z, v side by side
+  const bool vec = ((p.D | p.V | p.ld) & 3) == 0;
+  auto fetch = [&](int t0, int buf) {
+    const int nt = min(kTok, it.n - t0), nv = min(ncols, p.V - col0);
+    const int step = vec ? 4 : 1, per = (2 * p.D + nv + step - 1) / step;
+    for (int i = threadIdx.x; i < nt * per; i += threads) {
+      const int t = i / per, e = (i - t * per) * step;
+      const float* src = p.qfv + static_cast<size_t>(it.base + t0 + t) * p.ld;
+      float* dst = raw + (buf * kTok + t) * kRaw;
+      if (e < p.D) { src += head * p.D + e; dst += e; }
+      else if (e < 2 * p.D) { src += HD + head * p.D + e - p.D; dst += DP + e - p.D; }
+      else { src += 2 * HD + head * p.V + col0 + e - 2 * p.D; dst += 2 * DP + e - 2 * p.D; }
+      if (vec) cp_async<16>(dst, src); else cp_async<4>(dst, src);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(0, 0);
+  for (int t0 = 0, buf = 0; t0 < it.n; t0 += kTok, buf ^= 1) {
     const int nt = min(kTok, it.n - t0);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    for (int i = threadIdx.x; i < kTok * DP; i += threads) {
+    if (t0 + kTok < it.n) fetch(t0 + kTok, buf ^ 1);
+    for (int i = threadIdx.x; i < nt * DP; i += threads) {
       const int t = i / DP, d = i % DP;
+      const float* row = raw + (buf * kTok + t) * kRaw;
       float q = 0.f, f = 0.f, k = 0.f;
-      if (t < nt && d < p.D) {
-        const float* row = p.qfv + static_cast<size_t>(it.base + t0 + t) * p.ld + head * p.D + d;
-        const float low = p.low[head * p.D + d];
-        const float z = row[HD] + p.bias[head * p.D + d];
+      if (d < p.D) {
+        const float low = slow[d], z = row[DP + d] + sbias[d];
         const float ez = __expf(-fabsf(z));      // sigmoid of both signs from one exponential that cannot overflow
         const float r = __fdividef(1.f, 1.f + ez), small = ez * r;
         f = fmaf(1.f - low, z >= 0.f ? r : small, low);
         k = (1.f - low) * (z >= 0.f ? small : r);     // 1 - f without the cancellation
-        if (MODE == kFull) { const float x = row[0]; q = __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
+        if (MODE == kFull) { const float x = row[d]; q = __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
       }
       if (MODE == kFull) sq[t][d] = q;
       sf[t][d] = f; sk[t][d] = k;
     }
-    for (int i = threadIdx.x; i < kTok * ncols; i += threads) {
-      const int t = i / ncols, c = i % ncols;
-      const float v = t < nt && col0 + c < p.V ? p.qfv[static_cast<size_t>(it.base + t0 + t) * p.ld + 2 * HD + head * p.V + col0 + c] : 0.f;
+    for (int i = threadIdx.x; i < nt * ncols; i += threads) {
+      const int t = i / ncols, c = i - t * ncols;
+      const float v = col0 + c < p.V ? raw[(buf * kTok + t) * kRaw + 2 * DP + c] : 0.f;
       sv[t][c] = make_float2(v, v);
     }
     __syncthreads();
@@ -270,11 +311,18 @@ static int launch_hgrn2(const RecParams& p, int items, cudaStream_t stream) {
   const int need = (DP + 31) / 32;               // the gate products of a segment take one thread per state row
   if (p.seg_len > 0 && warps < need) warps = need;
   const dim3 grid((p.V + warps * 2 * CPT - 1) / (warps * 2 * CPT), p.heads, items);
+  constexpr int smem = RecCfg<DP, CPT>::kSmemBytes;
+  static bool attr_set = false;
+  if (!attr_set) {
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(hgrn2_kernel<DP, CPT, kLocal>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(hgrn2_kernel<DP, CPT, kFull>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    attr_set = true;
+  }
   if (p.seg_len > 0) {
-    hgrn2_kernel<DP, CPT, kLocal><<<grid, warps * 32, 0, stream>>>(p);
+    hgrn2_kernel<DP, CPT, kLocal><<<grid, warps * 32, smem, stream>>>(p);
     hgrn2_chain_kernel<<<dim3((p.V * DP / 4 + 255) / 256, p.heads, p.num_prefill), 256, 0, stream>>>(p, DP);
   }
-  hgrn2_kernel<DP, CPT, kFull><<<grid, warps * 32, 0, stream>>>(p);
+  hgrn2_kernel<DP, CPT, kFull><<<grid, warps * 32, smem, stream>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 
