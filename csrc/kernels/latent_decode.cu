@@ -4,10 +4,10 @@
 // their shared-memory traffic on rows that do not exist.  Here the products run on mma.sync m16n8k16 with 16 or 32 rows and
 // the kernel is laid out around the byte stream instead:
 //
-//   warp 8    : TMA producer, 64 tokens (4 pages) x R values per stage, 128-byte swizzled column chunks
-//   warps 0-7 : S = Q' C^T split four ways over the latent's columns and two ways over the tokens (a warp keeps its slice of
-//               Q' in registers where they suffice), partial scores summed through shared memory, softmax by eight threads a
-//               row, then O += P C with a warp owning R / 8 output columns
+//   last warp    : TMA producer, 64 tokens (4 pages) x R values per stage, 128-byte swizzled column chunks
+//   8 or 16 warps: S = Q' C^T split four ways over the latent's columns and two or four ways over the tokens (a warp keeps its
+//                  slice of Q' in registers where they suffice), partial scores summed through shared memory, softmax with all
+//                  threads, then O += P C with every warp owning its share of the output columns
 //
 // Keys split `num_splits` ways leave fp32 partials for latent_combine_kernel.  Waits are bounded; page ids are checked.
 #include "attention_common.cuh"
@@ -18,11 +18,9 @@
 namespace ogb {
 
 constexpr int kLdKeys = 64;
-constexpr int kLdWarps = 8;
-constexpr int kLdThreads = (kLdWarps + 1) * 32;
 constexpr int kLdPitch = 72;             // floats per row of partial scores: conflict-free 8-byte stores
 
-template <int R, int MT, int ST>
+template <int R, int MT, int ST, int NW>
 struct LdCfg {
   static constexpr int kRows = 16 * MT;
   static constexpr int kChunks = R / 64;
@@ -39,12 +37,14 @@ OGB_DEVICE uint32_t ld_off(int rows, int row, int col) {
   return static_cast<uint32_t>(((col >> 6) * rows + row) * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4));
 }
 
-template <int R, int MT, int ST>
-__global__ void __launch_bounds__(kLdThreads, 1)
+template <int R, int MT, int ST, int NW>
+__global__ void __launch_bounds__((NW + 1) * 32, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap c_map, const LatParams p) {
-  using Cfg = LdCfg<R, MT, ST>;
+  using Cfg = LdCfg<R, MT, ST, NW>;
   constexpr int KS = R / 64;             // k-steps of a warp's column slice (R / 4 columns)
-  constexpr int NT = R / 64;             // 8-column output tiles of a warp
+  constexpr int NT = R / (8 * NW);       // 8-column output tiles of a warp
+  constexpr int KN = 4 / (NW / 4);       // 16-token score tiles of a warp: NW / 4 warps share a column slice
+  constexpr int TPR = NW * 32 / (16 * MT), KPT = kLdKeys / TPR;   // softmax: threads a row, tokens a thread
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sK = smem;
@@ -80,14 +80,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < ST; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], kLdWarps); }
+    for (int i = 0; i < ST; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], NW); }
     mbar_init(q_full, 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
   __syncthreads();
 
-  if (warp == kLdWarps) {
+  if (warp == NW) {
     if (lane == 0) {
       mbar_expect_tx(q_full, Cfg::kQBytes);
       for (int h = 0; h < Cfg::kChunks; ++h) tma_load_2d(sQ + h * Cfg::kRows * 128, &q_map, q_full, h * 64, static_cast<int>(row0));
@@ -121,10 +121,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
 
   // ------------------------------ consumers ------------------------------
   const int g = lane >> 2, t = lane & 3;
-  const int ks = warp >> 1, kh = warp & 1;               // column slice and token half of the score product
+  const int ks = warp & 3, kh = warp >> 2;               // column slice and token group of the score product
   const uint32_t aK = smem_u32(sK), aQ = smem_u32(sQ), aP = smem_u32(sP);
   bool ok = fa_wait(q_full, 0, abort_flag);
-  constexpr bool kQRegs = MT * KS <= 8;                  // else the registers are worth more as loads in flight
+  constexpr bool kQRegs = MT * KS <= (NW == 16 ? 4 : 8);                  // else the registers are worth more as loads in flight
   uint32_t qf[MT][kQRegs ? KS : 1][4];
   auto load_q = [&](int m, int k, uint32_t (&f)[4]) {
     ldsm_x4(aQ + ld_off(Cfg::kRows, m * 16 + (lane & 15), ks * (R / 4) + k * 16 + (lane >> 4) * 8), f[0], f[1], f[2], f[3]);
@@ -136,7 +136,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       for (int k = 0; k < KS; ++k) load_q(m, k, qf[m][k]);
   }
   float o[MT][NT][4] = {};
-  const int srow = threadIdx.x / 8, sub = threadIdx.x & 7;      // softmax: eight threads a row (rows past 16 * MT idle)
+  const int srow = threadIdx.x / TPR, sub = threadIdx.x % TPR;
   float m_run = -INFINITY, l_run = 0.f;
   const float scale = p.scale * 1.4426950408889634f;
   for (int it = 0; it < nblk; ++it) {
@@ -145,7 +145,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
     if (!ok && lane == 0) { atomicOr(p.status, kStatusWaitTimeout); *abort_flag = 1; }
     const uint32_t kb = aK + st * Cfg::kStage;
     // ---- partial scores ----
-    float s[MT][4][4] = {};
+    float s[MT][2 * KN][4] = {};
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
       if constexpr (!kQRegs) {
@@ -153,9 +153,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
         for (int m = 0; m < MT; ++m) load_q(m, k, qf[m][0]);
       }
 #pragma unroll
-      for (int n2 = 0; n2 < 2; ++n2) {
+      for (int n2 = 0; n2 < KN; ++n2) {
         uint32_t b[4];
-        ldsm_x4(kb + ld_off(kLdKeys, kh * 32 + n2 * 16 + (lane >> 4) * 8 + (lane & 7), ks * (R / 4) + k * 16 + ((lane >> 3) & 1) * 8), b[0], b[1], b[2], b[3]);
+        ldsm_x4(kb + ld_off(kLdKeys, (kh * KN + n2) * 16 + (lane >> 4) * 8 + (lane & 7), ks * (R / 4) + k * 16 + ((lane >> 3) & 1) * 8), b[0], b[1], b[2], b[3]);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma_bf16_16816(s[m][2 * n2], qf[m][kQRegs ? k : 0], b[0], b[1]);
@@ -166,48 +166,55 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        float* d = sS + (ks * Cfg::kRows + m * 16 + g) * kLdPitch + kh * 32 + n * 8 + 2 * t;
+      for (int n = 0; n < 2 * KN; ++n) {
+        float* d = sS + (ks * Cfg::kRows + m * 16 + g) * kLdPitch + kh * KN * 16 + n * 8 + 2 * t;
         *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
         *reinterpret_cast<float2*>(d + 8 * kLdPitch) = make_float2(s[m][n][2], s[m][n][3]);
       }
-    asm volatile("bar.sync 1, 256;" ::: "memory");
+    asm volatile("bar.sync 1, %0;" ::"n"(NW * 32) : "memory");
     // ---- softmax ----
-    if (srow < Cfg::kRows) {
-      float v[8];
+    {
+      float v[KPT];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        float4 a = *reinterpret_cast<const float4*>(sS + srow * kLdPitch + sub * 8 + 4 * h);
+      for (int j = 0; j < KPT; ++j) v[j] = 0.f;
 #pragma unroll
-        for (int x = 1; x < 4; ++x) {
-          const float4 b = *reinterpret_cast<const float4*>(sS + (x * Cfg::kRows + srow) * kLdPitch + sub * 8 + 4 * h);
-          a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
+      for (int x = 0; x < 4; ++x) {
+        const float* src = sS + (x * Cfg::kRows + srow) * kLdPitch + sub * KPT;
+#pragma unroll
+        for (int j = 0; j < KPT; j += 2) {
+          const float2 b = *reinterpret_cast<const float2*>(src + j);
+          v[j] += b.x; v[j + 1] += b.y;
         }
-        v[4 * h] = a.x; v[4 * h + 1] = a.y; v[4 * h + 2] = a.z; v[4 * h + 3] = a.w;
       }
-      const int key0 = (b0 + it) * kLdKeys + sub * 8;
+      const int key0 = (b0 + it) * kLdKeys + sub * KPT;
       float mx = -INFINITY;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
+      for (int j = 0; j < KPT; ++j) {
         v[j] = key0 + j >= lo && key0 + j < ctx ? v[j] * scale : -INFINITY;
         mx = fmaxf(mx, v[j]);
       }
-      const unsigned act = __activemask();
 #pragma unroll
-      for (int x = 1; x < 8; x <<= 1) mx = fmaxf(mx, __shfl_xor_sync(act, mx, x));
+      for (int x = 1; x < TPR; x <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
       const float m_new = fmaxf(m_run, mx);
       const float alpha = m_run == -INFINITY ? 0.f : exp2f(m_run - m_new);
       const float neg = m_new == -INFINITY ? 0.f : -m_new;
       float sum = 0.f;
+      uint32_t pk[KPT / 2];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) { v[j] = exp2f(v[j] + neg); sum += v[j]; }
+      for (int j = 0; j < KPT; j += 2) {
+        const float e0 = exp2f(v[j] + neg), e1 = exp2f(v[j + 1] + neg);
+        sum += e0 + e1;
+        pk[j / 2] = pack_bf16(e0, e1);
+      }
       l_run = l_run * alpha + sum;                       // this thread's keys; the row's sum is formed at the end
       m_run = m_new;
-      *reinterpret_cast<uint4*>(sP + ld_off(Cfg::kRows, srow, sub * 8)) =
-          make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+      uint8_t* pd = sP + ld_off(Cfg::kRows, srow, sub * KPT) + (sub * KPT & 7) * 2;
+      if constexpr (KPT == 8) *reinterpret_cast<uint4*>(pd) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+      else if constexpr (KPT == 4) *reinterpret_cast<uint2*>(pd) = make_uint2(pk[0], pk[1]);
+      else *reinterpret_cast<uint32_t*>(pd) = pk[0];
       if (sub == 0) sA[srow] = alpha;
     }
-    asm volatile("bar.sync 1, 256;" ::: "memory");
+    asm volatile("bar.sync 1, %0;" ::"n"(NW * 32) : "memory");
     // ---- O += P C ----
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
@@ -228,7 +235,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         uint32_t b[4];
-        ldsm_x4_t(kb + ld_off(kLdKeys, kk * 32 + lane, warp * (R / 8) + n * 8), b[0], b[1], b[2], b[3]);
+        ldsm_x4_t(kb + ld_off(kLdKeys, kk * 32 + lane, warp * (R / NW) + n * 8), b[0], b[1], b[2], b[3]);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma_bf16_16816(o[m][n], pf[m][0], b[0], b[1]);
@@ -240,12 +247,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
     if (lane == 0) mbar_arrive(&empty[st]);
   }
   // ---- row sums, output ----
-  asm volatile("bar.sync 1, 256;" ::: "memory");
+  asm volatile("bar.sync 1, %0;" ::"n"(NW * 32) : "memory");
   const bool split = p.num_splits > 1;
-  if (srow < Cfg::kRows) {
-    const unsigned act = __activemask();
+  {
 #pragma unroll
-    for (int x = 1; x < 8; x <<= 1) l_run += __shfl_xor_sync(act, l_run, x);
+    for (int x = 1; x < TPR; x <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
     if (sub == 0) {
       sA[srow] = split ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
       if (split && srow < heads) {
@@ -255,7 +261,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       }
     }
   }
-  asm volatile("bar.sync 1, 256;" ::: "memory");
+  asm volatile("bar.sync 1, %0;" ::"n"(NW * 32) : "memory");
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -265,7 +271,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       const float f = sA[row];
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
-        const int col = warp * (R / 8) + n * 8 + 2 * t;
+        const int col = warp * (R / NW) + n * 8 + 2 * t;
         if (col >= p.rank) continue;
         const float x = o[m][n][2 * hrow] * f, y = o[m][n][2 * hrow + 1] * f;
         if (split)
@@ -281,9 +287,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   }
 }
 
-template <int R, int MT, int ST>
+template <int R, int MT, int ST, int NW>
 static int launch_ld(const LatParams& p, cudaStream_t stream) {
-  using Cfg = LdCfg<R, MT, ST>;
+  using Cfg = LdCfg<R, MT, ST, NW>;
   CUtensorMap q_map, c_map;
   int rc = make_tmap_bf16_2d(&q_map, p.q, static_cast<uint64_t>(p.rows) * p.heads, p.rank, p.ldq, Cfg::kRows, 64);
   if (rc != 0) return rc;
@@ -291,20 +297,20 @@ static int launch_ld(const LatParams& p, cudaStream_t stream) {
   if (rc != 0) return rc;
   static bool attr_set = false;
   if (!attr_set) {
-    OGB_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<R, MT, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<R, MT, ST, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
     attr_set = true;
   }
   const dim3 grid(p.rows, (p.heads + Cfg::kRows - 1) / Cfg::kRows, p.num_splits);
-  latent_decode_kernel<R, MT, ST><<<grid, kLdThreads, Cfg::kSmemBytes, stream>>>(q_map, c_map, p);
+  latent_decode_kernel<R, MT, ST, NW><<<grid, (NW + 1) * 32, Cfg::kSmemBytes, stream>>>(q_map, c_map, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <int MT>
 static int dispatch_ld(const LatParams& p, cudaStream_t stream) {
-  if (p.rank <= 64) return launch_ld<64, MT, 4>(p, stream);
-  if (p.rank <= 128) return launch_ld<128, MT, 4>(p, stream);
-  if (p.rank <= 256) return launch_ld<256, MT, 4>(p, stream);
-  return launch_ld<512, MT, 2>(p, stream);
+  if (p.rank <= 64) return launch_ld<64, MT, 4, 8>(p, stream);
+  if (p.rank <= 128) return launch_ld<128, MT, 4, 8>(p, stream);
+  if (p.rank <= 256) return launch_ld<256, MT, 4, 16>(p, stream);
+  return launch_ld<512, MT, 2, 16>(p, stream);
 }
 
 int launch_latent_decode(const LatParams& p, cudaStream_t stream) {
