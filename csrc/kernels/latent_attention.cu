@@ -201,16 +201,19 @@ extern "C" int ogb_latent_set_tc(int on) {
 extern "C" int ogb_latent_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
                                     const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages,
                                     int num_tiles, int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml,
-                                    int elem, int* status, void* stream) {
+                                    int* counters, int elem, int* status, void* stream) {
   if (rows <= 0 || (cu_q != nullptr && num_tiles <= 0)) return 0;
   if (heads <= 0 || rank <= 0 || rank > ldq || rank > ldp) return -3;
   if (cu_q != nullptr) num_splits = 1;
   if (num_splits > 1 && (part_o == nullptr || part_ml == nullptr)) return -3;
   LatParams p{q, out, pool, page_table, ctx_len, cu_q, tile_seq, tile_q0, rows, heads, rank, ldq, ldp, max_pages, num_tiles, window,
-              num_splits < 1 ? 1 : num_splits, num_pages, scale, part_o, part_ml, status};
+              num_splits < 1 ? 1 : num_splits, num_pages, scale, part_o, part_ml, counters, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   int rc = -2;                                    // the tensor-core kernel declines what it cannot take
-  if (elem == kElemBF16 && use_tensor_cores()) rc = launch_latent_tc(p, s);
+  if (elem == kElemBF16 && use_tensor_cores()) {
+    rc = launch_latent_tc(p, s);
+    if (rc == 0 && counters != nullptr) return 0;
+  }
   if (rc == -2) rc = elem == kElemBF16 ? launch_warp<__nv_bfloat16>(p, s) : elem == kElemF32 ? launch_warp<float>(p, s) : -3;
   if (rc != 0 || p.num_splits == 1) return rc;
   const int blocks = (rows * heads + 3) / 4;

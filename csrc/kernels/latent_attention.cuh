@@ -19,12 +19,13 @@ struct LatParams {
   int64_t num_pages;
   float scale;
   float *part_o, *part_ml;
+  int* counters;          // zeroed words, one per (decode row, 16 heads): the last split of a row merges them (null: a second kernel does)
   int* status;
 };
 
 // Tensor-core launch; -2 when it does not take the call (rank above 512, alignment).
 int launch_latent_tc(const LatParams& p, cudaStream_t stream);
-// Decode rows (latent_decode.cu); launch_latent_tc hands them over.
+// Decode rows (latent_decode.cu); launch_latent_tc hands them over.  It merges split keys itself when it has counters.
 int launch_latent_decode(const LatParams& p, cudaStream_t stream);
 
 }  // namespace ogb

@@ -37,6 +37,43 @@ OGB_DEVICE uint32_t ld_off(int rows, int row, int col) {
   return static_cast<uint32_t>(((col >> 6) * rows + row) * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4));
 }
 
+// Called by the consumer threads of every split of a row once its partials are written: the last one to arrive merges them.
+template <int NW>
+OGB_DEVICE void ld_merge(const LatParams& p, int* counter, size_t row0, int heads, volatile int* flag) {
+  __threadfence();
+  asm volatile("bar.sync 1, %0;" ::"n"(NW * 32) : "memory");
+  if (threadIdx.x == 0) {
+    const int last = atomicAdd(counter, 1) == p.num_splits - 1;
+    if (last) *counter = 0;              // every split has arrived: ready for the next launch
+    *flag = last;
+  }
+  asm volatile("bar.sync 1, %0;" ::"n"(NW * 32) : "memory");
+  if (*flag == 0) return;
+  __threadfence();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int row = warp; row < heads; row += NW) {
+    const float* ml = p.part_ml + 2 * (row0 + row) * p.num_splits;
+    float m = -INFINITY, l = 0.f;
+    for (int s = 0; s < p.num_splits; ++s) m = fmaxf(m, __ldcg(ml + 2 * s));
+    for (int s = 0; s < p.num_splits; ++s) {
+      const float ms = __ldcg(ml + 2 * s);
+      if (ms != -INFINITY) l += __ldcg(ml + 2 * s + 1) * expf(ms - m);
+    }
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    for (int c = lane * 4; c < p.rank; c += 128) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int s = 0; s < p.num_splits; ++s) {
+        const float ms = __ldcg(ml + 2 * s);
+        if (ms == -INFINITY) continue;
+        const float w = expf(ms - m) * inv;
+        const float4 o = __ldcg(reinterpret_cast<const float4*>(p.part_o + ((row0 + row) * p.num_splits + s) * p.rank + c));
+        a.x = fmaf(w, o.x, a.x); a.y = fmaf(w, o.y, a.y); a.z = fmaf(w, o.z, a.z); a.w = fmaf(w, o.w, a.w);
+      }
+      *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldq + c) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
+    }
+  }
+}
+
 template <int R, int MT, int ST, int NW>
 __global__ void __launch_bounds__((NW + 1) * 32, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap c_map, const LatParams p) {
@@ -76,6 +113,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       p.part_ml[2 * pr] = -INFINITY;
       p.part_ml[2 * pr + 1] = 0.f;
     }
+    if (p.counters != nullptr && threadIdx.x < NW * 32)
+      ld_merge<NW>(p, p.counters + entry * gridDim.y + blockIdx.y, row0, heads, abort_flag);
     return;
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -280,7 +319,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
           *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldq + col) = pack_bf16(x, y);
       }
     }
-  if (*abort_flag != 0) {
+  const bool aborted = *abort_flag != 0;
+  if (split && p.counters != nullptr) ld_merge<NW>(p, p.counters + entry * gridDim.y + blockIdx.y, row0, heads, reinterpret_cast<volatile int*>(sS));
+  if (aborted) {
     // a wait ran out: give copies that may still be in flight a bounded time to land
     const uint64_t t0 = global_timer_ns();
     while (global_timer_ns() - t0 < 200000ull) { __nanosleep(1000); }

@@ -171,7 +171,7 @@ int ogb_latent_append(const void* c, int ldc, const float* w, float eps, const i
                       int64_t num_slots, int elem, int* status, void* stream);
 int ogb_latent_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
                          const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages, int num_tiles,
-                         int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml, int elem, int* status,
+                         int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml, int* counters, int elem, int* status,
                          void* stream);
 int ogb_latent_gather(const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, int entries, int max_pages, int64_t num_pages,
                       int window, int ldp, int blocks, void* out, int* scratch_table, int* status, void* stream);

@@ -152,7 +152,7 @@ def kernel_rows(size: str, timer, pk):
         rows.append({"kernel": name, "step": phase, "ms": round(ms, 4), "roofline_ms": round(bound, 4), "of_roofline": round(bound / ms, 3),
                      "TF/s": round(flops / ms / 1e9, 1) if flops else None, "GB/s": round(nbytes / ms / 1e6, 1) if nbytes else None})
 
-    for phase, chunks in (("prefill 4096", [(0, 4096)]), ("prefill 4x1024", [(0, 1024)] * 4), ("decode 64", [(2047, 1)] * 64)):
+    for phase, chunks in (("prefill 4096", [(0, 4096)]), ("prefill 4x1024", [(0, 1024)] * 4), ("decode 64", [(2047, 1)] * 64), ("decode 64, context 8192", [(8191, 1)] * 64)):
         t, nseq = sum(n for _, n in chunks), len(chunks)
         ctx = max(a + n for a, n in chunks)
         mp, npages = (ctx + 15) // 16, sum((a + n + 15) // 16 for a, n in chunks)
@@ -196,14 +196,24 @@ def kernel_rows(size: str, timer, pk):
         qa = rnd(t * heads, rank)
         oc = torch.empty_like(qa)
         pairs, keys = seen_pairs(chunks, window), sum(min(a + n, window + n) for a, n in chunks)
-        best = None
-        for splits in ((1,) if si.num_prefill_seqs else (1, 2, 4, 8)):
+        if si.num_prefill_seqs:
+            row("latent_attention (latents as keys)", phase, lambda: hops.latent_attention(qa, oc, pool, si, heads, rank, 0.1, window),
+                4 * pairs * heads * rank, keys * rank * 2 + 2 * t * heads * rank * 2)
+            if rank > d:      # what prompts of this shape run on
+                pages = hops.visible_pages(si, window)
+                dense, kvp = torch.empty(pages * 16, rank, dtype=bf, device="cuda"), torch.empty(pages, heads, 2, 16, d, dtype=bf, device="cuda")
+                table, kvw, qd = torch.zeros(nseq, mp, dtype=torch.int32, device="cuda"), rnd(heads * 2 * d, rank), rnd(t, heads * d)
+                od = torch.empty(t, heads * d, dtype=bf, device="cuda")
+                row("latent prompt, expanded K/V (3 kernels)", phase, lambda: hops.latent_prefill_expanded(qd, od, pool, kvw, si, heads, d, 0.1, window,
+                                                                                                          pages, dense, kvp, table),
+                    4 * pairs * heads * d + 2 * pages * 16 * rank * heads * 2 * d, 2 * pages * 16 * heads * 2 * d * 2)
+        else:
+            cnt = torch.zeros(4096, dtype=torch.int32, device="cuda")
+            splits = max(1, 148 * (2 if rank <= 128 else 1) // nseq // 2 * 2)
             po, pm = torch.empty(t * heads * splits * rank, device="cuda"), torch.empty(t * heads * splits * 2, device="cuda")
-            ms, _ = timer.time(lambda: hops.latent_attention(qa, oc, pool, si, heads, rank, 0.1, window, splits, po, pm))
-            best = (ms, splits) if best is None or ms < best[0] else best
-        po, pm = torch.empty(t * heads * best[1] * rank, device="cuda"), torch.empty(t * heads * best[1] * 2, device="cuda")
-        row(f"latent_attention (splits {best[1]})", phase, lambda: hops.latent_attention(qa, oc, pool, si, heads, rank, 0.1, window, best[1], po, pm),
-            4 * pairs * heads * rank, keys * rank * 2 + 2 * t * heads * rank * 2)
+            row(f"latent_attention (decode, {splits} splits)", phase, lambda: hops.latent_attention(qa, oc, pool, si, heads, rank, 0.1, window, splits, po,
+                                                                                                   pm, cnt),
+                4 * pairs * heads * rank, keys * rank * 2 + 2 * t * heads * rank * 2)
         # the dense model's attention and projections
         nq = (heads + 2 * kvh) * d
         qkv, out, kv = rnd(t, nq), torch.empty(t, heads * d, dtype=bf, device="cuda"), rnd(npages, kvh, 2, 16, d)

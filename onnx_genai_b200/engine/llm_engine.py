@@ -447,9 +447,15 @@ class LLMEngine:
             return self.cfg.decode_splits
         ctas = nd * self.model.hkv
         target = 2 * (ops.num_sms() if self.device.type == "cuda" else 148)
-        if getattr(self.model, "split_by_window", False) and self.cfg.model.sliding_window > 0:
-            max_ctx = min(max_ctx, self.cfg.model.sliding_window)
-            target //= 2                 # one CTA per SM, and a split costs fp32 partials of the latent's width
+        if getattr(self.model, "split_by_window", False):
+            # decode attends to a window at most, and a split leaves fp32 partials as wide as the latent: split only while every
+            # CTA still has a place of its own
+            if self.cfg.model.sliding_window > 0:
+                max_ctx = min(max_ctx, self.cfg.model.sliding_window)
+            s = 1
+            while 2 * s * ctas <= self.model.decode_ctas and max_ctx // (2 * s) >= 128:
+                s *= 2
+            return s
         if ctas >= target or max_ctx < 256:
             return 1
         s = 1

@@ -279,7 +279,7 @@ class HybridModel:
 
     native = None
     fused_comm = None
-    split_by_window = True             # decode work is bounded by the window: the engine splits keys by it
+    split_by_window = True             # how the engine picks decode splits (decode_ctas)
 
     def __init__(self, cfg: HybridConfig, weights: HybridWeights, device, max_tokens: int, max_seqs: int, tp: int = 1, rank: int = 0, comm=None):
         cfg.validate()
@@ -312,9 +312,12 @@ class HybridModel:
         self.logits_buf = z(max_seqs, pad8(cfg.vocab) if dev.type == "cuda" else cfg.vocab)
         self.logits = self.logits_buf[:, : cfg.vocab]
         per_cta = 32 if dt == torch.bfloat16 else 4                     # heads a decode CTA takes
-        self.hkv = max((-(-m.heads // per_cta) for m in lat), default=1)      # CTAs per decode row: what the engine fills the device with
+        self.hkv = max((-(-m.heads // per_cta) for m in lat), default=1)      # CTAs per decode row ...
+        per_sm = 8 if dt == torch.float32 else (2 if max((m.rank for m in lat), default=0) <= 128 else 1)
+        self.decode_ctas = per_sm * (ops.num_sms() if dev.type == "cuda" else 148)       # ... and the device's places for them
         self.decode_splits, self._split_capacity = 1, 1
         self.part_o = self.part_ml = None
+        self.counters = z(max_seqs * max((-(-m.heads // 16) for m in lat), default=1), dtype=torch.int32) if dev.type == "cuda" else None
         self.state = None
         self.scratch: dict = {}
         self.capture = None            # list: gets the summed streams [rows, hidden] after every layer (tests, debugging)
@@ -382,7 +385,7 @@ class HybridModel:
             qa, oc = self._rows(self.qa, rows, hp * rp), self._rows(self.oc, rows, hp * rp)
             hops.linear_batched(qc[:rows], w.uk, qa, hp, dp, rp)
             hops.latent_attention(qa.view(rows * hp, rp), oc.view(rows * hp, rp), pool, si, hp, rp, m.scale, m.window, self.decode_splits,
-                                  self.part_o, self.part_ml, decode_only=bool(pages))
+                                  self.part_o, self.part_ml, self.counters, decode_only=bool(pages))
             hops.linear_batched(oc, w.uv, attn[:rows], hp, rp, vp)
         if pages:
             hops.latent_prefill_expanded(qc, attn, pool, w.kv, si, hp, m.dim, m.scale, m.window, pages,

@@ -18,7 +18,7 @@ P, I, F, L = _native.P, _native.I, _native.F, _native.L
 _native.register("ogb_hyper_step", [P] * 13 + [I] * 6 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_embed_streams", [P, P, P, I, I, I, I, I, P, P])
 _native.register("ogb_latent_append", [P, I, P, F, P, P, I, I, I, L, I, P, P])
-_native.register("ogb_latent_attention", [P] * 8 + [I] * 7 + [L, I, F, I, P, P, I, P, P])
+_native.register("ogb_latent_attention", [P] * 8 + [I] * 7 + [L, I, F, I, P, P, P, I, P, P])
 _native.register("ogb_latent_gather", [P, P, P, P, I, I, L, I, I, I, P, P, P, P])
 _native.register("ogb_latent_set_tc", [I])
 _native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
@@ -174,8 +174,9 @@ def latent_append(c, w, eps, slots, pool, rank):
 
 
 @_timed("latent_attention")
-def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None, decode_only=False):
+def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None, counters=None, decode_only=False):
     """Rows (token, head) of q [T * heads, ld] over the latents of their sequences' pages; window <= 0: causal only.
+    ``counters``: zeroed int32 words, one per decode row and 16 heads, with which the last split of a row merges the splits.
     ``decode_only``: leave the prefill rows to :func:`latent_prefill_expanded`."""
     if not q.is_cuda:
         reference.latent_attention(q, out, pool, si, heads, rank, scale, window)
@@ -187,14 +188,14 @@ def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, par
     if nd > 0:
         rc = lib.ogb_latent_attention(q.data_ptr(), out.data_ptr(), pool.data_ptr(), si.page_table.data_ptr(), si.ctx_len.data_ptr(), 0, 0, 0,
                                       nd, heads, rank, q.stride(0), pool.shape[2], mp, 0, pages, int(window), float(scale), int(splits),
-                                      _ptr(part_o), _ptr(part_ml), elem, st, _stream())
+                                      _ptr(part_o), _ptr(part_ml), _ptr(counters), elem, st, _stream())
         _native.check(rc, "ogb_latent_attention")
         launch_counts["latent_decode"] += 1
     if npf > 0 and not decode_only:
         qp, op = q[nd * heads:], out[nd * heads:]
         rc = lib.ogb_latent_attention(qp.data_ptr(), op.data_ptr(), pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(),
                                       si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), t - nd, heads, rank, q.stride(0),
-                                      pool.shape[2], mp, si.num_tiles, pages, int(window), float(scale), 1, 0, 0, elem, st, _stream())
+                                      pool.shape[2], mp, si.num_tiles, pages, int(window), float(scale), 1, 0, 0, 0, elem, st, _stream())
         _native.check(rc, "ogb_latent_attention")
         launch_counts["latent_prefill"] += 1
     return out

@@ -179,7 +179,7 @@ def test_hgrn2_recurrence(device, heads, dim, vdim, segment):
     torch.testing.assert_close(normed.cpu(), want, atol=1e-5, rtol=1e-5)
 
 
-def latent_case(device, dtype, heads, rank, window, chunks, spike, splits=1):
+def latent_case(device, dtype, heads, rank, window, chunks, spike, splits=1, counters=None):
     """Latent attention over random pages; with ``spike`` one latent outshines all others at a chosen distance."""
     g = torch.Generator().manual_seed(heads * 1000 + rank)
     si, order, pages = step_of(chunks, device, page_seed=3)
@@ -205,7 +205,7 @@ def latent_case(device, dtype, heads, rank, window, chunks, spike, splits=1):
     out = torch.zeros(si.num_tokens * heads, ld, dtype=dtype, device=device)
     part_o = torch.empty(si.num_tokens * heads * splits * ld, device=device)
     part_ml = torch.empty(si.num_tokens * heads * splits * 2, device=device)
-    H.latent_attention(q.to(dtype).to(device), out, pool.to(dtype).to(device), si, heads, rank, 0.37, window, splits, part_o, part_ml)
+    H.latent_attention(q.to(dtype).to(device), out, pool.to(dtype).to(device), si, heads, rank, 0.37, window, splits, part_o, part_ml, counters)
     base = 0
     for e, (a, n) in enumerate(order):
         c = lat[e].double()
@@ -235,8 +235,11 @@ def test_latent_attention_window_edges(where, heads, rank, window):
 @pytest.mark.parametrize("heads,rank,window,splits", [(3, 56, 0, 4), (16, 128, 300, 3), (2, 512, 200, 8), (32, 256, 0, 5)])
 def test_latent_decode_with_split_keys(dtype, heads, rank, window, splits):
     chunks = [(7, 1), (0, 1), (400, 1), (255, 1), (15, 1), (16, 1), (299, 1), (300, 1)]
-    latent_case("cuda", dtype, heads, rank, window, chunks, None, splits)
-    latent_case("cuda", dtype, heads, rank, window, chunks, window if window else 380, splits)
+    counters = torch.zeros(len(chunks) * -(-heads // 16), dtype=torch.int32, device="cuda")
+    for c in (None, counters, counters):                  # merged by a second kernel, or by a row's last split (counters come back as zeros)
+        latent_case("cuda", dtype, heads, rank, window, chunks, None, splits, c)
+        latent_case("cuda", dtype, heads, rank, window, chunks, window if window else 380, splits, c)
+    assert (counters == 0).all()
 
 
 @pytest.mark.parametrize("device", DEVICES)
