@@ -179,7 +179,7 @@ int ogb_latent_set_tc(int on);
 int ogb_hgrn2_state_rows(int D);
 int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D, int V,
               const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int seg_len,
-              int num_segments, float* seg_state, float* seg_gate, int* status, void* stream);
+              int num_segments, float* seg_state, float* seg_gate, int split, int* status, void* stream);
 int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, int elem, void* stream);
 int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, int elem, void* stream);
 int ogb_argmax_f32(const float* logits, int* out_tokens, int rows, int vocab, int ld, void* stream);

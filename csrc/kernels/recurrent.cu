@@ -28,6 +28,7 @@ struct RecParams {
   float* seg_state;       // [segments, heads, V, DP] (segmented runs)
   float* seg_gate;        // [segments, heads, DP]
   int ld, ldo, heads, D, V, num_prefill, seg_len;   // seg_len 0: not segmented
+  int z0;                 // first work item of the launch (decode rows come first)
   StepRows sr;
   int* status;
 };
@@ -82,6 +83,17 @@ OGB_DEVICE bool rec_item(const RecParams& p, int z, RecItem& it) {
   return false;
 }
 
+// State at a segment's start: the end of the segment before, or -- for the first one -- the sequence's state, which the chain
+// kernel has put into the place of the last segment (whose own end state goes straight to the sequence).
+OGB_DEVICE const float* rec_segment_start(const RecParams& p, const RecItem& it, int head, size_t head_state) {
+  int seg = it.seg - 1;
+  if (it.first == 0) {
+    const int s = it.entry - p.sr.num_decode, len = p.sr.cu_q[s + 1] - p.sr.cu_q[s];
+    seg = it.seg + (len + p.seg_len - 1) / p.seg_len - 1;
+  }
+  return p.seg_state + (static_cast<size_t>(seg) * p.heads + head) * head_state;
+}
+
 template <int DP, int CPT>
 struct RecCfg {
   static constexpr int kTok = DP == 256 ? 8 : 16;       // tokens staged at a time
@@ -117,7 +129,7 @@ __global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
   const int threads = blockDim.x, ncols = threads / 32 * 2 * CPT;
   const int head = blockIdx.y, col0 = blockIdx.x * ncols;
   RecItem it;
-  if (!rec_item(p, blockIdx.z, it)) return;
+  if (!rec_item(p, blockIdx.z + p.z0, it)) return;
   if (MODE == kLocal && it.last) return;         // nothing follows this segment: its end state comes out of the second pass
   const StepRows& sr = p.sr;
   const int ctx = sr.ctx_len[it.entry];
@@ -136,7 +148,7 @@ __global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
   // where the run starts: zero, the sequence's slot, or the chained state of the segment before
   const float* init = nullptr;
   if (MODE == kFull) {
-    if (it.first > 0) init = segs - static_cast<size_t>(p.heads) * head_state;
+    if (segs != nullptr && (it.first > 0 || !it.last)) init = rec_segment_start(p, it, head, head_state);
     else if (ctx - (sr.num_decode > it.entry ? 1 : sr.cu_q[it.entry - sr.num_decode + 1] - sr.cu_q[it.entry - sr.num_decode]) > 0) init = own;
   }
   f32x2 s[CPT][QPT][2];
@@ -280,6 +292,250 @@ __global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
     p.seg_gate[(static_cast<size_t>(it.seg) * p.heads + head) * DP + threadIdx.x] = gate;
 }
 
+// ------------------------------------------------------------------------------------------------------
+// The same recurrence on the tensor cores, 16 tokens at a time, for prompts of the bf16 engine.  With P_t the product of the
+// gates up to token t of the block, G = P_15 and X_s the product of the gates after token s,
+//
+//   o_t = (q_t P_t) S + sum_{s <= t} A[t][s] v_s,     A[t][s] = sum_d q_t k_s prod_{s < r <= t} f_r,     S <- G S + (k_s X_s)^T v_s
+//
+// so every factor is a product of gates (at most 1): nothing is divided by a decay and nothing overflows.  A is formed on the
+// fp32 units by running products; the three products with S and v run on mma.sync tf32 with their fp32 factors split in two
+// (S, q P, k X, A: about 21 bits; v, a projection, is rounded to tf32).  The transposed state [column][row] sits in a warp's
+// accumulators, 16 columns a warp, and is read as the A operand of the next product without moving: the contraction index is
+// relabelled so that accumulator and operand fragments agree.
+// ------------------------------------------------------------------------------------------------------
+constexpr int kMbTok = 16;
+
+template <int DP>
+struct MbCfg {
+  static constexpr int kRaw = 2 * DP + 128 + 8;                  // floats per raw row: q, z, v
+  static constexpr int kQp = 2 * DP + 16, kKp = 2 * DP + 8, kAp = 2 * kMbTok + 8;
+  static constexpr int kSmemBytes = 4 * (2 * kMbTok * kRaw + 3 * kMbTok * DP + kMbTok * (kQp + kKp + kAp) + 3 * DP);
+};
+
+OGB_DEVICE float tf32_round(float x) {
+  uint32_t r;
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
+  return __uint_as_float(r);
+}
+OGB_DEVICE float2 tf32_split(float x) {
+  const float hi = tf32_round(x);
+  return make_float2(hi, tf32_round(x - hi));
+}
+OGB_DEVICE void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1) {
+  asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)),
+        "r"(__float_as_uint(b1)));
+}
+
+template <int DP, int MODE>
+__global__ void __launch_bounds__(256, 2) hgrn2_mma_kernel(RecParams p) {
+  using Cfg = MbCfg<DP>;
+  constexpr int NT = DP / 8;                     // 8-row tiles of the state
+  constexpr int EP = DP / 32;                    // gate channels per lane in the running products
+  extern __shared__ __align__(16) uint8_t rec_smem[];
+  float* raw = reinterpret_cast<float*>(rec_smem);                // [2][16][kRaw]
+  float* sf = raw + 2 * kMbTok * Cfg::kRaw;                       // [16][DP] gate, key, query
+  float* sk = sf + kMbTok * DP;
+  float* sq = sk + kMbTok * DP;
+  float* qp = sq + kMbTok * DP;                                   // [16][kQp]: (hi, hi, lo, lo) of two channels
+  float* kx = qp + kMbTok * Cfg::kQp;                             // [16][kKp]: (hi, lo)
+  float* sA = kx + kMbTok * Cfg::kKp;                             // [16][kAp]: (hi, lo)
+  float* sG = sA + kMbTok * Cfg::kAp;                             // [DP] gate product of the block, lower bound, bias
+  float* slow = sG + DP;
+  float* sbias = slow + DP;
+  const int threads = blockDim.x, warps = threads >> 5, ncols = warps * 16;
+  const int head = blockIdx.y, col0 = blockIdx.x * ncols;
+  RecItem it;
+  if (!rec_item(p, blockIdx.z + p.z0, it)) return;
+  if (MODE == kLocal && it.last) return;
+  const StepRows& sr = p.sr;
+  const int ctx = sr.ctx_len[it.entry], slot = sr.state_slot[it.entry];
+  if (ctx <= 0 || slot < 0) return;
+  if (slot >= sr.num_slots) {
+    if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
+  const size_t head_state = static_cast<size_t>(p.V) * DP;
+  float* own = p.state + (static_cast<size_t>(slot) * p.heads + head) * head_state;
+  float* segs = p.seg_len > 0 ? p.seg_state + (static_cast<size_t>(it.seg) * p.heads + head) * head_state : nullptr;
+  const float* init = nullptr;
+  if (MODE == kFull) {
+    const int s = it.entry - sr.num_decode;
+    if (segs != nullptr && (it.first > 0 || !it.last)) init = rec_segment_start(p, it, head, head_state);
+    else if (ctx > sr.cu_q[s + 1] - sr.cu_q[s]) init = own;
+  }
+  const int vr = col0 + warp * 16 + g;           // state columns of this thread: vr, vr + 8
+  float S[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      float2 v = make_float2(0.f, 0.f);
+      if (init != nullptr && vr + 8 * h < p.V) v = *reinterpret_cast<const float2*>(init + static_cast<size_t>(vr + 8 * h) * DP + 8 * j + 2 * tq);
+      S[j][2 * h] = v.x; S[j][2 * h + 1] = v.y;
+    }
+  const int HD = p.heads * p.D;
+  for (int d = threadIdx.x; d < DP; d += threads) {
+    slow[d] = d < p.D ? p.low[head * p.D + d] : 0.f;
+    sbias[d] = d < p.D ? p.bias[head * p.D + d] : 0.f;
+  }
+  for (int i = threadIdx.x; i < kMbTok * kMbTok; i += threads)     // A stays zero above the diagonal
+    *reinterpret_cast<float2*>(sA + (i / kMbTok) * Cfg::kAp + 2 * (i % kMbTok)) = make_float2(0.f, 0.f);
+  const bool vec = ((p.D | p.V | p.ld) & 3) == 0;
+  auto fetch = [&](int t0, int buf) {
+    const int nt = min(kMbTok, it.n - t0), nv = min(ncols, p.V - col0);
+    const int step = vec ? 4 : 1, per = (2 * p.D + nv + step - 1) / step;
+    for (int i = threadIdx.x; i < nt * per; i += threads) {
+      const int t = i / per, e = (i - t * per) * step;
+      const float* src = p.qfv + static_cast<size_t>(it.base + t0 + t) * p.ld;
+      float* dst = raw + (buf * kMbTok + t) * Cfg::kRaw;
+      if (e < p.D) { src += head * p.D + e; dst += e; }
+      else if (e < 2 * p.D) { src += HD + head * p.D + e - p.D; dst += DP + e - p.D; }
+      else { src += 2 * HD + head * p.V + col0 + e - 2 * p.D; dst += 2 * DP + e - 2 * p.D; }
+      if (vec) cp_async<16>(dst, src); else cp_async<4>(dst, src);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(0, 0);
+  float seg_gate = 1.f;
+  for (int t0 = 0, buf = 0; t0 < it.n; t0 += kMbTok, buf ^= 1) {
+    const int nt = min(kMbTok, it.n - t0);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (t0 + kMbTok < it.n) fetch(t0 + kMbTok, buf ^ 1);
+    // ---- gates (tokens past the end: gate 1, key and query 0) ----
+    for (int i = threadIdx.x; i < kMbTok * DP; i += threads) {
+      const int t = i / DP, d = i % DP;
+      const float* row = raw + (buf * kMbTok + t) * Cfg::kRaw;
+      float q = 0.f, f = 1.f, k = 0.f;
+      if (t < nt && d < p.D) {
+        const float low = slow[d], z = row[DP + d] + sbias[d];
+        const float ez = __expf(-fabsf(z));
+        const float r = __fdividef(1.f, 1.f + ez), small = ez * r;
+        f = fmaf(1.f - low, z >= 0.f ? r : small, low);
+        k = (1.f - low) * (z >= 0.f ? small : r);
+        if (MODE == kFull) { const float x = row[d]; q = __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
+      }
+      if (MODE == kFull) sq[i] = q;
+      sf[i] = f; sk[i] = k;
+    }
+    __syncthreads();
+    // ---- products of gates from the block's start and to its end ----
+    for (int i = threadIdx.x; i < 2 * DP; i += threads) {
+      const int d = i % DP;
+      float x = 1.f;
+      if (i < DP) {
+        float* dst = qp + (d >> 1) * 4 + (d & 1);
+#pragma unroll
+        for (int t = 0; t < kMbTok; ++t) {
+          x *= sf[t * DP + d];
+          if (MODE == kFull) {
+            const float2 h = tf32_split(sq[t * DP + d] * x);
+            dst[t * Cfg::kQp] = h.x; dst[t * Cfg::kQp + 2] = h.y;
+          }
+        }
+        sG[d] = x;
+        if (MODE == kLocal && blockIdx.x == 0) seg_gate *= x;      // channel threadIdx.x: segmented launches have DP threads or more
+      } else {
+#pragma unroll
+        for (int t = kMbTok - 1; t >= 0; --t) {
+          *reinterpret_cast<float2*>(kx + t * Cfg::kKp + 2 * d) = tf32_split(sk[t * DP + d] * x);
+          x *= sf[t * DP + d];
+        }
+      }
+    }
+    // ---- A: running products from key s to every later query ----
+    if (MODE == kFull) {
+      for (int i = warp; i < kMbTok; i += warps) {
+        // warp w takes s = w, then 15 - w: as many pairs for every warp when there are eight
+        const int s = i < 8 ? i : 23 - i;
+        float x[EP];
+#pragma unroll
+        for (int e = 0; e < EP; ++e) x[e] = sk[s * DP + lane + 32 * e];
+        for (int t = s; t < kMbTok; ++t) {
+          float a = 0.f;
+#pragma unroll
+          for (int e = 0; e < EP; ++e) {
+            if (t > s) x[e] *= sf[t * DP + lane + 32 * e];
+            a = fmaf(sq[t * DP + lane + 32 * e], x[e], a);
+          }
+          a = warp_sum(a);
+          if (lane == 0) *reinterpret_cast<float2*>(sA + t * Cfg::kAp + 2 * s) = tf32_split(a);
+        }
+      }
+    }
+    __syncthreads();
+    // ---- v^T as the A operand of both products with v ----
+    float v[2][4];
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int t = 8 * k + tq + (x >> 1) * 4, c = warp * 16 + g + (x & 1) * 8;
+        v[k][x] = t < nt && col0 + c < p.V ? tf32_round(raw[(buf * kMbTok + t) * Cfg::kRaw + 2 * DP + c]) : 0.f;
+      }
+    if (MODE == kFull) {
+      float o[2][4] = {};
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        float hi[4], lo[4];
+        const int at[4] = {0, 2, 1, 3};                            // accumulator -> operand: (g, 2 tq) is index tq, (g, 2 tq + 1) is tq + 4
+#pragma unroll
+        for (int x = 0; x < 4; ++x) { const float2 h = tf32_split(S[j][at[x]]); hi[x] = h.x; lo[x] = h.y; }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          const float4 b = *reinterpret_cast<const float4*>(qp + (8 * n + g) * Cfg::kQp + (4 * j + tq) * 4);
+          mma_tf32(o[n], hi, b.x, b.y);
+          mma_tf32(o[n], lo, b.x, b.y);
+          mma_tf32(o[n], hi, b.z, b.w);
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          const float2 b0 = *reinterpret_cast<const float2*>(sA + (8 * n + g) * Cfg::kAp + 2 * (8 * k + tq));
+          const float2 b1 = *reinterpret_cast<const float2*>(sA + (8 * n + g) * Cfg::kAp + 2 * (8 * k + tq + 4));
+          mma_tf32(o[n], v[k], b0.x, b1.x);
+          mma_tf32(o[n], v[k], b0.y, b1.y);
+        }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int t = 8 * n + 2 * tq + (x & 1), c = vr + (x >> 1) * 8;
+          if (t < nt && c < p.V) p.out[static_cast<size_t>(it.base + t0 + t) * p.ldo + head * p.V + c] = o[n][x];
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const float2 gm = *reinterpret_cast<const float2*>(sG + 8 * j + 2 * tq);
+      S[j][0] *= gm.x; S[j][1] *= gm.y; S[j][2] *= gm.x; S[j][3] *= gm.y;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const float2 b0 = *reinterpret_cast<const float2*>(kx + (8 * k + tq) * Cfg::kKp + 2 * (8 * j + g));
+        const float2 b1 = *reinterpret_cast<const float2*>(kx + (8 * k + tq + 4) * Cfg::kKp + 2 * (8 * j + g));
+        mma_tf32(S[j], v[k], b0.x, b1.x);
+        mma_tf32(S[j], v[k], b0.y, b1.y);
+      }
+    }
+  }
+  float* dst = MODE == kLocal ? segs : (it.last ? own : nullptr);
+  if (dst != nullptr) {
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+        if (vr + 8 * h < p.V)
+          *reinterpret_cast<float2*>(dst + static_cast<size_t>(vr + 8 * h) * DP + 8 * j + 2 * tq) = make_float2(S[j][2 * h], S[j][2 * h + 1]);
+  }
+  if (MODE == kLocal && blockIdx.x == 0 && static_cast<int>(threadIdx.x) < DP)
+    p.seg_gate[(static_cast<size_t>(it.seg) * p.heads + head) * DP + threadIdx.x] = seg_gate;
+}
+
 // Turns every segment's local end state into the true state at its end: S_i <- gates_i * S_(i-1) + local_i, starting from the
 // sequence's state.  One thread per four state values of a (head, chunk).
 __global__ void __launch_bounds__(256) hgrn2_chain_kernel(RecParams p, int DP) {
@@ -294,6 +550,7 @@ __global__ void __launch_bounds__(256) hgrn2_chain_kernel(RecParams p, int DP) {
   if (i >= quads) return;
   float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
   if (ctx > len) a = reinterpret_cast<const float4*>(p.state + (static_cast<size_t>(slot) * p.heads + head) * p.V * DP)[i];
+  reinterpret_cast<float4*>(p.seg_state + (static_cast<size_t>(seg0 + segs - 1) * p.heads + head) * p.V * DP)[i] = a;   // where segment 0 starts
   for (int j = 0; j < segs - 1; ++j) {
     const size_t at = static_cast<size_t>(seg0 + j) * p.heads + head;
     float4* u = reinterpret_cast<float4*>(p.seg_state + at * p.V * DP) + i;
@@ -305,12 +562,13 @@ __global__ void __launch_bounds__(256) hgrn2_chain_kernel(RecParams p, int DP) {
 }
 
 template <int DP, int CPT>
-static int launch_hgrn2(const RecParams& p, int items, cudaStream_t stream) {
+static int launch_fma(RecParams p, int items, cudaStream_t stream) {
+  if (items <= p.z0) return 0;
   int warps = (p.V + 2 * CPT - 1) / (2 * CPT);
   if (warps > 8) warps = 8;
   const int need = (DP + 31) / 32;               // the gate products of a segment take one thread per state row
   if (p.seg_len > 0 && warps < need) warps = need;
-  const dim3 grid((p.V + warps * 2 * CPT - 1) / (warps * 2 * CPT), p.heads, items);
+  const dim3 grid((p.V + warps * 2 * CPT - 1) / (warps * 2 * CPT), p.heads, items - p.z0);
   constexpr int smem = RecCfg<DP, CPT>::kSmemBytes;
   static bool attr_set = false;
   if (!attr_set) {
@@ -326,6 +584,45 @@ static int launch_hgrn2(const RecParams& p, int items, cudaStream_t stream) {
   return static_cast<int>(cudaGetLastError());
 }
 
+template <int DP>
+static int launch_mma(const RecParams& p, int items, cudaStream_t stream) {
+  if (items <= p.z0) return 0;
+  int warps = (p.V + 15) / 16;
+  if (warps > 8) warps = 8;
+  if (p.seg_len > 0 && warps < DP / 32) warps = DP / 32;
+  const dim3 grid((p.V + warps * 16 - 1) / (warps * 16), p.heads, items - p.z0);
+  constexpr int smem = MbCfg<DP>::kSmemBytes;
+  static bool attr_set = false;
+  if (!attr_set) {
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(hgrn2_mma_kernel<DP, kLocal>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(hgrn2_mma_kernel<DP, kFull>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    attr_set = true;
+  }
+  if (p.seg_len > 0) {
+    hgrn2_mma_kernel<DP, kLocal><<<grid, warps * 32, smem, stream>>>(p);
+    hgrn2_chain_kernel<<<dim3((p.V * DP / 4 + 255) / 256, p.heads, p.num_prefill), 256, 0, stream>>>(p, DP);
+  }
+  hgrn2_mma_kernel<DP, kFull><<<grid, warps * 32, smem, stream>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// decode rows step by step on the fp32 units; prompts there too, or (split) in blocks on the tensor cores
+template <int DP, int CPT>
+static int launch_hgrn2(RecParams p, int items, bool split, cudaStream_t stream) {
+  if constexpr (DP <= 128) {
+    if (split) {
+      RecParams d = p;
+      d.seg_len = 0;
+      d.num_prefill = 0;
+      const int rc = launch_fma<DP, CPT>(d, p.sr.num_decode, stream);
+      if (rc != 0) return rc;
+      p.z0 = p.sr.num_decode;
+      return launch_mma<DP>(p, items, stream);
+    }
+  }
+  return launch_fma<DP, CPT>(p, items, stream);
+}
+
 }  // namespace ogb
 
 using namespace ogb;
@@ -334,19 +631,20 @@ using namespace ogb;
 extern "C" int ogb_hgrn2_state_rows(int D) { return D <= 0 ? 0 : D <= 64 ? 64 : D <= 128 ? 128 : D <= 256 ? 256 : 0; }
 
 // seg_len > 0: prefill chunks run as segments of that many tokens; num_segments counts them over all chunks, and seg_state
-// [num_segments, heads, V, rows] / seg_gate [num_segments, heads, rows] are scratch.
+// [num_segments, heads, V, rows] / seg_gate [num_segments, heads, rows] are scratch.  split: prompts may run on the tensor cores with
+// split fp32 factors (states of up to 128 rows).
 extern "C" int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D,
                          int V, const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots,
-                         int seg_len, int num_segments, float* seg_state, float* seg_gate, int* status, void* stream) {
+                         int seg_len, int num_segments, float* seg_state, float* seg_gate, int split, int* status, void* stream) {
   if (num_decode + num_prefill <= 0 || heads <= 0 || V <= 0) return 0;
   const int dp = ogb_hgrn2_state_rows(D);
   if (dp == 0) return -2;
   if (seg_len > 0 && (seg_state == nullptr || seg_gate == nullptr || num_segments < num_prefill)) return -3;
-  RecParams p{qfv, bias, low, state, out, seg_state, seg_gate, ld, ldo, heads, D, V, num_prefill, seg_len > 0 ? seg_len : 0,
+  RecParams p{qfv, bias, low, state, out, seg_state, seg_gate, ld, ldo, heads, D, V, num_prefill, seg_len > 0 ? seg_len : 0, 0,
               StepRows{ctx_len, state_slot, cu_q, nullptr, nullptr, num_decode, 0, num_slots}, status};
   const int items = num_decode + (seg_len > 0 ? num_segments : num_prefill);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dp == 64) return launch_hgrn2<64, 8>(p, items, s);
-  if (dp == 128) return launch_hgrn2<128, 8>(p, items, s);
-  return launch_hgrn2<256, 4>(p, items, s);
+  if (dp == 64) return launch_hgrn2<64, 8>(p, items, split != 0, s);
+  if (dp == 128) return launch_hgrn2<128, 8>(p, items, split != 0, s);
+  return launch_hgrn2<256, 4>(p, items, split != 0, s);
 }

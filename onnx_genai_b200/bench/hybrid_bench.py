@@ -175,7 +175,7 @@ def kernel_rows(size: str, timer, pk):
         qfv.normal_()
         state, raw = torch.zeros(nseq, heads, d, d, device="cuda"), torch.empty(t, heads * d, device="cuda")
         bias, low = f32(heads * d) * 2, f32(heads * d) * 0.5
-        row("hgrn2", phase, lambda: hops.hgrn2(qfv, bias, low, state, raw, heads, d, d, si), nbytes=t * heads * d * 16 + 2 * nseq * heads * d * d * 4)
+        row("hgrn2", phase, lambda: hops.hgrn2(qfv, bias, low, state, raw, heads, d, d, si, split=True), nbytes=t * heads * d * 16 + 2 * nseq * heads * d * d * 4)
         nw, attn = f32(d), torch.empty(t, heads * d, dtype=bf, device="cuda")
         row("head_rmsnorm", phase, lambda: hops.head_rmsnorm(raw, nw, 1e-6, attn, heads, d), nbytes=t * heads * d * 6)
         if phase.startswith("prefill"):

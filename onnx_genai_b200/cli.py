@@ -627,8 +627,10 @@ def cmd_validate(args, profiler):
         from .models.registry import load_checkpoint
 
         try:
-            cfg, _ = load_checkpoint(d.root, d.native, torch.bfloat16, "cpu")
-            notes.append(f"{d.native['architecture']} checkpoint: {cfg.num_layers} layers, hidden {cfg.hidden}, vocab {cfg.vocab}, every tensor read")
+            cfg, weights = load_checkpoint(d.root, d.native, torch.bfloat16, "cpu")
+            notes.append(f"{d.native['architecture']} checkpoint: {cfg.num_layers} layers, hidden {cfg.hidden}, vocab {cfg.vocab}, every tensor it names read")
+            if weights.unused:
+                notes.append(f"tensors the configuration does not use: {', '.join(weights.unused[:5])}{' ...' if len(weights.unused) > 5 else ''}")
             if meta is not None and meta.vocab_size and meta.vocab_size != cfg.vocab:
                 problems.append(f"metadata model.vocab_size={meta.vocab_size} but the embedding has {cfg.vocab} rows")
         except Exception as exc:

@@ -195,6 +195,7 @@ class HybridWeights:
     layers: list = field(default_factory=list)
     final_norm: DynamicTanh | None = None
     lm_head: torch.Tensor | None = None
+    unused: list = field(default_factory=list)   # tensors of the checkpoint that its configuration does not name
 
 
 def pad_cols(w, to=None):
@@ -361,7 +362,8 @@ class HybridModel:
         qfv = self._rows(self.qfv, t, pad8(n))
         hops.linear(h, w.qfv, qfv[:, :n], f32_out=True)
         raw = hops.hgrn2(qfv, w.gate_bias, w.gate_low, self.state.layers[li]["recurrent"], self._rows(self.rec_o, t, m.heads * m.vdim), m.heads,
-                         m.dim, m.vdim, si, scratch=lambda name, shape: self._scratch(name, shape, torch.float32))
+                         m.dim, m.vdim, si, scratch=lambda name, shape: self._scratch(name, shape, torch.float32),
+                         split=h.dtype == torch.bfloat16)
         width = m.heads * m.vdim
         attn = self._rows(self.attn, t, pad8(width))
         if pad8(width) != width:

@@ -26,7 +26,7 @@ def read_config(doc: dict, name: str = "rilelorn") -> HybridConfig:
         if mlp is not None and mlp["kind"] != "dense":
             raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
         layers.append(LayerSpec(mixer, MlpSpec(int(mlp["ff"])) if mlp is not None else None))
-    cfg = HybridConfig(vocab=int(doc["vocab"]), hidden=int(doc["width"]), layers=layers, streams=int(doc["streams"]),
+    cfg = HybridConfig(vocab=int(doc["vocab"]), hidden=int(doc["width"]), layers=layers, streams=int(doc.get("streams", 1)),
                        norm_eps=float(doc["norm"]["eps"]), name=name)
     cfg.validate()
     return cfg
@@ -62,7 +62,5 @@ def load_weights(cfg: HybridConfig, tensors, dtype, device) -> HybridWeights:
             pack_mlp(layer, take(p + "mlp.gate"), take(p + "mlp.up"), take(p + "mlp.down"))
         w.layers.append(layer)
     w.final_norm, w.lm_head = norm("final.norm"), pad_cols(take("head"))
-    left = sorted(set(tensors) - used)
-    if left:
-        raise ValueError(f"the checkpoint holds tensors its configuration does not use: {left[:5]}")
+    w.unused = sorted(set(tensors) - used)
     return w

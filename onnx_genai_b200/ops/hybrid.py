@@ -23,7 +23,7 @@ _native.register("ogb_latent_gather", [P, P, P, P, I, I, L, I, I, I, P, P, P, P]
 _native.register("ogb_latent_set_tc", [I])
 _native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
 _native.register("ogb_hgrn2_state_rows", [I])
-_native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P] * 4)
+_native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P, P, I, P, P])
 _native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, I, P])
 _native.register("ogb_act_mul_packed", [P, P, I, I, I, I, I, P])
 
@@ -244,10 +244,11 @@ def segment_length(si, heads: int, vdim: int) -> int:
 
 
 @_timed("hgrn2")
-def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si, segment=None, scratch=None):
+def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si, segment=None, scratch=None, split=False):
     """Advance the recurrence over the step's rows: qfv [T, ld] fp32 (query, gate and value projections), state
     [slots, heads, vdim, state_rows(dim)] fp32 in place, raw head outputs to out [T, ld] fp32.  ``segment``: tokens per segment of
-    the prompts (None: chosen, 0: whole); ``scratch(name, shape)`` provides fp32 scratch for segmented runs."""
+    the prompts (None: chosen, 0: whole); ``scratch(name, shape)`` provides fp32 scratch for segmented runs.
+    ``split``: prompts in blocks on the tensor cores, fp32 factors split in two tf32 terms (v rounded to one)."""
     if not qfv.is_cuda:
         reference.hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si)
         return out
@@ -260,7 +261,7 @@ def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si, segment=None, scratc
     rc = _native.load().ogb_hgrn2(qfv.data_ptr(), bias.data_ptr(), low.data_ptr(), state.data_ptr(), out.data_ptr(), qfv.stride(0),
                                   out.stride(0), heads, dim, vdim, si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(),
                                   si.num_decode, si.num_prefill_seqs, state.shape[0], seg if nseg else 0, nseg, _ptr(us), _ptr(ug),
-                                  status_word().data_ptr(), _stream())
+                                  int(split), status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_hgrn2")
     launch_counts["hgrn2"] += 1
     return out
