@@ -25,6 +25,9 @@ OGB_DEVICE void load_vec(const T* p, float (&r)[V]) {
     const uint2 u = *reinterpret_cast<const uint2*>(p);
     const float2 a = unpack_bf16(u.x), b = unpack_bf16(u.y);
     r[0] = a.x; r[1] = a.y; r[2] = b.x; r[3] = b.y;
+  } else if constexpr (V == 2 && sizeof(T) == 4) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    r[0] = f.x; r[1] = f.y;
   } else {
 #pragma unroll
     for (int i = 0; i < V; ++i) r[i] = to_f32<T>(p[i]);

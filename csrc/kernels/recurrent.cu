@@ -449,22 +449,59 @@ __global__ void __launch_bounds__(256, 2) hgrn2_mma_kernel(RecParams p) {
     }
     // ---- A: running products from key s to every later query ----
     if (MODE == kFull) {
-      for (int i = warp; i < kMbTok; i += warps) {
-        // warp w takes s = w, then 15 - w: as many pairs for every warp when there are eight
-        const int s = i < 8 ? i : 23 - i;
-        float x[EP];
+      for (int i = warp; i < kMbTok / 2; i += warps) {
+        // keys i and 15 - i at a time (they share the loads); a lane holds EP neighbouring channels
+        float x[2][EP], a[kMbTok];
+        float f[EP], q[EP];
+        load_vec<EP>(sk + i * DP + lane * EP, x[0]);
+        load_vec<EP>(sk + (kMbTok - 1 - i) * DP + lane * EP, x[1]);
+        float a2[kMbTok / 2];                                      // key 15 - i starts in the upper half
 #pragma unroll
-        for (int e = 0; e < EP; ++e) x[e] = sk[s * DP + lane + 32 * e];
-        for (int t = s; t < kMbTok; ++t) {
-          float a = 0.f;
+        for (int t = 0; t < kMbTok; ++t) {
+          load_vec<EP>(sf + t * DP + lane * EP, f);
+          load_vec<EP>(sq + t * DP + lane * EP, q);
+          float u = 0.f, w = 0.f;
 #pragma unroll
           for (int e = 0; e < EP; ++e) {
-            if (t > s) x[e] *= sf[t * DP + lane + 32 * e];
-            a = fmaf(sq[t * DP + lane + 32 * e], x[e], a);
+            if (t > i) x[0][e] *= f[e];
+            u = fmaf(q[e], x[0][e], u);
+            if (t >= kMbTok / 2) {
+              if (t > kMbTok - 1 - i) x[1][e] *= f[e];
+              w = fmaf(q[e], x[1][e], w);
+            }
           }
-          a = warp_sum(a);
-          if (lane == 0) *reinterpret_cast<float2*>(sA + t * Cfg::kAp + 2 * s) = tf32_split(a);
+          a[t] = u;
+          if (t >= kMbTok / 2) a2[t - kMbTok / 2] = w;
         }
+        // lane sums by halving: lane L ends with a[L mod 16 bit-reversed] and a2[L mod 8 bit-reversed]
+        int ta = 0, tb = 0;
+#pragma unroll
+        for (int w = kMbTok / 2, bit = 1; w >= 1; w >>= 1, bit <<= 1) {
+          const bool up = (lane & bit) != 0;
+#pragma unroll
+          for (int c = 0; c < w; ++c) {
+            const float send = up ? a[c] : a[c + w], keep = up ? a[c + w] : a[c];
+            a[c] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+          }
+          ta += up ? w : 0;
+        }
+        a[0] += __shfl_xor_sync(0xffffffffu, a[0], 16);
+#pragma unroll
+        for (int w = kMbTok / 4, bit = 1; w >= 1; w >>= 1, bit <<= 1) {
+          const bool up = (lane & bit) != 0;
+#pragma unroll
+          for (int c = 0; c < w; ++c) {
+            const float send = up ? a2[c] : a2[c + w], keep = up ? a2[c + w] : a2[c];
+            a2[c] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+          }
+          tb += up ? w : 0;
+        }
+        a2[0] += __shfl_xor_sync(0xffffffffu, a2[0], 8);
+        a2[0] += __shfl_xor_sync(0xffffffffu, a2[0], 16);
+        if (lane < 16 && ta >= i) *reinterpret_cast<float2*>(sA + ta * Cfg::kAp + 2 * i) = tf32_split(a[0]);
+        tb += kMbTok / 2;
+        if (lane < 8 && tb >= kMbTok - 1 - i)
+          *reinterpret_cast<float2*>(sA + tb * Cfg::kAp + 2 * (kMbTok - 1 - i)) = tf32_split(a2[0]);
       }
     }
     __syncthreads();
@@ -478,7 +515,7 @@ __global__ void __launch_bounds__(256, 2) hgrn2_mma_kernel(RecParams p) {
         v[k][x] = t < nt && col0 + c < p.V ? tf32_round(raw[(buf * kMbTok + t) * Cfg::kRaw + 2 * DP + c]) : 0.f;
       }
     if (MODE == kFull) {
-      float o[2][4] = {};
+      float o[2][4] = {}, oc[2][4] = {};                           // leading products and corrections: four chains of accumulation
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
         float hi[4], lo[4];
@@ -489,8 +526,8 @@ __global__ void __launch_bounds__(256, 2) hgrn2_mma_kernel(RecParams p) {
         for (int n = 0; n < 2; ++n) {
           const float4 b = *reinterpret_cast<const float4*>(qp + (8 * n + g) * Cfg::kQp + (4 * j + tq) * 4);
           mma_tf32(o[n], hi, b.x, b.y);
-          mma_tf32(o[n], lo, b.x, b.y);
-          mma_tf32(o[n], hi, b.z, b.w);
+          mma_tf32(oc[n], lo, b.x, b.y);
+          mma_tf32(oc[n], hi, b.z, b.w);
         }
       }
 #pragma unroll
@@ -500,14 +537,14 @@ __global__ void __launch_bounds__(256, 2) hgrn2_mma_kernel(RecParams p) {
           const float2 b0 = *reinterpret_cast<const float2*>(sA + (8 * n + g) * Cfg::kAp + 2 * (8 * k + tq));
           const float2 b1 = *reinterpret_cast<const float2*>(sA + (8 * n + g) * Cfg::kAp + 2 * (8 * k + tq + 4));
           mma_tf32(o[n], v[k], b0.x, b1.x);
-          mma_tf32(o[n], v[k], b0.y, b1.y);
+          mma_tf32(oc[n], v[k], b0.y, b1.y);
         }
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
           const int t = 8 * n + 2 * tq + (x & 1), c = vr + (x >> 1) * 8;
-          if (t < nt && c < p.V) p.out[static_cast<size_t>(it.base + t0 + t) * p.ldo + head * p.V + c] = o[n][x];
+          if (t < nt && c < p.V) p.out[static_cast<size_t>(it.base + t0 + t) * p.ldo + head * p.V + c] = o[n][x] + oc[n][x];
         }
     }
 #pragma unroll

@@ -231,14 +231,14 @@ def latent_prefill_expanded(q, out, pool, kv_w, si, heads, d, scale, window, pag
 
 def segment_length(si, heads: int, vdim: int) -> int:
     """Tokens per segment of a step's prompts, 0 to run every chunk in one piece: chunks are cut while the (head, chunk) pairs
-    leave the device half empty (a segmented run costs two thirds of a pass more)."""
+    leave much of the device empty (a segmented run goes over the gates twice)."""
     if si.num_prefill_seqs == 0 or si.prefill_len is None:
         return 0
     longest, per = int(si.prefill_len.max()), heads * max(1, -(-vdim // 128))
-    if per * si.num_prefill_seqs >= 148 or longest < 256:
+    if per * si.num_prefill_seqs >= 100 or longest < 256:
         return 0
     seg = 1 << (longest - 1).bit_length()
-    while seg > 128 and per * int((-(-si.prefill_len // seg)).sum()) < 296:
+    while seg > 128 and per * int((-(-si.prefill_len // seg)).sum()) < 256:
         seg //= 2
     return seg if seg < longest else 0
 
