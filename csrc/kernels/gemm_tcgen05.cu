@@ -46,7 +46,7 @@ constexpr int kGemmThreads = 192;
 constexpr int kGemmThreadsScatter = 224;  // + one warp that publishes finished tiles to peer GPUs
 
 enum GemmEpilogue : int { kEpiNone = 0, kEpiResidual = 1, kEpiSwiGLU = 2, kEpiScatter = 3 };
-enum GemmAct : int { kActSilu = 0, kActGeluTanh = 1 };   // gate activation of the gated epilogue
+enum GemmAct : int { kActSilu = 0, kActGeluTanh = 1, kActRelu2 = 2 };   // the gate of the gated epilogue; Relu2: every value of the plain one
 
 // 0.5 z (1 + tanh(a)) = z / (1 + exp(-2 a)); relative error of a few 1e-7, ahead of a bf16 rounding
 OGB_DEVICE float gelu_tanh_fast(float z) {
@@ -352,6 +352,9 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
             }
           }
           if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+          // this warp is the only reader of those flags: lowered again, so that a replayed graph, which brings the same
+          // sequence number back, waits for the partials of its own run
+          for (int x = fix_lo + lane; x < fix_hi; x += 32) sk_flags[x * 4 + q] = 0;
         }
       }
       if (C_f32 != nullptr) {
@@ -437,6 +440,14 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                     if (col + j < N) r[j] = __float_as_uint(__uint_as_float(r[j]) + __bfloat162float(bias[col + j]));
                 }
               }
+              if constexpr (EPI == kEpiNone)
+                if (act == kActRelu2) {
+#pragma unroll
+                  for (int j = 0; j < 32; ++j) {
+                    const float v = fmaxf(__uint_as_float(r[j]), 0.f);
+                    r[j] = __float_as_uint(v * v);
+                  }
+                }
 #pragma unroll
               for (int j = 0; j < 16; ++j) o[j] = pack_bf16(__uint_as_float(r[2 * j]), __uint_as_float(r[2 * j + 1]));
             }
@@ -961,21 +972,53 @@ extern "C" int ogb_gemm_bf16_scatter(const void* A, const void* W, int M, int N,
 
 // Grouped GEMM over experts (MoE): rows of A are sorted by expert; `group_tab` holds one int4 per
 // 128-row tile {expert, first row, end row, 0} and `group_mtiles` their count, both produced on the
-// device by ogb_moe_permute, so no routing information crosses to the host.  W is [experts, N, K].
-// epilogue 0 = plain, 2 = SwiGLU over per-expert packed gate|up weights (output width N/2).
+// device by ogb_moe_permute, so no routing information crosses to the host.  W is [experts, N, ldw].
+// epilogue 0 = plain (act 2: square of relu), 2 = SwiGLU over per-expert packed gate|up weights (output width N/2, N a multiple
+// of bn).  A tile that reaches past an expert's N rows of W computes columns that are not stored.
+static int grouped_gemm(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows,
+                        int max_mtiles, int N, int K, int lda, int ldw, int ldc, int epilogue, int act, int bn, int* status, cudaStream_t stream) {
+  if (max_rows <= 0 || experts <= 0) return 0;
+  if ((K % 8) != 0 || (lda % 8) != 0 || (ldw % 8) != 0 || (ldc % 8) != 0) return -3;
+  if (epilogue == kEpiSwiGLU && (N % bn) != 0) return -3;
+#define OGB_GROUPED(BN, EPI)                                                                                                                     \
+  return launch_gemm<BN, EPI>(A, W, C, nullptr, nullptr, nullptr, max_rows, N, K, lda, ldw, ldc, 0, status, stream, nullptr, group_tab,          \
+                              group_mtiles, experts, max_mtiles, nullptr, nullptr, 0, GemmBatch(), act)
+  if (epilogue == kEpiNone) {
+    if (bn == 256) OGB_GROUPED(256, kEpiNone);
+    if (bn == 128) OGB_GROUPED(128, kEpiNone);
+    if (bn == 64) OGB_GROUPED(64, kEpiNone);
+  } else if (epilogue == kEpiSwiGLU) {
+    if (bn == 256) OGB_GROUPED(256, kEpiSwiGLU);
+    if (bn == 128) OGB_GROUPED(128, kEpiSwiGLU);
+  }
+#undef OGB_GROUPED
+  return -2;
+}
+
 extern "C" int ogb_grouped_gemm_bf16(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles,
                                      int experts, int max_rows, int max_mtiles, int N, int K, int epilogue, int bn, int* status,
-                                     void* stream_) {
-  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (max_rows <= 0 || experts <= 0) return 0;
-  if ((K % 8) != 0 || (N % bn) != 0) return -3;
-  const int ldc = epilogue == kEpiSwiGLU ? N / 2 : N;
-  if (epilogue == kEpiNone) {
-    if (bn == 256) return launch_gemm<256, kEpiNone>(A, W, C, nullptr, nullptr, nullptr, max_rows, N, K, K, K, ldc, 0, status, stream, nullptr, group_tab, group_mtiles, experts, max_mtiles);
-    if (bn == 128) return launch_gemm<128, kEpiNone>(A, W, C, nullptr, nullptr, nullptr, max_rows, N, K, K, K, ldc, 0, status, stream, nullptr, group_tab, group_mtiles, experts, max_mtiles);
-  } else if (epilogue == kEpiSwiGLU) {
-    if (bn == 256) return launch_gemm<256, kEpiSwiGLU>(A, W, C, nullptr, nullptr, nullptr, max_rows, N, K, K, K, ldc, 0, status, stream, nullptr, group_tab, group_mtiles, experts, max_mtiles);
-    if (bn == 128) return launch_gemm<128, kEpiSwiGLU>(A, W, C, nullptr, nullptr, nullptr, max_rows, N, K, K, K, ldc, 0, status, stream, nullptr, group_tab, group_mtiles, experts, max_mtiles);
+                                     void* stream) {
+  if (bn <= 0 || (N % bn) != 0) return -3;
+  return grouped_gemm(A, W, C, group_tab, group_mtiles, experts, max_rows, max_mtiles, N, K, K, K, epilogue == kEpiSwiGLU ? N / 2 : N, epilogue,
+                      kActSilu, bn, status, static_cast<cudaStream_t>(stream));
+}
+
+// Plain products with any N, row strides of their own and an activation (0 none, 2 square of relu).  bn 0: picked from the most
+// tiles the launch can have.
+extern "C" int ogb_grouped_gemm_act(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows,
+                                    int max_mtiles, int N, int K, int lda, int ldw, int ldc, int act, int bn, int* status, void* stream) {
+  if (act != 0 && act != kActRelu2) return -7;
+  if (bn == 0) {
+    const int sms = ogb_num_sms();
+    const int cand[3] = {256, 128, 64};
+    const float cost[3] = {1.0f, 0.62f, 0.40f};
+    float best = 1e30f;
+    for (int i = 0; i < 3; ++i) {
+      const int tiles = max_mtiles * ((N + cand[i] - 1) / cand[i]);
+      const float t = static_cast<float>((tiles + sms - 1) / sms) * cost[i];
+      if (t < best - 1e-6f) { best = t; bn = cand[i]; }
+    }
   }
-  return -2;
+  return grouped_gemm(A, W, C, group_tab, group_mtiles, experts, max_rows, max_mtiles, N, K, lda, ldw, ldc, kEpiNone, act, bn, status,
+                      static_cast<cudaStream_t>(stream));
 }

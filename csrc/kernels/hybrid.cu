@@ -195,6 +195,141 @@ static int dispatch_hyper(const HyperParams& p, cudaStream_t stream) {
 }
 
 // ------------------------------------------------------------------------------------------------------
+// norm_step is the pass between two products for designs with one residual stream and RMS norms on both sides of a sublayer:
+//
+//   x <- x + rms(y) post        h = rms(x) w
+//
+// y is the sublayer's output row, or -- behind routed experts -- the weighted sum of the token's expert rows
+// (sum_j weight[t][j] ys[pos[t][j]]), taken here so that it never exists in memory.  One block per row, the row in registers; all
+// fp32.
+// ------------------------------------------------------------------------------------------------------
+struct NormStepParams {
+  float* x;                // [rows, W]
+  const void* y;           // [rows, ldy], or the expert rows
+  const int* pos;          // [rows, k] or null
+  const float* weight;     // [rows, k]
+  const float *post, *w;   // norm weights
+  void* h;                 // [rows, ldh] or null
+  const int* gather;       // row r of h comes from row gather[r]; x is then left alone
+  float eps;
+  int rows, total_rows, W, k, ldy, ldh;
+  int64_t y_rows;
+  int* status;
+};
+
+OGB_DEVICE float block_sum(float v, float* red) {
+  const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  v = warp_sum(v);
+  __syncthreads();                             // the last sum has been read
+  if ((threadIdx.x & 31) == 0) red[warp] = v;
+  __syncthreads();
+  float s = 0.f;
+  for (int i = 0; i < warps; ++i) s += red[i];
+  return s;
+}
+
+template <typename T, int V, int N>
+__global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
+  __shared__ float red[32];
+  const int r = blockIdx.x;
+  int t = r;
+  if (p.gather != nullptr) {
+    t = p.gather[r];
+    if (t < 0 || t >= p.total_rows) {
+      if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
+      t = 0;
+    }
+  }
+  float x[N][V];
+  float* xr = p.x + static_cast<size_t>(t) * p.W;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[i][v] = 0.f;
+    if (c < p.W) load_vec<V>(xr + c, x[i]);
+  }
+  if (p.y != nullptr) {
+    float y[N][V], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int v = 0; v < V; ++v) y[i][v] = 0.f;
+    const int k = p.pos != nullptr ? p.k : 1;
+    for (int j = 0; j < k; ++j) {
+      int64_t row = t;
+      float f = 1.f;
+      if (p.pos != nullptr) {
+        row = p.pos[static_cast<size_t>(t) * k + j];
+        f = p.weight[static_cast<size_t>(t) * k + j];
+        if (row < 0 || row >= p.y_rows) {
+          if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
+          continue;
+        }
+      }
+      const T* src = static_cast<const T*>(p.y) + row * p.ldy;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int c = (i * blockDim.x + threadIdx.x) * V;
+        if (c < p.W) {
+          float z[V];
+          load_vec<V>(src + c, z);
+#pragma unroll
+          for (int v = 0; v < V; ++v) y[i][v] = fmaf(f, z[v], y[i][v]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int v = 0; v < V; ++v) ss = fmaf(y[i][v], y[i][v], ss);
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(p.W) + p.eps);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < p.W) {
+        float g[V];
+        load_vec<V>(p.post + c, g);
+#pragma unroll
+        for (int v = 0; v < V; ++v) x[i][v] = fmaf(y[i][v] * inv, g[v], x[i][v]);
+        if (p.gather == nullptr) store_vec<V>(xr + c, x[i]);
+      }
+    }
+  }
+  if (p.h == nullptr) return;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+#pragma unroll
+    for (int v = 0; v < V; ++v) ss = fmaf(x[i][v], x[i][v], ss);
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(p.W) + p.eps);
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+    if (c < p.W) {
+      float g[V];
+      load_vec<V>(p.w + c, g);
+#pragma unroll
+      for (int v = 0; v < V; ++v) x[i][v] *= inv * g[v];
+      store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r) * p.ldh + c, x[i]);
+    }
+  }
+}
+
+template <typename T, int V>
+static int launch_norm_step(const NormStepParams& p, cudaStream_t s) {
+  const int units = (p.W + V - 1) / V;
+  const int threads = units >= 4096 ? 1024 : units >= 256 ? 256 : (units + 31) / 32 * 32;
+  const int n = (units + threads - 1) / threads;
+  if (n <= 1) norm_step_kernel<T, V, 1><<<p.rows, threads, 0, s>>>(p);
+  else if (n <= 2) norm_step_kernel<T, V, 2><<<p.rows, threads, 0, s>>>(p);
+  else if (n <= 4) norm_step_kernel<T, V, 4><<<p.rows, threads, 0, s>>>(p);
+  else if (n <= 16) norm_step_kernel<T, V, 16><<<p.rows, threads, 0, s>>>(p);
+  else return -2;
+  return static_cast<int>(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------------
 // all streams of a row start as the token's embedding
 // ------------------------------------------------------------------------------------------------------
 template <typename T>
@@ -239,19 +374,23 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const T* __restrict_
 }
 
 // ------------------------------------------------------------------------------------------------------
-// RMS norm of every group of `n` columns (a head) with one shared weight: fp32 in, activation type out; one warp per group
+// RMS norm of every group of `n` columns (a head) with one shared weight, times silu of a gate of the same layout where there is
+// one: fp32 in, activation type out; one warp per group
 // ------------------------------------------------------------------------------------------------------
+OGB_DEVICE float silu_f32(float z) { return z / (1.f + expf(-z)); }
+
 template <typename T>
 __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, T* __restrict__ out,
-                                                           int rows, int heads, int n, int ldx, int ldo) {
+                                                           int rows, int heads, int n, int ldx, int ldo, const T* __restrict__ gate, int ldg) {
   const int lane = threadIdx.x & 31;
   const long long g = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   if (g >= static_cast<long long>(rows) * heads) return;
   const int t = static_cast<int>(g / heads), h = static_cast<int>(g % heads);
   const float* src = x + static_cast<size_t>(t) * ldx + static_cast<size_t>(h) * n;
   T* dst = out + static_cast<size_t>(t) * ldo + static_cast<size_t>(h) * n;
+  const T* gt = gate != nullptr ? gate + static_cast<size_t>(t) * ldg + static_cast<size_t>(h) * n : nullptr;
   float ss = 0.f;
-  if ((n & 127) == 0 && n <= 512 && (ldx & 3) == 0 && (ldo & 3) == 0) {
+  if ((n & 127) == 0 && n <= 512 && ((ldx | ldo | ldg) & 3) == 0) {
     float v[4][4];
     const int per = n >> 7;
 #pragma unroll
@@ -269,13 +408,18 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restri
         load_vec<4>(w + k * 128 + lane * 4, wv);
 #pragma unroll
         for (int i = 0; i < 4; ++i) v[k][i] *= inv * wv[i];
+        if (gt != nullptr) {
+          load_vec<4>(gt + k * 128 + lane * 4, wv);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) v[k][i] *= silu_f32(wv[i]);
+        }
         store_vec<4>(dst + k * 128 + lane * 4, v[k]);
       }
     return;
   }
   for (int i = lane; i < n; i += 32) ss = fmaf(src[i], src[i], ss);
   const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
-  for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(src[i] * inv * w[i]);
+  for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(src[i] * inv * w[i] * (gt != nullptr ? silu_f32(to_f32<T>(gt[i])) : 1.f));
 }
 
 // ------------------------------------------------------------------------------------------------------
@@ -295,16 +439,27 @@ __global__ void __launch_bounds__(256) act_mul_packed_kernel(const T* __restrict
 
 // ------------------------------------------------------------------------------------------------------
 // fp32 matrix product (no reduced-precision mode): C[M,N] = A[M,K] W[N,K]^T for `batch` problems whose operands start at
-// column offsets of A and C and at row offsets of W.  64 x 64 tile, 4 x 4 results per thread.
+// column offsets of A and C and at row offsets of W.  64 x 64 tile, 4 x 4 results per thread.  Grouped: rows of A are sorted by
+// expert, `tab` / `mtiles` are the 128-row tile table of moe.cu, and W holds one matrix per expert.
 // ------------------------------------------------------------------------------------------------------
 constexpr int kF32Tile = 64, kF32K = 16;
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W, float* __restrict__ C, int M,
-                                                       int N, int K, int lda, int ldw, int ldc, int a_step, int c_step) {
+                                                       int N, int K, int lda, int ldw, int ldc, int a_step, int c_step, const int* __restrict__ tab,
+                                                       const int* __restrict__ mtiles, int relu2) {
   __shared__ float sa[kF32K][kF32Tile + 4], sw[kF32K][kF32Tile + 4];
   A += static_cast<size_t>(blockIdx.z) * a_step;
   W += static_cast<size_t>(blockIdx.z) * N * ldw;
   C += static_cast<size_t>(blockIdx.z) * c_step;
-  const int m0 = blockIdx.y * kF32Tile, n0 = blockIdx.x * kF32Tile;
+  const int n0 = blockIdx.x * kF32Tile;
+  int m0 = blockIdx.y * kF32Tile;
+  if (tab != nullptr) {
+    const int mt = blockIdx.y / 2;
+    if (mt >= *mtiles) return;
+    W += static_cast<size_t>(tab[4 * mt]) * N * ldw;
+    m0 = tab[4 * mt + 1] + (blockIdx.y & 1) * kF32Tile;
+    M = min(M, tab[4 * mt + 2]);
+    if (m0 >= M) return;
+  }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kF32K) {
@@ -331,7 +486,10 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int r = m0 + ty * 4 + i, c = n0 + tx * 4 + j;
-      if (r < M && c < N) C[static_cast<size_t>(r) * ldc + c] = acc[i][j];
+      if (r < M && c < N) {
+        const float v = relu2 ? fmaxf(acc[i][j], 0.f) * fmaxf(acc[i][j], 0.f) : acc[i][j];
+        C[static_cast<size_t>(r) * ldc + c] = v;
+      }
     }
 }
 
@@ -354,6 +512,20 @@ extern "C" int ogb_hyper_step(const float* x_in, float* x_out, const void* y, co
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (elem == kElemBF16) return vec ? dispatch_hyper<__nv_bfloat16, 4>(p, s) : dispatch_hyper<__nv_bfloat16, 1>(p, s);
   if (elem == kElemF32) return vec ? dispatch_hyper<float, 4>(p, s) : dispatch_hyper<float, 1>(p, s);
+  return -3;
+}
+
+// pos / weight (null: y has one row per token): y holds y_rows expert rows, of which token t sums k.  w / h null: no read-out.
+extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const float* post, const float* w, void* h,
+                             const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int ldh, int64_t y_rows, int elem,
+                             int* status, void* stream) {
+  if (rows <= 0) return 0;
+  if (W < 1 || (y != nullptr && post == nullptr) || (h != nullptr && w == nullptr) || (pos != nullptr && (weight == nullptr || k < 1))) return -3;
+  NormStepParams p{x, y, pos, weight, post, w, h, gather, eps, rows, total_rows, W, k, ldy, ldh, y_rows, status};
+  const bool vec = ((W | ldy | ldh) & 3) == 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (elem == kElemBF16) return vec ? launch_norm_step<__nv_bfloat16, 4>(p, s) : launch_norm_step<__nv_bfloat16, 1>(p, s);
+  if (elem == kElemF32) return vec ? launch_norm_step<float, 4>(p, s) : launch_norm_step<float, 1>(p, s);
   return -3;
 }
 
@@ -383,13 +555,15 @@ extern "C" int ogb_latent_append(const void* c, int ldc, const float* w, float e
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, int elem,
-                                void* stream) {
+extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate,
+                                int ldg, int elem, void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * heads + 7) / 8);
-  if (elem == kElemBF16) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo);
-  else if (elem == kElemF32) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo);
+  if (elem == kElemBF16) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo,
+                                                                           static_cast<const __nv_bfloat16*>(gate), ldg);
+  else if (elem == kElemF32) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo,
+                                                                              static_cast<const float*>(gate), ldg);
   else return -3;
   return static_cast<int>(cudaGetLastError());
 }
@@ -411,6 +585,16 @@ extern "C" int ogb_gemm_f32(const float* A, const float* W, float* C, int M, int
                             int c_step, void* stream) {
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
   const dim3 grid((N + kF32Tile - 1) / kF32Tile, (M + kF32Tile - 1) / kF32Tile, batch);
-  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, M, N, K, lda, ldw, ldc, a_step, c_step);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, M, N, K, lda, ldw, ldc, a_step, c_step, nullptr, nullptr, 0);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Products over experts (see ogb_grouped_gemm_bf16); act 2: square of relu.
+extern "C" int ogb_grouped_gemm_f32(const float* A, const float* W, float* C, const int* group_tab, const int* group_mtiles, int max_rows,
+                                    int max_mtiles, int N, int K, int lda, int ldw, int ldc, int act, void* stream) {
+  if (max_rows <= 0 || max_mtiles <= 0 || N <= 0) return 0;
+  if (act != 0 && act != 2) return -7;
+  const dim3 grid((N + kF32Tile - 1) / kF32Tile, 2 * max_mtiles);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, max_rows, N, K, lda, ldw, ldc, 0, 0, group_tab, group_mtiles, act == 2);
   return static_cast<int>(cudaGetLastError());
 }

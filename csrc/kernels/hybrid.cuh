@@ -1,5 +1,6 @@
 // Shared pieces of the kernels behind models with a per-layer mixer choice (hybrid.cu, recurrent.cu,
-// latent_attention.cu): the row structure of a step and loads / stores of the two activation types.
+// latent_attention.cu): the row structure of a step, loads / stores of the two activation types, packed fp32
+// arithmetic and the split tf32 products of the recurrences.
 // These files are compiled without fast math: tanh, exponentials, divisions and roots keep their full precision.
 #pragma once
 #include "common.cuh"
@@ -56,5 +57,47 @@ struct StepRows {
   const int* tile_q0;
   int num_decode, num_tiles, num_slots;
 };
+
+// two fp32 values in one 64-bit register
+typedef unsigned long long f32x2;
+OGB_DEVICE f32x2 f2_fma(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+OGB_DEVICE f32x2 f2_mul(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+OGB_DEVICE float f2_sum(f32x2 a) {
+  float x, y;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
+  return x + y;
+}
+
+template <int BYTES>
+OGB_DEVICE void cp_async(void* dst, const void* src) {
+  if constexpr (BYTES == 16)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  else
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+
+OGB_DEVICE float tf32_round(float x) {
+  uint32_t r;
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
+  return __uint_as_float(r);
+}
+OGB_DEVICE float2 tf32_split(float x) {
+  const float hi = tf32_round(x);
+  return make_float2(hi, tf32_round(x - hi));
+}
+OGB_DEVICE void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1) {
+  asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)),
+        "r"(__float_as_uint(b1)));
+}
 
 }  // namespace ogb

@@ -19,9 +19,13 @@ namespace ogb {
 
 constexpr int kMaxExperts = 256;
 
-__global__ void moe_route_topk_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ topk_ids,
-                                      float* __restrict__ topk_w, int tokens, int experts, int k, int renormalize, int ld) {
+// `groups` > 1: experts form that many equal groups of neighbours, a group scores as its best expert, and only the `keep` best
+// groups can be chosen from.
+template <typename T>
+__global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict__ logits, int* __restrict__ topk_ids, float* __restrict__ topk_w,
+                                                             int tokens, int experts, int k, int renormalize, int ld, int groups, int keep) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  __shared__ float s_group[8][kMaxExperts];
   if (warp >= tokens) return;
   constexpr int PER = kMaxExperts / 32;
   float v[PER];
@@ -29,38 +33,80 @@ __global__ void moe_route_topk_kernel(const __nv_bfloat16* __restrict__ logits, 
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
-    v[i] = (e < experts) ? __bfloat162float(logits[static_cast<size_t>(warp) * ld + e]) : -INFINITY;
+    v[i] = (e < experts) ? static_cast<float>(logits[static_cast<size_t>(warp) * ld + e]) : -INFINITY;
     mx = fmaxf(mx, v[i]);
   }
   mx = warp_max(mx);
   float sum = 0.f;
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
-    v[i] = (i * 32 + lane < experts) ? __expf(v[i] - mx) : 0.f;
+    v[i] = (i * 32 + lane < experts) ? expf(v[i] - mx) : 0.f;
     sum += v[i];
   }
   sum = warp_sum(sum);
   const float inv = 1.f / sum;
-  float chosen_sum = 0.f;
-  float my_w = 0.f;
-  int my_id = 0;
-  for (int r = 0; r < k; ++r) {
-    float best = -1.f;
-    int best_e = 0x7fffffff;
+  // the largest of a set of values with the lowest index among equals
+  auto best_of = [&](const float (&x)[PER], int count, float& best, int& at) {
+    best = -1.f;
+    at = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int e = i * 32 + lane;
-      if (e < experts && (v[i] > best || (v[i] == best && e < best_e))) { best = v[i]; best_e = e; }
+      if (e < count && (x[i] > best || (x[i] == best && e < at))) { best = x[i]; at = e; }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-      if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
+      const int oe = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ob > best || (ob == best && oe < at)) { best = ob; at = oe; }
     }
+  };
+  if (groups > 1 && keep < groups) {
+    float* s = s_group[threadIdx.x >> 5];
+    const int size = experts / groups;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) s[i * 32 + lane] = v[i];
+    __syncwarp();
+    float gs[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int g = i * 32 + lane;
+      gs[i] = -1.f;
+      if (g < groups)
+        for (int e = 0; e < size; ++e) gs[i] = fmaxf(gs[i], s[g * size + e]);
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < PER; ++i) s[i * 32 + lane] = 0.f;      // 1: the group stays
+    __syncwarp();
+    for (int r = 0; r < keep; ++r) {
+      float best;
+      int at;
+      best_of(gs, groups, best, at);
+      if (lane == 0 && at < groups) s[at] = 1.f;
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (i * 32 + lane == at) gs[i] = -2.f;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int e = i * 32 + lane;
+      if (e < experts && s[e / size] == 0.f) v[i] = -1.f;
+    }
+  }
+  float chosen_sum = 0.f;
+  float my_w = 0.f;
+  int my_id = 0;
+  for (int r = 0; r < k; ++r) {
+    float best;
+    int best_e;
+    best_of(v, experts, best, best_e);
     if (lane == r) { my_w = best * inv; my_id = best_e; }
     chosen_sum += best * inv;
-    if ((best_e & 31) == lane) v[best_e >> 5] = -1.f;   // remove the winner
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (i * 32 + lane == best_e) v[i] = -1.f;                // remove the winner
   }
   if (lane < k) {
     topk_ids[static_cast<size_t>(warp) * k + lane] = my_id;
@@ -122,14 +168,14 @@ __global__ void moe_assign_kernel(const int* __restrict__ topk_ids, const int* _
   route_pos[i] = pos;
 }
 
-__global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ sorted_route,
-                                       const int* __restrict__ meta, __nv_bfloat16* __restrict__ xs, int k, int hidden) {
+__global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, const int* __restrict__ sorted_route, const int* __restrict__ meta,
+                                       uint4* __restrict__ xs, int k, int vecs) {
   const int pos = blockIdx.x;
   if (pos >= meta[1]) return;
   const int token = sorted_route[pos] / k;
-  const uint4* src = reinterpret_cast<const uint4*>(x + static_cast<size_t>(token) * hidden);
-  uint4* dst = reinterpret_cast<uint4*>(xs + static_cast<size_t>(pos) * hidden);
-  for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x) dst[i] = src[i];
+  const uint4* src = x + static_cast<size_t>(token) * vecs;
+  uint4* dst = xs + static_cast<size_t>(pos) * vecs;
+  for (int i = threadIdx.x; i < vecs; i += blockDim.x) dst[i] = src[i];
 }
 
 __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ ys, const int* __restrict__ route_pos,
@@ -166,15 +212,28 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ ys, const i
 
 using namespace ogb;
 
-extern "C" int ogb_moe_route_topk(const void* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k,
-                                  int renormalize, int ld, void* stream) {
+template <typename T>
+static int route_topk(const T* logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize, int ld, int groups, int keep,
+                      void* stream) {
   if (tokens <= 0) return 0;
   if (experts > kMaxExperts || k > 32 || k > experts) return -3;
+  if (groups < 1 || experts % groups != 0 || keep < 1 || keep > groups || k > keep * (experts / groups)) return -3;
   const int warps_per_block = 8;
   const int blocks = (tokens + warps_per_block - 1) / warps_per_block;
-  moe_route_topk_kernel<<<blocks, warps_per_block * 32, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const __nv_bfloat16*>(router_logits), topk_ids, topk_w, tokens, experts, k, renormalize, ld);
+  moe_route_topk_kernel<T><<<blocks, warps_per_block * 32, 0, static_cast<cudaStream_t>(stream)>>>(logits, topk_ids, topk_w, tokens, experts, k,
+                                                                                                 renormalize, ld, groups, keep);
   return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int ogb_moe_route_topk(const void* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k,
+                                  int renormalize, int ld, void* stream) {
+  return route_topk(static_cast<const __nv_bfloat16*>(router_logits), topk_ids, topk_w, tokens, experts, k, renormalize, ld, 1, 1, stream);
+}
+
+// fp32 logits; `groups` equal groups of experts of which the `keep` best can be chosen from (1, 1: all).
+extern "C" int ogb_moe_route_grouped(const float* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize,
+                                     int ld, int groups, int keep, void* stream) {
+  return route_topk(router_logits, topk_ids, topk_w, tokens, experts, k, renormalize, ld, groups, keep, stream);
 }
 
 // counts must be zero on entry (the caller clears it); e0 = first expert owned by this rank.
@@ -191,13 +250,23 @@ extern "C" int ogb_moe_permute(const int* topk_ids, int* counts, int* offsets, i
   return static_cast<int>(cudaGetLastError());
 }
 
+static int gather_rows(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int row_bytes, void* stream) {
+  if (max_routes <= 0) return 0;
+  if (row_bytes % 16) return -3;
+  const int vecs = row_bytes / 16;
+  moe_gather_rows_kernel<<<max_routes, vecs < 128 ? (vecs + 31) / 32 * 32 : 128, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const uint4*>(x), sorted_route, meta, static_cast<uint4*>(xs), k, vecs);
+  return static_cast<int>(cudaGetLastError());
+}
+
 extern "C" int ogb_moe_gather_rows(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k,
                                    int hidden, void* stream) {
-  if (max_routes <= 0) return 0;
-  if (hidden % 8) return -3;
-  moe_gather_rows_kernel<<<max_routes, 128, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const __nv_bfloat16*>(x), sorted_route, meta, static_cast<__nv_bfloat16*>(xs), k, hidden);
-  return static_cast<int>(cudaGetLastError());
+  return gather_rows(x, sorted_route, meta, xs, max_routes, k, 2 * hidden, stream);
+}
+// Rows of any type, row_bytes a multiple of 16.
+extern "C" int ogb_moe_gather_bytes(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int row_bytes,
+                                    void* stream) {
+  return gather_rows(x, sorted_route, meta, xs, max_routes, k, row_bytes, stream);
 }
 
 extern "C" int ogb_moe_combine(const void* ys, const int* route_pos, const float* topk_w, void* out, int tokens, int k,

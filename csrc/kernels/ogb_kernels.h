@@ -180,7 +180,31 @@ int ogb_hgrn2_state_rows(int D);
 int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D, int V,
               const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int seg_len,
               int num_segments, float* seg_state, float* seg_gate, int split, int* status, void* stream);
-int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, int elem, void* stream);
+int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate, int ldg,
+                     int elem, void* stream);
+// norm_step: x += rms(y) post, h = rms(x) w over one fp32 residual stream; y may be the weighted sum of a token's expert rows.
+int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const float* post, const float* w, void* h, const int* gather, float eps,
+                  int rows, int total_rows, int W, int k, int ldy, int ldh, int64_t y_rows, int elem, int* status, void* stream);
+// Short causal convolutions (short_conv.cu): w [taps, channels], state [slots, taps - 1, channels].
+// Attention: q (nq heads of d) | k (nk) | v (nv heads of dv); rotated queries to q, keys and values to pages [nk][16][dp] | [nv][16][vp].
+int ogb_conv_rope_append(const void* u, int ldu, const float* w, const float* bias, float* state, int taps, void* q, int ldq, void* pool,
+                         const int* slots, const double* freq, int64_t num_slots, int64_t page_elems, int nq, int nk, int nv, int d, int dv, int dp,
+                         int vp, int rot, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0,
+                         int num_decode, int num_tiles, int state_slots, int elem, int* status, void* stream);
+// Delta rule: unit queries and keys (fp32), values, and per head (log of the decay, step size).
+int ogb_conv_unit_gates(const void* u, int ldu, const float* w, float* state, int taps, const float* ab, int ldab, const float* a_log,
+                        const float* dt_bias, float* qk, void* v, void* gates, int nk, int nv, int d, int dv, const int* ctx_len, const int* state_slot,
+                        const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode, int num_tiles, int state_slots, int elem, int* status,
+                        void* stream);
+// Gated delta rule over state [slots, heads, V, ogb_hgrn2_state_rows(D)].
+int ogb_delta_rule(const float* qk, const void* v, const void* gates, float* state, float* out, int heads, int groups, int D, int V, const int* ctx_len,
+                   const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int elem, int* status, void* stream);
+// Differential attention over the pages of ogb_conv_rope_append (nk = 2 hkv maps); cu_q null: decode rows.
+int ogb_diff_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, const int* tile_seq,
+                       const int* tile_q0, int rows, int num_tiles, int max_pages, int64_t num_pages, int64_t page_elems, int hq, int hkv, int d, int dv,
+                       int dp, int vp, int ldq, int ldo, int window, int keep, float scale, float lambda, float eps, float gain, int num_splits,
+                       float* part_o, float* part_ml, int* counters, int elem, int* status, void* stream);
+int ogb_diff_set_tc(int on);
 int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, int elem, void* stream);
 int ogb_argmax_f32(const float* logits, int* out_tokens, int rows, int vocab, int ld, void* stream);
 int ogb_sample_f32(const float* logits, int* out_tokens, const float* temperature, const int* top_k, const float* top_p, const float* min_p,
@@ -193,6 +217,13 @@ int ogb_moe_permute(const int* topk_ids, int* counts, int* offsets, int* cursor,
                     int* tile_tab, int* meta, int tokens, int k, int e0, int experts, int max_mtiles, void* stream);
 int ogb_moe_gather_rows(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int hidden,
                         void* stream);
+int ogb_moe_route_grouped(const float* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize, int ld,
+                          int groups, int keep, void* stream);
+int ogb_moe_gather_bytes(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int row_bytes, void* stream);
+int ogb_grouped_gemm_act(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows, int max_mtiles,
+                         int N, int K, int lda, int ldw, int ldc, int act, int bn, int* status, void* stream);
+int ogb_grouped_gemm_f32(const float* A, const float* W, float* C, const int* group_tab, const int* group_mtiles, int max_rows, int max_mtiles, int N,
+                         int K, int lda, int ldw, int ldc, int act, void* stream);
 int ogb_moe_combine(const void* ys, const int* route_pos, const float* topk_w, void* out, int tokens, int k, int hidden,
                     int accumulate, void* stream);
 int ogb_grouped_gemm_bf16(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts,

@@ -35,24 +35,6 @@ struct RecParams {
 
 enum RecMode : int { kFull = 0, kLocal = 1 };
 
-// two fp32 values in one 64-bit register
-typedef unsigned long long f32x2;
-OGB_DEVICE f32x2 f2_fma(f32x2 a, f32x2 b, f32x2 c) {
-  f32x2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-OGB_DEVICE f32x2 f2_mul(f32x2 a, f32x2 b) {
-  f32x2 r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-OGB_DEVICE float f2_sum(f32x2 a) {
-  float x, y;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
-  return x + y;
-}
-
 // Rows of work item z: a decode row, or a (segment of a) prefill chunk.
 struct RecItem {
   int entry, base, n, first, seg;        // first: tokens of the chunk before this segment; seg: global segment index
@@ -100,14 +82,6 @@ struct RecCfg {
   static constexpr int kMaxCols = 8 * 2 * CPT;          // columns of a CTA of eight warps
   static constexpr int kSmemBytes = 4 * (kTok * (3 * DP + 3 * kMaxCols) + 2 * DP + 2 * kTok * (2 * DP + kMaxCols));
 };
-
-template <int BYTES>
-OGB_DEVICE void cp_async(void* dst, const void* src) {
-  if constexpr (BYTES == 16)
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-  else
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
 
 template <int DP, int CPT, int MODE>
 __global__ void __launch_bounds__(256, 2) hgrn2_kernel(RecParams p) {
@@ -312,22 +286,6 @@ struct MbCfg {
   static constexpr int kQp = 2 * DP + 16, kKp = 2 * DP + 8, kAp = 2 * kMbTok + 8;
   static constexpr int kSmemBytes = 4 * (2 * kMbTok * kRaw + 3 * kMbTok * DP + kMbTok * (kQp + kKp + kAp) + 3 * DP);
 };
-
-OGB_DEVICE float tf32_round(float x) {
-  uint32_t r;
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
-  return __uint_as_float(r);
-}
-OGB_DEVICE float2 tf32_split(float x) {
-  const float hi = tf32_round(x);
-  return make_float2(hi, tf32_round(x - hi));
-}
-OGB_DEVICE void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1) {
-  asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)),
-        "r"(__float_as_uint(b1)));
-}
 
 template <int DP, int MODE>
 __global__ void __launch_bounds__(256, 2) hgrn2_mma_kernel(RecParams p) {

@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from . import decoder, hybrid, rilelorn
+from . import decoder, dezudra, hybrid, rilelorn
 from .config import DecoderConfig
 
 
@@ -36,7 +36,8 @@ FAMILIES = (
     Family(hybrid.HybridConfig, hybrid.HybridModel, lambda cfg, device, tp, rank, seed, dtype: hybrid.random_weights(cfg, device, seed=seed, dtype=dtype),
            ("bf16", "f32")),
 )
-ARCHITECTURES = {a.name: a for a in (Architecture("Rilelorn", rilelorn.read_config, rilelorn.load_weights, "hybrid"),)}
+ARCHITECTURES = {a.name: a for a in (Architecture("Rilelorn", rilelorn.read_config, rilelorn.load_weights, "hybrid"),
+                                     Architecture("Dezudra", dezudra.read_config, dezudra.load_weights, "delta"))}
 
 
 def family_of(cfg) -> Family:

@@ -1,6 +1,8 @@
-"""Ops of models that choose a mixer per layer (csrc/kernels/hybrid.cu, recurrent.cu, latent_attention.cu): hyper-connected
-residual streams with a Dynamic-Tanh norm and token shift, HGRN2 recurrence over per-sequence state, attention over paged
-latents, batched per-head products, and the fp32 matrix product of the 32-bit engine.
+"""Ops of models that choose a mixer per layer (csrc/kernels/hybrid.cu, recurrent.cu, latent_attention.cu, short_conv.cu,
+delta_rule.cu, diff_attention.cu): hyper-connected residual streams with a Dynamic-Tanh norm and token shift, one residual stream
+with RMS norms on both sides of a sublayer, HGRN2 and gated delta-rule recurrences over per-sequence state, short causal
+convolutions, attention over paged latents, differential attention over paged keys and values, batched per-head products, and
+the fp32 matrix product of the 32-bit engine.
 
 CUDA tensors run the kernels; CPU tensors run the statements in :mod:`onnx_genai_b200.ops.reference`, as the other ops do.
 ``si`` is the step's :class:`~onnx_genai_b200.models.decoder.StepInputs`.
@@ -24,7 +26,13 @@ _native.register("ogb_latent_set_tc", [I])
 _native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
 _native.register("ogb_hgrn2_state_rows", [I])
 _native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P, P, I, P, P])
-_native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, I, P])
+_native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, P, I, I, P])
+_native.register("ogb_norm_step", [P] * 8 + [F] + [I] * 6 + [L, I, P, P])
+_native.register("ogb_conv_rope_append", [P, I, P, P, P, I, P, I, P, P, P, L, L] + [I] * 8 + [P] * 5 + [I] * 4 + [P, P])
+_native.register("ogb_conv_unit_gates", [P, I, P, P, I, P, I] + [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, P])
+_native.register("ogb_delta_rule", [P] * 5 + [I] * 4 + [P] * 3 + [I] * 4 + [P, P])
+_native.register("ogb_diff_attention", [P] * 8 + [I] * 3 + [L, L] + [I] * 10 + [F] * 4 + [I, P, P, P, I, P, P])
+_native.register("ogb_diff_set_tc", [I])
 _native.register("ogb_act_mul_packed", [P, P, I, I, I, I, I, P])
 
 ACTS = {"silu": 0, "gelu_tanh": 1}
@@ -46,6 +54,21 @@ class HyperConnection:
     read: torch.Tensor
     write: torch.Tensor
     mix: torch.Tensor
+
+
+@dataclass
+class RmsNorm:
+    """x / sqrt(mean(x^2) + eps) w; w fp32."""
+    w: torch.Tensor
+    eps: float
+
+
+@dataclass
+class ExpertRows:
+    """A sublayer's output that is still spread over expert rows: token t's is sum_j weight[t, j] rows[pos[t, j]]."""
+    rows: torch.Tensor
+    pos: torch.Tensor
+    weight: torch.Tensor
 
 
 def state_rows(dim: int) -> int:
@@ -268,13 +291,126 @@ def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si, segment=None, scratc
 
 
 @_timed("head_rmsnorm")
-def head_rmsnorm(x, w, eps, out, heads, n):
-    """RMS norm of each head's n columns of x [T, ld] (fp32) with one shared weight."""
+def head_rmsnorm(x, w, eps, out, heads, n, gate=None):
+    """RMS norm of each head's n columns of x [T, ld] (fp32) with one shared weight, times silu(gate) [T, heads * n] where given."""
     if not x.is_cuda:
-        out[:, : heads * n] = reference.head_rmsnorm(x, w, eps, heads, n, out.dtype)
+        out[:, : heads * n] = reference.head_rmsnorm(x, w, eps, heads, n, out.dtype, gate)
         return out
     rc = _native.load().ogb_head_rmsnorm(x.data_ptr(), w.data_ptr(), float(eps), out.data_ptr(), x.shape[0], heads, n, x.stride(0),
-                                         out.stride(0), _ELEM[out.dtype], _stream())
+                                         out.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, _ELEM[out.dtype], _stream())
     _native.check(rc, "ogb_head_rmsnorm")
     launch_counts["head_rmsnorm"] += 1
     return out
+
+
+@_timed("norm_step")
+def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
+    """x [T, W] fp32 += post(y); h = norm(x).  ``y``: rows of the last sublayer's output, :class:`ExpertRows`, or None.  ``gather``:
+    h gets the rows it names only, and x stays as it is."""
+    rows = h.shape[0] if h is not None else x.shape[0]
+    routed = y if isinstance(y, ExpertRows) else None
+    if not x.is_cuda:
+        new = reference.norm_step(x, y, post)
+        if gather is None:
+            x.copy_(new)
+        else:
+            new = new[gather.long()]
+        if h is not None:
+            h[:, : x.shape[1]] = reference.rms(new, norm.w, norm.eps).to(h.dtype)
+        return h
+    src = routed.rows if routed is not None else y
+    eps = norm.eps if norm is not None else post.eps
+    assert post is None or post.eps == eps
+    rc = _native.load().ogb_norm_step(
+        x.data_ptr(), _ptr(src), _ptr(routed.pos if routed else None), _ptr(routed.weight if routed else None), _ptr(post.w if post is not None else None),
+        _ptr(norm.w if norm is not None else None), _ptr(h), _ptr(gather), float(eps), rows, x.shape[0], x.shape[1],
+        routed.pos.shape[1] if routed else 1, src.stride(0) if src is not None else 0, h.stride(0) if h is not None else 0,
+        routed.rows.shape[0] if routed else 0, _ELEM[h.dtype if h is not None else src.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_norm_step")
+    launch_counts["norm_step"] += 1
+    return h
+
+
+def _rows_args(si, state):
+    return (si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), si.num_decode,
+            si.num_tiles, state.shape[0])
+
+
+@_timed("conv_rope_append")
+def conv_rope_append(u, w, bias, state, q, pool, freq, si, nq, nk, nv, d, dv, dp, vp):
+    """Short convolution over the projected rows u [T, nq d | nk d | nv dv] (w [taps, channels], bias added first, state
+    [slots, taps - 1, channels] advanced), rotation of the first 2 len(freq) dimensions of every query and key (angles position x
+    freq, fp64), queries to q [T, nq * dp], keys and values to the pages [nk][16][dp] | [nv][16][vp] of pool [pages, elements]."""
+    if not u.is_cuda:
+        reference.conv_rope_append(u, w, bias, state, q, pool, freq, si, nq, nk, nv, d, dv, dp, vp)
+        return
+    assert pool.dtype == u.dtype == q.dtype and freq.dtype == torch.float64
+    rc = _native.load().ogb_conv_rope_append(
+        u.data_ptr(), u.stride(0), w.data_ptr(), _ptr(bias), state.data_ptr(), w.shape[0], q.data_ptr(), q.stride(0), pool.data_ptr(), si.slots.data_ptr(),
+        freq.data_ptr(), backed_pages(pool) * PAGE, pool.stride(0), nq, nk, nv, d, dv, dp, vp, 2 * freq.numel(), *_rows_args(si, state), _ELEM[u.dtype],
+        status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_conv_rope_append")
+    launch_counts["conv_rope_append"] += 1
+
+
+@_timed("conv_unit_gates")
+def conv_unit_gates(u, w, state, ab, a_log, dt_bias, qk, v, gates, si, nk, nv, d, dv):
+    """Short convolution and silu over the projected rows u [T, nk d | nk d | nv dv]; queries (times d^-1/2) and keys as unit vectors
+    to qk [T, 2 nk d] fp32, values to v, and from ab [T, nv | nv] fp32 the log decay -exp(a_log) softplus(a + dt_bias) and the step size
+    sigmoid(b) of every head to gates [T, nv, 2] fp32."""
+    if not u.is_cuda:
+        reference.conv_unit_gates(u, w, state, ab, a_log, dt_bias, qk, v, gates, si, nk, nv, d, dv)
+        return
+    assert qk.is_contiguous() and v.is_contiguous() and gates.is_contiguous() and v.dtype == u.dtype
+    rc = _native.load().ogb_conv_unit_gates(
+        u.data_ptr(), u.stride(0), w.data_ptr(), state.data_ptr(), w.shape[0], ab.data_ptr(), ab.stride(0), a_log.data_ptr(), dt_bias.data_ptr(),
+        qk.data_ptr(), v.data_ptr(), gates.data_ptr(), nk, nv, d, dv, *_rows_args(si, state), _ELEM[u.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_conv_unit_gates")
+    launch_counts["conv_unit_gates"] += 1
+
+
+@_timed("delta_rule")
+def delta_rule(qk, v, gates, state, out, heads, groups, dim, vdim, si):
+    """Advance the gated delta rule over the step's rows (inputs of :func:`conv_unit_gates`): state [slots, heads, vdim,
+    state_rows(dim)] fp32 in place, raw head outputs to out [T, heads * vdim] fp32."""
+    if not qk.is_cuda:
+        reference.delta_rule(qk, v, gates, state, out, heads, groups, dim, vdim, si)
+        return out
+    assert out.is_contiguous()
+    rc = _native.load().ogb_delta_rule(qk.data_ptr(), v.data_ptr(), gates.data_ptr(), state.data_ptr(), out.data_ptr(), heads, groups, dim, vdim,
+                                       si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(), si.num_decode, si.num_prefill_seqs,
+                                       state.shape[0], _ELEM[v.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_delta_rule")
+    launch_counts["delta_rule"] += 1
+    return out
+
+
+@_timed("diff_attention")
+def diff_attention(q, out, pool, si, hq, hkv, d, dv, dp, vp, scale, lam, eps, gain, window=0, keep=0, splits=1, part_o=None, part_ml=None,
+                   counters=None):
+    """Differential attention: q [T, (head, map) dp], pages of :func:`conv_rope_append` (2 hkv key maps), out [T, hq * vp] =
+    gain rms(a1 - lam a2).  ``window`` > 0: a query sees its last ``window`` keys and the first ``keep`` of the sequence."""
+    if not q.is_cuda:
+        reference.diff_attention(q, out, pool, si, hq, hkv, d, dv, dp, vp, scale, lam, eps, gain, window, keep)
+        return out
+    lib, st = _native.load(), status_word().data_ptr()
+    nd, npf, t = si.num_decode, si.num_prefill_seqs, si.num_tokens
+    tail = (si.page_table.shape[1], backed_pages(pool), pool.stride(0), hq, hkv, d, dv, dp, vp, q.stride(0), out.stride(0), int(window), int(keep),
+            float(scale), float(lam), float(eps), float(gain))
+    if nd > 0:
+        rc = lib.ogb_diff_attention(q.data_ptr(), out.data_ptr(), pool.data_ptr(), si.page_table.data_ptr(), si.ctx_len.data_ptr(), 0, 0, 0, nd, 0, *tail,
+                                    int(splits), _ptr(part_o), _ptr(part_ml), _ptr(counters), _ELEM[q.dtype], st, _stream())
+        _native.check(rc, "ogb_diff_attention")
+        launch_counts["diff_decode"] += 1
+    if npf > 0:
+        rc = lib.ogb_diff_attention(q[nd:].data_ptr(), out[nd:].data_ptr(), pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(),
+                                    si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), t - nd, si.num_tiles, *tail, 1, 0, 0, 0,
+                                    _ELEM[q.dtype], st, _stream())
+        _native.check(rc, "ogb_diff_attention")
+        launch_counts["diff_prefill"] += 1
+    return out
+
+
+def set_diff_tc(on: bool) -> bool:
+    """Switch the tensor-core kernels of differential attention (on by default); returns the old setting."""
+    return bool(_native.load().ogb_diff_set_tc(int(on)))

@@ -11,6 +11,10 @@ _native.register("ogb_moe_permute", [P] * 8 + [I] * 5 + [P])
 _native.register("ogb_moe_gather_rows", [P, P, P, P, I, I, I, P])
 _native.register("ogb_moe_combine", [P, P, P, P, I, I, I, I, P])
 _native.register("ogb_grouped_gemm_bf16", [P] * 5 + [I] * 7 + [P, P])
+_native.register("ogb_moe_route_grouped", [P, P, P] + [I] * 7 + [P])
+_native.register("ogb_moe_gather_bytes", [P, P, P, P, I, I, I, P])
+_native.register("ogb_grouped_gemm_act", [P] * 5 + [I] * 10 + [P, P])
+_native.register("ogb_grouped_gemm_f32", [P] * 5 + [I] * 8 + [P])
 
 
 def _stream():
@@ -95,3 +99,50 @@ def moe_experts(h, router_logits, expert_gate_up, expert_down, ws: MoEWorkspace,
     launch_counts["moe_grouped_gemm"] += 2
     launch_counts["moe_combine"] += 1
     return out
+
+
+def relu2_experts(h, logits, up, down, ws: MoEWorkspace, k, groups=1, keep=1, renormalize=False):
+    """Experts without a gate: down(relu(up h)^2), routed by softmax scores over fp32 ``logits`` [T, experts] with the experts in
+    ``groups`` of which ``keep`` stay (``reference.moe_route``).  up [E, inter, ld(h)], down [E, hidden, inter].  Returns the
+    tokens' outputs as :class:`~.hybrid.ExpertRows`: the residual step sums them."""
+    from .hybrid import ExpertRows
+
+    t, e = h.shape[0], up.shape[0]
+    inter, hidden = up.shape[1], down.shape[1]
+    if not h.is_cuda:
+        ids, w = reference.moe_route(logits, k, renormalize, groups, keep)
+        rows = torch.zeros(t * k, ws.ys.shape[1], dtype=h.dtype)
+        flat = ids.reshape(-1)
+        for x in range(e):
+            at = (flat == x).nonzero().flatten()
+            if at.numel():
+                a = torch.relu(reference.gemm(h[at // k], up[x], out_dtype=torch.float32)).pow(2).to(h.dtype)
+                rows[at, :hidden] = reference.gemm(a, down[x])
+        return ExpertRows(rows, torch.arange(t * k, dtype=torch.int32).view(t, k), w)
+    lib, st, s = _native.load(), status_word(h.device).data_ptr(), _stream()
+    f32 = h.dtype == torch.float32
+    with timed_region("moe_route_permute"):
+        rc = lib.ogb_moe_route_grouped(logits.data_ptr(), ws.topk_ids.data_ptr(), ws.topk_w.data_ptr(), t, e, k, int(renormalize), logits.stride(0),
+                                       groups, keep, s)
+        _native.check(rc, "ogb_moe_route_grouped")
+        rc = lib.ogb_moe_permute(ws.topk_ids.data_ptr(), ws.counts.data_ptr(), ws.offsets.data_ptr(), ws.cursor.data_ptr(), ws.sorted_route.data_ptr(),
+                                 ws.route_pos.data_ptr(), ws.tile_tab.data_ptr(), ws.meta.data_ptr(), t, k, 0, e, ws.max_mtiles, s)
+        _native.check(rc, "ogb_moe_permute")
+        rc = lib.ogb_moe_gather_bytes(h.data_ptr(), ws.sorted_route.data_ptr(), ws.meta.data_ptr(), ws.xs.data_ptr(), t * k, k,
+                                      h.stride(0) * h.element_size(), s)
+        _native.check(rc, "ogb_moe_gather_bytes")
+    mtiles = min(ws.max_mtiles, (t * k + 127) // 128 + e, t * k)
+    for name, a, w, c, act in (("up", ws.xs, up, ws.act, 2), ("down", ws.act, down, ws.ys, 0)):
+        with timed_region("moe_grouped_gemm_" + name):
+            if f32:
+                rc = lib.ogb_grouped_gemm_f32(a.data_ptr(), w.data_ptr(), c.data_ptr(), ws.tile_tab.data_ptr(), ws.meta.data_ptr(), a.shape[0], mtiles,
+                                              w.shape[1], w.shape[2], a.stride(0), w.shape[2], c.stride(0), act, s)
+            else:
+                rc = lib.ogb_grouped_gemm_act(a.data_ptr(), w.data_ptr(), c.data_ptr(), ws.tile_tab.data_ptr(), ws.meta.data_ptr(), e, a.shape[0], mtiles,
+                                              w.shape[1], w.shape[2], a.stride(0), w.shape[2], c.stride(0), act, 0, st, s)
+        _native.check(rc, "grouped product " + name)
+    launch_counts["moe_route_topk"] += 1
+    launch_counts["moe_permute"] += 4
+    launch_counts["moe_gather_rows"] += 1
+    launch_counts["moe_grouped_gemm"] += 2
+    return ExpertRows(ws.ys, ws.route_pos[: t * k].view(t, k), ws.topk_w[: t * k].view(t, k))

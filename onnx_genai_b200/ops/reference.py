@@ -332,8 +332,13 @@ def quantize_w4(w, block=32, symmetric=True):
     return q, scales, zp
 
 
-def moe_route(router_logits, k, renormalize=True):
+def moe_route(router_logits, k, renormalize=True, groups=1, keep=1):
+    """``groups`` > 1: only experts of the ``keep`` groups of neighbours whose best expert scores highest can be chosen."""
     probs = torch.softmax(router_logits.float(), dim=-1)
+    if groups > 1:
+        best = probs.view(probs.shape[0], groups, -1).amax(-1)
+        kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, torch.topk(best, keep, dim=-1).indices, True)
+        probs = probs.masked_fill(~kept.repeat_interleave(probs.shape[1] // groups, 1), -1.0)
     w, ids = torch.topk(probs, k, dim=-1)
     if renormalize:
         w = w / w.sum(-1, keepdim=True)
@@ -405,10 +410,110 @@ def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si):
         state[slot, :, :, :dim] = s
 
 
-def head_rmsnorm(x, w, eps, heads, n, out_dtype=None):
-    y = x[:, : heads * n].float().view(-1, heads, n)
-    y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w
-    return y.reshape(x.shape[0], heads * n).to(out_dtype or x.dtype)
+def rms(x, w, eps):
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
+
+
+def head_rmsnorm(x, w, eps, heads, n, out_dtype=None, gate=None):
+    y = rms(x[:, : heads * n].float().view(-1, heads, n), w, eps).reshape(x.shape[0], heads * n)
+    if gate is not None:
+        y = y * torch.nn.functional.silu(gate.float())
+    return y.to(out_dtype or x.dtype)
+
+
+def norm_step(x, y, post):
+    """x + post(y) for rows of y, or the weighted sum of a token's expert rows (ops.hybrid.ExpertRows)."""
+    if y is None:
+        return x
+    if not torch.is_tensor(y):
+        y = (y.rows[y.pos.long()].float() * y.weight[:, :, None]).sum(1)
+    return x + rms(y[:, : x.shape[1]].float(), post.w, post.eps)
+
+
+def short_conv(u, w, state, si):
+    """u [T, C] fp32 -> sum_j w[j] u_(t - taps + 1 + j) along every sequence; state [slots, taps - 1, C] is advanced."""
+    taps, out = w.shape[0], torch.empty_like(u)
+    for _, base, n, start, slot in step_entries(si):
+        before = state[slot].clone()
+        before[: max(0, taps - 1 - start)] = 0
+        rows = torch.cat([before, u[base:base + n]])
+        out[base:base + n] = sum(w[j] * rows[j:j + n] for j in range(taps))
+        if taps > 1:
+            state[slot] = rows[-(taps - 1):]
+    return out
+
+
+def rotate_half(x, pos, freq):
+    """x [T, heads, d]: dimension i turns with i + len(freq) by pos * freq[i]; dimensions past 2 len(freq) pass."""
+    half = freq.numel()
+    a = pos.double()[:, None] * freq[None, :]
+    c, s = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
+    u, v = x[..., :half], x[..., half:2 * half]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
+
+
+def conv_rope_append(u, w, bias, state, q, pool, freq, si, nq, nk, nv, d, dv, dp, vp):
+    t, n = si.num_tokens, (nq + nk) * d + nv * dv
+    y = short_conv(u[:, :n].float() + bias, w, state, si)
+    x = rotate_half(y[:, :(nq + nk) * d].view(t, nq + nk, d), si.positions[:t], freq)
+    q.view(t, nq, dp)[..., :d] = x[:, :nq].to(q.dtype)
+    live = si.slots[:t] >= 0
+    page, off = (si.slots[:t][live] // PAGE).long(), (si.slots[:t][live] % PAGE).long()
+    keys, values = diff_pages(pool, nk, nv, dp, vp)
+    keys[page, :, off, :d] = x[live, nq:].to(pool.dtype)
+    values[page, :, off, :dv] = y[live, (nq + nk) * d:].view(-1, nv, dv).to(pool.dtype)
+
+
+def diff_pages(pool, nk, nv, dp, vp):
+    """Views of a pool of pages [nk][16][dp] | [nv][16][vp]: keys [pages, nk, 16, dp], values [pages, nv, 16, vp]."""
+    k = nk * PAGE * dp
+    return pool[:, :k].view(-1, nk, PAGE, dp), pool[:, k:k + nv * PAGE * vp].view(-1, nv, PAGE, vp)
+
+
+def conv_unit_gates(u, w, state, ab, a_log, dt_bias, qk, v, gates, si, nk, nv, d, dv):
+    t = si.num_tokens
+    y = torch.nn.functional.silu(short_conv(u[:, :2 * nk * d + nv * dv].float(), w, state, si))
+    x = y[:, :2 * nk * d].view(t, 2, nk, d)
+    x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
+    x[:, 0] *= d ** -0.5
+    qk[:t] = x.reshape(t, -1)
+    v[:t] = y[:, 2 * nk * d:].to(v.dtype)
+    gates[:t, :, 0] = -torch.exp(a_log) * torch.nn.functional.softplus(ab[:, :nv] + dt_bias)
+    gates[:t, :, 1] = torch.sigmoid(ab[:, nv:2 * nv])
+
+
+def delta_rule(qk, v, gates, state, out, heads, groups, dim, vdim, si):
+    t, per = qk.shape[0], heads // groups
+    q, k = (x.repeat_interleave(per, 1) for x in qk.view(t, 2, groups, dim).unbind(1))
+    vv = v.float().view(t, heads, vdim)
+    for _, base, n, start, slot in step_entries(si):
+        s = state[slot, :, :, :dim].clone() if start > 0 else torch.zeros(heads, vdim, dim)
+        for r in range(base, base + n):
+            s = s * torch.exp(gates[r, :, 0])[:, None, None]
+            w = gates[r, :, 1][:, None] * (vv[r] - torch.einsum("hvd,hd->hv", s, k[r]))
+            s = s + w[:, :, None] * k[r][:, None, :]
+            out[r, : heads * vdim] = torch.einsum("hvd,hd->hv", s, q[r]).reshape(-1)
+        state[slot, :, :, :dim] = s
+
+
+def diff_attention(q, out, pool, si, hq, hkv, d, dv, dp, vp, scale, lam, eps, gain, window, keep):
+    keys, values = diff_pages(pool, 2 * hkv, hkv, dp, vp)
+    for e, base, n, start, _ in step_entries(si):
+        ctx = start + n
+        lo = max(0, start - window + 1) if window > 0 else 0
+        i, j = torch.arange(start, ctx)[:, None], torch.arange(ctx)[None, :]
+        seen = j <= i
+        if window > 0:
+            seen &= (i - j < window) | (j < keep)
+        near = (torch.arange(ctx) >= lo) | (torch.arange(ctx) < keep)      # pages in between may be gone
+        j = j[0][near]
+        page, off = si.page_table[e].long()[j // PAGE], j % PAGE
+        k = keys[page, :, off, :d].float().view(-1, hkv, 2, d).repeat_interleave(hq // hkv, 1)
+        v = values[page, :, off, :dv].float().repeat_interleave(hq // hkv, 1)
+        s = torch.einsum("nhmd,khmd->hmnk", q[base:base + n].view(n, hq, 2, dp)[..., :d].float(), k) * scale
+        p = torch.softmax(s.masked_fill(~seen[:, near], float("-inf")), -1)
+        a = torch.einsum("hmnk,khd->mnhd", p, v)
+        out[base:base + n].view(n, hq, vp)[..., :dv] = rms(a[0] - lam * a[1], gain, eps).to(out.dtype)
 
 
 def latent_append(c, w, eps, slots, pool, rank):
