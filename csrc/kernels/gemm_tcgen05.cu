@@ -684,6 +684,20 @@ int encode_tmap_bf16_2d(CUtensorMap* out, const void* base, uint64_t rows, uint6
 }
 
 
+// 3-D bf16 array [planes][rows][cols] with strides in elements; box = box_planes x box_rows x box_cols, 128-byte swizzled (box_cols 64).
+int encode_tmap_bf16_3d(CUtensorMap* out, const void* base, uint64_t cols, uint64_t rows, uint64_t planes, uint64_t row_stride, uint64_t plane_stride,
+                        uint32_t box_cols, uint32_t box_rows, uint32_t box_planes) {
+  EncodeTiledFn fn = get_encode_fn();
+  if (fn == nullptr) return -1;
+  cuuint64_t dims[3] = {cols, rows, planes};
+  cuuint64_t strides[2] = {row_stride * 2, plane_stride * 2};
+  cuuint32_t box[3] = {box_cols, box_rows, box_planes};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -static_cast<int>(r) - 1000;
+}
+
 // 2-D row-major byte matrix [rows, cols] (e4m3 KV pages); box = {box_cols bytes (<= 128), box_rows}.
 int make_tmap_u8_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows,
                     uint32_t box_cols) {
