@@ -93,6 +93,11 @@ OGB_DEVICE float2 tf32_split(float x) {
   const float hi = tf32_round(x);
   return make_float2(hi, tf32_round(x - hi));
 }
+// The cheaper split: the leading 11 bits as they are, and the rest (of which a tf32 operand keeps the leading 11 again).
+OGB_DEVICE float2 tf32_cut(float x) {
+  const float hi = __uint_as_float(__float_as_uint(x) & 0xffffe000u);
+  return make_float2(hi, x - hi);
+}
 OGB_DEVICE void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1) {
   asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])

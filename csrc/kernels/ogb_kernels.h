@@ -196,9 +196,11 @@ int ogb_conv_unit_gates(const void* u, int ldu, const float* w, float* state, in
                         const float* dt_bias, float* qk, void* v, void* gates, int nk, int nv, int d, int dv, const int* ctx_len, const int* state_slot,
                         const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode, int num_tiles, int state_slots, int elem, int* status,
                         void* stream);
-// Gated delta rule over state [slots, heads, V, ogb_hgrn2_state_rows(D)].
+// Gated delta rule over state [slots, heads, V, ogb_hgrn2_state_rows(D)]; with scratch, prompts run in blocks on the tensor cores.
+int ogb_delta_block_floats(int heads, int groups, int D, int V);
 int ogb_delta_rule(const float* qk, const void* v, const void* gates, float* state, float* out, int heads, int groups, int D, int V, const int* ctx_len,
-                   const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int elem, int* status, void* stream);
+                   const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode, int num_prefill, int num_tiles,
+                   int num_slots, float* scratch, int elem, int* status, void* stream);
 // Differential attention over the pages of ogb_conv_rope_append (nk = 2 hkv maps); cu_q null: decode rows.
 int ogb_diff_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, const int* tile_seq,
                        const int* tile_q0, int rows, int num_tiles, int max_pages, int64_t num_pages, int64_t page_elems, int hq, int hkv, int d, int dv,

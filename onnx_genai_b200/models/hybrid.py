@@ -568,7 +568,8 @@ class HybridModel:
         qk, v = self._rows(self.unit_qk, t, 2 * m.kv_heads * m.dim), self._rows(self.unit_v, t, width)
         gates = self._rows(self.gates, t, 2 * m.heads).view(t, m.heads, 2)
         hops.conv_unit_gates(proj, w.conv, st["conv"], ab, w.a_log, w.dt_bias, qk, v, gates, si, m.kv_heads, m.heads, m.dim, m.vdim)
-        raw = hops.delta_rule(qk, v, gates, st["recurrent"], self._rows(self.rec_o, t, width), m.heads, m.kv_heads, m.dim, m.vdim, si)
+        raw = hops.delta_rule(qk, v, gates, st["recurrent"], self._rows(self.rec_o, t, width), m.heads, m.kv_heads, m.dim, m.vdim, si,
+                              blocks=h.dtype == torch.bfloat16, scratch=lambda name, shape: self._scratch(name, shape, torch.float32))
         attn = self._rows(self.attn, t, pad8(width))
         if pad8(width) != width:
             attn[:, width:].zero_()    # the buffer is shared with layers of other widths

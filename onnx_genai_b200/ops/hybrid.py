@@ -30,7 +30,8 @@ _native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, P, I, I, P])
 _native.register("ogb_norm_step", [P] * 8 + [F] + [I] * 6 + [L, I, P, P])
 _native.register("ogb_conv_rope_append", [P, I, P, P, P, I, P, I, P, P, P, L, L] + [I] * 8 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_conv_unit_gates", [P, I, P, P, I, P, I] + [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, P])
-_native.register("ogb_delta_rule", [P] * 5 + [I] * 4 + [P] * 3 + [I] * 4 + [P, P])
+_native.register("ogb_delta_rule", [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, I, P, P])
+_native.register("ogb_delta_block_floats", [I] * 4)
 _native.register("ogb_diff_attention", [P] * 8 + [I] * 3 + [L, L] + [I] * 10 + [F] * 4 + [I, P, P, P, I, P, P])
 _native.register("ogb_diff_set_tc", [I])
 _native.register("ogb_act_mul_packed", [P, P, I, I, I, I, I, P])
@@ -370,16 +371,23 @@ def conv_unit_gates(u, w, state, ab, a_log, dt_bias, qk, v, gates, si, nk, nv, d
 
 
 @_timed("delta_rule")
-def delta_rule(qk, v, gates, state, out, heads, groups, dim, vdim, si):
+def delta_rule(qk, v, gates, state, out, heads, groups, dim, vdim, si, blocks=False, scratch=None):
     """Advance the gated delta rule over the step's rows (inputs of :func:`conv_unit_gates`): state [slots, heads, vdim,
-    state_rows(dim)] fp32 in place, raw head outputs to out [T, heads * vdim] fp32."""
+    state_rows(dim)] fp32 in place, raw head outputs to out [T, heads * vdim] fp32.  ``blocks``: prompts in blocks of 64 tokens on
+    the tensor cores, fp32 factors split in two tf32 terms; ``scratch(name, shape)`` provides fp32 scratch for them."""
     if not qk.is_cuda:
         reference.delta_rule(qk, v, gates, state, out, heads, groups, dim, vdim, si)
         return out
     assert out.is_contiguous()
-    rc = _native.load().ogb_delta_rule(qk.data_ptr(), v.data_ptr(), gates.data_ptr(), state.data_ptr(), out.data_ptr(), heads, groups, dim, vdim,
-                                       si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(), si.num_decode, si.num_prefill_seqs,
-                                       state.shape[0], _ELEM[v.dtype], status_word().data_ptr(), _stream())
+    lib, work = _native.load(), None
+    per_block = lib.ogb_delta_block_floats(heads, groups, dim, vdim) if blocks and si.num_prefill_seqs else 0
+    if per_block:
+        n = si.num_tiles * per_block
+        work = scratch("delta_blocks", (n,)) if scratch is not None else torch.empty(n, dtype=torch.float32, device=qk.device)
+    rc = lib.ogb_delta_rule(qk.data_ptr(), v.data_ptr(), gates.data_ptr(), state.data_ptr(), out.data_ptr(), heads, groups, dim, vdim,
+                            si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(),
+                            si.num_decode, si.num_prefill_seqs, si.num_tiles, state.shape[0], _ptr(work), _ELEM[v.dtype], status_word().data_ptr(),
+                            _stream())
     _native.check(rc, "ogb_delta_rule")
     launch_counts["delta_rule"] += 1
     return out

@@ -194,9 +194,13 @@ LONG = [(7, 1), (0, 1), (30, 2), (0, 2), (0, 16), (5, 17), (64, 64), (1, 130), (
 @pytest.mark.parametrize("heads,groups,dim,vdim", [(2, 1, 44, 56), (3, 3, 20, 36), (1, 1, 64, 10), (4, 2, 128, 130), (1, 1, 200, 33), (4, 1, 100, 32), (2, 2, 256, 140),
                                                    (2, 2, 128, 128), (6, 2, 64, 64)])
 @pytest.mark.parametrize("kind", ["plain", "fast", "closed"])
-def test_delta_rule(where, heads, groups, dim, vdim, kind):
-    """``fast``: decays near zero; ``closed``: no decay and full steps, keys that repeat (every write replaces one)."""
+@pytest.mark.parametrize("blocks", [False, True])
+def test_delta_rule(where, heads, groups, dim, vdim, kind, blocks):
+    """``fast``: decays near zero; ``closed``: no decay and full steps, keys that repeat (every write replaces one).  ``blocks``:
+    prompts in blocks on the tensor cores, as exact as the steps."""
     device, dt = where
+    if device == "cpu" and blocks:
+        pytest.skip("a variant of the CUDA kernel")
     g = torch.Generator().manual_seed(dim)
     si, order, _ = step_of(LONG, device)
     t = si.num_tokens
@@ -214,7 +218,7 @@ def test_delta_rule(where, heads, groups, dim, vdim, kind):
     start = torch.randn(len(order), heads, vdim, rows, generator=g)
     start[..., dim:] = 0
     state, out = start.to(device).clone(), torch.zeros(t, heads * vdim, device=device)
-    H.delta_rule(qk.reshape(t, -1).to(device), v.to(device), gates.to(device), state, out, heads, groups, dim, vdim, si)
+    H.delta_rule(qk.reshape(t, -1).to(device), v.to(device), gates.to(device), state, out, heads, groups, dim, vdim, si, blocks=blocks)
     for e, slot, b, a, n in entries(si, order):
         for h in range(heads):
             q, k = (qk[b:b + n, i, h // (heads // groups)].double() for i in range(2))
