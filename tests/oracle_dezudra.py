@@ -203,7 +203,7 @@ def random_tensors(cfg, seed=0, sharp=2.0):
             for n, rows, s in (("q", 2 * H * d, sharp), ("k", 2 * G * d, 1.0), ("v", G * dv, 1.0)):
                 t[x + n], t[x + n + ".b"], t[x + n + ".conv"] = lin(rows, w, s), 0.3 * torch.randn(rows, generator=g), taps(rows)
             for n in ("lq1", "lk1", "lq2", "lk2"):
-                t[x + n] = torch.randn(d, generator=g) * 0.5 / d ** 0.25
+                t[x + n] = torch.randn(d, generator=g) * 0.35 / d ** 0.25
         else:
             for n, rows in (("q", G * d), ("k", G * d), ("v", H * dv)):
                 t[x + n], t[x + n + ".conv"] = lin(rows, w, 1.5), taps(rows)

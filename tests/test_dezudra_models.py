@@ -40,10 +40,11 @@ def models():
 
 
 def model_for(models, name, where):
-    """In bf16 every expert is used: rounding could otherwise tip a close choice (choosing is tested on fixed logits)."""
+    """In bf16 every expert is used, since rounding could tip a close choice (choosing is tested on fixed logits), and attention is
+    less sharp, which magnifies rounding less."""
     cfg, tensors = models[name]
     if where[1] == "bf16":
-        cfg = json.loads(json.dumps(cfg))
+        cfg, tensors = json.loads(json.dumps(cfg)), O.random_tensors(cfg, seed=40, sharp=1.0)
         for layer in cfg["layers"]:
             if layer["mlp"]:
                 r = layer["mlp"]["router"]
