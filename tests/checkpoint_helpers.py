@@ -29,12 +29,16 @@ def tokens_of(cfg, n, seed):
     return np.random.default_rng(seed).integers(0, cfg["vocab"], n).tolist()
 
 
-def assert_logits(got, want, where):
+def assert_logits(got, want, where, outliers=0.0):
     """Root mean square of every row's difference against the spread of the logits.  The 32-bit engine is the sharp test; in
-    bf16 the bound is what rounding leaves in these sharply weighted models, far below what one wrong key or state costs."""
+    bf16 the bound is what rounding leaves in these sharply weighted models, far below what one wrong key or state costs.
+    ``outliers``: share of rows that bf16 may leave up to three times further away (designs that norm a head's output, which
+    magnifies rounding where that output is next to nothing)."""
     err = (got.double() - want).pow(2).mean(-1).sqrt() / want.std()
     worst, mean = (0.12, 0.04) if where[1] == "bf16" else (1e-4, 2e-5)
-    assert err.max() < worst and err.mean() < mean, (float(err.max()), float(err.mean()), int(err.argmax()))
+    over = (err >= worst).sum() if where[1] == "bf16" and outliers else 0
+    top = 3 * worst if over else worst
+    assert err.max() < top and over <= max(1.0, outliers * len(err)) and err.mean() < mean, (float(err.max()), float(err.mean()), int(err.argmax()))
 
 
 def replay_cuts(eng, tokens, cuts, name="a"):
