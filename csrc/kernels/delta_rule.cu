@@ -642,7 +642,7 @@ static int launch_delta_blocks(DeltaParams p, const DeltaBlocks& bl, int entries
   if (rc != 0) return rc;
   p.z0 = p.sr.num_decode;
   // narrow slices put more SMs to work on few heads; wide ones read the shared operands less often
-  if (static_cast<long long>((p.V + 15) / 16) * p.heads * entries <= 148) return launch_delta_walk<DP, 16>(p, bl, entries, stream);
+  if (static_cast<long long>((p.V + 15) / 16) * p.heads * entries <= ogb_num_sms()) return launch_delta_walk<DP, 16>(p, bl, entries, stream);
   return launch_delta_walk<DP, 32>(p, bl, entries, stream);
 }
 

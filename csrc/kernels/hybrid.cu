@@ -381,7 +381,7 @@ OGB_DEVICE float silu_f32(float z) { return z / (1.f + expf(-z)); }
 
 template <typename T>
 __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, T* __restrict__ out,
-                                                           int rows, int heads, int n, int ldx, int ldo, const T* __restrict__ gate, int ldg) {
+                                                           int rows, int heads, int n, int ldx, int ldo, const T* __restrict__ gate, int ldg, bool vec) {
   const int lane = threadIdx.x & 31;
   const long long g = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   if (g >= static_cast<long long>(rows) * heads) return;
@@ -390,7 +390,7 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restri
   T* dst = out + static_cast<size_t>(t) * ldo + static_cast<size_t>(h) * n;
   const T* gt = gate != nullptr ? gate + static_cast<size_t>(t) * ldg + static_cast<size_t>(h) * n : nullptr;
   float ss = 0.f;
-  if ((n & 127) == 0 && n <= 512 && ((ldx | ldo | ldg) & 3) == 0) {
+  if (vec) {                                   // rows and heads of x, out and gate start on four elements; n is 128 .. 512 in steps of 128
     float v[4][4];
     const int per = n >> 7;
 #pragma unroll
@@ -522,7 +522,10 @@ extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const floa
   if (rows <= 0) return 0;
   if (W < 1 || (y != nullptr && post == nullptr) || (h != nullptr && w == nullptr) || (pos != nullptr && (weight == nullptr || k < 1))) return -3;
   NormStepParams p{x, y, pos, weight, post, w, h, gather, eps, rows, total_rows, W, k, ldy, ldh, y_rows, status};
-  const bool vec = ((W | ldy | ldh) & 3) == 0;
+  // four elements at a time need rows that start on them, and pointers too
+  const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h);
+  const uintptr_t f32 = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(post) | reinterpret_cast<uintptr_t>(w);
+  const bool vec = ((W | ldy | ldh) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (elem == kElemBF16) return vec ? launch_norm_step<__nv_bfloat16, 4>(p, s) : launch_norm_step<__nv_bfloat16, 1>(p, s);
   if (elem == kElemF32) return vec ? launch_norm_step<float, 4>(p, s) : launch_norm_step<float, 1>(p, s);
@@ -560,10 +563,14 @@ extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void*
   if (rows <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * heads + 7) / 8);
-  if (elem == kElemBF16) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo,
-                                                                           static_cast<const __nv_bfloat16*>(gate), ldg);
-  else if (elem == kElemF32) head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo,
-                                                                              static_cast<const float*>(gate), ldg);
+  const uintptr_t unaligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) |
+                              ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(gate)) & (elem == kElemBF16 ? 7 : 15));
+  const bool vec = (n & 127) == 0 && n <= 512 && ((ldx | ldo | ldg) & 3) == 0 && unaligned == 0;
+  if (elem == kElemBF16)
+    head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo,
+                                               static_cast<const __nv_bfloat16*>(gate), ldg, vec);
+  else if (elem == kElemF32)
+    head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo, static_cast<const float*>(gate), ldg, vec);
   else return -3;
   return static_cast<int>(cudaGetLastError());
 }

@@ -300,16 +300,24 @@ static int launch_unit(const UnitParams& p, cudaStream_t stream) {
   return static_cast<int>(cudaGetLastError());
 }
 
+// four channels at a time: their places in the projected row, the filters and the outputs start on four elements
+template <typename T>
+static bool conv_aligned(const ConvIn& in, const void* out0, const void* out1, int sizes) {
+  const uintptr_t act = reinterpret_cast<uintptr_t>(in.u) | reinterpret_cast<uintptr_t>(out0) | reinterpret_cast<uintptr_t>(out1);
+  const uintptr_t f32 = reinterpret_cast<uintptr_t>(in.w) | reinterpret_cast<uintptr_t>(in.bias) | reinterpret_cast<uintptr_t>(in.state);
+  return ((sizes | in.ldu) & 3) == 0 && (f32 & 15) == 0 && (act & (4 * sizeof(T) - 1)) == 0;
+}
+
 template <typename T>
 static int dispatch_rope(const RopeParams& p, cudaStream_t s) {
   const int half = p.rot / 2;
-  const bool vec = ((half | p.d | p.dv | p.in.ldu) & 3) == 0;
+  const bool vec = conv_aligned<T>(p.in, p.q, p.pool, half | p.d | p.dv);
   if (p.in.taps <= 4) return vec ? launch_rope<T, 4, 4>(p, s) : launch_rope<T, 1, 4>(p, s);
   return vec ? launch_rope<T, 4, 8>(p, s) : launch_rope<T, 1, 8>(p, s);
 }
 template <typename T>
 static int dispatch_unit(const UnitParams& p, cudaStream_t s) {
-  const bool vec = ((p.d | p.dv | p.in.ldu) & 3) == 0;
+  const bool vec = conv_aligned<T>(p.in, p.v, nullptr, p.d | p.dv) && (reinterpret_cast<uintptr_t>(p.qk) & 15) == 0;
   if (p.in.taps <= 4) {
     if (!vec) return launch_unit<T, 1, 4, 8>(p, s);
     return p.d <= 128 ? launch_unit<T, 4, 4, 1>(p, s) : launch_unit<T, 4, 4, 2>(p, s);

@@ -127,13 +127,13 @@ def kernel_rows(size: str, timer, pk):
         # delta rule
         c = (2 * dg + dh) * DV
         wd, wab, ud, ab = rnd(c + dh * DV, hid), rnd(2 * dh, hid), empty(t, c + dh * DV), empty(t, 2 * dh, dtype=torch.float32)
-        row("gemm q|k|v|gate", phase, lambda: hops.linear(h, wd, ud), 2 * t * wd.shape[0] * hid, (wd.shape[0] + t) * hid * 2 + t * wd.shape[0] * 2)
+        row("gemm gate|q|k|v", phase, lambda: hops.linear(h, wd, ud), 2 * t * wd.shape[0] * hid, (wd.shape[0] + t) * hid * 2 + t * wd.shape[0] * 2)
         row("gemm decay|step (fp32 out)", phase, lambda: hops.linear(h, wab, ab, f32_out=True), 2 * t * 2 * dh * hid, (2 * dh + t) * hid * 2 + t * 2 * dh * 4)
         ud.normal_()
         cd, sd = f32(TAPS, c), torch.zeros(nseq, TAPS - 1, c, device="cuda")
         qk, v, gates = empty(t, 2 * dg * DV, dtype=torch.float32), empty(t, dh * DV), empty(t, dh, 2, dtype=torch.float32)
         al, dt = -f32(dh), f32(dh) - 3
-        row("conv_unit_gates", phase, lambda: hops.conv_unit_gates(ud, cd, sd, ab, al, dt, qk, v, gates, si, dg, dh, DV, DV),
+        row("conv_unit_gates", phase, lambda: hops.conv_unit_gates(ud[:, dh * DV:], cd, sd, ab, al, dt, qk, v, gates, si, dg, dh, DV, DV),
             nbytes=t * (c * 2 + 2 * dg * DV * 4 + dh * DV * 2 + dh * 16) + 2 * nseq * (TAPS - 1) * c * 4)
         rec, raw = torch.zeros(nseq, dh, DV, DV, device="cuda"), empty(t, dh * DV, dtype=torch.float32)
         work: dict = {}
@@ -149,7 +149,7 @@ def kernel_rows(size: str, timer, pk):
         b2, lo = f32(dh * DV) * 2, f32(dh * DV) * 0.5
         row("like: hgrn2", phase, lambda: hops.hgrn2(qfv, b2, lo, rec, raw, dh, DV, DV, si, split=True), nbytes=t * dh * DV * 16 + 2 * nseq * dh * DV * DV * 4)
         nw, gated = f32(DV), empty(t, dh * DV)
-        row("head_rmsnorm * gate", phase, lambda: hops.head_rmsnorm(raw, nw, 1e-6, gated, dh, DV, gate=ud[:, c:]), nbytes=t * dh * DV * 8)
+        row("head_rmsnorm * gate", phase, lambda: hops.head_rmsnorm(raw, nw, 1e-6, gated, dh, DV, gate=ud[:, :dh * DV]), nbytes=t * dh * DV * 8)
         row("like: head_rmsnorm", phase, lambda: hops.head_rmsnorm(raw, nw, 1e-6, gated, dh, DV), nbytes=t * dh * DV * 6)
         # experts
         wr, logits = rnd(e, hid), empty(t, e, dtype=torch.float32)

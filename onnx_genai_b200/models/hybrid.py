@@ -8,7 +8,7 @@ a layer to a fixed list of launches over buffers allocated once:
     hyper_step (fold the last sublayer's output into the streams, read-out, norm, token shift), or
     norm_step  (x += norm(the last sublayer's output), norm; sums the rows of routed experts on the way)
     recurrent:  gemm(q | gate | v, fp32 out) | hgrn2 | head_rmsnorm | gemm(o)
-    delta:      gemm(q | k | v | gate) | gemm(decay | step size, fp32 out) | conv_unit_gates | delta_rule | head_rmsnorm * gate | gemm(o)
+    delta:      gemm(gate | q | k | v) | gemm(decay | step size, fp32 out) | conv_unit_gates | delta_rule | head_rmsnorm * gate | gemm(o)
     latent:     gemm(q | latent) | latent_append | gemm per head (W_uk^T q) | latent_attention | gemm per head (W_uv o) | gemm(o);
                 prompts over wide latents: latent_gather | gemm (K | V pages) | paged_prefill | gemm(o)
     diff:       gemm(q | k | v) | conv_rope_append | diff_attention (both maps, difference and norm) | gemm(o)
@@ -276,7 +276,7 @@ class LatentWeights:
 
 @dataclass
 class DeltaWeights:
-    qkvg: torch.Tensor       # [conv_width + heads * vdim, hidden]: query, key, value and output-gate projections
+    gqkv: torch.Tensor       # [heads * vdim + conv_width, hidden]: output-gate, query, key and value projections
     ab: torch.Tensor         # [2 * heads, hidden]: decay and step-size projections
     conv: torch.Tensor       # fp32 [taps, conv_width]
     a_log: torch.Tensor      # fp32 [heads]
@@ -368,7 +368,7 @@ def pack_latent(spec: LatentSpec, q, dkv, dkv_norm, uk, uv, o) -> LatentWeights:
 def pack_delta(spec: DeltaSpec, q, k, v, g, a, b, conv, a_log, dt_bias, norm, o) -> DeltaWeights:
     """``conv``: filters of the q, k and v channels, [channels, taps] each."""
     f32 = lambda t: t.float().contiguous()
-    return DeltaWeights(qkvg=pad_cols(torch.cat([q, k, v, g], 0)), ab=pad_cols(torch.cat([a, b], 0)), conv=f32(torch.cat(conv, 0).t()), a_log=f32(a_log),
+    return DeltaWeights(gqkv=pad_cols(torch.cat([g, q, k, v], 0)), ab=pad_cols(torch.cat([a, b], 0)), conv=f32(torch.cat(conv, 0).t()), a_log=f32(a_log),
                         dt_bias=f32(dt_bias), norm=f32(norm), o=pad_cols(o))
 
 
@@ -562,18 +562,18 @@ class HybridModel:
     def _delta(self, li, m: DeltaSpec, w: DeltaWeights, h, y, si):
         t, width, st = h.shape[0], m.heads * m.vdim, self.state.layers[li]
         proj = self._rows(self.proj, t, pad8(m.conv_width + width))
-        hops.linear(h, w.qkvg, proj[:, : m.conv_width + width])
+        hops.linear(h, w.gqkv, proj[:, : m.conv_width + width])
         ab = self._rows(self.ab, t, pad8(2 * m.heads))
         hops.linear(h, w.ab, ab[:, : 2 * m.heads], f32_out=True)
         qk, v = self._rows(self.unit_qk, t, 2 * m.kv_heads * m.dim), self._rows(self.unit_v, t, width)
         gates = self._rows(self.gates, t, 2 * m.heads).view(t, m.heads, 2)
-        hops.conv_unit_gates(proj, w.conv, st["conv"], ab, w.a_log, w.dt_bias, qk, v, gates, si, m.kv_heads, m.heads, m.dim, m.vdim)
+        hops.conv_unit_gates(proj[:, width:], w.conv, st["conv"], ab, w.a_log, w.dt_bias, qk, v, gates, si, m.kv_heads, m.heads, m.dim, m.vdim)
         raw = hops.delta_rule(qk, v, gates, st["recurrent"], self._rows(self.rec_o, t, width), m.heads, m.kv_heads, m.dim, m.vdim, si,
                               blocks=h.dtype == torch.bfloat16, scratch=lambda name, shape: self._scratch(name, shape, torch.float32))
         attn = self._rows(self.attn, t, pad8(width))
         if pad8(width) != width:
             attn[:, width:].zero_()    # the buffer is shared with layers of other widths
-        hops.head_rmsnorm(raw, w.norm, self.cfg.norm_eps, attn, m.heads, m.vdim, gate=proj[:, m.conv_width:m.conv_width + width])
+        hops.head_rmsnorm(raw, w.norm, self.cfg.norm_eps, attn, m.heads, m.vdim, gate=proj[:, :width])
         hops.linear(attn, w.o, y)
 
     def _diff(self, li, m: DiffSpec, w: DiffWeights, h, y, kv, si):

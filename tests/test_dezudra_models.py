@@ -31,7 +31,10 @@ RECURRENT = O.make_config(64, 64, [O.layer_delta(4, 1, 16, 16, X(4, 2, 64, 2, 2)
 WIDE = O.make_config(80, 128, [O.layer_attention(8, 2, 64, 128, 70, 33, X(8, 2, 128, 4, 2)), O.layer_attention(16, 1, 32, 64, 128, 0, X(4, 1, 64)),
                                O.layer_delta(4, 2, 128, 128, X(8, 4, 64, 2, 2)), O.layer_attention(2, 2, 128, 128, 200, 16, None, rot=64),
                                O.layer_attention(3, 1, 96, 192, 45, 7, None)])
-CONFIGS = {"mixed": MIXED, "odd": ODD, "recurrent": RECURRENT, "wide": WIDE}
+# heads in steps of the vector width beside key widths and channel counts that are not
+UNEVEN = O.make_config(70, 68, [O.layer_delta(3, 3, 7, 128, X(4, 2, 20, 2, 1), conv=3), O.layer_attention(2, 1, 9, 64, 30, 6, X(3, 1, 12), rot=4, conv=4),
+                                O.layer_delta(2, 1, 64, 9, None, conv=5), O.layer_attention(9, 3, 64, 20, 18, 2, None, rot=22)])
+CONFIGS = {"mixed": MIXED, "odd": ODD, "recurrent": RECURRENT, "wide": WIDE, "uneven": UNEVEN}
 WHERE = [("cpu", torch.float32), pytest.param(("cuda", torch.float32), marks=GPU), pytest.param(("cuda", torch.bfloat16), marks=GPU)]
 
 
