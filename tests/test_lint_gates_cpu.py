@@ -31,7 +31,8 @@ def _sources(exts, roots=("onnx_genai_b200", "csrc", "tests", "examples")):
 
 def test_every_kernel_entry_point_in_the_header_is_bound_with_the_same_arity():
     from onnx_genai_b200.ops import _native
-    import onnx_genai_b200.ops.moe  # noqa: F401  (registers its entry points)
+    import onnx_genai_b200.ops.hybrid  # noqa: F401  (registers its entry points)
+    import onnx_genai_b200.ops.moe  # noqa: F401
     import onnx_genai_b200.ops.quant  # noqa: F401
     import onnx_genai_b200.ops.sequence  # noqa: F401
     import onnx_genai_b200.utils.vmm  # noqa: F401
