@@ -82,6 +82,10 @@ struct AttnParams {
   int kv_fmt;               // one-byte pages only: 0 = e4m3, 1 = int8
   unsigned long long* dbg;  // optional (tcgen05 prefill): per-role wait / work nanoseconds of the CTA (dbg_tile, head 0)
   int dbg_tile;
+  // pages in 64-column chunks (tcgen05 prefill): columns between the heads of q and of out, value columns that are stored, and a gate
+  int q_head, o_head, d_v;
+  const __nv_bfloat16* gate;   // [rows, ldg] or null: a head's output is multiplied by the sigmoid of its column
+  int ldg;
 };
 
 // Sliding window with attention sinks (the retention policy of crates/onnx-genai-kv/src/paged_cache.rs:483-585, done

@@ -43,24 +43,26 @@ constexpr int kFaThreads = (kFaFirstSoftmaxWarp + kFaSoftmaxWarps) * 32;
 // range of bf16 and of the fp32 sums, and the quotient O / l does not depend on the centre.
 constexpr float kFaRecentre = 24.f;
 
-template <int D, int BN>
+template <int DK, int DV, int BN>
 struct FaCfg {
-  static constexpr int kHalves = D / 64;
-  static constexpr int kQBytes = kFaBM * D * 2;
-  static constexpr int kKvBytes = BN * D * 2;          // one K or one V block
+  static constexpr int kHalvesK = DK / 64, kHalvesV = DV / 64;
+  static constexpr int kQBytes = kFaBM * DK * 2;
+  static constexpr int kKBytes = BN * DK * 2;          // one K block
+  static constexpr int kVBytes = BN * DV * 2;          // one V block
   static constexpr int kHalfStrideQ = kFaBM * 128;     // bytes between the 64-dim halves of Q
   static constexpr int kHalfStrideKv = BN * 128;       // bytes between the 64-dim halves of a K / V block
   static constexpr int kStages = 2;
-  static constexpr int kSmemBytes = kQBytes + kStages * 2 * kKvBytes + 1024 /*alignment*/ + 512 /*barriers*/ +
+  static constexpr int kSmemBytes = kQBytes + kStages * (kKBytes + kVBytes) + 1024 /*alignment*/ + 512 /*barriers*/ +
                                     2 * kFaBM * 8 /*(m, l) of both groups*/;
   // TMEM columns: O_A | O_B | S0 (P0 over its first 64 columns) | S1 (P1)
   static constexpr int kColO = 0;
-  static constexpr int kColS = 2 * D;
+  static constexpr int kColS = 2 * DV;
   static constexpr int kTmemCols = 512;
-  static constexpr int kXPitch = (D / 2 + 4) * 4;      // bytes per row of the accumulator halves exchanged in the epilogue
-  static_assert(2 * D + 2 * BN <= 512, "TMEM budget");
+  static constexpr int kXPitch = (DV / 2 + 4) * 4;      // bytes per row of the accumulator halves exchanged in the epilogue
+  static_assert(2 * DV + 2 * BN <= 512, "TMEM budget");
+  static_assert(kSmemBytes <= 227 * 1024, "shared memory");
   static_assert(BN == 128, "a row of scores is processed as two 64-column chunks");
-  static_assert(2 * kFaBM * kXPitch <= kStages * 2 * kKvBytes, "the exchange slab reuses the K/V rings");
+  static_assert(2 * kFaBM * kXPitch <= kStages * (kKBytes + kVBytes), "the exchange slab reuses the K/V rings");
 };
 
 // Optional stamps: when p.dbg is set, the CTA (dbg_tile, head 0) accumulates, per role, the nanoseconds spent
@@ -145,17 +147,19 @@ OGB_DEVICE float fa_max_chunk(uint32_t s_addr, int hi, int lo) {
   return fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
 }
 
-template <int D, int BN>
+// CHUNKED: pages are [16 tokens][64 columns] chunks, the DK / 64 of a head's keys and then the DV / 64 of its values, head by head;
+// otherwise [kv_heads][K | V][16][D] with DK = DV = D.
+template <int DK, int DV, int BN, bool CHUNKED>
 __global__ void __launch_bounds__(kFaThreads, 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
                         const AttnParams p) {
-  using Cfg = FaCfg<D, BN>;
+  using Cfg = FaCfg<DK, DV, BN>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
-  uint8_t* sK = sQ + Cfg::kQBytes;                      // [stage][kKvBytes]
-  uint8_t* sV = sK + Cfg::kStages * Cfg::kKvBytes;      // [stage][kKvBytes]
-  FaBars* bars = reinterpret_cast<FaBars*>(sV + Cfg::kStages * Cfg::kKvBytes);
+  uint8_t* sK = sQ + Cfg::kQBytes;                      // [stage][kKBytes]
+  uint8_t* sV = sK + Cfg::kStages * Cfg::kKBytes;       // [stage][kVBytes]
+  FaBars* bars = reinterpret_cast<FaBars*>(sV + Cfg::kStages * Cfg::kVBytes);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float2* x_ml = reinterpret_cast<float2*>(reinterpret_cast<uint8_t*>(bars) + 512);   // [group][row] (m, l)
@@ -218,15 +222,15 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
       if (!is_v) {
         mbar_expect_tx(&bars->q_full, Cfg::kQBytes);
 #pragma unroll
-        for (int h = 0; h < Cfg::kHalves; ++h)
-          tma_load_2d(sQ + h * Cfg::kHalfStrideQ, &q_map, &bars->q_full, head * D + h * 64, q_begin + q0);
+        for (int h = 0; h < Cfg::kHalvesK; ++h)
+          tma_load_2d(sQ + h * Cfg::kHalfStrideQ, &q_map, &bars->q_full, head * (CHUNKED ? p.q_head : DK) + h * 64, q_begin + q0);
       }
       const int n_pages = (ctx + kPageTokens - 1) / kPageTokens;
       const int* table = p.page_table + static_cast<size_t>(seq) * p.max_pages;
       uint64_t* full = is_v ? bars->v_full : bars->k_full;
       uint64_t* empty = is_v ? bars->v_empty : bars->k_empty;
       uint8_t* ring = is_v ? sV : sK;
-      const int row_add = is_v ? kPageTokens : 0;
+      const int kv_bytes = is_v ? Cfg::kVBytes : Cfg::kKBytes;
       for (int it = 0; it < nblk && ok; ++it) {
         const int b = b_begin + it;
         const int buf = it & 1;
@@ -243,19 +247,22 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
             atomicOr(p.status, kStatusIndexOutOfRange);
             page = 0;
           }
-          row_of_page[i] = static_cast<int>(((page * p.hkv + kvh) * 2) * kPageTokens) + row_add;
+          row_of_page[i] = CHUNKED ? static_cast<int>(((page * p.hkv + kvh) * (Cfg::kHalvesK + Cfg::kHalvesV) + (is_v ? Cfg::kHalvesK : 0)) * kPageTokens)
+                                   : static_cast<int>(((page * p.hkv + kvh) * 2 + (is_v ? 1 : 0)) * kPageTokens);
         }
         st.begin();
         if (!fa_wait(&empty[buf], par ^ 1, abort_flag)) { ok = false; break; }
         st.end(4);
         st.begin();
-        mbar_expect_tx(&full[buf], Cfg::kKvBytes);
-        uint8_t* dst = ring + buf * Cfg::kKvBytes;
+        mbar_expect_tx(&full[buf], kv_bytes);
+        uint8_t* dst = ring + buf * kv_bytes;
 #pragma unroll
         for (int i = 0; i < BN / kPageTokens; ++i) {
 #pragma unroll
-          for (int h = 0; h < Cfg::kHalves; ++h)
-            tma_load_2d(dst + h * Cfg::kHalfStrideKv + (i << 11), &kv_map, &full[buf], h * 64, row_of_page[i]);
+          for (int h = 0; h < (Cfg::kHalvesK > Cfg::kHalvesV ? Cfg::kHalvesK : Cfg::kHalvesV); ++h)
+            if (h < (is_v ? Cfg::kHalvesV : Cfg::kHalvesK))
+              tma_load_2d(dst + h * Cfg::kHalfStrideKv + (i << 11), &kv_map, &full[buf], CHUNKED ? 0 : h * 64,
+                          row_of_page[i] + (CHUNKED ? h * kPageTokens : 0));
         }
         st.end(5);
       }
@@ -267,7 +274,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
     // overwrite the columns of P_j (which live inside score buffer j & 1) before that product has read them.
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc_bf16(kFaBM, BN);
-      constexpr uint32_t idesc_o = make_idesc_bf16(kFaBM, D) | (1u << 16);   // B (= V) is MN-major
+      constexpr uint32_t idesc_o = make_idesc_bf16(kFaBM, DV) | (1u << 16);   // B (= V) is MN-major
       bool ok = fa_wait(&bars->q_full, 0, abort_flag);
       FaStamp st{dbg, 0};
       auto issue_pv = [&](int t) -> bool {
@@ -280,9 +287,9 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
         if (!fa_wait(&bars->v_full[buf], par, abort_flag)) return false;
         st.end(9);
         tc_fence_after();
-        const uint32_t sv = smem_u32(sV + buf * Cfg::kKvBytes);
+        const uint32_t sv = smem_u32(sV + buf * Cfg::kVBytes);
         const uint32_t p_addr = tmem_base + Cfg::kColS + buf * BN;            // P_t: first BN/2 columns of score buffer t & 1
-        const uint32_t o_addr = tmem_base + Cfg::kColO + buf * D;            // accumulator of the group that owns block t
+        const uint32_t o_addr = tmem_base + Cfg::kColO + buf * DV;           // accumulator of the group that owns block t
 #pragma unroll
         for (int k = 0; k < BN / 16; ++k) {
           const uint64_t db = make_mnmajor_sw128_desc(sv + k * 2048, Cfg::kHalfStrideKv);
@@ -300,10 +307,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
         st.end(6);
         tc_fence_after();
         const uint32_t sq = smem_u32(sQ);
-        const uint32_t sk = smem_u32(sK + buf * Cfg::kKvBytes);
+        const uint32_t sk = smem_u32(sK + buf * Cfg::kKBytes);
         const uint32_t s_addr = tmem_base + Cfg::kColS + buf * BN;
 #pragma unroll
-        for (int h = 0; h < Cfg::kHalves; ++h) {
+        for (int h = 0; h < Cfg::kHalvesK; ++h) {
           const uint64_t da = make_kmajor_sw128_desc(sq + h * Cfg::kHalfStrideQ);
           const uint64_t db = make_kmajor_sw128_desc(sk + h * Cfg::kHalfStrideKv);
 #pragma unroll
@@ -323,7 +330,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
     const int row = q * 32 + lane;                       // query row of this thread
     const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
     const uint32_t s_addr = lane_base + Cfg::kColS + g * BN;
-    const uint32_t o_addr = lane_base + Cfg::kColO + g * D;
+    const uint32_t o_addr = lane_base + Cfg::kColO + g * DV;
     const int qpos = pos0 + row;
     const int hi_abs = min(qpos, ctx - 1);
     const int lo_abs = (p.window > 0) ? (qpos - p.window + 1) : 0;
@@ -393,7 +400,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
             l_run *= alpha;
           }
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t o[32];
             tmem_ld_32x32(o_addr + 32 * c, o);
             tmem_ld_wait();
@@ -429,7 +436,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
     }
     st.begin();
     // ---- merge the two groups: each finalises one half of the columns ----
-    constexpr int OC = D / 2;
+    constexpr int OC = DV / 2;
     uint8_t* xo = sK;                                    // [group][row][OC floats], pitch kXPitch; the rings are idle by now
     asm volatile("bar.sync 1, 256;" ::: "memory");       // every tensor-core read of the rings has completed
     const bool live = ok && last >= 0;                   // this group accumulated something
@@ -456,10 +463,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
       const float w_mine = (m_mine == -INFINITY) ? 0.f : exp2f(m_mine - m_all);
       const float w_other = (other.x == -INFINITY) ? 0.f : exp2f(other.x - m_all);
       const float l_tot = (live ? l_run : 0.f) * w_mine + other.y * w_other;
-      const float inv = (l_tot > 0.f) ? 1.f / l_tot : 0.f;
+      float inv = (l_tot > 0.f) ? 1.f / l_tot : 0.f;
+      if (CHUNKED && p.gate != nullptr && row < rows)
+        inv *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(q_begin + q0 + row) * p.ldg + head])));
       const float a = w_mine * inv, b = w_other * inv;
       const float* src = reinterpret_cast<const float*>(xo + (static_cast<size_t>(g ^ 1) * kFaBM + row) * Cfg::kXPitch);
-      __nv_bfloat16* out = p.out + static_cast<size_t>(q_begin + q0 + row) * p.o_stride + head * D + g * OC;
+      __nv_bfloat16* out = p.out + static_cast<size_t>(q_begin + q0 + row) * p.o_stride + head * (CHUNKED ? p.o_head : DV) + g * OC;
 #pragma unroll
       for (int c = 0; c < OC / 32; ++c) {
         uint32_t o[32];
@@ -468,6 +477,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
         if (row < rows) {
 #pragma unroll
           for (int v = 0; v < 4; ++v) {
+            if (CHUNKED && g * OC + 32 * c + 8 * v >= p.d_v) continue;
             float r[8];
             const uint4 x0 = *reinterpret_cast<const uint4*>(src + 32 * c + 8 * v);
             const uint4 x1 = *reinterpret_cast<const uint4*>(src + 32 * c + 8 * v + 4);
@@ -540,23 +550,25 @@ static int cached_tmap(const void* base, uint64_t rows, uint64_t cols, uint64_t 
   return 0;
 }
 
-template <int D>
+template <int DK, int DV, bool CHUNKED>
 static int launch_prefill_tc(const AttnParams& p, const void* pool, int q_rows, cudaStream_t stream) {
   constexpr int BN = 128;
-  using Cfg = FaCfg<D, BN>;
+  using Cfg = FaCfg<DK, DV, BN>;
   CUtensorMap q_map, kv_map;
-  int rc = cached_tmap(p.q, static_cast<uint64_t>(q_rows), static_cast<uint64_t>(p.hq) * D, static_cast<uint64_t>(p.q_stride),
+  int rc = cached_tmap(p.q, static_cast<uint64_t>(q_rows), static_cast<uint64_t>(p.hq) * (CHUNKED ? p.q_head : DK), static_cast<uint64_t>(p.q_stride),
                        kFaBM, &q_map);
   if (rc != 0) return rc;
-  rc = cached_tmap(pool, static_cast<uint64_t>(p.num_pages) * p.hkv * 2 * kPageTokens, D, D, kPageTokens, &kv_map);
+  const uint64_t page_rows = static_cast<uint64_t>(p.num_pages) * p.hkv * kPageTokens;
+  rc = CHUNKED ? cached_tmap(pool, page_rows * (Cfg::kHalvesK + Cfg::kHalvesV), 64, 64, kPageTokens, &kv_map)
+               : cached_tmap(pool, page_rows * 2, DV, DV, kPageTokens, &kv_map);
   if (rc != 0) return rc;
   static bool attr_set = false;
   if (!attr_set) {
-    OGB_CUDA_CHECK(cudaFuncSetAttribute(paged_prefill_tc_kernel<D, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(paged_prefill_tc_kernel<DK, DV, BN, CHUNKED>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
     attr_set = true;
   }
   dim3 grid(p.num_tiles, p.hq);
-  paged_prefill_tc_kernel<D, BN><<<grid, kFaThreads, Cfg::kSmemBytes, stream>>>(q_map, kv_map, p);
+  paged_prefill_tc_kernel<DK, DV, BN, CHUNKED><<<grid, kFaThreads, Cfg::kSmemBytes, stream>>>(q_map, kv_map, p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -594,6 +606,33 @@ extern "C" int ogb_paged_prefill_tc_bf16(const void* q, void* out, const void* p
   p.hq = hq; p.hkv = hkv; p.group = hq / hkv; p.q_stride = q_stride; p.o_stride = o_stride;
   p.scale_log2e = scale * 1.4426950408889634f; p.window = window; p.num_splits = 1; p.status = status;
   p.dbg = g_fa_dbg; p.dbg_tile = g_fa_dbg_tile;
-  return d == 128 ? launch_prefill_tc<128>(p, pool, q_rows, static_cast<cudaStream_t>(stream))
-                  : launch_prefill_tc<64>(p, pool, q_rows, static_cast<cudaStream_t>(stream));
+  return d == 128 ? launch_prefill_tc<128, 128, false>(p, pool, q_rows, static_cast<cudaStream_t>(stream))
+                  : launch_prefill_tc<64, 64, false>(p, pool, q_rows, static_cast<cudaStream_t>(stream));
+}
+
+// The same over pages of [heads][kc key chunks | vc value chunks][16][64] (keys and values expanded per head, each padded with zeros to
+// whole chunks): queries of q_head columns per head, dv value columns to columns o_head apart, times the sigmoid of gate [rows, ldg]
+// where it is given.  scale > 0.
+extern "C" int ogb_paged_prefill_chunks_bf16(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
+                                             const int* tile_seq, const int* tile_q0, const void* gate, int num_tiles, int num_seqs, int q_rows,
+                                             int max_pages, int64_t num_pages, int heads, int kc, int vc, int dv, int q_head, int o_head, int q_stride,
+                                             int o_stride, int ldg, float scale, int window, int* status, void* stream) {
+  if (num_tiles <= 0) return 0;
+  if (((q_head | o_head | q_stride | o_stride | dv) & 7) != 0 || q_rows <= 0 || dv > 64 * vc || q_head > 64 * kc || scale <= 0.f) return -3;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(pool)) & 15) return -4;
+  AttnParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.page_table = page_table; p.ctx_len = ctx_len; p.cu_q = cu_q; p.tile_seq = tile_seq; p.tile_q0 = tile_q0;
+  p.num_tiles = num_tiles; p.num_seqs = num_seqs; p.max_pages = max_pages; p.num_pages = num_pages;
+  p.hq = heads; p.hkv = heads; p.group = 1; p.q_stride = q_stride; p.o_stride = o_stride;
+  p.scale_log2e = scale * 1.4426950408889634f; p.window = window; p.num_splits = 1; p.status = status;
+  p.q_head = q_head; p.o_head = o_head; p.d_v = dv; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (kc == 1 && vc == 1) return launch_prefill_tc<64, 64, true>(p, pool, q_rows, s);
+  if (kc == 2 && vc == 1) return launch_prefill_tc<128, 64, true>(p, pool, q_rows, s);
+  if (kc == 2 && vc == 2) return launch_prefill_tc<128, 128, true>(p, pool, q_rows, s);
+  if (kc == 3 && vc == 1) return launch_prefill_tc<192, 64, true>(p, pool, q_rows, s);
+  if (kc == 3 && vc == 2) return launch_prefill_tc<192, 128, true>(p, pool, q_rows, s);
+  return -2;
 }

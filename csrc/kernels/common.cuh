@@ -16,6 +16,19 @@
 
 namespace ogb {
 
+// Activations between the two products of a feed-forward.  Gated ones take a gate g and an up value u, the others one value v; a and b
+// are numbers of the model.
+//   relu2      max(v, 0)^2
+//   clamp_glu  g' sigmoid(1.702 g') (u' + 1), g' = min(g, a), u' = clamp(u, -a, a)
+//   xielu      v / 2 + a v^2 for v > 0, v / 2 + b (exp(v) - 1 - v) otherwise
+enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2, kActRelu2 = 3, kActClampGlu = 4, kActXielu = 5 };
+struct ActArgs {
+  int kind = kActNone;
+  float a = 0.f, b = 0.f;
+};
+constexpr float kClampGluSlope = 1.702f;
+inline bool act_gated(int kind) { return kind == kActSilu || kind == kActGeluTanh || kind == kActClampGlu; }
+
 enum StatusBits : int {
   kStatusOk = 0,
   kStatusWaitTimeout = 1,      // a bounded mbarrier / flag wait ran out

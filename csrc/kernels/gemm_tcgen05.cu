@@ -46,12 +46,31 @@ constexpr int kGemmThreads = 192;
 constexpr int kGemmThreadsScatter = 224;  // + one warp that publishes finished tiles to peer GPUs
 
 enum GemmEpilogue : int { kEpiNone = 0, kEpiResidual = 1, kEpiSwiGLU = 2, kEpiScatter = 3 };
-enum GemmAct : int { kActSilu = 0, kActGeluTanh = 1, kActRelu2 = 2 };   // the gate of the gated epilogue; Relu2: every value of the plain one
 
-// 0.5 z (1 + tanh(a)) = z / (1 + exp(-2 a)); relative error of a few 1e-7, ahead of a bf16 rounding
+// Activations ahead of a bf16 rounding: relative errors of a few 1e-7, absolute ones of 1e-7 next to zero.
+// 0.5 z (1 + tanh(a)) = z / (1 + exp(-2 a))
 OGB_DEVICE float gelu_tanh_fast(float z) {
   const float a = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
   return z / (1.f + __expf(fminf(-2.f * a, 80.f)));
+}
+// the gated epilogue's value for a gate and an up column
+OGB_DEVICE float gated_act(const ActArgs& act, float g, float u) {
+  if (act.kind == kActGeluTanh) return gelu_tanh_fast(g) * u;
+  if (act.kind == kActClampGlu) {
+    g = fminf(g, act.a);
+    u = fminf(fmaxf(u, -act.a), act.a);
+    return g / (1.f + __expf(fminf(-kClampGluSlope * g, 80.f))) * (u + 1.f);
+  }
+  return g / (1.f + __expf(-g)) * u;
+}
+// the plain epilogue's value for a result
+OGB_DEVICE float plain_act(const ActArgs& act, float v) {
+  if (act.kind == kActRelu2) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  if (act.kind == kActXielu) return fmaf(0.5f, v, v > 0.f ? act.a * v * v : act.b * (__expf(v) - 1.f - v));
+  return v;
 }
 
 constexpr int kStagingPitch = 272;                       // bytes per staged row: 128 bf16 + 16 bytes of padding
@@ -158,7 +177,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                          const __nv_bfloat16* residual, float* __restrict__ C_f32, int M, int N, int K, int ldc, int ldr,
                          int* status, const TpScatter* __restrict__ sc, const int* __restrict__ group_tab,
                          const int* __restrict__ group_mtiles, uint32_t* a_ready, uint32_t* a_done, unsigned long long a_wait_ns,
-                         float* sk_ws, uint32_t* sk_flags, uint32_t sk_seq, const GemmBatch batch, const int act) {
+                         float* sk_ws, uint32_t* sk_flags, uint32_t sk_seq, const GemmBatch batch, const ActArgs act) {
   using Cfg = GemmCfg<BN>;
   const bool stream_k = sk_ws != nullptr;
   if constexpr (EPI == kEpiScatter) pdl_trigger();   // the exchange kernel may start: it waits on the tile counters this kernel bumps
@@ -414,8 +433,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
               for (int j = 0; j < 16; ++j) {
                 const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
                 const float u0 = __uint_as_float(u[2 * j]), u1 = __uint_as_float(u[2 * j + 1]);
-                o[j] = act == kActGeluTanh ? pack_bf16(gelu_tanh_fast(g0) * u0, gelu_tanh_fast(g1) * u1)
-                                           : pack_bf16(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
+                o[j] = pack_bf16(gated_act(act, g0, u0), gated_act(act, g1, u1));
               }
             } else {
               uint32_t r[32];
@@ -441,12 +459,9 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
                 }
               }
               if constexpr (EPI == kEpiNone)
-                if (act == kActRelu2) {
+                if (act.kind != kActNone) {
 #pragma unroll
-                  for (int j = 0; j < 32; ++j) {
-                    const float v = fmaxf(__uint_as_float(r[j]), 0.f);
-                    r[j] = __float_as_uint(v * v);
-                  }
+                  for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(plain_act(act, __uint_as_float(r[j])));
                 }
 #pragma unroll
               for (int j = 0; j < 16; ++j) o[j] = pack_bf16(__uint_as_float(r[2 * j]), __uint_as_float(r[2 * j + 1]));
@@ -787,7 +802,7 @@ static int launch_gemm(const void* A, const void* W, void* C, const void* bias, 
                        int N, int K, int lda, int ldw, int ldc, int ldr, int* status, cudaStream_t stream,
                        const TpScatter* sc = nullptr, const int* group_tab = nullptr, const int* group_mtiles = nullptr,
                        int experts = 1, int max_mtiles = 0, uint32_t* a_ready = nullptr, uint32_t* a_done = nullptr,
-                       unsigned long long a_wait_ns = 0, GemmBatch batch = GemmBatch(), int act = kActSilu) {
+                       unsigned long long a_wait_ns = 0, GemmBatch batch = GemmBatch(), ActArgs act = ActArgs()) {
   using Cfg = GemmCfg<BN>;
   CUtensorMap ta, tb;
   int rc = make_tmap_bf16_2d(&ta, A, M, static_cast<uint64_t>(batch.count - 1) * batch.a_step + K, lda, kBM, kBK);
@@ -869,7 +884,7 @@ extern "C" int ogb_gemm_bf16(const void* A, const void* W, void* C, const void* 
 
 static int gemm_bf16_dispatch(const void* A, const void* W, void* C, const void* bias, const void* residual, void* C_f32, int M, int N, int K,
                               int lda, int ldw, int ldc, int ldr, int epilogue, int bn, uint32_t* a_ready, uint32_t* a_done,
-                              unsigned long long a_wait_ns, GemmBatch batch, int act, int* status, void* stream_) {
+                              unsigned long long a_wait_ns, GemmBatch batch, ActArgs act, int* status, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (a_ready != nullptr && a_done == nullptr) return -8;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
@@ -915,15 +930,16 @@ extern "C" int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const v
                                   int M, int N, int K, int lda, int ldw, int ldc, int ldr, int epilogue, int bn,
                                   uint32_t* a_ready, uint32_t* a_done, unsigned long long a_wait_ns, int* status, void* stream_) {
   return gemm_bf16_dispatch(A, W, C, bias, residual, C_f32, M, N, K, lda, ldw, ldc, ldr, epilogue, bn, a_ready, a_done, a_wait_ns, GemmBatch(),
-                            kActSilu, status, stream_);
+                            ActArgs(), status, stream_);
 }
 
-// Gated product over a packed gate | up weight with the activation chosen by `act` (0 silu, 1 tanh form of gelu).
-extern "C" int ogb_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, int bn,
-                                   int* status, void* stream) {
-  if (act != kActSilu && act != kActGeluTanh) return -7;
-  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, kEpiSwiGLU, bn, nullptr, nullptr, 0, GemmBatch(), act,
-                            status, stream);
+// Product with an activation (common.cuh Act) and its two numbers: a gated one over a packed gate | up weight whose half-width is
+// bn / 2, or one of every result (bn 0: picked).
+extern "C" int ogb_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b,
+                                 int bn, int* status, void* stream) {
+  if (act < 0 || act > kActXielu) return -7;
+  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, act_gated(act) ? kEpiSwiGLU : kEpiNone, bn, nullptr, nullptr, 0,
+                            GemmBatch(), ActArgs{act, act_a, act_b}, status, stream);
 }
 
 // `batch` products of one shape (see GemmBatch): C[:, z*c_step : +N] = A[:, z*a_step : +K] * W[z*N : +N, :]^T.
@@ -931,7 +947,7 @@ extern "C" int ogb_gemm_bf16_batched(const void* A, const void* W, void* C, int 
                                      int a_step, int c_step, int* status, void* stream) {
   GemmBatch b;
   b.count = batch; b.a_step = a_step; b.c_step = c_step;
-  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, kEpiNone, 0, nullptr, nullptr, 0, b, kActSilu, status,
+  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, ldc, 0, kEpiNone, 0, nullptr, nullptr, 0, b, ActArgs(), status,
                             stream);
 }
 
@@ -941,7 +957,7 @@ extern "C" int ogb_gemm_bf16_paged(const void* A, const void* W, void* C, int M,
   if (page_d <= 0 || page_d % 8 != 0 || N % page_d != 0) return -9;
   GemmBatch b;
   b.page_d = page_d;
-  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, N, 0, kEpiNone, 0, nullptr, nullptr, 0, b, kActSilu, status, stream);
+  return gemm_bf16_dispatch(A, W, C, nullptr, nullptr, nullptr, M, N, K, lda, ldw, N, 0, kEpiNone, 0, nullptr, nullptr, 0, b, ActArgs(), status, stream);
 }
 
 // Row-parallel GEMM of a tensor-parallel group: the partial product A[M,K_local] * W[N,K_local]^T of
@@ -987,10 +1003,10 @@ extern "C" int ogb_gemm_bf16_scatter(const void* A, const void* W, int M, int N,
 // Grouped GEMM over experts (MoE): rows of A are sorted by expert; `group_tab` holds one int4 per
 // 128-row tile {expert, first row, end row, 0} and `group_mtiles` their count, both produced on the
 // device by ogb_moe_permute, so no routing information crosses to the host.  W is [experts, N, ldw].
-// epilogue 0 = plain (act 2: square of relu), 2 = SwiGLU over per-expert packed gate|up weights (output width N/2, N a multiple
-// of bn).  A tile that reaches past an expert's N rows of W computes columns that are not stored.
+// epilogue 0 = plain (with an activation of every result), 2 = gated over per-expert packed gate|up weights (output width N/2, N a
+// multiple of bn).  A tile that reaches past an expert's N rows of W computes columns that are not stored.
 static int grouped_gemm(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows,
-                        int max_mtiles, int N, int K, int lda, int ldw, int ldc, int epilogue, int act, int bn, int* status, cudaStream_t stream) {
+                        int max_mtiles, int N, int K, int lda, int ldw, int ldc, int epilogue, ActArgs act, int bn, int* status, cudaStream_t stream) {
   if (max_rows <= 0 || experts <= 0) return 0;
   if ((K % 8) != 0 || (lda % 8) != 0 || (ldw % 8) != 0 || (ldc % 8) != 0) return -3;
   if (epilogue == kEpiSwiGLU && (N % bn) != 0) return -3;
@@ -1004,6 +1020,7 @@ static int grouped_gemm(const void* A, const void* W, void* C, const int* group_
   } else if (epilogue == kEpiSwiGLU) {
     if (bn == 256) OGB_GROUPED(256, kEpiSwiGLU);
     if (bn == 128) OGB_GROUPED(128, kEpiSwiGLU);
+    if (bn == 64) OGB_GROUPED(64, kEpiSwiGLU);
   }
 #undef OGB_GROUPED
   return -2;
@@ -1014,14 +1031,15 @@ extern "C" int ogb_grouped_gemm_bf16(const void* A, const void* W, void* C, cons
                                      void* stream) {
   if (bn <= 0 || (N % bn) != 0) return -3;
   return grouped_gemm(A, W, C, group_tab, group_mtiles, experts, max_rows, max_mtiles, N, K, K, K, epilogue == kEpiSwiGLU ? N / 2 : N, epilogue,
-                      kActSilu, bn, status, static_cast<cudaStream_t>(stream));
+                      ActArgs(), bn, status, static_cast<cudaStream_t>(stream));
 }
 
-// Plain products with any N, row strides of their own and an activation (0 none, 2 square of relu).  bn 0: picked from the most
-// tiles the launch can have.
+// Products with any N, row strides of their own and an activation (ogb_gemm_bf16_act).  Plain ones: bn 0 picks from the most tiles
+// the launch can have.
 extern "C" int ogb_grouped_gemm_act(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows,
-                                    int max_mtiles, int N, int K, int lda, int ldw, int ldc, int act, int bn, int* status, void* stream) {
-  if (act != 0 && act != kActRelu2) return -7;
+                                    int max_mtiles, int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b, int bn, int* status,
+                                    void* stream) {
+  if (act < 0 || act > kActXielu || (act_gated(act) && bn == 0)) return -7;
   if (bn == 0) {
     const int sms = ogb_num_sms();
     const int cand[3] = {256, 128, 64};
@@ -1033,6 +1051,6 @@ extern "C" int ogb_grouped_gemm_act(const void* A, const void* W, void* C, const
       if (t < best - 1e-6f) { best = t; bn = cand[i]; }
     }
   }
-  return grouped_gemm(A, W, C, group_tab, group_mtiles, experts, max_rows, max_mtiles, N, K, lda, ldw, ldc, kEpiNone, act, bn, status,
-                      static_cast<cudaStream_t>(stream));
+  return grouped_gemm(A, W, C, group_tab, group_mtiles, experts, max_rows, max_mtiles, N, K, lda, ldw, ldc, act_gated(act) ? kEpiSwiGLU : kEpiNone,
+                      ActArgs{act, act_a, act_b}, bn, status, static_cast<cudaStream_t>(stream));
 }

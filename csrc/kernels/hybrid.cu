@@ -1,5 +1,6 @@
-// Row-wise kernels of models with hyper-connected residual streams, Dynamic-Tanh norms, token shift and latent KV pages,
-// plus the fp32 matrix product of the 32-bit engine.
+// Row-wise kernels of models with a mixer per layer: hyper-connected residual streams with Dynamic-Tanh norms and token shift, one
+// residual stream with RMS norms and input convolutions, embeddings, latent KV pages; plus the fp32 matrix product of the 32-bit
+// engine.
 //
 // hyper_step is the one pass between two matrix products: it folds a sublayer's output y into the residual streams
 // (x_t <- sum_s mix[s][t] x_s + out[t] y), reads the next sublayer's input (u = sum_s in[s] x_s), applies the
@@ -195,42 +196,104 @@ static int dispatch_hyper(const HyperParams& p, cudaStream_t stream) {
 }
 
 // ------------------------------------------------------------------------------------------------------
-// norm_step is the pass between two products for designs with one residual stream and RMS norms on both sides of a sublayer:
+// What a sublayer left for the residual: a row per token, or -- behind routed experts -- the weighted sum of the token's expert rows
+// (sum_j weight[t][j] y[pos[t][j]]) and of a shared expert's row times the sigmoid of its gate, taken here so that it never
+// exists in memory.
+// ------------------------------------------------------------------------------------------------------
+struct SublayerOut {
+  const void* y;           // [rows, ldy], or the expert rows; null: nothing
+  const int* pos;          // [rows, k] or null
+  const float* weight;     // [rows, k]
+  const void* shared;      // [rows, lds] or null
+  const float* gate;       // [rows, ldg]: logits
+  int k, ldy, lds, ldg;
+  int64_t y_rows;
+};
+
+// Outputs of rows t0 .. t0 + n - 1 (n <= NB) at this thread's columns (i * blockDim.x + threadIdx.x) * V of W.
+template <typename T, int NB, int N, int V>
+OGB_DEVICE void sublayer_rows(const SublayerOut& o, int t0, int n, int W, float (&y)[NB][N][V], int* status) {
+#pragma unroll
+  for (int b = 0; b < NB; ++b)
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int v = 0; v < V; ++v) y[b][i][v] = 0.f;
+  if (o.y == nullptr) return;
+  auto add = [&](const void* base, int64_t row, int ld, float f, float (&acc)[N][V]) {
+    const T* src = static_cast<const T*>(base) + row * ld;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < W) {
+        float z[V];
+        load_vec<V>(src + c, z);
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[i][v] = fmaf(f, z[v], acc[i][v]);
+      }
+    }
+  };
+  if (o.pos == nullptr) {
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+      if (b < n) add(o.y, t0 + b, o.ldy, 1.f, y[b]);
+    return;
+  }
+  for (int j = 0; j < o.k; ++j) {
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      if (b >= n) continue;
+      const size_t at = static_cast<size_t>(t0 + b) * o.k + j;
+      const int row = o.pos[at];
+      if (row < 0 || row >= o.y_rows) {
+        if (threadIdx.x == 0) atomicOr(status, kStatusIndexOutOfRange);
+        continue;
+      }
+      add(o.y, row, o.ldy, o.weight[at], y[b]);
+    }
+  }
+  if (o.shared == nullptr) return;
+#pragma unroll
+  for (int b = 0; b < NB; ++b)
+    if (b < n) add(o.shared, t0 + b, o.lds, 1.f / (1.f + expf(-o.gate[static_cast<size_t>(t0 + b) * o.ldg])), y[b]);
+}
+
+// sums over the block of NB values a thread; `red` [2][NB][32] alternates with `parity`, so one barrier a call is enough
+template <int NB>
+OGB_DEVICE void block_sums(float (&v)[NB], float (&red)[2][NB][32], int parity) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+#pragma unroll
+  for (int b = 0; b < NB; ++b) {
+    v[b] = warp_sum(v[b]);
+    if (lane == 0) red[parity][b][warp] = v[b];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int b = 0; b < NB; ++b) v[b] = warp_sum(lane < warps ? red[parity][b][lane] : 0.f);
+}
+
+// ------------------------------------------------------------------------------------------------------
+// norm_step is the pass between two products for designs with one residual stream:
 //
 //   x <- x + rms(y) post        h = rms(x) w
 //
-// y is the sublayer's output row, or -- behind routed experts -- the weighted sum of the token's expert rows
-// (sum_j weight[t][j] ys[pos[t][j]]), taken here so that it never exists in memory.  One block per row, the row in registers; all
+// Without `post` the output is added as it is, without `w` h is the residual itself.  One block per row, the row in registers; all
 // fp32.
 // ------------------------------------------------------------------------------------------------------
 struct NormStepParams {
   float* x;                // [rows, W]
-  const void* y;           // [rows, ldy], or the expert rows
-  const int* pos;          // [rows, k] or null
-  const float* weight;     // [rows, k]
-  const float *post, *w;   // norm weights
+  SublayerOut out;
+  const float *post, *w;   // norm weights or null
   void* h;                 // [rows, ldh] or null
   const int* gather;       // row r of h comes from row gather[r]; x is then left alone
   float eps;
-  int rows, total_rows, W, k, ldy, ldh;
-  int64_t y_rows;
+  int rows, total_rows, W, ldh;
   int* status;
 };
 
-OGB_DEVICE float block_sum(float v, float* red) {
-  const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-  v = warp_sum(v);
-  __syncthreads();                             // the last sum has been read
-  if ((threadIdx.x & 31) == 0) red[warp] = v;
-  __syncthreads();
-  float s = 0.f;
-  for (int i = 0; i < warps; ++i) s += red[i];
-  return s;
-}
-
 template <typename T, int V, int N>
 __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
-  __shared__ float red[32];
+  __shared__ float red[2][1][32];
   const int r = blockIdx.x;
   int t = r;
   if (p.gather != nullptr) {
@@ -249,68 +312,49 @@ __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
     for (int v = 0; v < V; ++v) x[i][v] = 0.f;
     if (c < p.W) load_vec<V>(xr + c, x[i]);
   }
-  if (p.y != nullptr) {
-    float y[N][V], ss = 0.f;
+  if (p.out.y != nullptr) {
+    float y[1][N][V], inv[1] = {0.f};
+    sublayer_rows<T, 1>(p.out, t, 1, p.W, y, p.status);
+    if (p.post != nullptr) {
 #pragma unroll
-    for (int i = 0; i < N; ++i)
+      for (int i = 0; i < N; ++i)
 #pragma unroll
-      for (int v = 0; v < V; ++v) y[i][v] = 0.f;
-    const int k = p.pos != nullptr ? p.k : 1;
-    for (int j = 0; j < k; ++j) {
-      int64_t row = t;
-      float f = 1.f;
-      if (p.pos != nullptr) {
-        row = p.pos[static_cast<size_t>(t) * k + j];
-        f = p.weight[static_cast<size_t>(t) * k + j];
-        if (row < 0 || row >= p.y_rows) {
-          if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
-          continue;
-        }
-      }
-      const T* src = static_cast<const T*>(p.y) + row * p.ldy;
-#pragma unroll
-      for (int i = 0; i < N; ++i) {
-        const int c = (i * blockDim.x + threadIdx.x) * V;
-        if (c < p.W) {
-          float z[V];
-          load_vec<V>(src + c, z);
-#pragma unroll
-          for (int v = 0; v < V; ++v) y[i][v] = fmaf(f, z[v], y[i][v]);
-        }
-      }
+        for (int v = 0; v < V; ++v) inv[0] = fmaf(y[0][i][v], y[0][i][v], inv[0]);
+      block_sums<1>(inv, red, 0);
+      inv[0] = 1.f / sqrtf(inv[0] / static_cast<float>(p.W) + p.eps);
     }
-#pragma unroll
-    for (int i = 0; i < N; ++i)
-#pragma unroll
-      for (int v = 0; v < V; ++v) ss = fmaf(y[i][v], y[i][v], ss);
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(p.W) + p.eps);
 #pragma unroll
     for (int i = 0; i < N; ++i) {
       const int c = (i * blockDim.x + threadIdx.x) * V;
       if (c < p.W) {
         float g[V];
-        load_vec<V>(p.post + c, g);
+        if (p.post != nullptr) load_vec<V>(p.post + c, g);
 #pragma unroll
-        for (int v = 0; v < V; ++v) x[i][v] = fmaf(y[i][v] * inv, g[v], x[i][v]);
+        for (int v = 0; v < V; ++v) x[i][v] = p.post != nullptr ? fmaf(y[0][i][v] * inv[0], g[v], x[i][v]) : x[i][v] + y[0][i][v];
         if (p.gather == nullptr) store_vec<V>(xr + c, x[i]);
       }
     }
   }
   if (p.h == nullptr) return;
-  float ss = 0.f;
+  float inv[1] = {0.f};
+  if (p.w != nullptr) {
 #pragma unroll
-  for (int i = 0; i < N; ++i)
+    for (int i = 0; i < N; ++i)
 #pragma unroll
-    for (int v = 0; v < V; ++v) ss = fmaf(x[i][v], x[i][v], ss);
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(p.W) + p.eps);
+      for (int v = 0; v < V; ++v) inv[0] = fmaf(x[i][v], x[i][v], inv[0]);
+    block_sums<1>(inv, red, 1);
+    inv[0] = 1.f / sqrtf(inv[0] / static_cast<float>(p.W) + p.eps);
+  }
 #pragma unroll
   for (int i = 0; i < N; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * V;
     if (c < p.W) {
-      float g[V];
-      load_vec<V>(p.w + c, g);
+      if (p.w != nullptr) {
+        float g[V];
+        load_vec<V>(p.w + c, g);
 #pragma unroll
-      for (int v = 0; v < V; ++v) x[i][v] *= inv * g[v];
+        for (int v = 0; v < V; ++v) x[i][v] *= inv[0] * g[v];
+      }
       store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r) * p.ldh + c, x[i]);
     }
   }
@@ -330,11 +374,227 @@ static int launch_norm_step(const NormStepParams& p, cudaStream_t s) {
 }
 
 // ------------------------------------------------------------------------------------------------------
-// all streams of a row start as the token's embedding
+// norm_conv_step is that pass for designs whose sublayers read a short causal convolution of the normed residual:
+//
+//   x_out <- x_in + y + add        h = rms(x_out) w        u_t = sum_j conv[j] h_(t - taps + 1 + j)
+//
+// A block is one decode row or kNcRows rows of one prefill chunk.  A thread keeps its columns' last taps - 1 values of h and walks the
+// rows, NB at a time (their loads and sums are under way together).  The rows before the block's first are normed once more -- x_in and
+// x_out are different buffers, so what they need is still there -- or come from the sequence's slot ([slots][taps - 1][W], oldest
+// first); only the block with a chunk's first row reads a slot, so it also leaves the chunk's last values there.
+// ------------------------------------------------------------------------------------------------------
+constexpr int kNcRows = 16;                   // divides the scheduler's 64-row tiles
+
+struct NormConvParams {
+  const float* x_in;       // [rows, ldx]
+  float* x_out;            // [rows, W], or null: nothing is added
+  SublayerOut out;
+  const float* add;        // [W] or null
+  const float* w;          // [W]
+  const float* conv;       // [taps, W]
+  float* state;            // [slots, taps - 1, W]
+  void* h;                 // [rows, ldh]
+  float eps;
+  int W, ldx, ldh, taps;
+  StepRows sr;
+  int* status;
+};
+
+template <typename T, int V, int N, int NB, int TM>
+__global__ void __launch_bounds__(512) norm_conv_kernel(NormConvParams p) {
+  __shared__ float red[2][NB][32];
+  const StepRows& sr = p.sr;
+  int entry, base, n, j0;                      // sequence entry, its first row, its rows, first row of this block within them
+  if (static_cast<int>(blockIdx.x) < sr.num_decode) {
+    entry = blockIdx.x; base = entry; n = 1; j0 = 0;
+  } else {
+    const int g = blockIdx.x - sr.num_decode, tile = g / (64 / kNcRows), s = sr.tile_seq[tile];
+    entry = sr.num_decode + s;
+    base = sr.num_decode + sr.cu_q[s];
+    n = sr.cu_q[s + 1] - sr.cu_q[s];
+    j0 = sr.tile_q0[tile] + (g % (64 / kNcRows)) * kNcRows;
+  }
+  const int start = sr.ctx_len[entry] - n;     // tokens before the chunk
+  if (j0 >= n || start < 0) return;            // a padding row has none
+  int slot = sr.state_slot[entry];
+  if (slot >= sr.num_slots) {
+    if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
+    slot = -1;
+  }
+  float conv[TM][N][V], w[N][V], h[TM > 1 ? TM - 1 : 1][N][V];    // filters aligned to their last tap; h: the last values, oldest first
+  const int col0 = threadIdx.x * V, step = blockDim.x * V, off = TM - p.taps;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = col0 + i * step;
+#pragma unroll
+    for (int k = 0; k < TM; ++k) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) conv[k][i][v] = 0.f;
+      if (c < p.W && k >= off) load_vec<V>(p.conv + static_cast<size_t>(k - off) * p.W + c, conv[k][i]);
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) w[i][v] = 0.f;
+    if (c < p.W) load_vec<V>(p.w + c, w[i]);
+  }
+  int parity = 0;
+  // normed rows j .. j + m - 1 of the chunk (m <= NB)
+  auto normed = [&](int j, int m, bool write, float (&o)[NB][N][V]) {
+    float x[NB][N][V], ss[NB];
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+#pragma unroll
+        for (int v = 0; v < V; ++v) x[b][i][v] = 0.f;
+        if (b < m && col0 + i * step < p.W) load_vec<V>(p.x_in + static_cast<size_t>(base + j + b) * p.ldx + col0 + i * step, x[b][i]);
+      }
+    sublayer_rows<T, NB>(p.out, base + j, m, p.W, o, p.status);
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      ss[b] = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int c = col0 + i * step;
+        if (p.add != nullptr && c < p.W) {
+          float a[V];
+          load_vec<V>(p.add + c, a);
+#pragma unroll
+          for (int v = 0; v < V; ++v) o[b][i][v] += a[v];
+        }
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+          x[b][i][v] += o[b][i][v];
+          ss[b] = c < p.W ? fmaf(x[b][i][v], x[b][i][v], ss[b]) : ss[b];
+        }
+        if (write && p.x_out != nullptr && b < m && c < p.W) store_vec<V>(p.x_out + static_cast<size_t>(base + j + b) * p.W + c, x[b][i]);
+      }
+    }
+    block_sums<NB>(ss, red, parity);
+    parity ^= 1;
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      const float inv = 1.f / sqrtf(ss[b] / static_cast<float>(p.W) + p.eps);
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+#pragma unroll
+        for (int v = 0; v < V; ++v) o[b][i][v] = x[b][i][v] * (inv * w[i][v]);
+    }
+  };
+  auto shift_in = [&](const float (&o)[N][V]) {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+#pragma unroll
+        for (int k = 0; k + 1 < TM - 1; ++k) h[k][i][v] = h[k + 1][i][v];
+        h[TM > 1 ? TM - 2 : 0][i][v] = o[i][v];
+      }
+  };
+  float* st = slot >= 0 ? p.state + static_cast<size_t>(slot) * (p.taps - 1) * p.W : nullptr;
+  auto keep = [&]() {                          // the chunk's last values to the slot
+    if (st == nullptr) return;
+#pragma unroll
+    for (int k = 0; k < TM - 1; ++k)
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+        if (k >= off && col0 + i * step < p.W) store_vec<V>(st + static_cast<size_t>(k - off) * p.W + col0 + i * step, h[k][i]);
+  };
+  float o[NB][N][V];
+  // rows from..from + m - 1 of the chunk into the last values
+  auto recompute = [&](int from, int m) {
+    for (int j = 0; j < m; j += NB) {
+      const int c = min(NB, m - j);
+      normed(from + j, c, false, o);
+#pragma unroll
+      for (int b = 0; b < NB; ++b)
+        if (b < c) shift_in(o[b]);
+    }
+  };
+#pragma unroll
+  for (int k = 0; k < (TM > 1 ? TM - 1 : 1); ++k)
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int v = 0; v < V; ++v) h[k][i][v] = 0.f;
+  if (p.taps > 1) {
+    if (j0 == 0) {
+      if (n > kNcRows) {                       // other blocks finish the chunk
+        float old[TM > 1 ? TM - 1 : 1][N][V];
+#pragma unroll
+        for (int k = 0; k < TM - 1; ++k)
+#pragma unroll
+          for (int i = 0; i < N; ++i) {
+#pragma unroll
+            for (int v = 0; v < V; ++v) old[k][i][v] = 0.f;
+            const int t = start - (TM - 1) + k;
+            if (st != nullptr && k >= off && t >= 0 && col0 + i * step < p.W) load_vec<V>(st + static_cast<size_t>(k - off) * p.W + col0 + i * step, old[k][i]);
+          }
+        recompute(n - (p.taps - 1), p.taps - 1);
+        keep();
+#pragma unroll
+        for (int k = 0; k < TM - 1; ++k)
+#pragma unroll
+          for (int i = 0; i < N; ++i)
+#pragma unroll
+            for (int v = 0; v < V; ++v) h[k][i][v] = old[k][i][v];
+      } else {
+#pragma unroll
+        for (int k = 0; k < TM - 1; ++k)
+#pragma unroll
+          for (int i = 0; i < N; ++i) {
+            const int t = start - (TM - 1) + k;
+            if (st != nullptr && k >= off && t >= 0 && col0 + i * step < p.W) load_vec<V>(st + static_cast<size_t>(k - off) * p.W + col0 + i * step, h[k][i]);
+          }
+      }
+    } else {
+      recompute(j0 - (p.taps - 1), p.taps - 1);
+    }
+  }
+  const int j1 = min(j0 + kNcRows, n);
+  for (int j = j0; j < j1; j += NB) {
+    const int m = min(NB, j1 - j);
+    normed(j, m, true, o);
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      if (b >= m) continue;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        float u[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+          u[v] = conv[TM - 1][i][v] * o[b][i][v];
+#pragma unroll
+          for (int k = 0; k < TM - 1; ++k) u[v] = fmaf(conv[k][i][v], h[k][i][v], u[v]);
+        }
+        if (col0 + i * step < p.W) store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(base + j + b) * p.ldh + col0 + i * step, u);
+      }
+      shift_in(o[b]);
+    }
+  }
+  if (p.taps > 1 && j0 == 0 && n <= kNcRows) keep();
+}
+
+template <typename T, int V, int TM>
+static int launch_norm_conv(const NormConvParams& p, cudaStream_t s) {
+  const int units = (p.W + V - 1) / V, blocks = p.sr.num_decode + p.sr.num_tiles * (64 / kNcRows);
+  const int n = units <= 256 ? 1 : units <= 1024 ? 2 : units <= 2048 ? 4 : 8;
+  const int threads = ((units + n - 1) / n + 31) / 32 * 32;
+  if (threads > 512 || n * V > 16) return -2;
+  if (n == 1) norm_conv_kernel<T, V, 1, 4, TM><<<blocks, threads, 0, s>>>(p);
+  else if (n == 2) norm_conv_kernel<T, V, 2, V == 1 ? 4 : 2, TM><<<blocks, threads, 0, s>>>(p);
+  else if (n == 4) norm_conv_kernel<T, V, 4, V == 1 ? 4 : 1, TM><<<blocks, threads, 0, s>>>(p);
+  else if constexpr (V == 1) norm_conv_kernel<T, V, 8, 2, TM><<<blocks, threads, 0, s>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------------
+// all streams of a row start as the token's embedding, normed where `w` is given; `copy` gets it too (read again by later layers)
 // ------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256) embed_streams_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
-                                                            int S, int W, int vocab, int* status) {
+                                                            int S, int W, int vocab, const float* __restrict__ w, float eps, T* __restrict__ copy,
+                                                            int ldc, int* status) {
+  __shared__ float red[2][1][32];
   const int t = blockIdx.x;
   int id = ids[t];
   if (id < 0 || id >= vocab) {
@@ -343,34 +603,94 @@ __global__ void __launch_bounds__(256) embed_streams_kernel(const int* __restric
   }
   const T* src = table + static_cast<size_t>(id) * W;
   float* dst = x + static_cast<size_t>(t) * S * W;
+  float inv[1] = {0.f};
+  if (w != nullptr) {
+    for (int c = threadIdx.x; c < W; c += blockDim.x) inv[0] = fmaf(to_f32<T>(src[c]), to_f32<T>(src[c]), inv[0]);
+    block_sums<1>(inv, red, 0);
+    inv[0] = 1.f / sqrtf(inv[0] / static_cast<float>(W) + eps);
+  }
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
-    const float v = to_f32<T>(src[c]);
+    float v = to_f32<T>(src[c]);
+    if (w != nullptr) v *= inv[0] * w[c];
     for (int s = 0; s < S; ++s) dst[static_cast<size_t>(s) * W + c] = v;
+    if (copy != nullptr) copy[static_cast<size_t>(t) * ldc + c] = from_f32<T>(v);
   }
 }
 
 // ------------------------------------------------------------------------------------------------------
-// latent pages: RMS norm of a projected row, written to its page.  pool [pages, 16, ldp]; one warp per token.
+// latent pages [pages, 16, ldp]: a row is the normed latent (rank values, zeros up to a multiple of 8) and the rotated key part that
+// all heads share (rot values).  A projected row holds the queries of `heads` heads (dim values, zeros up to a multiple of 8, and rot
+// values each), the latent and the key part.  Neighbours 2i, 2i + 1 of a rotated part turn by position * freq[i].  Rotated query parts
+// go to column `q_col` of a head's row of q_out for tokens below `split`, and back to where they came from for the others.
+// One block per token: warp 0 has the latent.  rot 0: the latent alone (one warp per token).
 // ------------------------------------------------------------------------------------------------------
+struct LatentAppendParams {
+  void* row;               // [tokens, ldr], queries first
+  const float* w;          // [rank]
+  const int* slots;
+  void* pool;
+  const double* freq;      // [rot / 2]
+  const int* positions;
+  void* q_out;             // [tokens * heads, ldq]
+  float eps;
+  int tokens, ldr, latent, rank, ldp, heads, dim, rot, ldq, q_col, split;
+  int64_t num_slots;
+  int* status;
+};
+
 template <typename T>
-__global__ void __launch_bounds__(128) latent_append_kernel(const T* __restrict__ c, int ldc, const float* __restrict__ w, float eps,
-                                                            const int* __restrict__ slots, T* __restrict__ pool, int tokens, int rank,
-                                                            int ldp, int64_t num_slots, int* status) {
-  const int lane = threadIdx.x & 31;
-  const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
-  if (t >= tokens) return;
-  const int slot = slots[t];
+OGB_DEVICE void append_latent(const LatentAppendParams& p, int t, int lane) {
+  const int64_t slot = p.slots[t];
   if (slot < 0) return;                        // padding row
-  if (slot >= num_slots) {
-    if (lane == 0) atomicOr(status, kStatusIndexOutOfRange);
+  if (slot >= p.num_slots) {
+    if (lane == 0) atomicOr(p.status, kStatusIndexOutOfRange);
     return;
   }
-  const T* src = c + static_cast<size_t>(t) * ldc;
+  const T* src = static_cast<const T*>(p.row) + static_cast<size_t>(t) * p.ldr + p.latent;
   float ss = 0.f;
-  for (int i = lane; i < rank; i += 32) { const float v = to_f32<T>(src[i]); ss = fmaf(v, v, ss); }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(rank) + eps);
-  T* dst = pool + static_cast<size_t>(slot) * ldp;
-  for (int i = lane; i < rank; i += 32) dst[i] = from_f32<T>(to_f32<T>(src[i]) * inv * w[i]);
+  for (int i = lane; i < p.rank; i += 32) { const float v = to_f32<T>(src[i]); ss = fmaf(v, v, ss); }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.rank) + p.eps);
+  T* dst = static_cast<T*>(p.pool) + slot * p.ldp;
+  for (int i = lane; i < p.rank; i += 32) dst[i] = from_f32<T>(to_f32<T>(src[i]) * inv * p.w[i]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_append_kernel(LatentAppendParams p) {
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (t < p.tokens) append_latent<T>(p, t, threadIdx.x & 31);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_rope_append_kernel(LatentAppendParams p) {
+  extern __shared__ float2 s_turn[];           // [rot / 2] cos, sin
+  const int t = blockIdx.x, half = p.rot / 2, dp = (p.dim + 7) / 8 * 8, rp = (p.rot + 7) / 8 * 8;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    // the angle is reduced in double, so that it is good to fp32 at every position
+    const double a = static_cast<double>(p.positions[t]) * p.freq[i] * 0.15915494309189535;
+    float s, c;
+    sincospif(static_cast<float>(2.0 * (a - rint(a))), &s, &c);
+    s_turn[i] = make_float2(c, s);
+  }
+  if (threadIdx.x < 32) append_latent<T>(p, t, threadIdx.x);
+  __syncthreads();
+  T* row = static_cast<T*>(p.row) + static_cast<size_t>(t) * p.ldr;
+  const int64_t slot = p.slots[t];
+  for (int i = threadIdx.x; i < (p.heads + 1) * half; i += blockDim.x) {
+    const int head = i / half, e = i - head * half;
+    const bool key = head == p.heads;
+    T* src = row + (key ? p.latent + (p.rank + 7) / 8 * 8 : head * (dp + rp) + dp) + 2 * e;
+    const float u = to_f32<T>(src[0]), v = to_f32<T>(src[1]);
+    const float2 cs = s_turn[e];
+    T* dst = src;
+    if (key) {
+      if (slot < 0 || slot >= p.num_slots) continue;
+      dst = static_cast<T*>(p.pool) + slot * p.ldp + (p.rank + 7) / 8 * 8 + 2 * e;
+    } else if (t < p.split) {
+      dst = static_cast<T*>(p.q_out) + (static_cast<size_t>(t) * p.heads + head) * p.ldq + p.q_col + 2 * e;
+    }
+    dst[0] = from_f32<T>(u * cs.x - v * cs.y);
+    dst[1] = from_f32<T>(v * cs.x + u * cs.y);
+  }
 }
 
 // ------------------------------------------------------------------------------------------------------
@@ -423,17 +743,31 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restri
 }
 
 // ------------------------------------------------------------------------------------------------------
-// gated activation over tile-interleaved gate | up columns (ops.pack_gate_up): act 0 = silu, 1 = tanh form of gelu
+// gated activation over tile-interleaved gate | up columns (ops.pack_gate_up), and an activation of every value (common.cuh Act)
 // ------------------------------------------------------------------------------------------------------
+OGB_DEVICE float gated_act_f32(const ActArgs& act, float g, float u) {
+  if (act.kind == kActGeluTanh) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  if (act.kind == kActClampGlu) {
+    g = fminf(g, act.a);
+    u = fminf(fmaxf(u, -act.a), act.a);
+    return g / (1.f + expf(-kClampGluSlope * g)) * (u + 1.f);
+  }
+  return g / (1.f + expf(-g)) * u;
+}
+OGB_DEVICE float plain_act_f32(const ActArgs& act, float v) {
+  if (act.kind == kActRelu2) return fmaxf(v, 0.f) * fmaxf(v, 0.f);
+  if (act.kind == kActXielu) return fmaf(0.5f, v, v > 0.f ? act.a * v * v : act.b * (expm1f(v) - v));
+  return v;
+}
+
 template <typename T>
-__global__ void __launch_bounds__(256) act_mul_packed_kernel(const T* __restrict__ gu, T* __restrict__ out, int rows, int inter, int half, int act) {
+__global__ void __launch_bounds__(256) act_mul_packed_kernel(const T* __restrict__ gu, T* __restrict__ out, int rows, int inter, int half, ActArgs act) {
   const long long total = static_cast<long long>(rows) * inter;
   for (long long i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
     const int t = static_cast<int>(i / inter), j = static_cast<int>(i % inter);
     const T* row = gu + static_cast<size_t>(t) * 2 * inter + static_cast<size_t>(j / half) * 2 * half + j % half;
     const float g = to_f32<T>(row[0]), u = to_f32<T>(row[half]);
-    const float a = act == 1 ? 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.f + expf(-g));
-    out[i] = from_f32<T>(a * u);
+    out[i] = from_f32<T>(gated_act_f32(act, g, u));
   }
 }
 
@@ -445,7 +779,7 @@ __global__ void __launch_bounds__(256) act_mul_packed_kernel(const T* __restrict
 constexpr int kF32Tile = 64, kF32K = 16;
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W, float* __restrict__ C, int M,
                                                        int N, int K, int lda, int ldw, int ldc, int a_step, int c_step, const int* __restrict__ tab,
-                                                       const int* __restrict__ mtiles, int relu2) {
+                                                       const int* __restrict__ mtiles, ActArgs act) {
   __shared__ float sa[kF32K][kF32Tile + 4], sw[kF32K][kF32Tile + 4];
   A += static_cast<size_t>(blockIdx.z) * a_step;
   W += static_cast<size_t>(blockIdx.z) * N * ldw;
@@ -486,10 +820,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int r = m0 + ty * 4 + i, c = n0 + tx * 4 + j;
-      if (r < M && c < N) {
-        const float v = relu2 ? fmaxf(acc[i][j], 0.f) * fmaxf(acc[i][j], 0.f) : acc[i][j];
-        C[static_cast<size_t>(r) * ldc + c] = v;
-      }
+      if (r < M && c < N) C[static_cast<size_t>(r) * ldc + c] = plain_act_f32(act, acc[i][j]);
     }
 }
 
@@ -515,47 +846,88 @@ extern "C" int ogb_hyper_step(const float* x_in, float* x_out, const void* y, co
   return -3;
 }
 
-// pos / weight (null: y has one row per token): y holds y_rows expert rows, of which token t sums k.  w / h null: no read-out.
-extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const float* post, const float* w, void* h,
-                             const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int ldh, int64_t y_rows, int elem,
-                             int* status, void* stream) {
+// pos / weight (null: y has one row per token): y holds y_rows expert rows, of which token t sums k; shared / gate: a row of every
+// token, times the sigmoid of its gate.
+static bool sublayer_ok(const SublayerOut& o) {
+  return (o.pos == nullptr || (o.weight != nullptr && o.k >= 1)) && (o.shared == nullptr || (o.pos != nullptr && o.gate != nullptr));
+}
+
+// post null: y as it is; w null: h is the residual; h null: no read-out.
+extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const void* shared, const float* gate, const float* post,
+                             const float* w, void* h, const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int lds, int ldg,
+                             int ldh, int64_t y_rows, int elem, int* status, void* stream) {
   if (rows <= 0) return 0;
-  if (W < 1 || (y != nullptr && post == nullptr) || (h != nullptr && w == nullptr) || (pos != nullptr && (weight == nullptr || k < 1))) return -3;
-  NormStepParams p{x, y, pos, weight, post, w, h, gather, eps, rows, total_rows, W, k, ldy, ldh, y_rows, status};
+  NormStepParams p{x, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, post, w, h, gather, eps, rows, total_rows, W, ldh, status};
+  if (W < 1 || !sublayer_ok(p.out)) return -3;
   // four elements at a time need rows that start on them, and pointers too
-  const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h);
+  const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared);
   const uintptr_t f32 = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(post) | reinterpret_cast<uintptr_t>(w);
-  const bool vec = ((W | ldy | ldh) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
+  const bool vec = ((W | ldy | ldh | lds) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (elem == kElemBF16) return vec ? launch_norm_step<__nv_bfloat16, 4>(p, s) : launch_norm_step<__nv_bfloat16, 1>(p, s);
   if (elem == kElemF32) return vec ? launch_norm_step<float, 4>(p, s) : launch_norm_step<float, 1>(p, s);
   return -3;
 }
 
-extern "C" int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, int elem, int* status,
-                                 void* stream) {
+// x_out null: nothing is added (y and add null).  At most 8 taps; rows of up to 8192 columns, 4096 where they do not start on four
+// elements.
+extern "C" int ogb_norm_conv_step(const float* x_in, float* x_out, const void* y, const int* pos, const float* weight, const void* shared,
+                                  const float* gate, const float* add, const float* w, const float* conv, float* state, void* h, float eps, int W,
+                                  int taps, int k, int ldx, int ldy, int lds, int ldg, int ldh, int64_t y_rows, const int* ctx_len,
+                                  const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode, int num_tiles,
+                                  int num_slots, int elem, int* status, void* stream) {
+  if (num_decode + num_tiles <= 0) return 0;
+  NormConvParams p{x_in, x_out, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, add, w, conv, state, h, eps, W, ldx, ldh, taps,
+                   StepRows{ctx_len, state_slot, cu_q, tile_seq, tile_q0, num_decode, num_tiles, num_slots}, status};
+  if (W < 1 || taps < 1 || taps > 8 || x_in == x_out || !sublayer_ok(p.out) || w == nullptr || conv == nullptr || h == nullptr) return -3;
+  if ((taps > 1 && state == nullptr) || ((y != nullptr || add != nullptr) && x_out == nullptr)) return -3;
+  const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared);
+  const uintptr_t f32 = reinterpret_cast<uintptr_t>(x_in) | reinterpret_cast<uintptr_t>(x_out) | reinterpret_cast<uintptr_t>(add) |
+                        reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(conv) | reinterpret_cast<uintptr_t>(state);
+  const bool vec = ((W | ldx | ldy | ldh | lds) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+#define OGB_NORM_CONV(T) \
+  return vec ? (taps <= 4 ? launch_norm_conv<T, 4, 4>(p, s) : launch_norm_conv<T, 4, 8>(p, s)) \
+             : (taps <= 4 ? launch_norm_conv<T, 1, 4>(p, s) : launch_norm_conv<T, 1, 8>(p, s))
+  if (elem == kElemBF16) OGB_NORM_CONV(__nv_bfloat16);
+  if (elem == kElemF32) OGB_NORM_CONV(float);
+#undef OGB_NORM_CONV
+  return -3;
+}
+
+extern "C" int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, const float* w, float eps, void* copy,
+                                 int ldc, int elem, int* status, void* stream) {
   if (tokens <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (elem == kElemBF16) embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const __nv_bfloat16*>(table), x, S, W, vocab, status);
-  else if (elem == kElemF32) embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const float*>(table), x, S, W, vocab, status);
+  if (elem == kElemBF16)
+    embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const __nv_bfloat16*>(table), x, S, W, vocab, w, eps, static_cast<__nv_bfloat16*>(copy),
+                                                ldc, status);
+  else if (elem == kElemF32)
+    embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const float*>(table), x, S, W, vocab, w, eps, static_cast<float*>(copy), ldc, status);
   else return -3;
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int ogb_latent_append(const void* c, int ldc, const float* w, float eps, const int* slots, void* pool, int tokens, int rank,
-                                 int ldp, int64_t num_slots, int elem, int* status, void* stream) {
-  if (tokens <= 0) return 0;
-  if (rank > ldp) return -3;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int blocks = (tokens + 3) / 4;
-  if (elem == kElemBF16)
-    latent_append_kernel<<<blocks, 128, 0, s>>>(static_cast<const __nv_bfloat16*>(c), ldc, w, eps, slots, static_cast<__nv_bfloat16*>(pool), tokens,
-                                                rank, ldp, num_slots, status);
-  else if (elem == kElemF32)
-    latent_append_kernel<<<blocks, 128, 0, s>>>(static_cast<const float*>(c), ldc, w, eps, slots, static_cast<float*>(pool), tokens, rank, ldp,
-                                                num_slots, status);
-  else return -3;
+template <typename T>
+static int launch_latent_append(const LatentAppendParams& p, cudaStream_t s) {
+  if (p.rot == 0) latent_append_kernel<T><<<(p.tokens + 3) / 4, 128, 0, s>>>(p);
+  else latent_rope_append_kernel<T><<<p.tokens, 128, p.rot / 2 * sizeof(float2), s>>>(p);
   return static_cast<int>(cudaGetLastError());
+}
+
+// `latent`: column of the latent in a projected row.
+extern "C" int ogb_latent_append(void* row, int ldr, int latent, const float* w, float eps, const int* slots, void* pool, int tokens, int rank, int ldp,
+                                 int64_t num_slots, const double* freq, const int* positions, void* q_out, int heads, int dim, int rot, int ldq,
+                                 int q_col, int split, int elem, int* status, void* stream) {
+  if (tokens <= 0) return 0;
+  if (rank > ldp || rot < 0 || (rot & 1) || rot > 4096) return -3;
+  if (rot > 0 && (freq == nullptr || positions == nullptr || (rank + 7) / 8 * 8 + rot > ldp || (split > 0 && (q_out == nullptr || q_col + rot > ldq)))) return -3;
+  LatentAppendParams p{row, w, slots, pool, freq, positions, q_out, eps, tokens, ldr, latent, rank, ldp, heads, dim, rot, ldq, q_col, split, num_slots,
+                       status};
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (elem == kElemBF16) return launch_latent_append<__nv_bfloat16>(p, s);
+  if (elem == kElemF32) return launch_latent_append<float>(p, s);
+  return -3;
 }
 
 extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate,
@@ -575,9 +947,11 @@ extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void*
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, int elem, void* stream) {
+extern "C" int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int kind, float act_a, float act_b, int elem,
+                                  void* stream) {
   if (rows <= 0) return 0;
-  if (half <= 0 || inter % half != 0 || act < 0 || act > 1) return -3;
+  if (half <= 0 || inter % half != 0 || !act_gated(kind)) return -3;
+  const ActArgs act{kind, act_a, act_b};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int blocks = static_cast<int>(std::min<long long>((static_cast<long long>(rows) * inter + 255) / 256, 148 * 16));
   if (elem == kElemBF16)
@@ -592,16 +966,27 @@ extern "C" int ogb_gemm_f32(const float* A, const float* W, float* C, int M, int
                             int c_step, void* stream) {
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
   const dim3 grid((N + kF32Tile - 1) / kF32Tile, (M + kF32Tile - 1) / kF32Tile, batch);
-  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, M, N, K, lda, ldw, ldc, a_step, c_step, nullptr, nullptr, 0);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, M, N, K, lda, ldw, ldc, a_step, c_step, nullptr, nullptr, ActArgs());
   return static_cast<int>(cudaGetLastError());
 }
 
-// Products over experts (see ogb_grouped_gemm_bf16); act 2: square of relu.
+// With an activation of every result (not a gated one).
+extern "C" int ogb_gemm_f32_act(const float* A, const float* W, float* C, int M, int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b,
+                                void* stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (act_gated(act)) return -7;
+  const dim3 grid((N + kF32Tile - 1) / kF32Tile, (M + kF32Tile - 1) / kF32Tile);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, M, N, K, lda, ldw, ldc, 0, 0, nullptr, nullptr, ActArgs{act, act_a, act_b});
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Products over experts (see ogb_grouped_gemm_act), with an activation of every result.
 extern "C" int ogb_grouped_gemm_f32(const float* A, const float* W, float* C, const int* group_tab, const int* group_mtiles, int max_rows,
-                                    int max_mtiles, int N, int K, int lda, int ldw, int ldc, int act, void* stream) {
+                                    int max_mtiles, int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b, void* stream) {
   if (max_rows <= 0 || max_mtiles <= 0 || N <= 0) return 0;
-  if (act != 0 && act != 2) return -7;
+  if (act_gated(act)) return -7;
   const dim3 grid((N + kF32Tile - 1) / kF32Tile, 2 * max_mtiles);
-  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, max_rows, N, K, lda, ldw, ldc, 0, 0, group_tab, group_mtiles, act == 2);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(A, W, C, max_rows, N, K, lda, ldw, ldc, 0, 0, group_tab, group_mtiles,
+                                                                       ActArgs{act, act_a, act_b});
   return static_cast<int>(cudaGetLastError());
 }

@@ -1,10 +1,11 @@
-// Attention over paged latents: every head of a layer reads the same cached row c_j (kv_rank values) as key and as value.
+// Attention over paged latents: every head of a layer reads the same cached row c_j as key and, in its first kv_rank values, as value.
 // The per-head expansions are folded into the query and the output by matrix products outside this file
-// (q' = W_uk^T q before, W_uv o after), so a query row is (token, head) with kv_rank values, score = q' . c * scale, and
-// the result is the softmax-weighted sum of the visible c_j.  A token at position i sees j with 0 <= i - j < window
+// (q' = W_uk^T q before, W_uv o after), so a query row is (token, head) with as many values as a cached row -- kv_rank, and
+// behind them those of a rotated part that all heads share, where there is one --, score = q' . c * scale, and the result is the
+// softmax-weighted sum of the visible c_j, times the sigmoid of the head's gate where there is one.  A token at position i sees j with 0 <= i - j < window
 // (window <= 0: every earlier token).
 //
-// bf16 rows of up to 512 values run on the tensor cores (latent_attention_tc.cu).  latent_attention_warp_kernel takes any rank
+// bf16 rows of up to 576 values run on the tensor cores (latent_attention_tc.cu).  latent_attention_warp_kernel takes any rank
 // and both activation types: one warp per query row, four keys at a time, online softmax in fp32.  Decode rows can split
 // their keys `num_splits` ways (combined by a second kernel).
 #include <stdlib.h>
@@ -102,40 +103,39 @@ __global__ void __launch_bounds__(kLatWarps * 32) latent_attention_warp_kernel(L
     const size_t pr = row * p.num_splits + blockIdx.y;
 #pragma unroll
     for (int e = 0; e < PER; ++e)
-      if (lane + 32 * e < p.rank) p.part_o[pr * p.rank + lane + 32 * e] = acc[e];
+      if (lane + 32 * e < p.vrank) p.part_o[pr * p.vrank + lane + 32 * e] = acc[e];
     if (lane == 0) { p.part_ml[2 * pr] = m; p.part_ml[2 * pr + 1] = l; }
     return;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  T* op = static_cast<T*>(p.out) + row * p.ldq;
+  const float inv = (l > 0.f ? 1.f / l : 0.f) * latent_gate<T>(p, row);
+  T* op = static_cast<T*>(p.out) + row * p.ldo;
 #pragma unroll
   for (int e = 0; e < PER; ++e)
-    if (lane + 32 * e < p.rank) op[lane + 32 * e] = from_f32<T>(acc[e] * inv);
+    if (lane + 32 * e < p.vrank) op[lane + 32 * e] = from_f32<T>(acc[e] * inv);
 }
 
 // combine the partial results of split keys: one warp per query row
 template <typename T>
-__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, T* __restrict__ out,
-                                                             const int* __restrict__ ctx_len, int rows, int heads, int rank, int ldo, int splits) {
-  const int lane = threadIdx.x & 31;
+__global__ void __launch_bounds__(128) latent_combine_kernel(LatParams p) {
+  const int lane = threadIdx.x & 31, splits = p.num_splits;
   const int row = blockIdx.x * 4 + (threadIdx.x >> 5);
-  if (row >= rows * heads || ctx_len[row / heads] <= 0) return;
+  if (row >= p.rows * p.heads || p.ctx_len[row / p.heads] <= 0) return;
   float m = -INFINITY;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, part_ml[2 * (static_cast<size_t>(row) * splits + s)]);
+  for (int s = 0; s < splits; ++s) m = fmaxf(m, p.part_ml[2 * (static_cast<size_t>(row) * splits + s)]);
   float l = 0.f;
   for (int s = 0; s < splits; ++s) {
-    const float* ml = part_ml + 2 * (static_cast<size_t>(row) * splits + s);
+    const float* ml = p.part_ml + 2 * (static_cast<size_t>(row) * splits + s);
     l += ml[0] == -INFINITY ? 0.f : ml[1] * expf(ml[0] - m);
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int i = lane; i < rank; i += 32) {
+  const float inv = (l > 0.f ? 1.f / l : 0.f) * latent_gate<T>(p, row);
+  for (int i = lane; i < p.vrank; i += 32) {
     float a = 0.f;
     for (int s = 0; s < splits; ++s) {
       const size_t pr = static_cast<size_t>(row) * splits + s;
-      const float ms = part_ml[2 * pr];
-      if (ms != -INFINITY) a = fmaf(part_o[pr * rank + i], expf(ms - m), a);
+      const float ms = p.part_ml[2 * pr];
+      if (ms != -INFINITY) a = fmaf(p.part_o[pr * p.vrank + i], expf(ms - m), a);
     }
-    out[static_cast<size_t>(row) * ldo + i] = from_f32<T>(a * inv);
+    static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + i] = from_f32<T>(a * inv);
   }
 }
 
@@ -199,14 +199,14 @@ extern "C" int ogb_latent_set_tc(int on) {
 }
 
 extern "C" int ogb_latent_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
-                                    const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages,
-                                    int num_tiles, int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml,
-                                    int* counters, int elem, int* status, void* stream) {
+                                    const int* tile_seq, const int* tile_q0, const void* gate, int rows, int heads, int rank, int vrank, int ldq,
+                                    int ldo, int ldp, int ldg, int max_pages, int num_tiles, int64_t num_pages, int window, float scale,
+                                    int num_splits, float* part_o, float* part_ml, int* counters, int elem, int* status, void* stream) {
   if (rows <= 0 || (cu_q != nullptr && num_tiles <= 0)) return 0;
-  if (heads <= 0 || rank <= 0 || rank > ldq || rank > ldp) return -3;
+  if (heads <= 0 || rank <= 0 || rank > ldq || rank > ldp || vrank <= 0 || vrank > rank || vrank > ldo) return -3;
   if (cu_q != nullptr) num_splits = 1;
   if (num_splits > 1 && (part_o == nullptr || part_ml == nullptr)) return -3;
-  LatParams p{q, out, pool, page_table, ctx_len, cu_q, tile_seq, tile_q0, rows, heads, rank, ldq, ldp, max_pages, num_tiles, window,
+  LatParams p{q, out, pool, page_table, ctx_len, cu_q, tile_seq, tile_q0, gate, rows, heads, rank, vrank, ldq, ldo, ldp, ldg, max_pages, num_tiles, window,
               num_splits < 1 ? 1 : num_splits, num_pages, scale, part_o, part_ml, counters, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   int rc = -2;                                    // the tensor-core kernel declines what it cannot take
@@ -217,10 +217,8 @@ extern "C" int ogb_latent_attention(const void* q, void* out, const void* pool, 
   if (rc == -2) rc = elem == kElemBF16 ? launch_warp<__nv_bfloat16>(p, s) : elem == kElemF32 ? launch_warp<float>(p, s) : -3;
   if (rc != 0 || p.num_splits == 1) return rc;
   const int blocks = (rows * heads + 3) / 4;
-  if (elem == kElemBF16)
-    latent_combine_kernel<<<blocks, 128, 0, s>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), ctx_len, rows, heads, rank, ldq, p.num_splits);
-  else
-    latent_combine_kernel<<<blocks, 128, 0, s>>>(part_o, part_ml, static_cast<float*>(out), ctx_len, rows, heads, rank, ldq, p.num_splits);
+  if (elem == kElemBF16) latent_combine_kernel<__nv_bfloat16><<<blocks, 128, 0, s>>>(p);
+  else latent_combine_kernel<float><<<blocks, 128, 0, s>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 

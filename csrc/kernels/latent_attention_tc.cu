@@ -11,7 +11,7 @@
 //               accumulator (the scheme of attention_tc.cu; a thread owns one row)
 //   epilogue  : the groups merge through shared memory and store bf16 rows, or fp32 partials when the keys are split
 //
-// A CTA produces OC of the R output columns (blockIdx.y picks them), so two accumulators and two score buffers fit tensor
+// A CTA produces OC of the output columns (blockIdx.y picks them; the values are the first columns of a key), so two accumulators and two score buffers fit tensor
 // memory for every R; for R > OC the scores are computed once per column chunk.  Ranks that are no multiple of 64 are
 // rounded up: the tensor maps fill the missing columns with zeros.  Every wait is bounded and watches an abort flag.
 #include <algorithm>
@@ -38,7 +38,7 @@ struct LtCfg {
   static constexpr int kColS = 2 * OC;
   static constexpr int kTmemCols = 512;
   static constexpr int kXPitch = (OC / 2 + 4) * 4;
-  static_assert(R % 64 == 0 && R % OC == 0 && (OC == 64 || OC == 128) && BN % 32 == 0, "tile shape");
+  static_assert(R % 64 == 0 && R >= OC && (OC == 64 || OC == 128) && BN % 32 == 0, "tile shape");
   static_assert(2 * OC + 2 * BN <= 512, "TMEM budget");
   static_assert(2 * kLtBM * kXPitch <= kQBytes + ST * kKBytes, "the exchange slab reuses the operand buffers");
   static_assert(kSmemBytes <= 227 * 1024, "shared memory");
@@ -350,7 +350,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __gr
     const float l_all = l_mine * a + other.y * b;
     const bool split = p.num_splits > 1;
     if (!split) {
-      const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+      const float inv = l_all > 0.f && row < rw.rows ? latent_gate<__nv_bfloat16>(p, static_cast<int64_t>(rw.row0) + row) / l_all : 0.f;
       a *= inv; b *= inv;
     }
     const float* src = reinterpret_cast<const float*>(xo + (static_cast<size_t>(g ^ 1) * kLtBM + row) * Cfg::kXPitch);
@@ -370,7 +370,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __gr
 #pragma unroll
       for (int v = 0; v < 4; ++v) {
         const int col = col0 + g * HC + 32 * c + 8 * v;
-        if (col >= p.rank) continue;                     // rank is a multiple of 8
+        if (col >= p.vrank) continue;                    // a multiple of 8
         float r[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
@@ -379,11 +379,11 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __gr
           r[j] = mine + (b > 0.f ? src[32 * c + 8 * v + j] * b : 0.f);
         }
         if (split) {
-          float4* po = reinterpret_cast<float4*>(p.part_o + pr * p.rank + col);
+          float4* po = reinterpret_cast<float4*>(p.part_o + pr * p.vrank + col);
           po[0] = make_float4(r[0], r[1], r[2], r[3]);
           po[1] = make_float4(r[4], r[5], r[6], r[7]);
         } else {
-          *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.out) + orow * p.ldq + col) =
+          *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.out) + orow * p.ldo + col) =
               make_uint4(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]), pack_bf16(r[4], r[5]), pack_bf16(r[6], r[7]));
         }
       }
@@ -418,23 +418,25 @@ static int launch_lt(const LatParams& p, cudaStream_t stream) {
     attr_set = true;
   }
   const int q_per_tile = ((p.cu_q == nullptr ? 1 : 64) * p.heads + kLtBM - 1) / kLtBM;
-  const dim3 grid((p.cu_q == nullptr ? p.rows : p.num_tiles) * q_per_tile, (std::min(R, p.rank) + OC - 1) / OC, p.num_splits);
+  const dim3 grid((p.cu_q == nullptr ? p.rows : p.num_tiles) * q_per_tile, (p.vrank + OC - 1) / OC, p.num_splits);
   latent_attention_tc_kernel<R, OC, BN, ST><<<grid, kLtThreads, Cfg::kSmemBytes, stream>>>(q_map, c_map, p, q_per_tile);
   return static_cast<int>(cudaGetLastError());
 }
 
 int launch_latent_tc(const LatParams& p, cudaStream_t stream) {
-  if (p.rank > 512 || p.rank % 8 != 0 || p.ldq % 8 != 0 || p.ldp % 8 != 0 || p.num_pages <= 0) return -2;
+  if (p.rank > 576 || p.vrank > 512 || (p.rank | p.vrank | p.ldo) % 8 != 0 || p.ldq % 8 != 0 || p.ldp % 8 != 0 || p.num_pages <= 0) return -2;
   if ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.out) | reinterpret_cast<uintptr_t>(p.pool) |
        reinterpret_cast<uintptr_t>(p.part_o)) & 15) return -2;
   if (p.cu_q == nullptr) return launch_latent_decode(p, stream);
   if (p.scale <= 0.f) return -2;           // the row maximum is taken before scaling
   if (p.rank <= 64) return launch_lt<64, 64, 128, 4>(p, stream);
   if (p.rank <= 128) return launch_lt<128, 128, 128, 4>(p, stream);
-  if (p.rank <= 192) return launch_lt<192, 64, 128, 3>(p, stream);
+  if (p.rank <= 192) return p.vrank <= 128 ? launch_lt<192, 128, 128, 3>(p, stream) : launch_lt<192, 64, 128, 3>(p, stream);
   if (p.rank <= 256) return launch_lt<256, 128, 64, 4>(p, stream);
+  if (p.rank <= 320 && p.vrank <= 256) return launch_lt<320, 128, 64, 3>(p, stream);
   if (p.rank <= 384) return launch_lt<384, 128, 64, 2>(p, stream);
-  return launch_lt<512, 128, 32, 2>(p, stream);
+  if (p.rank <= 512) return launch_lt<512, 128, 32, 2>(p, stream);
+  return launch_lt<576, 128, 32, 2>(p, stream);
 }
 
 }  // namespace ogb

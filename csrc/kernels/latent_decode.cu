@@ -5,7 +5,7 @@
 // the kernel is laid out around the byte stream instead:
 //
 //   last warp    : TMA producer, 64 tokens (4 pages) x R values per stage, 128-byte swizzled column chunks
-//   8 or 16 warps: S = Q' C^T split four ways over the latent's columns and two or four ways over the tokens (a warp keeps its
+//   8 or 16 warps: (R key columns, of which the first V are values) S = Q' C^T split four ways over the latent's columns and two or four ways over the tokens (a warp keeps its
 //                  slice of Q' in registers where they suffice), partial scores summed through shared memory, softmax with all
 //                  threads, then O += P C with every warp owning its share of the output columns
 //
@@ -20,7 +20,7 @@ namespace ogb {
 constexpr int kLdKeys = 64;
 constexpr int kLdPitch = 72;             // floats per row of partial scores: conflict-free 8-byte stores
 
-template <int R, int MT, int ST, int NW>
+template <int R, int V, int MT, int ST, int NW>
 struct LdCfg {
   static constexpr int kRows = 16 * MT;
   static constexpr int kChunks = R / 64;
@@ -29,6 +29,7 @@ struct LdCfg {
   static constexpr int kPBytes = kRows * 128;
   static constexpr int kSBytes = 4 * kRows * kLdPitch * 4;
   static constexpr int kSmemBytes = ST * kStage + kQBytes + kPBytes + kSBytes + 1024 /*alignment*/ + 512 /*barriers, row factors*/ + 256;
+  static_assert(R % 64 == 0 && V % (8 * NW) == 0 && V <= R, "tile shape");
   static_assert(kSmemBytes <= 227 * 1024, "shared memory");
 };
 
@@ -59,27 +60,27 @@ OGB_DEVICE void ld_merge(const LatParams& p, int* counter, size_t row0, int head
       const float ms = __ldcg(ml + 2 * s);
       if (ms != -INFINITY) l += __ldcg(ml + 2 * s + 1) * expf(ms - m);
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    for (int c = lane * 4; c < p.rank; c += 128) {
+    const float inv = (l > 0.f ? 1.f / l : 0.f) * latent_gate<__nv_bfloat16>(p, row0 + row);
+    for (int c = lane * 4; c < p.vrank; c += 128) {
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int s = 0; s < p.num_splits; ++s) {
         const float ms = __ldcg(ml + 2 * s);
         if (ms == -INFINITY) continue;
         const float w = expf(ms - m) * inv;
-        const float4 o = __ldcg(reinterpret_cast<const float4*>(p.part_o + ((row0 + row) * p.num_splits + s) * p.rank + c));
+        const float4 o = __ldcg(reinterpret_cast<const float4*>(p.part_o + ((row0 + row) * p.num_splits + s) * p.vrank + c));
         a.x = fmaf(w, o.x, a.x); a.y = fmaf(w, o.y, a.y); a.z = fmaf(w, o.z, a.z); a.w = fmaf(w, o.w, a.w);
       }
-      *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldq + c) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
+      *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldo + c) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
     }
   }
 }
 
-template <int R, int MT, int ST, int NW>
+template <int R, int V, int MT, int ST, int NW>
 __global__ void __launch_bounds__((NW + 1) * 32, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap c_map, const LatParams p) {
-  using Cfg = LdCfg<R, MT, ST, NW>;
+  using Cfg = LdCfg<R, V, MT, ST, NW>;
   constexpr int KS = R / 64;             // k-steps of a warp's column slice (R / 4 columns)
-  constexpr int NT = R / (8 * NW);       // 8-column output tiles of a warp
+  constexpr int NT = V / (8 * NW);       // 8-column output tiles of a warp
   constexpr int KN = 4 / (NW / 4);       // 16-token score tiles of a warp: NW / 4 warps share a column slice
   constexpr int TPR = NW * 32 / (16 * MT), KPT = kLdKeys / TPR;   // softmax: threads a row, tokens a thread
   extern __shared__ uint8_t smem_raw[];
@@ -274,7 +275,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         uint32_t b[4];
-        ldsm_x4_t(kb + ld_off(kLdKeys, kk * 32 + lane, warp * (R / NW) + n * 8), b[0], b[1], b[2], b[3]);
+        ldsm_x4_t(kb + ld_off(kLdKeys, kk * 32 + lane, warp * (V / NW) + n * 8), b[0], b[1], b[2], b[3]);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma_bf16_16816(o[m][n], pf[m][0], b[0], b[1]);
@@ -292,7 +293,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
 #pragma unroll
     for (int x = 1; x < TPR; x <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
     if (sub == 0) {
-      sA[srow] = split ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
+      sA[srow] = split ? 1.f : (l_run > 0.f && srow < heads ? latent_gate<__nv_bfloat16>(p, row0 + srow) / l_run : 0.f);
       if (split && srow < heads) {
         const size_t pr = (row0 + srow) * p.num_splits + blockIdx.z;
         p.part_ml[2 * pr] = m_run * 0.6931471805599453f;
@@ -310,13 +311,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       const float f = sA[row];
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
-        const int col = warp * (R / NW) + n * 8 + 2 * t;
-        if (col >= p.rank) continue;
+        const int col = warp * (V / NW) + n * 8 + 2 * t;
+        if (col >= p.vrank) continue;
         const float x = o[m][n][2 * hrow] * f, y = o[m][n][2 * hrow + 1] * f;
         if (split)
-          *reinterpret_cast<float2*>(p.part_o + ((row0 + row) * p.num_splits + blockIdx.z) * p.rank + col) = make_float2(x, y);
+          *reinterpret_cast<float2*>(p.part_o + ((row0 + row) * p.num_splits + blockIdx.z) * p.vrank + col) = make_float2(x, y);
         else
-          *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldq + col) = pack_bf16(x, y);
+          *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + row) * p.ldo + col) = pack_bf16(x, y);
       }
     }
   const bool aborted = *abort_flag != 0;
@@ -328,9 +329,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   }
 }
 
-template <int R, int MT, int ST, int NW>
+template <int R, int V, int MT, int ST, int NW>
 static int launch_ld(const LatParams& p, cudaStream_t stream) {
-  using Cfg = LdCfg<R, MT, ST, NW>;
+  using Cfg = LdCfg<R, V, MT, ST, NW>;
   CUtensorMap q_map, c_map;
   int rc = make_tmap_bf16_2d(&q_map, p.q, static_cast<uint64_t>(p.rows) * p.heads, p.rank, p.ldq, Cfg::kRows, 64);
   if (rc != 0) return rc;
@@ -338,20 +339,24 @@ static int launch_ld(const LatParams& p, cudaStream_t stream) {
   if (rc != 0) return rc;
   static bool attr_set = false;
   if (!attr_set) {
-    OGB_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<R, MT, ST, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    OGB_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<R, V, MT, ST, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
     attr_set = true;
   }
   const dim3 grid(p.rows, (p.heads + Cfg::kRows - 1) / Cfg::kRows, p.num_splits);
-  latent_decode_kernel<R, MT, ST, NW><<<grid, (NW + 1) * 32, Cfg::kSmemBytes, stream>>>(q_map, c_map, p);
+  latent_decode_kernel<R, V, MT, ST, NW><<<grid, (NW + 1) * 32, Cfg::kSmemBytes, stream>>>(q_map, c_map, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <int MT>
 static int dispatch_ld(const LatParams& p, cudaStream_t stream) {
-  if (p.rank <= 64) return launch_ld<64, MT, 4, 8>(p, stream);
-  if (p.rank <= 128) return launch_ld<128, MT, 4, 8>(p, stream);
-  if (p.rank <= 256) return launch_ld<256, MT, 4, 16>(p, stream);
-  return launch_ld<512, MT, 2, 16>(p, stream);
+  if (p.rank <= 64) return launch_ld<64, 64, MT, 4, 8>(p, stream);
+  if (p.rank <= 128) return launch_ld<128, 128, MT, 4, 8>(p, stream);
+  if (p.rank <= 192 && p.vrank <= 128) return launch_ld<192, 128, MT, 4, 8>(p, stream);
+  if (p.rank <= 256) return launch_ld<256, 256, MT, 4, 16>(p, stream);
+  if (p.rank <= 320 && p.vrank <= 256) return launch_ld<320, 256, MT, 3, 16>(p, stream);
+  if (p.rank <= 512) return launch_ld<512, 512, MT, 2, 16>(p, stream);
+  if (p.vrank <= 512) return launch_ld<576, 512, MT, 2, 16>(p, stream);
+  return -2;
 }
 
 int launch_latent_decode(const LatParams& p, cudaStream_t stream) {

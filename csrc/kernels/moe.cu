@@ -19,10 +19,12 @@ namespace ogb {
 
 constexpr int kMaxExperts = 256;
 
-// `groups` > 1: experts form that many equal groups of neighbours, a group scores as its best expert, and only the `keep` best
-// groups can be chosen from.
+// `bias` (fp32, or null) is added to the logits.  The choice compares logits, which order experts as their scores do.  `groups` > 1:
+// experts form that many equal groups of neighbours, a group scores as its best expert, and only the `keep` best groups can be
+// chosen from.
 template <typename T>
-__global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict__ logits, int* __restrict__ topk_ids, float* __restrict__ topk_w,
+__global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ topk_ids,
+                                                             float* __restrict__ topk_w,
                                                              int tokens, int experts, int k, int renormalize, int ld, int groups, int keep) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   __shared__ float s_group[8][kMaxExperts];
@@ -33,26 +35,23 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
-    v[i] = (e < experts) ? static_cast<float>(logits[static_cast<size_t>(warp) * ld + e]) : -INFINITY;
+    v[i] = (e < experts) ? static_cast<float>(logits[static_cast<size_t>(warp) * ld + e]) + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
     mx = fmaxf(mx, v[i]);
   }
   mx = warp_max(mx);
   float sum = 0.f;
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    v[i] = (i * 32 + lane < experts) ? expf(v[i] - mx) : 0.f;
-    sum += v[i];
-  }
+  for (int i = 0; i < PER; ++i) sum += (i * 32 + lane < experts) ? expf(v[i] - mx) : 0.f;
   sum = warp_sum(sum);
   const float inv = 1.f / sum;
-  // the largest of a set of values with the lowest index among equals
+  // the largest of a set of values with the lowest index among equals (-inf: not a candidate)
   auto best_of = [&](const float (&x)[PER], int count, float& best, int& at) {
-    best = -1.f;
+    best = -INFINITY;
     at = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int e = i * 32 + lane;
-      if (e < count && (x[i] > best || (x[i] == best && e < at))) { best = x[i]; at = e; }
+      if (e < count && x[i] > best) { best = x[i]; at = e; }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -71,7 +70,7 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int g = i * 32 + lane;
-      gs[i] = -1.f;
+      gs[i] = -INFINITY;
       if (g < groups)
         for (int e = 0; e < size; ++e) gs[i] = fmaxf(gs[i], s[g * size + e]);
     }
@@ -86,13 +85,13 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
       if (lane == 0 && at < groups) s[at] = 1.f;
 #pragma unroll
       for (int i = 0; i < PER; ++i)
-        if (i * 32 + lane == at) gs[i] = -2.f;
+        if (i * 32 + lane == at) gs[i] = -INFINITY;
     }
     __syncwarp();
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int e = i * 32 + lane;
-      if (e < experts && s[e / size] == 0.f) v[i] = -1.f;
+      if (e < experts && s[e / size] == 0.f) v[i] = -INFINITY;
     }
   }
   float chosen_sum = 0.f;
@@ -102,15 +101,16 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
     float best;
     int best_e;
     best_of(v, experts, best, best_e);
-    if (lane == r) { my_w = best * inv; my_id = best_e; }
-    chosen_sum += best * inv;
+    best = expf(best - mx);
+    if (lane == r) { my_w = best; my_id = best_e; }
+    chosen_sum += best;
 #pragma unroll
     for (int i = 0; i < PER; ++i)
-      if (i * 32 + lane == best_e) v[i] = -1.f;                // remove the winner
+      if (i * 32 + lane == best_e) v[i] = -INFINITY;           // remove the winner
   }
   if (lane < k) {
     topk_ids[static_cast<size_t>(warp) * k + lane] = my_id;
-    topk_w[static_cast<size_t>(warp) * k + lane] = renormalize ? my_w / chosen_sum : my_w;
+    topk_w[static_cast<size_t>(warp) * k + lane] = renormalize ? my_w / chosen_sum : my_w * inv;
   }
 }
 
@@ -213,27 +213,27 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ ys, const i
 using namespace ogb;
 
 template <typename T>
-static int route_topk(const T* logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize, int ld, int groups, int keep,
+static int route_topk(const T* logits, const float* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize, int ld, int groups, int keep,
                       void* stream) {
   if (tokens <= 0) return 0;
   if (experts > kMaxExperts || k > 32 || k > experts) return -3;
   if (groups < 1 || experts % groups != 0 || keep < 1 || keep > groups || k > keep * (experts / groups)) return -3;
   const int warps_per_block = 8;
   const int blocks = (tokens + warps_per_block - 1) / warps_per_block;
-  moe_route_topk_kernel<T><<<blocks, warps_per_block * 32, 0, static_cast<cudaStream_t>(stream)>>>(logits, topk_ids, topk_w, tokens, experts, k,
-                                                                                                 renormalize, ld, groups, keep);
+  moe_route_topk_kernel<T><<<blocks, warps_per_block * 32, 0, static_cast<cudaStream_t>(stream)>>>(logits, bias, topk_ids, topk_w, tokens,
+                                                                                                 experts, k, renormalize, ld, groups, keep);
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int ogb_moe_route_topk(const void* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k,
                                   int renormalize, int ld, void* stream) {
-  return route_topk(static_cast<const __nv_bfloat16*>(router_logits), topk_ids, topk_w, tokens, experts, k, renormalize, ld, 1, 1, stream);
+  return route_topk(static_cast<const __nv_bfloat16*>(router_logits), nullptr, topk_ids, topk_w, tokens, experts, k, renormalize, ld, 1, 1, stream);
 }
 
-// fp32 logits; `groups` equal groups of experts of which the `keep` best can be chosen from (1, 1: all).
-extern "C" int ogb_moe_route_grouped(const float* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize,
+// fp32 logits and bias (or null); `groups` equal groups of experts of which the `keep` best can be chosen from (1, 1: all).
+extern "C" int ogb_moe_route_grouped(const float* router_logits, const float* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize,
                                      int ld, int groups, int keep, void* stream) {
-  return route_topk(router_logits, topk_ids, topk_w, tokens, experts, k, renormalize, ld, groups, keep, stream);
+  return route_topk(router_logits, bias, topk_ids, topk_w, tokens, experts, k, renormalize, ld, groups, keep, stream);
 }
 
 // counts must be zero on entry (the caller clears it); e0 = first expert owned by this rank.

@@ -24,9 +24,10 @@ int ogb_gemm_bf16_wait(const void* A, const void* W, void* C, const void* bias, 
                        int N, int K, int lda, int ldw, int ldc, int ldr, int epilogue, int bn, uint32_t* a_ready,
                        uint32_t* a_done, unsigned long long a_wait_ns, int* status, void* stream);
 
-// Gated product over a packed gate | up weight (tile width bn), activation act: 0 = silu, 1 = tanh form of gelu.
-int ogb_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, int bn,
-                        int* status, void* stream);
+// Product with an activation (common.cuh Act: 1 silu, 2 tanh form of gelu, 4 clamped gate over a packed gate | up weight, tile width
+// bn; 3 square of relu, 5 xielu on every result) and its numbers.
+int ogb_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b, int bn,
+                      int* status, void* stream);
 // `batch` products of one shape: C[:, z*c_step : +N] = A[:, z*a_step : +K] * W[z*N : +N, :]^T (steps are multiples of 8).
 int ogb_gemm_bf16_batched(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step,
                           int c_step, int* status, void* stream);
@@ -35,6 +36,8 @@ int ogb_gemm_bf16_paged(const void* A, const void* W, void* C, int M, int N, int
 // Products as ogb_gemm_bf16_batched in fp32 without any reduced-precision mode.
 int ogb_gemm_f32(const float* A, const float* W, float* C, int M, int N, int K, int lda, int ldw, int ldc, int batch, int a_step, int c_step,
                  void* stream);
+int ogb_gemm_f32_act(const float* A, const float* W, float* C, int M, int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b,
+                     void* stream);
 
 // Stream-K decomposition of the GEMMs (on by default; OGB_STREAM_K=0 disables it): 1 / 0 sets it, the old value is returned.
 int ogb_gemm_set_stream_k(int on);
@@ -73,6 +76,11 @@ int ogb_paged_prefill_tc_bf16(const void* q, void* out, const void* pool, const 
                               const int* cu_q, const int* tile_seq, const int* tile_q0, int num_tiles, int num_seqs,
                               int q_rows, int max_pages, int64_t num_pages, int hq, int hkv, int d, int q_stride,
                               int o_stride, float scale, int window, int sink, int* status, void* stream);
+// Over pages of 64-column chunks (attention_tc.cu): keys of kc chunks, values of vc chunks, per head.
+int ogb_paged_prefill_chunks_bf16(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
+                                  const int* tile_seq, const int* tile_q0, const void* gate, int num_tiles, int num_seqs, int q_rows, int max_pages,
+                                  int64_t num_pages, int heads, int kc, int vc, int dv, int q_head, int o_head, int q_stride, int o_stride, int ldg,
+                                  float scale, int window, int* status, void* stream);
 int ogb_paged_decode_bf16(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len,
                           int num_seqs, int max_pages, int64_t num_pages, int hq, int hkv, int d, int q_stride,
                           int o_stride, float scale, int num_splits, float* part_o, float* part_ml, int window,
@@ -166,13 +174,18 @@ int ogb_hyper_step(const float* x_in, float* x_out, const void* y, const float* 
                    const float* w, const float* b, const float* shift, float* prev, void* h, const int* gather, int rows, int total_rows, int S,
                    int W, int ldy, int ldh, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0,
                    int num_decode, int num_tiles, int num_slots, int elem, int* status, void* stream);
-int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, int elem, int* status, void* stream);
-int ogb_latent_append(const void* c, int ldc, const float* w, float eps, const int* slots, void* pool, int tokens, int rank, int ldp,
-                      int64_t num_slots, int elem, int* status, void* stream);
+// embed_streams: w (or null): RMS norm of the embedding; copy (or null): the same row again, [tokens, ldc].
+int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, const float* w, float eps, void* copy, int ldc,
+                      int elem, int* status, void* stream);
+// Latents and rotated key parts to their pages, rotated query parts to q_out or in place (hybrid.cu).
+int ogb_latent_append(void* row, int ldr, int latent, const float* w, float eps, const int* slots, void* pool, int tokens, int rank, int ldp,
+                      int64_t num_slots, const double* freq, const int* positions, void* q_out, int heads, int dim, int rot, int ldq, int q_col, int split,
+                      int elem, int* status, void* stream);
+// rank values of a page row are the key, the first vrank the value; gate (or null) [rows, ldg]: a head's output times its sigmoid.
 int ogb_latent_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q,
-                         const int* tile_seq, const int* tile_q0, int rows, int heads, int rank, int ldq, int ldp, int max_pages, int num_tiles,
-                         int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml, int* counters, int elem, int* status,
-                         void* stream);
+                         const int* tile_seq, const int* tile_q0, const void* gate, int rows, int heads, int rank, int vrank, int ldq, int ldo, int ldp,
+                         int ldg, int max_pages, int num_tiles, int64_t num_pages, int window, float scale, int num_splits, float* part_o, float* part_ml,
+                         int* counters, int elem, int* status, void* stream);
 int ogb_latent_gather(const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, int entries, int max_pages, int64_t num_pages,
                       int window, int ldp, int blocks, void* out, int* scratch_table, int* status, void* stream);
 int ogb_latent_set_tc(int on);
@@ -182,9 +195,16 @@ int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* stat
               int num_segments, float* seg_state, float* seg_gate, int split, int* status, void* stream);
 int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate, int ldg,
                      int elem, void* stream);
-// norm_step: x += rms(y) post, h = rms(x) w over one fp32 residual stream; y may be the weighted sum of a token's expert rows.
-int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const float* post, const float* w, void* h, const int* gather, float eps,
-                  int rows, int total_rows, int W, int k, int ldy, int ldh, int64_t y_rows, int elem, int* status, void* stream);
+// norm_step: x += rms(y) post, h = rms(x) w over one fp32 residual stream; y may be the weighted sum of a token's expert rows and a
+// gated row of a shared expert.
+int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const void* shared, const float* gate, const float* post, const float* w,
+                  void* h, const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int lds, int ldg, int ldh, int64_t y_rows,
+                  int elem, int* status, void* stream);
+// norm_conv_step: x_out = x_in + y + add, h = a causal convolution over rms(x_out) w.
+int ogb_norm_conv_step(const float* x_in, float* x_out, const void* y, const int* pos, const float* weight, const void* shared, const float* gate,
+                       const float* add, const float* w, const float* conv, float* state, void* h, float eps, int W, int taps, int k, int ldx, int ldy,
+                       int lds, int ldg, int ldh, int64_t y_rows, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq,
+                       const int* tile_q0, int num_decode, int num_tiles, int num_slots, int elem, int* status, void* stream);
 // Short causal convolutions (short_conv.cu): w [taps, channels], state [slots, taps - 1, channels].
 // Attention: q (nq heads of d) | k (nk) | v (nv heads of dv); rotated queries to q, keys and values to pages [nk][16][dp] | [nv][16][vp].
 int ogb_conv_rope_append(const void* u, int ldu, const float* w, const float* bias, float* state, int taps, void* q, int ldq, void* pool,
@@ -207,7 +227,7 @@ int ogb_diff_attention(const void* q, void* out, const void* pool, const int* pa
                        int dp, int vp, int ldq, int ldo, int window, int keep, float scale, float lambda, float eps, float gain, int num_splits,
                        float* part_o, float* part_ml, int* counters, int elem, int* status, void* stream);
 int ogb_diff_set_tc(int on);
-int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, int elem, void* stream);
+int ogb_act_mul_packed(const void* gate_up, void* out, int rows, int inter, int half, int act, float act_a, float act_b, int elem, void* stream);
 int ogb_argmax_f32(const float* logits, int* out_tokens, int rows, int vocab, int ld, void* stream);
 int ogb_sample_f32(const float* logits, int* out_tokens, const float* temperature, const int* top_k, const float* top_p, const float* min_p,
                    const float* uniform, uint32_t* work, int rows, int vocab, int ld, void* stream);
@@ -219,13 +239,13 @@ int ogb_moe_permute(const int* topk_ids, int* counts, int* offsets, int* cursor,
                     int* tile_tab, int* meta, int tokens, int k, int e0, int experts, int max_mtiles, void* stream);
 int ogb_moe_gather_rows(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int hidden,
                         void* stream);
-int ogb_moe_route_grouped(const float* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize, int ld,
-                          int groups, int keep, void* stream);
+int ogb_moe_route_grouped(const float* router_logits, const float* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize,
+                          int ld, int groups, int keep, void* stream);
 int ogb_moe_gather_bytes(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int row_bytes, void* stream);
 int ogb_grouped_gemm_act(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows, int max_mtiles,
-                         int N, int K, int lda, int ldw, int ldc, int act, int bn, int* status, void* stream);
+                         int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b, int bn, int* status, void* stream);
 int ogb_grouped_gemm_f32(const float* A, const float* W, float* C, const int* group_tab, const int* group_mtiles, int max_rows, int max_mtiles, int N,
-                         int K, int lda, int ldw, int ldc, int act, void* stream);
+                         int K, int lda, int ldw, int ldc, int act, float act_a, float act_b, void* stream);
 int ogb_moe_combine(const void* ys, const int* route_pos, const float* topk_w, void* out, int tokens, int k, int hidden,
                     int accumulate, void* stream);
 int ogb_grouped_gemm_bf16(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts,

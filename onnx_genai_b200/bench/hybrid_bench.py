@@ -187,7 +187,7 @@ def kernel_rows(size: str, timer, pk):
             row("graph operator: linear_attention (gated)", phase, la, nbytes=t * heads * d * 10 + 2 * b * heads * d * d * 2)
         # latent attention
         c, wn, pool = rnd(t, rank), f32(rank), rnd(npages, 16, rank)
-        row("latent_append", phase, lambda: hops.latent_append(c, wn, 1e-6, si.slots, pool, rank), nbytes=2 * t * rank * 2)
+        row("latent_append", phase, lambda: hops.latent_append(c, 0, wn, 1e-6, si.slots, pool, rank), nbytes=2 * t * rank * 2)
         q, uk, qa, oc = rnd(t, heads * d), rnd(heads * rank, d), rnd(t, heads * rank), torch.empty(t, heads * rank, dtype=bf, device="cuda")
         uv, o = rnd(heads * d, rank), torch.empty(t, heads * d, dtype=bf, device="cuda")
         wb = heads * rank * d * 2
@@ -201,11 +201,11 @@ def kernel_rows(size: str, timer, pk):
                 4 * pairs * heads * rank, keys * rank * 2 + 2 * t * heads * rank * 2)
             if rank > d:      # what prompts of this shape run on
                 pages = hops.visible_pages(si, window)
-                dense, kvp = torch.empty(pages * 16, rank, dtype=bf, device="cuda"), torch.empty(pages, heads, 2, 16, d, dtype=bf, device="cuda")
+                dense, kvp = torch.empty(pages * 16, rank, dtype=bf, device="cuda"), torch.empty(pages, heads, 2 * d // 64, 16, 64, dtype=bf, device="cuda")
                 table, kvw, qd = torch.zeros(nseq, mp, dtype=torch.int32, device="cuda"), rnd(heads * 2 * d, rank), rnd(t, heads * d)
                 od = torch.empty(t, heads * d, dtype=bf, device="cuda")
-                row("latent prompt, expanded K/V (3 kernels)", phase, lambda: hops.latent_prefill_expanded(qd, od, pool, kvw, si, heads, d, 0.1, window,
-                                                                                                          pages, dense, kvp, table),
+                row("latent prompt, expanded K/V (3 kernels)", phase, lambda: hops.latent_prefill_expanded(qd, od, pool, kvw, si, heads, d // 64, d // 64, d, d, 0.1,
+                                                                                                          window, pages, dense, kvp, table),
                     4 * pairs * heads * d + 2 * pages * 16 * rank * heads * 2 * d, 2 * pages * 16 * heads * 2 * d * 2)
         else:
             cnt = torch.zeros(4096, dtype=torch.int32, device="cuda")

@@ -45,7 +45,9 @@ PRECISE_SOURCES = {"hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_a
 SUBSETS = {"hybrid": ("hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_attention_tc.cu", "latent_decode.cu", "attention_tc.cu", "attention.cu", "gemm_tcgen05.cu",
                       "sampling.cu", "tp_comm.cu"),
            "delta": ("hybrid.cu", "short_conv.cu", "delta_rule.cu", "diff_attention.cu", "diff_attention_tc.cu", "moe.cu", "gemm_tcgen05.cu", "sampling.cu",
-                     "tp_comm.cu")}
+                     "tp_comm.cu"),
+           "latent_moe": ("hybrid.cu", "latent_attention.cu", "latent_attention_tc.cu", "latent_decode.cu", "attention_tc.cu", "attention.cu", "moe.cu",
+                          "gemm_tcgen05.cu", "sampling.cu", "tp_comm.cu")}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-fopenmp", "-mavx2", "-mfma"]
 
 

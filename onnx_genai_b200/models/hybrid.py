@@ -1,19 +1,24 @@
 """Decoder whose layers each choose a mixer -- recurrent (HGRN2, gated delta rule) or attention (over paged latents, differential) --
-and a feed-forward (gated, routed experts), on hyper-connected residual streams or on one stream normed around every sublayer.
+and a feed-forward (gated or not, routed experts), on hyper-connected residual streams or on one stream normed before -- and
+behind -- every sublayer.  A range of layers may run several times in a row with the same weights.
 
 A design of this kind is a :class:`HybridConfig` (layer specs plus constants) and a :class:`HybridWeights`;
 ``models/registry.py`` says which checkpoint architectures map here and how their files are read.  The executor lowers
-a layer to a fixed list of launches over buffers allocated once:
+a layer run to a fixed list of launches over buffers allocated once:
 
     hyper_step (fold the last sublayer's output into the streams, read-out, norm, token shift), or
-    norm_step  (x += norm(the last sublayer's output), norm; sums the rows of routed experts on the way)
+    norm_step  (x += norm(the last sublayer's output), norm; sums the rows of routed experts on the way), or
+    norm_conv_step (x += the last sublayer's output, norm, causal convolution of what the sublayer reads)
+    pass:       norm_step (x += the last sublayer's output, copy beside the embedding) | gemm(x | embedding, fp32 out)
     recurrent:  gemm(q | gate | v, fp32 out) | hgrn2 | head_rmsnorm | gemm(o)
     delta:      gemm(gate | q | k | v) | gemm(decay | step size, fp32 out) | conv_unit_gates | delta_rule | head_rmsnorm * gate | gemm(o)
-    latent:     gemm(q | latent) | latent_append | gemm per head (W_uk^T q) | latent_attention | gemm per head (W_uv o) | gemm(o);
+    latent:     gemm(q | latent | rotated key | head gates) | latent_append (norm, rotations) | gemm per head (W_uk^T q) |
+                latent_attention (head gates in its epilogue) | gemm per head (W_uv o) | gemm(o);
                 prompts over wide latents: latent_gather | gemm (K | V pages) | paged_prefill | gemm(o)
     diff:       gemm(q | k | v) | conv_rope_append | diff_attention (both maps, difference and norm) | gemm(o)
-    dense:      hyper_step or norm_step | gemm(gate_up, gated epilogue) | gemm(down)
-    experts:    norm_step | gemm(router, fp32 out) | route, permute, gather | grouped gemm(up, relu^2 epilogue) | grouped gemm(down)
+    dense:      gemm(gate_up or up, activation in the epilogue) | gemm(down)
+    experts:    gemm(router | shared gate, fp32 out) | route, permute, gather | grouped gemm(up, activation epilogue) | grouped gemm(down)
+                shared expert: gemm(gate_up, gated epilogue) | gemm(down)
 
 The residual streams, norms, gates and recurrent state are fp32 in every engine; matrix products and the activations
 between them are bf16, or fp32 throughout in the 32-bit engine (``EngineConfig.compute_dtype``).
@@ -30,7 +35,7 @@ import torch
 from .. import ops
 from ..ops import hybrid as hops
 from ..ops import moe as moe_ops
-from ..ops.hybrid import DynamicTanh, HyperConnection, RmsNorm
+from ..ops.hybrid import Act, DynamicTanh, ExpertRows, HyperConnection, LatentRope, RmsNorm
 from .decoder import pad_mlp, pick_swiglu_half
 
 
@@ -51,7 +56,9 @@ class RecurrentSpec:
 
 @dataclass
 class LatentSpec:
-    """Latent attention: ``window`` 0 means every earlier token; ``kv_from`` names the layer whose latents are read."""
+    """Latent attention: ``window`` 0 means every earlier token; ``kv_from`` names the layer whose latents are read.  ``rot_dim``: rotated
+    dimensions of every query head, and of a key part that all heads share and that lies behind the latent in its page row;
+    ``gated``: every head's output is multiplied by the sigmoid of a projection of the mixer's input."""
     heads: int
     dim: int
     vdim: int
@@ -59,6 +66,32 @@ class LatentSpec:
     scale: float
     window: int = 0
     kv_from: int | None = None
+    rot_dim: int = 0
+    rot_base: float = 10000.0
+    gated: bool = False
+
+    @property
+    def q_width(self) -> int:
+        """Columns of a projected query head."""
+        return pad8(self.dim) + pad8(self.rot_dim)
+
+    @property
+    def key_width(self) -> int:
+        """Columns of a page row, and of a query head folded to meet it."""
+        return pad8(self.rank) + pad8(self.rot_dim)
+
+    @property
+    def latent_col(self) -> int:
+        """Where the latent begins in a projected row."""
+        return self.heads * self.q_width
+
+    @property
+    def gate_col(self) -> int:
+        return self.latent_col + (self.key_width if self.kv_from is None else 0)
+
+    @property
+    def proj_width(self) -> int:
+        return self.gate_col + (self.heads if self.gated else 0)
 
 
 @dataclass
@@ -102,25 +135,51 @@ class DiffSpec:
 
 @dataclass
 class MlpSpec:
+    """``act``: a gated activation, or "xielu" (one projection, two numbers per layer)."""
     inter: int
     act: str = "gelu_tanh"
 
 
 @dataclass
 class MoeSpec:
-    """Routed experts down(relu(up h)^2), ``top`` of ``experts`` per token, chosen from the ``keep`` best of ``groups`` equal groups."""
+    """Routed experts down(act(up h)), ``top`` of ``experts`` per token, chosen from the ``keep`` best of ``groups`` equal groups; ``act``:
+    "relu2", or "clamp_glu" with a gate and ``limit``.  ``shared_inter`` > 0: an expert of that size (and ``shared_limit``) runs for every
+    token, times the sigmoid of a projection."""
     experts: int
     top: int
     inter: int
     groups: int = 1
     keep: int = 1
     renormalize: bool = False
+    act: str = "relu2"
+    limit: float = 0.0
+    shared_inter: int = 0
+    shared_limit: float = 0.0
+    bias: bool = False
+
+    @property
+    def gated(self) -> bool:
+        return Act(self.act).gated
+
+    @property
+    def logits(self) -> int:
+        """Columns of the router's product: experts, and the shared expert's gate."""
+        return self.experts + (self.shared_inter > 0)
 
 
 @dataclass
 class LayerSpec:
     mixer: RecurrentSpec | LatentSpec | DeltaSpec | DiffSpec
     mlp: MlpSpec | MoeSpec | None = None
+
+
+@dataclass
+class LoopSpec:
+    """Layers start .. stop - 1 run ``times`` times in a row.  Ahead of every pass the residual becomes a projection of itself and the
+    embedding, plus a vector of the pass."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -132,14 +191,26 @@ class HybridConfig:
     norm_eps: float = 1e-6
     name: str = "hybrid"
     logit_scale: float = 1.0           # folded into the final norm's weight
-    residual: str = "hyper"            # "hyper": connected streams, Dynamic-Tanh norms, token shift; "sandwich": RMS norms around a sublayer
+    residual: str = "hyper"            # "hyper": connected streams, Dynamic-Tanh norms, token shift; "sandwich": RMS norms around a sublayer;
+                                       # "pre": RMS norms before a sublayer
+    input_taps: int = 0                # "pre": what a sublayer reads is h plus a causal convolution of h over this many taps (0: h)
+    loop: LoopSpec | None = None
     eos_token: int = -1
     max_position: int = 1 << 20        # no positional table: bounded by the pool only
     default_seq_len: int = 8192        # sequence limit when neither the caller nor the package names one
 
     @property
+    def runs(self) -> list:
+        """The layers in the order they run; every run has a cache and state of its own."""
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            return list(range(n))
+        return [*range(lp.start), *list(range(lp.start, lp.stop)) * lp.times, *range(lp.stop, n)]
+
+    @property
     def num_layers(self) -> int:
-        return len(self.layers)
+        """Layer runs: what caches and state are counted by."""
+        return len(self.runs)
 
     @property
     def latent_layers(self) -> list:
@@ -169,16 +240,21 @@ class HybridConfig:
     has_state = True                   # token shift, convolutions and recurrences are per-sequence state
 
     def kv_page_shape(self, layer: int, kv_heads: int = 1):
-        """Shape of one KV page of a layer, None when the layer caches nothing of its own."""
-        m = self.layers[layer].mixer
+        """Shape of one KV page of a layer run, None when it caches nothing of its own."""
+        m = self.layers[self.runs[layer]].mixer
         if isinstance(m, DiffSpec):
             return (m.page_elems,)
-        return (ops.PAGE, pad8(m.rank)) if isinstance(m, LatentSpec) and m.kv_from is None else None
+        return (ops.PAGE, m.key_width) if isinstance(m, LatentSpec) and m.kv_from is None else None
 
     def state_shapes(self, layer: int) -> dict:
-        """Per-sequence fp32 state of a layer: name -> shape."""
-        m = self.layers[layer].mixer
+        """Per-sequence fp32 state of a layer run: name -> shape."""
+        spec = self.layers[self.runs[layer]]
+        m = spec.mixer
         shapes = {"shift": (self.hidden,)} if self.residual == "hyper" else {}
+        if self.input_taps:
+            shapes["input1"] = (self.input_taps - 1, self.hidden)
+            if spec.mlp is not None:
+                shapes["input2"] = (self.input_taps - 1, self.hidden)
         if isinstance(m, (DeltaSpec, DiffSpec)):
             shapes["conv"] = (m.taps - 1, m.conv_width)
         if isinstance(m, (RecurrentSpec, DeltaSpec)):
@@ -186,15 +262,28 @@ class HybridConfig:
         return shapes
 
     def validate(self) -> None:
-        if self.residual not in ("hyper", "sandwich"):
+        if self.residual not in ("hyper", "sandwich", "pre"):
             raise ValueError(f"unknown residual {self.residual!r}")
-        if not 1 <= self.streams <= 8 or (self.residual == "sandwich" and self.streams != 1):
+        if self.input_taps and (self.residual != "pre" or not 0 <= self.input_taps <= 8):
+            raise ValueError(f"input convolutions of {self.input_taps} taps are not supported (1 to 8, behind norms before the sublayers)")
+        if self.input_taps and self.hidden > (8192 if self.hidden % 4 == 0 else 4096):
+            raise ValueError(f"input convolutions of {self.hidden} channels are not supported (8192, 4096 where they are no multiple of 4)")
+        if self.loop is not None:
+            lp = self.loop
+            if self.residual != "pre" or not 0 <= lp.start < lp.stop <= len(self.layers) or lp.times < 1:
+                raise ValueError(f"a loop over layers {lp.start} .. {lp.stop} of {len(self.layers)}, {lp.times} times, is not supported "
+                                 "(with norms before the sublayers only)")
+            if any(isinstance(l.mixer, LatentSpec) and l.mixer.kv_from is not None for l in self.layers):
+                raise ValueError("layers that read another layer's latents cannot be combined with a loop")
+        if not 1 <= self.streams <= 8 or (self.residual != "hyper" and self.streams != 1):
             raise ValueError(f"{self.streams} residual streams are not supported (1 to 8, 1 with norms around the sublayers)")
         for i, layer in enumerate(self.layers):
             m, f = layer.mixer, layer.mlp
             if isinstance(f, MoeSpec):
-                if self.residual != "sandwich":
-                    raise ValueError(f"layer {i}: routed experts need the residual with norms around the sublayers")
+                if self.residual == "hyper":
+                    raise ValueError(f"layer {i}: routed experts need a residual of one stream")
+                if f.act not in ("relu2", "clamp_glu"):
+                    raise ValueError(f"layer {i}: unknown activation {f.act!r} of routed experts")
                 if f.experts > 256 or f.top > 32 or f.groups < 1 or f.experts % f.groups or not 1 <= f.keep <= f.groups:
                     raise ValueError(f"layer {i}: {f.experts} experts in {f.groups} groups, {f.keep} kept, {f.top} chosen are not supported "
                                      "(at most 256 experts in equal groups, 32 chosen)")
@@ -214,8 +303,12 @@ class HybridConfig:
                     raise ValueError(f"layer {i}: {m.rot_dims} rotated dimensions of {m.dim}")
             if not isinstance(m, LatentSpec):
                 continue
-            if m.rank > 1024:
-                raise ValueError(f"layer {i}: latent size {m.rank} is not supported (at most 1024)")
+            if m.key_width > 1024:
+                raise ValueError(f"layer {i}: latent size {m.rank} with {m.rot_dim} rotated dimensions is not supported (at most 1024 together)")
+            if m.rot_dim % 2:
+                raise ValueError(f"layer {i}: {m.rot_dim} rotated dimensions")
+            if m.rot_dim and m.kv_from is not None:
+                raise ValueError(f"layer {i}: rotated dimensions need latents of the layer's own")
             if m.kv_from is not None:
                 if not 0 <= m.kv_from < i:
                     raise ValueError(f"layer {i}: kv_from {m.kv_from} does not name an earlier layer")
@@ -239,17 +332,21 @@ class HybridConfig:
             elif isinstance(m, DiffSpec):
                 n += self.hidden * (m.conv_width + m.heads * m.vdim)
             else:
-                n += self.hidden * m.heads * (m.dim + m.vdim) + m.rank * m.heads * (m.dim + m.vdim)
-                n += self.hidden * m.rank if m.kv_from is None else 0
+                n += self.hidden * m.heads * (m.dim + m.rot_dim + m.vdim + m.gated) + m.rank * m.heads * (m.dim + m.vdim)
+                n += self.hidden * (m.rank + m.rot_dim) if m.kv_from is None else 0
             if isinstance(layer.mlp, MoeSpec):
-                n += self.hidden * layer.mlp.experts * (2 * layer.mlp.inter + 1)
+                f = layer.mlp
+                n += self.hidden * (f.experts * (2 + f.gated) * f.inter + 3 * f.shared_inter + f.logits)
             elif layer.mlp:
-                n += 3 * self.hidden * layer.mlp.inter
+                n += (2 + Act(layer.mlp.act).gated) * self.hidden * layer.mlp.inter
+        if self.loop is not None:
+            n += 2 * self.hidden * self.hidden
         return 2 * n
 
     def kv_bytes_per_token(self, kv_dtype_bytes: int = 2) -> int:
-        return kv_dtype_bytes * (sum(pad8(m.rank) for m in self.latent_layers if m.kv_from is None) +
-                                 sum(m.page_elems // ops.PAGE for m in self.attention_layers if isinstance(m, DiffSpec)))
+        mixers = [self.layers[li].mixer for li in self.runs]
+        return kv_dtype_bytes * (sum(m.key_width for m in mixers if isinstance(m, LatentSpec) and m.kv_from is None) +
+                                 sum(m.page_elems // ops.PAGE for m in mixers if isinstance(m, DiffSpec)))
 
 
 # ------------------------------------------------------------------------------------------
@@ -266,12 +363,13 @@ class RecurrentWeights:
 
 @dataclass
 class LatentWeights:
-    qc: torch.Tensor              # [heads * dim_p (+ rank_p), hidden]: query (and latent) projections
+    qc: torch.Tensor              # [LatentSpec.proj_width, hidden]: query (latent and rotated key, head gate) projections
     c_norm: torch.Tensor | None   # fp32 [rank]
     uk: torch.Tensor              # [heads * rank_p, dim_p]: W_uk^T per head, folds the key expansion into the query
     uv: torch.Tensor              # [heads * vdim_p, rank_p]: value expansion, applied to the attended latent
     o: torch.Tensor               # [hidden, heads * vdim_p]
-    kv: torch.Tensor | None = None   # [heads * (key | value) * dim, rank_p]: both expansions, for prompts (see expand_prompts)
+    kv: torch.Tensor | None = None     # [heads * (key | value chunks) * 64, key_width]: both expansions, for prompts (see expand_prompts)
+    freq: torch.Tensor | None = None   # fp64 [rot_dim / 2]
 
 
 @dataclass
@@ -297,17 +395,22 @@ class DiffWeights:
 
 @dataclass
 class MoeWeights:
-    router: torch.Tensor     # [experts, hidden]
-    up: torch.Tensor         # [experts, inter_p, hidden_p]
+    router: torch.Tensor     # [experts (+ the shared expert's gate), hidden]
+    up: torch.Tensor         # [experts, inter_p, hidden_p]; gated: [experts, 2 inter_p, hidden_p], gate and up rows packed with ``half``
     down: torch.Tensor       # [experts, hidden, inter_p]
+    half: int = 0
+    bias: torch.Tensor | None = None             # fp32 [experts]
+    shared_up: torch.Tensor | None = None        # [2 inter_p, hidden_p], packed with ``shared_half``
+    shared_down: torch.Tensor | None = None
+    shared_half: int = 0
 
 
 @dataclass
 class HybridLayer:
     """Norms and residual connections follow ``HybridConfig.residual``: Dynamic-Tanh, hyper-connections and a token shift, or RMS
-    norms before (norm1, norm2) and behind (hc1, hc2) the sublayers."""
+    norms before (norm1, norm2) and, for "sandwich", behind (hc1, hc2) the sublayers."""
     norm1: DynamicTanh | RmsNorm
-    hc1: HyperConnection | RmsNorm
+    hc1: HyperConnection | RmsNorm | None
     mixer: RecurrentWeights | LatentWeights | DeltaWeights | DiffWeights
     shift: torch.Tensor | None = None             # fp32 [hidden]
     norm2: DynamicTanh | RmsNorm | None = None
@@ -316,6 +419,9 @@ class HybridLayer:
     down: torch.Tensor | None = None
     half: int = 0
     moe: MoeWeights | None = None
+    act: Act | None = None                        # feed-forward; a gated one has gate_up packed with ``half``, another up rows alone
+    conv1: torch.Tensor | None = None             # fp32 [input_taps, hidden]: what the sublayer reads, the identity included
+    conv2: torch.Tensor | None = None
 
 
 @dataclass
@@ -324,6 +430,9 @@ class HybridWeights:
     layers: list = field(default_factory=list)
     final_norm: DynamicTanh | None = None
     lm_head: torch.Tensor | None = None
+    embed_norm: RmsNorm | None = None
+    loop_in: torch.Tensor | None = None          # [hidden, 2 * hidden_p]: residual, embedding
+    loop_step: torch.Tensor | None = None        # fp32 [times, hidden]
     unused: list = field(default_factory=list)   # tensors of the checkpoint that its configuration does not name
 
 
@@ -344,25 +453,53 @@ def pack_recurrent(spec: RecurrentSpec, q, f, f_bias, low, v, norm, o) -> Recurr
                             norm=norm.float().contiguous(), o=pad_cols(o))
 
 
+def chunks(n: int) -> int:
+    """64-column chunks that hold n columns."""
+    return -(-n // 64)
+
+
 def expand_prompts(spec: LatentSpec, dtype) -> bool:
-    """Whether prompts of a layer may run on expanded keys and values: the heads fit the paged prefill kernel, and a latent is
+    """Whether prompts of a layer may run on expanded keys and values: the heads fit the paged prefill kernel, and a page row is
     wider than a head (otherwise attending to the latent itself is no more work)."""
-    return dtype == torch.bfloat16 and spec.dim == spec.vdim and spec.dim in (64, 128) and spec.rank > spec.dim
+    return (dtype == torch.bfloat16 and chunks(spec.q_width) <= 3 and chunks(spec.vdim) <= min(2, chunks(spec.q_width)) and spec.scale > 0
+            and spec.key_width > spec.q_width)
 
 
-def pack_latent(spec: LatentSpec, q, dkv, dkv_norm, uk, uv, o) -> LatentWeights:
-    h, dp, rp, vp = spec.heads, pad8(spec.dim), pad8(spec.rank), pad8(spec.vdim)
-    qc = pad_head_rows(q, h, dp)
+def rotation(dims: int, base: float, device) -> torch.Tensor:
+    """Angles per position of the pairs of ``dims`` rotated dimensions, fp64."""
+    return (base ** (-2 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1))).to(device)
+
+
+def pack_latent(spec: LatentSpec, q, dkv, dkv_norm, uk, uv, o, g=None) -> LatentWeights:
+    """q: heads of dim (+ rot_dim) rows; dkv: the latent's rows (and the rotated key part's); g: head gates."""
+    h, d, r, rank = spec.heads, spec.dim, spec.rot_dim, spec.rank
+    dp, rp, vp, cp, kw = pad8(d), pad8(r), pad8(spec.vdim), pad8(rank), spec.key_width
+    pad = torch.nn.functional.pad
+
+    def two_parts(w, first, second):
+        """[n, first + second, k] -> both parts padded to multiples of 8 rows, [n * .., k]."""
+        n, k = w.shape[0], w.shape[-1]
+        return torch.cat([pad(w[:, :first], (0, 0, 0, pad8(first) - first)), pad(w[:, first:], (0, 0, 0, pad8(second) - second))], 1).reshape(-1, k)
+
+    qc = [two_parts(q.reshape(h, d + r, -1), d, r)]
     if dkv is not None:
-        qc = torch.cat([qc, pad_head_rows(dkv, 1, rp)], 0)
-    ukt = uk.reshape(h, spec.dim, spec.rank).transpose(1, 2)                                   # [h, rank, dim]
-    ukt = torch.nn.functional.pad(ukt, (0, dp - spec.dim, 0, rp - spec.rank)).reshape(h * rp, dp)
+        qc.append(two_parts(dkv[None], rank, r))
+    if g is not None:
+        qc.append(g)
+    ukh, uvh = uk.reshape(h, d, rank), uv.reshape(h, spec.vdim, rank)
+    ukt = pad(ukh.transpose(1, 2), (0, dp - d, 0, cp - rank)).reshape(h * cp, dp)             # [h, rank, dim]
     kv = None
     if expand_prompts(spec, q.dtype):
-        kv = pad_cols(torch.stack([uk.reshape(h, spec.dim, spec.rank), uv.reshape(h, spec.vdim, spec.rank)], 1).reshape(2 * h * spec.dim, spec.rank), rp)
-    return LatentWeights(kv=kv, qc=pad_cols(qc), c_norm=None if dkv_norm is None else dkv_norm.float().contiguous(), uk=ukt.contiguous(),
-                         uv=pad_cols(pad_head_rows(uv, h, vp), rp),
-                         o=torch.nn.functional.pad(o.reshape(o.shape[0], h, spec.vdim), (0, vp - spec.vdim)).reshape(o.shape[0], h * vp).contiguous())
+        # a head's expanded key is [W_uk c | rotated part]: the part passes through rows of the identity
+        kv = q.new_zeros(h, 64 * (chunks(spec.q_width) + chunks(spec.vdim)), kw)
+        kv[:, :d, :rank] = ukh
+        kv[:, dp:dp + r, cp:cp + r] = torch.eye(r, dtype=q.dtype, device=q.device)
+        v0 = 64 * chunks(spec.q_width)
+        kv[:, v0:v0 + spec.vdim, :rank] = uvh
+        kv = kv.reshape(-1, kw)
+    return LatentWeights(kv=kv, qc=pad_cols(torch.cat(qc, 0)), c_norm=None if dkv_norm is None else dkv_norm.float().contiguous(), uk=ukt.contiguous(),
+                         uv=pad_cols(pad_head_rows(uv, h, vp), cp), freq=rotation(r, spec.rot_base, q.device) if r else None,
+                         o=pad(o.reshape(o.shape[0], h, spec.vdim), (0, vp - spec.vdim)).reshape(o.shape[0], h * vp).contiguous())
 
 
 def pack_delta(spec: DeltaSpec, q, k, v, g, a, b, conv, a_log, dt_bias, norm, o) -> DeltaWeights:
@@ -376,9 +513,7 @@ def pack_diff(spec: DiffSpec, q, k, v, bias, conv, lam: float, o) -> DiffWeights
     """``bias``, ``conv``: of the q, k and v channels; ``lam``: the layer's weight of the second map."""
     vp = pad8(spec.vdim)
     f32 = lambda t: t.float().contiguous()
-    i = torch.arange(spec.rot_dims // 2, dtype=torch.float64)
-    freq = spec.rot_base ** (-2 * i / max(spec.rot_dims, 1))
-    return DiffWeights(qkv=pad_cols(torch.cat([q, k, v], 0)), bias=f32(torch.cat(bias, 0)), conv=f32(torch.cat(conv, 0).t()), freq=freq.to(q.device),
+    return DiffWeights(qkv=pad_cols(torch.cat([q, k, v], 0)), bias=f32(torch.cat(bias, 0)), conv=f32(torch.cat(conv, 0).t()), freq=rotation(spec.rot_dims, spec.rot_base, q.device),
                        lam=float(lam), o=torch.nn.functional.pad(o.reshape(o.shape[0], spec.heads, spec.vdim), (0, vp - spec.vdim)).reshape(o.shape[0], -1).contiguous())
 
 
@@ -389,12 +524,53 @@ def pack_moe(router, ups, downs) -> MoeWeights:
     return MoeWeights(router=pad_cols(router), up=up, down=pad_cols(torch.stack(list(downs))))
 
 
-def pack_mlp(layer: HybridLayer, gate, up, down) -> None:
+def pack_gated(gate, up, down):
+    """(gate and up rows packed for the gated epilogue, down, half-width)."""
     if gate.shape[0] % 32:
         gate, up, down = pad_mlp(gate, up, down)
-    layer.half = pick_swiglu_half(gate.shape[0])
-    layer.gate_up = pad_cols(ops.pack_gate_up(gate.contiguous(), up.contiguous(), layer.half))
-    layer.down = down.contiguous()
+    half = pick_swiglu_half(gate.shape[0])
+    return pad_cols(ops.pack_gate_up(gate.contiguous(), up.contiguous(), half)), down.contiguous(), half
+
+
+def pack_gated_moe(router, bias, gates, ups, downs, shared=None) -> MoeWeights:
+    """Gated experts: ``gates``, ``ups`` [inter, hidden] and ``downs`` [hidden, inter] of every one; ``shared``: (gate, up, down, sigmoid gate
+    [1, hidden]) of the expert that runs for every token."""
+    packed = [pack_gated(*w) for w in zip(gates, ups, downs)]
+    w = MoeWeights(router=pad_cols(router if shared is None else torch.cat([router, shared[3]], 0)), up=torch.stack([p[0] for p in packed]),
+                   down=torch.stack([p[1] for p in packed]), half=packed[0][2], bias=bias.float().contiguous() if bias is not None else None)
+    if shared is not None:
+        w.shared_up, w.shared_down, w.shared_half = pack_gated(*shared[:3])
+    return w
+
+
+def pack_mlp(layer: HybridLayer, gate, up, down, act="gelu_tanh") -> None:
+    layer.gate_up, layer.down, layer.half = pack_gated(gate, up, down)
+    layer.act = hops.as_act(act)
+
+
+def pack_plain_mlp(layer: HybridLayer, up, down, act: Act) -> None:
+    """A feed-forward without a gate."""
+    layer.gate_up = torch.nn.functional.pad(pad_cols(up), (0, 0, 0, pad8(up.shape[0]) - up.shape[0])).contiguous()
+    layer.down, layer.act = pad_cols(down), act
+
+
+def pack_input_conv(w) -> torch.Tensor:
+    """[hidden, taps] of a sublayer that reads h + conv(h): one filter, last tap first met by the token itself."""
+    f = w.float().t().clone()
+    f[-1] += 1
+    return f.contiguous()
+
+
+def xielu(p: float, q: float) -> Act:
+    """xIELU with its two numbers as they are stored."""
+    soft = lambda v: float(torch.nn.functional.softplus(torch.tensor(v, dtype=torch.float64)))
+    return Act("xielu", soft(p), 0.5 + soft(q))
+
+
+def pack_loop_in(w) -> torch.Tensor:
+    """[hidden, residual | embedding], each half padded to multiples of 8 columns."""
+    n = w.shape[1] // 2
+    return torch.cat([pad_cols(w[:, :n]), pad_cols(w[:, n:])], 1).contiguous()
 
 
 def random_weights(cfg: HybridConfig, device, seed: int = 0, std: float = 0.02, dtype=torch.bfloat16) -> HybridWeights:
@@ -408,9 +584,15 @@ def random_weights(cfg: HybridConfig, device, seed: int = 0, std: float = 0.02, 
         norm = lambda: DynamicTanh(0.5 + rand(1), 1 + 0.1 * (rand(hid) - 0.5), 0.1 * (rand(hid) - 0.5))
         conn = lambda: HyperConnection(rand(st) / st + 0.5 / st, 0.5 + rand(st), torch.eye(st, device=dev) * 0.8 + 0.2 * rand(st, st) / st)
     else:
-        norm = conn = lambda: RmsNorm(1 + 0.1 * (rand(hid) - 0.5), cfg.norm_eps)
+        norm = lambda: RmsNorm(1 + 0.1 * (rand(hid) - 0.5), cfg.norm_eps)
+        conn = norm if cfg.residual == "sandwich" else lambda: None
     taps = lambda m, *rows: [torch.randn(n, m.taps, generator=gen, device=dev) * 0.5 / m.taps for n in rows]
+    input_conv = lambda: pack_input_conv(torch.randn(hid, cfg.input_taps, generator=gen, device=dev) * 0.5 / cfg.input_taps) if cfg.input_taps else None
     w = HybridWeights(embed=draw(cfg.vocab, hid))
+    if cfg.residual == "pre":
+        w.embed_norm = norm()
+    if cfg.loop is not None:
+        w.loop_in, w.loop_step = pack_loop_in(draw(hid, 2 * hid)), torch.randn(cfg.loop.times, hid, generator=gen, device=dev) * std
     for spec in cfg.layers:
         m = spec.mixer
         if isinstance(m, RecurrentSpec):
@@ -425,16 +607,24 @@ def random_weights(cfg: HybridConfig, device, seed: int = 0, std: float = 0.02, 
             mixer = pack_diff(m, *(draw(n, hid) for n in rows), [draw(n) for n in rows], taps(m, *rows), m.diff, draw(hid, m.heads * m.vdim))
         else:
             own = m.kv_from is None
-            mixer = pack_latent(m, draw(m.heads * m.dim, hid), draw(m.rank, hid) if own else None, torch.ones(m.rank, device=dev) if own else None,
-                                draw(m.heads * m.dim, m.rank), draw(m.heads * m.vdim, m.rank), draw(hid, m.heads * m.vdim))
-        layer = HybridLayer(norm1=norm(), shift=rand(hid) if cfg.residual == "hyper" else None, hc1=conn(), mixer=mixer)
+            mixer = pack_latent(m, draw(m.heads * (m.dim + m.rot_dim), hid), draw(m.rank + m.rot_dim, hid) if own else None,
+                                torch.ones(m.rank, device=dev) if own else None, draw(m.heads * m.dim, m.rank), draw(m.heads * m.vdim, m.rank),
+                                draw(hid, m.heads * m.vdim), draw(m.heads, hid) if m.gated else None)
+        layer = HybridLayer(norm1=norm(), shift=rand(hid) if cfg.residual == "hyper" else None, hc1=conn(), mixer=mixer, conv1=input_conv())
         if spec.mlp is not None:
-            layer.norm2, layer.hc2 = norm(), conn()
-        if isinstance(spec.mlp, MoeSpec):
-            f = spec.mlp
+            layer.norm2, layer.hc2, layer.conv2 = norm(), conn(), input_conv()
+        f = spec.mlp
+        if isinstance(f, MoeSpec) and f.gated:
+            expert = lambda n: (draw(n, hid), draw(n, hid), draw(hid, n))
+            layer.moe = pack_gated_moe(draw(f.experts, hid), torch.randn(f.experts, generator=gen, device=dev) * std if f.bias else None,
+                                       *zip(*(expert(f.inter) for _ in range(f.experts))),
+                                       shared=(*expert(f.shared_inter), draw(1, hid)) if f.shared_inter else None)
+        elif isinstance(f, MoeSpec):
             layer.moe = pack_moe(draw(f.experts, hid), [draw(f.inter, hid) for _ in range(f.experts)], [draw(hid, f.inter) for _ in range(f.experts)])
-        elif spec.mlp is not None:
-            pack_mlp(layer, draw(spec.mlp.inter, hid), draw(spec.mlp.inter, hid), draw(hid, spec.mlp.inter))
+        elif f is not None and f.act == "xielu":
+            pack_plain_mlp(layer, draw(f.inter, hid), draw(hid, f.inter), xielu(0.3, -0.2))
+        elif f is not None:
+            pack_mlp(layer, draw(f.inter, hid), draw(f.inter, hid), draw(hid, f.inter), f.act)
         w.layers.append(layer)
     w.final_norm, w.lm_head = norm(), pad_cols(draw(cfg.vocab, hid))
     return w
@@ -463,7 +653,7 @@ class HybridModel:
         z = lambda *s, dtype=dt: torch.zeros(*s, dtype=dtype, device=dev)
         hid = cfg.hidden
         # residual streams, double buffered where a row reads its neighbour
-        self.xs = [z(max_tokens, cfg.streams, hid, dtype=torch.float32) for _ in range(2 if cfg.residual == "hyper" else 1)]
+        self.xs = [z(max_tokens, cfg.streams, hid, dtype=torch.float32) for _ in range(1 if cfg.residual == "sandwich" else 2)]
         self.h, self.y = z(max_tokens, pad8(hid)), z(max_tokens, pad8(hid))
         of = lambda kind: [l.mixer for l in cfg.layers if isinstance(l.mixer, kind)]
         rec, lat, delta, diff = of(RecurrentSpec), of(LatentSpec), of(DeltaSpec), of(DiffSpec)
@@ -472,24 +662,29 @@ class HybridModel:
         flat = lambda width, dtype=dt: z(max_tokens * width, dtype=dtype) if width else None    # viewed per layer: rows stay contiguous
         self.qfv = flat(most(pad8(m.heads * (2 * m.dim + m.vdim)) for m in rec), torch.float32)
         self.rec_o = flat(most(m.heads * m.vdim for m in rec + delta), torch.float32)
-        self.qc = flat(most(m.heads * pad8(m.dim) + pad8(m.rank) for m in lat))
-        self.qa = flat(most(m.heads * pad8(m.rank) for m in lat))
+        self.loop_in = self.loop_x = None
+        if cfg.loop is not None:       # residual | embedding, and the residual a pass begins with
+            self.loop_in, self.loop_x = z(max_tokens, 2 * pad8(hid)), z(max_tokens, pad8(hid), dtype=torch.float32)
+        self.qc = flat(most(pad8(m.proj_width) for m in lat))
+        self.qa = flat(most(m.heads * m.key_width for m in lat))
         self.oc = flat(most(m.heads * pad8(m.rank) for m in lat))
         self.proj = flat(most([pad8(m.conv_width + m.heads * m.vdim) for m in delta] + [pad8(m.conv_width) for m in diff]))
-        self.ab = flat(most([pad8(2 * m.heads) for m in delta] + [pad8(f.experts) for f in experts]), torch.float32)
+        self.ab = flat(most([pad8(2 * m.heads) for m in delta] + [pad8(f.logits) for f in experts]), torch.float32)
         self.unit_qk = flat(most(2 * m.kv_heads * m.dim for m in delta), torch.float32)
         self.unit_v = flat(most(m.heads * m.vdim for m in delta))
         self.gates = flat(most(2 * m.heads for m in delta), torch.float32)
         self.diff_q = flat(most(2 * m.heads * pad8(m.dim) for m in diff))
         self.attn = flat(most([pad8(m.heads * m.vdim) for m in rec + delta] + [m.heads * pad8(m.vdim) for m in lat + diff]))
-        inter = most(l.down.shape[1] for l in weights.layers if l.down is not None)
+        inter = most([l.down.shape[1] for l in weights.layers if l.down is not None] +
+                     [l.moe.shared_down.shape[1] for l in weights.layers if l.moe is not None and l.moe.shared_down is not None])
         self.act = flat(inter)
         self.gate_up = flat(2 * inter) if dt == torch.float32 and dev.type == "cuda" else None
         self.moe_ws = None
         if experts:
             if dev.type == "cuda":
                 self.moe_ws = moe_ops.MoEWorkspace(max_tokens, most(f.top for f in experts), most(f.experts for f in experts), pad8(hid),
-                                                   most(pad8(f.inter) for f in experts), dev, dt)
+                                                   most(l.moe.down.shape[2] for l in weights.layers if l.moe is not None), dev, dt,
+                                                   gated_f32=dt == torch.float32 and any(f.gated for f in experts))
             else:
                 self.moe_ws = moe_ops.MoEWorkspace(1, 1, 1, pad8(hid), 8, dev, dt)
         self.h_last_buf = z(max_seqs, pad8(hid))
@@ -499,7 +694,7 @@ class HybridModel:
         per_cta = 32 if dt == torch.bfloat16 else 4                     # latent heads a decode CTA takes
         diff_ctas = [m.kv_heads * -(-(m.heads // m.kv_heads) // 8) for m in diff]
         self.hkv = most([-(-m.heads // per_cta) for m in lat] + diff_ctas) or 1      # CTAs per decode row ...
-        per_sm = 8 if dt == torch.float32 else (2 if most(m.rank for m in lat) <= 128 else 1)
+        per_sm = 8 if dt == torch.float32 else (2 if most(m.key_width for m in lat) <= 128 else 1)
         self.decode_ctas = per_sm * (ops.num_sms() if dev.type == "cuda" else 148)       # ... and the device's places for them
         self.decode_splits, self._split_capacity = 1, 1
         # fp32 partial results of a decode row and split: 16 rows per CTA, and (maximum, sum) of each
@@ -588,32 +783,54 @@ class HybridModel:
         hops.linear(attn, w.o, y)
 
     def _experts(self, f: MoeSpec, w: MoeWeights, h):
-        logits = self._rows(self.ab, h.shape[0], pad8(f.experts))
-        hops.linear(h, w.router, logits[:, : f.experts], f32_out=True)
-        return moe_ops.relu2_experts(h, logits[:, : f.experts], w.up, w.down, self.moe_ws, f.top, f.groups, f.keep, f.renormalize)
+        t = h.shape[0]
+        logits = self._rows(self.ab, t, pad8(f.logits))
+        hops.linear(h, w.router, logits[:, : f.logits], f32_out=True)
+        out = moe_ops.routed_experts(h, logits[:, : f.experts], w.up, w.down, self.moe_ws, f.top, Act(f.act, f.limit), w.half, f.groups, f.keep,
+                                     f.renormalize, w.bias)
+        if w.shared_up is not None:
+            y = self.y[:t]
+            self._mlp(h, w.shared_up, w.shared_down, Act(f.act, f.shared_limit), w.shared_half, y[:, : self.cfg.hidden])
+            out = ExpertRows(out.rows, out.pos, out.weight, y, logits[:, f.experts])
+        return out
+
+    def _mlp(self, h, up, down, act: Act, half, y):
+        """y = down(act(up h)); ``up`` packed with ``half`` for a gated activation."""
+        t = h.shape[0]
+        mid = self._rows(self.act, t, down.shape[1])
+        if act.gated:
+            hops.gated_linear(h, up, half, act, mid, self._rows(self.gate_up, t, up.shape[0]) if self.gate_up is not None else None)
+        else:
+            hops.act_linear(h, up, act, mid)
+        hops.linear(mid, down, y)
 
     def _latent(self, li, m: LatentSpec, w: LatentWeights, h, y, kv, si):
         t, hp = h.shape[0], m.heads
-        dp, rp, vp = pad8(m.dim), pad8(m.rank), pad8(m.vdim)
+        dp, cp, vp, kw = pad8(m.dim), pad8(m.rank), pad8(m.vdim), m.key_width
         own = m.kv_from is None
         pool = kv.pools[li if own else m.kv_from]
-        qc = self._rows(self.qc, t, hp * dp + (rp if own else 0))
-        hops.linear(h, w.qc, qc)
-        if own:
-            hops.latent_append(qc[:, hp * dp:], w.c_norm, self.cfg.norm_eps, si.slots, pool, m.rank)
+        qc = self._rows(self.qc, t, pad8(m.proj_width))
+        hops.linear(h, w.qc, qc[:, : m.proj_width])
         attn = self._rows(self.attn, t, hp * vp)
         pages = self._expanded_pages(m, w, si)
         rows = si.num_decode if pages else t      # rows that attend to the latents themselves
+        qa, oc = self._rows(self.qa, rows, hp * kw), self._rows(self.oc, rows, hp * cp)
+        if own:
+            rope = None
+            if m.rot_dim:
+                rope = LatentRope(w.freq, si.positions, hp, m.dim, qa.view(rows * hp, kw) if rows else None, cp, rows)
+            hops.latent_append(qc, m.latent_col, w.c_norm, self.cfg.norm_eps, si.slots, pool, m.rank, rope)
+        gate = qc[:, m.gate_col:m.gate_col + hp] if m.gated else None
         if rows:
-            qa, oc = self._rows(self.qa, rows, hp * rp), self._rows(self.oc, rows, hp * rp)
-            hops.linear_batched(qc[:rows], w.uk, qa, hp, dp, rp)
-            hops.latent_attention(qa.view(rows * hp, rp), oc.view(rows * hp, rp), pool, si, hp, rp, m.scale, m.window, self.decode_splits,
-                                  self.part_o, self.part_ml, self.counters, decode_only=bool(pages))
-            hops.linear_batched(oc, w.uv, attn[:rows], hp, rp, vp)
+            hops.linear_batched(qc[:rows], w.uk, qa, hp, m.q_width, kw)
+            hops.latent_attention(qa.view(rows * hp, kw), oc.view(rows * hp, cp), pool, si, hp, kw, m.scale, m.window, self.decode_splits,
+                                  self.part_o, self.part_ml, self.counters, decode_only=bool(pages), vrank=cp, gate=gate)
+            hops.linear_batched(oc, w.uv, attn[:rows], hp, cp, vp)
         if pages:
-            hops.latent_prefill_expanded(qc, attn, pool, w.kv, si, hp, m.dim, m.scale, m.window, pages,
-                                         self._scratch("dense", (pages * ops.PAGE, rp)), self._scratch("kv", (pages, hp, 2, ops.PAGE, m.dim)),
-                                         self._scratch("table", (si.num_prefill_seqs, si.page_table.shape[1]), torch.int32))
+            kc, vc = chunks(m.q_width), chunks(m.vdim)
+            hops.latent_prefill_expanded(qc, attn, pool, w.kv, si, hp, kc, vc, m.q_width, vp, m.scale, m.window, pages,
+                                         self._scratch("dense", (pages * ops.PAGE, kw)), self._scratch("kv", (pages, hp, kc + vc, ops.PAGE, 64)),
+                                         self._scratch("table", (si.num_prefill_seqs, si.page_table.shape[1]), torch.int32), gate)
         hops.linear(attn, w.o, y)
 
     EXPAND_BYTES = 1 << 30             # most memory the expanded keys and values of a step may take
@@ -628,9 +845,10 @@ class HybridModel:
         seen = start + (n + 1) // 2
         pairs = int((n * (seen.clip(max=m.window) if m.window > 0 else seen)).sum())
         # operations per head: the latent kernel computes scores once per 128 output columns of a wide latent
-        direct = pairs * 2 * m.rank * (1 + max(1, -(-m.rank // 128)))
-        expanded = pairs * 4 * m.dim + pages * ops.PAGE * 4 * m.dim * m.rank
-        return pages if direct > expanded and pages * ops.PAGE * m.heads * m.dim * 4 <= self.EXPAND_BYTES else 0
+        head = 64 * (chunks(m.q_width) + chunks(m.vdim))
+        direct = pairs * 2 * (m.key_width * max(1, -(-m.rank // 128)) + m.rank)
+        expanded = pairs * 2 * head + pages * ops.PAGE * 2 * head * m.key_width
+        return pages if direct > expanded and pages * ops.PAGE * m.heads * head * 2 <= self.EXPAND_BYTES else 0
 
     def _scratch(self, name, shape, dtype=None):
         """Step scratch that grows to the largest step seen (prompt steps only: never inside a captured graph)."""
@@ -647,12 +865,21 @@ class HybridModel:
         cfg, w, t = self.cfg, self.w, si.num_tokens
         cur, nxt = self.xs[0][:t], self.xs[-1][:t]
         h, y = self.h[:t], self.y[:t]
-        hops.embed_streams(si.token_ids, w.embed, cur)
+        wp = pad8(cfg.hidden)
+        hops.embed_streams(si.token_ids, w.embed, cur, w.embed_norm, self.loop_in[:t, wp:wp + cfg.hidden] if cfg.loop is not None else None)
         written, out = None, None      # connection whose sublayer output the residual still has to take in, and that output
+        entered, add = None, None      # residual that a pass begins with instead of ``cur``, and what is still to be added to it
 
-        def step(conn, norm, h, gather=None, **kw):
-            nonlocal cur, nxt
-            if cfg.residual == "sandwich":
+        def step(conn, norm, h, gather=None, conv=None, state=None, **kw):
+            nonlocal cur, nxt, entered, add
+            if conv is not None:
+                fold = entered is not None or out is not None
+                hops.norm_conv_step(entered if entered is not None else cur[:, 0], nxt[:, 0] if fold else None, out, add, norm, conv, state, h, si)
+                entered = add = None
+                if fold:
+                    cur, nxt = nxt, cur
+                return
+            if cfg.residual != "hyper":
                 hops.norm_step(cur[:, 0], out, written, norm, h, gather)
                 return
             fold = written is not None and gather is None
@@ -660,32 +887,42 @@ class HybridModel:
             if fold:
                 cur, nxt = nxt, cur
 
-        for li, (spec, lw) in enumerate(zip(cfg.layers, w.layers)):
-            m = spec.mixer
-            step(lw.hc1, lw.norm1, h, **({"shift": lw.shift, "prev": self.state.layers[li]["shift"]} if lw.shift is not None else {}))
-            if self.capture is not None and li > 0:
+        lp, passes = cfg.loop, 0
+        for ri, li in enumerate(cfg.runs):
+            spec, lw, m = cfg.layers[li], w.layers[li], cfg.layers[li].mixer
+            state = self.state.layers[ri]
+            begins = lp is not None and li == lp.start
+            if begins:
+                step(None, None, self.loop_in[:t, : cfg.hidden])
+                if self.capture is not None and ri > 0:
+                    self.capture.append(cur.sum(1))
+                hops.linear(self.loop_in[:t], w.loop_in, self.loop_x[:t, : cfg.hidden], f32_out=True)
+                entered, add, written, out = self.loop_x[:t, : cfg.hidden], w.loop_step[passes], None, None
+                passes += 1
+                if lw.conv1 is None:   # the passes that follow work on the stream itself
+                    torch.add(entered, add, out=cur[:, 0])
+                    entered = add = None
+            step(lw.hc1, lw.norm1, h, conv=lw.conv1, state=state.get("input1"),
+                 **({"shift": lw.shift, "prev": state["shift"]} if lw.shift is not None else {}))
+            if self.capture is not None and ri > 0 and not begins:
                 self.capture.append(cur.sum(1))
             if isinstance(m, RecurrentSpec):
-                self._recurrent(li, m, lw.mixer, h, y[:, : cfg.hidden], si)
+                self._recurrent(ri, m, lw.mixer, h, y[:, : cfg.hidden], si)
             elif isinstance(m, DeltaSpec):
-                self._delta(li, m, lw.mixer, h, y[:, : cfg.hidden], si)
+                self._delta(ri, m, lw.mixer, h, y[:, : cfg.hidden], si)
             elif isinstance(m, DiffSpec):
-                self._diff(li, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
+                self._diff(ri, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
             else:
-                self._latent(li, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
+                self._latent(ri, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
             written, out = lw.hc1, y
             if spec.mlp is None:
                 continue
-            step(lw.hc2, lw.norm2, h)
-            written = lw.hc2
+            step(lw.hc2, lw.norm2, h, conv=lw.conv2, state=state.get("input2"))
+            written, out = lw.hc2, y
             if isinstance(spec.mlp, MoeSpec):
                 out = self._experts(spec.mlp, lw.moe, h)
-                continue
-            act = self._rows(self.act, t, lw.down.shape[1])
-            hops.gated_linear(h, lw.gate_up, lw.half, spec.mlp.act, act,
-                              self._rows(self.gate_up, t, lw.gate_up.shape[0]) if self.gate_up is not None else None)
-            hops.linear(act, lw.down, y[:, : cfg.hidden])
-            out = y
+            else:
+                self._mlp(h, lw.gate_up, lw.down, lw.act, lw.half, y[:, : cfg.hidden])
         if self.capture is not None:
             step(None, None, None)
             self.capture.append(cur.sum(1))

@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from . import decoder, dezudra, hybrid, rilelorn
+from . import decoder, dezudra, fizesun, hybrid, rilelorn
 from .config import DecoderConfig
 
 
@@ -37,7 +37,8 @@ FAMILIES = (
            ("bf16", "f32")),
 )
 ARCHITECTURES = {a.name: a for a in (Architecture("Rilelorn", rilelorn.read_config, rilelorn.load_weights, "hybrid"),
-                                     Architecture("Dezudra", dezudra.read_config, dezudra.load_weights, "delta"))}
+                                     Architecture("Dezudra", dezudra.read_config, dezudra.load_weights, "delta"),
+                                     Architecture("Fizesun", fizesun.read_config, fizesun.load_weights, "latent_moe"))}
 
 
 def family_of(cfg) -> Family:

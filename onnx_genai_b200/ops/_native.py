@@ -40,7 +40,6 @@ _SIGNATURES = {
     "ogb_rope_kv_append_q8": ([P, P, P, P, P, P, I, I, I, I, I, I, I, I, L, I, P, P], I),
     "ogb_paged_decode_q8": ([P, P, P, P, I, P, P, I, I, L, I, I, I, I, I, F, I, P, P, I, I, P, P], I),
     "ogb_paged_prefill_q8": ([P, P, P, P, I, P, P, P, P, P, I, I, I, L, I, I, I, I, I, F, I, I, P, P], I),
-    "ogb_gemm_bf16_gated": ([P, P, P, I, I, I, I, I, I, I, I, P, P], I),
     "ogb_gemm_bf16_batched": ([P, P, P, I, I, I, I, I, I, I, I, I, P, P], I),
     "ogb_gemm_f32": ([P, P, P, I, I, I, I, I, I, I, I, I, P], I),
     "ogb_argmax_f32": ([P, P, I, I, I, P], I),

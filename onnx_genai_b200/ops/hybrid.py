@@ -1,8 +1,9 @@
 """Ops of models that choose a mixer per layer (csrc/kernels/hybrid.cu, recurrent.cu, latent_attention.cu, short_conv.cu,
 delta_rule.cu, diff_attention.cu): hyper-connected residual streams with a Dynamic-Tanh norm and token shift, one residual stream
-with RMS norms on both sides of a sublayer, HGRN2 and gated delta-rule recurrences over per-sequence state, short causal
-convolutions, attention over paged latents, differential attention over paged keys and values, batched per-head products, and
-the fp32 matrix product of the 32-bit engine.
+with RMS norms before (and behind) a sublayer and convolutions of what a sublayer reads, HGRN2 and gated delta-rule recurrences
+over per-sequence state, short causal convolutions, attention over paged latents with or without a rotated part, differential
+attention over paged keys and values, products with activations, batched per-head products, and the fp32 matrix product of the
+32-bit engine.
 
 CUDA tensors run the kernels; CPU tensors run the statements in :mod:`onnx_genai_b200.ops.reference`, as the other ops do.
 ``si`` is the step's :class:`~onnx_genai_b200.models.decoder.StepInputs`.
@@ -18,25 +19,29 @@ from . import PAGE, gemm
 
 P, I, F, L = _native.P, _native.I, _native.F, _native.L
 _native.register("ogb_hyper_step", [P] * 13 + [I] * 6 + [P] * 5 + [I] * 4 + [P, P])
-_native.register("ogb_embed_streams", [P, P, P, I, I, I, I, I, P, P])
-_native.register("ogb_latent_append", [P, I, P, F, P, P, I, I, I, L, I, P, P])
-_native.register("ogb_latent_attention", [P] * 8 + [I] * 7 + [L, I, F, I, P, P, P, I, P, P])
+_native.register("ogb_embed_streams", [P, P, P, I, I, I, I, P, F, P, I, I, P, P])
+_native.register("ogb_latent_append", [P, I, I, P, F, P, P, I, I, I, L, P, P, P] + [I] * 7 + [P, P])
+_native.register("ogb_latent_attention", [P] * 9 + [I] * 10 + [L, I, F, I, P, P, P, I, P, P])
+_native.register("ogb_paged_prefill_chunks_bf16", [P] * 9 + [I] * 4 + [L] + [I] * 9 + [F, I, P, P])
+_native.register("ogb_gemm_bf16_act", [P] * 3 + [I] * 7 + [F, F, I, P, P])
+_native.register("ogb_gemm_f32_act", [P] * 3 + [I] * 7 + [F, F, P])
 _native.register("ogb_latent_gather", [P, P, P, P, I, I, L, I, I, I, P, P, P, P])
 _native.register("ogb_latent_set_tc", [I])
 _native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
 _native.register("ogb_hgrn2_state_rows", [I])
 _native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P, P, I, P, P])
 _native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, P, I, I, P])
-_native.register("ogb_norm_step", [P] * 8 + [F] + [I] * 6 + [L, I, P, P])
+_native.register("ogb_norm_step", [P] * 10 + [F] + [I] * 8 + [L, I, P, P])
+_native.register("ogb_norm_conv_step", [P] * 12 + [F] + [I] * 8 + [L] + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_conv_rope_append", [P, I, P, P, P, I, P, I, P, P, P, L, L] + [I] * 8 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_conv_unit_gates", [P, I, P, P, I, P, I] + [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_delta_rule", [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, I, P, P])
 _native.register("ogb_delta_block_floats", [I] * 4)
 _native.register("ogb_diff_attention", [P] * 8 + [I] * 3 + [L, L] + [I] * 10 + [F] * 4 + [I, P, P, P, I, P, P])
 _native.register("ogb_diff_set_tc", [I])
-_native.register("ogb_act_mul_packed", [P, P, I, I, I, I, I, P])
+_native.register("ogb_act_mul_packed", [P, P, I, I, I, I, F, F, I, P])
 
-ACTS = {"silu": 0, "gelu_tanh": 1}
+ACTS = {"none": 0, "silu": 1, "gelu_tanh": 2, "relu2": 3, "clamp_glu": 4, "xielu": 5}
 _ELEM = {torch.float32: 0, torch.bfloat16: 1}
 
 
@@ -66,10 +71,34 @@ class RmsNorm:
 
 @dataclass
 class ExpertRows:
-    """A sublayer's output that is still spread over expert rows: token t's is sum_j weight[t, j] rows[pos[t, j]]."""
+    """A sublayer's output that is still spread over expert rows: token t's is sum_j weight[t, j] rows[pos[t, j]], and a shared
+    expert's row times sigmoid(gate[t]) (a column of fp32 logits) where there is one."""
     rows: torch.Tensor
     pos: torch.Tensor
     weight: torch.Tensor
+    shared: torch.Tensor | None = None
+    gate: torch.Tensor | None = None
+
+
+@dataclass(frozen=True)
+class Act:
+    """Activation of a feed-forward and its numbers.  Gated: silu, gelu_tanh, clamp_glu (a: limit); of one value: relu2, xielu
+    (a, b: weights of its rising and its falling side)."""
+    kind: str
+    a: float = 0.0
+    b: float = 0.0
+
+    @property
+    def gated(self) -> bool:
+        return self.kind in ("silu", "gelu_tanh", "clamp_glu")
+
+    @property
+    def args(self):
+        return ACTS[self.kind], float(self.a), float(self.b)
+
+
+def as_act(act) -> Act:
+    return act if isinstance(act, Act) else Act(act)
 
 
 def state_rows(dim: int) -> int:
@@ -116,36 +145,70 @@ def linear_batched(a, w, out, batch, a_step, c_step):
 
 @_timed("gated_linear")
 def gated_linear(a, w_packed, half, act, out, scratch=None):
-    """out = act(a @ gate^T) * (a @ up^T) over a weight packed by ``ops.pack_gate_up``; bf16 in one product with the gate in its
-    epilogue, fp32 through ``scratch`` [rows, 2 * inter]."""
+    """out = act(a @ gate^T, a @ up^T) over a weight packed by ``ops.pack_gate_up``; ``act``: a gated :class:`Act` or its name.  bf16 in
+    one product with the gate in its epilogue, fp32 through ``scratch`` [rows, 2 * inter]."""
+    act = as_act(act)
     if not a.is_cuda:
         out.copy_(reference.act_mul_packed(reference.gemm(a, w_packed, out_dtype=torch.float32), half, act, out.dtype))
         return out
     m, n = a.shape[0], w_packed.shape[0]
     if a.dtype == torch.bfloat16:
-        rc = _native.load().ogb_gemm_bf16_gated(a.data_ptr(), w_packed.data_ptr(), out.data_ptr(), m, n, a.shape[1], a.stride(0),
-                                                w_packed.stride(0), out.stride(0), ACTS[act], 2 * half, status_word().data_ptr(), _stream())
-        _native.check(rc, "ogb_gemm_bf16_gated")
+        rc = _native.load().ogb_gemm_bf16_act(a.data_ptr(), w_packed.data_ptr(), out.data_ptr(), m, n, a.shape[1], a.stride(0), w_packed.stride(0),
+                                              out.stride(0), *act.args, 2 * half, status_word().data_ptr(), _stream())
+        _native.check(rc, "ogb_gemm_bf16_act")
         launch_counts["gemm_bf16_tcgen05"] += 1
         return out
     gu = scratch[:m, :n]
     assert gu.is_contiguous() and out.is_contiguous()
     linear(a, w_packed, gu)
-    rc = _native.load().ogb_act_mul_packed(gu.data_ptr(), out.data_ptr(), m, n // 2, half, ACTS[act], _ELEM[a.dtype], _stream())
+    return act_mul_packed(gu, half, act, out)
+
+
+def act_mul_packed(gate_up, half, act, out):
+    """Gated activation over columns packed by ``ops.pack_gate_up`` (contiguous rows)."""
+    m, n = gate_up.shape
+    rc = _native.load().ogb_act_mul_packed(gate_up.data_ptr(), out.data_ptr(), m, n // 2, half, *as_act(act).args, _ELEM[out.dtype], _stream())
     _native.check(rc, "ogb_act_mul_packed")
     launch_counts["act_mul_packed"] += 1
     return out
 
 
+@_timed("act_linear")
+def act_linear(a, w, act, out):
+    """out = act(a @ w^T) for an :class:`Act` of one value."""
+    act = as_act(act)
+    if not a.is_cuda:
+        out.copy_(reference.plain_act(reference.gemm(a, w, out_dtype=torch.float32), act).to(out.dtype))
+        return out
+    m, n, k = a.shape[0], w.shape[0], w.shape[1]
+    lib, ld = _native.load(), (a.stride(0), w.stride(0), out.stride(0))
+    if a.dtype == torch.bfloat16:
+        rc = lib.ogb_gemm_bf16_act(a.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, *ld, *act.args, 0, status_word().data_ptr(), _stream())
+        _native.check(rc, "ogb_gemm_bf16_act")
+        launch_counts["gemm_bf16_tcgen05"] += 1
+    else:
+        rc = lib.ogb_gemm_f32_act(a.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, *ld, *act.args, _stream())
+        _native.check(rc, "ogb_gemm_f32_act")
+        launch_counts["gemm_f32"] += 1
+    return out
+
+
 @_timed("embed_streams")
-def embed_streams(ids, table, x):
-    """Every stream of row t of x [T, S, W] (fp32) becomes the embedding of ids[t]."""
+def embed_streams(ids, table, x, norm: RmsNorm | None = None, copy=None):
+    """Every stream of row t of x [T, S, W] (fp32) becomes the embedding of ids[t], normed where ``norm`` is given; so does row t of
+    ``copy`` [T, W]."""
     t, s, w = x.shape
     if not x.is_cuda:
-        x.copy_(table[ids[:t].long()].float()[:, None, :].expand(-1, s, -1))
+        rows = table[ids[:t].long()].float()
+        if norm is not None:
+            rows = reference.rms(rows, norm.w, norm.eps)
+        x.copy_(rows[:, None, :].expand(-1, s, -1))
+        if copy is not None:
+            copy.copy_(rows)
         return x
-    rc = _native.load().ogb_embed_streams(ids.data_ptr(), table.data_ptr(), x.data_ptr(), t, s, w, table.shape[0], _ELEM[table.dtype],
-                                          status_word().data_ptr(), _stream())
+    rc = _native.load().ogb_embed_streams(ids.data_ptr(), table.data_ptr(), x.data_ptr(), t, s, w, table.shape[0], _ptr(norm.w if norm is not None else None),
+                                          float(norm.eps) if norm is not None else 0.0, _ptr(copy), copy.stride(0) if copy is not None else 0,
+                                          _ELEM[table.dtype], status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_embed_streams")
     launch_counts["embed_streams"] += 1
     return x
@@ -184,42 +247,66 @@ def hyper_step(x_in, x_out, y, written: HyperConnection | None, read, norm: Dyna
 
 
 @_timed("latent_append")
-def latent_append(c, w, eps, slots, pool, rank):
-    """RMS-norm the projected latents c [T, >= rank] and write them to their slots of pool [pages, 16, ld]."""
-    t = c.shape[0]
-    if not c.is_cuda:
-        reference.latent_append(c, w, eps, slots[:t], pool, rank)
+def latent_append(row, latent, w, eps, slots, pool, rank, rope=None):
+    """RMS-norm the latents in columns latent .. latent + rank of the projected rows [T, ld] and write them to their slots of pool
+    [pages, 16, ld].  ``rope``: a :class:`LatentRope`, which turns the rows' rotated parts."""
+    t = row.shape[0]
+    if not row.is_cuda:
+        reference.latent_append(row, latent, w, eps, slots[:t], pool, rank, rope)
         return
-    assert pool.dtype == c.dtype
-    rc = _native.load().ogb_latent_append(c.data_ptr(), c.stride(0), w.data_ptr(), float(eps), slots.data_ptr(), pool.data_ptr(), t, rank,
-                                          pool.shape[2], backed_pages(pool) * PAGE, _ELEM[c.dtype], status_word().data_ptr(), _stream())
+    assert pool.dtype == row.dtype
+    turn = [0, 0, 0, 0, 0, 0, 0, 0, 0]
+    if rope is not None:
+        q = rope.q_out
+        turn = [rope.freq.data_ptr(), rope.positions.data_ptr(), _ptr(q), rope.heads, rope.dim, 2 * rope.freq.numel(), q.stride(0) if q is not None else 0,
+                rope.q_col, rope.split]
+    rc = _native.load().ogb_latent_append(row.data_ptr(), row.stride(0), latent, w.data_ptr(), float(eps), slots.data_ptr(), pool.data_ptr(), t, rank,
+                                          pool.shape[2], backed_pages(pool) * PAGE, *turn, _ELEM[row.dtype], status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_latent_append")
     launch_counts["latent_append"] += 1
 
 
+@dataclass
+class LatentRope:
+    """Rotated parts beside a latent.  A projected row holds ``heads`` queries of pad8(dim) + pad8(rot) columns, then the latent (in
+    pad8(rank) columns) and the key part that all heads share; neighbours 2i, 2i + 1 of a part turn by position x freq[i].  Query parts
+    go to columns q_col .. of q_out [T * heads, ld] for rows below ``split`` and stay where they are for the others."""
+    freq: torch.Tensor           # fp64 [rot / 2]
+    positions: torch.Tensor
+    heads: int
+    dim: int
+    q_out: torch.Tensor | None
+    q_col: int
+    split: int
+
+
 @_timed("latent_attention")
-def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None, counters=None, decode_only=False):
-    """Rows (token, head) of q [T * heads, ld] over the latents of their sequences' pages; window <= 0: causal only.
-    ``counters``: zeroed int32 words, one per decode row and 16 heads, with which the last split of a row merges the splits.
-    ``decode_only``: leave the prefill rows to :func:`latent_prefill_expanded`."""
+def latent_attention(q, out, pool, si, heads, rank, scale, window, splits=1, part_o=None, part_ml=None, counters=None, decode_only=False, vrank=None,
+                     gate=None):
+    """Rows (token, head) of q [T * heads, ld] over the latents of their sequences' pages; window <= 0: causal only.  The first ``rank``
+    values of a page row are the key, the first ``vrank`` (None: all of them) the value.  ``gate`` [T, heads]: every head's output times
+    the sigmoid.  ``counters``: zeroed int32 words, one per decode row and 16 heads, with which the last split of a row merges the
+    splits.  ``decode_only``: leave the prefill rows to :func:`latent_prefill_expanded`."""
+    vrank = rank if vrank is None else vrank
     if not q.is_cuda:
-        reference.latent_attention(q, out, pool, si, heads, rank, scale, window)
+        reference.latent_attention(q, out, pool, si, heads, rank, scale, window, vrank, gate)
         return out
     lib, st = _native.load(), status_word().data_ptr()
     nd, npf, t = si.num_decode, si.num_prefill_seqs, si.num_tokens
     pages, mp = backed_pages(pool), si.page_table.shape[1]
     elem = _ELEM[q.dtype]
+    sizes = (heads, rank, vrank, q.stride(0), out.stride(0), pool.shape[2], gate.stride(0) if gate is not None else 0, mp)
     if nd > 0:
-        rc = lib.ogb_latent_attention(q.data_ptr(), out.data_ptr(), pool.data_ptr(), si.page_table.data_ptr(), si.ctx_len.data_ptr(), 0, 0, 0,
-                                      nd, heads, rank, q.stride(0), pool.shape[2], mp, 0, pages, int(window), float(scale), int(splits),
-                                      _ptr(part_o), _ptr(part_ml), _ptr(counters), elem, st, _stream())
+        rc = lib.ogb_latent_attention(q.data_ptr(), out.data_ptr(), pool.data_ptr(), si.page_table.data_ptr(), si.ctx_len.data_ptr(), 0, 0, 0, _ptr(gate),
+                                      nd, *sizes, 0, pages, int(window), float(scale), int(splits), _ptr(part_o), _ptr(part_ml), _ptr(counters), elem, st,
+                                      _stream())
         _native.check(rc, "ogb_latent_attention")
         launch_counts["latent_decode"] += 1
     if npf > 0 and not decode_only:
         qp, op = q[nd * heads:], out[nd * heads:]
         rc = lib.ogb_latent_attention(qp.data_ptr(), op.data_ptr(), pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(),
-                                      si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), t - nd, heads, rank, q.stride(0),
-                                      pool.shape[2], mp, si.num_tiles, pages, int(window), float(scale), 1, 0, 0, 0, elem, st, _stream())
+                                      si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), _ptr(gate[nd:] if gate is not None else None),
+                                      t - nd, *sizes, si.num_tiles, pages, int(window), float(scale), 1, 0, 0, 0, elem, st, _stream())
         _native.check(rc, "ogb_latent_attention")
         launch_counts["latent_prefill"] += 1
     return out
@@ -232,13 +319,12 @@ def visible_pages(si, window):
     return int(((si.prefill_ctx + PAGE - 1) // PAGE - lo).sum())
 
 
-def latent_prefill_expanded(q, out, pool, kv_w, si, heads, d, scale, window, pages, dense, kv, table):
-    """Prefill rows with keys and values expanded: the visible latents are packed (``dense`` [16 * pages, ld]), one product with
-    ``kv_w`` [heads * (key | value) * d, ld] writes K/V pages (``kv`` [pages, heads, 2, 16, d]), and the paged prefill kernel of the
-    dense decoders runs over them through ``table``.  Worth it when many queries share a latent and the latent is wider
-    than a head: a (query, key) pair then costs 4 d instead of 4 rank operations per head."""
-    from . import paged_prefill
-
+def latent_prefill_expanded(q, out, pool, kv_w, si, heads, kc, vc, q_head, dv, scale, window, pages, dense, kv, table, gate=None):
+    """Prefill rows with keys and values expanded: the visible page rows are packed (``dense`` [16 * pages, ld]), one product with
+    ``kv_w`` [heads * (kc key | vc value chunks) * 64, ld] writes pages of 64-column chunks (``kv`` [pages, heads, kc + vc, 16, 64]), and the
+    paged prefill kernel of the dense decoders runs over them through ``table``.  q: heads of ``q_head`` columns, out: of ``dv``.  Worth it
+    when many queries share a latent and the latent is wider than a head: a (query, key) pair then costs the head's widths in operations
+    instead of the latent's."""
     nd, npf, t = si.num_decode, si.num_prefill_seqs, si.num_tokens
     lib, st = _native.load(), status_word().data_ptr()
     mp = si.page_table.shape[1]
@@ -246,11 +332,15 @@ def latent_prefill_expanded(q, out, pool, kv_w, si, heads, d, scale, window, pag
                                backed_pages(pool), int(window), pool.shape[2], pages, dense.data_ptr(), table.data_ptr(), st, _stream())
     _native.check(rc, "ogb_latent_gather")
     rc = lib.ogb_gemm_bf16_paged(dense.data_ptr(), kv_w.data_ptr(), kv.data_ptr(), pages * PAGE, kv_w.shape[0], kv_w.shape[1], dense.stride(0),
-                                 kv_w.stride(0), d, st, _stream())
+                                 kv_w.stride(0), 64, st, _stream())
     _native.check(rc, "ogb_gemm_bf16_paged")
+    rc = lib.ogb_paged_prefill_chunks_bf16(q[nd:].data_ptr(), out[nd:].data_ptr(), kv.data_ptr(), table.data_ptr(), si.ctx_len[nd:].data_ptr(),
+                                           si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), _ptr(gate[nd:] if gate is not None else None),
+                                           si.num_tiles, npf, t - nd, mp, pages, heads, kc, vc, dv, q_head, dv, q.stride(0), out.stride(0),
+                                           gate.stride(0) if gate is not None else 0, float(scale), int(window), st, _stream())
+    _native.check(rc, "ogb_paged_prefill_chunks_bf16")
     launch_counts["latent_expand"] += 1
-    paged_prefill(q[nd:t], out[nd:t], kv[:pages], table[:npf], si.ctx_len[nd:nd + npf], si.cu_q, si.tile_seq, si.tile_q0, si.num_tiles, heads, heads,
-                  d, scale, window)
+    launch_counts["paged_prefill_tc"] += 1
 
 
 def segment_length(si, heads: int, vdim: int) -> int:
@@ -304,12 +394,21 @@ def head_rmsnorm(x, w, eps, out, heads, n, gate=None):
     return out
 
 
+def _sublayer(y):
+    """(output rows, kernel pointers, (k, ldy, lds, ldg), expert rows) of a sublayer's output: rows, :class:`ExpertRows` or None."""
+    if not isinstance(y, ExpertRows):
+        return y, (_ptr(y), 0, 0, 0, 0), (1, y.stride(0) if y is not None else 0, 0, 0), 0
+    shared = (_ptr(y.shared), _ptr(y.gate))
+    assert y.shared is None or (y.shared.dtype == y.rows.dtype and y.gate.dtype == torch.float32)
+    lds, ldg = (y.shared.stride(0), y.gate.stride(0)) if y.shared is not None else (0, 0)
+    return y.rows, (y.rows.data_ptr(), y.pos.data_ptr(), y.weight.data_ptr(), *shared), (y.pos.shape[1], y.rows.stride(0), lds, ldg), y.rows.shape[0]
+
+
 @_timed("norm_step")
 def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
-    """x [T, W] fp32 += post(y); h = norm(x).  ``y``: rows of the last sublayer's output, :class:`ExpertRows`, or None.  ``gather``:
-    h gets the rows it names only, and x stays as it is."""
+    """x [T, W] fp32 += post(y) (None: y as it is); h = norm(x) (None: x).  ``y``: rows of the last sublayer's output, :class:`ExpertRows`,
+    or None.  ``gather``: h gets the rows it names only, and x stays as it is."""
     rows = h.shape[0] if h is not None else x.shape[0]
-    routed = y if isinstance(y, ExpertRows) else None
     if not x.is_cuda:
         new = reference.norm_step(x, y, post)
         if gather is None:
@@ -317,18 +416,40 @@ def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
         else:
             new = new[gather.long()]
         if h is not None:
-            h[:, : x.shape[1]] = reference.rms(new, norm.w, norm.eps).to(h.dtype)
+            h[:, : x.shape[1]] = (reference.rms(new, norm.w, norm.eps) if norm is not None else new).to(h.dtype)
         return h
-    src = routed.rows if routed is not None else y
-    eps = norm.eps if norm is not None else post.eps
+    src, ptrs, (k, ldy, lds, ldg), y_rows = _sublayer(y)
+    eps = norm.eps if norm is not None else post.eps if post is not None else 0.0
     assert post is None or post.eps == eps
+    assert x.is_contiguous()
     rc = _native.load().ogb_norm_step(
-        x.data_ptr(), _ptr(src), _ptr(routed.pos if routed else None), _ptr(routed.weight if routed else None), _ptr(post.w if post is not None else None),
-        _ptr(norm.w if norm is not None else None), _ptr(h), _ptr(gather), float(eps), rows, x.shape[0], x.shape[1],
-        routed.pos.shape[1] if routed else 1, src.stride(0) if src is not None else 0, h.stride(0) if h is not None else 0,
-        routed.rows.shape[0] if routed else 0, _ELEM[h.dtype if h is not None else src.dtype], status_word().data_ptr(), _stream())
+        x.data_ptr(), *ptrs, _ptr(post.w if post is not None else None), _ptr(norm.w if norm is not None else None), _ptr(h), _ptr(gather), float(eps), rows,
+        x.shape[0], x.shape[1], k, ldy, lds, ldg, h.stride(0) if h is not None else 0, y_rows, _ELEM[h.dtype if h is not None else src.dtype],
+        status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_norm_step")
     launch_counts["norm_step"] += 1
+    return h
+
+
+@_timed("norm_conv_step")
+def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si):
+    """x_out [T, W] = x_in + y + add (y as for :func:`norm_step`, add [W] or None); h_t = sum_j conv[j] n_(t - taps + 1 + j) along every sequence
+    with n = norm(x_out), conv [taps, W] fp32, state [slots, taps - 1, W] advanced.  Where nothing is added x_out may be None."""
+    t, w = x_in.shape
+    if not x_in.is_cuda:
+        new = reference.norm_step(x_in, y, None)
+        if add is not None:
+            new = new + add
+        if x_out is not None:
+            x_out.copy_(new)
+        h[:, :w] = reference.short_conv(reference.rms(new, norm.w, norm.eps), conv, state, si).to(h.dtype)
+        return h
+    src, ptrs, (k, ldy, lds, ldg), y_rows = _sublayer(y)
+    rc = _native.load().ogb_norm_conv_step(
+        x_in.data_ptr(), _ptr(x_out), *ptrs, _ptr(add), norm.w.data_ptr(), conv.data_ptr(), state.data_ptr(), h.data_ptr(), float(norm.eps), w, conv.shape[0], k,
+        x_in.stride(0), ldy, lds, ldg, h.stride(0), y_rows, *_rows_args(si, state), _ELEM[h.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_norm_conv_step")
+    launch_counts["norm_conv_step"] += 1
     return h
 
 

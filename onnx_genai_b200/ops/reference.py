@@ -332,9 +332,10 @@ def quantize_w4(w, block=32, symmetric=True):
     return q, scales, zp
 
 
-def moe_route(router_logits, k, renormalize=True, groups=1, keep=1):
+def moe_route(router_logits, k, renormalize=True, groups=1, keep=1, bias=None):
     """``groups`` > 1: only experts of the ``keep`` groups of neighbours whose best expert scores highest can be chosen."""
-    probs = torch.softmax(router_logits.float(), dim=-1)
+    logits = router_logits.float()
+    probs = torch.softmax(logits if bias is None else logits + bias, dim=-1)
     if groups > 1:
         best = probs.view(probs.shape[0], groups, -1).amax(-1)
         kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, torch.topk(best, keep, dim=-1).indices, True)
@@ -352,14 +353,28 @@ def gelu_tanh(z):
     return torch.nn.functional.gelu(z, approximate="tanh")
 
 
-GATED_ACTS = {"silu": torch.nn.functional.silu, "gelu_tanh": gelu_tanh}
+def gated_act(act, g, u):
+    """``act``: ops.hybrid.Act of a gate and an up value."""
+    if act.kind == "clamp_glu":
+        g, u = g.clamp(max=act.a), u.clamp(-act.a, act.a)
+        return g * torch.sigmoid(1.702 * g) * (u + 1)
+    return {"silu": torch.nn.functional.silu, "gelu_tanh": gelu_tanh}[act.kind](g) * u
+
+
+def plain_act(v, act):
+    """``act``: ops.hybrid.Act of one value."""
+    if act.kind == "relu2":
+        return torch.relu(v).pow(2)
+    if act.kind == "xielu":
+        return v / 2 + torch.where(v > 0, act.a * v * v, act.b * (torch.expm1(v.clamp(max=0)) - v))
+    return v
 
 
 def act_mul_packed(gate_up, half, act, out_dtype=None):
-    """act(gate) * up over columns interleaved by :func:`pack_gate_up`."""
+    """Gated activation over columns interleaved by :func:`pack_gate_up`."""
     t, n = gate_up.shape
     y = gate_up.float().view(t, n // (2 * half), 2, half)
-    return (GATED_ACTS[act](y[:, :, 0]) * y[:, :, 1]).reshape(t, n // 2).to(out_dtype or gate_up.dtype)
+    return gated_act(act, y[:, :, 0], y[:, :, 1]).reshape(t, n // 2).to(out_dtype or gate_up.dtype)
 
 
 def hyper_step(x, y=None, mix=None, out_w=None, in_w=None, norm=None):
@@ -422,12 +437,17 @@ def head_rmsnorm(x, w, eps, heads, n, out_dtype=None, gate=None):
 
 
 def norm_step(x, y, post):
-    """x + post(y) for rows of y, or the weighted sum of a token's expert rows (ops.hybrid.ExpertRows)."""
+    """x + post(y) for rows of y, or the weighted sum of a token's expert rows (ops.hybrid.ExpertRows); y as it is without post."""
     if y is None:
         return x
     if not torch.is_tensor(y):
-        y = (y.rows[y.pos.long()].float() * y.weight[:, :, None]).sum(1)
-    return x + rms(y[:, : x.shape[1]].float(), post.w, post.eps)
+        rows = (y.rows[y.pos.long()].float() * y.weight[:, :, None]).sum(1)
+        if y.shared is not None:
+            w = min(rows.shape[1], y.shared.shape[1])
+            rows = rows[:, :w] + torch.sigmoid(y.gate)[:, None] * y.shared[:, :w].float()
+        y = rows
+    y = y[:, : x.shape[1]].float()
+    return x + (rms(y, post.w, post.eps) if post is not None else y)
 
 
 def short_conv(u, w, state, si):
@@ -516,17 +536,39 @@ def diff_attention(q, out, pool, si, hq, hkv, d, dv, dp, vp, scale, lam, eps, ga
         out[base:base + n].view(n, hq, vp)[..., :dv] = rms(a[0] - lam * a[1], gain, eps).to(out.dtype)
 
 
-def latent_append(c, w, eps, slots, pool, rank):
-    """RMS norm of every row of c, written to its slot of pool [pages, 16, >= rank]."""
-    y = c[:, :rank].float()
+def rotate_pairs(x, pos, freq):
+    """x [T, heads, 2 len(freq)]: dimension 2i turns with 2i + 1 by pos * freq[i]."""
+    a = pos.double()[:, None] * freq[None, :]
+    c, s = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+
+
+def latent_append(row, latent, w, eps, slots, pool, rank, rope=None):
+    """RMS norm of columns latent .. latent + rank, written to the rows' slots of pool [pages, 16, ld]; ``rope``: ops.hybrid.LatentRope."""
+    y = row[:, latent:latent + rank].float()
     y = (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w).to(pool.dtype)
     flat = pool.view(-1, pool.shape[-1])
     live = slots >= 0
-    flat[slots[live].long(), :rank] = y[live]
+    at = slots[live].long()
+    flat[at, :rank] = y[live]
+    if rope is None:
+        return
+    t, rot = row.shape[0], 2 * rope.freq.numel()
+    up8 = lambda n: n + (-n) % 8
+    pos, part = rope.positions[:t], latent + up8(rank)
+    flat[at, up8(rank):up8(rank) + rot] = rotate_pairs(row[:, None, part:part + rot], pos, rope.freq)[live, 0].to(pool.dtype)
+    dp, step = up8(rope.dim), up8(rope.dim) + up8(rot)
+    q = row[:, : rope.heads * step].unflatten(1, (rope.heads, step))[..., dp:dp + rot]
+    turned = rotate_pairs(q, pos, rope.freq).to(row.dtype)
+    if rope.split > 0:
+        rope.q_out[: rope.split * rope.heads, rope.q_col:rope.q_col + rot] = turned[: rope.split].reshape(-1, rot)
+    q[rope.split:] = turned[rope.split:]
 
 
-def latent_attention(q, out, pool, si, heads, rank, scale, window):
-    """q / out [T * heads, >= rank]: every head attends to the latents of its sequence's pages (key and value alike)."""
+def latent_attention(q, out, pool, si, heads, rank, scale, window, vrank=None, gate=None):
+    """q [T * heads, >= rank]: every head attends to the page rows of its sequence (keys, and values in the first vrank columns)."""
+    vrank = rank if vrank is None else vrank
     for e, base, n, start, _ in step_entries(si):
         ctx = start + n
         lo = max(0, start - window + 1) if window > 0 else 0
@@ -540,5 +582,7 @@ def latent_attention(q, out, pool, si, heads, rank, scale, window):
         qs = q[base * heads:(base + n) * heads, :rank].float().view(n, heads, rank)
         s = torch.einsum("nhr,kr->nhk", qs, c) * scale
         p = torch.softmax(s.masked_fill(~seen[:, None, :], float("-inf")), -1)
-        o = torch.einsum("nhk,kr->nhr", p, c)
-        out[base * heads:(base + n) * heads, :rank] = o.reshape(n * heads, rank).to(out.dtype)
+        o = torch.einsum("nhk,kr->nhr", p, c[:, :vrank])
+        if gate is not None:
+            o = o * torch.sigmoid(gate[base:base + n].float())[..., None]
+        out[base * heads:(base + n) * heads, :vrank] = o.reshape(n * heads, vrank).to(out.dtype)

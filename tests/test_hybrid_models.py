@@ -189,7 +189,7 @@ def test_latent_append_norms_and_places(device):
     c = torch.randn(9, 40, generator=g)
     w, slots = torch.rand(36, generator=g) + 0.5, torch.tensor([5, 16, 17, -1, 31, 0, 47, 33, 2], dtype=torch.int32)
     pool = torch.zeros(3, 16, 40, device=device)
-    H.latent_append(c.to(device), w.to(device), 1e-3, slots.to(device), pool, 36)
+    H.latent_append(c.to(device), 0, w.to(device), 1e-3, slots.to(device), pool, 36)
     flat = pool.cpu().view(48, 40)
     want = O.root_mean_square_norm(c[:, :36], w, 1e-3)
     for r, s in enumerate(slots.tolist()):
