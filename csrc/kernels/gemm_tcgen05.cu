@@ -782,8 +782,13 @@ static bool stream_k_enabled() {
 // the tensor-parallel path, whose tiles end in stores to other GPUs, keeps the 13 it was tuned with.
 constexpr float kSkFixPlain = 40.0f;
 constexpr float kSkFixScatter = 13.0f;
+// A finisher adds the partials of a tile one after the other, so the fix-up grows with the CTAs that share a tile once they are many
+// (8 tiles on 148 SMs, 19 each, took 123 us where whole tiles take 20).
+constexpr float kSkShared = 6.0f;
 static bool stream_k_applies(int tiles, int k_blocks, int sms, float fix) {
   if (!stream_k_enabled() || tiles % sms == 0 || static_cast<long long>(tiles) * k_blocks < 2LL * sms) return false;
+  const float shared = static_cast<float>(sms) / static_cast<float>(tiles);
+  if (shared > kSkShared) fix *= shared / kSkShared;
   const float w = static_cast<float>(tiles) / static_cast<float>(sms);
   const float dp = static_cast<float>((tiles + sms - 1) / sms);
   const float sk = w + fix / static_cast<float>(k_blocks);

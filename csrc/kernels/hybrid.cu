@@ -277,17 +277,20 @@ OGB_DEVICE void block_sums(float (&v)[NB], float (&red)[2][NB][32], int parity) 
 //
 //   x <- x + rms(y) post        h = rms(x) w
 //
-// Without `post` the output is added as it is, without `w` h is the residual itself.  One block per row, the row in registers; all
-// fp32.
+// Without `post` the output is added as it is, without `w` h is the residual itself.  The residual may come from elsewhere (x_in), and a
+// vector may be added to it.  One block per row, the row in registers; all fp32.
 // ------------------------------------------------------------------------------------------------------
 struct NormStepParams {
-  float* x;                // [rows, W]
+  const float* x_in;       // [rows, ldx]
+  float* x;                // [rows, W], or null where nothing is added
   SublayerOut out;
+  const float* add;        // [W] or null
   const float *post, *w;   // norm weights or null
   void* h;                 // [rows, ldh] or null
+  float* factor;           // [rows] or null: gets 1 / root mean square of x
   const int* gather;       // row r of h comes from row gather[r]; x is then left alone
   float eps;
-  int rows, total_rows, W, ldh;
+  int rows, total_rows, W, ldx, ldh;
   int* status;
 };
 
@@ -304,13 +307,23 @@ __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
     }
   }
   float x[N][V];
-  float* xr = p.x + static_cast<size_t>(t) * p.W;
+  const float* xr = p.x_in + static_cast<size_t>(t) * p.ldx;
+  float* xw = p.gather == nullptr ? p.x + static_cast<size_t>(t) * p.W : nullptr;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * V;
 #pragma unroll
     for (int v = 0; v < V; ++v) x[i][v] = 0.f;
-    if (c < p.W) load_vec<V>(xr + c, x[i]);
+    if (c < p.W) {
+      load_vec<V>(xr + c, x[i]);
+      if (p.add != nullptr) {
+        float a[V];
+        load_vec<V>(p.add + c, a);
+#pragma unroll
+        for (int v = 0; v < V; ++v) x[i][v] += a[v];
+        if (p.out.y == nullptr && xw != nullptr) store_vec<V>(xw + c, x[i]);
+      }
+    }
   }
   if (p.out.y != nullptr) {
     float y[1][N][V], inv[1] = {0.f};
@@ -331,20 +344,22 @@ __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
         if (p.post != nullptr) load_vec<V>(p.post + c, g);
 #pragma unroll
         for (int v = 0; v < V; ++v) x[i][v] = p.post != nullptr ? fmaf(y[0][i][v] * inv[0], g[v], x[i][v]) : x[i][v] + y[0][i][v];
-        if (p.gather == nullptr) store_vec<V>(xr + c, x[i]);
+        if (xw != nullptr) store_vec<V>(xw + c, x[i]);
       }
     }
   }
-  if (p.h == nullptr) return;
+  if (p.h == nullptr && p.factor == nullptr) return;
   float inv[1] = {0.f};
-  if (p.w != nullptr) {
+  if (p.w != nullptr || p.factor != nullptr) {
 #pragma unroll
     for (int i = 0; i < N; ++i)
 #pragma unroll
       for (int v = 0; v < V; ++v) inv[0] = fmaf(x[i][v], x[i][v], inv[0]);
     block_sums<1>(inv, red, 1);
     inv[0] = 1.f / sqrtf(inv[0] / static_cast<float>(p.W) + p.eps);
+    if (p.factor != nullptr && threadIdx.x == 0) p.factor[r] = inv[0];
   }
+  if (p.h == nullptr) return;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * V;
@@ -403,24 +418,9 @@ struct NormConvParams {
 template <typename T, int V, int N, int NB, int TM>
 __global__ void __launch_bounds__(512) norm_conv_kernel(NormConvParams p) {
   __shared__ float red[2][NB][32];
-  const StepRows& sr = p.sr;
-  int entry, base, n, j0;                      // sequence entry, its first row, its rows, first row of this block within them
-  if (static_cast<int>(blockIdx.x) < sr.num_decode) {
-    entry = blockIdx.x; base = entry; n = 1; j0 = 0;
-  } else {
-    const int g = blockIdx.x - sr.num_decode, tile = g / (64 / kNcRows), s = sr.tile_seq[tile];
-    entry = sr.num_decode + s;
-    base = sr.num_decode + sr.cu_q[s];
-    n = sr.cu_q[s + 1] - sr.cu_q[s];
-    j0 = sr.tile_q0[tile] + (g % (64 / kNcRows)) * kNcRows;
-  }
-  const int start = sr.ctx_len[entry] - n;     // tokens before the chunk
-  if (j0 >= n || start < 0) return;            // a padding row has none
-  int slot = sr.state_slot[entry];
-  if (slot >= sr.num_slots) {
-    if (threadIdx.x == 0) atomicOr(p.status, kStatusIndexOutOfRange);
-    slot = -1;
-  }
+  RowSpan<kNcRows> r;
+  if (!r.set(p.sr, blockIdx.x, p.status)) return;
+  const int base = r.base, n = r.n, j0 = r.j0, j1 = r.j1, start = r.start, slot = r.slot;
   float conv[TM][N][V], w[N][V], h[TM > 1 ? TM - 1 : 1][N][V];    // filters aligned to their last tap; h: the last values, oldest first
   const int col0 = threadIdx.x * V, step = blockDim.x * V, off = TM - p.taps;
 #pragma unroll
@@ -550,7 +550,6 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(NormConvParams p) {
       recompute(j0 - (p.taps - 1), p.taps - 1);
     }
   }
-  const int j1 = min(j0 + kNcRows, n);
   for (int j = j0; j < j1; j += NB) {
     const int m = min(NB, j1 - j);
     normed(j, m, true, o);
@@ -576,7 +575,7 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(NormConvParams p) {
 
 template <typename T, int V, int TM>
 static int launch_norm_conv(const NormConvParams& p, cudaStream_t s) {
-  const int units = (p.W + V - 1) / V, blocks = p.sr.num_decode + p.sr.num_tiles * (64 / kNcRows);
+  const int units = (p.W + V - 1) / V, blocks = span_blocks<kNcRows>(p.sr);
   const int n = units <= 256 ? 1 : units <= 1024 ? 2 : units <= 2048 ? 4 : 8;
   const int threads = ((units + n - 1) / n + 31) / 32 * 32;
   if (threads > 512 || n * V > 16) return -2;
@@ -584,6 +583,96 @@ static int launch_norm_conv(const NormConvParams& p, cudaStream_t s) {
   else if (n == 2) norm_conv_kernel<T, V, 2, V == 1 ? 4 : 2, TM><<<blocks, threads, 0, s>>>(p);
   else if (n == 4) norm_conv_kernel<T, V, 4, V == 1 ? 4 : 1, TM><<<blocks, threads, 0, s>>>(p);
   else if constexpr (V == 1) norm_conv_kernel<T, V, 8, 2, TM><<<blocks, threads, 0, s>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------------
+// input_conv is the second half of that pass for steps of many rows: norm_step has left the residual and its rows' factors, and the
+// convolution is elementwise in the column.  A thread keeps V columns and walks a block's rows; slots as above.
+// ------------------------------------------------------------------------------------------------------
+struct InputConvParams {
+  const float* x;          // [rows, W]
+  const float* factor;     // [rows]
+  const float* w;          // [W]
+  const float* conv;       // [taps, W]
+  float* state;            // [slots, taps - 1, W]
+  void* h;                 // [rows, ldh]
+  int W, ldh, taps;
+  StepRows sr;
+  int* status;
+};
+
+template <typename T, int V, int TM>
+__global__ void __launch_bounds__(128) input_conv_kernel(InputConvParams p) {
+  RowSpan<kNcRows> r;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V, off = TM - p.taps;
+  if (!r.set(p.sr, blockIdx.x, p.status) || c >= p.W) return;
+  float conv[TM][V], w[V], h[TM > 1 ? TM - 1 : 1][V];        // filters aligned to their last tap; h: the last values, oldest first
+  load_vec<V>(p.w + c, w);
+#pragma unroll
+  for (int k = 0; k < TM; ++k) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) conv[k][v] = 0.f;
+    if (k >= off) load_vec<V>(p.conv + static_cast<size_t>(k - off) * p.W + c, conv[k]);
+  }
+  auto normed = [&](int t, float (&o)[V]) {
+    load_vec<V>(p.x + static_cast<size_t>(r.base + t) * p.W + c, o);
+    const float f = p.factor[r.base + t];
+#pragma unroll
+    for (int v = 0; v < V; ++v) o[v] *= f * w[v];
+  };
+  float* st = r.slot >= 0 ? p.state + static_cast<size_t>(r.slot) * (p.taps - 1) * p.W + c : nullptr;
+#pragma unroll
+  for (int k = 0; k < (TM > 1 ? TM - 1 : 1); ++k) {
+    const int t = r.j0 - (TM - 1) + k;                       // within the chunk
+#pragma unroll
+    for (int v = 0; v < V; ++v) h[k][v] = 0.f;
+    if (k < off || TM == 1) continue;
+    if (t >= 0) normed(t, h[k]);
+    else if (st != nullptr && r.start + t >= 0) load_vec<V>(st + static_cast<size_t>(k - off) * p.W, h[k]);
+  }
+  if (r.j0 == 0 && st != nullptr) {
+#pragma unroll
+    for (int k = 0; k < TM - 1; ++k) {
+      if (k < off) continue;
+      const int t = r.n - (TM - 1) + k;
+      float o[V];
+#pragma unroll
+      for (int q = 0; q < TM - 1; ++q)                       // fewer rows than taps: older values move up
+#pragma unroll
+        for (int v = 0; v < V; ++v) o[v] = (q == 0 || q == k + r.n) ? h[q][v] : o[v];
+      if (t >= 0) normed(t, o);
+      store_vec<V>(st + static_cast<size_t>(k - off) * p.W, o);
+    }
+  }
+  constexpr int NB = 4;
+  for (int j = r.j0; j < r.j1; j += NB) {
+    float o[NB][V];
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+      if (j + b < r.j1) normed(j + b, o[b]);
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      if (j + b >= r.j1) continue;
+      float u[V];
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        u[v] = conv[TM - 1][v] * o[b][v];
+#pragma unroll
+        for (int k = 0; k < TM - 1; ++k) u[v] = fmaf(conv[k][v], h[k][v], u[v]);
+#pragma unroll
+        for (int k = 0; k + 1 < TM - 1; ++k) h[k][v] = h[k + 1][v];
+        h[TM > 1 ? TM - 2 : 0][v] = o[b][v];
+      }
+      store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r.base + j + b) * p.ldh + c, u);
+    }
+  }
+}
+
+template <typename T, int V, int TM>
+static int launch_input_conv(const InputConvParams& p, cudaStream_t s) {
+  const dim3 grid(span_blocks<kNcRows>(p.sr), (p.W + 128 * V - 1) / (128 * V));
+  input_conv_kernel<T, V, TM><<<grid, 128, 0, s>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -678,8 +767,9 @@ __global__ void __launch_bounds__(128) latent_rope_append_kernel(LatentAppendPar
   for (int i = threadIdx.x; i < (p.heads + 1) * half; i += blockDim.x) {
     const int head = i / half, e = i - head * half;
     const bool key = head == p.heads;
-    T* src = row + (key ? p.latent + (p.rank + 7) / 8 * 8 : head * (dp + rp) + dp) + 2 * e;
-    const float u = to_f32<T>(src[0]), v = to_f32<T>(src[1]);
+    T* src = row + (key ? p.latent + (p.rank + 7) / 8 * 8 : head * (dp + rp) + dp) + 2 * e;      // parts start on 8 elements
+    float x[2];
+    load_vec<2>(src, x);
     const float2 cs = s_turn[e];
     T* dst = src;
     if (key) {
@@ -688,8 +778,8 @@ __global__ void __launch_bounds__(128) latent_rope_append_kernel(LatentAppendPar
     } else if (t < p.split) {
       dst = static_cast<T*>(p.q_out) + (static_cast<size_t>(t) * p.heads + head) * p.ldq + p.q_col + 2 * e;
     }
-    dst[0] = from_f32<T>(u * cs.x - v * cs.y);
-    dst[1] = from_f32<T>(v * cs.x + u * cs.y);
+    const float o[2] = {x[0] * cs.x - x[1] * cs.y, x[1] * cs.x + x[0] * cs.y};
+    store_vec<2>(dst, o);
   }
 }
 
@@ -857,7 +947,8 @@ extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const floa
                              const float* w, void* h, const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int lds, int ldg,
                              int ldh, int64_t y_rows, int elem, int* status, void* stream) {
   if (rows <= 0) return 0;
-  NormStepParams p{x, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, post, w, h, gather, eps, rows, total_rows, W, ldh, status};
+  NormStepParams p{x, x, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, nullptr, post, w, h, nullptr, gather, eps, rows, total_rows,
+                   W, W, ldh, status};
   if (W < 1 || !sublayer_ok(p.out)) return -3;
   // four elements at a time need rows that start on them, and pointers too
   const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared);
@@ -869,29 +960,38 @@ extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const floa
   return -3;
 }
 
-// x_out null: nothing is added (y and add null).  At most 8 taps; rows of up to 8192 columns, 4096 where they do not start on four
-// elements.
+// x_out null: nothing is added (y and add null).  At most 8 taps.  factor null: one kernel, for few rows (of up to 8192 columns, 4096
+// where they do not start on four elements); else [rows] of scratch, norm_step and input_conv.
+template <typename T>
+static int norm_conv(const NormConvParams& p, float* factor, int rows, bool vec, cudaStream_t s) {
+  if (factor == nullptr)
+    return vec ? (p.taps <= 4 ? launch_norm_conv<T, 4, 4>(p, s) : launch_norm_conv<T, 4, 8>(p, s))
+               : (p.taps <= 4 ? launch_norm_conv<T, 1, 4>(p, s) : launch_norm_conv<T, 1, 8>(p, s));
+  const NormStepParams n{p.x_in, p.x_out, p.out, p.add, nullptr, nullptr, nullptr, factor, nullptr, p.eps, rows, rows, p.W, p.ldx, 0, p.status};
+  const int rc = vec ? launch_norm_step<T, 4>(n, s) : launch_norm_step<T, 1>(n, s);
+  if (rc != 0) return rc;
+  const InputConvParams q{p.x_out != nullptr ? p.x_out : p.x_in, factor, p.w, p.conv, p.state, p.h, p.W, p.ldh, p.taps, p.sr, p.status};
+  return vec ? (p.taps <= 4 ? launch_input_conv<T, 4, 4>(q, s) : launch_input_conv<T, 4, 8>(q, s))
+             : (p.taps <= 4 ? launch_input_conv<T, 1, 4>(q, s) : launch_input_conv<T, 1, 8>(q, s));
+}
+
 extern "C" int ogb_norm_conv_step(const float* x_in, float* x_out, const void* y, const int* pos, const float* weight, const void* shared,
-                                  const float* gate, const float* add, const float* w, const float* conv, float* state, void* h, float eps, int W,
-                                  int taps, int k, int ldx, int ldy, int lds, int ldg, int ldh, int64_t y_rows, const int* ctx_len,
-                                  const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode, int num_tiles,
-                                  int num_slots, int elem, int* status, void* stream) {
+                                  const float* gate, const float* add, const float* w, const float* conv, float* state, void* h, float* factor,
+                                  float eps, int rows, int W, int taps, int k, int ldx, int ldy, int lds, int ldg, int ldh, int64_t y_rows,
+                                  const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode,
+                                  int num_tiles, int num_slots, int elem, int* status, void* stream) {
   if (num_decode + num_tiles <= 0) return 0;
   NormConvParams p{x_in, x_out, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, add, w, conv, state, h, eps, W, ldx, ldh, taps,
                    StepRows{ctx_len, state_slot, cu_q, tile_seq, tile_q0, num_decode, num_tiles, num_slots}, status};
   if (W < 1 || taps < 1 || taps > 8 || x_in == x_out || !sublayer_ok(p.out) || w == nullptr || conv == nullptr || h == nullptr) return -3;
-  if ((taps > 1 && state == nullptr) || ((y != nullptr || add != nullptr) && x_out == nullptr)) return -3;
+  if ((taps > 1 && state == nullptr) || ((y != nullptr || add != nullptr) && x_out == nullptr) || (x_out == nullptr && ldx != W)) return -3;
   const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared);
   const uintptr_t f32 = reinterpret_cast<uintptr_t>(x_in) | reinterpret_cast<uintptr_t>(x_out) | reinterpret_cast<uintptr_t>(add) |
                         reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(conv) | reinterpret_cast<uintptr_t>(state);
   const bool vec = ((W | ldx | ldy | ldh | lds) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-#define OGB_NORM_CONV(T) \
-  return vec ? (taps <= 4 ? launch_norm_conv<T, 4, 4>(p, s) : launch_norm_conv<T, 4, 8>(p, s)) \
-             : (taps <= 4 ? launch_norm_conv<T, 1, 4>(p, s) : launch_norm_conv<T, 1, 8>(p, s))
-  if (elem == kElemBF16) OGB_NORM_CONV(__nv_bfloat16);
-  if (elem == kElemF32) OGB_NORM_CONV(float);
-#undef OGB_NORM_CONV
+  if (elem == kElemBF16) return norm_conv<__nv_bfloat16>(p, factor, rows, vec, s);
+  if (elem == kElemF32) return norm_conv<float>(p, factor, rows, vec, s);
   return -3;
 }
 

@@ -16,7 +16,7 @@ template <typename T> OGB_DEVICE T from_f32(float v);
 template <> OGB_DEVICE float from_f32<float>(float v) { return v; }
 template <> OGB_DEVICE __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
-// V consecutive elements as fp32 (one vector access where V = 4; the pointer is then aligned to it)
+// V consecutive elements as fp32 (one vector access where V is 2 or 4; the pointer is then aligned to it)
 template <int V, typename T>
 OGB_DEVICE void load_vec(const T* p, float (&r)[V]) {
   if constexpr (V == 4 && sizeof(T) == 4) {
@@ -29,6 +29,9 @@ OGB_DEVICE void load_vec(const T* p, float (&r)[V]) {
   } else if constexpr (V == 2 && sizeof(T) == 4) {
     const float2 f = *reinterpret_cast<const float2*>(p);
     r[0] = f.x; r[1] = f.y;
+  } else if constexpr (V == 2) {
+    const float2 f = unpack_bf16(*reinterpret_cast<const uint32_t*>(p));
+    r[0] = f.x; r[1] = f.y;
   } else {
 #pragma unroll
     for (int i = 0; i < V; ++i) r[i] = to_f32<T>(p[i]);
@@ -40,6 +43,10 @@ OGB_DEVICE void store_vec(T* p, const float (&r)[V]) {
     *reinterpret_cast<float4*>(p) = make_float4(r[0], r[1], r[2], r[3]);
   } else if constexpr (V == 4) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]));
+  } else if constexpr (V == 2 && sizeof(T) == 4) {
+    *reinterpret_cast<float2*>(p) = make_float2(r[0], r[1]);
+  } else if constexpr (V == 2) {
+    *reinterpret_cast<uint32_t*>(p) = pack_bf16(r[0], r[1]);
   } else {
 #pragma unroll
     for (int i = 0; i < V; ++i) p[i] = from_f32<T>(r[i]);
@@ -57,6 +64,35 @@ struct StepRows {
   const int* tile_q0;
   int num_decode, num_tiles, num_slots;
 };
+
+// The rows of block `b`: a decode row, or up to R (a divisor of 64) rows of one prefill chunk; a grid has span_blocks of them.
+template <int R>
+struct RowSpan {
+  int base, n, j0, j1, start, slot;            // first row of the entry, its rows, this block's rows within them, tokens before, slot (-1: none)
+  OGB_DEVICE bool set(const StepRows& sr, int b, int* status) {
+    int entry;
+    if (b < sr.num_decode) {
+      entry = b; base = b; n = 1; j0 = 0;
+    } else {
+      const int g = b - sr.num_decode, tile = g / (64 / R), s = sr.tile_seq[tile];
+      entry = sr.num_decode + s;
+      base = sr.num_decode + sr.cu_q[s];
+      n = sr.cu_q[s + 1] - sr.cu_q[s];
+      j0 = sr.tile_q0[tile] + (g % (64 / R)) * R;
+    }
+    j1 = min(j0 + R, n);
+    start = sr.ctx_len[entry] - n;
+    if (j0 >= n || start < 0) return false;    // a padding row has no tokens
+    slot = sr.state_slot[entry];
+    if (slot >= sr.num_slots) {
+      if (threadIdx.x == 0) atomicOr(status, kStatusIndexOutOfRange);
+      slot = -1;
+    }
+    return true;
+  }
+};
+template <int R>
+inline int span_blocks(const StepRows& sr) { return sr.num_decode + sr.num_tiles * (64 / R); }
 
 // two fp32 values in one 64-bit register
 typedef unsigned long long f32x2;

@@ -202,8 +202,8 @@ int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, 
                   int elem, int* status, void* stream);
 // norm_conv_step: x_out = x_in + y + add, h = a causal convolution over rms(x_out) w.
 int ogb_norm_conv_step(const float* x_in, float* x_out, const void* y, const int* pos, const float* weight, const void* shared, const float* gate,
-                       const float* add, const float* w, const float* conv, float* state, void* h, float eps, int W, int taps, int k, int ldx, int ldy,
-                       int lds, int ldg, int ldh, int64_t y_rows, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq,
+                       const float* add, const float* w, const float* conv, float* state, void* h, float* factor, float eps, int rows, int W, int taps,
+                       int k, int ldx, int ldy, int lds, int ldg, int ldh, int64_t y_rows, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq,
                        const int* tile_q0, int num_decode, int num_tiles, int num_slots, int elem, int* status, void* stream);
 // Short causal convolutions (short_conv.cu): w [taps, channels], state [slots, taps - 1, channels].
 // Attention: q (nq heads of d) | k (nk) | v (nv heads of dv); rotated queries to q, keys and values to pages [nk][16][dp] | [nv][16][vp].

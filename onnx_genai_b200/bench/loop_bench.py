@@ -72,9 +72,10 @@ def kernel_rows(size: str, timer, pk):
         w = hops.RmsNorm(f32(hid), 1e-6)
         conv, state = f32(TAPS, hid), torch.zeros(nseq, TAPS - 1, hid, device="cuda")
         sb = 2 * nseq * (TAPS - 1) * hid * 4
-        row("norm_conv_step", phase, lambda: hops.norm_conv_step(x0, x1, y, None, w, conv, state, h, si), nbytes=t * hid * (8 + 4) + sb)
+        factor = f32(t) if prompt else None
+        row("norm_conv_step", phase, lambda: hops.norm_conv_step(x0, x1, y, None, w, conv, state, h, si, factor), nbytes=t * hid * (8 + 4) + sb)
         routed = hops.ExpertRows(rnd(t * top, hid), torch.randperm(t * top, device="cuda").int().view(t, top), f32(t, top), rnd(t, hid), f32(t, e + 8)[:, e])
-        row("norm_conv_step over expert rows", phase, lambda: hops.norm_conv_step(x0, x1, routed, None, w, conv, state, h, si),
+        row("norm_conv_step over expert rows", phase, lambda: hops.norm_conv_step(x0, x1, routed, None, w, conv, state, h, si, factor),
             nbytes=t * hid * (8 + 2 + 2 * (top + 1)) + sb)
         xs0, xs1, prev, amount = rnd(t, 2, hid, dtype=torch.float32), empty(t, 2, hid, dtype=torch.float32), f32(nseq, hid), f32(hid)
         hc, dyn = hops.HyperConnection(f32(2), f32(2), f32(2, 2)), hops.DynamicTanh(f32(1), f32(hid), f32(hid))

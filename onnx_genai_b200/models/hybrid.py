@@ -662,6 +662,7 @@ class HybridModel:
         flat = lambda width, dtype=dt: z(max_tokens * width, dtype=dtype) if width else None    # viewed per layer: rows stay contiguous
         self.qfv = flat(most(pad8(m.heads * (2 * m.dim + m.vdim)) for m in rec), torch.float32)
         self.rec_o = flat(most(m.heads * m.vdim for m in rec + delta), torch.float32)
+        self.factor = z(max_tokens, dtype=torch.float32) if cfg.input_taps else None
         self.loop_in = self.loop_x = None
         if cfg.loop is not None:       # residual | embedding, and the residual a pass begins with
             self.loop_in, self.loop_x = z(max_tokens, 2 * pad8(hid)), z(max_tokens, pad8(hid), dtype=torch.float32)
@@ -833,6 +834,7 @@ class HybridModel:
                                          self._scratch("table", (si.num_prefill_seqs, si.page_table.shape[1]), torch.int32), gate)
         hops.linear(attn, w.o, y)
 
+    FUSED_ROWS = 512                   # steps of more rows split norms and input convolutions in two kernels
     EXPAND_BYTES = 1 << 30             # most memory the expanded keys and values of a step may take
 
     def _expanded_pages(self, m: LatentSpec, w: LatentWeights, si) -> int:
@@ -874,7 +876,8 @@ class HybridModel:
             nonlocal cur, nxt, entered, add
             if conv is not None:
                 fold = entered is not None or out is not None
-                hops.norm_conv_step(entered if entered is not None else cur[:, 0], nxt[:, 0] if fold else None, out, add, norm, conv, state, h, si)
+                hops.norm_conv_step(entered if entered is not None else cur[:, 0], nxt[:, 0] if fold else None, out, add, norm, conv, state, h, si,
+                                    self.factor if t > self.FUSED_ROWS else None)
                 entered = add = None
                 if fold:
                     cur, nxt = nxt, cur

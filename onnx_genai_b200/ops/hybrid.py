@@ -32,7 +32,7 @@ _native.register("ogb_hgrn2_state_rows", [I])
 _native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P, P, I, P, P])
 _native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, P, I, I, P])
 _native.register("ogb_norm_step", [P] * 10 + [F] + [I] * 8 + [L, I, P, P])
-_native.register("ogb_norm_conv_step", [P] * 12 + [F] + [I] * 8 + [L] + [P] * 5 + [I] * 4 + [P, P])
+_native.register("ogb_norm_conv_step", [P] * 13 + [F] + [I] * 9 + [L] + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_conv_rope_append", [P, I, P, P, P, I, P, I, P, P, P, L, L] + [I] * 8 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_conv_unit_gates", [P, I, P, P, I, P, I] + [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_delta_rule", [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, I, P, P])
@@ -432,9 +432,10 @@ def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
 
 
 @_timed("norm_conv_step")
-def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si):
+def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si, factor=None):
     """x_out [T, W] = x_in + y + add (y as for :func:`norm_step`, add [W] or None); h_t = sum_j conv[j] n_(t - taps + 1 + j) along every sequence
-    with n = norm(x_out), conv [taps, W] fp32, state [slots, taps - 1, W] advanced.  Where nothing is added x_out may be None."""
+    with n = norm(x_out), conv [taps, W] fp32, state [slots, taps - 1, W] advanced.  Where nothing is added x_out may be None.
+    ``factor`` [>= T] fp32 scratch: the pass runs as two kernels, which steps of many rows gain from."""
     t, w = x_in.shape
     if not x_in.is_cuda:
         new = reference.norm_step(x_in, y, None)
@@ -446,10 +447,11 @@ def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si):
         return h
     src, ptrs, (k, ldy, lds, ldg), y_rows = _sublayer(y)
     rc = _native.load().ogb_norm_conv_step(
-        x_in.data_ptr(), _ptr(x_out), *ptrs, _ptr(add), norm.w.data_ptr(), conv.data_ptr(), state.data_ptr(), h.data_ptr(), float(norm.eps), w, conv.shape[0], k,
+        x_in.data_ptr(), _ptr(x_out), *ptrs, _ptr(add), norm.w.data_ptr(), conv.data_ptr(), state.data_ptr(), h.data_ptr(), _ptr(factor), float(norm.eps), t, w,
+        conv.shape[0], k,
         x_in.stride(0), ldy, lds, ldg, h.stride(0), y_rows, *_rows_args(si, state), _ELEM[h.dtype], status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_norm_conv_step")
-    launch_counts["norm_conv_step"] += 1
+    launch_counts["norm_conv_step"] += 1 if factor is None else 2
     return h
 
 
