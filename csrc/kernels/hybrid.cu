@@ -588,8 +588,9 @@ static int launch_norm_conv(const NormConvParams& p, cudaStream_t s) {
 
 // ------------------------------------------------------------------------------------------------------
 // input_conv is the second half of that pass for steps of many rows: norm_step has left the residual and its rows' factors, and the
-// convolution is elementwise in the column.  A thread keeps V columns and walks a block's rows; slots as above.
+// convolution is elementwise in the column.  A thread loads V columns of a block's rows at once; slots as above.
 // ------------------------------------------------------------------------------------------------------
+constexpr int kIcRows = 8;                    // rows of a block (before them taps - 1 more are read)
 struct InputConvParams {
   const float* x;          // [rows, W]
   const float* factor;     // [rows]
@@ -604,7 +605,7 @@ struct InputConvParams {
 
 template <typename T, int V, int TM>
 __global__ void __launch_bounds__(128) input_conv_kernel(InputConvParams p) {
-  RowSpan<kNcRows> r;
+  RowSpan<kIcRows> r;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V, off = TM - p.taps;
   if (!r.set(p.sr, blockIdx.x, p.status) || c >= p.W) return;
   float conv[TM][V], w[V], h[TM > 1 ? TM - 1 : 1][V];        // filters aligned to their last tap; h: the last values, oldest first
@@ -631,47 +632,44 @@ __global__ void __launch_bounds__(128) input_conv_kernel(InputConvParams p) {
     if (t >= 0) normed(t, h[k]);
     else if (st != nullptr && r.start + t >= 0) load_vec<V>(st + static_cast<size_t>(k - off) * p.W, h[k]);
   }
+  float o[kIcRows][V];
+#pragma unroll
+  for (int b = 0; b < kIcRows; ++b) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) o[b][v] = 0.f;
+    if (r.j0 + b < r.j1) normed(r.j0 + b, o[b]);
+  }
   if (r.j0 == 0 && st != nullptr) {
 #pragma unroll
     for (int k = 0; k < TM - 1; ++k) {
       if (k < off) continue;
       const int t = r.n - (TM - 1) + k;
-      float o[V];
+      float last[V];
 #pragma unroll
       for (int q = 0; q < TM - 1; ++q)                       // fewer rows than taps: older values move up
 #pragma unroll
-        for (int v = 0; v < V; ++v) o[v] = (q == 0 || q == k + r.n) ? h[q][v] : o[v];
-      if (t >= 0) normed(t, o);
-      store_vec<V>(st + static_cast<size_t>(k - off) * p.W, o);
+        for (int v = 0; v < V; ++v) last[v] = (q == 0 || q == k + r.n) ? h[q][v] : last[v];
+      if (t >= 0) normed(t, last);
+      store_vec<V>(st + static_cast<size_t>(k - off) * p.W, last);
     }
   }
-  constexpr int NB = 4;
-  for (int j = r.j0; j < r.j1; j += NB) {
-    float o[NB][V];
 #pragma unroll
-    for (int b = 0; b < NB; ++b)
-      if (j + b < r.j1) normed(j + b, o[b]);
+  for (int b = 0; b < kIcRows; ++b) {
+    if (r.j0 + b >= r.j1) continue;
+    float u[V];
 #pragma unroll
-    for (int b = 0; b < NB; ++b) {
-      if (j + b >= r.j1) continue;
-      float u[V];
+    for (int v = 0; v < V; ++v) {
+      u[v] = conv[TM - 1][v] * o[b][v];
 #pragma unroll
-      for (int v = 0; v < V; ++v) {
-        u[v] = conv[TM - 1][v] * o[b][v];
-#pragma unroll
-        for (int k = 0; k < TM - 1; ++k) u[v] = fmaf(conv[k][v], h[k][v], u[v]);
-#pragma unroll
-        for (int k = 0; k + 1 < TM - 1; ++k) h[k][v] = h[k + 1][v];
-        h[TM > 1 ? TM - 2 : 0][v] = o[b][v];
-      }
-      store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r.base + j + b) * p.ldh + c, u);
+      for (int k = 0; k < TM - 1; ++k) u[v] = fmaf(conv[k][v], b + k < TM - 1 ? h[b + k < TM - 1 ? b + k : 0][v] : o[b + k < TM - 1 ? 0 : b + k - (TM - 1)][v], u[v]);
     }
+    store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r.base + r.j0 + b) * p.ldh + c, u);
   }
 }
 
 template <typename T, int V, int TM>
 static int launch_input_conv(const InputConvParams& p, cudaStream_t s) {
-  const dim3 grid(span_blocks<kNcRows>(p.sr), (p.W + 128 * V - 1) / (128 * V));
+  const dim3 grid(span_blocks<kIcRows>(p.sr), (p.W + 128 * V - 1) / (128 * V));
   input_conv_kernel<T, V, TM><<<grid, 128, 0, s>>>(p);
   return static_cast<int>(cudaGetLastError());
 }

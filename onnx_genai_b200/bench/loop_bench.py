@@ -112,6 +112,10 @@ def kernel_rows(size: str, timer, pk):
             t * heads * (d + rank) * 2 + wb * d)
         row("gemm per head (W_uv o)", phase, lambda: hops.linear_batched(oc.view(t, -1), uv, attn, heads, rank, dv), 2 * t * heads * dv * rank,
             t * heads * (dv + rank) * 2 + wb * dv)
+        uk1, qa1 = rnd(heads * rank, dv), empty(t, heads * rank)
+        row("like: gemm per head (W_uk^T q)", phase, lambda: hops.linear_batched(qp, uk1, qa1, heads, dv, rank), 2 * t * heads * dv * rank,
+            t * heads * (dv + rank) * 2 + wb * dv)
+        del uk1, qa1
         gate = qc[:, m.gate_col:m.gate_col + heads]
         pairs, keys = seen_pairs(parts, 0), sum(a + n for a, n in parts)
         qa1 = rnd(t * heads, rank)
