@@ -213,33 +213,6 @@ struct DbCfg {
   static constexpr int kSmemBytes = 4 * (2 * kDbTok * kPitch + 2 * kDbTok * kTP + 32 * 33 + 3 * kDbTok) + 8 * kDbTok;
 };
 
-// C += A B^T over K in steps of 8: A rows a + g, B rows b + g (K-major, row pitches pa, pb); the first nt tiles of eight B rows
-template <int KS, int NT>
-OGB_DEVICE void db_product(float (&c)[NT][4], const float* a, int pa, const float* b, int pb, int nt, int g, int tq) {
-  float e[NT][4] = {};
-#pragma unroll 2
-  for (int k = 0; k < KS; ++k) {
-    float hi[4], lo[4];
-#pragma unroll
-    for (int x = 0; x < 4; ++x) {
-      const float2 h = tf32_cut(a[(g + (x & 1) * 8) * pa + 8 * k + tq + (x >> 1) * 4]);
-      hi[x] = h.x; lo[x] = h.y;
-    }
-#pragma unroll
-    for (int n = 0; n < NT; ++n)
-      if (n < nt) {
-        const float2 b0 = tf32_cut(b[(8 * n + g) * pb + 8 * k + tq]), b1 = tf32_cut(b[(8 * n + g) * pb + 8 * k + tq + 4]);
-        mma_tf32(c[n], hi, b0.x, b1.x);
-        mma_tf32(e[n], lo, b0.x, b1.x);
-        mma_tf32(e[n], hi, b0.y, b1.y);
-      }
-  }
-#pragma unroll
-  for (int n = 0; n < NT; ++n)
-#pragma unroll
-    for (int x = 0; x < 4; ++x) c[n][x] += e[n][x];
-}
-
 template <typename T, int DP>
 __global__ void __launch_bounds__(256, 2) delta_prepare_kernel(DeltaParams p, DeltaBlocks bl) {
   using Cfg = DbCfg<DP>;
@@ -313,7 +286,7 @@ __global__ void __launch_bounds__(256, 2) delta_prepare_kernel(DeltaParams p, De
       const int n_tiles = min(4, 2 * m + 2 - n0);
       float c[4][4] = {};
       if (n_tiles > 0)
-        db_product<DP / 8, 4>(c, (isq ? sq : sk) + 16 * m * Cfg::kPitch, Cfg::kPitch, sk + 8 * n0 * Cfg::kPitch, Cfg::kPitch, n_tiles, g, tq);
+        split_product<DP / 8, 4>(c, (isq ? sq : sk) + 16 * m * Cfg::kPitch, Cfg::kPitch, sk + 8 * n0 * Cfg::kPitch, Cfg::kPitch, n_tiles, g, tq);
 #pragma unroll
       for (int n = 0; n < 4; ++n)
 #pragma unroll

@@ -198,7 +198,7 @@ static int dispatch_hyper(const HyperParams& p, cudaStream_t stream) {
 // ------------------------------------------------------------------------------------------------------
 // What a sublayer left for the residual: a row per token, or -- behind routed experts -- the weighted sum of the token's expert rows
 // (sum_j weight[t][j] y[pos[t][j]]) and of a shared expert's row times the sigmoid of its gate, taken here so that it never
-// exists in memory.
+// exists in memory.  With res_gate the output reaches the residual as (output + y_bias) sigmoid(res_gate + res_bias).
 // ------------------------------------------------------------------------------------------------------
 struct SublayerOut {
   const void* y;           // [rows, ldy], or the expert rows; null: nothing
@@ -206,7 +206,10 @@ struct SublayerOut {
   const float* weight;     // [rows, k]
   const void* shared;      // [rows, lds] or null
   const float* gate;       // [rows, ldg]: logits
-  int k, ldy, lds, ldg;
+  const float* y_bias;     // [W] or null
+  const void* res_gate;    // [rows, ldr] or null
+  const float* res_bias;   // [W]
+  int k, ldy, lds, ldg, ldr;
   int64_t y_rows;
 };
 
@@ -233,10 +236,32 @@ OGB_DEVICE void sublayer_rows(const SublayerOut& o, int t0, int n, int W, float 
       }
     }
   };
+  auto gate = [&]() {
+    if (o.res_gate == nullptr) return;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c >= W) continue;
+      float bias[V], yb[V];
+      load_vec<V>(o.res_bias + c, bias);
+#pragma unroll
+      for (int v = 0; v < V; ++v) yb[v] = 0.f;
+      if (o.y_bias != nullptr) load_vec<V>(o.y_bias + c, yb);
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        if (b >= n) continue;
+        float z[V];
+        load_vec<V>(static_cast<const T*>(o.res_gate) + static_cast<size_t>(t0 + b) * o.ldr + c, z);
+#pragma unroll
+        for (int v = 0; v < V; ++v) y[b][i][v] = (y[b][i][v] + yb[v]) / (1.f + expf(-(z[v] + bias[v])));
+      }
+    }
+  };
   if (o.pos == nullptr) {
 #pragma unroll
     for (int b = 0; b < NB; ++b)
       if (b < n) add(o.y, t0 + b, o.ldy, 1.f, y[b]);
+    gate();
     return;
   }
   for (int j = 0; j < o.k; ++j) {
@@ -252,10 +277,12 @@ OGB_DEVICE void sublayer_rows(const SublayerOut& o, int t0, int n, int W, float 
       add(o.y, row, o.ldy, o.weight[at], y[b]);
     }
   }
-  if (o.shared == nullptr) return;
+  if (o.shared != nullptr) {
 #pragma unroll
-  for (int b = 0; b < NB; ++b)
-    if (b < n) add(o.shared, t0 + b, o.lds, 1.f / (1.f + expf(-o.gate[static_cast<size_t>(t0 + b) * o.ldg])), y[b]);
+    for (int b = 0; b < NB; ++b)
+      if (b < n) add(o.shared, t0 + b, o.lds, 1.f / (1.f + expf(-o.gate[static_cast<size_t>(t0 + b) * o.ldg])), y[b]);
+  }
+  gate();
 }
 
 // sums over the block of NB values a thread; `red` [2][NB][32] alternates with `parity`, so one barrier a call is enough
@@ -272,13 +299,41 @@ OGB_DEVICE void block_sums(float (&v)[NB], float (&red)[2][NB][32], int parity) 
   for (int b = 0; b < NB; ++b) v[b] = warp_sum(lane < warps ? red[parity][b][lane] : 0.f);
 }
 
+// 1 / root mean square of every one of `groups` equal parts of a row of W columns, V of which a thread holds at (i * blockDim.x +
+// threadIdx.x) * V: `part` [W / V] and `inv` [groups] are shared memory, in which the thread finds the factors of its columns
+// (group_of) after the call.  A part is a multiple of V.
+template <int N, int V>
+OGB_DEVICE void group_factors(const float (&x)[N][V], int W, int groups, float eps, float* part, float* inv) {
+  const int units = W / V, per = units / groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  __syncthreads();                             // the arrays may still be read from the call before
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int u = i * blockDim.x + threadIdx.x;
+    float ss = 0.f;
+#pragma unroll
+    for (int v = 0; v < V; ++v) ss = fmaf(x[i][v], x[i][v], ss);
+    if (u < units) part[u] = ss;
+  }
+  __syncthreads();
+  for (int g = warp; g < groups; g += warps) {
+    float a = 0.f;
+    for (int u = lane; u < per; u += 32) a += part[g * per + u];
+    a = warp_sum(a);
+    if (lane == 0) inv[g] = 1.f / sqrtf(a / static_cast<float>(per * V) + eps);
+  }
+  __syncthreads();
+}
+// shared memory of group_factors: part and inv of `rows` rows
+inline size_t group_bytes(int W, int V, int groups, int rows) { return groups > 1 ? static_cast<size_t>(rows) * (W / V + groups) * sizeof(float) : 0; }
+
 // ------------------------------------------------------------------------------------------------------
 // norm_step is the pass between two products for designs with one residual stream:
 //
 //   x <- x + rms(y) post        h = rms(x) w
 //
 // Without `post` the output is added as it is, without `w` h is the residual itself.  The residual may come from elsewhere (x_in), and a
-// vector may be added to it.  One block per row, the row in registers; all fp32.
+// vector may be added to it.  `groups` > 1: that many equal parts of x have a root mean square each.  One block per row, the row in
+// registers; all fp32.
 // ------------------------------------------------------------------------------------------------------
 struct NormStepParams {
   const float* x_in;       // [rows, ldx]
@@ -287,16 +342,17 @@ struct NormStepParams {
   const float* add;        // [W] or null
   const float *post, *w;   // norm weights or null
   void* h;                 // [rows, ldh] or null
-  float* factor;           // [rows] or null: gets 1 / root mean square of x
+  float* factor;           // [rows, groups] or null: gets 1 / root mean square of x
   const int* gather;       // row r of h comes from row gather[r]; x is then left alone
   float eps;
-  int rows, total_rows, W, ldx, ldh;
+  int rows, total_rows, W, groups, ldx, ldh;
   int* status;
 };
 
 template <typename T, int V, int N>
 __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
   __shared__ float red[2][1][32];
+  extern __shared__ float ns_groups[];         // groups > 1: [W / V] sums, [groups] factors
   const int r = blockIdx.x;
   int t = r;
   if (p.gather != nullptr) {
@@ -350,7 +406,12 @@ __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
   }
   if (p.h == nullptr && p.factor == nullptr) return;
   float inv[1] = {0.f};
-  if (p.w != nullptr || p.factor != nullptr) {
+  float* ginv = ns_groups + p.W / V;
+  if (p.groups > 1 && (p.w != nullptr || p.factor != nullptr)) {
+    group_factors<N, V>(x, p.W, p.groups, p.eps, ns_groups, ginv);
+    if (p.factor != nullptr)
+      for (int g = threadIdx.x; g < p.groups; g += blockDim.x) p.factor[static_cast<size_t>(r) * p.groups + g] = ginv[g];
+  } else if (p.w != nullptr || p.factor != nullptr) {
 #pragma unroll
     for (int i = 0; i < N; ++i)
 #pragma unroll
@@ -367,8 +428,9 @@ __global__ void __launch_bounds__(1024) norm_step_kernel(NormStepParams p) {
       if (p.w != nullptr) {
         float g[V];
         load_vec<V>(p.w + c, g);
+        const float f = p.groups > 1 ? ginv[c / (p.W / p.groups)] : inv[0];
 #pragma unroll
-        for (int v = 0; v < V; ++v) x[i][v] *= inv[0] * g[v];
+        for (int v = 0; v < V; ++v) x[i][v] *= f * g[v];
       }
       store_vec<V>(static_cast<T*>(p.h) + static_cast<size_t>(r) * p.ldh + c, x[i]);
     }
@@ -380,10 +442,12 @@ static int launch_norm_step(const NormStepParams& p, cudaStream_t s) {
   const int units = (p.W + V - 1) / V;
   const int threads = units >= 4096 ? 1024 : units >= 256 ? 256 : (units + 31) / 32 * 32;
   const int n = (units + threads - 1) / threads;
-  if (n <= 1) norm_step_kernel<T, V, 1><<<p.rows, threads, 0, s>>>(p);
-  else if (n <= 2) norm_step_kernel<T, V, 2><<<p.rows, threads, 0, s>>>(p);
-  else if (n <= 4) norm_step_kernel<T, V, 4><<<p.rows, threads, 0, s>>>(p);
-  else if (n <= 16) norm_step_kernel<T, V, 16><<<p.rows, threads, 0, s>>>(p);
+  const size_t smem = group_bytes(p.W, V, p.groups, 1);
+  if (smem > 40 * 1024) return -2;
+  if (n <= 1) norm_step_kernel<T, V, 1><<<p.rows, threads, smem, s>>>(p);
+  else if (n <= 2) norm_step_kernel<T, V, 2><<<p.rows, threads, smem, s>>>(p);
+  else if (n <= 4) norm_step_kernel<T, V, 4><<<p.rows, threads, smem, s>>>(p);
+  else if (n <= 16) norm_step_kernel<T, V, 16><<<p.rows, threads, smem, s>>>(p);
   else return -2;
   return static_cast<int>(cudaGetLastError());
 }
@@ -409,8 +473,9 @@ struct NormConvParams {
   const float* conv;       // [taps, W]
   float* state;            // [slots, taps - 1, W]
   void* h;                 // [rows, ldh]
+  void* plain;             // [rows, ldp] or null: gets the normed rows
   float eps;
-  int W, ldx, ldh, taps;
+  int W, groups, ldx, ldh, ldp, taps;
   StepRows sr;
   int* status;
 };
@@ -418,6 +483,7 @@ struct NormConvParams {
 template <typename T, int V, int N, int NB, int TM>
 __global__ void __launch_bounds__(512) norm_conv_kernel(NormConvParams p) {
   __shared__ float red[2][NB][32];
+  extern __shared__ float nc_groups[];         // groups > 1: [NB][W / V] sums, [NB][groups] factors
   RowSpan<kNcRows> r;
   if (!r.set(p.sr, blockIdx.x, p.status)) return;
   const int base = r.base, n = r.n, j0 = r.j0, j1 = r.j1, start = r.start, slot = r.slot;
@@ -469,15 +535,55 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(NormConvParams p) {
         if (write && p.x_out != nullptr && b < m && c < p.W) store_vec<V>(p.x_out + static_cast<size_t>(base + j + b) * p.W + c, x[b][i]);
       }
     }
-    block_sums<NB>(ss, red, parity);
-    parity ^= 1;
+    if (p.groups > 1) {
+      const int units = p.W / V, per = units / p.groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+      float* ginv = nc_groups + NB * units;
+      __syncthreads();
 #pragma unroll
-    for (int b = 0; b < NB; ++b) {
-      const float inv = 1.f / sqrtf(ss[b] / static_cast<float>(p.W) + p.eps);
+      for (int b = 0; b < NB; ++b)
 #pragma unroll
-      for (int i = 0; i < N; ++i)
+        for (int i = 0; i < N; ++i) {
+          const int u = i * blockDim.x + threadIdx.x;
+          float a = 0.f;
 #pragma unroll
-        for (int v = 0; v < V; ++v) o[b][i][v] = x[b][i][v] * (inv * w[i][v]);
+          for (int v = 0; v < V; ++v) a = fmaf(x[b][i][v], x[b][i][v], a);
+          if (u < units) nc_groups[b * units + u] = a;
+        }
+      __syncthreads();
+      for (int g = warp; g < NB * p.groups; g += warps) {       // groups of the NB rows one after the other
+        float a = 0.f;
+        for (int u = lane; u < per; u += 32) a += nc_groups[(g / p.groups) * units + (g % p.groups) * per + u];
+        a = warp_sum(a);
+        if (lane == 0) ginv[g] = 1.f / sqrtf(a / static_cast<float>(per * V) + p.eps);
+      }
+      __syncthreads();
+#pragma unroll
+      for (int b = 0; b < NB; ++b)
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          const int c = col0 + i * step;
+          const float f = c < p.W ? ginv[b * p.groups + c / (p.W / p.groups)] : 0.f;
+#pragma unroll
+          for (int v = 0; v < V; ++v) o[b][i][v] = x[b][i][v] * (f * w[i][v]);
+        }
+    } else {
+      block_sums<NB>(ss, red, parity);
+      parity ^= 1;
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        const float inv = 1.f / sqrtf(ss[b] / static_cast<float>(p.W) + p.eps);
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+#pragma unroll
+          for (int v = 0; v < V; ++v) o[b][i][v] = x[b][i][v] * (inv * w[i][v]);
+      }
+    }
+    if (write && p.plain != nullptr) {
+#pragma unroll
+      for (int b = 0; b < NB; ++b)
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+          if (b < m && col0 + i * step < p.W) store_vec<V>(static_cast<T*>(p.plain) + static_cast<size_t>(base + j + b) * p.ldp + col0 + i * step, o[b][i]);
     }
   };
   auto shift_in = [&](const float (&o)[N][V]) {
@@ -579,10 +685,11 @@ static int launch_norm_conv(const NormConvParams& p, cudaStream_t s) {
   const int n = units <= 256 ? 1 : units <= 1024 ? 2 : units <= 2048 ? 4 : 8;
   const int threads = ((units + n - 1) / n + 31) / 32 * 32;
   if (threads > 512 || n * V > 16) return -2;
-  if (n == 1) norm_conv_kernel<T, V, 1, 4, TM><<<blocks, threads, 0, s>>>(p);
-  else if (n == 2) norm_conv_kernel<T, V, 2, V == 1 ? 4 : 2, TM><<<blocks, threads, 0, s>>>(p);
-  else if (n == 4) norm_conv_kernel<T, V, 4, V == 1 ? 4 : 1, TM><<<blocks, threads, 0, s>>>(p);
-  else if constexpr (V == 1) norm_conv_kernel<T, V, 8, 2, TM><<<blocks, threads, 0, s>>>(p);
+  auto smem = [&](int nb) { return group_bytes(p.W, V, p.groups, nb); };
+  if (n == 1) norm_conv_kernel<T, V, 1, 4, TM><<<blocks, threads, smem(4), s>>>(p);
+  else if (n == 2) norm_conv_kernel<T, V, 2, V == 1 ? 4 : 2, TM><<<blocks, threads, smem(V == 1 ? 4 : 2), s>>>(p);
+  else if (n == 4) norm_conv_kernel<T, V, 4, V == 1 ? 4 : 1, TM><<<blocks, threads, smem(V == 1 ? 4 : 1), s>>>(p);
+  else if constexpr (V == 1) norm_conv_kernel<T, V, 8, 2, TM><<<blocks, threads, smem(2), s>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -593,12 +700,13 @@ static int launch_norm_conv(const NormConvParams& p, cudaStream_t s) {
 constexpr int kIcRows = 8;                    // rows of a block (before them taps - 1 more are read)
 struct InputConvParams {
   const float* x;          // [rows, W]
-  const float* factor;     // [rows]
+  const float* factor;     // [rows, groups]
   const float* w;          // [W]
   const float* conv;       // [taps, W]
   float* state;            // [slots, taps - 1, W]
   void* h;                 // [rows, ldh]
-  int W, ldh, taps;
+  void* plain;             // [rows, ldp] or null: gets the normed rows
+  int W, groups, ldh, ldp, taps;
   StepRows sr;
   int* status;
 };
@@ -616,9 +724,10 @@ __global__ void __launch_bounds__(128) input_conv_kernel(InputConvParams p) {
     for (int v = 0; v < V; ++v) conv[k][v] = 0.f;
     if (k >= off) load_vec<V>(p.conv + static_cast<size_t>(k - off) * p.W + c, conv[k]);
   }
+  const int group = p.groups > 1 ? c / (p.W / p.groups) : 0;
   auto normed = [&](int t, float (&o)[V]) {
     load_vec<V>(p.x + static_cast<size_t>(r.base + t) * p.W + c, o);
-    const float f = p.factor[r.base + t];
+    const float f = p.factor[static_cast<size_t>(r.base + t) * p.groups + group];
 #pragma unroll
     for (int v = 0; v < V; ++v) o[v] *= f * w[v];
   };
@@ -638,6 +747,11 @@ __global__ void __launch_bounds__(128) input_conv_kernel(InputConvParams p) {
 #pragma unroll
     for (int v = 0; v < V; ++v) o[b][v] = 0.f;
     if (r.j0 + b < r.j1) normed(r.j0 + b, o[b]);
+  }
+  if (p.plain != nullptr) {
+#pragma unroll
+    for (int b = 0; b < kIcRows; ++b)
+      if (r.j0 + b < r.j1) store_vec<V>(static_cast<T*>(p.plain) + static_cast<size_t>(r.base + r.j0 + b) * p.ldp + c, o[b]);
   }
   if (r.j0 == 0 && st != nullptr) {
 #pragma unroll
@@ -675,12 +789,12 @@ static int launch_input_conv(const InputConvParams& p, cudaStream_t s) {
 }
 
 // ------------------------------------------------------------------------------------------------------
-// all streams of a row start as the token's embedding, normed where `w` is given; `copy` gets it too (read again by later layers)
+// all streams of a row start as the token's embedding times `scale`, normed where `w` is given; `copy` gets it too (read again by later layers)
 // ------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256) embed_streams_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
-                                                            int S, int W, int vocab, const float* __restrict__ w, float eps, T* __restrict__ copy,
-                                                            int ldc, int* status) {
+                                                            int S, int W, int vocab, const float* __restrict__ w, float eps, float scale,
+                                                            T* __restrict__ copy, int ldc, int* status) {
   __shared__ float red[2][1][32];
   const int t = blockIdx.x;
   int id = ids[t];
@@ -692,12 +806,15 @@ __global__ void __launch_bounds__(256) embed_streams_kernel(const int* __restric
   float* dst = x + static_cast<size_t>(t) * S * W;
   float inv[1] = {0.f};
   if (w != nullptr) {
-    for (int c = threadIdx.x; c < W; c += blockDim.x) inv[0] = fmaf(to_f32<T>(src[c]), to_f32<T>(src[c]), inv[0]);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      const float v = to_f32<T>(src[c]) * scale;
+      inv[0] = fmaf(v, v, inv[0]);
+    }
     block_sums<1>(inv, red, 0);
     inv[0] = 1.f / sqrtf(inv[0] / static_cast<float>(W) + eps);
   }
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
-    float v = to_f32<T>(src[c]);
+    float v = to_f32<T>(src[c]) * scale;
     if (w != nullptr) v *= inv[0] * w[c];
     for (int s = 0; s < S; ++s) dst[static_cast<size_t>(s) * W + c] = v;
     if (copy != nullptr) copy[static_cast<size_t>(t) * ldc + c] = from_f32<T>(v);
@@ -782,20 +899,23 @@ __global__ void __launch_bounds__(128) latent_rope_append_kernel(LatentAppendPar
 }
 
 // ------------------------------------------------------------------------------------------------------
-// RMS norm of every group of `n` columns (a head) with one shared weight, times silu of a gate of the same layout where there is
-// one: fp32 in, activation type out; one warp per group
+// RMS norm of every group of `n` columns (a head) with a weight (null: none; head h's begins at h * wstep: 0 is one for all), times silu
+// or sigmoid of a gate of the same layout where there is one: fp32 in, activation type out; one warp per group
 // ------------------------------------------------------------------------------------------------------
 OGB_DEVICE float silu_f32(float z) { return z / (1.f + expf(-z)); }
+OGB_DEVICE float gate_f32(float z, bool sigmoid) { return sigmoid ? 1.f / (1.f + expf(-z)) : silu_f32(z); }
 
 template <typename T>
-__global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, T* __restrict__ out,
-                                                           int rows, int heads, int n, int ldx, int ldo, const T* __restrict__ gate, int ldg, bool vec) {
+__global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, int wstep, float eps,
+                                                           T* __restrict__ out, int rows, int heads, int n, int ldx, int ldo, const T* __restrict__ gate,
+                                                           int ldg, bool sigmoid, bool vec) {
   const int lane = threadIdx.x & 31;
   const long long g = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   if (g >= static_cast<long long>(rows) * heads) return;
   const int t = static_cast<int>(g / heads), h = static_cast<int>(g % heads);
   const float* src = x + static_cast<size_t>(t) * ldx + static_cast<size_t>(h) * n;
   T* dst = out + static_cast<size_t>(t) * ldo + static_cast<size_t>(h) * n;
+  if (w != nullptr) w += static_cast<size_t>(h) * wstep;
   const T* gt = gate != nullptr ? gate + static_cast<size_t>(t) * ldg + static_cast<size_t>(h) * n : nullptr;
   float ss = 0.f;
   if (vec) {                                   // rows and heads of x, out and gate start on four elements; n is 128 .. 512 in steps of 128
@@ -812,14 +932,14 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restri
 #pragma unroll
     for (int k = 0; k < 4; ++k)
       if (k < per) {
-        float wv[4];
-        load_vec<4>(w + k * 128 + lane * 4, wv);
+        float wv[4] = {1.f, 1.f, 1.f, 1.f};
+        if (w != nullptr) load_vec<4>(w + k * 128 + lane * 4, wv);
 #pragma unroll
         for (int i = 0; i < 4; ++i) v[k][i] *= inv * wv[i];
         if (gt != nullptr) {
           load_vec<4>(gt + k * 128 + lane * 4, wv);
 #pragma unroll
-          for (int i = 0; i < 4; ++i) v[k][i] *= silu_f32(wv[i]);
+          for (int i = 0; i < 4; ++i) v[k][i] *= gate_f32(wv[i], sigmoid);
         }
         store_vec<4>(dst + k * 128 + lane * 4, v[k]);
       }
@@ -827,7 +947,7 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(const float* __restri
   }
   for (int i = lane; i < n; i += 32) ss = fmaf(src[i], src[i], ss);
   const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
-  for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(src[i] * inv * w[i] * (gt != nullptr ? silu_f32(to_f32<T>(gt[i])) : 1.f));
+  for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(src[i] * inv * (w != nullptr ? w[i] : 1.f) * (gt != nullptr ? gate_f32(to_f32<T>(gt[i]), sigmoid) : 1.f));
 }
 
 // ------------------------------------------------------------------------------------------------------
@@ -937,21 +1057,28 @@ extern "C" int ogb_hyper_step(const float* x_in, float* x_out, const void* y, co
 // pos / weight (null: y has one row per token): y holds y_rows expert rows, of which token t sums k; shared / gate: a row of every
 // token, times the sigmoid of its gate.
 static bool sublayer_ok(const SublayerOut& o) {
-  return (o.pos == nullptr || (o.weight != nullptr && o.k >= 1)) && (o.shared == nullptr || (o.pos != nullptr && o.gate != nullptr));
+  return (o.pos == nullptr || (o.weight != nullptr && o.k >= 1)) && (o.shared == nullptr || (o.pos != nullptr && o.gate != nullptr)) &&
+         (o.res_gate != nullptr ? o.y != nullptr && o.res_bias != nullptr : o.y_bias == nullptr);
+}
+// four elements at a time need rows that start on them, and pointers too
+static bool sublayer_vec(const SublayerOut& o, int elem) {
+  const uintptr_t act = reinterpret_cast<uintptr_t>(o.y) | reinterpret_cast<uintptr_t>(o.shared) | reinterpret_cast<uintptr_t>(o.res_gate);
+  const uintptr_t f32 = reinterpret_cast<uintptr_t>(o.y_bias) | reinterpret_cast<uintptr_t>(o.res_bias);
+  return ((o.ldy | o.lds | o.ldr) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
 }
 
-// post null: y as it is; w null: h is the residual; h null: no read-out.
-extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const void* shared, const float* gate, const float* post,
-                             const float* w, void* h, const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int lds, int ldg,
-                             int ldh, int64_t y_rows, int elem, int* status, void* stream) {
+// post null: y as it is; w null: h is the residual; h null: no read-out.  A gathered row's gate is the one of the row it comes from.
+extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const void* shared, const float* gate, const float* y_bias,
+                             const void* res_gate, const float* res_bias, const float* post, const float* w, void* h, const int* gather, float eps, int rows,
+                             int total_rows, int W, int groups, int k, int ldy, int lds, int ldg, int ldr, int ldh, int64_t y_rows, int elem, int* status,
+                             void* stream) {
   if (rows <= 0) return 0;
-  NormStepParams p{x, x, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, nullptr, post, w, h, nullptr, gather, eps, rows, total_rows,
-                   W, W, ldh, status};
-  if (W < 1 || !sublayer_ok(p.out)) return -3;
-  // four elements at a time need rows that start on them, and pointers too
-  const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared);
+  NormStepParams p{x, x, SublayerOut{y, pos, weight, shared, gate, y_bias, res_gate, res_bias, k, ldy, lds, ldg, ldr, y_rows}, nullptr, post, w, h, nullptr,
+                   gather, eps, rows, total_rows, W, groups, W, ldh, status};
+  if (W < 1 || groups < 1 || W % groups != 0 || !sublayer_ok(p.out)) return -3;
   const uintptr_t f32 = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(post) | reinterpret_cast<uintptr_t>(w);
-  const bool vec = ((W | ldy | ldh | lds) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
+  const bool vec = ((W | ldh) & 3) == 0 && (groups == 1 || (W / groups & 3) == 0) && (f32 & 15) == 0 &&
+                   (reinterpret_cast<uintptr_t>(h) & (elem == kElemBF16 ? 7 : 15)) == 0 && sublayer_vec(p.out, elem);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (elem == kElemBF16) return vec ? launch_norm_step<__nv_bfloat16, 4>(p, s) : launch_norm_step<__nv_bfloat16, 1>(p, s);
   if (elem == kElemF32) return vec ? launch_norm_step<float, 4>(p, s) : launch_norm_step<float, 1>(p, s);
@@ -959,49 +1086,54 @@ extern "C" int ogb_norm_step(float* x, const void* y, const int* pos, const floa
 }
 
 // x_out null: nothing is added (y and add null).  At most 8 taps.  factor null: one kernel, for few rows (of up to 8192 columns, 4096
-// where they do not start on four elements); else [rows] of scratch, norm_step and input_conv.
+// where they do not start on four elements); else [rows, groups] of scratch, norm_step and input_conv.
 template <typename T>
 static int norm_conv(const NormConvParams& p, float* factor, int rows, bool vec, cudaStream_t s) {
   if (factor == nullptr)
     return vec ? (p.taps <= 4 ? launch_norm_conv<T, 4, 4>(p, s) : launch_norm_conv<T, 4, 8>(p, s))
                : (p.taps <= 4 ? launch_norm_conv<T, 1, 4>(p, s) : launch_norm_conv<T, 1, 8>(p, s));
-  const NormStepParams n{p.x_in, p.x_out, p.out, p.add, nullptr, nullptr, nullptr, factor, nullptr, p.eps, rows, rows, p.W, p.ldx, 0, p.status};
+  const NormStepParams n{p.x_in, p.x_out, p.out, p.add, nullptr, nullptr, nullptr, factor, nullptr, p.eps, rows, rows, p.W, p.groups, p.ldx, 0, p.status};
   const int rc = vec ? launch_norm_step<T, 4>(n, s) : launch_norm_step<T, 1>(n, s);
   if (rc != 0) return rc;
-  const InputConvParams q{p.x_out != nullptr ? p.x_out : p.x_in, factor, p.w, p.conv, p.state, p.h, p.W, p.ldh, p.taps, p.sr, p.status};
+  const InputConvParams q{p.x_out != nullptr ? p.x_out : p.x_in, factor, p.w, p.conv, p.state, p.h, p.plain, p.W, p.groups, p.ldh, p.ldp, p.taps, p.sr,
+                         p.status};
   return vec ? (p.taps <= 4 ? launch_input_conv<T, 4, 4>(q, s) : launch_input_conv<T, 4, 8>(q, s))
              : (p.taps <= 4 ? launch_input_conv<T, 1, 4>(q, s) : launch_input_conv<T, 1, 8>(q, s));
 }
 
 extern "C" int ogb_norm_conv_step(const float* x_in, float* x_out, const void* y, const int* pos, const float* weight, const void* shared,
-                                  const float* gate, const float* add, const float* w, const float* conv, float* state, void* h, float* factor,
-                                  float eps, int rows, int W, int taps, int k, int ldx, int ldy, int lds, int ldg, int ldh, int64_t y_rows,
+                                  const float* gate, const float* y_bias, const void* res_gate, const float* res_bias, const float* add, const float* w,
+                                  const float* conv, float* state, void* h, void* plain, float* factor, float eps, int rows, int W, int groups, int taps,
+                                  int k, int ldx, int ldy, int lds, int ldg, int ldr, int ldh, int ldp, int64_t y_rows,
                                   const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode,
                                   int num_tiles, int num_slots, int elem, int* status, void* stream) {
   if (num_decode + num_tiles <= 0) return 0;
-  NormConvParams p{x_in, x_out, SublayerOut{y, pos, weight, shared, gate, k, ldy, lds, ldg, y_rows}, add, w, conv, state, h, eps, W, ldx, ldh, taps,
+  NormConvParams p{x_in, x_out, SublayerOut{y, pos, weight, shared, gate, y_bias, res_gate, res_bias, k, ldy, lds, ldg, ldr, y_rows}, add, w, conv, state,
+                   h, plain, eps, W, groups, ldx, ldh, ldp, taps,
                    StepRows{ctx_len, state_slot, cu_q, tile_seq, tile_q0, num_decode, num_tiles, num_slots}, status};
+  if (groups < 1 || W % groups != 0) return -3;
   if (W < 1 || taps < 1 || taps > 8 || x_in == x_out || !sublayer_ok(p.out) || w == nullptr || conv == nullptr || h == nullptr) return -3;
   if ((taps > 1 && state == nullptr) || ((y != nullptr || add != nullptr) && x_out == nullptr) || (x_out == nullptr && ldx != W)) return -3;
-  const uintptr_t act = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(shared);
+  const uintptr_t act = reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(plain);
   const uintptr_t f32 = reinterpret_cast<uintptr_t>(x_in) | reinterpret_cast<uintptr_t>(x_out) | reinterpret_cast<uintptr_t>(add) |
                         reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(conv) | reinterpret_cast<uintptr_t>(state);
-  const bool vec = ((W | ldx | ldy | ldh | lds) & 3) == 0 && (f32 & 15) == 0 && (act & (elem == kElemBF16 ? 7 : 15)) == 0;
+  const bool vec = ((W | ldx | ldh | ldp) & 3) == 0 && (groups == 1 || (W / groups & 3) == 0) && (f32 & 15) == 0 &&
+                   (act & (elem == kElemBF16 ? 7 : 15)) == 0 && sublayer_vec(p.out, elem);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (elem == kElemBF16) return norm_conv<__nv_bfloat16>(p, factor, rows, vec, s);
   if (elem == kElemF32) return norm_conv<float>(p, factor, rows, vec, s);
   return -3;
 }
 
-extern "C" int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, const float* w, float eps, void* copy,
-                                 int ldc, int elem, int* status, void* stream) {
+extern "C" int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, const float* w, float eps, float scale,
+                                 void* copy, int ldc, int elem, int* status, void* stream) {
   if (tokens <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (elem == kElemBF16)
-    embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const __nv_bfloat16*>(table), x, S, W, vocab, w, eps, static_cast<__nv_bfloat16*>(copy),
-                                                ldc, status);
+    embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const __nv_bfloat16*>(table), x, S, W, vocab, w, eps, scale,
+                                                static_cast<__nv_bfloat16*>(copy), ldc, status);
   else if (elem == kElemF32)
-    embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const float*>(table), x, S, W, vocab, w, eps, static_cast<float*>(copy), ldc, status);
+    embed_streams_kernel<<<tokens, 256, 0, s>>>(ids, static_cast<const float*>(table), x, S, W, vocab, w, eps, scale, static_cast<float*>(copy), ldc, status);
   else return -3;
   return static_cast<int>(cudaGetLastError());
 }
@@ -1028,19 +1160,20 @@ extern "C" int ogb_latent_append(void* row, int ldr, int latent, const float* w,
   return -3;
 }
 
-extern "C" int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate,
-                                int ldg, int elem, void* stream) {
+extern "C" int ogb_head_rmsnorm(const float* x, const float* w, int wstep, float eps, void* out, int rows, int heads, int n, int ldx, int ldo,
+                                const void* gate, int ldg, int sigmoid, int elem, void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * heads + 7) / 8);
   const uintptr_t unaligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) |
                               ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(gate)) & (elem == kElemBF16 ? 7 : 15));
-  const bool vec = (n & 127) == 0 && n <= 512 && ((ldx | ldo | ldg) & 3) == 0 && unaligned == 0;
+  const bool vec = (n & 127) == 0 && n <= 512 && ((ldx | ldo | ldg | wstep) & 3) == 0 && unaligned == 0;
   if (elem == kElemBF16)
-    head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo,
-                                               static_cast<const __nv_bfloat16*>(gate), ldg, vec);
+    head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, wstep, eps, static_cast<__nv_bfloat16*>(out), rows, heads, n, ldx, ldo,
+                                               static_cast<const __nv_bfloat16*>(gate), ldg, sigmoid != 0, vec);
   else if (elem == kElemF32)
-    head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo, static_cast<const float*>(gate), ldg, vec);
+    head_rmsnorm_kernel<<<blocks, 256, 0, s>>>(x, w, wstep, eps, static_cast<float*>(out), rows, heads, n, ldx, ldo, static_cast<const float*>(gate), ldg,
+                                               sigmoid != 0, vec);
   else return -3;
   return static_cast<int>(cudaGetLastError());
 }

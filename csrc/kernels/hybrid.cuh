@@ -141,4 +141,32 @@ OGB_DEVICE void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1)
         "r"(__float_as_uint(b1)));
 }
 
+// C += A B^T over K in steps of 8, fp32 factors split in two tf32 terms (about 20 bits): A rows a + g, B rows b + g (K-major, row pitches
+// pa, pb); the first nt tiles of eight B rows
+template <int KS, int NT>
+OGB_DEVICE void split_product(float (&c)[NT][4], const float* a, int pa, const float* b, int pb, int nt, int g, int tq) {
+  float e[NT][4] = {};
+#pragma unroll 2
+  for (int k = 0; k < KS; ++k) {
+    float hi[4], lo[4];
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const float2 h = tf32_cut(a[(g + (x & 1) * 8) * pa + 8 * k + tq + (x >> 1) * 4]);
+      hi[x] = h.x; lo[x] = h.y;
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+      if (n < nt) {
+        const float2 b0 = tf32_cut(b[(8 * n + g) * pb + 8 * k + tq]), b1 = tf32_cut(b[(8 * n + g) * pb + 8 * k + tq + 4]);
+        mma_tf32(c[n], hi, b0.x, b1.x);
+        mma_tf32(e[n], lo, b0.x, b1.x);
+        mma_tf32(e[n], hi, b0.y, b1.y);
+      }
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int x = 0; x < 4; ++x) c[n][x] += e[n][x];
+}
+
 }  // namespace ogb

@@ -19,13 +19,15 @@ namespace ogb {
 
 constexpr int kMaxExperts = 256;
 
-// `bias` (fp32, or null) is added to the logits.  The choice compares logits, which order experts as their scores do.  `groups` > 1:
-// experts form that many equal groups of neighbours, a group scores as its best expert, and only the `keep` best groups can be
-// chosen from.
+// Softmax scores: `bias` (fp32, or null) is added to the logits, and the choice compares logits, which order experts as their scores do.
+// Sigmoid scores: the choice compares scores plus `bias`, the weights are the scores (over their sum + 1e-20 when renormalised).
+// `groups` > 1: experts form that many equal groups of neighbours, a group scores as its best expert (`group_best` 2: as the sum of its
+// best two), and only the `keep` best groups can be chosen from.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ topk_ids,
                                                              float* __restrict__ topk_w,
-                                                             int tokens, int experts, int k, int renormalize, int ld, int groups, int keep) {
+                                                             int tokens, int experts, int k, int renormalize, int ld, int groups, int keep, bool sigmoid,
+                                                             int group_best) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   __shared__ float s_group[8][kMaxExperts];
   if (warp >= tokens) return;
@@ -35,15 +37,22 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
-    v[i] = (e < experts) ? static_cast<float>(logits[static_cast<size_t>(warp) * ld + e]) + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
+    v[i] = -INFINITY;
+    if (e < experts) {
+      const float z = static_cast<float>(logits[static_cast<size_t>(warp) * ld + e]);
+      v[i] = (sigmoid ? 1.f / (1.f + expf(-z)) : z) + (bias != nullptr ? bias[e] : 0.f);
+    }
     mx = fmaxf(mx, v[i]);
   }
-  mx = warp_max(mx);
-  float sum = 0.f;
+  float inv = 1.f;
+  if (!sigmoid) {
+    mx = warp_max(mx);
+    float sum = 0.f;
 #pragma unroll
-  for (int i = 0; i < PER; ++i) sum += (i * 32 + lane < experts) ? expf(v[i] - mx) : 0.f;
-  sum = warp_sum(sum);
-  const float inv = 1.f / sum;
+    for (int i = 0; i < PER; ++i) sum += (i * 32 + lane < experts) ? expf(v[i] - mx) : 0.f;
+    sum = warp_sum(sum);
+    inv = 1.f / sum;
+  }
   // the largest of a set of values with the lowest index among equals (-inf: not a candidate)
   auto best_of = [&](const float (&x)[PER], int count, float& best, int& at) {
     best = -INFINITY;
@@ -71,8 +80,15 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
     for (int i = 0; i < PER; ++i) {
       const int g = i * 32 + lane;
       gs[i] = -INFINITY;
-      if (g < groups)
-        for (int e = 0; e < size; ++e) gs[i] = fmaxf(gs[i], s[g * size + e]);
+      if (g < groups) {
+        float second = -INFINITY;
+        for (int e = 0; e < size; ++e) {
+          const float x = s[g * size + e];
+          second = fmaxf(second, fminf(gs[i], x));
+          gs[i] = fmaxf(gs[i], x);
+        }
+        if (group_best > 1 && size > 1) gs[i] += second;
+      }
     }
     __syncwarp();
 #pragma unroll
@@ -101,7 +117,12 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
     float best;
     int best_e;
     best_of(v, experts, best, best_e);
-    best = expf(best - mx);
+    if (sigmoid) {
+      const float z = best_e < experts ? static_cast<float>(logits[static_cast<size_t>(warp) * ld + best_e]) : -INFINITY;
+      best = 1.f / (1.f + expf(-z));
+    } else {
+      best = expf(best - mx);
+    }
     if (lane == r) { my_w = best; my_id = best_e; }
     chosen_sum += best;
 #pragma unroll
@@ -110,7 +131,7 @@ __global__ void __launch_bounds__(256) moe_route_topk_kernel(const T* __restrict
   }
   if (lane < k) {
     topk_ids[static_cast<size_t>(warp) * k + lane] = my_id;
-    topk_w[static_cast<size_t>(warp) * k + lane] = renormalize ? my_w / chosen_sum : my_w * inv;
+    topk_w[static_cast<size_t>(warp) * k + lane] = renormalize ? my_w / (chosen_sum + (sigmoid ? 1e-20f : 0.f)) : my_w * inv;
   }
 }
 
@@ -214,26 +235,29 @@ using namespace ogb;
 
 template <typename T>
 static int route_topk(const T* logits, const float* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize, int ld, int groups, int keep,
-                      void* stream) {
+                      bool sigmoid, int group_best, void* stream) {
   if (tokens <= 0) return 0;
   if (experts > kMaxExperts || k > 32 || k > experts) return -3;
   if (groups < 1 || experts % groups != 0 || keep < 1 || keep > groups || k > keep * (experts / groups)) return -3;
   const int warps_per_block = 8;
   const int blocks = (tokens + warps_per_block - 1) / warps_per_block;
   moe_route_topk_kernel<T><<<blocks, warps_per_block * 32, 0, static_cast<cudaStream_t>(stream)>>>(logits, bias, topk_ids, topk_w, tokens,
-                                                                                                 experts, k, renormalize, ld, groups, keep);
+                                                                                                 experts, k, renormalize, ld, groups, keep, sigmoid,
+                                                                                                 group_best);
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int ogb_moe_route_topk(const void* router_logits, int* topk_ids, float* topk_w, int tokens, int experts, int k,
                                   int renormalize, int ld, void* stream) {
-  return route_topk(static_cast<const __nv_bfloat16*>(router_logits), nullptr, topk_ids, topk_w, tokens, experts, k, renormalize, ld, 1, 1, stream);
+  return route_topk(static_cast<const __nv_bfloat16*>(router_logits), nullptr, topk_ids, topk_w, tokens, experts, k, renormalize, ld, 1, 1, false, 1, stream);
 }
 
-// fp32 logits and bias (or null); `groups` equal groups of experts of which the `keep` best can be chosen from (1, 1: all).
+// fp32 logits and bias (or null); `groups` equal groups of experts of which the `keep` best can be chosen from (1, 1: all).  sigmoid,
+// group_best: how experts and groups score (moe_route_topk_kernel).
 extern "C" int ogb_moe_route_grouped(const float* router_logits, const float* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize,
-                                     int ld, int groups, int keep, void* stream) {
-  return route_topk(router_logits, bias, topk_ids, topk_w, tokens, experts, k, renormalize, ld, groups, keep, stream);
+                                     int ld, int groups, int keep, int sigmoid, int group_best, void* stream) {
+  if (group_best < 1 || group_best > 2) return -3;
+  return route_topk(router_logits, bias, topk_ids, topk_w, tokens, experts, k, renormalize, ld, groups, keep, sigmoid != 0, group_best, stream);
 }
 
 // counts must be zero on entry (the caller clears it); e0 = first expert owned by this rank.

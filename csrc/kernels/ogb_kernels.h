@@ -174,9 +174,9 @@ int ogb_hyper_step(const float* x_in, float* x_out, const void* y, const float* 
                    const float* w, const float* b, const float* shift, float* prev, void* h, const int* gather, int rows, int total_rows, int S,
                    int W, int ldy, int ldh, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0,
                    int num_decode, int num_tiles, int num_slots, int elem, int* status, void* stream);
-// embed_streams: w (or null): RMS norm of the embedding; copy (or null): the same row again, [tokens, ldc].
-int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, const float* w, float eps, void* copy, int ldc,
-                      int elem, int* status, void* stream);
+// embed_streams: the embedding times scale; w (or null): RMS norm of it; copy (or null): the same row again, [tokens, ldc].
+int ogb_embed_streams(const int* ids, const void* table, float* x, int tokens, int S, int W, int vocab, const float* w, float eps, float scale, void* copy,
+                      int ldc, int elem, int* status, void* stream);
 // Latents and rotated key parts to their pages, rotated query parts to q_out or in place (hybrid.cu).
 int ogb_latent_append(void* row, int ldr, int latent, const float* w, float eps, const int* slots, void* pool, int tokens, int rank, int ldp,
                       int64_t num_slots, const double* freq, const int* positions, void* q_out, int heads, int dim, int rot, int ldq, int q_col, int split,
@@ -193,18 +193,36 @@ int ogb_hgrn2_state_rows(int D);
 int ogb_hgrn2(const float* qfv, const float* bias, const float* low, float* state, float* out, int ld, int ldo, int heads, int D, int V,
               const int* ctx_len, const int* state_slot, const int* cu_q, int num_decode, int num_prefill, int num_slots, int seg_len,
               int num_segments, float* seg_state, float* seg_gate, int split, int* status, void* stream);
-int ogb_head_rmsnorm(const float* x, const float* w, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate, int ldg,
-                     int elem, void* stream);
-// norm_step: x += rms(y) post, h = rms(x) w over one fp32 residual stream; y may be the weighted sum of a token's expert rows and a
-// gated row of a shared expert.
-int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const void* shared, const float* gate, const float* post, const float* w,
-                  void* h, const int* gather, float eps, int rows, int total_rows, int W, int k, int ldy, int lds, int ldg, int ldh, int64_t y_rows,
-                  int elem, int* status, void* stream);
-// norm_conv_step: x_out = x_in + y + add, h = a causal convolution over rms(x_out) w.
+int ogb_head_rmsnorm(const float* x, const float* w, int wstep, float eps, void* out, int rows, int heads, int n, int ldx, int ldo, const void* gate,
+                     int ldg, int sigmoid, int elem, void* stream);
+// norm_step: x += rms(y) post, h = rms(x) w over one fp32 residual stream, in `groups` parts; y may be the weighted sum of a token's expert
+// rows and a gated row of a shared expert, and may reach x as (y + y_bias) sigmoid(res_gate + res_bias).
+int ogb_norm_step(float* x, const void* y, const int* pos, const float* weight, const void* shared, const float* gate, const float* y_bias,
+                  const void* res_gate, const float* res_bias, const float* post, const float* w, void* h, const int* gather, float eps, int rows,
+                  int total_rows, int W, int groups, int k, int ldy, int lds, int ldg, int ldr, int ldh, int64_t y_rows, int elem, int* status,
+                  void* stream);
+// norm_conv_step: x_out = x_in + y + add, plain (or null) = rms(x_out) w, h = a causal convolution over it.
 int ogb_norm_conv_step(const float* x_in, float* x_out, const void* y, const int* pos, const float* weight, const void* shared, const float* gate,
-                       const float* add, const float* w, const float* conv, float* state, void* h, float* factor, float eps, int rows, int W, int taps,
-                       int k, int ldx, int ldy, int lds, int ldg, int ldh, int64_t y_rows, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq,
+                       const float* y_bias, const void* res_gate, const float* res_bias, const float* add, const float* w, const float* conv, float* state,
+                       void* h, void* plain, float* factor, float eps, int rows, int W, int groups, int taps, int k, int ldx, int ldy, int lds, int ldg,
+                       int ldr, int ldh, int ldp, int64_t y_rows, const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq,
                        const int* tile_q0, int num_decode, int num_tiles, int num_slots, int elem, int* status, void* stream);
+// Matrix memories with one decay per head (decay_memory.cu).  turns [tokens, half]: (cos, sin) of turn_table.
+int ogb_turn_table(const int* positions, const double* freq, float* out, int tokens, int half, void* stream);
+int ogb_decay_block_floats(int heads, int D, int V, int gated);
+int ogb_decay_memory(const void* row, int ld, const float* turns, int half, const float* logits, int ldl, const float* bias, float cap,
+                     const float* decay, float* state, float* peak, float* out, int heads, int D, int V, int DP, float q_scale, float k_scale,
+                     const int* ctx_len, const int* state_slot, const int* cu_q, const int* tile_seq, const int* tile_q0, int num_decode,
+                     int num_prefill, int num_tiles, int num_slots, float* work, int elem, int* status, void* stream);
+// Attention over paged keys that are the values too (tied_attention.cu): pages [hkv][16][dp] keys | [16] fp32 factors.
+int ogb_tied_append(const void* row, int ldr, const float* q_bias, const float* k_bias, const float* q_gain, float eps, float factor, void* q, int ldq,
+                    void* pool, const int* slots, int64_t num_slots, int64_t page_elems, int tokens, int hq, int hkv, int d, int dp, int elem,
+                    int* status, void* stream);
+int ogb_tied_attention(const void* q, void* out, const void* pool, const int* page_table, const int* ctx_len, const int* cu_q, const int* tile_seq,
+                       const int* tile_q0, const void* gate, const float* slope, const float* sink, int rows, int num_tiles, int max_pages,
+                       int64_t num_pages, int64_t page_elems, int hq, int hkv, int d, int dp, int ldq, int ldo, int ldg, int window, float cap,
+                       int num_splits, float* part_o, float* part_ml, int* counters, int elem, int* status, void* stream);
+int ogb_tied_set_tc(int on);
 // Short causal convolutions (short_conv.cu): w [taps, channels], state [slots, taps - 1, channels].
 // Attention: q (nq heads of d) | k (nk) | v (nv heads of dv); rotated queries to q, keys and values to pages [nk][16][dp] | [nv][16][vp].
 int ogb_conv_rope_append(const void* u, int ldu, const float* w, const float* bias, float* state, int taps, void* q, int ldq, void* pool,
@@ -240,7 +258,7 @@ int ogb_moe_permute(const int* topk_ids, int* counts, int* offsets, int* cursor,
 int ogb_moe_gather_rows(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int hidden,
                         void* stream);
 int ogb_moe_route_grouped(const float* router_logits, const float* bias, int* topk_ids, float* topk_w, int tokens, int experts, int k, int renormalize,
-                          int ld, int groups, int keep, void* stream);
+                          int ld, int groups, int keep, int sigmoid, int group_best, void* stream);
 int ogb_moe_gather_bytes(const void* x, const int* sorted_route, const int* meta, void* xs, int max_routes, int k, int row_bytes, void* stream);
 int ogb_grouped_gemm_act(const void* A, const void* W, void* C, const int* group_tab, const int* group_mtiles, int experts, int max_rows, int max_mtiles,
                          int N, int K, int lda, int ldw, int ldc, int act, float act_a, float act_b, int bn, int* status, void* stream);

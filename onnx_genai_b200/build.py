@@ -39,7 +39,7 @@ NVCC_FLAGS = [
 # paths call exp2f/__expf explicitly.  Sources whose tanh, exp, divisions and roots belong to a model's 32-bit part are
 # compiled without it.
 PRECISE_SOURCES = {"hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_attention_tc.cu", "latent_decode.cu", "short_conv.cu", "delta_rule.cu",
-                   "diff_attention.cu", "diff_attention_tc.cu", "moe.cu"}
+                   "diff_attention.cu", "diff_attention_tc.cu", "moe.cu", "decay_memory.cu", "tied_attention.cu", "tied_attention_tc.cu"}
 # A library of its own for models that need only a few of the kernel sources: built when the full library is not there, so
 # that the first load compiles no more than the model uses (ops/_native.py ``prefer``).
 SUBSETS = {"hybrid": ("hybrid.cu", "recurrent.cu", "latent_attention.cu", "latent_attention_tc.cu", "latent_decode.cu", "attention_tc.cu", "attention.cu", "gemm_tcgen05.cu",
@@ -47,7 +47,8 @@ SUBSETS = {"hybrid": ("hybrid.cu", "recurrent.cu", "latent_attention.cu", "laten
            "delta": ("hybrid.cu", "short_conv.cu", "delta_rule.cu", "diff_attention.cu", "diff_attention_tc.cu", "moe.cu", "gemm_tcgen05.cu", "sampling.cu",
                      "tp_comm.cu"),
            "latent_moe": ("hybrid.cu", "latent_attention.cu", "latent_attention_tc.cu", "latent_decode.cu", "attention_tc.cu", "attention.cu", "moe.cu",
-                          "gemm_tcgen05.cu", "sampling.cu", "tp_comm.cu")}
+                          "gemm_tcgen05.cu", "sampling.cu", "tp_comm.cu"),
+           "memory": ("hybrid.cu", "decay_memory.cu", "tied_attention.cu", "tied_attention_tc.cu", "moe.cu", "gemm_tcgen05.cu", "sampling.cu", "tp_comm.cu")}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-fopenmp", "-mavx2", "-mfma"]
 
 

@@ -1,6 +1,7 @@
-"""Decoder whose layers each choose a mixer -- recurrent (HGRN2, gated delta rule) or attention (over paged latents, differential) --
-and a feed-forward (gated or not, routed experts), on hyper-connected residual streams or on one stream normed before -- and
-behind -- every sublayer.  A range of layers may run several times in a row with the same weights.
+"""Decoder whose layers each choose a mixer -- recurrent (HGRN2, gated delta rule, matrix memories with one decay per head) or attention
+(over paged latents, over keys that are the values, differential) -- and a feed-forward (gated or not, routed experts), on hyper-connected
+residual streams or on one stream normed before -- and behind -- every sublayer.  A range of layers may run several times in a row with
+the same weights.
 
 A design of this kind is a :class:`HybridConfig` (layer specs plus constants) and a :class:`HybridWeights`;
 ``models/registry.py`` says which checkpoint architectures map here and how their files are read.  The executor lowers
@@ -8,13 +9,17 @@ a layer run to a fixed list of launches over buffers allocated once:
 
     hyper_step (fold the last sublayer's output into the streams, read-out, norm, token shift), or
     norm_step  (x += norm(the last sublayer's output), norm; sums the rows of routed experts on the way), or
-    norm_conv_step (x += the last sublayer's output, norm, causal convolution of what the sublayer reads)
+    norm_conv_step (x += the last sublayer's output, norm, causal convolution of what the sublayer reads); both passes take the
+                bias and the gate of an output on its way to x: gemm(residual gate) over the normed rows stands behind them
     pass:       norm_step (x += the last sublayer's output, copy beside the embedding) | gemm(x | embedding, fp32 out)
     recurrent:  gemm(q | gate | v, fp32 out) | hgrn2 | head_rmsnorm | gemm(o)
     delta:      gemm(gate | q | k | v) | gemm(decay | step size, fp32 out) | conv_unit_gates | delta_rule | head_rmsnorm * gate | gemm(o)
     latent:     gemm(q | latent | rotated key | head gates) | latent_append (norm, rotations) | gemm per head (W_uk^T q) |
                 latent_attention (head gates in its epilogue) | gemm per head (W_uv o) | gemm(o);
                 prompts over wide latents: latent_gather | gemm (K | V pages) | paged_prefill | gemm(o)
+    tied:       gemm(q | k | head gates) | tied_append (biases, norms, pages) | tied_attention (bias by distance, cap, sink, head gates) | gemm(o)
+    memory:     gemm(q | k | v | gate) | gemm(input | forget gates, fp32 out) | decay_memory (rotations, gates, read-out) | head_rmsnorm * gate |
+                gemm(o)
     diff:       gemm(q | k | v) | conv_rope_append | diff_attention (both maps, difference and norm) | gemm(o)
     dense:      gemm(gate_up or up, activation in the epilogue) | gemm(down)
     experts:    gemm(router | shared gate, fp32 out) | route, permute, gather | grouped gemm(up, activation epilogue) | grouped gemm(down)
@@ -35,7 +40,7 @@ import torch
 from .. import ops
 from ..ops import hybrid as hops
 from ..ops import moe as moe_ops
-from ..ops.hybrid import Act, DynamicTanh, ExpertRows, HyperConnection, LatentRope, RmsNorm
+from ..ops.hybrid import Act, DynamicTanh, ExpertRows, GatedRows, HyperConnection, LatentRope, RmsNorm
 from .decoder import pad_mlp, pick_swiglu_half
 
 
@@ -134,6 +139,64 @@ class DiffSpec:
 
 
 @dataclass
+class TiedSpec:
+    """Attention whose values are its keys before their norm: ``heads`` queries of ``dim`` over ``kv_heads`` keys, both normed over the whole
+    projection.  Scores times ``scale`` are capped to softcap tanh(s / softcap) (0: not), and lose a number per head times the distance;
+    ``sink``: a number per head joins the softmax; ``window`` 0 means every earlier token; ``gated``: a sigmoid per head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    softcap: float = 0.0
+    window: int = 0
+    sink: bool = True
+    gated: bool = True
+
+    @property
+    def gate_col(self) -> int:
+        return (self.heads + self.kv_heads) * self.dim
+
+    @property
+    def proj_width(self) -> int:
+        return self.gate_col + (self.heads if self.gated else 0)
+
+    @property
+    def factor(self) -> float:
+        """What a page's factors hold besides the key's norm."""
+        return self.scale / self.softcap if self.softcap > 0 else self.scale
+
+    @property
+    def page_elems(self) -> int:
+        return hops.tied_page_elems(self.kv_heads, pad8(self.dim))
+
+
+@dataclass
+class MemorySpec:
+    """Matrix memories of ``dim`` x ``vdim`` with one decay per head and an output gate.  ``gate_cap`` 0: retention -- fixed decays, queries and
+    keys rotated in their first ``rot_dims``, keys scaled by dim^-1/2, a silu gate; otherwise mLSTM -- exponential input gates and
+    sigmoid forget gates capped at +-gate_cap under a running maximum, a normalizer, queries scaled, a sigmoid gate."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float = 0.0
+    decay: tuple = ()                  # a fixed one per head
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+
+    @property
+    def gated(self) -> bool:
+        return self.gate_cap > 0
+
+    @property
+    def gate_col(self) -> int:
+        return self.heads * (2 * self.dim + self.vdim)
+
+    @property
+    def proj_width(self) -> int:
+        return self.gate_col + self.heads * self.vdim
+
+
+@dataclass
 class MlpSpec:
     """``act``: a gated activation, or "xielu" (one projection, two numbers per layer)."""
     inter: int
@@ -142,8 +205,9 @@ class MlpSpec:
 
 @dataclass
 class MoeSpec:
-    """Routed experts down(act(up h)), ``top`` of ``experts`` per token, chosen from the ``keep`` best of ``groups`` equal groups; ``act``:
-    "relu2", or "clamp_glu" with a gate and ``limit``.  ``shared_inter`` > 0: an expert of that size (and ``shared_limit``) runs for every
+    """Routed experts down(act(up h)), ``top`` of ``experts`` per token, chosen from the ``keep`` best of ``groups`` equal groups, which score as
+    their ``group_best`` best experts; ``score``: "softmax" (``bias``: added to the logits) or "sigmoid" (added to the scores that are
+    compared).  ``act``: "relu2", or with a gate "silu" or "clamp_glu" (``limit``).  ``shared_inter`` > 0: an expert of that size (and ``shared_limit``) runs for every
     token, times the sigmoid of a projection."""
     experts: int
     top: int
@@ -156,6 +220,8 @@ class MoeSpec:
     shared_inter: int = 0
     shared_limit: float = 0.0
     bias: bool = False
+    score: str = "softmax"
+    group_best: int = 1
 
     @property
     def gated(self) -> bool:
@@ -169,7 +235,7 @@ class MoeSpec:
 
 @dataclass
 class LayerSpec:
-    mixer: RecurrentSpec | LatentSpec | DeltaSpec | DiffSpec
+    mixer: RecurrentSpec | LatentSpec | DeltaSpec | DiffSpec | TiedSpec | MemorySpec
     mlp: MlpSpec | MoeSpec | None = None
 
 
@@ -194,6 +260,11 @@ class HybridConfig:
     residual: str = "hyper"            # "hyper": connected streams, Dynamic-Tanh norms, token shift; "sandwich": RMS norms around a sublayer;
                                        # "pre": RMS norms before a sublayer
     input_taps: int = 0                # "pre": what a sublayer reads is h plus a causal convolution of h over this many taps (0: h)
+    ff_input_conv: bool = True         # feed-forwards too, not only mixers
+    residual_gates: bool = False       # "pre": a sublayer's output reaches the residual times sigmoid(W h + b), h the normed residual
+    norm_groups: int = 1
+    embed_scale: float = 1.0
+    embed_normed: bool = True          # "pre": random weights have a norm of the embedding
     loop: LoopSpec | None = None
     eos_token: int = -1
     max_position: int = 1 << 20        # no positional table: bounded by the pool only
@@ -218,7 +289,7 @@ class HybridConfig:
 
     @property
     def attention_layers(self) -> list:
-        return [l.mixer for l in self.layers if isinstance(l.mixer, (LatentSpec, DiffSpec))]
+        return [l.mixer for l in self.layers if isinstance(l.mixer, (LatentSpec, DiffSpec, TiedSpec))]
 
     @property
     def num_heads(self) -> int:
@@ -242,7 +313,7 @@ class HybridConfig:
     def kv_page_shape(self, layer: int, kv_heads: int = 1):
         """Shape of one KV page of a layer run, None when it caches nothing of its own."""
         m = self.layers[self.runs[layer]].mixer
-        if isinstance(m, DiffSpec):
+        if isinstance(m, (DiffSpec, TiedSpec)):
             return (m.page_elems,)
         return (ops.PAGE, m.key_width) if isinstance(m, LatentSpec) and m.kv_from is None else None
 
@@ -253,12 +324,16 @@ class HybridConfig:
         shapes = {"shift": (self.hidden,)} if self.residual == "hyper" else {}
         if self.input_taps:
             shapes["input1"] = (self.input_taps - 1, self.hidden)
-            if spec.mlp is not None:
+            if spec.mlp is not None and self.ff_input_conv:
                 shapes["input2"] = (self.input_taps - 1, self.hidden)
         if isinstance(m, (DeltaSpec, DiffSpec)):
             shapes["conv"] = (m.taps - 1, m.conv_width)
         if isinstance(m, (RecurrentSpec, DeltaSpec)):
             shapes["recurrent"] = (m.heads, m.vdim, hops.state_rows(m.dim))
+        if isinstance(m, MemorySpec):
+            shapes["recurrent"] = (m.heads, m.vdim + m.gated, hops.state_rows(m.dim))
+            if m.gated:
+                shapes["peak"] = (m.heads,)
         return shapes
 
     def validate(self) -> None:
@@ -266,8 +341,15 @@ class HybridConfig:
             raise ValueError(f"unknown residual {self.residual!r}")
         if self.input_taps and (self.residual != "pre" or not 0 <= self.input_taps <= 8):
             raise ValueError(f"input convolutions of {self.input_taps} taps are not supported (1 to 8, behind norms before the sublayers)")
-        if self.input_taps and self.hidden > (8192 if self.hidden % 4 == 0 else 4096):
-            raise ValueError(f"input convolutions of {self.hidden} channels are not supported (8192, 4096 where they are no multiple of 4)")
+        if self.norm_groups < 1 or self.hidden % self.norm_groups or (self.norm_groups > 1 and self.residual != "pre"):
+            raise ValueError(f"norms of {self.hidden} channels in {self.norm_groups} groups are not supported (equal groups, before the sublayers)")
+        quads = self.hidden // self.norm_groups % 4 == 0
+        if self.input_taps and self.hidden > (8192 if quads else 4096):
+            raise ValueError(f"input convolutions of {self.hidden} channels are not supported (8192, 4096 where a norm's groups are no multiple of 4)")
+        if self.residual_gates and self.residual != "pre":
+            raise ValueError("gates of the residual need norms before the sublayers")
+        if self.norm_groups > 1 and self.hidden > (16384 if quads else 4096):
+            raise ValueError(f"norms in groups of {self.hidden} channels are not supported (16384, 4096 where they are no multiple of 4)")
         if self.loop is not None:
             lp = self.loop
             if self.residual != "pre" or not 0 <= lp.start < lp.stop <= len(self.layers) or lp.times < 1:
@@ -282,15 +364,29 @@ class HybridConfig:
             if isinstance(f, MoeSpec):
                 if self.residual == "hyper":
                     raise ValueError(f"layer {i}: routed experts need a residual of one stream")
-                if f.act not in ("relu2", "clamp_glu"):
+                if f.score not in ("softmax", "sigmoid") or f.group_best < 1 or f.group_best > 2:
+                    raise ValueError(f"layer {i}: routing by {f.score!r} scores and the {f.group_best} best experts of a group is not supported")
+                if f.act not in ("relu2", "silu", "clamp_glu"):
                     raise ValueError(f"layer {i}: unknown activation {f.act!r} of routed experts")
                 if f.experts > 256 or f.top > 32 or f.groups < 1 or f.experts % f.groups or not 1 <= f.keep <= f.groups:
                     raise ValueError(f"layer {i}: {f.experts} experts in {f.groups} groups, {f.keep} kept, {f.top} chosen are not supported "
                                      "(at most 256 experts in equal groups, 32 chosen)")
                 if not 1 <= f.top <= f.keep * (f.experts // f.groups):
                     raise ValueError(f"layer {i}: {f.top} experts cannot be chosen from {f.keep} groups of {f.experts // f.groups}")
-            if isinstance(m, (RecurrentSpec, DeltaSpec)):
+            if isinstance(m, (RecurrentSpec, DeltaSpec, MemorySpec)):
                 hops.state_rows(m.dim)
+            if isinstance(m, MemorySpec):
+                if not m.gated and (len(m.decay) != m.heads or not all(0 <= a <= 1 for a in m.decay)):
+                    raise ValueError(f"layer {i}: {len(m.decay)} decays for {m.heads} heads (one each, between 0 and 1)")
+                if m.rot_dims % 2 or not 0 <= m.rot_dims <= m.dim:
+                    raise ValueError(f"layer {i}: {m.rot_dims} rotated dimensions of {m.dim}")
+                if m.gated and m.vdim > 512:
+                    raise ValueError(f"layer {i}: gated memories of {m.vdim} value channels are not supported (at most 512)")
+            if isinstance(m, TiedSpec):
+                if m.kv_heads < 1 or m.heads % m.kv_heads:
+                    raise ValueError(f"layer {i}: {m.heads} heads do not divide over {m.kv_heads} key heads")
+                if m.dim > 512:
+                    raise ValueError(f"layer {i}: heads of {m.dim} are not supported (at most 512)")
             if isinstance(m, (DeltaSpec, DiffSpec)):
                 if not 1 <= m.taps <= 8:
                     raise ValueError(f"layer {i}: convolutions of {m.taps} taps are not supported (1 to 8)")
@@ -331,6 +427,10 @@ class HybridConfig:
                 n += self.hidden * (m.conv_width + 2 * m.heads * m.vdim + 2 * m.heads)
             elif isinstance(m, DiffSpec):
                 n += self.hidden * (m.conv_width + m.heads * m.vdim)
+            elif isinstance(m, TiedSpec):
+                n += self.hidden * (m.proj_width + m.heads * m.dim)
+            elif isinstance(m, MemorySpec):
+                n += self.hidden * (m.proj_width + m.heads * m.vdim + 2 * m.heads * m.gated)
             else:
                 n += self.hidden * m.heads * (m.dim + m.rot_dim + m.vdim + m.gated) + m.rank * m.heads * (m.dim + m.vdim)
                 n += self.hidden * (m.rank + m.rot_dim) if m.kv_from is None else 0
@@ -339,6 +439,8 @@ class HybridConfig:
                 n += self.hidden * (f.experts * (2 + f.gated) * f.inter + 3 * f.shared_inter + f.logits)
             elif layer.mlp:
                 n += (2 + Act(layer.mlp.act).gated) * self.hidden * layer.mlp.inter
+            if self.residual_gates:
+                n += (1 + (layer.mlp is not None)) * self.hidden * self.hidden
         if self.loop is not None:
             n += 2 * self.hidden * self.hidden
         return 2 * n
@@ -346,7 +448,7 @@ class HybridConfig:
     def kv_bytes_per_token(self, kv_dtype_bytes: int = 2) -> int:
         mixers = [self.layers[li].mixer for li in self.runs]
         return kv_dtype_bytes * (sum(m.key_width for m in mixers if isinstance(m, LatentSpec) and m.kv_from is None) +
-                                 sum(m.page_elems // ops.PAGE for m in mixers if isinstance(m, DiffSpec)))
+                                 sum(m.page_elems // ops.PAGE for m in mixers if isinstance(m, (DiffSpec, TiedSpec))))
 
 
 # ------------------------------------------------------------------------------------------
@@ -394,6 +496,28 @@ class DiffWeights:
 
 
 @dataclass
+class TiedWeights:
+    qkg: torch.Tensor                  # [TiedSpec.proj_width, hidden]: queries, keys, head gates
+    q_bias: torch.Tensor | None        # fp32 [heads * dim]
+    k_bias: torch.Tensor | None        # fp32 [kv_heads * dim]
+    q_gain: torch.Tensor               # fp32 [heads * dim]: the query norm's weight times the key norm's of the head's keys
+    slope: torch.Tensor | None         # fp32 [heads]
+    sink: torch.Tensor | None          # fp32 [heads]
+    o: torch.Tensor                    # [hidden, heads * dim_p]
+    o_bias: torch.Tensor | None = None
+
+
+@dataclass
+class MemoryWeights:
+    qkvg: torch.Tensor                 # [MemorySpec.proj_width, hidden]: queries, keys, values, output gate
+    o: torch.Tensor                    # [hidden, heads * vdim]
+    decay: torch.Tensor | None = None          # fp32 [2, heads]: decays, their logarithms
+    gates: torch.Tensor | None = None          # [2 * heads, hidden]: input, forget
+    gates_bias: torch.Tensor | None = None     # fp32 [2 * heads]
+    norm: torch.Tensor | None = None           # fp32 [heads * vdim]
+
+
+@dataclass
 class MoeWeights:
     router: torch.Tensor     # [experts (+ the shared expert's gate), hidden]
     up: torch.Tensor         # [experts, inter_p, hidden_p]; gated: [experts, 2 inter_p, hidden_p], gate and up rows packed with ``half``
@@ -411,7 +535,7 @@ class HybridLayer:
     norms before (norm1, norm2) and, for "sandwich", behind (hc1, hc2) the sublayers."""
     norm1: DynamicTanh | RmsNorm
     hc1: HyperConnection | RmsNorm | None
-    mixer: RecurrentWeights | LatentWeights | DeltaWeights | DiffWeights
+    mixer: RecurrentWeights | LatentWeights | DeltaWeights | DiffWeights | TiedWeights | MemoryWeights
     shift: torch.Tensor | None = None             # fp32 [hidden]
     norm2: DynamicTanh | RmsNorm | None = None
     hc2: HyperConnection | RmsNorm | None = None
@@ -422,6 +546,10 @@ class HybridLayer:
     act: Act | None = None                        # feed-forward; a gated one has gate_up packed with ``half``, another up rows alone
     conv1: torch.Tensor | None = None             # fp32 [input_taps, hidden]: what the sublayer reads, the identity included
     conv2: torch.Tensor | None = None
+    gate1: torch.Tensor | None = None             # [hidden, hidden] and fp32 [hidden]: gates of what the sublayers add to the residual
+    gate1_bias: torch.Tensor | None = None
+    gate2: torch.Tensor | None = None
+    gate2_bias: torch.Tensor | None = None
 
 
 @dataclass
@@ -517,6 +645,32 @@ def pack_diff(spec: DiffSpec, q, k, v, bias, conv, lam: float, o) -> DiffWeights
                        lam=float(lam), o=torch.nn.functional.pad(o.reshape(o.shape[0], spec.heads, spec.vdim), (0, vp - spec.vdim)).reshape(o.shape[0], -1).contiguous())
 
 
+def pack_tied(spec: TiedSpec, q, k, g, q_bias, k_bias, q_norm, k_norm, slope, sink, o, o_bias) -> TiedWeights:
+    """q_norm, k_norm: weights over the whole projections."""
+    h, d, dp = spec.heads, spec.dim, pad8(spec.dim)
+    f32 = lambda t: None if t is None else t.float().contiguous()
+    keys = k_norm.float().view(spec.kv_heads, 1, d).expand(-1, h // spec.kv_heads, -1).reshape(-1)
+    return TiedWeights(qkg=pad_cols(torch.cat([q, k] + ([g] if g is not None else []), 0)), q_bias=f32(q_bias), k_bias=f32(k_bias),
+                       q_gain=(q_norm.float() * keys).contiguous(), slope=f32(slope), sink=f32(sink), o_bias=f32(o_bias),
+                       o=torch.nn.functional.pad(o.reshape(o.shape[0], h, d), (0, dp - d)).reshape(o.shape[0], h * dp).contiguous())
+
+
+def distance_slopes(heads: int, device) -> torch.Tensor:
+    """Slopes 2^(-8 (h + 1) / heads) of biases by distance."""
+    return torch.exp2(-8 * torch.arange(1, heads + 1, dtype=torch.float64) / heads).float().to(device)
+
+
+def pack_memory(spec: MemorySpec, q, k, v, g, o, gates=None, gates_bias=None, norm=None) -> MemoryWeights:
+    """``gates``: input and forget projections."""
+    f32 = lambda t: None if t is None else t.float().contiguous()
+    decay = None
+    if not spec.gated:                 # a decay of zero forgets everything at once; its logarithm stays finite
+        decay = torch.tensor(spec.decay, dtype=torch.float64)
+        decay = torch.stack([decay, torch.log(decay).clamp(min=-1e30)]).float().to(q.device)
+    return MemoryWeights(qkvg=pad_cols(torch.cat([q, k, v, g], 0)), o=pad_cols(o), decay=decay, gates=None if gates is None else pad_cols(gates),
+                         gates_bias=f32(gates_bias), norm=f32(norm))
+
+
 def pack_moe(router, ups, downs) -> MoeWeights:
     """``ups`` [inter, hidden] and ``downs`` [hidden, inter] of every expert."""
     inter = ups[0].shape[0]
@@ -584,12 +738,12 @@ def random_weights(cfg: HybridConfig, device, seed: int = 0, std: float = 0.02, 
         norm = lambda: DynamicTanh(0.5 + rand(1), 1 + 0.1 * (rand(hid) - 0.5), 0.1 * (rand(hid) - 0.5))
         conn = lambda: HyperConnection(rand(st) / st + 0.5 / st, 0.5 + rand(st), torch.eye(st, device=dev) * 0.8 + 0.2 * rand(st, st) / st)
     else:
-        norm = lambda: RmsNorm(1 + 0.1 * (rand(hid) - 0.5), cfg.norm_eps)
+        norm = lambda: RmsNorm(1 + 0.1 * (rand(hid) - 0.5), cfg.norm_eps, cfg.norm_groups)
         conn = norm if cfg.residual == "sandwich" else lambda: None
     taps = lambda m, *rows: [torch.randn(n, m.taps, generator=gen, device=dev) * 0.5 / m.taps for n in rows]
     input_conv = lambda: pack_input_conv(torch.randn(hid, cfg.input_taps, generator=gen, device=dev) * 0.5 / cfg.input_taps) if cfg.input_taps else None
     w = HybridWeights(embed=draw(cfg.vocab, hid))
-    if cfg.residual == "pre":
+    if cfg.residual == "pre" and cfg.embed_normed:
         w.embed_norm = norm()
     if cfg.loop is not None:
         w.loop_in, w.loop_step = pack_loop_in(draw(hid, 2 * hid)), torch.randn(cfg.loop.times, hid, generator=gen, device=dev) * std
@@ -605,6 +759,14 @@ def random_weights(cfg: HybridConfig, device, seed: int = 0, std: float = 0.02, 
         elif isinstance(m, DiffSpec):
             rows = (2 * m.heads * m.dim, 2 * m.kv_heads * m.dim, m.kv_heads * m.vdim)
             mixer = pack_diff(m, *(draw(n, hid) for n in rows), [draw(n) for n in rows], taps(m, *rows), m.diff, draw(hid, m.heads * m.vdim))
+        elif isinstance(m, TiedSpec):
+            nq, nk = m.heads * m.dim, m.kv_heads * m.dim
+            mixer = pack_tied(m, draw(nq, hid), draw(nk, hid), draw(m.heads, hid) if m.gated else None, draw(nq), draw(nk), 1 + 0.1 * (rand(nq) - 0.5),
+                              1 + 0.1 * (rand(nk) - 0.5), distance_slopes(m.heads, dev), rand(m.heads) if m.sink else None, draw(hid, nq), draw(hid))
+        elif isinstance(m, MemorySpec):
+            k, v = m.heads * m.dim, m.heads * m.vdim
+            own = dict(gates=draw(2 * m.heads, hid), gates_bias=torch.cat([rand(m.heads) - 1, rand(m.heads) + 3]), norm=1 + 0.1 * (rand(v) - 0.5)) if m.gated else {}
+            mixer = pack_memory(m, draw(k, hid), draw(k, hid), draw(v, hid), draw(v, hid), draw(hid, v), **own)
         else:
             own = m.kv_from is None
             mixer = pack_latent(m, draw(m.heads * (m.dim + m.rot_dim), hid), draw(m.rank + m.rot_dim, hid) if own else None,
@@ -612,7 +774,11 @@ def random_weights(cfg: HybridConfig, device, seed: int = 0, std: float = 0.02, 
                                 draw(hid, m.heads * m.vdim), draw(m.heads, hid) if m.gated else None)
         layer = HybridLayer(norm1=norm(), shift=rand(hid) if cfg.residual == "hyper" else None, hc1=conn(), mixer=mixer, conv1=input_conv())
         if spec.mlp is not None:
-            layer.norm2, layer.hc2, layer.conv2 = norm(), conn(), input_conv()
+            layer.norm2, layer.hc2, layer.conv2 = norm(), conn(), input_conv() if cfg.ff_input_conv else None
+        if cfg.residual_gates:
+            layer.gate1, layer.gate1_bias = pad_cols(draw(hid, hid)), rand(hid)
+            if spec.mlp is not None:
+                layer.gate2, layer.gate2_bias = pad_cols(draw(hid, hid)), rand(hid)
         f = spec.mlp
         if isinstance(f, MoeSpec) and f.gated:
             expert = lambda n: (draw(n, hid), draw(n, hid), draw(hid, n))
@@ -656,26 +822,32 @@ class HybridModel:
         self.xs = [z(max_tokens, cfg.streams, hid, dtype=torch.float32) for _ in range(1 if cfg.residual == "sandwich" else 2)]
         self.h, self.y = z(max_tokens, pad8(hid)), z(max_tokens, pad8(hid))
         of = lambda kind: [l.mixer for l in cfg.layers if isinstance(l.mixer, kind)]
-        rec, lat, delta, diff = of(RecurrentSpec), of(LatentSpec), of(DeltaSpec), of(DiffSpec)
+        rec, lat, delta, diff, tied, mem = (of(kind) for kind in (RecurrentSpec, LatentSpec, DeltaSpec, DiffSpec, TiedSpec, MemorySpec))
         experts = [l.mlp for l in cfg.layers if isinstance(l.mlp, MoeSpec)]
         most = lambda widths: max(widths, default=0)
         flat = lambda width, dtype=dt: z(max_tokens * width, dtype=dtype) if width else None    # viewed per layer: rows stay contiguous
         self.qfv = flat(most(pad8(m.heads * (2 * m.dim + m.vdim)) for m in rec), torch.float32)
-        self.rec_o = flat(most(m.heads * m.vdim for m in rec + delta), torch.float32)
-        self.factor = z(max_tokens, dtype=torch.float32) if cfg.input_taps else None
+        self.rec_o = flat(most(m.heads * m.vdim for m in rec + delta + mem), torch.float32)
+        self.factor = z(max_tokens * cfg.norm_groups, dtype=torch.float32) if cfg.input_taps else None
+        self.plain, self.res_gate = (z(max_tokens, pad8(hid)) if cfg.residual_gates else None for _ in range(2))
+        # rotations of a step's rows, shared by the layers that turn alike
+        self.turns = {key: (rotation(*key, dev), z(max_tokens, key[0] // 2, 2, dtype=torch.float32))
+                      for key in {(m.rot_dims, m.rot_base) for m in mem if m.rot_dims}}
         self.loop_in = self.loop_x = None
         if cfg.loop is not None:       # residual | embedding, and the residual a pass begins with
             self.loop_in, self.loop_x = z(max_tokens, 2 * pad8(hid)), z(max_tokens, pad8(hid), dtype=torch.float32)
         self.qc = flat(most(pad8(m.proj_width) for m in lat))
         self.qa = flat(most(m.heads * m.key_width for m in lat))
         self.oc = flat(most(m.heads * pad8(m.rank) for m in lat))
-        self.proj = flat(most([pad8(m.conv_width + m.heads * m.vdim) for m in delta] + [pad8(m.conv_width) for m in diff]))
-        self.ab = flat(most([pad8(2 * m.heads) for m in delta] + [pad8(f.logits) for f in experts]), torch.float32)
+        self.proj = flat(most([pad8(m.conv_width + m.heads * m.vdim) for m in delta] + [pad8(m.conv_width) for m in diff] +
+                              [pad8(m.proj_width) for m in tied + mem]))
+        self.ab = flat(most([pad8(2 * m.heads) for m in delta + mem] + [pad8(f.logits) for f in experts]), torch.float32)
         self.unit_qk = flat(most(2 * m.kv_heads * m.dim for m in delta), torch.float32)
         self.unit_v = flat(most(m.heads * m.vdim for m in delta))
         self.gates = flat(most(2 * m.heads for m in delta), torch.float32)
-        self.diff_q = flat(most(2 * m.heads * pad8(m.dim) for m in diff))
-        self.attn = flat(most([pad8(m.heads * m.vdim) for m in rec + delta] + [m.heads * pad8(m.vdim) for m in lat + diff]))
+        self.diff_q = flat(most([2 * m.heads * pad8(m.dim) for m in diff] + [m.heads * pad8(m.dim) for m in tied]))
+        self.attn = flat(most([pad8(m.heads * m.vdim) for m in rec + delta + mem] + [m.heads * pad8(m.vdim) for m in lat + diff] +
+                              [m.heads * pad8(m.dim) for m in tied]))
         inter = most([l.down.shape[1] for l in weights.layers if l.down is not None] +
                      [l.moe.shared_down.shape[1] for l in weights.layers if l.moe is not None and l.moe.shared_down is not None])
         self.act = flat(inter)
@@ -693,14 +865,14 @@ class HybridModel:
         self.logits_buf = z(max_seqs, pad8(cfg.vocab) if dev.type == "cuda" else cfg.vocab)
         self.logits = self.logits_buf[:, : cfg.vocab]
         per_cta = 32 if dt == torch.bfloat16 else 4                     # latent heads a decode CTA takes
-        diff_ctas = [m.kv_heads * -(-(m.heads // m.kv_heads) // 8) for m in diff]
+        diff_ctas = [m.kv_heads * -(-(m.heads // m.kv_heads) // 8) for m in diff] + [m.kv_heads * -(-(m.heads // m.kv_heads) // 16) for m in tied]
         self.hkv = most([-(-m.heads // per_cta) for m in lat] + diff_ctas) or 1      # CTAs per decode row ...
         per_sm = 8 if dt == torch.float32 else (2 if most(m.key_width for m in lat) <= 128 else 1)
         self.decode_ctas = per_sm * (ops.num_sms() if dev.type == "cuda" else 148)       # ... and the device's places for them
         self.decode_splits, self._split_capacity = 1, 1
         # fp32 partial results of a decode row and split: 16 rows per CTA, and (maximum, sum) of each
         self.part_rows = most([m.heads for m in lat] + [16 * n for n in diff_ctas])
-        self.part_width = most([pad8(m.rank) for m in lat] + [pad8(m.vdim) for m in diff])
+        self.part_width = most([pad8(m.rank) for m in lat] + [pad8(m.vdim) for m in diff] + [pad8(m.dim) for m in tied])
         self.part_o = self.part_ml = None
         self.counters = z(max_seqs * (most([-(-m.heads // 16) for m in lat] + diff_ctas) or 1), dtype=torch.int32) if dev.type == "cuda" else None
         self.state = None
@@ -783,12 +955,42 @@ class HybridModel:
                             m.window, m.keep, self.decode_splits, self.part_o, self.part_ml, self.counters)
         hops.linear(attn, w.o, y)
 
+    def _tied(self, li, m: TiedSpec, w: TiedWeights, h, y, kv, si):
+        t, dp = h.shape[0], pad8(m.dim)
+        proj = self._rows(self.proj, t, pad8(m.proj_width))
+        hops.linear(h, w.qkg, proj[:, : m.proj_width])
+        q, attn = self._rows(self.diff_q, t, m.heads * dp), self._rows(self.attn, t, m.heads * dp)
+        hops.tied_append(proj, w.q_bias, w.k_bias, w.q_gain, self.cfg.norm_eps, m.factor, q, kv.pools[li], si.slots, m.heads, m.kv_heads, m.dim, dp)
+        hops.tied_attention(q, attn, kv.pools[li], si, m.heads, m.kv_heads, m.dim, dp, m.softcap, w.slope, w.sink, m.window,
+                            proj[:, m.gate_col:m.gate_col + m.heads] if m.gated else None, self.decode_splits, self.part_o, self.part_ml, self.counters)
+        hops.linear(attn, w.o, y)
+
+    def _memory(self, li, m: MemorySpec, w: MemoryWeights, h, y, si):
+        t, width, st = h.shape[0], m.heads * m.vdim, self.state.layers[li]
+        proj = self._rows(self.proj, t, pad8(m.proj_width))
+        hops.linear(h, w.qkvg, proj[:, : m.proj_width])
+        logits = None
+        if m.gated:
+            logits = self._rows(self.ab, t, pad8(2 * m.heads))
+            hops.linear(h, w.gates, logits[:, : 2 * m.heads], f32_out=True)
+        turns = self.turns[m.rot_dims, m.rot_base][1][:t] if m.rot_dims else None
+        unit = m.dim ** -0.5
+        raw = hops.decay_memory(proj, turns, logits, w.gates_bias, m.gate_cap, w.decay, st["recurrent"], st.get("peak"),
+                                self._rows(self.rec_o, t, width), m.heads, m.dim, m.vdim, unit if m.gated else 1.0, 1.0 if m.gated else unit, si,
+                                blocks=h.dtype == torch.bfloat16, scratch=lambda name, shape: self._scratch(name, shape, torch.float32))
+        attn = self._rows(self.attn, t, pad8(width))
+        if pad8(width) != width:
+            attn[:, width:].zero_()    # the buffer is shared with layers of other widths
+        hops.head_rmsnorm(raw, w.norm, self.cfg.norm_eps, attn, m.heads, m.vdim, gate=proj[:, m.gate_col:m.gate_col + width],
+                          gate_act="sigmoid" if m.gated else "silu")
+        hops.linear(attn, w.o, y)
+
     def _experts(self, f: MoeSpec, w: MoeWeights, h):
         t = h.shape[0]
         logits = self._rows(self.ab, t, pad8(f.logits))
         hops.linear(h, w.router, logits[:, : f.logits], f32_out=True)
         out = moe_ops.routed_experts(h, logits[:, : f.experts], w.up, w.down, self.moe_ws, f.top, Act(f.act, f.limit), w.half, f.groups, f.keep,
-                                     f.renormalize, w.bias)
+                                     f.renormalize, w.bias, f.score, f.group_best)
         if w.shared_up is not None:
             y = self.y[:t]
             self._mlp(h, w.shared_up, w.shared_down, Act(f.act, f.shared_limit), w.shared_half, y[:, : self.cfg.hidden])
@@ -868,16 +1070,27 @@ class HybridModel:
         cur, nxt = self.xs[0][:t], self.xs[-1][:t]
         h, y = self.h[:t], self.y[:t]
         wp = pad8(cfg.hidden)
-        hops.embed_streams(si.token_ids, w.embed, cur, w.embed_norm, self.loop_in[:t, wp:wp + cfg.hidden] if cfg.loop is not None else None)
+        hops.embed_streams(si.token_ids, w.embed, cur, w.embed_norm, self.loop_in[:t, wp:wp + cfg.hidden] if cfg.loop is not None else None,
+                           cfg.embed_scale)
+        for freq, table in self.turns.values():
+            hops.turn_table(si.positions, freq, table[:t])
         written, out = None, None      # connection whose sublayer output the residual still has to take in, and that output
         entered, add = None, None      # residual that a pass begins with instead of ``cur``, and what is still to be added to it
 
-        def step(conn, norm, h, gather=None, conv=None, state=None, **kw):
+        def gated(y, source, weight, gate_bias, bias=None):
+            """What the residual takes of a sublayer's output: gates over the normed rows the sublayer (before its convolution) came from."""
+            if weight is None:
+                return y
+            gate = self.res_gate[:t]
+            hops.linear(source, weight, gate[:, : cfg.hidden])
+            return GatedRows(y, gate, gate_bias, bias)
+
+        def step(conn, norm, h, gather=None, conv=None, state=None, plain=None, **kw):
             nonlocal cur, nxt, entered, add
             if conv is not None:
                 fold = entered is not None or out is not None
                 hops.norm_conv_step(entered if entered is not None else cur[:, 0], nxt[:, 0] if fold else None, out, add, norm, conv, state, h, si,
-                                    self.factor if t > self.FUSED_ROWS else None)
+                                    self.factor if t > self.FUSED_ROWS else None, plain)
                 entered = add = None
                 if fold:
                     cur, nxt = nxt, cur
@@ -905,7 +1118,8 @@ class HybridModel:
                 if lw.conv1 is None:   # the passes that follow work on the stream itself
                     torch.add(entered, add, out=cur[:, 0])
                     entered = add = None
-            step(lw.hc1, lw.norm1, h, conv=lw.conv1, state=state.get("input1"),
+            plain = self.plain[:t] if lw.gate1 is not None and lw.conv1 is not None else None
+            step(lw.hc1, lw.norm1, h, conv=lw.conv1, state=state.get("input1"), plain=plain,
                  **({"shift": lw.shift, "prev": state["shift"]} if lw.shift is not None else {}))
             if self.capture is not None and ri > 0 and not begins:
                 self.capture.append(cur.sum(1))
@@ -915,9 +1129,13 @@ class HybridModel:
                 self._delta(ri, m, lw.mixer, h, y[:, : cfg.hidden], si)
             elif isinstance(m, DiffSpec):
                 self._diff(ri, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
+            elif isinstance(m, TiedSpec):
+                self._tied(ri, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
+            elif isinstance(m, MemorySpec):
+                self._memory(ri, m, lw.mixer, h, y[:, : cfg.hidden], si)
             else:
                 self._latent(ri, m, lw.mixer, h, y[:, : cfg.hidden], kv, si)
-            written, out = lw.hc1, y
+            written, out = lw.hc1, gated(y, h if plain is None else plain, lw.gate1, lw.gate1_bias, getattr(lw.mixer, "o_bias", None))
             if spec.mlp is None:
                 continue
             step(lw.hc2, lw.norm2, h, conv=lw.conv2, state=state.get("input2"))
@@ -926,6 +1144,7 @@ class HybridModel:
                 out = self._experts(spec.mlp, lw.moe, h)
             else:
                 self._mlp(h, lw.gate_up, lw.down, lw.act, lw.half, y[:, : cfg.hidden])
+            out = gated(out, h, lw.gate2, lw.gate2_bias)
         if self.capture is not None:
             step(None, None, None)
             self.capture.append(cur.sum(1))

@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from . import decoder, dezudra, fizesun, hybrid, rilelorn
+from . import decoder, dezudra, fizesun, hybrid, midisun, rilelorn
 from .config import DecoderConfig
 
 
@@ -38,7 +38,8 @@ FAMILIES = (
 )
 ARCHITECTURES = {a.name: a for a in (Architecture("Rilelorn", rilelorn.read_config, rilelorn.load_weights, "hybrid"),
                                      Architecture("Dezudra", dezudra.read_config, dezudra.load_weights, "delta"),
-                                     Architecture("Fizesun", fizesun.read_config, fizesun.load_weights, "latent_moe"))}
+                                     Architecture("Fizesun", fizesun.read_config, fizesun.load_weights, "latent_moe"),
+                                     Architecture("Midisun", midisun.read_config, midisun.load_weights, "memory"))}
 
 
 def family_of(cfg) -> Family:

@@ -1,9 +1,9 @@
 """Ops of models that choose a mixer per layer (csrc/kernels/hybrid.cu, recurrent.cu, latent_attention.cu, short_conv.cu,
-delta_rule.cu, diff_attention.cu): hyper-connected residual streams with a Dynamic-Tanh norm and token shift, one residual stream
-with RMS norms before (and behind) a sublayer and convolutions of what a sublayer reads, HGRN2 and gated delta-rule recurrences
-over per-sequence state, short causal convolutions, attention over paged latents with or without a rotated part, differential
-attention over paged keys and values, products with activations, batched per-head products, and the fp32 matrix product of the
-32-bit engine.
+delta_rule.cu, diff_attention.cu, decay_memory.cu, tied_attention.cu): hyper-connected residual streams with a Dynamic-Tanh norm and
+token shift, one residual stream with RMS norms before (and behind) a sublayer, convolutions of what a sublayer reads and gates of
+what it adds, HGRN2, gated delta-rule and one-decay-per-head recurrences over per-sequence state, short causal convolutions, attention
+over paged latents with or without a rotated part, over paged keys that are the values too, differential attention over paged keys
+and values, products with activations, batched per-head products, and the fp32 matrix product of the 32-bit engine.
 
 CUDA tensors run the kernels; CPU tensors run the statements in :mod:`onnx_genai_b200.ops.reference`, as the other ops do.
 ``si`` is the step's :class:`~onnx_genai_b200.models.decoder.StepInputs`.
@@ -19,7 +19,7 @@ from . import PAGE, gemm
 
 P, I, F, L = _native.P, _native.I, _native.F, _native.L
 _native.register("ogb_hyper_step", [P] * 13 + [I] * 6 + [P] * 5 + [I] * 4 + [P, P])
-_native.register("ogb_embed_streams", [P, P, P, I, I, I, I, P, F, P, I, I, P, P])
+_native.register("ogb_embed_streams", [P, P, P, I, I, I, I, P, F, F, P, I, I, P, P])
 _native.register("ogb_latent_append", [P, I, I, P, F, P, P, I, I, I, L, P, P, P] + [I] * 7 + [P, P])
 _native.register("ogb_latent_attention", [P] * 9 + [I] * 10 + [L, I, F, I, P, P, P, I, P, P])
 _native.register("ogb_paged_prefill_chunks_bf16", [P] * 9 + [I] * 4 + [L] + [I] * 9 + [F, I, P, P])
@@ -30,9 +30,15 @@ _native.register("ogb_latent_set_tc", [I])
 _native.register("ogb_gemm_bf16_paged", [P, P, P, I, I, I, I, I, I, P, P])
 _native.register("ogb_hgrn2_state_rows", [I])
 _native.register("ogb_hgrn2", [P] * 5 + [I] * 5 + [P] * 3 + [I] * 5 + [P, P, I, P, P])
-_native.register("ogb_head_rmsnorm", [P, P, F, P, I, I, I, I, I, P, I, I, P])
-_native.register("ogb_norm_step", [P] * 10 + [F] + [I] * 8 + [L, I, P, P])
-_native.register("ogb_norm_conv_step", [P] * 13 + [F] + [I] * 9 + [L] + [P] * 5 + [I] * 4 + [P, P])
+_native.register("ogb_head_rmsnorm", [P, P, I, F, P, I, I, I, I, I, P, I, I, I, P])
+_native.register("ogb_norm_step", [P] * 13 + [F] + [I] * 10 + [L, I, P, P])
+_native.register("ogb_norm_conv_step", [P] * 17 + [F] + [I] * 12 + [L] + [P] * 5 + [I] * 4 + [P, P])
+_native.register("ogb_turn_table", [P, P, P, I, I, P])
+_native.register("ogb_tied_append", [P, I, P, P, P, F, F, P, I, P, P, L, L] + [I] * 6 + [P, P])
+_native.register("ogb_tied_attention", [P] * 11 + [I] * 3 + [L, L] + [I] * 8 + [F, I, P, P, P, I, P, P])
+_native.register("ogb_tied_set_tc", [I])
+_native.register("ogb_decay_memory", [P, I, P, I, P, I, P, F] + [P] * 4 + [I] * 4 + [F, F] + [P] * 5 + [I] * 4 + [P, I, P, P])
+_native.register("ogb_decay_block_floats", [I] * 4)
 _native.register("ogb_conv_rope_append", [P, I, P, P, P, I, P, I, P, P, P, L, L] + [I] * 8 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_conv_unit_gates", [P, I, P, P, I, P, I] + [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, P])
 _native.register("ogb_delta_rule", [P] * 5 + [I] * 4 + [P] * 5 + [I] * 4 + [P, I, P, P])
@@ -64,9 +70,10 @@ class HyperConnection:
 
 @dataclass
 class RmsNorm:
-    """x / sqrt(mean(x^2) + eps) w; w fp32."""
+    """x / sqrt(mean(x^2) + eps) w; w fp32.  ``groups``: equal consecutive parts of x, each over its own root mean square."""
     w: torch.Tensor
     eps: float
+    groups: int = 1
 
 
 @dataclass
@@ -78,6 +85,16 @@ class ExpertRows:
     weight: torch.Tensor
     shared: torch.Tensor | None = None
     gate: torch.Tensor | None = None
+
+
+@dataclass
+class GatedRows:
+    """A sublayer's output (``rows``: a row per token, or :class:`ExpertRows`; plus ``bias`` [W] fp32 where given) that reaches the residual
+    times sigmoid(gate + gate_bias), coordinate by coordinate: gate [T, ld], gate_bias [W] fp32."""
+    rows: object
+    gate: torch.Tensor
+    gate_bias: torch.Tensor
+    bias: torch.Tensor | None = None
 
 
 @dataclass(frozen=True)
@@ -194,12 +211,12 @@ def act_linear(a, w, act, out):
 
 
 @_timed("embed_streams")
-def embed_streams(ids, table, x, norm: RmsNorm | None = None, copy=None):
-    """Every stream of row t of x [T, S, W] (fp32) becomes the embedding of ids[t], normed where ``norm`` is given; so does row t of
-    ``copy`` [T, W]."""
+def embed_streams(ids, table, x, norm: RmsNorm | None = None, copy=None, scale=1.0):
+    """Every stream of row t of x [T, S, W] (fp32) becomes the embedding of ids[t] times ``scale``, normed where ``norm`` is given; so does
+    row t of ``copy`` [T, W]."""
     t, s, w = x.shape
     if not x.is_cuda:
-        rows = table[ids[:t].long()].float()
+        rows = table[ids[:t].long()].float() * scale
         if norm is not None:
             rows = reference.rms(rows, norm.w, norm.eps)
         x.copy_(rows[:, None, :].expand(-1, s, -1))
@@ -207,7 +224,7 @@ def embed_streams(ids, table, x, norm: RmsNorm | None = None, copy=None):
             copy.copy_(rows)
         return x
     rc = _native.load().ogb_embed_streams(ids.data_ptr(), table.data_ptr(), x.data_ptr(), t, s, w, table.shape[0], _ptr(norm.w if norm is not None else None),
-                                          float(norm.eps) if norm is not None else 0.0, _ptr(copy), copy.stride(0) if copy is not None else 0,
+                                          float(norm.eps) if norm is not None else 0.0, float(scale), _ptr(copy), copy.stride(0) if copy is not None else 0,
                                           _ELEM[table.dtype], status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_embed_streams")
     launch_counts["embed_streams"] += 1
@@ -382,32 +399,41 @@ def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si, segment=None, scratc
 
 
 @_timed("head_rmsnorm")
-def head_rmsnorm(x, w, eps, out, heads, n, gate=None):
-    """RMS norm of each head's n columns of x [T, ld] (fp32) with one shared weight, times silu(gate) [T, heads * n] where given."""
+def head_rmsnorm(x, w, eps, out, heads, n, gate=None, gate_act="silu"):
+    """RMS norm of each head's n columns of x [T, ld] (fp32) with a weight (None, [n] for every head, or [heads * n]), times silu or sigmoid
+    (``gate_act``) of gate [T, heads * n] where given."""
     if not x.is_cuda:
-        out[:, : heads * n] = reference.head_rmsnorm(x, w, eps, heads, n, out.dtype, gate)
+        out[:, : heads * n] = reference.head_rmsnorm(x, w, eps, heads, n, out.dtype, gate, gate_act)
         return out
-    rc = _native.load().ogb_head_rmsnorm(x.data_ptr(), w.data_ptr(), float(eps), out.data_ptr(), x.shape[0], heads, n, x.stride(0),
-                                         out.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, _ELEM[out.dtype], _stream())
+    step = n if w is not None and w.numel() != n else 0
+    rc = _native.load().ogb_head_rmsnorm(x.data_ptr(), _ptr(w), step, float(eps), out.data_ptr(), x.shape[0], heads, n, x.stride(0), out.stride(0),
+                                         _ptr(gate), gate.stride(0) if gate is not None else 0, int(gate_act == "sigmoid"), _ELEM[out.dtype], _stream())
     _native.check(rc, "ogb_head_rmsnorm")
     launch_counts["head_rmsnorm"] += 1
     return out
 
 
 def _sublayer(y):
-    """(output rows, kernel pointers, (k, ldy, lds, ldg), expert rows) of a sublayer's output: rows, :class:`ExpertRows` or None."""
+    """(output rows, kernel pointers, (k, ldy, lds, ldg, ldr), expert rows) of a sublayer's output: rows, :class:`ExpertRows`,
+    :class:`GatedRows` of either, or None."""
+    scaled, ldr = (0, 0, 0), 0
+    if isinstance(y, GatedRows):
+        scaled, ldr = (_ptr(y.bias), y.gate.data_ptr(), y.gate_bias.data_ptr()), y.gate.stride(0)
+        assert y.gate.dtype == (y.rows.rows if isinstance(y.rows, ExpertRows) else y.rows).dtype
+        y = y.rows
     if not isinstance(y, ExpertRows):
-        return y, (_ptr(y), 0, 0, 0, 0), (1, y.stride(0) if y is not None else 0, 0, 0), 0
+        return y, (_ptr(y), 0, 0, 0, 0, *scaled), (1, y.stride(0) if y is not None else 0, 0, 0, ldr), 0
     shared = (_ptr(y.shared), _ptr(y.gate))
     assert y.shared is None or (y.shared.dtype == y.rows.dtype and y.gate.dtype == torch.float32)
     lds, ldg = (y.shared.stride(0), y.gate.stride(0)) if y.shared is not None else (0, 0)
-    return y.rows, (y.rows.data_ptr(), y.pos.data_ptr(), y.weight.data_ptr(), *shared), (y.pos.shape[1], y.rows.stride(0), lds, ldg), y.rows.shape[0]
+    return (y.rows, (y.rows.data_ptr(), y.pos.data_ptr(), y.weight.data_ptr(), *shared, *scaled), (y.pos.shape[1], y.rows.stride(0), lds, ldg, ldr),
+            y.rows.shape[0])
 
 
 @_timed("norm_step")
 def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
     """x [T, W] fp32 += post(y) (None: y as it is); h = norm(x) (None: x).  ``y``: rows of the last sublayer's output, :class:`ExpertRows`,
-    or None.  ``gather``: h gets the rows it names only, and x stays as it is."""
+    :class:`GatedRows`, or None.  ``gather``: h gets the rows it names only, and x stays as it is."""
     rows = h.shape[0] if h is not None else x.shape[0]
     if not x.is_cuda:
         new = reference.norm_step(x, y, post)
@@ -416,15 +442,15 @@ def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
         else:
             new = new[gather.long()]
         if h is not None:
-            h[:, : x.shape[1]] = (reference.rms(new, norm.w, norm.eps) if norm is not None else new).to(h.dtype)
+            h[:, : x.shape[1]] = (reference.rms(new, norm.w, norm.eps, norm.groups) if norm is not None else new).to(h.dtype)
         return h
-    src, ptrs, (k, ldy, lds, ldg), y_rows = _sublayer(y)
+    src, ptrs, (k, ldy, lds, ldg, ldr), y_rows = _sublayer(y)
     eps = norm.eps if norm is not None else post.eps if post is not None else 0.0
-    assert post is None or post.eps == eps
+    assert post is None or (post.eps == eps and post.groups == 1)
     assert x.is_contiguous()
     rc = _native.load().ogb_norm_step(
         x.data_ptr(), *ptrs, _ptr(post.w if post is not None else None), _ptr(norm.w if norm is not None else None), _ptr(h), _ptr(gather), float(eps), rows,
-        x.shape[0], x.shape[1], k, ldy, lds, ldg, h.stride(0) if h is not None else 0, y_rows, _ELEM[h.dtype if h is not None else src.dtype],
+        x.shape[0], x.shape[1], norm.groups if norm is not None else 1, k, ldy, lds, ldg, ldr, h.stride(0) if h is not None else 0, y_rows, _ELEM[h.dtype if h is not None else src.dtype],
         status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_norm_step")
     launch_counts["norm_step"] += 1
@@ -432,10 +458,10 @@ def norm_step(x, y, post: RmsNorm | None, norm: RmsNorm | None, h, gather=None):
 
 
 @_timed("norm_conv_step")
-def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si, factor=None):
+def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si, factor=None, plain=None):
     """x_out [T, W] = x_in + y + add (y as for :func:`norm_step`, add [W] or None); h_t = sum_j conv[j] n_(t - taps + 1 + j) along every sequence
     with n = norm(x_out), conv [taps, W] fp32, state [slots, taps - 1, W] advanced.  Where nothing is added x_out may be None.
-    ``factor`` [>= T] fp32 scratch: the pass runs as two kernels, which steps of many rows gain from."""
+    ``factor`` [>= T * norm groups] fp32 scratch: the pass runs as two kernels, which steps of many rows gain from.  ``plain`` [T, ld] gets n."""
     t, w = x_in.shape
     if not x_in.is_cuda:
         new = reference.norm_step(x_in, y, None)
@@ -443,13 +469,16 @@ def norm_conv_step(x_in, x_out, y, add, norm: RmsNorm, conv, state, h, si, facto
             new = new + add
         if x_out is not None:
             x_out.copy_(new)
-        h[:, :w] = reference.short_conv(reference.rms(new, norm.w, norm.eps), conv, state, si).to(h.dtype)
+        n = reference.rms(new, norm.w, norm.eps, norm.groups)
+        if plain is not None:
+            plain[:, :w] = n.to(plain.dtype)
+        h[:, :w] = reference.short_conv(n, conv, state, si).to(h.dtype)
         return h
-    src, ptrs, (k, ldy, lds, ldg), y_rows = _sublayer(y)
+    src, ptrs, (k, ldy, lds, ldg, ldr), y_rows = _sublayer(y)
+    assert plain is None or plain.dtype == h.dtype
     rc = _native.load().ogb_norm_conv_step(
-        x_in.data_ptr(), _ptr(x_out), *ptrs, _ptr(add), norm.w.data_ptr(), conv.data_ptr(), state.data_ptr(), h.data_ptr(), _ptr(factor), float(norm.eps), t, w,
-        conv.shape[0], k,
-        x_in.stride(0), ldy, lds, ldg, h.stride(0), y_rows, *_rows_args(si, state), _ELEM[h.dtype], status_word().data_ptr(), _stream())
+        x_in.data_ptr(), _ptr(x_out), *ptrs, _ptr(add), norm.w.data_ptr(), conv.data_ptr(), state.data_ptr(), h.data_ptr(), _ptr(plain), _ptr(factor),
+        float(norm.eps), t, w, norm.groups, conv.shape[0], k, x_in.stride(0), ldy, lds, ldg, ldr, h.stride(0), plain.stride(0) if plain is not None else 0, y_rows, *_rows_args(si, state), _ELEM[h.dtype], status_word().data_ptr(), _stream())
     _native.check(rc, "ogb_norm_conv_step")
     launch_counts["norm_conv_step"] += 1 if factor is None else 2
     return h
@@ -545,3 +574,100 @@ def diff_attention(q, out, pool, si, hq, hkv, d, dv, dp, vp, scale, lam, eps, ga
 def set_diff_tc(on: bool) -> bool:
     """Switch the tensor-core kernels of differential attention (on by default); returns the old setting."""
     return bool(_native.load().ogb_diff_set_tc(int(on)))
+
+
+@_timed("turn_table")
+def turn_table(positions, freq, out):
+    """Cosine and sine of position x freq (fp64 [n], angles reduced in double) to out [T, n, 2] fp32."""
+    t = out.shape[0]
+    if not out.is_cuda:
+        reference.turn_table(positions[:t], freq, out)
+        return out
+    assert out.is_contiguous() and freq.dtype == torch.float64
+    rc = _native.load().ogb_turn_table(positions.data_ptr(), freq.data_ptr(), out.data_ptr(), t, freq.numel(), _stream())
+    _native.check(rc, "ogb_turn_table")
+    launch_counts["turn_table"] += 1
+    return out
+
+
+@_timed("decay_memory")
+def decay_memory(row, turns, logits, bias, cap, decay, state, peak, out, heads, dim, vdim, q_scale, k_scale, si, blocks=False, scratch=None):
+    """Advance the matrix memories S <- a S + b k v^T of the step's rows and read o = S^T q out: row [T, ld] holds the projections
+    [heads dim | heads dim | heads vdim] of q, k and v; q and k are rotated by ``turns`` (:func:`turn_table`; dimension i with i + n) where
+    given, and scaled.  ``decay`` [2, heads] fp32 (decays, their logarithms): a = decay, b = 1.  Else ``logits`` [T, (input | forget) heads] fp32 plus
+    ``bias``, capped at +-``cap``, are the gates of a memory with a running maximum (``peak`` [slots, heads]) and a normalizer (the state's
+    last column), over which o is divided.  state [slots, heads, vdim (+ 1), state_rows(dim)] fp32 in place, out [T, heads * vdim] fp32.
+    ``blocks``: prompts in blocks of 64 tokens on the tensor cores; ``scratch(name, shape)`` provides fp32 scratch for them."""
+    if not row.is_cuda:
+        reference.decay_memory(row, turns, logits, bias, cap, decay, state, peak, out, heads, dim, vdim, q_scale, k_scale, si)
+        return out
+    assert out.is_contiguous() and (logits is None) != (decay is None)
+    lib, work = _native.load(), None
+    per_block = lib.ogb_decay_block_floats(heads, dim, vdim, int(logits is not None)) if blocks and si.num_prefill_seqs else 0
+    if per_block:
+        n = si.num_tiles * per_block
+        work = scratch("decay_blocks", (n,)) if scratch is not None else torch.empty(n, dtype=torch.float32, device=row.device)
+    rc = lib.ogb_decay_memory(
+        row.data_ptr(), row.stride(0), _ptr(turns), turns.shape[1] if turns is not None else 0, _ptr(logits), logits.stride(0) if logits is not None else 0,
+        _ptr(bias), float(cap), _ptr(decay), state.data_ptr(), _ptr(peak), out.data_ptr(), heads, dim, vdim, state.shape[3], float(q_scale),
+        float(k_scale), si.ctx_len.data_ptr(), si.state_slot.data_ptr(), si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), si.num_decode,
+        si.num_prefill_seqs, si.num_tiles, state.shape[0], _ptr(work), _ELEM[row.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_decay_memory")
+    launch_counts["decay_memory"] += 1
+    return out
+
+
+def tied_page_elems(hkv, dp):
+    """Elements of a page of keys that are values too: [hkv][16][dp] keys, and 16 fp32 factors (in room for two elements each)."""
+    return hkv * PAGE * dp + 2 * PAGE
+
+
+@_timed("tied_append")
+def tied_append(row, q_bias, k_bias, q_gain, eps, factor, q, pool, slots, hq, hkv, d, dp):
+    """Rows [T, hq d | hkv d] of projected queries and keys, biases added: queries over their root mean square (of the whole projection)
+    times ``q_gain`` to q [T, hq * dp]; keys as they are to their slots of pool [pages, elements], with ``factor`` over their root mean
+    square beside them -- the keys' norm and its weight reach a score through that number and the query's gain."""
+    t = row.shape[0]
+    if not row.is_cuda:
+        reference.tied_append(row, q_bias, k_bias, q_gain, eps, factor, q, pool, slots, hq, hkv, d, dp)
+        return
+    assert pool.dtype == row.dtype == q.dtype
+    rc = _native.load().ogb_tied_append(row.data_ptr(), row.stride(0), _ptr(q_bias), _ptr(k_bias), q_gain.data_ptr(), float(eps), float(factor), q.data_ptr(),
+                                        q.stride(0), pool.data_ptr(), slots.data_ptr(), backed_pages(pool) * PAGE, pool.stride(0), t, hq, hkv, d, dp,
+                                        _ELEM[row.dtype], status_word().data_ptr(), _stream())
+    _native.check(rc, "ogb_tied_append")
+    launch_counts["tied_append"] += 1
+
+
+@_timed("tied_attention")
+def tied_attention(q, out, pool, si, hq, hkv, d, dp, cap=0.0, slope=None, sink=None, window=0, gate=None, splits=1, part_o=None, part_ml=None,
+                   counters=None):
+    """Attention over pages of :func:`tied_append`, whose keys are the values: s = (q . k) factor, capped to cap tanh(s) where ``cap`` > 0
+    (the factor then holds 1 / cap), less slope[head] x distance; softmax with exp(sink[head]) in the denominator; every head's output
+    times the sigmoid of gate [T, hq].  ``window`` > 0: a query sees its last ``window`` keys.  slope, sink: fp32 [hq] or None."""
+    if not q.is_cuda:
+        reference.tied_attention(q, out, pool, si, hq, hkv, d, dp, cap, slope, sink, window, gate)
+        return out
+    lib, st = _native.load(), status_word().data_ptr()
+    nd, npf, t = si.num_decode, si.num_prefill_seqs, si.num_tokens
+    assert gate is None or gate.dtype == q.dtype
+    tail = (si.page_table.shape[1], backed_pages(pool), pool.stride(0), hq, hkv, d, dp, q.stride(0), out.stride(0), gate.stride(0) if gate is not None else 0,
+            int(window), float(cap))
+    if nd > 0:
+        rc = lib.ogb_tied_attention(q.data_ptr(), out.data_ptr(), pool.data_ptr(), si.page_table.data_ptr(), si.ctx_len.data_ptr(), 0, 0, 0, _ptr(gate),
+                                    _ptr(slope), _ptr(sink), nd, 0, *tail, int(splits), _ptr(part_o), _ptr(part_ml), _ptr(counters), _ELEM[q.dtype], st,
+                                    _stream())
+        _native.check(rc, "ogb_tied_attention")
+        launch_counts["tied_decode"] += 1
+    if npf > 0:
+        rc = lib.ogb_tied_attention(q[nd:].data_ptr(), out[nd:].data_ptr(), pool.data_ptr(), si.page_table[nd:].data_ptr(), si.ctx_len[nd:].data_ptr(),
+                                    si.cu_q.data_ptr(), si.tile_seq.data_ptr(), si.tile_q0.data_ptr(), _ptr(gate[nd:] if gate is not None else None),
+                                    _ptr(slope), _ptr(sink), t - nd, si.num_tiles, *tail, 1, 0, 0, 0, _ELEM[q.dtype], st, _stream())
+        _native.check(rc, "ogb_tied_attention")
+        launch_counts["tied_prefill"] += 1
+    return out
+
+
+def set_tied_tc(on: bool) -> bool:
+    """Switch the tensor-core kernels of attention over keys that are values (on by default); returns the old setting."""
+    return bool(_native.load().ogb_tied_set_tc(int(on)))

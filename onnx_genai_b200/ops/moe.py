@@ -11,7 +11,7 @@ _native.register("ogb_moe_permute", [P] * 8 + [I] * 5 + [P])
 _native.register("ogb_moe_gather_rows", [P, P, P, P, I, I, I, P])
 _native.register("ogb_moe_combine", [P, P, P, P, I, I, I, I, P])
 _native.register("ogb_grouped_gemm_bf16", [P] * 5 + [I] * 7 + [P, P])
-_native.register("ogb_moe_route_grouped", [P, P, P, P] + [I] * 7 + [P])
+_native.register("ogb_moe_route_grouped", [P, P, P, P] + [I] * 9 + [P])
 _native.register("ogb_moe_gather_bytes", [P, P, P, P, I, I, I, P])
 _native.register("ogb_grouped_gemm_act", [P] * 5 + [I] * 9 + [F, F, I, P, P])
 _native.register("ogb_grouped_gemm_f32", [P] * 5 + [I] * 8 + [F, F, P])
@@ -108,9 +108,9 @@ def relu2_experts(h, logits, up, down, ws: MoEWorkspace, k, groups=1, keep=1, re
     return routed_experts(h, logits, up, down, ws, k, "relu2", 0, groups, keep, renormalize)
 
 
-def routed_experts(h, logits, up, down, ws: MoEWorkspace, k, act, half=0, groups=1, keep=1, renormalize=False, bias=None):
-    """Experts down(act(up h)), routed by softmax scores over fp32 ``logits`` [T, experts] plus ``bias`` with the experts in ``groups`` of
-    which ``keep`` stay (``reference.moe_route``).  ``act``: ops.hybrid.Act or its name; up [E, inter, ld(h)], for a gated one the gate and
+def routed_experts(h, logits, up, down, ws: MoEWorkspace, k, act, half=0, groups=1, keep=1, renormalize=False, bias=None, score="softmax", group_best=1):
+    """Experts down(act(up h)), routed by scores of fp32 ``logits`` [T, experts] and ``bias`` with the experts in ``groups`` of which ``keep``
+    stay (``score``, ``group_best``: see ``reference.moe_route``).  ``act``: ops.hybrid.Act or its name; up [E, inter, ld(h)], for a gated one the gate and
     up rows of every expert packed with half-width ``half`` [E, 2 inter, ld(h)]; down [E, hidden, inter].  Returns the tokens' outputs as
     :class:`~.hybrid.ExpertRows`: the residual step sums them."""
     from .hybrid import ExpertRows, act_mul_packed, as_act
@@ -119,7 +119,7 @@ def routed_experts(h, logits, up, down, ws: MoEWorkspace, k, act, half=0, groups
     t, e = h.shape[0], up.shape[0]
     inter, hidden = down.shape[2], down.shape[1]
     if not h.is_cuda:
-        ids, w = reference.moe_route(logits, k, renormalize, groups, keep, bias)
+        ids, w = reference.moe_route(logits, k, renormalize, groups, keep, bias, score, group_best)
         rows = torch.zeros(t * k, ws.ys.shape[1], dtype=h.dtype)
         flat = ids.reshape(-1)
         for x in range(e):
@@ -133,7 +133,7 @@ def routed_experts(h, logits, up, down, ws: MoEWorkspace, k, act, half=0, groups
     f32 = h.dtype == torch.float32
     with timed_region("moe_route_permute"):
         rc = lib.ogb_moe_route_grouped(logits.data_ptr(), bias.data_ptr() if bias is not None else 0, ws.topk_ids.data_ptr(), ws.topk_w.data_ptr(), t, e, k,
-                                       int(renormalize), logits.stride(0), groups, keep, s)
+                                       int(renormalize), logits.stride(0), groups, keep, int(score == "sigmoid"), group_best, s)
         _native.check(rc, "ogb_moe_route_grouped")
         rc = lib.ogb_moe_permute(ws.topk_ids.data_ptr(), ws.counts.data_ptr(), ws.offsets.data_ptr(), ws.cursor.data_ptr(), ws.sorted_route.data_ptr(),
                                  ws.route_pos.data_ptr(), ws.tile_tab.data_ptr(), ws.meta.data_ptr(), t, k, 0, e, ws.max_mtiles, s)

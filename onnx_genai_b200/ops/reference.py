@@ -332,17 +332,25 @@ def quantize_w4(w, block=32, symmetric=True):
     return q, scales, zp
 
 
-def moe_route(router_logits, k, renormalize=True, groups=1, keep=1, bias=None):
-    """``groups`` > 1: only experts of the ``keep`` groups of neighbours whose best expert scores highest can be chosen."""
+def moe_route(router_logits, k, renormalize=True, groups=1, keep=1, bias=None, score="softmax", group_best=1):
+    """``groups`` > 1: only experts of the ``keep`` groups of neighbours whose ``group_best`` best experts score highest together can be
+    chosen.  ``score`` "softmax": of logits plus ``bias``; "sigmoid": of the logits, and ``bias`` corrects the scores that are compared
+    but not the weights."""
     logits = router_logits.float()
-    probs = torch.softmax(logits if bias is None else logits + bias, dim=-1)
+    if score == "sigmoid":
+        probs = torch.sigmoid(logits)
+        ranked = probs if bias is None else probs + bias
+    else:
+        ranked = probs = torch.softmax(logits if bias is None else logits + bias, dim=-1)
     if groups > 1:
-        best = probs.view(probs.shape[0], groups, -1).amax(-1)
+        best = ranked.view(probs.shape[0], groups, -1)
+        best = torch.topk(best, min(group_best, best.shape[-1]), dim=-1).values.sum(-1)
         kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, torch.topk(best, keep, dim=-1).indices, True)
-        probs = probs.masked_fill(~kept.repeat_interleave(probs.shape[1] // groups, 1), -1.0)
-    w, ids = torch.topk(probs, k, dim=-1)
+        ranked = ranked.masked_fill(~kept.repeat_interleave(probs.shape[1] // groups, 1), float("-inf"))
+    ids = torch.topk(ranked, k, dim=-1).indices
+    w = probs.gather(1, ids)
     if renormalize:
-        w = w / w.sum(-1, keepdim=True)
+        w = w / (w.sum(-1, keepdim=True) + (1e-20 if score == "sigmoid" else 0.0))
     return ids.to(torch.int32), w
 
 
@@ -425,21 +433,34 @@ def hgrn2(qfv, bias, low, state, out, heads, dim, vdim, si):
         state[slot, :, :, :dim] = s
 
 
-def rms(x, w, eps):
+def rms(x, w, eps, groups=1):
+    """``groups``: equal consecutive parts with a root mean square each."""
+    if groups > 1:
+        parts = x.unflatten(-1, (groups, -1))
+        return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2) * w
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
 
 
-def head_rmsnorm(x, w, eps, heads, n, out_dtype=None, gate=None):
-    y = rms(x[:, : heads * n].float().view(-1, heads, n), w, eps).reshape(x.shape[0], heads * n)
+def head_rmsnorm(x, w, eps, heads, n, out_dtype=None, gate=None, gate_act="silu"):
+    """w: None, [n] for every head, or [heads * n]."""
+    y = x[:, : heads * n].float().view(-1, heads, n)
+    y = rms(y, 1.0 if w is None else w if w.numel() == n else w.view(heads, n), eps).reshape(x.shape[0], heads * n)
     if gate is not None:
-        y = y * torch.nn.functional.silu(gate.float())
+        y = y * (torch.sigmoid(gate.float()) if gate_act == "sigmoid" else torch.nn.functional.silu(gate.float()))
     return y.to(out_dtype or x.dtype)
 
 
 def norm_step(x, y, post):
-    """x + post(y) for rows of y, or the weighted sum of a token's expert rows (ops.hybrid.ExpertRows); y as it is without post."""
+    """x + post(y) for rows of y, or the weighted sum of a token's expert rows (ops.hybrid.ExpertRows); y as it is without post.
+    ops.hybrid.GatedRows: those times the sigmoid of a gate, coordinate by coordinate."""
     if y is None:
         return x
+    if hasattr(y, "gate_bias"):
+        w = x.shape[1]
+        inner = norm_step(torch.zeros_like(x), y.rows, None)
+        if y.bias is not None:
+            inner = inner + y.bias
+        return x + inner * torch.sigmoid(y.gate[:, :w].float() + y.gate_bias)
     if not torch.is_tensor(y):
         rows = (y.rows[y.pos.long()].float() * y.weight[:, :, None]).sum(1)
         if y.shared is not None:
@@ -447,7 +468,7 @@ def norm_step(x, y, post):
             rows = rows[:, :w] + torch.sigmoid(y.gate)[:, None] * y.shared[:, :w].float()
         y = rows
     y = y[:, : x.shape[1]].float()
-    return x + (rms(y, post.w, post.eps) if post is not None else y)
+    return x + (rms(y, post.w, post.eps, post.groups) if post is not None else y)
 
 
 def short_conv(u, w, state, si):
@@ -586,3 +607,97 @@ def latent_attention(q, out, pool, si, heads, rank, scale, window, vrank=None, g
         if gate is not None:
             o = o * torch.sigmoid(gate[base:base + n].float())[..., None]
         out[base * heads:(base + n) * heads, :vrank] = o.reshape(n * heads, vrank).to(out.dtype)
+
+
+# ------------------------------------------------------------------------------------------
+# attention whose values are its keys, and recurrences with one decay per head (ops/hybrid.py)
+# ------------------------------------------------------------------------------------------
+def tied_pages(pool, hkv, dp):
+    """Views of a pool of pages [hkv][16][dp] | [16] factors: keys [pages, hkv, 16, dp], factors [pages, 16] fp32."""
+    n = hkv * PAGE * dp
+    tail = PAGE * 4 // pool.element_size()
+    return pool[:, :n].view(-1, hkv, PAGE, dp), pool.view(torch.float32)[:, n * pool.element_size() // 4:(n + tail) * pool.element_size() // 4]
+
+
+def tied_append(row, q_bias, k_bias, q_gain, eps, factor, q, pool, slots, hq, hkv, d, dp):
+    t = row.shape[0]
+    qs = row[:, : hq * d].float() + q_bias
+    ks = row[:, hq * d:(hq + hkv) * d].float() + k_bias
+    q[:t].view(t, hq, dp)[..., :d] = rms(qs, q_gain, eps).view(t, hq, d).to(q.dtype)
+    live = slots[:t] >= 0
+    page, off = (slots[:t][live] // PAGE).long(), (slots[:t][live] % PAGE).long()
+    keys, factors = tied_pages(pool, hkv, dp)
+    keys[page, :, off, :d] = ks.view(t, hkv, d)[live].to(pool.dtype)
+    factors[page, off] = (torch.rsqrt(ks.pow(2).mean(-1) + eps) * factor)[live]
+
+
+def tied_attention(q, out, pool, si, hq, hkv, d, dp, cap, slope, sink, window, gate):
+    keys, factors = tied_pages(pool, hkv, dp)
+    for e, base, n, start, _ in step_entries(si):
+        ctx = start + n
+        lo = max(0, start - window + 1) if window > 0 else 0
+        j = torch.arange(lo, ctx)
+        dist = torch.arange(start, ctx)[:, None] - j[None, :]
+        seen = dist >= 0
+        if window > 0:
+            seen &= dist < window
+        page, off = si.page_table[e].long()[j // PAGE], j % PAGE
+        k = keys[page, :, off, :d].float().repeat_interleave(hq // hkv, 1)
+        s = torch.einsum("nhd,khd->hnk", q[base:base + n].view(n, hq, dp)[..., :d].float(), k) * factors[page, off]
+        if cap > 0:
+            s = cap * torch.tanh(s)
+        if slope is not None:
+            s = s - slope[:, None, None] * dist
+        s = s.masked_fill(~seen, float("-inf"))
+        if sink is not None:
+            s = torch.cat([s, sink[:, None, None].expand(-1, n, 1)], -1)
+        p = torch.softmax(s, -1)[..., : j.numel()]
+        o = torch.einsum("hnk,khd->nhd", p, k)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[base:base + n, :hq].float())[..., None]
+        out[base:base + n].view(n, hq, dp)[..., :d] = o.to(out.dtype)
+
+
+def turn_table(positions, freq, out):
+    """out [T, len(freq), 2] fp32: cosine and sine of position x freq."""
+    a = positions.double()[:, None] * freq[None, :]
+    out[: a.shape[0], :, 0], out[: a.shape[0], :, 1] = torch.cos(a).float(), torch.sin(a).float()
+
+
+def memory_gates(logits, bias, cap, heads):
+    """(log input gate, log forget gate) [T, heads] of logits [T, >= 2 heads] (input | forget)."""
+    z = cap * torch.tanh((logits[:, : 2 * heads].float() + bias) / cap)
+    return z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:])
+
+
+def decay_memory(row, turns, logits, bias, cap, decay, state, peak, out, heads, dim, vdim, q_scale, k_scale, si):
+    t, hd = row.shape[0], heads * dim
+    q, k = row[:, :hd].float().view(t, heads, dim), row[:, hd:2 * hd].float().view(t, heads, dim)
+    v = row[:, 2 * hd:2 * hd + heads * vdim].float().view(t, heads, vdim)
+    if turns is not None:
+        half = turns.shape[1]
+        c, s = turns[:t, None, :, 0], turns[:t, None, :, 1]
+        turn = lambda x: torch.cat([x[..., :half] * c - x[..., half:2 * half] * s, x[..., half:2 * half] * c + x[..., :half] * s, x[..., 2 * half:]], -1)
+        q, k = turn(q), turn(k)
+    q, k = q * q_scale, k * k_scale
+    gated = logits is not None
+    if gated:
+        gi, gf = memory_gates(logits, bias, cap, heads)
+        v = torch.cat([v, torch.ones(t, heads, 1)], -1)              # one more value column holds the normalizer
+    for _, base, n, start, slot in step_entries(si):
+        s = state[slot, :, :, :dim].clone() if start > 0 else torch.zeros(heads, v.shape[2], dim)
+        m = peak[slot].clone() if gated and start > 0 else torch.zeros(heads)
+        for r in range(base, base + n):
+            if gated:
+                new = torch.maximum(gf[r] + m, gi[r])
+                keep, take, m = torch.exp(gf[r] + m - new), torch.exp(gi[r] - new), new
+            else:
+                keep, take = decay[0], torch.ones(heads)
+            s = s * keep[:, None, None] + (take[:, None] * v[r])[:, :, None] * k[r][:, None, :]
+            o = torch.einsum("hvd,hd->hv", s, q[r])
+            if gated:
+                o = o[:, :vdim] / (torch.maximum(o[:, vdim].abs(), torch.exp(-m)) + 1e-6)[:, None]
+            out[r, : heads * vdim] = o.reshape(-1)
+        state[slot, :, :, :dim] = s
+        if gated:
+            peak[slot] = m

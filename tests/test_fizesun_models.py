@@ -427,7 +427,7 @@ def test_chosen_experts_share_a_softmax_of_their_own(device):
     bias = torch.tensor([0.0, 0.0, 0.0, 0.0, -20.0, 30.0], device="cuda")
     ids, w = torch.zeros(2, 4, dtype=torch.int32, device="cuda"), torch.zeros(2, 4, device="cuda")
     lib = ops._native.load()
-    assert lib.ogb_moe_route_grouped(z.data_ptr(), bias.data_ptr(), ids.data_ptr(), w.data_ptr(), 2, 6, 4, 1, 6, 1, 1, torch.cuda.current_stream().cuda_stream) == 0
+    assert lib.ogb_moe_route_grouped(z.data_ptr(), bias.data_ptr(), ids.data_ptr(), w.data_ptr(), 2, 6, 4, 1, 6, 1, 1, 0, 1, torch.cuda.current_stream().cuda_stream) == 0
     for t in range(2):
         want, ww = O.choose((z + bias)[t].cpu(), 4)
         assert ids[t].tolist() == want
