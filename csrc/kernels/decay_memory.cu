@@ -104,6 +104,7 @@ __global__ void __launch_bounds__(256, DP == 256 ? 1 : 2) memory_step_kernel(Mem
   if (GATED) {                                           // every block keeps the normalizer and the maximum; the first one stores them
     load(p.V, n);
     if (threadIdx.x == 0) sm[kMemTok] = it.fresh ? 0.f : p.peak[static_cast<size_t>(it.slot) * p.heads + head];
+    __syncwarp();
     if (gridDim.x > 1) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   }
   for (int t0 = 0; t0 < it.n; t0 += kMemTok) {
@@ -208,6 +209,7 @@ __global__ void __launch_bounds__(256, DP == 256 ? 1 : 2) memory_step_kernel(Mem
   for (int c = 0; c < CPT; ++c)
     if (col0 + lc + c < p.V) store(col0 + lc + c, s[c]);
   if (GATED) {
+    __syncwarp();
     if (gridDim.x > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");      // every block has read them
     if (blockIdx.x == 0 && threadIdx.x < 16) store(p.V, n);
     if (blockIdx.x == 0 && threadIdx.x == 0) p.peak[static_cast<size_t>(it.slot) * p.heads + head] = sm[kMemTok];

@@ -141,7 +141,6 @@ tied_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
   const int kvh = blockIdx.y % p.hkv, col0 = blockIdx.y / p.hkv * OC;       // output columns of this CTA
   const int kv_lo = p.window > 0 ? max(0, rw.pos_first - p.window + 1) : 0;
   const int b_begin = kv_lo / BN, nblk = (rw.pos_last + BN) / BN - b_begin;  // last visible key is pos_last
-  const int n_out = min(OC, (p.dp - col0 + 15) / 16 * 16), k_steps = (p.dp + 15) / 16;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -207,7 +206,7 @@ tied_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
     // MMAs of one thread execute in issue order: S_{j+2}, issued after PV_j, cannot overwrite the P_j it has yet to read.
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc_bf16(kTtBM, BN);
-      const uint32_t idesc_o = make_idesc_bf16(kTtBM, n_out) | (1u << 16);   // B is MN-major
+      constexpr uint32_t idesc_o = make_idesc_bf16(kTtBM, OC) | (1u << 16);   // B is MN-major
       bool ok = fa_wait(&bars->q_full, 0, abort_flag);
       auto issue_pv = [&](int t) -> bool {
         const int buf = t & 1, st = t % ST;
@@ -231,8 +230,7 @@ tied_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
         for (int h = 0; h < Cfg::kChunks; ++h) {
           const uint64_t da = make_kmajor_sw128_desc(sq + h * kTtBM * 128), db = make_kmajor_sw128_desc(sk + h * BN * 128);
 #pragma unroll
-          for (int k = 0; k < 4; ++k)
-            if (4 * h + k < k_steps) umma_f16(tmem_base + Cfg::kColS + buf * BN, da + 2 * k, db + 2 * k, idesc_s, (h | k) != 0 ? 1u : 0u);
+          for (int k = 0; k < 4; ++k) umma_f16(tmem_base + Cfg::kColS + buf * BN, da + 2 * k, db + 2 * k, idesc_s, (h | k) != 0 ? 1u : 0u);
         }
         umma_commit(&bars->s_full[buf]);
         if (it >= 1 && !issue_pv(it - 1)) ok = false;
