@@ -123,19 +123,21 @@ def main():
     ap.add_argument("--hybrid", action="store_true", help="instead of the headline workload: prefill / decode throughput of the hybrid decoder "
                     "(Rilelorn layers) beside a dense decoder of equal size, and every kernel against its roofline (table on stderr, JSON on stdout)")
     ap.add_argument("--hybrid-sizes", default="small,medium,large")
-    ap.add_argument("--hybrid-design", default="rilelorn", choices=["rilelorn", "dezudra", "fizesun"], help="which hybrid decoder: Rilelorn layers "
-                    "beside a dense GQA decoder, Dezudra layers beside a GQA decoder with experts, or Fizesun layers beside Rilelorn's latent layers")
+    ap.add_argument("--hybrid-design", default="rilelorn", choices=["rilelorn", "dezudra", "fizesun", "midisun"], help="which hybrid decoder: "
+                    "Rilelorn layers beside a dense GQA decoder, Dezudra layers beside a GQA decoder with experts, Fizesun layers beside Rilelorn's "
+                    "latent layers, or Midisun layers beside Dezudra layers")
     ap.add_argument("--hybrid-json", default="")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
     if args.hybrid:
-        from onnx_genai_b200.bench import delta_bench, hybrid_bench, loop_bench
+        from onnx_genai_b200.bench import delta_bench, hybrid_bench, loop_bench, memory_bench
 
         sampler = ClockSampler(0)
         sampler.start()
         t0 = time.perf_counter()
-        designs = {"rilelorn": (hybrid_bench, "a GQA decoder"), "dezudra": (delta_bench, "a GQA decoder"), "fizesun": (loop_bench, "a decoder of latent layers")}
+        designs = {"rilelorn": (hybrid_bench, "a GQA decoder"), "dezudra": (delta_bench, "a GQA decoder"), "fizesun": (loop_bench, "a decoder of latent layers"),
+                   "midisun": (memory_bench, "a decoder of delta-rule layers")}
         bench, beside = designs[args.hybrid_design]
         doc = bench.main(args.hybrid_sizes.split(","), args.hybrid_json)
         t1 = time.perf_counter()

@@ -260,7 +260,8 @@ static int dispatch_memory_step(const MemoryParams& p, int items, cudaStream_t s
 // g are kept in double, so that differences of large sums stay good to fp32.  Products run on mma.sync tf32, fp32 factors split in
 // two (values are bf16, which tf32 holds as they are).
 // ------------------------------------------------------------------------------------------------------
-constexpr int kMbTok = 64, kMbCols = 64;                          // tokens of a block, value columns of a CTA's tile
+constexpr int kMbThreads = 256;
+constexpr int kMbTok = 64, kMbCols = 64;                          // tokens of a block, value columns of a tile
 constexpr int kMbVP = kMbCols + 8, kMbPP = kMbTok + 4;            // row pitches of values and of the products of queries and keys
 
 struct MemoryBlocks {
@@ -294,142 +295,183 @@ struct MbTile {
   }
 };
 
-// rotated, scaled queries or keys of the block's rows to dst [64][pitch]; zeros behind the head's channels and the last token
-template <typename T>
-OGB_DEVICE void mb_channels(const MemoryParams& p, const MbTile& b, const T* src, float scale, float* dst, int DP, int pitch) {
+// rotated, scaled queries or keys of the block's rows to dst [64][pitch]; zeros behind the head's channels and the last token.  A thread
+// has the same four channels in all its rows, whose loads are under way together.
+template <typename T, int DP>
+OGB_DEVICE void mb_channels(const MemoryParams& p, const MbTile& b, const T* src, float scale, float* dst, int pitch) {
   const bool vec = ((p.D | p.half) & 3) == 0 && (p.ld & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(T) - 1)) == 0;
-  if (vec) {
-    for (int i = threadIdx.x; i < kMbTok * DP / 4; i += blockDim.x) {
-      const int t = i / (DP / 4), d = i % (DP / 4) * 4;
-      float x[4] = {0.f, 0.f, 0.f, 0.f};
-      if (t < b.nt && d < p.D) {
-        const T* s = src + (b.row0 + t) * p.ld;
-        load_vec<4>(s + d, x);
-        if (d < 2 * p.half) {
-          const bool low = d < p.half;
-          const float2* cs = p.turns + (b.row0 + t) * p.half + (low ? d : d - p.half);
-          float y[4];
-          load_vec<4>(s + (low ? d + p.half : d - p.half), y);
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const float2 c = cs[j];
-            x[j] = low ? x[j] * c.x - y[j] * c.y : x[j] * c.x + y[j] * c.y;
-          }
-        }
-      }
-      *reinterpret_cast<float4*>(dst + t * pitch + d) = make_float4(x[0] * scale, x[1] * scale, x[2] * scale, x[3] * scale);
+  if (!vec) {
+    for (int i = threadIdx.x; i < kMbTok * DP; i += kMbThreads) {
+      const int t = i / DP, d = i % DP;
+      dst[t * pitch + d] = t < b.nt && d < p.D ? memory_channel<T>(p, src + (b.row0 + t) * p.ld, static_cast<int>(b.row0) + t, d) * scale : 0.f;
     }
     return;
   }
-  for (int i = threadIdx.x; i < kMbTok * DP; i += blockDim.x) {
-    const int t = i / DP, d = i % DP;
-    dst[t * pitch + d] = t < b.nt && d < p.D ? memory_channel<T>(p, src + (b.row0 + t) * p.ld, static_cast<int>(b.row0) + t, d) * scale : 0.f;
-  }
-}
-
-// value columns v0 .. v0 + 63 of the block's rows to dst [64][kMbVP]
-template <typename T>
-OGB_DEVICE void mb_values(const MemoryParams& p, const MbTile& b, int head, int v0, float* dst) {
-  const T* src = static_cast<const T*>(p.row) + 2 * p.heads * p.D + static_cast<size_t>(head) * p.V + v0;
-  const bool vec = ((p.V | p.ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(T) - 1)) == 0;
-  for (int i = threadIdx.x; i < kMbTok * kMbCols / 4; i += blockDim.x) {
-    const int t = i / (kMbCols / 4), c = i % (kMbCols / 4) * 4;
-    float x[4] = {0.f, 0.f, 0.f, 0.f};
-    if (t < b.nt) {
-      const T* s = src + (b.row0 + t) * p.ld + c;
-      if (vec && v0 + c < p.V) load_vec<4>(s, x);
-      else
+  constexpr int kStep = kMbThreads / (DP / 4), kBatch = 4;         // rows between a thread's, rows at a time
+  const int d = threadIdx.x % (DP / 4) * 4, t0 = threadIdx.x / (DP / 4);
+  const bool live = d < p.D, turn = d < 2 * p.half, low = d < p.half;
+  const int dx = live ? d : 0, dy = turn ? (low ? d + p.half : d - p.half) : dx;
+  const float2* cs = p.turns + (turn ? (low ? d : d - p.half) : 0);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (v0 + c + j < p.V) x[j] = to_f32<T>(s[j]);
-    }
-    *reinterpret_cast<float4*>(dst + t * kMbVP + c) = make_float4(x[0], x[1], x[2], x[3]);
-  }
-}
-
-// c of every token of the block (threads below 64 return theirs in c, g as above; tokens behind the last have no weight: g = -inf).  `sg` is
-// shared scratch [128] doubles and holds the g's on return.
-OGB_DEVICE void mb_sums(const MemoryParams& p, const MbTile& b, int head, double* sg, double& c, double& g) {
-  const int t = threadIdx.x;
-  float gi = 0.f;
-  if (t < kMbTok) {
-    float f = 0.f;
-    if (t < b.nt) {
-      if (p.logits != nullptr) {
-        const float2 x = memory_log_gates(p, static_cast<int>(b.row0) + t, head);
-        gi = x.x; f = x.y;
-      } else {
-        f = p.decay[p.heads + head];
+  for (int j0 = 0; j0 < kMbTok / kStep; j0 += kBatch) {
+    float x[kBatch][4], y[kBatch][4];
+    float4 c[kBatch][2];
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j) {
+      const size_t row = b.row0 + min(t0 + (j0 + j) * kStep, b.nt - 1);
+      load_vec<4>(src + row * p.ld + dx, x[j]);
+      if (turn) {
+        load_vec<4>(src + row * p.ld + dy, y[j]);
+        c[j][0] = *reinterpret_cast<const float4*>(cs + row * p.half);
+        c[j][1] = *reinterpret_cast<const float4*>(cs + row * p.half + 2);
       }
     }
-    sg[kMbTok + t] = static_cast<double>(f);
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j) {
+      const int t = t0 + (j0 + j) * kStep;
+      if (turn) {
+        const float co[4] = {c[j][0].x, c[j][0].z, c[j][1].x, c[j][1].z}, si[4] = {c[j][0].y, c[j][0].w, c[j][1].y, c[j][1].w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) x[j][k] = low ? x[j][k] * co[k] - y[j][k] * si[k] : x[j][k] * co[k] + y[j][k] * si[k];
+      }
+      const float f = live && t < b.nt ? scale : 0.f;
+      *reinterpret_cast<float4*>(dst + t * pitch + d) = make_float4(x[j][0] * f, x[j][1] * f, x[j][2] * f, x[j][3] * f);
+    }
   }
-  __syncthreads();
-  if (t < kMbTok) {
-    c = 0.0;
-    for (int j = 0; j <= t; ++j) c += sg[kMbTok + j];
-    g = t < b.nt ? static_cast<double>(gi) - c : -INFINITY;
-    sg[t] = g;
-  }
-  __syncthreads();
 }
 
-template <typename T, int DP>
-__global__ void __launch_bounds__(256) memory_write_kernel(MemoryParams p, MemoryBlocks bl) {
-  constexpr int kPitch = DP + 8, NT = DP / 16;
-  extern __shared__ __align__(16) uint8_t mb_smem[];
-  double* sg = reinterpret_cast<double*>(mb_smem);                // [128]
-  float* sw = reinterpret_cast<float*>(sg + 2 * kMbTok);          // [64] weights
-  float* sv = sw + kMbTok;                                        // [64][kMbVP]
-  float* sk = sv + kMbTok * kMbVP;                                // [64][kPitch]
-  MbTile b;
-  if (!b.set(p, bl)) return;
-  const int head = blockIdx.y, v0 = blockIdx.z * kMbCols, VS = p.columns();
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, tq = lane & 3;
-  double c = 0.0, g = 0.0;
-  mb_sums(p, b, head, sg, c, g);
-  mb_channels<T>(p, b, static_cast<const T*>(p.row) + static_cast<size_t>(p.heads + head) * p.D, p.k_scale, sk, DP, kPitch);
-  mb_values<T>(p, b, head, v0, sv);
-  if (tid < kMbTok) {
-    double top = sg[b.nt - 1];                                    // without gates: -c of the last token
-    if (p.logits != nullptr)
-      for (int j = 0; j < b.nt - 1; ++j) top = fmax(top, sg[j]);
-    sw[tid] = tid < b.nt ? expf(static_cast<float>(g - top)) : 0.f;
-    if (tid == b.nt - 1 && blockIdx.z == 0) bl.num[b.block * p.heads + head] = make_float4(static_cast<float>(c), static_cast<float>(c + top), 0.f, 0.f);
-  }
-  __syncthreads();
-  const int m = warp & 3, d0 = (warp >> 2) * (DP / 2);
-  float* u = bl.u + (b.block * p.heads + head) * static_cast<size_t>(VS) * DP;
-  float acc[NT][4] = {};
-#pragma unroll 2
-  for (int k = 0; k < kMbTok / 8; ++k) {
-    const int s0 = 8 * k + tq, s1 = s0 + 4, v = 16 * m + gr;
-    const float a[4] = {sv[s0 * kMbVP + v], sv[s0 * kMbVP + v + 8], sv[s1 * kMbVP + v], sv[s1 * kMbVP + v + 8]};
-    const float w0 = sw[s0], w1 = sw[s1];
-    float lo[4];
-    bool exact = sizeof(T) == 2;                                  // a bf16 value is a tf32 one
-    if (!exact) {
+// value columns v0 .. v0 + 63 of the block's rows to dst [64][pitch]
+template <typename T>
+OGB_DEVICE void mb_values(const MemoryParams& p, const MbTile& b, int head, int v0, float* dst, int pitch) {
+  const T* src = static_cast<const T*>(p.row) + 2 * p.heads * p.D + static_cast<size_t>(head) * p.V + v0;
+  const bool vec = ((p.V | p.ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(T) - 1)) == 0;
+  constexpr int kRows = kMbTok * kMbCols / 4 / kMbThreads, kStep = kMbThreads / (kMbCols / 4);
+  const int c = threadIdx.x % (kMbCols / 4) * 4, t0 = threadIdx.x / (kMbCols / 4);
+  float x[kRows][4];
 #pragma unroll
-      for (int x = 0; x < 4; ++x) lo[x] = a[x] - tf32_cut(a[x]).x;
-    }
+  for (int k = 0; k < kRows; ++k) {
+    const T* s = src + (b.row0 + min(t0 + k * kStep, b.nt - 1)) * p.ld;
+    if (vec) {
+      load_vec<4>(s + (v0 + c < p.V ? c : 0), x[k]);
+    } else {
 #pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      const int d = d0 + 8 * n + gr;
-      const float2 b0 = tf32_cut(w0 * sk[s0 * kPitch + d]), b1 = tf32_cut(w1 * sk[s1 * kPitch + d]);
-      mma_tf32(acc[n], a, b0.x, b1.x);
-      mma_tf32(acc[n], a, b0.y, b1.y);
-      if (!exact) mma_tf32(acc[n], lo, b0.x, b1.x);
+      for (int j = 0; j < 4; ++j) x[k][j] = v0 + c + j < p.V ? to_f32<T>(s[c + j]) : 0.f;
     }
   }
 #pragma unroll
-  for (int n = 0; n < NT; ++n)
+  for (int k = 0; k < kRows; ++k) {
+    const bool live = t0 + k * kStep < b.nt && v0 + c < p.V;
+    *reinterpret_cast<float4*>(dst + (t0 + k * kStep) * pitch + c) =
+        live ? make_float4(x[k][0], x[k][1], x[k][2], x[k][3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+}
+
+// The sums of a block in the first warp's hands: lane l has tokens l and l + 32 (tokens behind the last have no weight: g = -inf).
+struct MbSums {
+  double c[2], g[2], top[2];   // c, g as above; the largest g up to the token (without gates: -c)
+  OGB_DEVICE void set(const MemoryParams& p, const MbTile& b, int head, double start) {
+    const int lane = threadIdx.x & 31;
+    const bool gated = p.logits != nullptr;
+    float in[2] = {0.f, 0.f};
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const int v = v0 + 16 * m + gr + 8 * h;
-      if (v < p.V) *reinterpret_cast<float2*>(u + static_cast<size_t>(v) * DP + d0 + 8 * n + 2 * tq) = make_float2(acc[n][2 * h], acc[n][2 * h + 1]);
+      const int t = lane + 32 * h;
+      c[h] = 0.0;
+      if (t >= b.nt) continue;
+      if (gated) {
+        const float2 x = memory_log_gates(p, static_cast<int>(b.row0) + t, head);
+        in[h] = x.x;
+        c[h] = static_cast<double>(x.y);
+      } else {
+        c[h] = static_cast<double>(p.decay[p.heads + head]);
+      }
     }
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const double x = __shfl_up_sync(0xffffffffu, c[h], o);
+        if (lane >= o) c[h] += x;
+      }
+    c[1] += __shfl_sync(0xffffffffu, c[0], 31);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      g[h] = lane + 32 * h < b.nt ? static_cast<double>(in[h]) - c[h] : -INFINITY;
+      top[h] = gated ? g[h] : -c[h];
+    }
+    if (!gated) return;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const double x = __shfl_up_sync(0xffffffffu, top[h], o);
+        if (lane >= o) top[h] = fmax(top[h], x);
+      }
+    top[0] = fmax(top[0], start);
+    top[1] = fmax(top[1], __shfl_sync(0xffffffffu, top[0], 31));
+  }
+};
+
+// 128 value columns of a block's writes: a warp has 16 of them and all channels of the keys, 128 at a time
+constexpr int kMwCols = 128, kMwVP = kMwCols + 8;
+template <int DP>
+struct MwCfg {
+  static constexpr int kPitch = DP + 8;
+  static constexpr int kSmemBytes = 4 * (kMbTok + kMbTok * kMwVP + kMbTok * kPitch);
+};
+
+template <typename T, int DP>
+__global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_write_kernel(MemoryParams p, MemoryBlocks bl) {
+  constexpr int kPitch = MwCfg<DP>::kPitch, DC = DP < 128 ? DP : 128, NT = DC / 8;
+  extern __shared__ __align__(16) uint8_t mb_smem[];
+  float* sw = reinterpret_cast<float*>(mb_smem);                  // [64] weights
+  float* sv = sw + kMbTok;                                        // [64][kMwVP]
+  float* sk = sv + kMbTok * kMwVP;                                // [64][kPitch]
+  MbTile b;
+  if (!b.set(p, bl)) return;
+  const int head = blockIdx.y, v0 = blockIdx.z * kMwCols, VS = p.columns();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, tq = lane & 3;
+  mb_channels<T, DP>(p, b, static_cast<const T*>(p.row) + static_cast<size_t>(p.heads + head) * p.D, p.k_scale, sk, kPitch);
+  mb_values<T>(p, b, head, v0, sv, kMwVP);
+  if (v0 + kMbCols < p.V) mb_values<T>(p, b, head, v0 + kMbCols, sv + kMbCols, kMwVP);
+  if (warp == 0) {
+    MbSums m;
+    m.set(p, b, head, -INFINITY);
+    const double c = __shfl_sync(0xffffffffu, m.c[1], 31), top = __shfl_sync(0xffffffffu, m.top[1], 31);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) sw[lane + 32 * h] = expf(static_cast<float>(m.g[h] - top));
+    if (lane == 0 && blockIdx.z == 0) bl.num[b.block * p.heads + head] = make_float4(static_cast<float>(c), static_cast<float>(c + top), 0.f, 0.f);
+  }
+  __syncthreads();
+  float* u = bl.u + (b.block * p.heads + head) * static_cast<size_t>(VS) * DP;
+  if (v0 + 16 * warp < p.V) {
+#pragma unroll 1
+    for (int d0 = 0; d0 < DP; d0 += DC) {
+      float acc[NT][4] = {};
+#pragma unroll 2
+      for (int k = 0; k < kMbTok / 8; ++k) {
+        const int s0 = 8 * k + tq, s1 = s0 + 4, v = 16 * warp + gr;
+        const float w0 = sw[s0], w1 = sw[s1];
+        const float a[4] = {sv[s0 * kMwVP + v], sv[s0 * kMwVP + v + 8], sv[s1 * kMwVP + v], sv[s1 * kMwVP + v + 8]};
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          const int d = d0 + 8 * n + gr;
+          const float2 b0 = tf32_cut(w0 * sk[s0 * kPitch + d]), b1 = tf32_cut(w1 * sk[s1 * kPitch + d]);
+          mma_tf32(acc[n], a, b0.x, b1.x);
+          mma_tf32(acc[n], a, b0.y, b1.y);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int v = v0 + 16 * warp + gr + 8 * h;
+          if (v < p.V) *reinterpret_cast<float2*>(u + static_cast<size_t>(v) * DP + d0 + 8 * n + 2 * tq) = make_float2(acc[n][2 * h], acc[n][2 * h + 1]);
+        }
+    }
+  }
   if (p.logits != nullptr && blockIdx.z == 0)
-    for (int d = tid; d < DP; d += 256) {
+    for (int d = tid; d < DP; d += kMbThreads) {
       float a = 0.f;
 #pragma unroll 8
       for (int s = 0; s < kMbTok; ++s) a = fmaf(sw[s], sk[s * kPitch + d], a);
@@ -437,10 +479,11 @@ __global__ void __launch_bounds__(256) memory_write_kernel(MemoryParams p, Memor
     }
 }
 
-__global__ void __launch_bounds__(256) memory_chain_kernel(MemoryParams p, MemoryBlocks bl) {
-  constexpr int kAhead = 4;
+constexpr int kMcThreads = 128;
+__global__ void __launch_bounds__(kMcThreads) memory_chain_kernel(MemoryParams p, MemoryBlocks bl) {
+  constexpr int kAhead = 8;                                       // blocks whose writes are under way
   MemoryItem it;
-  const int seq = blockIdx.z, head = blockIdx.y, quads = p.columns() * p.DP / 4, e = blockIdx.x * 256 + threadIdx.x;
+  const int seq = blockIdx.z, head = blockIdx.y, quads = p.columns() * p.DP / 4, e = blockIdx.x * kMcThreads + threadIdx.x;
   if (!it.set(p, p.sr.num_decode + seq) || e >= quads) return;
   const size_t b0 = mb_first_block(p.sr, seq), at = (b0 * p.heads + head), step = p.heads;
   const int blocks = (it.n + kMbTok - 1) / kMbTok;
@@ -449,47 +492,54 @@ __global__ void __launch_bounds__(256) memory_chain_kernel(MemoryParams p, Memor
   const bool gated = p.logits != nullptr;
   float m = gated && !it.fresh ? p.peak[static_cast<size_t>(it.slot) * p.heads + head] : 0.f;
   float4* u = reinterpret_cast<float4*>(bl.u) + at * quads + e;
-  for (int i0 = 0; i0 < blocks; i0 += kAhead) {
-    float4 w[kAhead], num[kAhead];
+  float4 w[kAhead];
+  float2 num[kAhead];
+  auto fetch = [&](int i, int j) {
+    w[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    num[j] = make_float2(0.f, 0.f);
+    if (i < blocks) {
+      w[j] = __ldcg(u + i * step * quads);
+      num[j] = __ldcg(reinterpret_cast<const float2*>(bl.num + at + i * step));
+    }
+  };
 #pragma unroll
-    for (int j = 0; j < kAhead; ++j)
-      if (i0 + j < blocks) {
-        w[j] = u[(i0 + j) * step * quads];
-        num[j] = bl.num[at + (i0 + j) * step];
-      }
+  for (int j = 0; j < kAhead; ++j) fetch(j, j);
+  for (int i0 = 0; i0 < blocks; i0 += kAhead)
 #pragma unroll
     for (int j = 0; j < kAhead; ++j) {
       if (i0 + j >= blocks) break;
-      u[(i0 + j) * step * quads] = s;
+      const float4 x = w[j];
+      const float2 y = num[j];
+      fetch(i0 + kAhead + j, j);
+      __stcg(u + (i0 + j) * step * quads, s);
       if (e == 0) bl.num[at + (i0 + j) * step].z = m;
       float a, f = 1.f;
       if (gated) {
-        const float next = fmaxf(num[j].x + m, num[j].y);
-        a = expf(num[j].x + m - next);
-        f = expf(num[j].y - next);
+        const float next = fmaxf(y.x + m, y.y);
+        a = expf(y.x + m - next);
+        f = expf(y.y - next);
         m = next;
       } else {
-        a = expf(num[j].x);
+        a = expf(y.x);
       }
-      s = make_float4(fmaf(f, w[j].x, a * s.x), fmaf(f, w[j].y, a * s.y), fmaf(f, w[j].z, a * s.z), fmaf(f, w[j].w, a * s.w));
+      s = make_float4(fmaf(f, x.x, a * s.x), fmaf(f, x.y, a * s.y), fmaf(f, x.z, a * s.z), fmaf(f, x.w, a * s.w));
     }
-  }
   *own = s;                                                       // the maximum is left by memory_read_kernel: others may yet read it here
 }
 
 template <int DP>
 struct MrCfg {
   static constexpr int kPitch = DP + 4;
-  static constexpr int kSmemBytes = 8 * (3 * kMbTok) + 4 * (2 * kMbTok * kPitch + kMbTok * kMbVP + kMbTok * kMbPP + 5 * kMbTok);
+  static constexpr int kSmemBytes = 8 * (2 * kMbTok) + 4 * (2 * kMbTok * kPitch + kMbTok * kMbVP + kMbTok * kMbPP + 5 * kMbTok);
 };
 
 template <typename T, int DP>
-__global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) memory_read_kernel(MemoryParams p, MemoryBlocks bl) {
+__global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_read_kernel(MemoryParams p, MemoryBlocks bl) {
   using Cfg = MrCfg<DP>;
   constexpr int kPitch = Cfg::kPitch;
   extern __shared__ __align__(16) uint8_t mb_smem[];
-  double* sg = reinterpret_cast<double*>(mb_smem);                // [128], [64] G
-  double* sG = sg + 2 * kMbTok;
+  double* sg = reinterpret_cast<double*>(mb_smem);                // [64] g, [64] G
+  double* sG = sg + kMbTok;
   float* se = reinterpret_cast<float*>(sG + kMbTok);              // [64] exp(m - G)
   float* sinv = se + kMbTok;                                      // [64] what read-outs are multiplied by
   float* sdot = sinv + kMbTok;                                    // [64] n . q
@@ -506,27 +556,27 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) memory_read_kernel(Mem
   const float* u = bl.u + (b.block * p.heads + head) * static_cast<size_t>(VS) * DP;
   const float m_in = gated ? bl.num[b.block * p.heads + head].z : 0.f;
   const T* src = static_cast<const T*>(p.row) + static_cast<size_t>(head) * p.D;
-  double c = 0.0, g = 0.0;
-  mb_sums(p, b, head, sg, c, g);
-  mb_channels<T>(p, b, src, p.q_scale, sq, DP, kPitch);
-  mb_channels<T>(p, b, src + p.heads * p.D, p.k_scale, sk, DP, kPitch);
-  float peak = 0.f;                                               // m_t of this thread's token
-  if (tid < kMbTok) {
-    double top = -c;
-    if (gated) {
-      top = static_cast<double>(m_in);
-      for (int j = 0; j <= tid; ++j) top = fmax(top, sg[j]);
-      peak = static_cast<float>(c + top);
+  mb_channels<T, DP>(p, b, src, p.q_scale, sq, kPitch);
+  mb_channels<T, DP>(p, b, src + p.heads * p.D, p.k_scale, sk, kPitch);
+  if (warp == 0) {
+    MbSums x;
+    x.set(p, b, head, static_cast<double>(m_in));
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = lane + 32 * h;
+      const float peak = gated ? static_cast<float>(x.c[h] + x.top[h]) : 0.f;      // m_t
+      sg[t] = x.g[h];
+      sG[t] = x.top[h];
+      se[t] = expf(static_cast<float>(static_cast<double>(m_in) - x.top[h]));
+      sinv[t] = expf(-peak);
+      // the last block of a chunk leaves the maximum for the next step
+      if (gated && t == b.nt - 1 && b.q0 + b.nt == b.len) {
+        const int slot = p.sr.state_slot[p.sr.num_decode + b.seq];
+        if (slot >= 0 && slot < p.sr.num_slots) p.peak[static_cast<size_t>(slot) * p.heads + head] = peak;
+      }
     }
-    sG[tid] = top;
-    se[tid] = expf(static_cast<float>(static_cast<double>(m_in) - top));
   }
   __syncthreads();
-  // the last block of a chunk leaves the maximum for the next step
-  if (gated && tid == b.nt - 1 && b.q0 + b.nt == b.len) {
-    const int slot = p.sr.state_slot[p.sr.num_decode + b.seq];
-    if (slot >= 0 && slot < p.sr.num_slots) p.peak[static_cast<size_t>(slot) * p.heads + head] = peak;
-  }
   const int m = warp & 3, half = warp >> 2;
   {
     float acc[4][4] = {};
@@ -560,17 +610,18 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) memory_read_kernel(Mem
   __syncthreads();
   if (tid < kMbTok) {
     float inv = 1.f;
-    if (gated) inv = 1.f / (fmaxf(fabsf(se[tid] * sdot[tid] + srow[tid] + srow[kMbTok + tid]), expf(-peak)) + 1e-6f);
+    if (gated) inv = 1.f / (fmaxf(fabsf(se[tid] * sdot[tid] + srow[tid] + srow[kMbTok + tid]), sinv[tid]) + 1e-6f);
     sinv[tid] = inv;
   }
   for (int v0 = 0; v0 < p.V; v0 += kMbCols) {
     if (v0 > 0) __syncthreads();
-    for (int i = tid; i < kMbCols * DP / 4; i += 256) {           // columns behind the last are read as the last and dropped
-      const int v = min(v0 + i / (DP / 4), VS - 1), d = i % (DP / 4) * 4;
+#pragma unroll
+    for (int j = 0; j < kMbCols * DP / 4 / kMbThreads; ++j) {     // columns behind the last are read as the last and dropped
+      const int i = j * kMbThreads + tid, v = min(v0 + i / (DP / 4), VS - 1), d = i % (DP / 4) * 4;
       cp_async<16>(sk + i / (DP / 4) * kPitch + d, u + static_cast<size_t>(v) * DP + d);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
-    mb_values<T>(p, b, head, v0, sv);
+    mb_values<T>(p, b, head, v0, sv, kMbVP);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     float o[4][4] = {};
@@ -589,15 +640,8 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) memory_read_kernel(Mem
 #pragma unroll
       for (int n = 0; n < 4; ++n) {
         const float w0 = sv[(8 * k + tq) * kMbVP + 32 * half + 8 * n + gr], w1 = sv[(8 * k + tq + 4) * kMbVP + 32 * half + 8 * n + gr];
-        if (sizeof(T) == 2) {
-          mma_tf32(o[n], hi, w0, w1);
-          mma_tf32(o[n], lo, w0, w1);
-        } else {
-          const float2 x0 = tf32_cut(w0), x1 = tf32_cut(w1);
-          mma_tf32(o[n], hi, x0.x, x1.x);
-          mma_tf32(o[n], lo, x0.x, x1.x);
-          mma_tf32(o[n], hi, x0.y, x1.y);
-        }
+        mma_tf32(o[n], hi, w0, w1);
+        mma_tf32(o[n], lo, w0, w1);
       }
     }
 #pragma unroll
@@ -621,7 +665,8 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) memory_read_kernel(Mem
 
 template <typename T, int DP>
 static int launch_memory_blocks(const MemoryParams& p, const MemoryBlocks& bl, int num_prefill, cudaStream_t stream) {
-  constexpr int write_bytes = 8 * 2 * kMbTok + 4 * (kMbTok + kMbTok * kMbVP + kMbTok * (DP + 8));
+  static_assert(sizeof(T) == 2, "values are taken for exact tf32 terms");
+  constexpr int write_bytes = MwCfg<DP>::kSmemBytes;
   static bool attr_set = false;
   if (!attr_set) {
     OGB_CUDA_CHECK(cudaFuncSetAttribute(memory_write_kernel<T, DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, write_bytes));
@@ -629,9 +674,9 @@ static int launch_memory_blocks(const MemoryParams& p, const MemoryBlocks& bl, i
     attr_set = true;
   }
   const int VS = p.V + (p.logits != nullptr), quads = VS * DP / 4;
-  memory_write_kernel<T, DP><<<dim3(bl.num_tiles, p.heads, (p.V + kMbCols - 1) / kMbCols), 256, write_bytes, stream>>>(p, bl);
-  memory_chain_kernel<<<dim3((quads + 255) / 256, p.heads, num_prefill), 256, 0, stream>>>(p, bl);
-  memory_read_kernel<T, DP><<<dim3(bl.num_tiles, p.heads), 256, MrCfg<DP>::kSmemBytes, stream>>>(p, bl);
+  memory_write_kernel<T, DP><<<dim3(bl.num_tiles, p.heads, (p.V + kMwCols - 1) / kMwCols), kMbThreads, write_bytes, stream>>>(p, bl);
+  memory_chain_kernel<<<dim3((quads + kMcThreads - 1) / kMcThreads, p.heads, num_prefill), kMcThreads, 0, stream>>>(p, bl);
+  memory_read_kernel<T, DP><<<dim3(bl.num_tiles, p.heads), kMbThreads, MrCfg<DP>::kSmemBytes, stream>>>(p, bl);
   return static_cast<int>(cudaGetLastError());
 }
 
