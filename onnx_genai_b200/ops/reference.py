@@ -621,13 +621,14 @@ def tied_pages(pool, hkv, dp):
 
 def tied_append(row, q_bias, k_bias, q_gain, eps, factor, q, pool, slots, hq, hkv, d, dp):
     t = row.shape[0]
-    qs = row[:, : hq * d].float() + q_bias
-    ks = row[:, hq * d:(hq + hkv) * d].float() + k_bias
-    q[:t].view(t, hq, dp)[..., :d] = rms(qs, q_gain, eps).view(t, hq, d).to(q.dtype)
+    qs, ks = row[:, : hq * d].float(), row[:, hq * d:(hq + hkv) * d].float()
+    qs, ks = qs if q_bias is None else qs + q_bias, ks if k_bias is None else ks + k_bias
+    pad = lambda x: torch.nn.functional.pad(x, (0, dp - d))
+    q[:t] = pad(rms(qs, q_gain, eps).view(t, hq, d)).to(q.dtype).reshape(t, -1)
     live = slots[:t] >= 0
     page, off = (slots[:t][live] // PAGE).long(), (slots[:t][live] % PAGE).long()
     keys, factors = tied_pages(pool, hkv, dp)
-    keys[page, :, off, :d] = ks.view(t, hkv, d)[live].to(pool.dtype)
+    keys[page, :, off] = pad(ks.view(t, hkv, d))[live].to(pool.dtype)
     factors[page, off] = (torch.rsqrt(ks.pow(2).mean(-1) + eps) * factor)[live]
 
 
@@ -655,7 +656,7 @@ def tied_attention(q, out, pool, si, hq, hkv, d, dp, cap, slope, sink, window, g
         o = torch.einsum("hnk,khd->nhd", p, k)
         if gate is not None:
             o = o * torch.sigmoid(gate[base:base + n, :hq].float())[..., None]
-        out[base:base + n].view(n, hq, dp)[..., :d] = o.to(out.dtype)
+        out[base:base + n] = torch.nn.functional.pad(o, (0, dp - d)).to(out.dtype).reshape(n, -1)
 
 
 def turn_table(positions, freq, out):
