@@ -255,14 +255,14 @@ static int dispatch_memory_step(const MemoryParams& p, int items, cudaStream_t s
 //   o_t = exp(m - G_t) S^T q_t + sum_{s <= t} exp(g_s - G_t) (q_t . k_s) v_s      (m = 0 without gates)
 //
 // and the block's own writes, up to a factor that the chain brings in, are  U = sum_s exp(g_s - g*) k_s v_s^T  with g* = max_s g_s
-// (without gates: -c_63).  Three kernels: all blocks write U side by side; a chain over the blocks of a sequence, elementwise in the
-// state, turns every U into the state its block starts with; all blocks read out side by side.  Exponents are never positive; c and
+// (without gates: -c_63).  A warp per block and head sums the gates up; all blocks write U side by side; a chain over the blocks of a
+// sequence, elementwise in the state, turns every U into the state its block starts with; all blocks read out side by side.  Exponents are never positive; c and
 // g are kept in double, so that differences of large sums stay good to fp32.  Products run on mma.sync tf32, fp32 factors split in
 // two (values are bf16, which tf32 holds as they are).
 // ------------------------------------------------------------------------------------------------------
 constexpr int kMbThreads = 256;
-constexpr int kMbTok = 64, kMbCols = 64;                          // tokens of a block, value columns of a tile
-constexpr int kMbVP = kMbCols + 8, kMbPP = kMbTok + 4;            // row pitches of values and of the products of queries and keys
+constexpr int kMbTok = 64;                                        // tokens of a block
+constexpr int kMbPP = kMbTok + 4;                                 // row pitch of the products of queries and keys
 
 struct MemoryBlocks {
   const int* tile_seq;     // 64-row tiles of the prefill chunks
@@ -270,6 +270,7 @@ struct MemoryBlocks {
   int num_tiles;
   float* u;                // [blocks, heads, VS, DP]: writes of the block, then the state it starts with
   float4* num;             // [blocks, heads]: sum of log decays, m* = c + g*, m at the block's start
+  double* sums;            // [blocks, heads, 3, 64], with gates: c, g, the largest g up to the token
 };
 
 OGB_DEVICE int mb_first_block(const StepRows& sr, int s) {        // blocks of the entries before prefill entry s
@@ -282,10 +283,10 @@ OGB_DEVICE int mb_first_block(const StepRows& sr, int s) {        // blocks of t
 struct MbTile {
   int seq, q0, len, nt;
   size_t row0, block;
-  OGB_DEVICE bool set(const MemoryParams& p, const MemoryBlocks& bl) {
+  OGB_DEVICE bool set(const MemoryParams& p, const MemoryBlocks& bl, int tile) {
     const StepRows& sr = p.sr;
-    seq = bl.tile_seq[blockIdx.x];
-    q0 = bl.tile_q0[blockIdx.x];
+    seq = bl.tile_seq[tile];
+    q0 = bl.tile_q0[tile];
     len = sr.cu_q[seq + 1] - sr.cu_q[seq];
     nt = min(kMbTok, len - q0);
     if (nt <= 0) return false;
@@ -295,33 +296,43 @@ struct MbTile {
   }
 };
 
-// rotated, scaled queries or keys of the block's rows to dst [64][pitch]; zeros behind the head's channels and the last token.  A thread
-// has the same four channels in all its rows, whose loads are under way together.
-template <typename T, int DP>
-OGB_DEVICE void mb_channels(const MemoryParams& p, const MbTile& b, const T* src, float scale, float* dst, int pitch) {
-  const bool vec = ((p.D | p.half) & 3) == 0 && (p.ld & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(T) - 1)) == 0;
+// Rotated, scaled channels of the block's rows to dst [64][pitch] -- of keys, or of queries and keys together (N = 2), which share their
+// rotations; zeros behind the head's channels and the last token.  A thread has the same four channels in all its rows, whose loads are
+// under way together.
+template <typename T, int DP, int N>
+OGB_DEVICE void mb_channels(const MemoryParams& p, const MbTile& b, const T* const (&src)[N], const float (&scale)[N], float* const (&dst)[N], int pitch) {
+  bool vec = ((p.D | p.half) & 3) == 0 && (p.ld & 3) == 0;
+#pragma unroll
+  for (int a = 0; a < N; ++a) vec = vec && (reinterpret_cast<uintptr_t>(src[a]) & (4 * sizeof(T) - 1)) == 0;
   if (!vec) {
-    for (int i = threadIdx.x; i < kMbTok * DP; i += kMbThreads) {
-      const int t = i / DP, d = i % DP;
-      dst[t * pitch + d] = t < b.nt && d < p.D ? memory_channel<T>(p, src + (b.row0 + t) * p.ld, static_cast<int>(b.row0) + t, d) * scale : 0.f;
-    }
+#pragma unroll
+    for (int a = 0; a < N; ++a)
+      for (int i = threadIdx.x; i < kMbTok * DP; i += kMbThreads) {
+        const int t = i / DP, d = i % DP;
+        dst[a][t * pitch + d] = t < b.nt && d < p.D ? memory_channel<T>(p, src[a] + (b.row0 + t) * p.ld, static_cast<int>(b.row0) + t, d) * scale[a] : 0.f;
+      }
     return;
   }
+  static_assert(sizeof(T) == 2, "four channels are two registers");
   constexpr int kStep = kMbThreads / (DP / 4), kBatch = 4;         // rows between a thread's, rows at a time
   const int d = threadIdx.x % (DP / 4) * 4, t0 = threadIdx.x / (DP / 4);
   const bool live = d < p.D, turn = d < 2 * p.half, low = d < p.half;
   const int dx = live ? d : 0, dy = turn ? (low ? d + p.half : d - p.half) : dx;
   const float2* cs = p.turns + (turn ? (low ? d : d - p.half) : 0);
+  const float sign = low ? -1.f : 1.f;
 #pragma unroll
   for (int j0 = 0; j0 < kMbTok / kStep; j0 += kBatch) {
-    float x[kBatch][4], y[kBatch][4];
+    uint2 x[kBatch][N], y[kBatch][N];
     float4 c[kBatch][2];
 #pragma unroll
     for (int j = 0; j < kBatch; ++j) {
       const size_t row = b.row0 + min(t0 + (j0 + j) * kStep, b.nt - 1);
-      load_vec<4>(src + row * p.ld + dx, x[j]);
+#pragma unroll
+      for (int a = 0; a < N; ++a) {
+        x[j][a] = *reinterpret_cast<const uint2*>(src[a] + row * p.ld + dx);
+        if (turn) y[j][a] = *reinterpret_cast<const uint2*>(src[a] + row * p.ld + dy);
+      }
       if (turn) {
-        load_vec<4>(src + row * p.ld + dy, y[j]);
         c[j][0] = *reinterpret_cast<const float4*>(cs + row * p.half);
         c[j][1] = *reinterpret_cast<const float4*>(cs + row * p.half + 2);
       }
@@ -329,90 +340,111 @@ OGB_DEVICE void mb_channels(const MemoryParams& p, const MbTile& b, const T* src
 #pragma unroll
     for (int j = 0; j < kBatch; ++j) {
       const int t = t0 + (j0 + j) * kStep;
-      if (turn) {
-        const float co[4] = {c[j][0].x, c[j][0].z, c[j][1].x, c[j][1].z}, si[4] = {c[j][0].y, c[j][0].w, c[j][1].y, c[j][1].w};
 #pragma unroll
-        for (int k = 0; k < 4; ++k) x[j][k] = low ? x[j][k] * co[k] - y[j][k] * si[k] : x[j][k] * co[k] + y[j][k] * si[k];
+      for (int a = 0; a < N; ++a) {
+        float2 x0 = unpack_bf16(x[j][a].x), x1 = unpack_bf16(x[j][a].y);
+        if (turn) {
+          const float2 y0 = unpack_bf16(y[j][a].x), y1 = unpack_bf16(y[j][a].y);
+          x0 = make_float2(x0.x * c[j][0].x + sign * (y0.x * c[j][0].y), x0.y * c[j][0].z + sign * (y0.y * c[j][0].w));
+          x1 = make_float2(x1.x * c[j][1].x + sign * (y1.x * c[j][1].y), x1.y * c[j][1].z + sign * (y1.y * c[j][1].w));
+        }
+        const float f = live && t < b.nt ? scale[a] : 0.f;
+        *reinterpret_cast<float4*>(dst[a] + t * pitch + d) = make_float4(x0.x * f, x0.y * f, x1.x * f, x1.y * f);
       }
-      const float f = live && t < b.nt ? scale : 0.f;
-      *reinterpret_cast<float4*>(dst + t * pitch + d) = make_float4(x[j][0] * f, x[j][1] * f, x[j][2] * f, x[j][3] * f);
     }
   }
 }
 
-// value columns v0 .. v0 + 63 of the block's rows to dst [64][pitch]
-template <typename T>
-OGB_DEVICE void mb_values(const MemoryParams& p, const MbTile& b, int head, int v0, float* dst, int pitch) {
-  const T* src = static_cast<const T*>(p.row) + 2 * p.heads * p.D + static_cast<size_t>(head) * p.V + v0;
-  const bool vec = ((p.V | p.ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(T) - 1)) == 0;
-  constexpr int kRows = kMbTok * kMbCols / 4 / kMbThreads, kStep = kMbThreads / (kMbCols / 4);
-  const int c = threadIdx.x % (kMbCols / 4) * 4, t0 = threadIdx.x / (kMbCols / 4);
+// NC value columns v0 .. of the block's rows: fetched to registers, stored to dst [64][PITCH]
+template <typename T, int NC, int PITCH>
+struct MbValues {
+  static constexpr int kRows = kMbTok * NC / 4 / kMbThreads, kStep = kMbThreads / (NC / 4);
   float x[kRows][4];
+  OGB_DEVICE void fetch(const MemoryParams& p, const MbTile& b, int head, int v0) {
+    const T* src = static_cast<const T*>(p.row) + 2 * p.heads * p.D + static_cast<size_t>(head) * p.V + v0;
+    const bool vec = ((p.V | p.ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(T) - 1)) == 0;
+    const int c = threadIdx.x % (NC / 4) * 4, t0 = threadIdx.x / (NC / 4);
 #pragma unroll
-  for (int k = 0; k < kRows; ++k) {
-    const T* s = src + (b.row0 + min(t0 + k * kStep, b.nt - 1)) * p.ld;
-    if (vec) {
-      load_vec<4>(s + (v0 + c < p.V ? c : 0), x[k]);
-    } else {
+    for (int k = 0; k < kRows; ++k) {
+      const int t = t0 + k * kStep;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) x[k][j] = v0 + c + j < p.V ? to_f32<T>(s[c + j]) : 0.f;
+      for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
+      if (t >= b.nt || v0 + c >= p.V) continue;
+      const T* s = src + (b.row0 + t) * p.ld + c;
+      if (vec) load_vec<4>(s, x[k]);
+      else
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (v0 + c + j < p.V) x[k][j] = to_f32<T>(s[j]);
     }
   }
+  OGB_DEVICE void store(float* dst) const {
+    const int c = threadIdx.x % (NC / 4) * 4, t0 = threadIdx.x / (NC / 4);
 #pragma unroll
-  for (int k = 0; k < kRows; ++k) {
-    const bool live = t0 + k * kStep < b.nt && v0 + c < p.V;
-    *reinterpret_cast<float4*>(dst + (t0 + k * kStep) * pitch + c) =
-        live ? make_float4(x[k][0], x[k][1], x[k][2], x[k][3]) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-}
-
-// The sums of a block in the first warp's hands: lane l has tokens l and l + 32 (tokens behind the last have no weight: g = -inf).
-struct MbSums {
-  double c[2], g[2], top[2];   // c, g as above; the largest g up to the token (without gates: -c)
-  OGB_DEVICE void set(const MemoryParams& p, const MbTile& b, int head, double start) {
-    const int lane = threadIdx.x & 31;
-    const bool gated = p.logits != nullptr;
-    float in[2] = {0.f, 0.f};
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int t = lane + 32 * h;
-      c[h] = 0.0;
-      if (t >= b.nt) continue;
-      if (gated) {
-        const float2 x = memory_log_gates(p, static_cast<int>(b.row0) + t, head);
-        in[h] = x.x;
-        c[h] = static_cast<double>(x.y);
-      } else {
-        c[h] = static_cast<double>(p.decay[p.heads + head]);
-      }
-    }
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const double x = __shfl_up_sync(0xffffffffu, c[h], o);
-        if (lane >= o) c[h] += x;
-      }
-    c[1] += __shfl_sync(0xffffffffu, c[0], 31);
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      g[h] = lane + 32 * h < b.nt ? static_cast<double>(in[h]) - c[h] : -INFINITY;
-      top[h] = gated ? g[h] : -c[h];
-    }
-    if (!gated) return;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const double x = __shfl_up_sync(0xffffffffu, top[h], o);
-        if (lane >= o) top[h] = fmax(top[h], x);
-      }
-    top[0] = fmax(top[0], start);
-    top[1] = fmax(top[1], __shfl_sync(0xffffffffu, top[0], 31));
+    for (int k = 0; k < kRows; ++k) *reinterpret_cast<float4*>(dst + (t0 + k * kStep) * PITCH + c) = make_float4(x[k][0], x[k][1], x[k][2], x[k][3]);
   }
 };
 
-// 128 value columns of a block's writes: a warp has 16 of them and all channels of the keys, 128 at a time
+// The sums of a block's gates: one warp, whose lane l has tokens l and l + 32 (tokens behind the last have no weight: g = -inf).
+__global__ void __launch_bounds__(256) memory_sums_kernel(MemoryParams p, MemoryBlocks bl) {
+  const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, tile = item / p.heads, head = item % p.heads;
+  MbTile b;
+  if (tile >= bl.num_tiles || !b.set(p, bl, tile)) return;
+  double c[2], g[2], top[2];
+  float in[2] = {0.f, 0.f};
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int t = lane + 32 * h;
+    c[h] = 0.0;
+    if (t >= b.nt) continue;
+    const float2 x = memory_log_gates(p, static_cast<int>(b.row0) + t, head);
+    in[h] = x.x;
+    c[h] = static_cast<double>(x.y);
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const double x = __shfl_up_sync(0xffffffffu, c[h], o);
+      if (lane >= o) c[h] += x;
+    }
+  c[1] += __shfl_sync(0xffffffffu, c[0], 31);
+#pragma unroll
+  for (int h = 0; h < 2; ++h) top[h] = g[h] = lane + 32 * h < b.nt ? static_cast<double>(in[h]) - c[h] : -INFINITY;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const double x = __shfl_up_sync(0xffffffffu, top[h], o);
+      if (lane >= o) top[h] = fmax(top[h], x);
+    }
+  top[1] = fmax(top[1], __shfl_sync(0xffffffffu, top[0], 31));
+  double* out = bl.sums + (b.block * p.heads + head) * (3 * kMbTok);
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    out[lane + 32 * h] = c[h];
+    out[kMbTok + lane + 32 * h] = g[h];
+    out[2 * kMbTok + lane + 32 * h] = top[h];
+  }
+}
+
+struct MbSums {            // c, g, the largest g up to the token (without gates: -c) of token t of a block
+  double c, g, top;
+  OGB_DEVICE MbSums(const MemoryParams& p, const MemoryBlocks& bl, const MbTile& b, int head, int t) {
+    if (p.logits != nullptr) {
+      const double* in = bl.sums + (b.block * p.heads + head) * (3 * kMbTok) + t;
+      c = in[0];
+      g = in[kMbTok];
+      top = in[2 * kMbTok];
+    } else {
+      c = static_cast<double>(p.decay[p.heads + head]) * (min(t, b.nt - 1) + 1);
+      top = -c;
+      g = t < b.nt ? -c : -INFINITY;
+    }
+  }
+};
+
+// 128 value columns of a block's writes: a warp has 16 of them and all channels of the keys, 64 at a time
 constexpr int kMwCols = 128, kMwVP = kMwCols + 8;
 template <int DP>
 struct MwCfg {
@@ -421,27 +453,31 @@ struct MwCfg {
 };
 
 template <typename T, int DP>
-__global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_write_kernel(MemoryParams p, MemoryBlocks bl) {
-  constexpr int kPitch = MwCfg<DP>::kPitch, DC = DP < 128 ? DP : 128, NT = DC / 8;
+__global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 3 : 1) memory_write_kernel(MemoryParams p, MemoryBlocks bl) {
+  constexpr int kPitch = MwCfg<DP>::kPitch, DC = 64, NT = DC / 8;
   extern __shared__ __align__(16) uint8_t mb_smem[];
   float* sw = reinterpret_cast<float*>(mb_smem);                  // [64] weights
   float* sv = sw + kMbTok;                                        // [64][kMwVP]
   float* sk = sv + kMbTok * kMwVP;                                // [64][kPitch]
   MbTile b;
-  if (!b.set(p, bl)) return;
-  const int head = blockIdx.y, v0 = blockIdx.z * kMwCols, VS = p.columns();
+  if (!b.set(p, bl, blockIdx.y)) return;
+  const int head = blockIdx.x, v0 = blockIdx.z * kMwCols, VS = p.columns();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, tq = lane & 3;
-  mb_channels<T, DP>(p, b, static_cast<const T*>(p.row) + static_cast<size_t>(p.heads + head) * p.D, p.k_scale, sk, kPitch);
-  mb_values<T>(p, b, head, v0, sv, kMwVP);
-  if (v0 + kMbCols < p.V) mb_values<T>(p, b, head, v0 + kMbCols, sv + kMbCols, kMwVP);
-  if (warp == 0) {
-    MbSums m;
-    m.set(p, b, head, -INFINITY);
-    const double c = __shfl_sync(0xffffffffu, m.c[1], 31), top = __shfl_sync(0xffffffffu, m.top[1], 31);
-#pragma unroll
-    for (int h = 0; h < 2; ++h) sw[lane + 32 * h] = expf(static_cast<float>(m.g[h] - top));
-    if (lane == 0 && blockIdx.z == 0) bl.num[b.block * p.heads + head] = make_float4(static_cast<float>(c), static_cast<float>(c + top), 0.f, 0.f);
+  if (tid < kMbTok) {
+    const MbSums x(p, bl, b, head, tid), last(p, bl, b, head, kMbTok - 1);
+    sw[tid] = expf(static_cast<float>(x.g - last.top));
+    if (tid == 0 && blockIdx.z == 0)
+      bl.num[b.block * p.heads + head] = make_float4(static_cast<float>(last.c), static_cast<float>(last.c + last.top), 0.f, 0.f);
   }
+  {
+    const T* const keys[1] = {static_cast<const T*>(p.row) + static_cast<size_t>(p.heads + head) * p.D};
+    const float scale[1] = {p.k_scale};
+    float* const to[1] = {sk};
+    mb_channels<T, DP, 1>(p, b, keys, scale, to, kPitch);
+  }
+  MbValues<T, kMwCols, kMwVP> val;
+  val.fetch(p, b, head, v0);
+  val.store(sv);
   __syncthreads();
   float* u = bl.u + (b.block * p.heads + head) * static_cast<size_t>(VS) * DP;
   if (v0 + 16 * warp < p.V) {
@@ -527,10 +563,18 @@ __global__ void __launch_bounds__(kMcThreads) memory_chain_kernel(MemoryParams p
   *own = s;                                                       // the maximum is left by memory_read_kernel: others may yet read it here
 }
 
+OGB_DEVICE float2 two_terms(double x) {
+  const float hi = static_cast<float>(x);
+  return make_float2(hi, hi == -INFINITY ? 0.f : static_cast<float>(x - static_cast<double>(hi)));
+}
+
+// A read-out: products of queries and keys, then 32 value columns at a time, whose states and values come in while the columns before
+// them are worked on.  Each of the eight warps has 16 tokens and half of the keys or columns.
+constexpr int kMrCols = 32, kMrVP = kMrCols + 8;
 template <int DP>
 struct MrCfg {
   static constexpr int kPitch = DP + 4;
-  static constexpr int kSmemBytes = 8 * (2 * kMbTok) + 4 * (2 * kMbTok * kPitch + kMbTok * kMbVP + kMbTok * kMbPP + 5 * kMbTok);
+  static constexpr int kSmemBytes = 8 * (2 * kMbTok) + 4 * (2 * kMbTok * kPitch + 2 * kMbTok * kMrVP + kMbTok * kMbPP + 5 * kMbTok);
 };
 
 template <typename T, int DP>
@@ -538,97 +582,111 @@ __global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_read_ker
   using Cfg = MrCfg<DP>;
   constexpr int kPitch = Cfg::kPitch;
   extern __shared__ __align__(16) uint8_t mb_smem[];
-  double* sg = reinterpret_cast<double*>(mb_smem);                // [64] g, [64] G
-  double* sG = sg + kMbTok;
+  float2* sg = reinterpret_cast<float2*>(mb_smem);                // [64] g, [64] G, as sums of two terms
+  float2* sG = sg + kMbTok;
   float* se = reinterpret_cast<float*>(sG + kMbTok);              // [64] exp(m - G)
-  float* sinv = se + kMbTok;                                      // [64] what read-outs are multiplied by
+  float* sinv = se + kMbTok;                                      // [64] exp(-m_t), then what read-outs are multiplied by
   float* sdot = sinv + kMbTok;                                    // [64] n . q
   float* srow = sdot + kMbTok;                                    // [2][64] sums of the rows of sP
   float* sq = srow + 2 * kMbTok;                                  // [64][kPitch]
-  float* sk = sq + kMbTok * kPitch;                               // [64][kPitch] keys, then 64 columns of the state
-  float* sv = sk + kMbTok * kPitch;                               // [64][kMbVP]
-  float* sP = sv + kMbTok * kMbVP;                                // [64][kMbPP]
+  float* sk = sq + kMbTok * kPitch;                               // [64][kPitch] keys, then twice 32 columns of the state
+  float* sv = sk + kMbTok * kPitch;                               // [2][64][kMrVP]
+  float* sP = sv + 2 * kMbTok * kMrVP;                            // [64][kMbPP]
   MbTile b;
-  if (!b.set(p, bl)) return;
-  const int head = blockIdx.y, VS = p.columns();
+  if (!b.set(p, bl, blockIdx.y)) return;
+  const int head = blockIdx.x, VS = p.columns();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, tq = lane & 3;
   const bool gated = p.logits != nullptr;
   const float* u = bl.u + (b.block * p.heads + head) * static_cast<size_t>(VS) * DP;
-  const float m_in = gated ? bl.num[b.block * p.heads + head].z : 0.f;
   const T* src = static_cast<const T*>(p.row) + static_cast<size_t>(head) * p.D;
-  mb_channels<T, DP>(p, b, src, p.q_scale, sq, kPitch);
-  mb_channels<T, DP>(p, b, src + p.heads * p.D, p.k_scale, sk, kPitch);
-  if (warp == 0) {
-    MbSums x;
-    x.set(p, b, head, static_cast<double>(m_in));
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int t = lane + 32 * h;
-      const float peak = gated ? static_cast<float>(x.c[h] + x.top[h]) : 0.f;      // m_t
-      sg[t] = x.g[h];
-      sG[t] = x.top[h];
-      se[t] = expf(static_cast<float>(static_cast<double>(m_in) - x.top[h]));
-      sinv[t] = expf(-peak);
-      // the last block of a chunk leaves the maximum for the next step
-      if (gated && t == b.nt - 1 && b.q0 + b.nt == b.len) {
-        const int slot = p.sr.state_slot[p.sr.num_decode + b.seq];
-        if (slot >= 0 && slot < p.sr.num_slots) p.peak[static_cast<size_t>(slot) * p.heads + head] = peak;
-      }
+  if (tid < kMbTok) {
+    const float m_in = gated ? bl.num[b.block * p.heads + head].z : 0.f;
+    const MbSums x(p, bl, b, head, tid);
+    const double top = gated ? fmax(static_cast<double>(m_in), x.top) : x.top;
+    const float peak = gated ? static_cast<float>(x.c + top) : 0.f;      // m_t
+    sg[tid] = two_terms(x.g);
+    sG[tid] = two_terms(top);
+    se[tid] = expf(static_cast<float>(static_cast<double>(m_in) - top));
+    sinv[tid] = expf(-peak);
+    // the last block of a chunk leaves the maximum for the next step
+    if (gated && tid == b.nt - 1 && b.q0 + b.nt == b.len) {
+      const int slot = p.sr.state_slot[p.sr.num_decode + b.seq];
+      if (slot >= 0 && slot < p.sr.num_slots) p.peak[static_cast<size_t>(slot) * p.heads + head] = peak;
     }
   }
+  {
+    const T* const both[2] = {src, src + p.heads * p.D};
+    const float scale[2] = {p.q_scale, p.k_scale};
+    float* const to[2] = {sq, sk};
+    mb_channels<T, DP, 2>(p, b, both, scale, to, kPitch);
+  }
+  MbValues<T, kMrCols, kMrVP> val;
+  val.fetch(p, b, head, 0);
+  val.store(sv);
   __syncthreads();
   const int m = warp & 3, half = warp >> 2;
+  float acc[4][4] = {};
   {
-    float acc[4][4] = {};
     const int tiles = min(4, max(0, 2 * m + 2 - 4 * half));       // key tiles up to the diagonal
     if (tiles > 0) split_product<DP / 8, 4>(acc, sq + 16 * m * kPitch, kPitch, sk + 32 * half * kPitch, kPitch, tiles, gr, tq);
+  }
+  __syncthreads();                                                // the keys have been read
+  auto fetch_state = [&](int v0, int buf) {                       // columns behind the last are read as the last and dropped
+    if (v0 < p.V) {
+#pragma unroll
+      for (int j = 0; j < kMrCols * DP / 4 / kMbThreads; ++j) {
+        const int i = j * kMbThreads + tid, v = min(v0 + i / (DP / 4), VS - 1), d = i % (DP / 4) * 4;
+        cp_async<16>(sk + (buf * kMrCols + i / (DP / 4)) * kPitch + d, u + static_cast<size_t>(v) * DP + d);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch_state(0, 0);
+  {
     float sum[2] = {0.f, 0.f};
 #pragma unroll
     for (int n = 0; n < 4; ++n)
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int t = 16 * m + gr + (x >> 1) * 8, s = 32 * half + 8 * n + 2 * tq + (x & 1);
-        const float f = s <= t ? acc[n][x] * expf(static_cast<float>(sg[s] - sG[t])) : 0.f;
+        const float f = s <= t ? acc[n][x] * expf((sg[s].x - sG[t].x) + (sg[s].y - sG[t].y)) : 0.f;
         sP[t * kMbPP + s] = f;
         sum[x >> 1] += f;
       }
+    if (gated) {
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 1);
-      sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
-      if (tq == 0) srow[half * kMbTok + 16 * m + gr + 8 * h] = sum[h];
-    }
-  }
-  if (gated) {
-    for (int t = warp; t < kMbTok; t += 8) {
-      float a = 0.f;
-      for (int d = lane; d < DP; d += 32) a = fmaf(sq[t * kPitch + d], u[static_cast<size_t>(p.V) * DP + d], a);
-      a = warp_sum(a);
-      if (lane == 0) sdot[t] = a;
-    }
-  }
-  __syncthreads();
-  if (tid < kMbTok) {
-    float inv = 1.f;
-    if (gated) inv = 1.f / (fmaxf(fabsf(se[tid] * sdot[tid] + srow[tid] + srow[kMbTok + tid]), sinv[tid]) + 1e-6f);
-    sinv[tid] = inv;
-  }
-  for (int v0 = 0; v0 < p.V; v0 += kMbCols) {
-    if (v0 > 0) __syncthreads();
+      for (int h = 0; h < 2; ++h) {
+        sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 1);
+        sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
+        if (tq == 0) srow[half * kMbTok + 16 * m + gr + 8 * h] = sum[h];
+      }
+      float n[DP / 32];
 #pragma unroll
-    for (int j = 0; j < kMbCols * DP / 4 / kMbThreads; ++j) {     // columns behind the last are read as the last and dropped
-      const int i = j * kMbThreads + tid, v = min(v0 + i / (DP / 4), VS - 1), d = i % (DP / 4) * 4;
-      cp_async<16>(sk + i / (DP / 4) * kPitch + d, u + static_cast<size_t>(v) * DP + d);
+      for (int d = 0; d < DP / 32; ++d) n[d] = u[static_cast<size_t>(p.V) * DP + 32 * d + lane];
+#pragma unroll 2
+      for (int t = warp; t < kMbTok; t += 8) {
+        float a = 0.f;
+#pragma unroll
+        for (int d = 0; d < DP / 32; ++d) a = fmaf(sq[t * kPitch + 32 * d + lane], n[d], a);
+        a = warp_sum(a);
+        if (lane == 0) sdot[t] = a;
+      }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    mb_values<T>(p, b, head, v0, sv, kMbVP);
+  }
+  for (int v0 = 0, buf = 0; v0 < p.V; v0 += kMrCols, buf ^= 1) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    float o[4][4] = {};
-    split_product<DP / 8, 4>(o, sq + 16 * m * kPitch, kPitch, sk + 32 * half * kPitch, kPitch, 4, gr, tq);
+    __syncthreads();                                              // these columns have arrived, the ones before are done
+    if (v0 == 0 && tid < kMbTok)
+      sinv[tid] = gated ? 1.f / (fmaxf(fabsf(se[tid] * sdot[tid] + srow[tid] + srow[kMbTok + tid]), sinv[tid]) + 1e-6f) : 1.f;
+    fetch_state(v0 + kMrCols, buf ^ 1);
+    val.fetch(p, b, head, v0 + kMrCols);
+    const float* s_state = sk + buf * kMrCols * kPitch;
+    const float* s_val = sv + buf * kMbTok * kMrVP;
+    float o[2][4] = {};
+    split_product<DP / 8, 2>(o, sq + 16 * m * kPitch, kPitch, s_state + 16 * half * kPitch, kPitch, 2, gr, tq);
     const float e0 = se[16 * m + gr], e1 = se[16 * m + gr + 8];
 #pragma unroll
-    for (int n = 0; n < 4; ++n) { o[n][0] *= e0; o[n][1] *= e0; o[n][2] *= e1; o[n][3] *= e1; }
+    for (int n = 0; n < 2; ++n) { o[n][0] *= e0; o[n][1] *= e0; o[n][2] *= e1; o[n][3] *= e1; }
 #pragma unroll 2
     for (int k = 0; k < 2 * m + 2; ++k) {
       float hi[4], lo[4];
@@ -638,12 +696,14 @@ __global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_read_ker
         hi[x] = h.x; lo[x] = h.y;
       }
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        const float w0 = sv[(8 * k + tq) * kMbVP + 32 * half + 8 * n + gr], w1 = sv[(8 * k + tq + 4) * kMbVP + 32 * half + 8 * n + gr];
+      for (int n = 0; n < 2; ++n) {
+        const float w0 = s_val[(8 * k + tq) * kMrVP + 16 * half + 8 * n + gr], w1 = s_val[(8 * k + tq + 4) * kMrVP + 16 * half + 8 * n + gr];
         mma_tf32(o[n], hi, w0, w1);
         mma_tf32(o[n], lo, w0, w1);
       }
     }
+    val.store(sv + (buf ^ 1) * kMbTok * kMrVP);                   // last read a step ago
+    if (v0 == 0) __syncthreads();                                 // sinv
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int t = 16 * m + gr + 8 * h;
@@ -651,8 +711,8 @@ __global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_read_ker
       const float f = sinv[t];
       float* dst = p.out + (b.row0 + t) * (static_cast<size_t>(p.heads) * p.V) + static_cast<size_t>(head) * p.V;
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        const int v = v0 + 32 * half + 8 * n + 2 * tq;
+      for (int n = 0; n < 2; ++n) {
+        const int v = v0 + 16 * half + 8 * n + 2 * tq;
         if ((p.V & 1) == 0 && v < p.V) *reinterpret_cast<float2*>(dst + v) = make_float2(o[n][2 * h] * f, o[n][2 * h + 1] * f);
         else {
           if (v < p.V) dst[v] = o[n][2 * h] * f;
@@ -661,6 +721,7 @@ __global__ void __launch_bounds__(kMbThreads, DP <= 128 ? 2 : 1) memory_read_ker
       }
     }
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
 template <typename T, int DP>
@@ -674,9 +735,10 @@ static int launch_memory_blocks(const MemoryParams& p, const MemoryBlocks& bl, i
     attr_set = true;
   }
   const int VS = p.V + (p.logits != nullptr), quads = VS * DP / 4;
-  memory_write_kernel<T, DP><<<dim3(bl.num_tiles, p.heads, (p.V + kMwCols - 1) / kMwCols), kMbThreads, write_bytes, stream>>>(p, bl);
+  if (p.logits != nullptr) memory_sums_kernel<<<(bl.num_tiles * p.heads + 7) / 8, 256, 0, stream>>>(p, bl);
+  memory_write_kernel<T, DP><<<dim3(p.heads, bl.num_tiles, (p.V + kMwCols - 1) / kMwCols), kMbThreads, write_bytes, stream>>>(p, bl);
   memory_chain_kernel<<<dim3((quads + kMcThreads - 1) / kMcThreads, p.heads, num_prefill), kMcThreads, 0, stream>>>(p, bl);
-  memory_read_kernel<T, DP><<<dim3(bl.num_tiles, p.heads), kMbThreads, MrCfg<DP>::kSmemBytes, stream>>>(p, bl);
+  memory_read_kernel<T, DP><<<dim3(p.heads, bl.num_tiles), kMbThreads, MrCfg<DP>::kSmemBytes, stream>>>(p, bl);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -709,7 +771,7 @@ extern "C" int ogb_turn_table(const int* positions, const double* freq, float* o
 // fp32 scratch per 64-row tile of a step's prompts
 extern "C" int ogb_decay_block_floats(int heads, int D, int V, int gated) {
   const int dp = D <= 64 ? 64 : D <= 128 ? 128 : 256;
-  return heads * ((V + (gated != 0)) * dp + 4);
+  return heads * ((V + (gated != 0)) * dp + 4 + (gated != 0 ? 6 * kMbTok : 0));
 }
 
 // row: q | k | v of `heads` heads; logits (or null) and decay (or null): one of them.  work (16-byte aligned, ogb_decay_block_floats of
@@ -724,7 +786,7 @@ extern "C" int ogb_decay_memory(const void* row, int ld, const float* turns, int
   MemoryParams p{row, reinterpret_cast<const float2*>(turns), logits, bias, decay, state, peak, out, ld, half, ldl, heads, D, V, DP, 0, cap, q_scale,
                  k_scale, StepRows{ctx_len, state_slot, cu_q, tile_seq, tile_q0, num_decode, num_tiles, num_slots}, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool in_blocks = work != nullptr && elem == kElemBF16 && num_prefill > 0 && num_tiles > 0 && (reinterpret_cast<uintptr_t>(work) & 15) == 0 &&
+  const bool in_blocks = work != nullptr && elem == kElemBF16 && num_prefill > 0 && num_tiles > 0 && num_tiles <= 65535 && (reinterpret_cast<uintptr_t>(work) & 15) == 0 &&
                          (reinterpret_cast<uintptr_t>(out) & 7) == 0;
   const int items = num_decode + (in_blocks ? 0 : num_prefill);
   int rc = -3;
@@ -735,7 +797,8 @@ extern "C" int ogb_decay_memory(const void* row, int ld, const float* turns, int
   const size_t n = static_cast<size_t>(num_tiles) * heads;
   bl.tile_seq = tile_seq; bl.tile_q0 = tile_q0; bl.num_tiles = num_tiles;
   bl.num = reinterpret_cast<float4*>(work);
-  bl.u = work + 4 * n;
+  bl.sums = reinterpret_cast<double*>(work + 4 * n);
+  bl.u = work + 4 * n + (logits != nullptr ? 6 * kMbTok * n : 0);
   if (DP == 64) return launch_memory_blocks<__nv_bfloat16, 64>(p, bl, num_prefill, s);
   if (DP == 128) return launch_memory_blocks<__nv_bfloat16, 128>(p, bl, num_prefill, s);
   return launch_memory_blocks<__nv_bfloat16, 256>(p, bl, num_prefill, s);
