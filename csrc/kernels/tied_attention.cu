@@ -221,7 +221,7 @@ template <int DP>
 struct TdCfg {
   static constexpr int kKBytes = kKvBlock * DP * 2;
   static constexpr int kStageBytes = kKBytes + 1024;   // keys, 4 x 16 factors (stages stay 1024-byte aligned)
-  static constexpr int kStages = 96 * 1024 / kStageBytes < 2 ? 2 : 96 * 1024 / kStageBytes > 5 ? 5 : 96 * 1024 / kStageBytes;
+  static constexpr int kStages = DP <= 128 ? 5 : 2;
   static constexpr int kQBytes = 16 * DP * 2;
   static constexpr int kSmemBytes = kStages * kStageBytes + kQBytes + 1024 /*alignment*/ + 1024 /*barriers, merge statistics*/;
   static_assert(4 * 16 * DP * 4 <= kStages * kStageBytes, "the merge slab reuses the ring");
@@ -363,8 +363,10 @@ __global__ void __launch_bounds__(kAttnThreads) tied_decode_kernel(const __grid_
           sum += s[j][2 * r] + s[j][2 * r + 1];
         }
         l_run[r] = l_run[r] * alpha + sum;
+        if (__any_sync(0xffffffffu, alpha != 1.f)) {       // some row has a new maximum
 #pragma unroll
-        for (int j = 0; j < DP / 8; ++j) { o[j][2 * r] *= alpha; o[j][2 * r + 1] *= alpha; }
+          for (int j = 0; j < DP / 8; ++j) { o[j][2 * r] *= alpha; o[j][2 * r + 1] *= alpha; }
+        }
       }
       const uint32_t a[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
 #pragma unroll

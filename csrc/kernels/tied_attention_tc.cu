@@ -1,7 +1,7 @@
 // Prompts of attention over keys that are the values, on the 5th-generation tensor cores (tcgen05 + TMEM), bf16.
 //
-// A CTA has one KV head and 128 rows: the (token, query head) pairs of 128 / group tokens.  One shared-memory block of keys serves both
-// products, as in latent_attention_tc.cu:
+// A CTA has 128 rows: the (token, query head) pairs of a KV head's group and 128 / group tokens, or one query head's 128 tokens where the
+// group does not divide 128.  One shared-memory block of keys serves both products, as in latent_attention_tc.cu:
 //
 //   warp 0    : TMA producer.  The queries once; then every 16-token page, 64 columns at a time (2 KB boxes, 128-byte swizzle), so a
 //               block is [column chunk][token][64 values]: the K-major operand of S = Q K^T and, read along the other axis, the
@@ -54,7 +54,7 @@ struct TtBars {
 };
 
 struct TtShape {                         // how a tile's rows are dealt out
-  int group, tokens, span, per_tile;     // query heads of a KV head, tokens of a CTA, tokens of its tiles, CTAs they take
+  int group, tokens, span, per_tile;     // query heads of a CTA, its tokens, tokens of its tiles, CTAs they take
 };
 
 struct TtRows {                          // the query rows of a CTA
@@ -138,7 +138,8 @@ tied_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
 
   TtRows rw;
   if (!tt_rows(p, sh, rw)) return;
-  const int kvh = blockIdx.y % p.hkv, col0 = blockIdx.y / p.hkv * OC;       // output columns of this CTA
+  const int units = p.hq / sh.group, head0 = blockIdx.y % units * sh.group, kvh = head0 / (p.hq / p.hkv);
+  const int col0 = blockIdx.y / units * OC;             // output columns of this CTA
   const int kv_lo = p.window > 0 ? max(0, rw.pos_first - p.window + 1) : 0;
   const int b_begin = kv_lo / BN, nblk = (rw.pos_last + BN) / BN - b_begin;  // last visible key is pos_last
 
@@ -171,7 +172,7 @@ tied_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
       bool ok = true;
       mbar_expect_tx(&bars->q_full, Cfg::kChunks * sh.tokens * sh.group * 128);
 #pragma unroll
-      for (int h = 0; h < Cfg::kChunks; ++h) tma_load_3d(sQ + h * kTtBM * 128, &q_map, &bars->q_full, h * 64, kvh * sh.group, rw.tok0);
+      for (int h = 0; h < Cfg::kChunks; ++h) tma_load_3d(sQ + h * kTtBM * 128, &q_map, &bars->q_full, h * 64, head0, rw.tok0);
       const int n_pages = (rw.ctx + kTaPage - 1) / kTaPage;
       const int* table = p.page_table + static_cast<size_t>(rw.entry) * p.max_pages;
       const __nv_bfloat16* factors = static_cast<const __nv_bfloat16*>(p.pool) + static_cast<size_t>(p.hkv) * kTaPage * p.dp;
@@ -246,7 +247,7 @@ tied_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
     const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
     const uint32_t s_addr = lane_base + Cfg::kColS + g * BN;
     const uint32_t o_addr = lane_base + g * OC;
-    const int tok = row / sh.group, head = kvh * sh.group + row - tok * sh.group;
+    const int tok = row / sh.group, head = head0 + row - tok * sh.group;
     const int pos = rw.pos_first + tok;                  // rows past the last are computed and dropped
     const int hi_abs = min(pos, rw.ctx - 1);
     const int lo_abs = p.window > 0 ? pos - p.window + 1 : 0;
@@ -440,11 +441,11 @@ template <int R, int OC, int BN, int ST>
 static int launch_tt(const TiedParams& p, cudaStream_t stream) {
   using Cfg = TtCfg<R, OC, BN, ST>;
   TtShape sh;
-  sh.group = p.hq / p.hkv;
-  sh.tokens = std::min(kTtBM / sh.group, 128);
+  const int group = p.hq / p.hkv;
+  sh.group = kTtBM % group == 0 ? group : 1;
   sh.span = sh.group == 1 ? 128 : 64;
-  sh.tokens = std::min(sh.tokens, sh.span);
-  sh.per_tile = (sh.span + sh.tokens - 1) / sh.tokens;
+  sh.tokens = kTtBM / sh.group;
+  sh.per_tile = sh.span / sh.tokens;
   CUtensorMap q_map, k_map;
   int rc = encode_tmap_bf16_3d(&q_map, p.q, p.dp, p.hq, p.rows, p.dp, p.ldq, 64, sh.group, sh.tokens);
   if (rc != 0) return rc;
@@ -455,13 +456,13 @@ static int launch_tt(const TiedParams& p, cudaStream_t stream) {
     OGB_CUDA_CHECK(cudaFuncSetAttribute(tied_attention_tc_kernel<R, OC, BN, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
     attr_set = true;
   }
-  const dim3 grid(p.num_tiles * sh.per_tile, p.hkv * ((p.dp + OC - 1) / OC));
+  const dim3 grid(p.num_tiles * sh.per_tile, p.hq / sh.group * ((p.dp + OC - 1) / OC));
   tied_attention_tc_kernel<R, OC, BN, ST><<<grid, kTtThreads, Cfg::kSmemBytes, stream>>>(q_map, k_map, p, sh);
   return static_cast<int>(cudaGetLastError());
 }
 
 int launch_tied_prefill_tc(const TiedParams& p, cudaStream_t stream) {
-  if (p.dp > 256 || p.hq / p.hkv > 64 || ((p.dp | p.ldq | p.ldo | p.page_elems) & 7) != 0) return -2;
+  if (p.dp > 256 || ((p.dp | p.ldq | p.ldo | p.page_elems) & 7) != 0) return -2;
   if ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.out) | reinterpret_cast<uintptr_t>(p.pool)) & 15) return -2;
   if (p.dp <= 64) return launch_tt<64, 64, 128, 4>(p, stream);
   if (p.dp <= 128) return launch_tt<128, 128, 128, 4>(p, stream);
