@@ -172,6 +172,7 @@ def kernel_rows(size: str, timer, pk):
         row("gemm router (fp32 out)", phase, lambda: hops.linear(h, wr, logits, f32_out=True), **product(e, hid, 4))
         logits.normal_()
         half, gu, down, lg, acc = 128, rnd(e, 2 * ff, hid), rnd(e, hid, ff), logits.to(bf), empty(t, hid)
+        corr *= 0.01                                      # choices stay spread over the experts
         ws = mops.MoEWorkspace(t, top, e, hid, ff, "cuda", bf)
         fl, by = 6 * t * top * ff * hid, min(e, t * top) * 3 * ff * hid * 2 + t * top * (2 * hid + 2 * ff) * 2
         row("experts: route, permute, gather, up, down", phase,
