@@ -35,9 +35,9 @@ TAPS, GROUPS = 4, 4
 def configs(size: str):
     hid, layers, hq, hkv, window, rh, mh, e, top, groups, kept, ff, dense = SIZES[size]
     moe = MoeSpec(e, top, ff, groups, kept, True, "silu", bias=True, score="sigmoid", group_best=2)
-    tied = TiedSpec(hq, hkv, D, D ** -0.5, 50.0, window)
+    tied = TiedSpec(hq, hkv, D, D ** -0.5, 30.0, window)
     ret = MemorySpec(rh, D, D, decay=tuple(1 - 2.0 ** -(5 + 6 * a / rh) for a in range(rh)), rot_dims=D, rot_base=1e4)
-    mem = MemorySpec(mh, D, MV, gate_cap=15.0)
+    mem = MemorySpec(mh, D, MV, gate_cap=10.0)
     new = HybridConfig(vocab=VOCAB, hidden=hid, layers=[LayerSpec((tied, ret, ret, mem)[i % 4], MlpSpec(dense, "silu") if i % 4 == 0 else moe) for i in range(layers)],
                        residual="pre", norm_groups=GROUPS, input_taps=TAPS, ff_input_conv=False, residual_gates=True, embed_normed=False, name=f"midisun-{size}")
     # experts there have two matrices: half as many channels again for as many operations
@@ -96,9 +96,9 @@ def kernel_rows(size: str, timer, pk):
         row("like: gemm qkv", phase, lambda: ops.gemm(h, wl, out=qkv), **product(wl.shape[0], hid))
         u.normal_()
         pool = rnd(npages, hops.tied_page_elems(hkv, D))
-        pool.view(f4)[:, hkv * 16 * D // 2:] = 0.1 / 50
+        pool.view(f4)[:, hkv * 16 * D // 2:] = 0.1 / 30
         qb, kb, qg = f32(hq * D), f32(hkv * D), f32(hq * D)
-        row("tied_append", phase, lambda: hops.tied_append(u, qb, kb, qg, 1e-6, D ** -0.5 / 50, q, pool, si.slots, hq, hkv, D, D), nbytes=2 * t * (hq + hkv) * D * 2)
+        row("tied_append", phase, lambda: hops.tied_append(u, qb, kb, qg, 1e-6, D ** -0.5 / 30, q, pool, si.slots, hq, hkv, D, D), nbytes=2 * t * (hq + hkv) * D * 2)
         kv = rnd(npages, hkv, 2, 16, D)
         table = ops.reference.rope_table(ctx + 1, D, 1e4, "cuda")
         row("like: rope_kv_append", phase, lambda: ops.rope_kv_append(qkv, si.positions, si.slots, table, kv, hq, hkv, D), nbytes=2 * t * (hq + 2 * hkv) * D * 2)
@@ -108,7 +108,7 @@ def kernel_rows(size: str, timer, pk):
         slope, sink, out = distance_slopes(hq, "cuda"), f32(hq), empty(t, hq * D)
         hg = u[:, (hq + hkv) * D:(hq + hkv) * D + hq]
         if prompt:
-            row("tied_attention (prompt)", phase, lambda: hops.tied_attention(q, attn, pool, si, hq, hkv, D, D, 50.0, slope, sink, window, hg), fl, by)
+            row("tied_attention (prompt)", phase, lambda: hops.tied_attention(q, attn, pool, si, hq, hkv, D, D, 30.0, slope, sink, window, hg), fl, by)
             row("  the same without a cap", phase, lambda: hops.tied_attention(q, attn, pool, si, hq, hkv, D, D, 0.0, slope, sink, window, hg), fl, by)
             row("like: paged_prefill (window, tcgen05)", phase, lambda: ops.paged_prefill(qkv, out, kv, si.page_table, si.ctx_len, si.cu_q, si.tile_seq, si.tile_q0,
                                                                                         si.num_tiles, hq, hkv, D, None, window), fl, lby)
@@ -119,7 +119,7 @@ def kernel_rows(size: str, timer, pk):
                 splits *= 2
             cnt = torch.zeros(nseq * ctas, dtype=torch.int32, device="cuda")
             po, pm = empty(nseq * ctas * 16 * splits * D, dtype=f4), empty(nseq * ctas * 32 * splits, dtype=f4)
-            row(f"tied_attention (decode, {splits} splits)", phase, lambda: hops.tied_attention(q, attn, pool, si, hq, hkv, D, D, 50.0, slope, sink, window, hg, splits, po, pm,
+            row(f"tied_attention (decode, {splits} splits)", phase, lambda: hops.tied_attention(q, attn, pool, si, hq, hkv, D, D, 30.0, slope, sink, window, hg, splits, po, pm,
                                                                                                cnt), fl, by)
             row("like: paged_decode (window)", phase, lambda: ops.paged_decode(qkv, out, kv, si.page_table, si.ctx_len, hq, hkv, D, None, 1, None, None, window), fl, lby)
         wo = rnd(hid, hq * D)
@@ -151,7 +151,7 @@ def kernel_rows(size: str, timer, pk):
                 wi = rnd(2 * heads, hid)
                 row("gemm input|forget gates (fp32 out)", phase, lambda: hops.linear(h, wi, logits, f32_out=True), **product(2 * heads, hid, 4))
             bias = f32(2 * heads) + 2 if gated else None
-            row(f"decay_memory ({what})", phase, lambda: hops.decay_memory(p, None if gated else turns, logits, bias, 15.0, None if gated else dec, st, peak if gated else None,
+            row(f"decay_memory ({what})", phase, lambda: hops.decay_memory(p, None if gated else turns, logits, bias, 10.0, None if gated else dec, st, peak if gated else None,
                                                                           raw, heads, D, vd, 1.0, 1.0, si, blocks=True, scratch=scratch),
                 nbytes=t * heads * ((2 * D + vd) * 2 + vd * 4) + 2 * nseq * heads * (vd + gated) * D * 4)
             nw = f32(heads * vd)

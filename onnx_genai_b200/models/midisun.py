@@ -46,7 +46,7 @@ def read_config(doc: dict, name: str = "midisun") -> HybridConfig:
     layers = [LayerSpec(read_mixer(i, entry["type"], entry["mixer"]), read_mlp(i, entry.get("mlp"))) for i, entry in enumerate(doc["layers"])]
     cfg = HybridConfig(vocab=int(doc["vocab"]), hidden=int(doc["width"]), layers=layers, norm_eps=float(doc["norm"]["eps"]), name=name, residual="pre",
                        norm_groups=int(doc["norm"].get("groups", 1)), input_taps=int(doc["canon"]["taps"]), ff_input_conv=False, residual_gates=True,
-                       embed_scale=float(doc["embedding"]["scale"]), embed_normed=False)
+                       embed_scale=float((doc.get("embedding") or {}).get("scale", 1.0)), embed_normed=False)
     cfg.validate()
     return cfg
 

@@ -328,7 +328,7 @@ def tied_case(where, hq, hkv, d, window, cap, chunks, spike, sloped=True, splits
     assert not out.view(t, hq, dp)[..., d:].any()
 
 
-TIED_SIZES = [(3, 1, 20, 21, 4.0), (1, 1, 10, 1, 0.0), (4, 2, 64, 70, 6.0), (8, 1, 32, 100, 3.0), (20, 1, 48, 64, 30.0), (2, 2, 128, 130, 5.0), (4, 4, 96, 96, 50.0),
+TIED_SIZES = [(3, 1, 20, 21, 4.0), (1, 1, 10, 1, 0.0), (4, 2, 64, 70, 6.0), (8, 1, 32, 100, 3.0), (20, 1, 48, 64, 30.0), (2, 2, 128, 130, 5.0), (3, 3, 104, 90, 20.0),
               (2, 1, 160, 40, 8.0), (2, 2, 256, 30, 0.0), (6, 3, 64, 0, 2.0), (1, 1, 300, 33, 7.0), (66, 1, 16, 50, 5.0)]
 
 
